@@ -22,8 +22,13 @@ using gemm::Params;
 
 namespace {
 
-enum Epi : int { kEpiStore = 0, kEpiSiluMul = 1 };
+using gemm::kEpiClampGlu;
+using gemm::kEpiF32;
+using gemm::kEpiSiluMul;
+using gemm::kEpiStore;
 
+template <int EPI>
+__device__ __forceinline__ float glu_pair(const Params& p, float g, float u);
 __device__ __forceinline__ float bf16_round(float x) { return __bfloat162float(__float2bfloat16_rn(x)); }
 // silu(g) * u with every intermediate rounded to bf16, which is what an unfused bf16
 // pipeline (gate, act(gate), act * up as separate bf16 tensors) produces.
@@ -34,6 +39,35 @@ __device__ __forceinline__ float silu_mul_bf16(float g, float u) {
   return s * u;
 }
 
+template <>
+__device__ __forceinline__ float glu_pair<kEpiSiluMul>(const Params& p, float g, float u) { return silu_mul_bf16(g, u); }
+template <>
+__device__ __forceinline__ float glu_pair<kEpiClampGlu>(const Params& p, float g, float u) { return gemm::clamp_glu(g, u, p.act_a, p.act_b); }
+
+// four consecutive fp32 features of one token: activation, store, optional bf16 copy
+__device__ __forceinline__ void store_f32x4(const Params& p, size_t off, int m, float4 v) {
+  v.x = gemm::apply_act(v.x, p.act, p.act_a);
+  v.y = gemm::apply_act(v.y, p.act, p.act_a);
+  v.z = gemm::apply_act(v.z, p.act, p.act_a);
+  v.w = gemm::apply_act(v.w, p.act, p.act_a);
+  if (m + 4 <= p.M) {
+    *reinterpret_cast<float4*>(p.yf + off) = v;
+    if (p.y2) {
+      __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+      uint2 pk;
+      pk.x = *reinterpret_cast<uint32_t*>(&lo);
+      pk.y = *reinterpret_cast<uint32_t*>(&hi);
+      *reinterpret_cast<uint2*>(p.y2 + off) = pk;
+    }
+  } else {
+    const float a4[4] = {v.x, v.y, v.z, v.w};
+    for (int e = 0; e < 4 && m + e < p.M; e++) {
+      p.yf[off + e] = a4[e];
+      if (p.y2) p.y2[off + e] = __float2bfloat16_rn(a4[e]);
+    }
+  }
+}
+
 template <int EPI>
 __global__ void __launch_bounds__(gemm::kThreads, 1)
 k_gemm(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB, const Params p) {
@@ -42,7 +76,16 @@ k_gemm(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensor
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   // Launch order follows blockIdx.x.  With many token tiles the CTAs that share one 128-row weight tile
   // must run together, so that the weights stream from HBM once and the activations stay in L2.
-  const int m0 = (p.raster ? blockIdx.y : blockIdx.x) * gemm::kBM, n0 = (p.raster ? blockIdx.x : blockIdx.y) * p.bn;
+  constexpr bool kGlu = EPI == kEpiSiluMul || EPI == kEpiClampGlu;
+  int m0 = (p.raster ? blockIdx.y : blockIdx.x) * gemm::kBM;
+  const int n0 = (p.raster ? blockIdx.x : blockIdx.y) * p.bn;
+  int grp = 0;                                   // group of a grouped problem; m0 becomes the feature inside the group
+  if (p.groups > 1) {
+    const int mt = (p.M + gemm::kBM - 1) / gemm::kBM;
+    grp = (m0 / gemm::kBM) / mt;
+    m0 -= grp * mt * gemm::kBM;
+  }
+  const size_t ycol = size_t(grp) * p.y_group;
   const int S = p.splits;
   const int split = S > 1 ? int(cluster_ctarank()) : 0;
   const int kb_per = (p.kb_total + S - 1) / S;
@@ -50,10 +93,10 @@ k_gemm(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensor
   int nkb = p.kb_total - kb0;
   nkb = nkb < 0 ? 0 : (nkb > kb_per ? kb_per : nkb);
 
-  uint8_t* sm = gemm::mainloop(&tmA, &tmB, p, s, smem_raw, m0, n0, kb0, nkb);
+  uint8_t* sm = gemm::mainloop(&tmA, &tmB, p, s, smem_raw, grp * p.M + m0, n0, kb0, nkb, grp * p.x_group);
   volatile int* abortp = &s.abort_flag;
   const int rows = (p.N - n0 < p.bn) ? (p.N - n0) : p.bn;  // valid tokens in this tile
-  constexpr int OUTW = EPI == kEpiSiluMul ? 64 : 128;       // output features per tile
+  constexpr int OUTW = kGlu ? 64 : 128;       // output features per tile
 
   if (warp >= 2) {
     const int quarter = warp & 3;             // TMEM lane quarter this warp may read
@@ -78,7 +121,10 @@ k_gemm(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensor
       if (S > 1) {
 #pragma unroll
         for (int j = 0; j < 16; j++) stage_f[(c + j) * 128 + ml] = __uint_as_float(r[j]);
-      } else if (EPI == kEpiSiluMul) {
+      } else if (EPI == kEpiF32) {
+#pragma unroll
+        for (int j = 0; j < 16; j++) stage_f[(c + j) * 128 + ml] = __uint_as_float(r[j]) + bias;
+      } else if (kGlu) {
         // Even lanes hold gate rows, odd lanes the matching up rows.  Per pair of token columns the two lanes
         // swap one value each, so that the even lane finishes column j and the odd lane column j + 1: every
         // lane does useful SiLU work and one shuffle serves two outputs.
@@ -86,7 +132,7 @@ k_gemm(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensor
         for (int j = 0; j < 16; j += 2) {
           const float v0 = __uint_as_float(r[j]) + bias, v1 = __uint_as_float(r[j + 1]) + bias;
           const float recv = __shfl_xor_sync(0xffffffffu, (lane & 1) ? v0 : v1, 1);
-          const float o = (lane & 1) ? silu_mul_bf16(recv, v1) : silu_mul_bf16(v0, recv);
+          const float o = (lane & 1) ? glu_pair<kGlu ? EPI : kEpiSiluMul>(p, recv, v1) : glu_pair<kGlu ? EPI : kEpiSiluMul>(p, v0, recv);
           stage_h[(c + j + (lane & 1)) * 64 + (ml >> 1)] = __float2bfloat16_rn(o);
         }
       } else {
@@ -94,21 +140,29 @@ k_gemm(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensor
         for (int j = 0; j < 16; j++) stage_h[(c + j) * 128 + ml] = __float2bfloat16_rn(__uint_as_float(r[j]) + bias);
       }
     }
-    if (S == 1) {
+    if (S == 1 && EPI == kEpiF32) {
+      asm volatile("bar.sync 1, 128;" ::: "memory");
+      const int te = threadIdx.x - 64;
+      for (int idx = te; idx < rows * 32; idx += 128) {
+        const int t = idx >> 5, m = m0 + (idx & 31) * 4;
+        if (m < p.M)
+          store_f32x4(p, size_t(n0 + t) * p.ldy + ycol + m, m, *reinterpret_cast<const float4*>(stage_f + t * 128 + (idx & 31) * 4));
+      }
+    } else if (S == 1) {
       // coalesced copy-out of the staged tile: 16-byte pieces, OUTW features per token row
       asm volatile("bar.sync 1, 128;" ::: "memory");
       const int te = threadIdx.x - 64;
       constexpr int PPR = OUTW / 8;  // 16-byte pieces per row
-      const int out_m0 = EPI == kEpiSiluMul ? (m0 >> 1) : m0;
-      const int out_M = EPI == kEpiSiluMul ? (p.M >> 1) : p.M;
+      const int out_m0 = kGlu ? (m0 >> 1) : m0;
+      const int out_M = kGlu ? (p.M >> 1) : p.M;
       for (int idx = te; idx < rows * PPR; idx += 128) {
         const int t = idx / PPR, pc = idx % PPR;
         const int m = out_m0 + pc * 8;
         if (m + 8 <= out_M) {
-          *reinterpret_cast<uint4*>(p.y + size_t(n0 + t) * p.ldy + m) =
+          *reinterpret_cast<uint4*>(p.y + size_t(n0 + t) * p.ldy + ycol + m) =
               *reinterpret_cast<const uint4*>(stage_h + t * OUTW + pc * 8);
         } else {
-          for (int e = 0; e < 8 && m + e < out_M; e++) p.y[size_t(n0 + t) * p.ldy + m + e] = stage_h[t * OUTW + pc * 8 + e];
+          for (int e = 0; e < 8 && m + e < out_M; e++) p.y[size_t(n0 + t) * p.ldy + ycol + m + e] = stage_h[t * OUTW + pc * 8 + e];
         }
       }
     }
@@ -133,11 +187,13 @@ k_gemm(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensor
           if (m + 2 < p.M) acc.z += __bfloat162float(p.bias[m + 2]);
           if (m + 3 < p.M) acc.w += __bfloat162float(p.bias[m + 3]);
         }
-        if (EPI == kEpiSiluMul) {
-          __nv_bfloat162 o = __floats2bfloat162_rn(silu_mul_bf16(acc.x, acc.y), silu_mul_bf16(acc.z, acc.w));
-          if (m + 4 <= p.M) *reinterpret_cast<__nv_bfloat162*>(p.y + size_t(n0 + t) * p.ldy + (m >> 1)) = o;
+        if (EPI == kEpiF32) {
+          if (m < p.M) store_f32x4(p, size_t(n0 + t) * p.ldy + ycol + m, m, acc);
+        } else if (kGlu) {
+          __nv_bfloat162 o = __floats2bfloat162_rn(glu_pair<kGlu ? EPI : kEpiSiluMul>(p, acc.x, acc.y), glu_pair<kGlu ? EPI : kEpiSiluMul>(p, acc.z, acc.w));
+          if (m + 4 <= p.M) *reinterpret_cast<__nv_bfloat162*>(p.y + size_t(n0 + t) * p.ldy + ycol + (m >> 1)) = o;
         } else {
-          __nv_bfloat16* dst = p.y + size_t(n0 + t) * p.ldy + m;
+          __nv_bfloat16* dst = p.y + size_t(n0 + t) * p.ldy + ycol + m;
           if (m + 4 <= p.M) {
             __nv_bfloat162 lo = __floats2bfloat162_rn(acc.x, acc.y), hi = __floats2bfloat162_rn(acc.z, acc.w);
             uint2 pk;
@@ -279,10 +335,10 @@ int sm_count() {
   return g_sm_count[dev & 15];
 }
 
-void gemm_config(int M, int N, int K, int splits_hint, int* bn_out, int* splits_out, int* stages_out) {
+void gemm_config(int M, int N, int K, int splits_hint, int* bn_out, int* splits_out, int* stages_out, int groups, bool f32_out) {
   int bn = N <= 16 ? 16 : (N <= 32 ? 32 : (N <= 64 ? 64 : (N <= 128 ? 128 : 256)));
   const int kb = (K + 63) / 64;
-  const int tiles = ((M + 127) / 128) * ((N + bn - 1) / bn);
+  const int tiles = groups * ((M + 127) / 128) * ((N + bn - 1) / bn);
   const int sms = sm_count();
   int splits = 1;
   if (splits_hint > 0) {
@@ -297,12 +353,64 @@ void gemm_config(int M, int N, int K, int splits_hint, int* bn_out, int* splits_
   const int budget = (tiles * splits > sms) ? 108 * 1024 : 200 * 1024;  // two CTAs per SM when the grid is larger than the GPU
   int stages = budget / stage_bytes;
   stages = stages < 2 ? 2 : (stages > gemm::kMaxStages ? gemm::kMaxStages : stages);
-  const int need = splits > 1 ? bn * 512 : bn * 256;  // epilogue staging reuses the ring
+  const int need = splits > 1 || f32_out ? bn * 512 : bn * 256;  // epilogue staging reuses the ring
   while (stages * stage_bytes < need) stages++;
   *bn_out = bn; *splits_out = splits; *stages_out = stages;
 }
 
 }  // namespace tbvops
+
+namespace {
+// Decode-form launch of a filled Params (M, N, K, ldy, output pointers, epilogue arguments, groups).
+int launch_decode_form(const void* w, const void* x, int ldx, Params& p, int epi, int splits_hint, cudaStream_t st) {
+  const int M = p.M, N = p.N, K = p.K, G = p.groups > 1 ? p.groups : 1;
+  int bn, splits, stages;
+  tbvops::gemm_config(M, N, K, splits_hint, &bn, &splits, &stages, G, epi == kEpiF32);
+  CUtensorMap tmA, tmB;
+  if (tbvops::make_tensor_map_bf16(&tmA, w, (unsigned long long)G * M, K, K, 128) != 0) return -3;
+  if (tbvops::make_tensor_map_bf16(&tmB, x, N, (unsigned long long)(G - 1) * p.x_group + K, ldx, bn) != 0) return -3;
+  p.bn = bn; p.splits = splits; p.stages = stages;
+  p.kb_total = (K + 63) / 64;
+  p.limit_ns = 2000000000ull;
+  p.err = tbvops::gemm_err_flag();
+  const size_t smem = size_t(stages) * (gemm::kATileBytes + bn * 128) + 1024;
+  if (!g_attr_done) {
+    // 227 KB per CTA in total; the kernel's static shared state comes out of the same budget
+    const cudaError_t a[4] = {cudaFuncSetAttribute(k_gemm<kEpiStore>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
+                              cudaFuncSetAttribute(k_gemm<kEpiSiluMul>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
+                              cudaFuncSetAttribute(k_gemm<kEpiF32>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
+                              cudaFuncSetAttribute(k_gemm<kEpiClampGlu>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024)};
+    for (cudaError_t e : a)
+      if (e != cudaSuccess) {
+        fprintf(stderr, "[tbvops] cudaFuncSetAttribute(max dynamic smem) failed: %s\n", cudaGetErrorString(e));
+        return -1;
+      }
+    g_attr_done = true;
+  }
+  const int mt = G * ((M + 127) / 128), nt = (N + bn - 1) / bn;
+  p.raster = nt > 1 ? 1 : 0;
+  const dim3 grid(p.raster ? nt : mt, p.raster ? mt : nt, splits), blk(gemm::kThreads);
+  cudaError_t e;
+  switch (epi) {
+    case kEpiSiluMul: e = pdl::launch(k_gemm<kEpiSiluMul>, grid, blk, smem, st, splits, tmA, tmB, p); break;
+    case kEpiF32: e = pdl::launch(k_gemm<kEpiF32>, grid, blk, smem, st, splits, tmA, tmB, p); break;
+    case kEpiClampGlu: e = pdl::launch(k_gemm<kEpiClampGlu>, grid, blk, smem, st, splits, tmA, tmB, p); break;
+    default: e = pdl::launch(k_gemm<kEpiStore>, grid, blk, smem, st, splits, tmA, tmB, p); break;
+  }
+  if (e != cudaSuccess) {
+    fprintf(stderr, "[tbvops] gemm launch failed: %s (M=%d N=%d K=%d groups=%d bn=%d splits=%d stages=%d)\n", cudaGetErrorString(e), M, N,
+            K, G, bn, splits, stages);
+    return -1;
+  }
+  return 0;
+}
+int persist_mode() {
+  // TBV_GEMM_PERSIST: 0 = never, 1 (default) = where it is estimated to be faster, 2 / 3 = its 128- / 256-token tile
+  // wherever the shape allows; read once, not per launch.
+  if (g_persist_mode == -1) { const char* pe = getenv("TBV_GEMM_PERSIST"); g_persist_mode = pe ? atoi(pe) : 1; }
+  return g_persist_mode;
+}
+}  // namespace
 
 extern "C" {
 
@@ -320,10 +428,8 @@ int tbv_op_gemm(const void* w, const void* x, void* y, const void* bias, int M, 
   const unsigned long long pf_bytes = tbvops::take_next_prefetch(&pf_ptr, (unsigned long long)(M > 0 ? M : 0) * (unsigned long long)(K > 0 ? K : 0) * 2ull);
   if (M <= 0 || N <= 0 || K <= 0 || (K % 8) || (ldx % 8) || (ldy % 8) || (reinterpret_cast<uintptr_t>(y) & 15u)) return -2;
   if (epi == kEpiSiluMul && (M % 2)) return -2;
-  // Hundreds of tokens: the persistent kernel with tokens on the UMMA M axis.  TBV_GEMM_PERSIST: 0 = never,
-  // 1 (default) = where it is estimated to be faster, 2 / 3 = its 128- / 256-token tile wherever the shape allows.
-  if (g_persist_mode == -1) { const char* pe = getenv("TBV_GEMM_PERSIST"); g_persist_mode = pe ? atoi(pe) : 1; }  // read once, not per launch
-  const int persist = g_persist_mode;
+  // Hundreds of tokens: the persistent kernel with tokens on the UMMA M axis.
+  const int persist = persist_mode();
   if (persist > 0 && splits_hint <= 0) {
     const int th = w_not_constant ? 0 : tbvops::gemm_tok_choose(M, N, K, ldy, epi, persist);   // the many-token kernel always prefetches w
     if (th > 0) return tbvops::gemm_tok_launch(w, x, y, bias, M, N, K, ldx, ldy, epi, th, stream);
@@ -331,44 +437,38 @@ int tbv_op_gemm(const void* w, const void* x, void* y, const void* bias, int M, 
   // Large weight matrices at decode batch sizes: the persistent kernel that splits the work evenly over the SMs.
   if (tbvops::gemm_streamk_wants(M, N, K, epi, splits_hint, w_not_constant != 0))
     return tbvops::gemm_streamk_launch(w, x, y, bias, M, N, K, ldx, ldy, epi, stream);
-  int bn, splits, stages;
-  tbvops::gemm_config(M, N, K, splits_hint, &bn, &splits, &stages);
-  CUtensorMap tmA, tmB;
-  if (tbvops::make_tensor_map_bf16(&tmA, w, M, K, K, 128) != 0) return -3;
-  if (tbvops::make_tensor_map_bf16(&tmB, x, N, K, ldx, bn) != 0) return -3;
   Params p{};
-  p.M = M; p.N = N; p.K = K; p.ldy = ldy; p.bn = bn; p.splits = splits; p.stages = stages;
-  p.kb_total = (K + 63) / 64;
+  p.M = M; p.N = N; p.K = K; p.ldy = ldy;
   p.a_after_wait = w_not_constant;
   p.bias = static_cast<const __nv_bfloat16*>(bias);
   p.y = static_cast<__nv_bfloat16*>(y);
-  p.limit_ns = 2000000000ull;
-  p.err = tbvops::gemm_err_flag();
   p.pf_ptr = pf_ptr;
   p.pf_bytes = pf_bytes;
-  const size_t smem = size_t(stages) * (gemm::kATileBytes + bn * 128) + 1024;
-  if (!g_attr_done) {
-    // 227 KB per CTA in total; the kernel's static shared state comes out of the same budget
-    cudaError_t a1 = cudaFuncSetAttribute(k_gemm<kEpiStore>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024);
-    cudaError_t a2 = cudaFuncSetAttribute(k_gemm<kEpiSiluMul>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024);
-    if (a1 != cudaSuccess || a2 != cudaSuccess) {
-      fprintf(stderr, "[tbvops] cudaFuncSetAttribute(max dynamic smem) failed: %s\n", cudaGetErrorString(a1 != cudaSuccess ? a1 : a2));
-      return -1;
-    }
-    g_attr_done = true;
+  return launch_decode_form(w, x, ldx, p, epi, splits_hint, static_cast<cudaStream_t>(stream));
+}
+
+// The GEMM with the wider set of epilogues: fp32 output with an activation, clamped gated unit, grouped weights.
+// y: fp32 [N, ldy] for epi 2, bf16 otherwise; y2: optional bf16 copy of an fp32 result (same ldy).  act (epi 2): 0 none,
+// 1 softplus, 2 act_a * tanh(v / act_a).  epi 3: rows of w interleaved (gate_i, up_i), act_a = clamp limit, act_b = slope of the
+// sigmoid.  groups > 1: w is [groups * M, K]; group g reads x columns g * x_group .. + K and writes y columns g * y_group .. .
+int tbv_op_gemm_ex(const void* w, const void* x, void* y, void* y2, const void* bias, int M, int N, int K, int ldx, int ldy, int epi,
+                   int act, float act_a, float act_b, int groups, int x_group, int y_group, void* stream) {
+  if (M <= 0 || N <= 0 || K <= 0 || (K % 8) || (ldx % 8) || (ldy % 8) || (reinterpret_cast<uintptr_t>(y) & 15u)) return -2;
+  if (epi < 0 || epi > 3 || (epi == kEpiClampGlu && (M % 2)) || (y2 && (epi != kEpiF32 || (reinterpret_cast<uintptr_t>(y2) & 7u)))) return -2;
+  if (groups > 1 && ((x_group % 8) || (y_group % 8) || bias)) return -2;
+  Params p{};
+  p.M = M; p.N = N; p.K = K; p.ldy = ldy;
+  p.bias = static_cast<const __nv_bfloat16*>(bias);
+  if (epi == kEpiF32) p.yf = static_cast<float*>(y);
+  else p.y = static_cast<__nv_bfloat16*>(y);
+  p.y2 = static_cast<__nv_bfloat16*>(y2);
+  p.act = act; p.act_a = act_a; p.act_b = act_b;
+  p.groups = groups > 1 ? groups : 1; p.x_group = groups > 1 ? x_group : 0; p.y_group = groups > 1 ? y_group : 0;
+  if (groups <= 1 && persist_mode() > 0) {
+    const int th = tbvops::gemm_tok_choose(M, N, K, ldy, epi, persist_mode());
+    if (th > 0) return tbvops::gemm_tok_launch_p(w, x, p, ldx, epi, th, stream);
   }
-  const int mt = (M + 127) / 128, nt = (N + bn - 1) / bn;
-  p.raster = nt > 1 ? 1 : 0;
-  const dim3 grid(p.raster ? nt : mt, p.raster ? mt : nt, splits);
-  cudaStream_t st = static_cast<cudaStream_t>(stream);
-  cudaError_t e = epi == kEpiSiluMul ? pdl::launch(k_gemm<kEpiSiluMul>, grid, dim3(gemm::kThreads), smem, st, splits, tmA, tmB, p)
-                                     : pdl::launch(k_gemm<kEpiStore>, grid, dim3(gemm::kThreads), smem, st, splits, tmA, tmB, p);
-  if (e != cudaSuccess) {
-    fprintf(stderr, "[tbvops] gemm launch failed: %s (M=%d N=%d K=%d bn=%d splits=%d stages=%d)\n", cudaGetErrorString(e), M, N, K,
-            bn, splits, stages);
-    return -1;
-  }
-  return 0;
+  return launch_decode_form(w, x, ldx, p, epi, 0, static_cast<cudaStream_t>(stream));
 }
 
 // Announce the weights of the GEMM that will run after the next one launched from this host thread: that launch's CTAs ask

@@ -34,11 +34,34 @@ struct Params {
   int a_after_wait;    // 1: operand A (w) may have been written by the preceding kernel: fetch it only after the dependency wait
   const __nv_bfloat16* bias;  // [M] or null
   __nv_bfloat16* y;
+  // fp32 output (kEpiF32): activation after the bias, and an optional bf16 copy of the result under the same indexing
+  float* yf;
+  __nv_bfloat16* y2;
+  int act;             // Act below
+  float act_a, act_b;  // softcap: limit; clamped GLU: limit, slope of the sigmoid
+  // grouped form (decode-form kernel): `groups` problems of M features side by side; group g multiplies rows g * M .. of w
+  // with columns g * x_group .. of x and writes at column g * y_group.  groups <= 1: one plain problem.
+  int groups, x_group, y_group;
   unsigned long long limit_ns;  // bound on every barrier wait
   int* err;                     // device flag: set to 1 if a wait gave up
   const char* pf_ptr;           // weights of the GEMM that runs next (or null): see the producer's last step
   unsigned long long pf_bytes;  // how much of them to ask into L2 (a multiple of 16), shared out over the CTAs
 };
+
+enum Epi : int { kEpiStore = 0, kEpiSiluMul = 1, kEpiF32 = 2, kEpiClampGlu = 3 };
+enum Act : int { kActNone = 0, kActSoftplus = 1, kActSoftcap = 2 };
+
+__device__ __forceinline__ float apply_act(float v, int act, float a) {
+  if (act == kActSoftplus) return v > 20.f ? v : log1pf(expf(v));
+  if (act == kActSoftcap) return a * tanhf(v / a);
+  return v;
+}
+// clamped gated unit: g = min(g, limit), u = clamp(u, -limit, limit); g * sigmoid(slope * g) * (u + 1), all in fp32
+__device__ __forceinline__ float clamp_glu(float g, float u, float limit, float slope) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g / (1.0f + __expf(-slope * g)) * (u + 1.0f);
+}
 
 struct Smem {  // static shared state of one CTA
   unsigned long long full[kMaxStages], empty[kMaxStages], accum;
@@ -53,10 +76,10 @@ __device__ __forceinline__ uint32_t tmem_cols(int bn) {
 }
 
 // Runs the TMA/MMA pipeline.  On return (for all threads) the accumulator for this CTA's
-// K range is complete in TMEM (unless s.abort_flag is set).  Returns the aligned dynamic
+// K range is complete in TMEM (unless s.abort_flag is set).  `xk0`: first column of X that belongs to this problem.  Returns the aligned dynamic
 // shared memory base, which the epilogue may reuse as staging space.
 __device__ __forceinline__ uint8_t* mainloop(const CUtensorMap* tmA, const CUtensorMap* tmB, const Params& p, Smem& s,
-                                             uint8_t* smem_raw, int m0, int n0, int kb0, int nkb) {
+                                             uint8_t* smem_raw, int m0, int n0, int kb0, int nkb, int xk0 = 0) {
   using namespace sm100;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const uint32_t raw = smem_u32(smem_raw);
@@ -107,7 +130,7 @@ __device__ __forceinline__ uint8_t* mainloop(const CUtensorMap* tmA, const CUten
     }
     if (!p.a_after_wait) pdl::grid_dependency_wait();
     for (int i = 0; i < pre; i++)
-      tma_load_2d_hint(b_base + i * b_tile_bytes, tmB, (kb0 + i) * kBK, n0, smem_u32(&s.full[i]), pol_x);
+      tma_load_2d_hint(b_base + i * b_tile_bytes, tmB, xk0 + (kb0 + i) * kBK, n0, smem_u32(&s.full[i]), pol_x);
     issued = pre;
     for (int i = pre; i < nkb; i++) {
       const int st = i % p.stages;
@@ -116,7 +139,7 @@ __device__ __forceinline__ uint8_t* mainloop(const CUtensorMap* tmA, const CUten
       const uint32_t fb = smem_u32(&s.full[st]);
       mbar_expect_tx(fb, kATileBytes + b_tile_bytes);
       tma_load_2d_hint(a_base + st * kATileBytes, tmA, (kb0 + i) * kBK, m0, fb, pol_w);
-      tma_load_2d_hint(b_base + st * b_tile_bytes, tmB, (kb0 + i) * kBK, n0, fb, pol_x);
+      tma_load_2d_hint(b_base + st * b_tile_bytes, tmB, xk0 + (kb0 + i) * kBK, n0, fb, pol_x);
       issued = i + 1;
     }
     // This CTA's own weight tiles are all requested.  Between here and the moment the NEXT GEMM may start (this

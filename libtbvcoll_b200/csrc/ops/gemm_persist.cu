@@ -88,7 +88,24 @@ __device__ __forceinline__ void store16(const gemm::Params& p, int n, int f, con
 #pragma unroll
     for (int j = 0; j < 16; j++) v[j] += __bfloat162float(p.bias[f + j]);
   }
-  if (EPI == 1) {
+  if (EPI == gemm::kEpiF32) {
+#pragma unroll
+    for (int j = 0; j < 16; j++) v[j] = gemm::apply_act(v[j], p.act, p.act_a);
+    float4* dst = reinterpret_cast<float4*>(p.yf + size_t(n) * p.ldy + f);
+#pragma unroll
+    for (int j = 0; j < 4; j++) dst[j] = make_float4(v[4 * j], v[4 * j + 1], v[4 * j + 2], v[4 * j + 3]);
+    if (p.y2) {
+      uint4* d2 = reinterpret_cast<uint4*>(p.y2 + size_t(n) * p.ldy + f);
+      d2[0] = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
+      d2[1] = make_uint4(pack_bf16(v[8], v[9]), pack_bf16(v[10], v[11]), pack_bf16(v[12], v[13]), pack_bf16(v[14], v[15]));
+    }
+  } else if (EPI == gemm::kEpiClampGlu) {
+    float o[8];
+#pragma unroll
+    for (int j = 0; j < 8; j++) o[j] = gemm::clamp_glu(v[2 * j], v[2 * j + 1], p.act_a, p.act_b);
+    *reinterpret_cast<uint4*>(p.y + size_t(n) * p.ldy + (f >> 1)) =
+        make_uint4(pack_bf16(o[0], o[1]), pack_bf16(o[2], o[3]), pack_bf16(o[4], o[5]), pack_bf16(o[6], o[7]));
+  } else if (EPI == 1) {
     uint4 o;
     o.x = pack_bf16(silu_mul_bf16(v[0], v[1]), silu_mul_bf16(v[2], v[3]));
     o.y = pack_bf16(silu_mul_bf16(v[4], v[5]), silu_mul_bf16(v[6], v[7]));
@@ -105,7 +122,8 @@ __device__ __forceinline__ void store16(const gemm::Params& p, int n, int f, con
   }
 }
 
-// EPI 0: store (+bias); 1: SiLU-mul over interleaved gate/up features (output has M / 2 features).
+// EPI 0: store (+bias); 1: SiLU-mul over interleaved gate/up features (output has M / 2 features); 2: fp32 store with
+// an activation; 3: clamped gated unit over interleaved gate/up features.
 template <int EPI, int TH>
 __global__ void __launch_bounds__(Shape<TH>::kThreads, 1)
 k_gemm_tok(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUtensorMap tmW, const gemm::Params p) {
@@ -287,14 +305,14 @@ namespace tbvops {
 // decode-form kernel runs 2 CTAs per SM scheduled by the hardware and costs tiles / SMs / efficiency.
 // Efficiencies are measured on B200 at 4096 tokens (Llama-3-8B shapes).
 int gemm_tok_choose(int M, int N, int K, int ldy, int epi, int mode) {
-  if (!(N >= 384 && (M % 16) == 0 && (K % 8) == 0 && (ldy % 8) == 0 && (epi == 0 || epi == 1))) return 0;
+  if (!(N >= 384 && (M % 16) == 0 && (K % 8) == 0 && (ldy % 8) == 0 && epi >= 0 && epi <= 3)) return 0;
   if (mode == 2) return 1;
   if (mode == 3) return 2;
   const double sms = sm_count();
   const long ft = (M + kFeatTile - 1) / kFeatTile;
   const long t1 = long((N + 127) / 128) * ft, t2 = long((N + 255) / 256) * ft;
   const double r1 = double((t1 + long(sms) - 1) / long(sms)), r2 = double((t2 + long(sms) - 1) / long(sms));
-  const double e_dec = double((M + 127) / 128) * ((N + 255) / 256) / sms / kEffDecode[epi];
+  const double e_dec = double((M + 127) / 128) * ((N + 255) / 256) / sms / kEffDecode[epi & 1];
   const double e1 = r1 / kEffTok1, e2 = 2.0 * r2 / kEffTok2;
   if (e_dec <= e1 && e_dec <= e2) return 0;
   return e1 <= e2 ? 1 : 2;
@@ -303,28 +321,46 @@ int gemm_tok_choose(int M, int N, int K, int ldy, int epi, int mode) {
 int gemm_tok_launch(const void* w, const void* x, void* y, const void* bias, int M, int N, int K, int ldx, int ldy, int epi, int th,
                     void* stream) {
   gemm::Params p{};
-  p.M = M; p.N = N; p.K = K; p.ldy = ldy; p.bn = kFeatTile; p.splits = 1; p.stages = th == 1 ? 4 : 3;
-  p.kb_total = (K + 63) / 64;
+  p.M = M; p.N = N; p.K = K; p.ldy = ldy;
   p.bias = static_cast<const __nv_bfloat16*>(bias);
   p.y = static_cast<__nv_bfloat16*>(y);
+  return gemm_tok_launch_p(w, x, p, ldx, epi, th, stream);
+}
+
+int gemm_tok_launch_p(const void* w, const void* x, gemm::Params& p, int ldx, int epi, int th, void* stream) {
+  p.bn = kFeatTile; p.splits = 1; p.stages = th == 1 ? 4 : 3;
+  p.kb_total = (p.K + 63) / 64;
   p.limit_ns = 2000000000ull;
   p.err = gemm_err_flag();
   if (!g_attr) {
-    cudaError_t a[4] = {cudaFuncSetAttribute(k_gemm_tok<0, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
+    cudaError_t a[8] = {cudaFuncSetAttribute(k_gemm_tok<0, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
                         cudaFuncSetAttribute(k_gemm_tok<1, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
+                        cudaFuncSetAttribute(k_gemm_tok<2, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
+                        cudaFuncSetAttribute(k_gemm_tok<3, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
                         cudaFuncSetAttribute(k_gemm_tok<0, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
-                        cudaFuncSetAttribute(k_gemm_tok<1, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024)};
+                        cudaFuncSetAttribute(k_gemm_tok<1, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
+                        cudaFuncSetAttribute(k_gemm_tok<2, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
+                        cudaFuncSetAttribute(k_gemm_tok<3, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024)};
     for (cudaError_t e : a)
       if (e != cudaSuccess) return -1;
     g_attr = true;
   }
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   int map_rc = 0;
-  cudaError_t e = th == 2 ? (epi == 1 ? launch<1, 2>(w, x, p, ldx, st, &map_rc) : launch<0, 2>(w, x, p, ldx, st, &map_rc))
-                          : (epi == 1 ? launch<1, 1>(w, x, p, ldx, st, &map_rc) : launch<0, 1>(w, x, p, ldx, st, &map_rc));
+  cudaError_t e;
+  switch (epi * 2 + (th == 2 ? 1 : 0)) {
+    case 1: e = launch<0, 2>(w, x, p, ldx, st, &map_rc); break;
+    case 2: e = launch<1, 1>(w, x, p, ldx, st, &map_rc); break;
+    case 3: e = launch<1, 2>(w, x, p, ldx, st, &map_rc); break;
+    case 4: e = launch<2, 1>(w, x, p, ldx, st, &map_rc); break;
+    case 5: e = launch<2, 2>(w, x, p, ldx, st, &map_rc); break;
+    case 6: e = launch<3, 1>(w, x, p, ldx, st, &map_rc); break;
+    case 7: e = launch<3, 2>(w, x, p, ldx, st, &map_rc); break;
+    default: e = launch<0, 1>(w, x, p, ldx, st, &map_rc); break;
+  }
   if (map_rc != 0) return map_rc;
   if (e != cudaSuccess) {
-    fprintf(stderr, "[tbvops] many-token gemm launch failed: %s (M=%d N=%d K=%d tile %dx256)\n", cudaGetErrorString(e), M, N, K, 128 * th);
+    fprintf(stderr, "[tbvops] many-token gemm launch failed: %s (M=%d N=%d K=%d tile %dx256)\n", cudaGetErrorString(e), p.M, p.N, p.K, 128 * th);
     return -1;
   }
   return 0;

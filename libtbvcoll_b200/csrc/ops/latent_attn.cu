@@ -1,0 +1,694 @@
+// latent_attn.cu — attention over a compressed (latent) paged cache, with a learned sink per head.
+//
+// A cached token is one row of Dk = Rp + rotp values shared by all heads: the normalised latent c (R values, padded to Rp)
+// and one rotated key part (padded to rotp).  Head h scores it as (q_h . W_uk,h c + q_rot,h . k_rot) * scale and its
+// value is W_uv,h c.  Two forms of the same sum:
+//   rows form     W_uk is folded into the query (qa_h = W_uk,h^T q_h), the cache rows serve as keys AND as values, and the
+//                 result is a latent per head that W_uv expands afterwards.  The cache is read once for all heads: the
+//                 decode form, and the form for portions of a few tokens.
+//   prefill form  keys and values of the visible context are expanded once into dense rows and many query rows share
+//                 them: a third of the arithmetic per (query, key) pair.
+// Scores, softmax and sums are fp32; the denominator contains exp(sink_h) once.
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <stdint.h>
+#include <stdio.h>
+
+#include "../pdl.cuh"
+
+namespace {
+
+constexpr float kNegBig = -1e30f;
+constexpr float kLog2e = 1.4426950408889634f;
+constexpr int kMaxPairs = 512;
+
+__device__ __forceinline__ float to_f(float v) { return v; }
+__device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ void from_f(float& d, float v) { d = v; }
+__device__ __forceinline__ void from_f(__nv_bfloat16& d, float v) { d = __float2bfloat16_rn(v); }
+
+// ---- rotation, latent norm, cache write ------------------------------------------------------------------------------
+struct PrepParams {
+  void* qkv;                // [rows, ldq]: head parts (q_off: rotated parts of all heads), latent (c_off), key part (k_off)
+  void* qa;                 // [n_rows_form, heads, Dk]: rotated query parts of the first n_rows_form rows go to column Rp
+  void* cache;              // [slots, Dk]
+  const float* gamma;       // [R]
+  const float* inv_freq;    // [pairs]
+  const int* positions;
+  const long long* slots;
+  int ldq, q_off, c_off, k_off, heads, R, Rp, rotp, pairs, n_rows_form;
+  float eps, mscale;        // mscale: factor on cos and sin
+};
+
+template <typename T>
+__global__ void __launch_bounds__(256) k_latent_prep(const PrepParams p) {
+  __shared__ float cs[kMaxPairs], sn[kMaxPairs], red[8];
+  pdl::launch_dependents();
+  pdl::grid_dependency_wait();
+  const int row = blockIdx.x, tid = threadIdx.x;
+  T* q = static_cast<T*>(p.qkv) + size_t(row) * p.ldq;
+  const float pos = float(p.positions[row]);
+  for (int i = tid; i < p.pairs; i += 256) {
+    float s, c;
+    sincosf(pos * p.inv_freq[i], &s, &c);
+    cs[i] = c * p.mscale;
+    sn[i] = s * p.mscale;
+  }
+  const T* cv = q + p.c_off;
+  float ss = 0.f;
+  for (int i = tid; i < p.R; i += 256) { const float v = to_f(cv[i]); ss = fmaf(v, v, ss); }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  if ((tid & 31) == 0) red[tid >> 5] = ss;
+  __syncthreads();
+  float tot = 0.f;
+#pragma unroll
+  for (int w = 0; w < 8; w++) tot += red[w];
+  const float r = 1.0f / sqrtf(tot / float(p.R) + p.eps);
+  const int Dk = p.Rp + p.rotp, half = p.rotp / 2;
+  const long long slot = p.slots[row];
+  if (slot >= 0) {
+    T* kc = static_cast<T*>(p.cache) + size_t(slot) * Dk;
+    for (int i = tid; i < p.Rp; i += 256) from_f(kc[i], i < p.R ? to_f(cv[i]) * r * p.gamma[i] : 0.f);
+    const T* kr = q + p.k_off;
+    for (int i = tid; i < half; i += 256) {
+      const float a = to_f(kr[2 * i]), b = to_f(kr[2 * i + 1]);
+      const bool rot = i < p.pairs;
+      from_f(kc[p.Rp + 2 * i], rot ? a * cs[i] - b * sn[i] : a);
+      from_f(kc[p.Rp + 2 * i + 1], rot ? b * cs[i] + a * sn[i] : b);
+    }
+  }
+  const bool rows_form = row < p.n_rows_form;
+  T* qr = q + p.q_off;
+  for (int j = tid; j < p.heads * half; j += 256) {
+    const int h = j / half, i = j - h * half;
+    const float a = to_f(qr[h * p.rotp + 2 * i]), b = to_f(qr[h * p.rotp + 2 * i + 1]);
+    const bool rot = i < p.pairs;
+    T* dst = rows_form ? static_cast<T*>(p.qa) + (size_t(row) * p.heads + h) * Dk + p.Rp + 2 * i : qr + h * p.rotp + 2 * i;
+    from_f(dst[0], rot ? a * cs[i] - b * sn[i] : a);
+    from_f(dst[1], rot ? b * cs[i] + a * sn[i] : b);
+  }
+}
+
+// ---- rows form ---------------------------------------------------------------------------------------------------------
+struct RowsParams {
+  const void* qa;           // [rows, heads, Dk]
+  const void* cache;        // [slots, Dk]
+  const int* tables;        // [nseq, max_blocks]
+  const int* seq_of_row;    // [rows] or null
+  const int* ctx_lens;      // [rows]
+  const float* sink;        // [heads] or null
+  void* out;                // [rows, heads, Rp]
+  int heads, R, Rp, rotp, block_size, max_blocks, splits;
+  float scale_log2;
+};
+
+// fp32: one CTA per (row, head), tiles of 128 keys
+__global__ void __launch_bounds__(128) k_latent_rows_f32(const RowsParams p) {
+  extern __shared__ float sm[];
+  __shared__ float red[4];
+  pdl::launch_dependents();
+  pdl::grid_dependency_wait();
+  const int row = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, Dk = p.Rp + p.rotp;
+  float* sq = sm;            // [Dk]
+  float* sp = sm + Dk;       // [128]
+  int* sl = reinterpret_cast<int*>(sp + 128);
+  const float* qa = static_cast<const float*>(p.qa) + (size_t(row) * p.heads + h) * Dk;
+  for (int i = tid; i < Dk; i += 128) sq[i] = qa[i];
+  const float* cache = static_cast<const float*>(p.cache);
+  const int ctx = min(p.ctx_lens[row], p.max_blocks * p.block_size);
+  const int* bt = p.tables + size_t(p.seq_of_row ? p.seq_of_row[row] : row) * p.max_blocks;
+  constexpr int kAcc = 16;   // Rp <= 2048
+  float o[kAcc];
+#pragma unroll
+  for (int k = 0; k < kAcc; k++) o[k] = 0.f;
+  float m = kNegBig, l = 0.f;
+  for (int t0 = 0; t0 < ctx; t0 += 128) {
+    const int n = min(128, ctx - t0);
+    __syncthreads();
+    float s = kNegBig;
+    if (tid < n) {
+      const int tok = t0 + tid, slot = bt[tok / p.block_size] * p.block_size + tok % p.block_size;
+      sl[tid] = slot;
+      const float4* kr = reinterpret_cast<const float4*>(cache + size_t(slot) * Dk);
+      const float4* q4 = reinterpret_cast<const float4*>(sq);
+      float a = 0.f;
+      for (int i = 0; i < Dk / 4; i++) {
+        const float4 k = kr[i], q = q4[i];
+        a = fmaf(q.x, k.x, a); a = fmaf(q.y, k.y, a); a = fmaf(q.z, k.z, a); a = fmaf(q.w, k.w, a);
+      }
+      s = a * p.scale_log2;
+    }
+    float mx = s;
+#pragma unroll
+    for (int d = 16; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
+    if ((tid & 31) == 0) red[tid >> 5] = mx;
+    __syncthreads();
+    const float mn = fmaxf(m, fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3])));
+    const float pr = tid < n ? exp2f(s - mn) : 0.f, corr = exp2f(m - mn);
+    sp[tid] = pr;
+    float ps = pr;
+#pragma unroll
+    for (int d = 16; d > 0; d >>= 1) ps += __shfl_xor_sync(0xffffffffu, ps, d);
+    __syncthreads();
+    if ((tid & 31) == 0) red[tid >> 5] = ps;
+    __syncthreads();
+    l = l * corr + (red[0] + red[1] + red[2] + red[3]);
+    m = mn;
+#pragma unroll
+    for (int k = 0; k < kAcc; k++) {
+      const int d = tid + k * 128;
+      if (d < p.R) {
+        float acc = o[k] * corr;
+        for (int t = 0; t < n; t++) acc = fmaf(sp[t], cache[size_t(sl[t]) * Dk + d], acc);
+        o[k] = acc;
+      }
+    }
+  }
+  float c = 1.f;
+  if (p.sink) {
+    const float sk = p.sink[h] * kLog2e, mf = fmaxf(m, sk);
+    c = exp2f(m - mf);
+    l = l * c + exp2f(sk - mf);
+  }
+  float* out = static_cast<float*>(p.out) + (size_t(row) * p.heads + h) * p.Rp;
+#pragma unroll
+  for (int k = 0; k < kAcc; k++) {
+    const int d = tid + k * 128;
+    if (d < p.Rp) out[d] = d < p.R && l > 0.f ? o[k] * c / l : 0.f;
+  }
+}
+
+__device__ __forceinline__ uint32_t smem_addr(const void* p) { return static_cast<uint32_t>(__cvta_generic_to_shared(p)); }
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+__device__ __forceinline__ void st_zero16(uint32_t dst) { asm volatile("st.shared.v4.u32 [%0], {%1,%1,%1,%1};" ::"r"(dst), "r"(0u) : "memory"); }
+__device__ __forceinline__ void ldmatrix_x4(uint32_t addr, uint32_t* r) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldmatrix_x2(uint32_t addr, uint32_t* r) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(addr));
+}
+__device__ __forceinline__ void ldmatrix_x4_trans(uint32_t addr, uint32_t* r) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void mma_bf16(float* d, const uint32_t* a, uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
+  __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
+  return *reinterpret_cast<uint32_t*>(&v);
+}
+__device__ __forceinline__ float ld_cluster_f32(uint32_t addr, uint32_t rank) {
+  uint32_t r;
+  float v;
+  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(addr), "r"(rank));
+  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(r) : "memory");
+  return v;
+}
+__device__ __forceinline__ void cluster_sync() {
+  asm volatile("barrier.cluster.arrive.release.aligned;\nbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+
+// bf16: 16 heads of one row per CTA on tensor cores.  Eight warps share tiles of TT cached tokens (two cp.async stages, row
+// pitch Dk * 2 + 16 bytes so that ldmatrix is conflict-free): for the scores warp w takes tokens 8w.. of the tile over all Dk
+// columns; for the weighted sum it takes the latent columns of the 16-column blocks w, w + 8, .. (CBW of them).  grid (rows, head tiles,
+// splits), cluster (1, 1, splits): the CTAs of a cluster cover disjoint token ranges and merge in split order.
+constexpr int kRW = 8;
+constexpr int kMaxSplits = 8;
+template <int CBW, int TT>
+__global__ void __launch_bounds__(kRW * 32, 1) k_latent_rows_mma(const RowsParams p) {
+  extern __shared__ __align__(128) uint8_t dsm[];
+  __shared__ float sh_max[kRW][16], sh_l[kRW][16], sh_ml[16][2], sh_fac[kMaxSplits][16];
+  __shared__ __align__(16) uint8_t sh_p[16 * (TT * 2 + 16)];
+  pdl::launch_dependents();
+  pdl::grid_dependency_wait();
+  const int row = blockIdx.x, h0 = blockIdx.y * 16, sp = blockIdx.z, S = p.splits;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r8 = lane >> 2, quad = lane & 3;
+  const int Dk = p.Rp + p.rotp, chunks = Dk / 8, pitch = Dk * 2 + 16, ksteps = Dk / 16, cblocks = p.Rp / 16;
+  const uint32_t sq = smem_addr(dsm), sk0 = sq + 16 * pitch, stage = uint32_t(TT) * pitch, spb = smem_addr(sh_p);
+  constexpr int kPP = TT * 2 + 16;
+  const int ctx = min(p.ctx_lens[row], p.max_blocks * p.block_size);
+  const int* bt = p.tables + size_t(p.seq_of_row ? p.seq_of_row[row] : row) * p.max_blocks;
+  int chunk = (ctx + S - 1) / S;
+  chunk = (chunk + TT - 1) / TT * TT;
+  const int t0 = min(ctx, sp * chunk), t1 = min(ctx, t0 + chunk);
+  const int ntiles = (t1 - t0 + TT - 1) / TT;
+
+  const __nv_bfloat16* qa = static_cast<const __nv_bfloat16*>(p.qa) + (size_t(row) * p.heads + h0) * Dk;
+  for (int r = warp; r < 16; r += kRW)
+    for (int c = lane; c < chunks; c += 32) {
+      if (h0 + r < p.heads) cp_async16(sq + r * pitch + c * 16, qa + size_t(r) * Dk + c * 8);
+      else st_zero16(sq + r * pitch + c * 16);
+    }
+  const __nv_bfloat16* cache = static_cast<const __nv_bfloat16*>(p.cache);
+  auto issue = [&](int i) {
+    if (i < ntiles) {
+      const uint32_t dst = sk0 + (i & 1) * stage;
+      for (int r = warp; r < TT; r += kRW) {
+        const int tok = t0 + i * TT + r;
+        if (tok < t1) {
+          const __nv_bfloat16* src = cache + (size_t(bt[tok / p.block_size]) * p.block_size + tok % p.block_size) * Dk;
+          for (int c = lane; c < chunks; c += 32) cp_async16(dst + r * pitch + c * 16, src + c * 8);
+        } else {
+          for (int c = lane; c < chunks; c += 32) st_zero16(dst + r * pitch + c * 16);
+        }
+      }
+    }
+    cp_async_commit();
+  };
+  float o[CBW][2][4];
+#pragma unroll
+  for (int b = 0; b < CBW; b++)
+#pragma unroll
+    for (int n = 0; n < 2; n++) o[b][n][0] = o[b][n][1] = o[b][n][2] = o[b][n][3] = 0.f;
+  float m_lo = kNegBig, m_hi = kNegBig, l_lo = 0.f, l_hi = 0.f;
+  issue(0);
+  for (int i = 0; i < ntiles; i++) {
+    issue(i + 1);
+    cp_async_wait<1>();
+    __syncthreads();
+    const uint32_t sk = sk0 + (i & 1) * stage;
+    float sc[4] = {0.f, 0.f, 0.f, 0.f}, sd[4] = {0.f, 0.f, 0.f, 0.f};
+    const bool has_s = warp * 8 < TT;
+    if (has_s) {
+      // two accumulators: consecutive k steps do not wait for one another
+      const uint32_t qaddr = sq + (lane & 15) * pitch + (lane >> 4) * 16;
+      const uint32_t kaddr = sk + (warp * 8 + (lane & 7)) * pitch + (lane >> 3) * 16;
+      int ks = 0;
+      for (; ks + 1 < ksteps; ks += 2) {
+        uint32_t a0[4], a1[4], b[4];
+        ldmatrix_x4(qaddr + ks * 32, a0);
+        ldmatrix_x4(qaddr + ks * 32 + 32, a1);
+        ldmatrix_x4(kaddr + ks * 32, b);
+        mma_bf16(sc, a0, b[0], b[1]);
+        mma_bf16(sd, a1, b[2], b[3]);
+      }
+      if (ks < ksteps) {
+        uint32_t a0[4], b[2];
+        ldmatrix_x4(qaddr + ks * 32, a0);
+        ldmatrix_x2(sk + (warp * 8 + (lane & 7)) * pitch + ((lane >> 3) & 1) * 16 + ks * 32, b);
+        mma_bf16(sc, a0, b[0], b[1]);
+      }
+      const int tok = t0 + i * TT + warp * 8 + quad * 2;
+#pragma unroll
+      for (int j = 0; j < 4; j++) sc[j] = tok + (j & 1) < t1 ? (sc[j] + sd[j]) * p.scale_log2 : kNegBig;
+      float x_lo = fmaxf(sc[0], sc[1]), x_hi = fmaxf(sc[2], sc[3]);
+      x_lo = fmaxf(x_lo, __shfl_xor_sync(0xffffffffu, x_lo, 1));
+      x_lo = fmaxf(x_lo, __shfl_xor_sync(0xffffffffu, x_lo, 2));
+      x_hi = fmaxf(x_hi, __shfl_xor_sync(0xffffffffu, x_hi, 1));
+      x_hi = fmaxf(x_hi, __shfl_xor_sync(0xffffffffu, x_hi, 2));
+      if (quad == 0) { sh_max[warp][r8] = x_lo; sh_max[warp][r8 + 8] = x_hi; }
+    }
+    __syncthreads();
+    float n_lo = m_lo, n_hi = m_hi;
+#pragma unroll
+    for (int w = 0; w < TT / 8; w++) { n_lo = fmaxf(n_lo, sh_max[w][r8]); n_hi = fmaxf(n_hi, sh_max[w][r8 + 8]); }
+    const float c_lo = exp2f(m_lo - n_lo), c_hi = exp2f(m_hi - n_hi);
+    m_lo = n_lo;
+    m_hi = n_hi;
+    l_lo *= c_lo;
+    l_hi *= c_hi;
+    if (has_s) {
+      const float p0 = exp2f(sc[0] - n_lo), p1 = exp2f(sc[1] - n_lo), p2 = exp2f(sc[2] - n_hi), p3 = exp2f(sc[3] - n_hi);
+      l_lo += p0 + p1;
+      l_hi += p2 + p3;
+      *reinterpret_cast<uint32_t*>(sh_p + r8 * kPP + (warp * 8 + quad * 2) * 2) = pack_bf16(p0, p1);
+      *reinterpret_cast<uint32_t*>(sh_p + (r8 + 8) * kPP + (warp * 8 + quad * 2) * 2) = pack_bf16(p2, p3);
+    }
+    __syncthreads();
+#pragma unroll
+    for (int b = 0; b < CBW; b++)
+#pragma unroll
+      for (int n = 0; n < 2; n++) { o[b][n][0] *= c_lo; o[b][n][1] *= c_lo; o[b][n][2] *= c_hi; o[b][n][3] *= c_hi; }
+#pragma unroll
+    for (int ks = 0; ks < TT / 16; ks++) {
+      uint32_t a[4];
+      ldmatrix_x4(spb + (lane & 15) * kPP + (lane >> 4) * 16 + ks * 32, a);
+#pragma unroll
+      for (int b = 0; b < CBW; b++) {
+        const int cb = warp + b * kRW;
+        if (cb < cblocks) {
+          uint32_t v[4];
+          ldmatrix_x4_trans(sk + (ks * 16 + (lane & 15)) * pitch + cb * 32 + (lane >> 4) * 16, v);
+          mma_bf16(o[b][0], a, v[0], v[1]);
+          mma_bf16(o[b][1], a, v[2], v[3]);
+        }
+      }
+    }
+    __syncthreads();   // this stage may be refilled
+  }
+  cp_async_wait<0>();
+  l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1);
+  l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
+  l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1);
+  l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
+  if (quad == 0) { sh_l[warp][r8] = l_lo; sh_l[warp][r8 + 8] = l_hi; }
+  if (warp == 0 && quad == 0) { sh_ml[r8][0] = m_lo; sh_ml[r8 + 8][0] = m_hi; }
+  __syncthreads();     // also: every warp is done with the tiles, whose space now takes the partial results
+  float* so = reinterpret_cast<float*>(dsm);   // [16][Rp]
+#pragma unroll
+  for (int b = 0; b < CBW; b++) {
+    const int cb = warp + b * kRW;
+    if (cb < cblocks) {
+#pragma unroll
+      for (int n = 0; n < 2; n++) {
+        const int col = cb * 16 + n * 8 + quad * 2;
+        *reinterpret_cast<float2*>(so + r8 * p.Rp + col) = make_float2(o[b][n][0], o[b][n][1]);
+        *reinterpret_cast<float2*>(so + (r8 + 8) * p.Rp + col) = make_float2(o[b][n][2], o[b][n][3]);
+      }
+    }
+  }
+  if (tid < 16) {
+    float l = 0.f;
+#pragma unroll
+    for (int w = 0; w < kRW; w++) l += sh_l[w][tid];
+    sh_ml[tid][1] = l;
+  }
+  if (S > 1) cluster_sync();
+  else __syncthreads();
+  // factor of every split's partial sum, the sink and the division included
+  if (tid < 16) {
+    const float sk = p.sink && h0 + tid < p.heads ? p.sink[h0 + tid] * kLog2e : kNegBig;
+    const uint32_t a = smem_addr(&sh_ml[tid][0]);
+    float ms[kMaxSplits], mx = sk, l = 0.f;
+    for (int r = 0; r < S; r++) { ms[r] = S > 1 ? ld_cluster_f32(a, r) : sh_ml[tid][0]; mx = fmaxf(mx, ms[r]); }
+    for (int r = 0; r < S; r++) l = fmaf(S > 1 ? ld_cluster_f32(a + 4, r) : sh_ml[tid][1], exp2f(ms[r] - mx), l);
+    if (p.sink) l += exp2f(sk - mx);
+    for (int r = 0; r < S; r++) sh_fac[r][tid] = l > 0.f ? exp2f(ms[r] - mx) / l : 0.f;
+  }
+  __syncthreads();
+  const int nh = min(16, p.heads - h0), total = nh * p.Rp / 2, per = (total + S - 1) / S;
+  __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + (size_t(row) * p.heads + h0) * p.Rp;
+  const uint32_t soa = smem_addr(so);
+  for (int i = tid; i < per; i += kRW * 32) {
+    const int idx = sp * per + i;
+    if (idx < total) {
+      const int h = idx * 2 / p.Rp;
+      float x = 0.f, y = 0.f;
+      for (int r = 0; r < S; r++) {
+        const float f = sh_fac[r][h];
+        if (S > 1) {
+          x = fmaf(ld_cluster_f32(soa + idx * 8, r), f, x);
+          y = fmaf(ld_cluster_f32(soa + idx * 8 + 4, r), f, y);
+        } else {
+          x = so[idx * 2] * f;
+          y = so[idx * 2 + 1] * f;
+        }
+      }
+      *reinterpret_cast<uint32_t*>(out + idx * 2) = pack_bf16(x, y);
+    }
+  }
+  if (S > 1) cluster_sync();   // nobody leaves while a peer may still read its shared memory
+}
+
+// ---- prefill form --------------------------------------------------------------------------------------------------------
+// cache rows of the visible context -> dense latents [n, Rp] and rotated key parts [n, rotp]
+__global__ void __launch_bounds__(256) k_latent_gather(const uint4* __restrict__ cache, const long long* __restrict__ slots, uint4* c, uint4* kr,
+                                                       int n, int cu, int ku) {
+  pdl::launch_dependents();
+  pdl::grid_dependency_wait();
+  const int w = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (w >= n) return;
+  const uint4* src = cache + size_t(slots[w]) * (cu + ku);
+  for (int i = lane; i < cu + ku; i += 32) {
+    const uint4 v = src[i];
+    if (i < cu) c[size_t(w) * cu + i] = v;
+    else kr[size_t(w) * ku + i - cu] = v;
+  }
+}
+
+struct PrefillParams {
+  const __nv_bfloat16 *q, *kv, *kr;   // q [rows, ldq]; kv [ctx rows, ldkv]: keys at h * dimp, values at v_off + h * vdp; kr [ctx rows, rotp]
+  __nv_bfloat16* out;                 // [rows, ldo], head h at h * vdp
+  const int* tiles;                   // [ntiles, 4]: first query row, rows (<= 64), first dense context row, keys the first row sees
+  const float* sink;
+  int ldq, q_rot_off, ldkv, v_off, ldo, dimp, rotp, vdp;
+  float scale_log2;
+};
+
+// 64 query rows of one sequence and one head per CTA, four warps of 16 rows; key / value tiles of 64 tokens in two cp.async stages.
+constexpr int kPK = 64;
+template <int VT>
+__global__ void __launch_bounds__(128, 2) k_latent_prefill_mma(const PrefillParams p) {
+  extern __shared__ __align__(128) uint8_t dsm[];
+  pdl::launch_dependents();
+  pdl::grid_dependency_wait();
+  const int* tl = p.tiles + 4 * blockIdx.y;
+  const int row0 = tl[0], nrows = tl[1], ctx0 = tl[2], see0 = tl[3], h = blockIdx.x;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r8 = lane >> 2, quad = lane & 3;
+  const int Dq = p.dimp + p.rotp, ksteps = Dq / 16, pq = Dq * 2 + 16, pv = p.vdp * 2 + 16, vblocks = p.vdp / 16;
+  const uint32_t sq = smem_addr(dsm), sk0 = sq + 64 * pq, sv0 = sk0 + 2 * kPK * pq;
+  const int nkeys = see0 + nrows - 1, ntiles = (nkeys + kPK - 1) / kPK;
+  const int nch = p.dimp / 8, rch = p.rotp / 8, vch = p.vdp / 8;
+
+  // rows are copied by groups of lanes: 4 rows per warp pass, 8 lanes per row
+  const int g8 = lane >> 3, l8 = lane & 7;
+  for (int r = warp * 4 + g8; r < 64; r += 16) {
+    const uint32_t d = sq + r * pq;
+    if (r < nrows) {
+      const __nv_bfloat16* src = p.q + size_t(row0 + r) * p.ldq;
+      for (int c = l8; c < nch; c += 8) cp_async16(d + c * 16, src + h * p.dimp + c * 8);
+      for (int c = l8; c < rch; c += 8) cp_async16(d + (nch + c) * 16, src + p.q_rot_off + h * p.rotp + c * 8);
+    } else {
+      for (int c = l8; c < nch + rch; c += 8) st_zero16(d + c * 16);
+    }
+  }
+  auto issue = [&](int i) {
+    if (i < ntiles) {
+      const uint32_t kb = sk0 + (i & 1) * kPK * pq, vb = sv0 + (i & 1) * kPK * pv;
+      for (int r = warp * 4 + g8; r < kPK; r += 16) {
+        const int tok = i * kPK + r;
+        const uint32_t kd = kb + r * pq, vd = vb + r * pv;
+        if (tok < nkeys) {
+          const __nv_bfloat16* src = p.kv + size_t(ctx0 + tok) * p.ldkv;
+          const __nv_bfloat16* srk = p.kr + size_t(ctx0 + tok) * p.rotp;
+          for (int c = l8; c < nch; c += 8) cp_async16(kd + c * 16, src + h * p.dimp + c * 8);
+          for (int c = l8; c < rch; c += 8) cp_async16(kd + (nch + c) * 16, srk + c * 8);
+          for (int c = l8; c < vch; c += 8) cp_async16(vd + c * 16, src + p.v_off + h * p.vdp + c * 8);
+        } else {
+          for (int c = l8; c < nch + rch; c += 8) st_zero16(kd + c * 16);
+          for (int c = l8; c < vch; c += 8) st_zero16(vd + c * 16);
+        }
+      }
+    }
+    cp_async_commit();
+  };
+  float o[VT * 2][4];
+#pragma unroll
+  for (int n = 0; n < VT * 2; n++) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
+  float m_lo = kNegBig, m_hi = kNegBig, l_lo = 0.f, l_hi = 0.f;
+  const int see_lo = see0 + warp * 16 + r8, see_hi = see_lo + 8;   // keys visible to this lane's two rows
+  issue(0);
+  for (int i = 0; i < ntiles; i++) {
+    issue(i + 1);
+    cp_async_wait<1>();
+    __syncthreads();
+    const int tok0 = i * kPK;
+    if (tok0 < see0 + warp * 16 + 15) {          // otherwise every key of the tile is hidden from this warp's rows
+      const uint32_t sk = sk0 + (i & 1) * kPK * pq, sv = sv0 + (i & 1) * kPK * pv;
+      float s[kPK / 8][4];
+#pragma unroll
+      for (int n = 0; n < kPK / 8; n++) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
+      const uint32_t qaddr = sq + (warp * 16 + (lane & 15)) * pq + (lane >> 4) * 16;
+      const uint32_t kaddr = sk + ((lane & 7) + ((lane >> 4) << 3)) * pq + ((lane >> 3) & 1) * 16;
+      for (int ks = 0; ks < ksteps; ks++) {
+        uint32_t a[4];
+        ldmatrix_x4(qaddr + ks * 32, a);
+#pragma unroll
+        for (int n = 0; n < kPK / 16; n++) {
+          uint32_t b[4];
+          ldmatrix_x4(kaddr + n * 16 * pq + ks * 32, b);
+          mma_bf16(s[2 * n], a, b[0], b[1]);
+          mma_bf16(s[2 * n + 1], a, b[2], b[3]);
+        }
+      }
+      float x_lo = m_lo, x_hi = m_hi;
+      if (tok0 + kPK > see0 + warp * 16) {       // the diagonal
+#pragma unroll
+        for (int n = 0; n < kPK / 8; n++)
+#pragma unroll
+          for (int j = 0; j < 2; j++) {
+            const int tok = tok0 + n * 8 + quad * 2 + j;
+            s[n][j] = tok < see_lo ? s[n][j] * p.scale_log2 : kNegBig;
+            s[n][2 + j] = tok < see_hi ? s[n][2 + j] * p.scale_log2 : kNegBig;
+          }
+      } else {
+#pragma unroll
+        for (int n = 0; n < kPK / 8; n++)
+#pragma unroll
+          for (int j = 0; j < 4; j++) s[n][j] *= p.scale_log2;
+      }
+#pragma unroll
+      for (int n = 0; n < kPK / 8; n++) { x_lo = fmaxf(x_lo, fmaxf(s[n][0], s[n][1])); x_hi = fmaxf(x_hi, fmaxf(s[n][2], s[n][3])); }
+      x_lo = fmaxf(x_lo, __shfl_xor_sync(0xffffffffu, x_lo, 1));
+      x_lo = fmaxf(x_lo, __shfl_xor_sync(0xffffffffu, x_lo, 2));
+      x_hi = fmaxf(x_hi, __shfl_xor_sync(0xffffffffu, x_hi, 1));
+      x_hi = fmaxf(x_hi, __shfl_xor_sync(0xffffffffu, x_hi, 2));
+      const float c_lo = exp2f(m_lo - x_lo), c_hi = exp2f(m_hi - x_hi);
+      m_lo = x_lo;
+      m_hi = x_hi;
+      float t_lo = 0.f, t_hi = 0.f;
+      uint32_t pa[kPK / 16][4];
+#pragma unroll
+      for (int n = 0; n < kPK / 8; n++) {
+        const float p0 = exp2f(s[n][0] - x_lo), p1 = exp2f(s[n][1] - x_lo), p2 = exp2f(s[n][2] - x_hi), p3 = exp2f(s[n][3] - x_hi);
+        t_lo += p0 + p1;
+        t_hi += p2 + p3;
+        pa[n >> 1][(n & 1) * 2] = pack_bf16(p0, p1);
+        pa[n >> 1][(n & 1) * 2 + 1] = pack_bf16(p2, p3);
+      }
+      l_lo = l_lo * c_lo + t_lo;
+      l_hi = l_hi * c_hi + t_hi;
+#pragma unroll
+      for (int n = 0; n < VT * 2; n++) { o[n][0] *= c_lo; o[n][1] *= c_lo; o[n][2] *= c_hi; o[n][3] *= c_hi; }
+#pragma unroll
+      for (int b = 0; b < VT; b++) {
+        if (b < vblocks) {
+#pragma unroll
+          for (int ks = 0; ks < kPK / 16; ks++) {
+            uint32_t v[4];
+            ldmatrix_x4_trans(sv + (ks * 16 + (lane & 15)) * pv + b * 32 + (lane >> 4) * 16, v);
+            mma_bf16(o[2 * b], pa[ks], v[0], v[1]);
+            mma_bf16(o[2 * b + 1], pa[ks], v[2], v[3]);
+          }
+        }
+      }
+    }
+    __syncthreads();
+  }
+  cp_async_wait<0>();
+  l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1);
+  l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
+  l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1);
+  l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
+  float f_lo = 1.f, f_hi = 1.f;
+  if (p.sink) {
+    const float sk = p.sink[h] * kLog2e, x_lo = fmaxf(m_lo, sk), x_hi = fmaxf(m_hi, sk);
+    f_lo = exp2f(m_lo - x_lo);
+    f_hi = exp2f(m_hi - x_hi);
+    l_lo = l_lo * f_lo + exp2f(sk - x_lo);
+    l_hi = l_hi * f_hi + exp2f(sk - x_hi);
+  }
+  f_lo = l_lo > 0.f ? f_lo / l_lo : 0.f;
+  f_hi = l_hi > 0.f ? f_hi / l_hi : 0.f;
+  const int rl = warp * 16 + r8, rh = rl + 8;
+#pragma unroll
+  for (int n = 0; n < VT * 2; n++) {
+    if (n < vblocks * 2) {
+      const int col = h * p.vdp + n * 8 + quad * 2;
+      if (rl < nrows) *reinterpret_cast<uint32_t*>(p.out + size_t(row0 + rl) * p.ldo + col) = pack_bf16(o[n][0] * f_lo, o[n][1] * f_lo);
+      if (rh < nrows) *reinterpret_cast<uint32_t*>(p.out + size_t(row0 + rh) * p.ldo + col) = pack_bf16(o[n][2] * f_hi, o[n][3] * f_hi);
+    }
+  }
+}
+
+constexpr size_t kMaxSmem = 226 * 1024;
+
+template <typename K>
+cudaError_t allow_smem(K kern, size_t bytes, bool* done) {
+  if (*done || bytes <= 48 * 1024) return cudaSuccess;
+  cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(kMaxSmem));
+  if (e == cudaSuccess) *done = true;
+  return e;
+}
+
+template <int CBW, int TT>
+cudaError_t launch_rows(const RowsParams& p, dim3 grid, size_t smem, cudaStream_t st) {
+  static bool done = false;
+  cudaError_t e = allow_smem(k_latent_rows_mma<CBW, TT>, smem, &done);
+  return e != cudaSuccess ? e : pdl::launch(k_latent_rows_mma<CBW, TT>, grid, dim3(kRW * 32), smem, st, p.splits, p);
+}
+template <int VT>
+cudaError_t launch_prefill(const PrefillParams& p, dim3 grid, size_t smem, cudaStream_t st) {
+  static bool done = false;
+  cudaError_t e = allow_smem(k_latent_prefill_mma<VT>, smem, &done);
+  return e != cudaSuccess ? e : pdl::launch(k_latent_prefill_mma<VT>, grid, dim3(128), smem, st, 1, p);
+}
+size_t rows_smem(int Dk, int TT) { return size_t(16 + 2 * TT) * (Dk * 2 + 16); }
+size_t prefill_smem(int Dq, int vdp) { return size_t(64 + 2 * kPK) * (Dq * 2 + 16) + size_t(2) * kPK * (vdp * 2 + 16); }
+
+}  // namespace
+
+extern "C" {
+
+int tbv_op_latent_prep(void* qkv, void* qa, void* cache, const void* gamma, const void* inv_freq, const void* positions, const void* slots,
+                       int rows, int n_rows_form, int ldq, int q_off, int c_off, int k_off, int heads, int R, int Rp, int rotp, int pairs,
+                       float eps, float mscale, int bf16, void* stream) {
+  if (rows <= 0) return 0;
+  if (pairs > kMaxPairs || pairs * 2 > rotp || R > Rp || (Rp % 16) || (rotp % 16) || n_rows_form > rows) return -2;
+  PrepParams p{qkv, qa, cache, static_cast<const float*>(gamma), static_cast<const float*>(inv_freq), static_cast<const int*>(positions),
+               static_cast<const long long*>(slots), ldq, q_off, c_off, k_off, heads, R, Rp, rotp, pairs, n_rows_form, eps, mscale};
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  cudaError_t e = bf16 ? pdl::launch(k_latent_prep<__nv_bfloat16>, dim3(rows), dim3(256), 0, st, 1, p)
+                       : pdl::launch(k_latent_prep<float>, dim3(rows), dim3(256), 0, st, 1, p);
+  return e == cudaSuccess ? 0 : -1;
+}
+
+int tbv_op_latent_attn_rows(const void* qa, const void* cache, const void* tables, const void* seq_of_row, const void* ctx_lens,
+                            const void* sink, void* out, int rows, int heads, int R, int Rp, int rotp, int block_size, int max_blocks,
+                            int splits, float scale, int bf16, void* stream) {
+  if (rows <= 0) return 0;
+  if (heads <= 0 || R > Rp || (Rp % 16) || (rotp % 16) || block_size <= 0) return -2;
+  RowsParams p{qa, cache, static_cast<const int*>(tables), static_cast<const int*>(seq_of_row), static_cast<const int*>(ctx_lens),
+               static_cast<const float*>(sink), out, heads, R, Rp, rotp, block_size, max_blocks, 1, scale * kLog2e};
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  cudaError_t e;
+  if (!bf16) {
+    if (Rp > 2048) return -2;
+    e = pdl::launch(k_latent_rows_f32, dim3(rows, heads), dim3(128), size_t(Rp + rotp + 256) * 4, st, 1, p);
+    return e == cudaSuccess ? 0 : -1;
+  }
+  p.splits = splits < 1 ? 1 : (splits > kMaxSplits ? kMaxSplits : splits);
+  const int Dk = Rp + rotp;
+  const dim3 grid(rows, (heads + 15) / 16, p.splits);
+  const size_t s64 = rows_smem(Dk, 64), s32 = rows_smem(Dk, 32);   // either holds the [16][Rp] fp32 partials too
+  if (Rp <= 128) e = launch_rows<1, 64>(p, grid, s64, st);
+  else if (Rp <= 256) e = launch_rows<2, 64>(p, grid, s64, st);
+  else if (Rp <= 512 && s64 <= kMaxSmem - 8192) e = launch_rows<4, 64>(p, grid, s64, st);
+  else if (Rp <= 1024 && s32 <= kMaxSmem - 8192) e = launch_rows<8, 32>(p, grid, s32, st);
+  else return -2;
+  if (e != cudaSuccess) fprintf(stderr, "[tbvops] latent attention launch failed: %s\n", cudaGetErrorString(e));
+  return e == cudaSuccess ? 0 : -1;
+}
+
+int tbv_op_latent_gather(const void* cache, const void* slots, void* c, void* kr, int n, int Rp, int rotp, void* stream) {
+  if (n <= 0) return 0;
+  if ((Rp % 16) || (rotp % 16)) return -2;
+  cudaError_t e = pdl::launch(k_latent_gather, dim3((n + 7) / 8), dim3(256), 0, static_cast<cudaStream_t>(stream), 1,
+                              static_cast<const uint4*>(cache), static_cast<const long long*>(slots), static_cast<uint4*>(c),
+                              static_cast<uint4*>(kr), n, Rp / 8, rotp / 8);
+  return e == cudaSuccess ? 0 : -1;
+}
+
+// 1 if the prefill form takes these sizes (bf16)
+int tbv_op_latent_prefill_fits(int dimp, int rotp, int vdp) { return vdp <= 256 && prefill_smem(dimp + rotp, vdp) <= kMaxSmem ? 1 : 0; }
+
+int tbv_op_latent_prefill(const void* q, const void* kv, const void* kr, const void* tiles, const void* sink, void* out, int ntiles,
+                          int heads, int ldq, int q_rot_off, int ldkv, int v_off, int ldo, int dimp, int rotp, int vdp, float scale,
+                          void* stream) {
+  if (ntiles <= 0) return 0;
+  if ((dimp % 16) || (rotp % 16) || (vdp % 16) || (ldq % 8) || (ldkv % 8) || (q_rot_off % 8) || (v_off % 8) || ntiles > 65535) return -2;
+  if (!tbv_op_latent_prefill_fits(dimp, rotp, vdp)) return -2;
+  PrefillParams p{static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(kv), static_cast<const __nv_bfloat16*>(kr),
+                  static_cast<__nv_bfloat16*>(out), static_cast<const int*>(tiles), static_cast<const float*>(sink),
+                  ldq, q_rot_off, ldkv, v_off, ldo, dimp, rotp, vdp, scale * kLog2e};
+  const size_t smem = prefill_smem(dimp + rotp, vdp);
+  const dim3 grid(heads, ntiles);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  cudaError_t e;
+  if (vdp <= 32) e = launch_prefill<2>(p, grid, smem, st);
+  else if (vdp <= 64) e = launch_prefill<4>(p, grid, smem, st);
+  else if (vdp <= 128) e = launch_prefill<8>(p, grid, smem, st);
+  else e = launch_prefill<16>(p, grid, smem, st);
+  if (e != cudaSuccess) fprintf(stderr, "[tbvops] latent prefill launch failed: %s\n", cudaGetErrorString(e));
+  return e == cudaSuccess ? 0 : -1;
+}
+
+}  // extern "C"

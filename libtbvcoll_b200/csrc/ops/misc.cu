@@ -118,18 +118,21 @@ __global__ void k_embedding(const long long* __restrict__ ids, const __nv_bfloat
 // holding it.  Stage 1: `nblk` CTAs per row write partials; stage 2: the last CTA of a row
 // (atomic ticket) folds them in block order — deterministic, first index wins ties like
 // torch.argmax.
-__global__ void k_argmax(const __nv_bfloat16* __restrict__ logits, int vocab, int ld, long long index_offset,
+__device__ __forceinline__ float logit(float v) { return v; }
+__device__ __forceinline__ float logit(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename T>
+__global__ void k_argmax(const T* __restrict__ logits, int vocab, int ld, long long index_offset,
                          float* part_val, long long* part_idx, unsigned* tickets, float* out_val, long long* out_idx) {
   pdl::launch_dependents();
   pdl::grid_dependency_wait();
   const int row = blockIdx.y, nblk = gridDim.x;
   const int per = (vocab + nblk - 1) / nblk;
   const int v0 = blockIdx.x * per, v1 = min(vocab, v0 + per);
-  const __nv_bfloat16* x = logits + size_t(row) * ld;
+  const T* x = logits + size_t(row) * ld;
   float best = -FLT_MAX;
   int bi = 0x7fffffff;
   for (int i = v0 + threadIdx.x; i < v1; i += blockDim.x) {
-    const float f = __bfloat162float(x[i]);
+    const float f = logit(x[i]);
     if (f > best) { best = f; bi = i; }  // ascending i per thread: first index kept on ties
   }
   __shared__ float sv[32];
@@ -209,6 +212,22 @@ __global__ void k_decode_advance(const long long* __restrict__ next_ids, long lo
   if (b == 0) *step_counter = step + 1;
 }
 
+template <typename T>
+int run_argmax(const void* logits, int tokens, int vocab, int ld, long long index_offset, void* workspace, void* out_val,
+                  void* out_idx, void* stream) {
+  if (tokens <= 0) return 0;
+  int nblk = (vocab + 4095) / 4096;
+  nblk = nblk < 1 ? 1 : (nblk > 64 ? 64 : nblk);
+  char* ws = static_cast<char*>(workspace);
+  unsigned* tickets = reinterpret_cast<unsigned*>(ws);
+  float* pv = reinterpret_cast<float*>(ws + ((size_t(tokens) * 4 + 255) & ~size_t(255)));
+  long long* pi = reinterpret_cast<long long*>(reinterpret_cast<char*>(pv) + size_t(tokens) * 64 * 4);
+  cudaError_t e = pdl::launch(k_argmax<T>, dim3(nblk, tokens), dim3(256), 0, static_cast<cudaStream_t>(stream), 1,
+                              static_cast<const T*>(logits), vocab, ld, index_offset, pv, pi, tickets,
+                              static_cast<float*>(out_val), static_cast<long long*>(out_idx));
+  return e == cudaSuccess ? 0 : -1;
+}
+
 }  // namespace
 
 extern "C" {
@@ -280,17 +299,11 @@ size_t tbv_op_argmax_workspace(int tokens) {
 }
 int tbv_op_argmax(const void* logits, int tokens, int vocab, int ld, long long index_offset, void* workspace, void* out_val,
                   void* out_idx, void* stream) {
-  if (tokens <= 0) return 0;
-  int nblk = (vocab + 4095) / 4096;
-  nblk = nblk < 1 ? 1 : (nblk > 64 ? 64 : nblk);
-  char* ws = static_cast<char*>(workspace);
-  unsigned* tickets = reinterpret_cast<unsigned*>(ws);
-  float* pv = reinterpret_cast<float*>(ws + ((size_t(tokens) * 4 + 255) & ~size_t(255)));
-  long long* pi = reinterpret_cast<long long*>(reinterpret_cast<char*>(pv) + size_t(tokens) * 64 * 4);
-  cudaError_t e = pdl::launch(k_argmax, dim3(nblk, tokens), dim3(256), 0, static_cast<cudaStream_t>(stream), 1,
-                              static_cast<const __nv_bfloat16*>(logits), vocab, ld, index_offset, pv, pi, tickets,
-                              static_cast<float*>(out_val), static_cast<long long*>(out_idx));
-  return e == cudaSuccess ? 0 : -1;
+  return run_argmax<__nv_bfloat16>(logits, tokens, vocab, ld, index_offset, workspace, out_val, out_idx, stream);
+}
+int tbv_op_argmax_f32(const void* logits, int tokens, int vocab, int ld, long long index_offset, void* workspace, void* out_val,
+                      void* out_idx, void* stream) {
+  return run_argmax<float>(logits, tokens, vocab, ld, index_offset, workspace, out_val, out_idx, stream);
 }
 // vals / idx point at rank 0's candidates; rank r's are rank_stride_bytes further on.
 int tbv_op_argmax_merge(const void* vals, const void* idx, int world, int tokens, long long rank_stride_bytes, void* out,

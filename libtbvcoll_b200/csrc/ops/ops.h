@@ -2,6 +2,8 @@
 #pragma once
 #include <cuda.h>
 
+namespace gemm { struct Params; }
+
 namespace tbvops {
 int make_tensor_map_bf16(CUtensorMap* out, const void* ptr, unsigned long long rows, unsigned long long cols,
                          unsigned long long ld, unsigned box_rows, bool cache = true);
@@ -12,11 +14,14 @@ int* gemm_err_flag();
 unsigned long long take_next_prefetch(const char** ptr, unsigned long long own_bytes);
 void set_next_prefetch(const void* ptr, unsigned long long bytes);
 int sm_count();
-void gemm_config(int M, int N, int K, int splits_hint, int* bn_out, int* splits_out, int* stages_out);
+void gemm_config(int M, int N, int K, int splits_hint, int* bn_out, int* splits_out, int* stages_out, int groups = 1,
+                 bool f32_out = false);
 // many-token (prefill) persistent kernel, gemm_persist.cu
 int gemm_tok_choose(int M, int N, int K, int ldy, int epi, int mode);
 int gemm_tok_launch(const void* w, const void* x, void* y, const void* bias, int M, int N, int K, int ldx, int ldy, int epi, int th,
                     void* stream);
+// the same for a filled parameter block (M, N, K, ldy, outputs, epilogue arguments)
+int gemm_tok_launch_p(const void* w, const void* x, gemm::Params& p, int ldx, int epi, int th, void* stream);
 // evenly-split (stream-K) decode GEMM, gemm_streamk.cu
 bool gemm_streamk_wants(int M, int N, int K, int epi, int splits_hint, bool w_not_constant);
 int gemm_streamk_launch(const void* w, const void* x, void* y, const void* bias, int M, int N, int K, int ldx, int ldy, int epi,

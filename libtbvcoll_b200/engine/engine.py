@@ -27,11 +27,11 @@ import numpy as np
 import torch
 
 from .. import ops
-from ..models.config import ModelConfig
-from ..models.llama import LlamaTP
+from ..models.registry import architecture_of
 from ..parallel.tp import TPGroup
-from ..utils.weights import RandomSource, shard_for_rank
-from .kv_cache import BlockManager
+from ..utils.weights import RandomSource
+from .batch import Portion, StepBatch, lay_out
+from .kv_cache import BlockManager, RequestTable
 
 
 def _nvtx(name: str):
@@ -43,18 +43,11 @@ def _nvtx(name: str):
 
 def prefill_rows(prompts: Sequence[Sequence[int]], tables: np.ndarray, block_size: int):
     """Flat per-row arrays over all prompts, rows grouped by sequence in position order:
-    (total rows, sequence of row, position, token id, KV-cache slot, is-last-row-of-its-prompt).
-    numpy throughout: a 4096-row prefill must not spend milliseconds in Python loops."""
-    B = len(prompts)
-    lens = np.fromiter((len(p) for p in prompts), dtype=np.int64, count=B)
-    total = int(lens.sum())
-    seq_all = np.repeat(np.arange(B, dtype=np.int64), lens)
-    starts = np.cumsum(lens) - lens
-    pos_all = np.arange(total, dtype=np.int64) - np.repeat(starts, lens)
-    ids_all = np.concatenate([np.asarray(p, dtype=np.int64) for p in prompts]) if total else np.zeros(0, dtype=np.int64)
-    slots_all = tables[seq_all, pos_all // block_size].astype(np.int64) * block_size + pos_all % block_size
-    is_last = pos_all == (lens[seq_all] - 1)
-    return total, seq_all, pos_all, ids_all, slots_all, is_last
+    (total rows, sequence of row, position, token id, KV-cache slot, is-last-row-of-its-prompt)."""
+    hb = lay_out([Portion(b, 0, p, (len(p) - 1,)) for b, p in enumerate(prompts)], tables, block_size)
+    is_last = np.zeros(hb.ids.size, dtype=bool)
+    is_last[hb.want_rows] = True
+    return int(hb.ids.size), hb.seq, hb.pos, hb.ids, hb.slots, is_last
 
 
 class _GraphChain:
@@ -69,22 +62,30 @@ class _GraphChain:
 
 
 class Engine:
-    def __init__(self, cfg: ModelConfig, tp: Optional[TPGroup] = None, device="cuda:0", weights: Optional[Dict[str, torch.Tensor]] = None,
+    def __init__(self, cfg, tp: Optional[TPGroup] = None, device="cuda:0", weights: Optional[Dict[str, torch.Tensor]] = None,
                  source=None, seed: int = 0, max_batch: int = 8, max_seq_len: int = 1024, block_size: int = 16,
-                 prefill_chunk: int = 2048, max_attn_splits: int = 32):
-        self.cfg = cfg
+                 prefill_chunk: int = 2048, max_attn_splits: int = 32, dtype: torch.dtype = torch.bfloat16,
+                 max_cache_tokens: Optional[int] = None):
+        """``cfg``: a configuration of any registered architecture.  ``max_cache_tokens``: size of the cache pool (default: ``max_batch``
+        sequences of ``max_seq_len`` tokens each)."""
+        arch = architecture_of(cfg)
+        if str(dtype).split(".")[-1] not in arch.dtypes:
+            raise ValueError(f"{arch.name} models do not run in {dtype}")
+        self.cfg, self.dtype = cfg, dtype
         self.tp = tp or TPGroup()
         self.device = torch.device(device)
         self.max_batch, self.max_seq_len, self.block_size = max_batch, max_seq_len, block_size
         self.prefill_chunk = prefill_chunk
         if weights is None:
             source = source or RandomSource(cfg, seed=seed, device=self.device)
-            weights = shard_for_rank(cfg, source, self.tp.rank, self.tp.world, self.device)
+            weights = arch.model().load_weights(cfg, source, self.tp, self.device, dtype)
         max_blocks_per_seq = (max_seq_len + block_size - 1) // block_size
-        num_blocks = max_batch * max_blocks_per_seq + 1
+        pool = max_batch * max_blocks_per_seq if max_cache_tokens is None else (max_cache_tokens + block_size - 1) // block_size
+        num_blocks = pool + 1          # block 0 is never handed out
         self.bm = BlockManager(num_blocks, block_size, max_batch, max_blocks_per_seq, self.device)
-        self.model = LlamaTP(cfg, self.tp, weights, self.device, max_tokens=max(prefill_chunk, max_batch), max_batch=max_batch,
-                             num_blocks=num_blocks, block_size=block_size, max_attn_splits=max_attn_splits)
+        self.requests = RequestTable(self.bm)
+        self.model = arch.model()(cfg, self.tp, weights, self.device, max_tokens=max(prefill_chunk, max_batch), max_batch=max_batch,
+                                  num_blocks=num_blocks, block_size=block_size, max_attn_splits=max_attn_splits, dtype=dtype)
         dev, B = self.device, max_batch
         # Static decode inputs (graph-captured addresses): ONE device block and ONE pinned mirror, so that a step's inputs
         # cross PCIe as a single copy:  ids int64[B] | cache slots int64[B] | positions int32[B] | context lengths int32[B]
@@ -102,6 +103,12 @@ class Engine:
         # serving loop: layers in a short first graph of a step (0 = one graph per step, the default: measured 3.327 ms per step
         # with 0, 3.323 / 3.327 / 3.348 with 1 / 2 / 4 head layers on the 8B shape; replaying the graph costs the host 13 us); see capture()
         self.serve_head_layers = int(os.environ.get("TBV_SERVE_HEAD", "0"))
+        # one-token segments of a decode step: row i is a sequence whose state slot is i + 1 (idle: the dummy slot 0)
+        seg = torch.zeros(B, 4, dtype=torch.int32)
+        seg[:, 0], seg[:, 1] = torch.arange(B), 1
+        self.idle_segs = seg.to(dev)
+        seg[:, 2] = torch.arange(B) + 1
+        self.decode_segs = seg.to(dev)
         self.step_counter = torch.zeros(1, dtype=torch.int32, device=dev)
         self.history = torch.zeros(max_seq_len, B, dtype=torch.int64, device=dev)
         # Sequence-parallel prefill (GEMM->reduce-scatter, all-gather->GEMM) for chunks whose row count divides evenly.
@@ -126,43 +133,100 @@ class Engine:
         Returns the first generated token of every sequence."""
         B = len(prompts)
         assert 0 < B <= self.max_batch
+        self.requests.end_all()
         self.bm.release_all()
         for b, p in enumerate(prompts):
             if len(p) + reserve_new > self.max_seq_len:
                 raise ValueError("prompt + new tokens exceed max_seq_len")
             self.bm.reserve(b, len(p) + reserve_new)
         self.bm.sync_to_device()
-        total, seq_all, pos_all, ids_all, slots_all, is_last = prefill_rows(prompts, self.bm.tables_host.numpy(), self.bm.block_size)
         first = [0] * B
-        dev = self.device
-        for c0 in range(0, total, self.prefill_chunk):
-            c1 = min(total, c0 + self.prefill_chunk)
-            T = c1 - c0
-            pos = torch.from_numpy(pos_all[c0:c1].astype(np.int32))
-            seqof = torch.from_numpy(seq_all[c0:c1].astype(np.int32))
-            last_r = np.nonzero(is_last[c0:c1])[0]
-            n_log = int(last_r.size)
-            out = torch.zeros(max(n_log, 1), dtype=torch.int64, device=dev)
-            logit_rows = torch.from_numpy(last_r if n_log else np.zeros(1, dtype=np.int64)).to(dev)
-            tiles = ops.prefill_tiles(seqof, self.model.nq // self.model.nkv).to(dev) if self.tiled_prefill_attention else None
-            ids_d, slots_d = torch.from_numpy(ids_all[c0:c1]).to(dev), torch.from_numpy(slots_all[c0:c1]).to(dev)
-            pos_d, ctx_d, seq_d = pos.to(dev), (pos + 1).to(dev), seqof.to(dev)
-            if self.sp_prefill and self.model.sp_ok(T):
-                self.model.forward_sp(T, ids_d, pos_d, slots_d, self.bm.tables, ctx_d, seq_d, logit_rows, max(n_log, 1), out, prefill_tiles=tiles)
+        for parts in self._chunks([Portion(b, 0, p, (len(p) - 1,)) for b, p in enumerate(prompts)]):
+            rows = [p.row for p in parts if len(p.want)]
+            out = torch.zeros(max(len(rows), 1), dtype=torch.int64, device=self.device)
+            batch = self.batch_of(parts, out_tokens=out)
+            if self.sp_prefill and hasattr(self.model, "sp_ok") and self.model.sp_ok(batch.T):
+                sel = batch.logit_rows if rows else torch.zeros(1, dtype=torch.int64, device=self.device)
+                self.model.forward_sp(batch.T, batch.ids, batch.positions, batch.slots, self.bm.tables, batch.ctx, batch.seq_of_row, sel,
+                                      max(len(rows), 1), out, prefill_tiles=batch.tiles)
                 self.sp_chunks += 1
             else:
-                self.model.forward(T, ids_d, pos_d, slots_d, self.bm.tables, ctx_d, seq_d, logit_rows, max(n_log, 1), out, attn_splits=1,
-                                   prefill_tiles=tiles)
-            if n_log:
-                toks = out[:n_log].tolist()
-                for r, t in zip(last_r.tolist(), toks):
-                    first[int(seq_all[c0 + r])] = t
+                self.model.forward_batch(batch)
+            if rows:
+                for b, t in zip(rows, out[: len(rows)].tolist()):
+                    first[b] = t
         return first
 
+    def _chunks(self, parts: Sequence[Portion]):
+        """The portions cut into passes of at most ``prefill_chunk`` rows (a sequence may straddle passes)."""
+        cur, room = [], self.prefill_chunk
+        for p in parts:
+            n, at = len(p.tokens), 0
+            while at < n:
+                k = min(room, n - at)
+                cur.append(Portion(p.row, p.start + at, p.tokens[at:at + k], tuple(w - at for w in p.want if at <= w < at + k)))
+                at += k
+                room -= k
+                if room == 0:
+                    yield cur
+                    cur, room = [], self.prefill_chunk
+        if cur:
+            yield cur
+
+    def batch_of(self, parts: Sequence[Portion], out_tokens: Optional[torch.Tensor] = None, logits_out: Optional[torch.Tensor] = None) -> StepBatch:
+        """Device arrays of one pass over ``parts`` (blocks reserved, tables on the device)."""
+        m, dev = self.model, self.device
+        hb = lay_out(parts, self._tables_np, self.block_size, m.rows_form_max)
+        put = lambda a, dt: torch.from_numpy(np.ascontiguousarray(a.astype(dt, copy=False))).to(dev)
+        T = int(hb.ids.size)
+        b = StepBatch(T=T, ids=put(hb.ids, np.int64), positions=put(hb.pos, np.int32), slots=put(hb.slots, np.int64), tables=self.bm.tables,
+                      ctx=put(hb.pos + 1, np.int32), n_logits=int(hb.want_rows.size), seq_of_row=put(hb.seq, np.int32),
+                      logit_rows=put(hb.want_rows, np.int64), out_tokens=out_tokens, logits_out=logits_out, n_rows_form=hb.n_rows_form)
+        if m.uses_state:
+            b.segs, b.seg_of_row = put(hb.segs, np.int32), put(hb.seg, np.int32)
+        if m.rows_form_max:
+            if hb.n_rows_form:
+                b.attn_splits = self.attn_splits_for(hb.n_rows_form, int(hb.pos[: hb.n_rows_form].max()) + 1)
+            if hb.n_rows_form < T:
+                b.dense_tiles, b.dense_slots = put(hb.dense_tiles, np.int32), put(hb.dense_slots, np.int64)
+        elif self.tiled_prefill_attention:
+            b.tiles = ops.prefill_tiles(torch.from_numpy(hb.seq.astype(np.int32)), m.nq // m.nkv).to(dev)
+        return b
+
+    # ---- one mixed step ---------------------------------------------------------------------------
+    def step(self, entries, end=(), sample: bool = False):
+        """One step over live requests: ``entries`` = (request id, next tokens, wanted offsets among them) per request — whole prompts,
+        portions of prompts and single tokens side by side.  A request is admitted at its first entry and keeps its row, blocks and
+        state until it is named in ``end`` (given back after this step).  Returns the fp32 logits [wanted, vocab] in the order of
+        the entries and offsets, or the greedy tokens (list) with ``sample``.  ``generate`` resets the same cache: do not mix the two
+        while requests are live."""
+        parts, n = [], 0
+        for key, tokens, want in entries:
+            r = self.requests.extend(key, len(tokens))
+            parts.append(Portion(r.row, r.length, list(tokens), tuple(want)))
+            n += len(want)
+        self.bm.sync_to_device()
+        out = torch.empty(n, dtype=torch.int64, device=self.device) if sample else \
+            torch.empty(n, self.cfg.vocab_size, dtype=torch.float32, device=self.device)
+        at = 0
+        for piece in self._chunks(parts):
+            k = sum(len(p.want) for p in piece)
+            self.model.forward_batch(self.batch_of(piece, **{"out_tokens" if sample else "logits_out": out[at: at + k]}))
+            at += k
+        for key in end:
+            self.requests.end(key)
+        if ops.gemm_error():
+            raise RuntimeError("a GEMM barrier wait gave up on the device (see the kernel's watchdog)")
+        return out.tolist() if sample else out
+
     # ---- decode -------------------------------------------------------------------------------
-    def _decode_step(self, B: int, splits: int, advance: bool, layer_begin: int = 0, layer_end: Optional[int] = None) -> None:
-        self.model.forward(B, self.ids[:B], self.positions[:B], self.slots[:B], self.bm.tables, self.ctx[:B], None, None, B,
-                           self.out_tokens, attn_splits=splits, layer_begin=layer_begin, layer_end=layer_end)
+    def _decode_step(self, B: int, splits: int, advance: bool, layer_begin: int = 0, layer_end: Optional[int] = None, idle: bool = False) -> None:
+        """One token per row.  ``idle``: a warm-up pass that must leave no trace — the cache rows it writes are written again
+        by the real step, and carried state goes to the dummy slot."""
+        self.model.forward_batch(StepBatch(T=B, ids=self.ids[:B], positions=self.positions[:B], slots=self.slots[:B], tables=self.bm.tables,
+                                           ctx=self.ctx[:B], n_logits=B, out_tokens=self.out_tokens, attn_splits=splits, n_rows_form=B,
+                                           segs=(self.idle_segs if idle else self.decode_segs)[:B]),
+                                 layer_begin=layer_begin, layer_end=layer_end)
         if advance and (layer_end is None or layer_end == self.cfg.num_layers):
             ops.decode_advance(self.out_tokens[:B], self.ids[:B], self.positions[:B], self.ctx[:B], self.slots[:B], self.bm.tables,
                                self.block_size, self.history, self.step_counter)
@@ -172,7 +236,7 @@ class Engine:
         # kv splits are the CTAs of one cluster: the largest power of two (<= 8) that keeps the whole
         # grid in one wave (two CTAs per SM) and leaves at least 64 cached tokens per CTA
         s = 1
-        while s < 8 and B * self.model.nkv * s * 2 <= 2 * sms and max_ctx // (s * 2) >= 64:
+        while s < 8 and B * self.model.attn_ctas_per_row * s * 2 <= self.model.attn_ctas_per_sm * sms and max_ctx // (s * 2) >= 64:
             s *= 2
         return min(s, self.model.max_attn_splits)
 
@@ -192,7 +256,7 @@ class Engine:
         s.wait_stream(torch.cuda.current_stream(self.device))
         parts = []
         with torch.cuda.stream(s):
-            self._decode_step(B, splits, False)      # eager warm-up: idempotent (no advance)
+            self._decode_step(B, splits, False, idle=True)      # eager warm-up: leaves no trace (no advance)
             s.synchronize()
             n0 = ops.launch_count + self.tp.launches
             for lo, hi in ([(0, head), (head, L)] if 0 < head < L else [(0, L)]):
@@ -225,8 +289,12 @@ class Engine:
                  eos_id: Optional[int] = None) -> List[List[int]]:
         """Greedy generation.  ``loop="host"``: per-step H2D inputs + D2H tokens (serving shape);
         ``loop="device"``: steps chained on the device, tokens read back once at the end.
-        EOS is ignored unless ``eos_id`` is given (the reference bench sets ignore_eos)."""
+        EOS is ignored unless ``eos_id`` is given (the reference bench sets ignore_eos).  More prompts than ``max_batch`` go
+        through the scheduler, which admits them as rows and cache blocks become free."""
         B = len(prompts)
+        if B > self.max_batch:
+            from .scheduler import Scheduler
+            return Scheduler(self).run(prompts, max_new_tokens, eos_id)
         t0 = time.perf_counter()
         with _nvtx("tbv.prefill"):
             first = self.prefill(prompts, max_new_tokens)

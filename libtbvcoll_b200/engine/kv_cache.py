@@ -8,7 +8,7 @@ warm-up point at it, so a stray write can never land in a live sequence.
 """
 from __future__ import annotations
 
-from typing import List
+from typing import Dict, List, NamedTuple
 
 import torch
 
@@ -54,3 +54,43 @@ class BlockManager:
 
     def sync_to_device(self) -> None:
         self.tables.copy_(self.tables_host, non_blocking=True)
+
+
+class Request(NamedTuple):
+    row: int        # batch row: block-table row, and state slot row + 1 in models that carry state (slot 0 is nobody's)
+    length: int     # tokens already in the cache / state
+
+
+class RequestTable:
+    """Live requests of ``Engine.step``: a batch row (with its blocks and state slot) from the first entry to the end, however many
+    steps lie between.  A row that is given back goes to the end of the line; blocks are handed out as tokens arrive.  What a previous owner left
+    in a state slot is never read: a sequence's first token starts from zero."""
+
+    def __init__(self, blocks: BlockManager):
+        self.blocks = blocks
+        self.free_rows: List[int] = list(range(blocks.max_batch))
+        self.live: Dict[object, Request] = {}
+
+    def admit(self, key) -> Request:
+        if key not in self.live:
+            if not self.free_rows:
+                raise RuntimeError(f"more than {self.blocks.max_batch} live requests")
+            self.live[key] = Request(self.free_rows.pop(0), 0)
+        return self.live[key]
+
+    def extend(self, key, tokens: int) -> Request:
+        """Admit if new, make room for ``tokens`` more and count them; returns the request as it was before them."""
+        r = self.admit(key)
+        self.blocks.reserve(r.row, r.length + tokens)
+        self.live[key] = r._replace(length=r.length + tokens)
+        return r
+
+    def end(self, key) -> None:
+        r = self.live.pop(key, None)
+        if r is not None:
+            self.blocks.release(r.row)
+            self.free_rows.append(r.row)
+
+    def end_all(self) -> None:
+        for k in list(self.live):
+            self.end(k)

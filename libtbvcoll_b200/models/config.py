@@ -6,7 +6,7 @@ from __future__ import annotations
 
 import json
 from dataclasses import dataclass, field
-from typing import Optional
+from typing import List, Optional, Union
 
 
 @dataclass
@@ -77,3 +77,139 @@ def from_hf_config(path: str) -> ModelConfig:
         rms_eps=c.get("rms_norm_eps", 1e-5), max_position=c.get("max_position_embeddings", 8192),
         qkv_bias=c.get("attention_bias", c.get("model_type") == "qwen2"), tie_embeddings=c.get("tie_word_embeddings", False),
         rope_scaling=c.get("rope_scaling"))
+
+
+# ---- Nubosun: selective-scan and latent-attention layers over several residual streams ------------------------------------
+@dataclass
+class MambaSpec:
+    inner: int
+    state: int
+    dt_rank: int
+    conv: int                              # taps of the causal convolution, the current token's included
+
+
+@dataclass
+class RotationSpec:
+    dims: int
+    base: float
+    scaling: Optional[dict] = None         # YaRN: factor, original, fast, slow
+
+
+@dataclass
+class LatentSpec:
+    heads: int
+    dim: int                               # unrotated query / key dimensions per head
+    rot_dim: int                           # rotated ones; the key's rotated part is shared by all heads
+    vdim: int
+    kv_rank: int                           # size of the cached latent
+    scale: float
+    rot: RotationSpec = None
+
+
+@dataclass
+class ClampedGluSpec:
+    ff: int
+    limit: float
+    slope: float = 1.702                   # of the sigmoid gate
+
+
+@dataclass
+class LayerSpec:
+    mixer: Union[MambaSpec, LatentSpec]
+    mlp: Optional[ClampedGluSpec] = None
+
+
+@dataclass
+class NubosunConfig:
+    name: str
+    vocab_size: int
+    hidden_size: int
+    layers: List[LayerSpec]
+    streams: int = 1
+    embedding_scale: float = 1.0
+    rms_eps: float = 1e-5
+    logit_softcap: Optional[float] = None
+    loop: Optional[tuple] = None           # (start, stop, times): layers start .. stop-1 run `times` times in a row
+
+    def __post_init__(self):
+        if self.loop is not None:
+            a, b, n = self.loop
+            if not (0 <= a <= b <= len(self.layers) and n >= 0):
+                raise ValueError(f"loop {self.loop} does not fit {len(self.layers)} layers")
+        if not 1 <= self.streams <= 8:
+            raise ValueError(f"{self.streams} residual streams: 1 to 8 are supported")
+
+    def check_tp(self, tp: int) -> None:
+        if tp != 1:
+            raise ValueError("Nubosun models run on one GPU (no tensor-parallel sharding of the scan and the latent cache)")
+
+    @property
+    def runs(self) -> List[int]:
+        """Layer index of every layer run, in order; each run has a cache or state of its own."""
+        n = list(range(len(self.layers)))
+        if self.loop is None:
+            return n
+        a, b, times = self.loop
+        return n[:a] + n[a:b] * times + n[b:]
+
+    @property
+    def num_layers(self) -> int:
+        return len(self.runs)
+
+    def param_count(self) -> int:
+        from ..utils.weights import tensor_shapes
+        total = 0
+        for shape in tensor_shapes(self).values():
+            k = 1
+            for d in shape:
+                k *= d
+            total += k
+        return total
+
+
+def parse_nubosun_config(c: dict) -> NubosunConfig:
+    """``config.json`` of a Nubosun checkpoint."""
+    layers = []
+    for i, e in enumerate(c["layers"]):
+        m = e["mixer"]
+        if e["type"] == "mamba1":
+            mixer = MambaSpec(inner=m["inner"], state=m["state"], dt_rank=m["dt_rank"], conv=m["conv"])
+        elif e["type"] == "latent_attention":
+            r = m["rot"]
+            if r["dims"] % 2 or not 0 <= r["dims"] <= m["rot_dim"]:
+                raise ValueError(f"layer {i}: {r['dims']} rotated dimensions of {m['rot_dim']}")
+            mixer = LatentSpec(heads=m["heads"], dim=m["dim"], rot_dim=m["rot_dim"], vdim=m["vdim"], kv_rank=m["kv_rank"], scale=float(m["scale"]),
+                               rot=RotationSpec(dims=r["dims"], base=float(r["base"]), scaling=r.get("scaling")))
+        else:
+            raise ValueError(f"layer {i}: unknown type {e['type']!r}")
+        mlp = e.get("mlp")
+        if mlp is not None and mlp["kind"] != "dense":
+            raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+        layers.append(LayerSpec(mixer, None if mlp is None else ClampedGluSpec(ff=mlp["ff"], limit=float(mlp["limit"]))))
+    loop = c.get("loop")
+    cap = c.get("logit_softcap")
+    return NubosunConfig(name=c.get("name", "nubosun"), vocab_size=c["vocab"], hidden_size=c["width"], layers=layers, streams=c.get("streams", 1),
+                         embedding_scale=float(c.get("embedding", {}).get("scale", 1.0)), rms_eps=float(c["norm"]["eps"]),
+                         logit_softcap=float(cap) if cap else None,
+                         loop=(loop["start"], loop["stop"], loop["times"]) if loop else None)
+
+
+def nubosun_like(hidden: int, layers: int, ff: int, heads: int, vocab: int, head_dim: int = 128, kv_rank: int = 512, state: int = 16,
+                 attention_every: int = 2, streams: int = 2, name: str = "nubosun") -> NubosunConfig:
+    """A Nubosun of ordinary proportions (inner = 2 x width, dt_rank = width / 16, four taps, half of head_dim rotated): a latent-
+    attention layer with a feed-forward after every ``attention_every`` - 1 selective-scan layers with one."""
+    lay = []
+    for i in range(layers):
+        if (i + 1) % attention_every:
+            mixer = MambaSpec(inner=2 * hidden, state=state, dt_rank=hidden // 16, conv=4)
+        else:
+            mixer = LatentSpec(heads=heads, dim=head_dim, rot_dim=head_dim // 2, vdim=head_dim, kv_rank=kv_rank, scale=(1.5 * head_dim) ** -0.5,
+                               rot=RotationSpec(head_dim // 2, 5e5, {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}))
+        lay.append(LayerSpec(mixer, ClampedGluSpec(ff=ff, limit=7.0)))
+    return NubosunConfig(name=name, vocab_size=vocab, hidden_size=hidden, layers=lay, streams=streams, logit_softcap=30.0)
+
+
+PRESETS["nubosun-8b"] = nubosun_like(4096, 32, 14336, 32, 128256, name="nubosun-8b")
+PRESETS["nubosun-2k"] = nubosun_like(2048, 16, 7168, 16, 32768, name="nubosun-2k")
+PRESETS["llama3-2k"] = ModelConfig(name="llama3-2k", hidden_size=2048, num_layers=16, num_heads=16, num_kv_heads=4, intermediate_size=7168,
+                                   vocab_size=32768)

@@ -26,14 +26,21 @@ from typing import Dict, Optional
 import torch
 
 from .. import ops
+from ..engine.batch import StepBatch
 from ..parallel.tp import TPGroup
 from .config import ModelConfig
 
 
 class LlamaTP:
+    rows_form_max = 0          # one attention form: rows of a step keep their order
+    uses_state = False         # nothing is carried from token to token besides the KV cache
+    attn_ctas_per_sm = 2
+
     def __init__(self, cfg: ModelConfig, tp: TPGroup, weights: Dict[str, torch.Tensor], device, max_tokens: int,
-                 max_batch: int, num_blocks: int, block_size: int = 16, max_attn_splits: int = 32):
+                 max_batch: int, num_blocks: int, block_size: int = 16, max_attn_splits: int = 32, dtype: torch.dtype = torch.bfloat16):
         cfg.check_tp(tp.world)
+        if dtype is not torch.bfloat16:
+            raise ValueError(f"{cfg.name}: the kernels of this model run in bfloat16 only")
         self.cfg, self.tp, self.w, self.device = cfg, tp, weights, torch.device(device)
         self.block_size, self.num_blocks = block_size, num_blocks
         self.nq = cfg.num_heads // tp.world
@@ -68,6 +75,40 @@ class LlamaTP:
         # paged KV cache, one pair per layer: [num_blocks * block_size, nkv, D]
         self.k_cache = [torch.zeros(num_blocks * block_size, self.nkv, self.D, dtype=bf, device=dev) for _ in range(cfg.num_layers)]
         self.v_cache = [torch.zeros(num_blocks * block_size, self.nkv, self.D, dtype=bf, device=dev) for _ in range(cfg.num_layers)]
+
+        self.attn_ctas_per_row = self.nkv
+
+    @staticmethod
+    def load_weights(cfg: ModelConfig, source, tp: TPGroup, device, dtype):
+        from ..utils.weights import shard_for_rank
+        return shard_for_rank(cfg, source, tp.rank, tp.world, device)
+
+    def forward_batch(self, b: StepBatch, layer_begin: int = 0, layer_end: Optional[int] = None) -> None:
+        """``forward`` on a step's batch; logits (gathered over the vocabulary shards) go to ``b.logits_out`` if it is set."""
+        if b.logits_out is None or b.n_logits == 0:
+            rows = b.logit_rows
+            if b.n_logits == 0:    # the pass still runs (it fills the cache); its sampled row is not used
+                rows = torch.zeros(1, dtype=torch.int64, device=self.device)
+            out = b.out_tokens if b.out_tokens is not None and b.n_logits else torch.empty(1, dtype=torch.int64, device=self.device)
+            self.forward(b.T, b.ids, b.positions, b.slots, b.tables, b.ctx, b.seq_of_row, rows, max(b.n_logits, 1), out,
+                         attn_splits=b.attn_splits, prefill_tiles=b.tiles, layer_begin=layer_begin, layer_end=layer_end)
+            return
+        n0 = min(b.n_logits, self.max_batch)
+        out = b.out_tokens if b.out_tokens is not None else torch.empty(n0, dtype=torch.int64, device=self.device)
+        assert b.out_tokens is None or b.n_logits <= self.max_batch
+        self.forward(b.T, b.ids, b.positions, b.slots, b.tables, b.ctx, b.seq_of_row, b.logit_rows[:n0], n0, out, attn_splits=b.attn_splits,
+                     prefill_tiles=b.tiles)
+        for c0 in range(0, b.n_logits, self.max_batch):
+            n = min(self.max_batch, b.n_logits - c0)
+            if c0:
+                torch.index_select(self.xn[: b.T], 0, b.logit_rows[c0: c0 + n], out=self.xl[:n])
+                ops.gemm(self.xl[:n], self.w["lm_head"], out=self.logits[:n])
+            shards = torch.empty(self.tp.world, n, self.vpr, dtype=self.logits.dtype, device=self.device)
+            if self.tp.world == 1:
+                shards[0].copy_(self.logits[:n])
+            else:
+                self.tp.all_gather(self.logits[:n].contiguous(), shards)
+            b.logits_out[c0: c0 + n].copy_(shards.transpose(0, 1).reshape(n, -1))
 
     # -- one forward pass over T token rows ----------------------------------------------------
     def forward(self, T: int, ids: torch.Tensor, positions: torch.Tensor, slot_mapping: torch.Tensor, block_tables: torch.Tensor,

@@ -1,0 +1,55 @@
+"""Which model class, weight layout and loader a configuration belongs to.  The engine, the trace replay, the command line and
+the benchmarks all choose through here."""
+from __future__ import annotations
+
+import json
+import os
+from dataclasses import dataclass
+from typing import Callable, Tuple
+
+from .config import ModelConfig, NubosunConfig, from_hf_config, parse_nubosun_config
+
+
+@dataclass(frozen=True)
+class Architecture:
+    name: str
+    config_type: type
+    model: Callable[[], type]              # imported on use: the model modules need the native library
+    dtypes: Tuple[str, ...]                # compute types the model runs in
+    tensor_parallel: bool
+
+
+def _llama():
+    from .llama import LlamaTP
+    return LlamaTP
+
+
+def _nubosun():
+    from .nubosun import Nubosun
+    return Nubosun
+
+
+ARCHITECTURES = {
+    "llama": Architecture("llama", ModelConfig, _llama, ("bfloat16",), True),
+    "nubosun": Architecture("nubosun", NubosunConfig, _nubosun, ("bfloat16", "float32"), False),
+}
+
+
+def architecture_of(cfg) -> Architecture:
+    for a in ARCHITECTURES.values():
+        if isinstance(cfg, a.config_type):
+            return a
+    raise ValueError(f"no architecture for a configuration of type {type(cfg).__name__}")
+
+
+def load_config(model_dir: str):
+    """Configuration object of a model directory, its kind chosen by ``config.json``."""
+    path = os.path.join(model_dir, "config.json")
+    with open(path) as f:
+        c = json.load(f)
+    arch = str(c.get("architecture", "")).lower()
+    if arch == "nubosun":
+        return parse_nubosun_config(c)
+    if arch:
+        raise ValueError(f"unknown architecture {c['architecture']!r}")
+    return from_hf_config(path)            # Llama / Qwen2 families in the HF layout

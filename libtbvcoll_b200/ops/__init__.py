@@ -33,6 +33,18 @@ def lib():
     I, F, LL, SZ = ctypes.c_int, ctypes.c_float, ctypes.c_longlong, ctypes.c_size_t
     l.tbv_op_gemm.argtypes = [c_vp, c_vp, c_vp, c_vp, I, I, I, I, I, I, I, c_vp]
     l.tbv_op_gemm_error.restype = I
+    l.tbv_op_gemm_ex.argtypes = [c_vp, c_vp, c_vp, c_vp, c_vp, I, I, I, I, I, I, I, F, F, I, I, I, c_vp]
+    l.tbv_op_gemm_f32.argtypes = [c_vp, c_vp, c_vp, c_vp, I, I, I, I, I, I, I, F, F, I, I, I, c_vp]
+    l.tbv_op_argmax_f32.argtypes = [c_vp, I, I, I, LL, c_vp, c_vp, c_vp, c_vp]
+    l.tbv_op_hyper_embed.argtypes = [c_vp, c_vp, LL, F, c_vp, c_vp, c_vp, c_vp, I, I, I, I, I, F, I, c_vp]
+    l.tbv_op_hyper_mix.argtypes = [c_vp, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp, I, I, I, I, I, I, F, I, c_vp]
+    l.tbv_op_causal_conv_silu.argtypes = [c_vp] * 8 + [I] * 6 + [c_vp]
+    l.tbv_op_selective_scan.argtypes = [c_vp] * 11 + [I] * 14 + [c_vp]
+    l.tbv_op_latent_prep.argtypes = [c_vp] * 7 + [I] * 11 + [F, F, I, c_vp]
+    l.tbv_op_latent_attn_rows.argtypes = [c_vp] * 7 + [I] * 8 + [F, I, c_vp]
+    l.tbv_op_latent_gather.argtypes = [c_vp] * 4 + [I] * 3 + [c_vp]
+    l.tbv_op_latent_prefill_fits.argtypes = [I, I, I]
+    l.tbv_op_latent_prefill.argtypes = [c_vp] * 6 + [I] * 10 + [F, c_vp]
     l.tbv_op_gemm_persist_mode.argtypes = [I]
     l.tbv_op_gemm_persist_mode.restype = None
     l.tbv_op_gemm_streamk_min_bytes.argtypes = [ctypes.c_long]
@@ -102,7 +114,8 @@ def _count(n=1):
     launch_count += n
 
 
-EPI_STORE, EPI_SILU_MUL = 0, 1
+EPI_STORE, EPI_SILU_MUL, EPI_F32, EPI_CLAMP_GLU = 0, 1, 2, 3
+ACT_NONE, ACT_SOFTPLUS, ACT_SOFTCAP = 0, 1, 2
 
 
 def gemm(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None,
@@ -125,6 +138,35 @@ def gemm(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, b
     assert out.shape == (N, om) and out.stride(1) == 1
     _chk(lib().tbv_op_gemm(_p(w), _p(x), _p(out), _p(bias), M, N, K, x.stride(0), out.stride(0), epi | (0 if w_is_constant else 0x100), splits, _st()),
          "tbv_op_gemm")
+    _count()
+    return out
+
+
+def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[torch.Tensor] = None, act: int = ACT_NONE, act_arg: float = 0.0,
+           glu: Optional[tuple] = None, copy: Optional[torch.Tensor] = None, groups: int = 1, x_group: int = 0, y_group: int = 0) -> torch.Tensor:
+    """out[N, M] = epilogue(x[N, K] @ w[M, K]^T + bias) for bf16 operands (tcgen05) or fp32 operands (CUDA cores, full 32-bit).
+
+    The output dtype is ``out``'s: fp32 results take an activation (``ACT_SOFTPLUS``, ``ACT_SOFTCAP`` with its limit in ``act_arg``)
+    and, from bf16 operands, an optional bf16 ``copy`` with the same row stride.  ``glu=(limit, slope)``: ``w`` holds gate / up rows
+    interleaved and out[N, M/2] = g * sigmoid(slope * g) * (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit).
+    ``groups`` > 1: w is [groups * M, K]; group g multiplies columns g * x_group .. of x and writes columns g * y_group .. of out."""
+    assert x.is_cuda and x.dtype is w.dtype and x.stride(1) == 1 and w.is_contiguous() and out.stride(1) == 1 and x.shape[0] == out.shape[0]
+    N, K = x.shape[0], w.shape[1]
+    M = w.shape[0] // groups
+    assert x.shape[1] >= (groups - 1) * x_group + K and out.shape[1] >= (groups - 1) * y_group + (M // 2 if glu else M)
+    if N == 0:
+        return out
+    limit, slope = glu if glu else (act_arg, 0.0)
+    if x.dtype is torch.float32:
+        assert out.dtype is torch.float32 and copy is None and (bias is None or bias.dtype is torch.float32)
+        _chk(lib().tbv_op_gemm_f32(_p(w), _p(x), _p(out), _p(bias), M, N, K, x.stride(0), out.stride(0), EPI_CLAMP_GLU if glu else EPI_F32, act,
+                                   limit, slope, groups, x_group, y_group, _st()), "tbv_op_gemm_f32")
+    else:
+        epi = EPI_CLAMP_GLU if glu else (EPI_F32 if out.dtype is torch.float32 else EPI_STORE)
+        assert x.dtype is torch.bfloat16 and (bias is None or bias.dtype is torch.bfloat16) and (epi == EPI_F32 or (act == ACT_NONE and copy is None))
+        assert copy is None or (copy.dtype is torch.bfloat16 and copy.stride(0) == out.stride(0))
+        _chk(lib().tbv_op_gemm_ex(_p(w), _p(x), _p(out), _p(copy), _p(bias), M, N, K, x.stride(0), out.stride(0), epi, act, limit, slope,
+                                  groups, x_group, y_group, _st()), "tbv_op_gemm_ex")
     _count()
     return out
 
@@ -201,6 +243,24 @@ def rope_cos_sin(head_dim: int, max_pos: int, theta: float, device, scaling: Opt
     return torch.cat((f.cos(), f.sin()), dim=-1).contiguous()
 
 
+def rope_frequencies(dims: int, base: float, scaling: Optional[dict] = None):
+    """([dims / 2] float64 frequencies, factor on cos and sin) of a rotation over ``dims`` dimensions; ``scaling`` = YaRN's
+    ``factor``, ``original`` (context), ``fast`` and ``slow`` (turns over that context between which the frequencies blend from
+    unscaled to divided by ``factor``)."""
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    f = float(base) ** (-2.0 * i / dims)
+    if not scaling:
+        return f, 1.0
+    factor, original = float(scaling["factor"]), float(scaling["original"])
+
+    def dim_of(turns):
+        return dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+    lo = max(math.floor(dim_of(float(scaling["fast"]))), 0)
+    hi = min(math.ceil(dim_of(float(scaling["slow"]))), dims - 1)
+    ramp = ((i - lo) / max(hi - lo, 1e-3)).clamp(0.0, 1.0)
+    return f / factor * ramp + f * (1.0 - ramp), 0.1 * math.log(factor) + 1.0
+
+
 def rope_kv(qkv: torch.Tensor, positions: torch.Tensor, cos_sin: torch.Tensor, slot_mapping: Optional[torch.Tensor],
             k_cache: Optional[torch.Tensor], v_cache: Optional[torch.Tensor], nq: int, nkv: int, head_dim: int) -> None:
     """In place: rotate the q and k heads of qkv [T, (nq+2nkv)*D]; write k, v rows into the
@@ -244,7 +304,8 @@ def argmax(logits: torch.Tensor, workspace: torch.Tensor, index_offset: int = 0,
     T, V = logits.shape
     out_val = torch.empty(T, dtype=torch.float32, device=logits.device) if out_val is None else out_val
     out_idx = torch.empty(T, dtype=torch.int64, device=logits.device) if out_idx is None else out_idx
-    _chk(lib().tbv_op_argmax(_p(logits), T, V, logits.stride(0), index_offset, _p(workspace), _p(out_val), _p(out_idx), _st()),
+    fn = lib().tbv_op_argmax_f32 if logits.dtype is torch.float32 else lib().tbv_op_argmax
+    _chk(fn(_p(logits), T, V, logits.stride(0), index_offset, _p(workspace), _p(out_val), _p(out_idx), _st()),
          "tbv_op_argmax")
     _count()
     return out_val, out_idx
@@ -347,3 +408,7 @@ def prefill_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
                                         block_tables.shape[1], scale, _st()), "tbv_op_prefill_attention")
     _count()
     return out
+
+
+from .mixers import (causal_conv_silu, hyper_embed, hyper_mix, latent_attention_prefill, latent_attention_rows, latent_gather,  # noqa: E402,F401
+                     latent_prefill_fits, latent_prep, selective_scan)

@@ -17,7 +17,7 @@ from typing import Callable, Dict, Iterable, Optional
 
 import torch
 
-from ..models.config import ModelConfig
+from ..models.config import LatentSpec, MambaSpec, ModelConfig, NubosunConfig
 
 
 def hf_tensor_shapes(cfg: ModelConfig) -> Dict[str, tuple]:
@@ -43,13 +43,68 @@ def hf_tensor_shapes(cfg: ModelConfig) -> Dict[str, tuple]:
     return shapes
 
 
+def nubosun_tensor_shapes(cfg: NubosunConfig) -> Dict[str, tuple]:
+    W, S = cfg.hidden_size, cfg.streams
+    shapes = {"embed": (cfg.vocab_size, W), "final.norm": (W,), "head": (cfg.vocab_size, W)}
+    for i, lay in enumerate(cfg.layers):
+        p, m = f"l{i}.", lay.mixer
+        for q in (1, 2) if lay.mlp is not None else (1,):
+            shapes[f"{p}norm{q}"] = shapes[f"{p}ls{q}"] = (W,)
+            shapes[f"{p}hc{q}.in"] = shapes[f"{p}hc{q}.out"] = (S,)
+            shapes[f"{p}hc{q}.mix"] = (S, S)
+        if isinstance(m, MambaSpec):
+            shapes.update({p + "mix.in": (2 * m.inner, W), p + "mix.conv": (m.inner, m.conv), p + "mix.conv.b": (m.inner,),
+                           p + "mix.x": (m.dt_rank + 2 * m.state, m.inner), p + "mix.dt": (m.inner, m.dt_rank), p + "mix.dt.b": (m.inner,),
+                           p + "mix.A_log": (m.inner, m.state), p + "mix.D": (m.inner,), p + "mix.o": (W, m.inner)})
+        else:
+            shapes.update({p + "mix.q": (m.heads * (m.dim + m.rot_dim), W), p + "mix.dkv": (m.kv_rank + m.rot_dim, W), p + "mix.dkv.norm": (m.kv_rank,),
+                           p + "mix.uk": (m.heads * m.dim, m.kv_rank), p + "mix.uv": (m.heads * m.vdim, m.kv_rank), p + "mix.sink": (m.heads,),
+                           p + "mix.o": (W, m.heads * m.vdim)})
+        if lay.mlp is not None:
+            shapes.update({p + "mlp.gate": (lay.mlp.ff, W), p + "mlp.up": (lay.mlp.ff, W), p + "mlp.down": (W, lay.mlp.ff)})
+    return shapes
+
+
+def tensor_shapes(cfg) -> Dict[str, tuple]:
+    """Checkpoint tensor names and shapes of a configuration of any architecture."""
+    return nubosun_tensor_shapes(cfg) if isinstance(cfg, NubosunConfig) else hf_tensor_shapes(cfg)
+
+
+def _nubosun_random(name: str, shape: tuple, g: torch.Generator, device) -> torch.Tensor:
+    """Random values that keep a Nubosun's activations near unit size: decays over many time scales, mixing near the identity."""
+    leaf = name.split(".", 1)[1] if name.startswith("l") and "." in name else name
+    n = lambda *s: torch.randn(s or shape, generator=g, device=device, dtype=torch.float32)
+    u = lambda: torch.rand(shape, generator=g, device=device, dtype=torch.float32)
+    if leaf.startswith("norm") or leaf in ("final.norm", "mix.dkv.norm") or leaf.startswith("ls"):
+        return 1.0 + 0.1 * n()
+    if leaf == "mix.A_log":
+        return torch.log(0.5 + 8.0 * u())
+    if leaf == "mix.dt.b":
+        return -4.0 + 3.0 * u()                       # softplus: steps of 0.02 .. 0.3
+    if leaf == "mix.D":
+        return 1.0 + 0.1 * n()
+    if leaf.endswith(".in") and leaf.startswith("hc"):
+        return 1.0 / shape[0] + 0.1 * n()
+    if leaf.endswith(".out"):
+        return 1.0 + 0.2 * n()
+    if leaf.endswith(".mix") and leaf.startswith("hc"):
+        return torch.eye(shape[0], device=device) * 0.9 + 0.05 * n()
+    if leaf in ("mix.sink", "mix.conv.b"):
+        return 0.5 * n()
+    if leaf == "mix.conv":
+        return n() / shape[1] ** 0.5
+    if leaf == "embed":
+        return n()
+    return n() / shape[1] ** 0.5
+
+
 class RandomSource:
     """Seeded random weights under HF names.  A tensor's values depend only on (seed, name),
     never on the TP degree, so every rank slices the same virtual checkpoint."""
 
     def __init__(self, cfg: ModelConfig, seed: int = 0, device="cpu", dtype=torch.bfloat16):
         self.cfg, self.seed, self.device, self.dtype = cfg, seed, torch.device(device), dtype
-        self.shapes = hf_tensor_shapes(cfg)
+        self.shapes = tensor_shapes(cfg)
 
     def names(self) -> Iterable[str]:
         return self.shapes.keys()
@@ -57,7 +112,9 @@ class RandomSource:
     def get(self, name: str) -> torch.Tensor:
         shape = self.shapes[name]
         g = torch.Generator(device=self.device).manual_seed((self.seed * 1000003 + zlib.crc32(name.encode())) & 0x7FFFFFFF)
-        if name.endswith("layernorm.weight") or name.endswith("norm.weight"):
+        if isinstance(self.cfg, NubosunConfig):
+            t = _nubosun_random(name, shape, g, self.device)
+        elif name.endswith("layernorm.weight") or name.endswith("norm.weight"):
             t = 1.0 + 0.1 * torch.randn(shape, generator=g, device=self.device, dtype=torch.float32)
         elif name.endswith(".bias"):
             t = 0.1 * torch.randn(shape, generator=g, device=self.device, dtype=torch.float32)
@@ -129,6 +186,100 @@ def _rows(source, name: str, r0: int, r1: int) -> torch.Tensor:
     if hasattr(source, "get_rows"):
         return source.get_rows(name, r0, r1)
     return source.get(name)[r0:r1]
+
+
+def _pad16(n: int) -> int:
+    return (n + 15) // 16 * 16
+
+
+def _padded(t: torch.Tensor, rows: int, cols: Optional[int] = None) -> torch.Tensor:
+    """Zero-padded copy: [rows] or [rows, cols]."""
+    out = torch.zeros((rows,) if cols is None else (rows, cols), dtype=t.dtype, device=t.device)
+    if cols is None:
+        out[: t.shape[0]] = t
+    else:
+        out[: t.shape[0], : t.shape[1]] = t
+    return out
+
+
+def _pad_heads(t: torch.Tensor, heads: int, dim: int, dim_p: int) -> torch.Tensor:
+    """[heads * dim, K] -> [heads * dim_p, K], each head's rows followed by zero rows."""
+    out = torch.zeros(heads, dim_p, t.shape[1], dtype=t.dtype, device=t.device)
+    out[:, :dim] = t.reshape(heads, dim, -1)
+    return out.reshape(heads * dim_p, -1)
+
+
+def load_nubosun(cfg: NubosunConfig, source, device, dtype=torch.bfloat16) -> Dict[str, torch.Tensor]:
+    """Tensors the way the kernels consume them.  Every dimension that a matrix product runs over is padded with zeros to a multiple
+    of 16 (so that any configuration meets the TMA alignment rules); small parameters that act in 32-bit are fp32.
+
+    Latent attention: ``qkv`` stacks the heads' unrotated query rows, their rotated rows, the latent rows and the rotated key rows;
+    ``wabs`` [heads * rank, dim] folds W_uk into the query, ``wuv`` [heads * vdim, rank] expands a latent, ``wukv`` [heads * (dim + vdim), rank]
+    gives keys then values.  Mamba: ``in`` stacks x rows and z rows, ``conv`` is transposed to [taps, inner], ``a2`` = -exp(A_log) * log2 e."""
+    dev, out = torch.device(device), {}
+    Wp = _pad16(cfg.hidden_size)
+    want = nubosun_tensor_shapes(cfg)
+
+    def get(name):
+        t = source.get(name)
+        if tuple(t.shape) != tuple(want[name]):
+            raise ValueError(f"{name}: shape {tuple(t.shape)}, expected {tuple(want[name])}")
+        return t
+
+    def put(name, t, as_dtype=dtype):
+        out[name] = t.to(as_dtype).to(dev).contiguous()
+
+    f32 = torch.float32
+    put("embed", _padded(get("embed"), cfg.vocab_size, Wp))
+    put("head", _padded(get("head"), _pad16(cfg.vocab_size), Wp))
+    put("final.norm", _padded(get("final.norm"), Wp), f32)
+    for i, lay in enumerate(cfg.layers):
+        p, m = f"l{i}.", lay.mixer
+        for q in (1, 2) if lay.mlp is not None else (1,):
+            put(f"{p}norm{q}", _padded(get(f"{p}norm{q}"), Wp), f32)
+            put(f"{p}ls{q}", _padded(get(f"{p}ls{q}"), Wp), f32)
+            for k in ("in", "out", "mix"):
+                put(f"{p}hc{q}.{k}", get(f"{p}hc{q}.{k}"), f32)
+        x = p + "mix."
+        if isinstance(m, MambaSpec):
+            ip, kd = _pad16(m.inner), _pad16(m.dt_rank)
+            w = get(x + "in")
+            put(x + "in", torch.cat((_padded(w[: m.inner], ip, Wp), _padded(w[m.inner:], ip, Wp))))
+            put(x + "conv", _padded(get(x + "conv").t(), m.conv, ip), f32)
+            put(x + "conv.b", _padded(get(x + "conv.b"), ip), f32)
+            put(x + "x", _padded(get(x + "x"), _pad16(m.dt_rank + 2 * m.state), ip))
+            put(x + "dt", _padded(get(x + "dt"), ip, kd))
+            put(x + "dt.b", _padded(get(x + "dt.b"), ip))
+            put(x + "a2", -torch.exp(get(x + "A_log").float()) * 1.4426950408889634, f32)
+            put(x + "D", get(x + "D"), f32)
+            put(x + "o", _padded(get(x + "o"), Wp, ip))
+        else:
+            H, D, V, R, rot = m.heads, _pad16(m.dim), _pad16(m.vdim), _pad16(m.kv_rank), _pad16(m.rot_dim)
+            q = get(x + "q").reshape(H, m.dim + m.rot_dim, -1)
+            kv = get(x + "dkv")
+            rows = torch.cat((_pad_heads(q[:, : m.dim].reshape(H * m.dim, -1), H, m.dim, D),
+                              _pad_heads(q[:, m.dim:].reshape(H * m.rot_dim, -1), H, m.rot_dim, rot),
+                              _padded(kv[: m.kv_rank], R, kv.shape[1]), _padded(kv[m.kv_rank:], rot, kv.shape[1])))
+            put(x + "qkv", _padded(rows, rows.shape[0], Wp))
+            put(x + "dkv.norm", get(x + "dkv.norm"), f32)
+            put(x + "sink", get(x + "sink"), f32)
+            uk, uv = get(x + "uk"), get(x + "uv")
+            wabs = torch.zeros(H, R, D, dtype=uk.dtype, device=uk.device)
+            wabs[:, : m.kv_rank, : m.dim] = uk.reshape(H, m.dim, m.kv_rank).transpose(1, 2)
+            put(x + "wabs", wabs.reshape(H * R, D))
+            wuv = _padded(_pad_heads(uv, H, m.vdim, V), H * V, R)
+            put(x + "wuv", wuv)
+            if dtype is torch.bfloat16:
+                put(x + "wukv", torch.cat((_padded(_pad_heads(uk, H, m.dim, D), H * D, R), wuv)))
+            o = torch.zeros(Wp, H, V, dtype=uv.dtype, device=uv.device)
+            o[: cfg.hidden_size, :, : m.vdim] = get(x + "o").reshape(cfg.hidden_size, H, m.vdim)
+            put(x + "o", o.reshape(Wp, H * V))
+        if lay.mlp is not None:
+            x, fp = p + "mlp.", _pad16(lay.mlp.ff)
+            g, u = _padded(get(x + "gate"), fp, Wp), _padded(get(x + "up"), fp, Wp)
+            put(x + "gate_up", torch.stack((g, u), 1).reshape(2 * fp, Wp))
+            put(x + "down", _padded(get(x + "down"), Wp, fp))
+    return out
 
 
 def shard_for_rank(cfg: ModelConfig, source, rank: int, tp: int, device, interleave_gate_up: bool = True) -> Dict[str, torch.Tensor]:
