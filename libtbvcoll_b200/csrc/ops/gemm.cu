@@ -464,7 +464,7 @@ int tbv_op_gemm_ex(const void* w, const void* x, void* y, void* y2, const void* 
   p.y2 = static_cast<__nv_bfloat16*>(y2);
   p.act = act; p.act_a = act_a; p.act_b = act_b;
   p.groups = groups > 1 ? groups : 1; p.x_group = groups > 1 ? x_group : 0; p.y_group = groups > 1 ? y_group : 0;
-  if (groups <= 1 && persist_mode() > 0) {
+  if (groups <= 1 && persist_mode() > 0 && !(reinterpret_cast<uintptr_t>(y) & 31u)) {   // its fp32 stores are 32 bytes wide
     const int th = tbvops::gemm_tok_choose(M, N, K, ldy, epi, persist_mode());
     if (th > 0) return tbvops::gemm_tok_launch_p(w, x, p, ldx, epi, th, stream);
   }

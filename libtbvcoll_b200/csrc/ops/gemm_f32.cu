@@ -38,6 +38,7 @@ __global__ void __launch_bounds__(256) k_gemm_f32(const F32Params p) {
       sw[k][r] = (m0 + r < p.M && k0 + k < p.K) ? w[size_t(m0 + r) * p.K + k0 + k] : 0.f;
     }
     __syncthreads();
+    float part[4][4] = {};      // one step's sum apart from the running total: the rounding error grows with K / 16, not with K
 #pragma unroll
     for (int k = 0; k < kKB; k++) {
       const float4 a = *reinterpret_cast<const float4*>(&sx[k][tn]), b = *reinterpret_cast<const float4*>(&sw[k][tm]);
@@ -45,8 +46,12 @@ __global__ void __launch_bounds__(256) k_gemm_f32(const F32Params p) {
 #pragma unroll
       for (int i = 0; i < 4; i++)
 #pragma unroll
-        for (int j = 0; j < 4; j++) acc[i][j] = fmaf(av[i], bv[j], acc[i][j]);
+        for (int j = 0; j < 4; j++) part[i][j] = fmaf(av[i], bv[j], part[i][j]);
     }
+#pragma unroll
+    for (int i = 0; i < 4; i++)
+#pragma unroll
+      for (int j = 0; j < 4; j++) acc[i][j] += part[i][j];
     __syncthreads();
   }
 #pragma unroll

@@ -78,6 +78,12 @@ __device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 
+// One 32-byte store: a whole sector per thread, where rows of different tokens sit in neighbouring threads.
+__device__ __forceinline__ void st_global_f32x8(float* p, const float* v) {
+  asm volatile("st.global.v8.f32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8};" ::"l"(p), "f"(v[0]), "f"(v[1]), "f"(v[2]), "f"(v[3]), "f"(v[4]), "f"(v[5]),
+               "f"(v[6]), "f"(v[7]) : "memory");
+}
+
 // One token row, 16 features starting at f: convert, apply the epilogue, store.
 template <int EPI>
 __device__ __forceinline__ void store16(const gemm::Params& p, int n, int f, const uint32_t* q) {
@@ -91,9 +97,9 @@ __device__ __forceinline__ void store16(const gemm::Params& p, int n, int f, con
   if (EPI == gemm::kEpiF32) {
 #pragma unroll
     for (int j = 0; j < 16; j++) v[j] = gemm::apply_act(v[j], p.act, p.act_a);
-    float4* dst = reinterpret_cast<float4*>(p.yf + size_t(n) * p.ldy + f);
-#pragma unroll
-    for (int j = 0; j < 4; j++) dst[j] = make_float4(v[4 * j], v[4 * j + 1], v[4 * j + 2], v[4 * j + 3]);
+    float* dst = p.yf + size_t(n) * p.ldy + f;      // 64-byte aligned rows: M and ldy are multiples of 16 and 8
+    st_global_f32x8(dst, v);
+    st_global_f32x8(dst + 8, v + 8);
     if (p.y2) {
       uint4* d2 = reinterpret_cast<uint4*>(p.y2 + size_t(n) * p.ldy + f);
       d2[0] = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));

@@ -100,10 +100,11 @@ struct RowsParams {
   const float* sink;        // [heads] or null
   void* out;                // [rows, heads, Rp]
   int heads, R, Rp, rotp, block_size, max_blocks, splits;
-  float scale_log2;
+  float scale_log2, scale;
 };
 
-// fp32: one CTA per (row, head), tiles of 128 keys
+// fp32: one CTA per (row, head), tiles of 128 keys.  Exponents are taken of differences of natural-unit scores: a score of
+// hundreds loses nothing to a multiplication by log2 e.
 __global__ void __launch_bounds__(128) k_latent_rows_f32(const RowsParams p) {
   extern __shared__ float sm[];
   __shared__ float red[4];
@@ -132,12 +133,12 @@ __global__ void __launch_bounds__(128) k_latent_rows_f32(const RowsParams p) {
       sl[tid] = slot;
       const float4* kr = reinterpret_cast<const float4*>(cache + size_t(slot) * Dk);
       const float4* q4 = reinterpret_cast<const float4*>(sq);
-      float a = 0.f;
+      float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
       for (int i = 0; i < Dk / 4; i++) {
         const float4 k = kr[i], q = q4[i];
-        a = fmaf(q.x, k.x, a); a = fmaf(q.y, k.y, a); a = fmaf(q.z, k.z, a); a = fmaf(q.w, k.w, a);
+        a.x = fmaf(q.x, k.x, a.x); a.y = fmaf(q.y, k.y, a.y); a.z = fmaf(q.z, k.z, a.z); a.w = fmaf(q.w, k.w, a.w);
       }
-      s = a * p.scale_log2;
+      s = ((a.x + a.y) + (a.z + a.w)) * p.scale;
     }
     float mx = s;
 #pragma unroll
@@ -145,7 +146,7 @@ __global__ void __launch_bounds__(128) k_latent_rows_f32(const RowsParams p) {
     if ((tid & 31) == 0) red[tid >> 5] = mx;
     __syncthreads();
     const float mn = fmaxf(m, fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3])));
-    const float pr = tid < n ? exp2f(s - mn) : 0.f, corr = exp2f(m - mn);
+    const float pr = tid < n ? expf(s - mn) : 0.f, corr = expf(m - mn);
     sp[tid] = pr;
     float ps = pr;
 #pragma unroll
@@ -159,17 +160,17 @@ __global__ void __launch_bounds__(128) k_latent_rows_f32(const RowsParams p) {
     for (int k = 0; k < kAcc; k++) {
       const int d = tid + k * 128;
       if (d < p.R) {
-        float acc = o[k] * corr;
+        float acc = 0.f;
         for (int t = 0; t < n; t++) acc = fmaf(sp[t], cache[size_t(sl[t]) * Dk + d], acc);
-        o[k] = acc;
+        o[k] = fmaf(o[k], corr, acc);
       }
     }
   }
   float c = 1.f;
   if (p.sink) {
-    const float sk = p.sink[h] * kLog2e, mf = fmaxf(m, sk);
-    c = exp2f(m - mf);
-    l = l * c + exp2f(sk - mf);
+    const float sk = p.sink[h], mf = fmaxf(m, sk);
+    c = expf(m - mf);
+    l = l * c + expf(sk - mf);
   }
   float* out = static_cast<float*>(p.out) + (size_t(row) * p.heads + h) * p.Rp;
 #pragma unroll
@@ -212,6 +213,13 @@ __device__ __forceinline__ float ld_cluster_f32(uint32_t addr, uint32_t rank) {
   asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(r) : "memory");
   return v;
 }
+__device__ __forceinline__ float4 ld_cluster_f32x4(uint32_t addr, uint32_t rank) {
+  uint32_t r;
+  float4 v;
+  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(addr), "r"(rank));
+  asm volatile("ld.shared::cluster.v4.f32 {%0,%1,%2,%3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(r) : "memory");
+  return v;
+}
 __device__ __forceinline__ void cluster_sync() {
   asm volatile("barrier.cluster.arrive.release.aligned;\nbarrier.cluster.wait.acquire.aligned;" ::: "memory");
 }
@@ -225,7 +233,7 @@ constexpr int kMaxSplits = 8;
 template <int CBW, int TT>
 __global__ void __launch_bounds__(kRW * 32, 1) k_latent_rows_mma(const RowsParams p) {
   extern __shared__ __align__(128) uint8_t dsm[];
-  __shared__ float sh_max[kRW][16], sh_l[kRW][16], sh_ml[16][2], sh_fac[kMaxSplits][16];
+  __shared__ float sh_max[kRW][16], sh_l[kRW][16], sh_ml[16][2], sh_fac[kMaxSplits][16], sh_sm[kMaxSplits][16];
   __shared__ __align__(16) uint8_t sh_p[16 * (TT * 2 + 16)];
   pdl::launch_dependents();
   pdl::grid_dependency_wait();
@@ -237,7 +245,7 @@ __global__ void __launch_bounds__(kRW * 32, 1) k_latent_rows_mma(const RowsParam
   const int ctx = min(p.ctx_lens[row], p.max_blocks * p.block_size);
   const int* bt = p.tables + size_t(p.seq_of_row ? p.seq_of_row[row] : row) * p.max_blocks;
   int chunk = (ctx + S - 1) / S;
-  chunk = (chunk + TT - 1) / TT * TT;
+  chunk = (chunk + 15) / 16 * 16;
   const int t0 = min(ctx, sp * chunk), t1 = min(ctx, t0 + chunk);
   const int ntiles = (t1 - t0 + TT - 1) / TT;
 
@@ -251,10 +259,15 @@ __global__ void __launch_bounds__(kRW * 32, 1) k_latent_rows_mma(const RowsParam
   auto issue = [&](int i) {
     if (i < ntiles) {
       const uint32_t dst = sk0 + (i & 1) * stage;
-      for (int r = warp; r < TT; r += kRW) {
-        const int tok = t0 + i * TT + r;
+      // the warp's TT / kRW table entries with one load, handed out by shuffles
+      const int mt = t0 + i * TT + warp + (lane & (TT / kRW - 1)) * kRW;
+      const int mine = mt < t1 ? bt[mt / p.block_size] * p.block_size + mt % p.block_size : 0;
+#pragma unroll
+      for (int k = 0; k < TT / kRW; k++) {
+        const int r = warp + k * kRW;
+        const int tok = t0 + i * TT + r, slot = __shfl_sync(0xffffffffu, mine, k);
         if (tok < t1) {
-          const __nv_bfloat16* src = cache + (size_t(bt[tok / p.block_size]) * p.block_size + tok % p.block_size) * Dk;
+          const __nv_bfloat16* src = cache + size_t(slot) * Dk;
           for (int c = lane; c < chunks; c += 32) cp_async16(dst + r * pitch + c * 16, src + c * 8);
         } else {
           for (int c = lane; c < chunks; c += 32) st_zero16(dst + r * pitch + c * 16);
@@ -373,36 +386,50 @@ __global__ void __launch_bounds__(kRW * 32, 1) k_latent_rows_mma(const RowsParam
   }
   if (S > 1) cluster_sync();
   else __syncthreads();
-  // factor of every split's partial sum, the sink and the division included
-  if (tid < 16) {
-    const float sk = p.sink && h0 + tid < p.heads ? p.sink[h0 + tid] * kLog2e : kNegBig;
-    const uint32_t a = smem_addr(&sh_ml[tid][0]);
-    float ms[kMaxSplits], mx = sk, l = 0.f;
-    for (int r = 0; r < S; r++) { ms[r] = S > 1 ? ld_cluster_f32(a, r) : sh_ml[tid][0]; mx = fmaxf(mx, ms[r]); }
-    for (int r = 0; r < S; r++) l = fmaf(S > 1 ? ld_cluster_f32(a + 4, r) : sh_ml[tid][1], exp2f(ms[r] - mx), l);
-    if (p.sink) l += exp2f(sk - mx);
-    for (int r = 0; r < S; r++) sh_fac[r][tid] = l > 0.f ? exp2f(ms[r] - mx) / l : 0.f;
+  // factor of every split's partial sum, the sink and the division included; all remote values are requested before one is used
+  if (tid < 16 * kMaxSplits) {
+    const int r = tid >> 4, h = tid & 15;
+    float m = kNegBig, l = 0.f;
+    if (r < S) {
+      const uint32_t a = smem_addr(&sh_ml[h][0]);
+      m = S > 1 ? ld_cluster_f32(a, r) : sh_ml[h][0];
+      l = S > 1 ? ld_cluster_f32(a + 4, r) : sh_ml[h][1];
+    }
+    sh_sm[r][h] = m;
+    sh_fac[r][h] = l;
   }
   __syncthreads();
-  const int nh = min(16, p.heads - h0), total = nh * p.Rp / 2, per = (total + S - 1) / S;
+  if (tid < 16) {
+    const float sk = p.sink && h0 + tid < p.heads ? p.sink[h0 + tid] * kLog2e : kNegBig;
+    float mx = sk, l = 0.f;
+    for (int r = 0; r < S; r++) mx = fmaxf(mx, sh_sm[r][tid]);
+    for (int r = 0; r < S; r++) l = fmaf(sh_fac[r][tid], exp2f(sh_sm[r][tid] - mx), l);
+    if (p.sink) l += exp2f(sk - mx);
+    for (int r = 0; r < S; r++) sh_fac[r][tid] = l > 0.f ? exp2f(sh_sm[r][tid] - mx) / l : 0.f;
+  }
+  __syncthreads();
+  const int nh = min(16, p.heads - h0), total = nh * p.Rp / 4, per = (total + S - 1) / S;
   __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + (size_t(row) * p.heads + h0) * p.Rp;
   const uint32_t soa = smem_addr(so);
   for (int i = tid; i < per; i += kRW * 32) {
     const int idx = sp * per + i;
     if (idx < total) {
-      const int h = idx * 2 / p.Rp;
-      float x = 0.f, y = 0.f;
-      for (int r = 0; r < S; r++) {
-        const float f = sh_fac[r][h];
-        if (S > 1) {
-          x = fmaf(ld_cluster_f32(soa + idx * 8, r), f, x);
-          y = fmaf(ld_cluster_f32(soa + idx * 8 + 4, r), f, y);
-        } else {
-          x = so[idx * 2] * f;
-          y = so[idx * 2 + 1] * f;
-        }
+      const int h = idx * 4 / p.Rp;
+      float4 v[kMaxSplits], a = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (S > 1) {
+#pragma unroll
+        for (int r = 0; r < kMaxSplits; r++)
+          if (r < S) v[r] = ld_cluster_f32x4(soa + idx * 16, r);
+      } else {
+        v[0] = *reinterpret_cast<const float4*>(so + idx * 4);
       }
-      *reinterpret_cast<uint32_t*>(out + idx * 2) = pack_bf16(x, y);
+#pragma unroll
+      for (int r = 0; r < kMaxSplits; r++)
+        if (r < S) {
+          const float f = sh_fac[r][h];
+          a.x = fmaf(v[r].x, f, a.x); a.y = fmaf(v[r].y, f, a.y); a.z = fmaf(v[r].z, f, a.z); a.w = fmaf(v[r].w, f, a.w);
+        }
+      *reinterpret_cast<uint2*>(out + idx * 4) = make_uint2(pack_bf16(a.x, a.y), pack_bf16(a.z, a.w));
     }
   }
   if (S > 1) cluster_sync();   // nobody leaves while a peer may still read its shared memory
@@ -593,8 +620,11 @@ constexpr size_t kMaxSmem = 226 * 1024;
 
 template <typename K>
 cudaError_t allow_smem(K kern, size_t bytes, bool* done) {
-  if (*done || bytes <= 48 * 1024) return cudaSuccess;
-  cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(kMaxSmem));
+  if (*done || bytes <= 32 * 1024) return cudaSuccess;   // up to 48 KB with the static part needs no opt-in
+  cudaFuncAttributes a;
+  cudaError_t e = cudaFuncGetAttributes(&a, kern);
+  if (e != cudaSuccess) return e;
+  e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(227 * 1024 - a.sharedSizeBytes));   // static + dynamic: 227 KB
   if (e == cudaSuccess) *done = true;
   return e;
 }
@@ -637,7 +667,7 @@ int tbv_op_latent_attn_rows(const void* qa, const void* cache, const void* table
   if (rows <= 0) return 0;
   if (heads <= 0 || R > Rp || (Rp % 16) || (rotp % 16) || block_size <= 0) return -2;
   RowsParams p{qa, cache, static_cast<const int*>(tables), static_cast<const int*>(seq_of_row), static_cast<const int*>(ctx_lens),
-               static_cast<const float*>(sink), out, heads, R, Rp, rotp, block_size, max_blocks, 1, scale * kLog2e};
+               static_cast<const float*>(sink), out, heads, R, Rp, rotp, block_size, max_blocks, 1, scale * kLog2e, scale};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   cudaError_t e;
   if (!bf16) {

@@ -4,8 +4,8 @@ several residual streams with hyper-connections, layers that run more than once,
 Per sublayer the residual streams (fp32) are read and written by ONE kernel (``ops.hyper_mix``: layer scale, stream mixing, next
 norm).  Between two of them:
 
-    mamba   in-projection GEMM -> convolution + SiLU -> x-projection GEMM (fp32 + bf16 copy) -> step-size GEMM with softplus
-            epilogue -> selective scan with the gate and the state update -> out-projection GEMM (fp32)
+    mamba   in-projection GEMM -> convolution + SiLU -> x-projection GEMM (fp32 + bf16 copy) -> step-size GEMM (fp32)
+            -> selective scan with the softplus before and the gate after it, replacing the carried state -> out-projection GEMM (fp32)
     latent  query + latent GEMM -> rotation, latent norm and cache write -> attention -> out-projection GEMM (fp32); attention is
             fold W_uk into the query (grouped GEMM) -> rows kernel over the cache -> expand with W_uv (grouped GEMM)    few rows
             or gather -> expand keys and values (GEMM) -> tiled kernel                                                  many rows
@@ -126,9 +126,9 @@ class Nubosun:
         else:
             low = proj
             ops.linear(u, w[p + "x"], proj)
-        ops.linear(low[:, :kd], w[p + "dt"], dt, bias=w[p + "dt.b"], act=ops.ACT_SOFTPLUS)
+        ops.linear(low[:, :kd], w[p + "dt"], dt, bias=w[p + "dt.b"])
         ops.selective_scan(u, xz, ip, dt, proj, m.dt_rank, m.dt_rank + m.state, w[p + "a2"], w[p + "D"], self.ssm[run], self.conv[run], u, b.segs,
-                           b.positions)
+                           b.positions, one_token=b.seg_of_row is None)
         ops.linear(u, w[p + "o"], y)
 
     def _latent(self, b: StepBatch, run: int, i: int, m: LatentSpec, h, y) -> None:

@@ -39,7 +39,7 @@ def lib():
     l.tbv_op_hyper_embed.argtypes = [c_vp, c_vp, LL, F, c_vp, c_vp, c_vp, c_vp, I, I, I, I, I, F, I, c_vp]
     l.tbv_op_hyper_mix.argtypes = [c_vp, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp, I, I, I, I, I, I, F, I, c_vp]
     l.tbv_op_causal_conv_silu.argtypes = [c_vp] * 8 + [I] * 6 + [c_vp]
-    l.tbv_op_selective_scan.argtypes = [c_vp] * 11 + [I] * 14 + [c_vp]
+    l.tbv_op_selective_scan.argtypes = [c_vp] * 11 + [I] * 15 + [c_vp]
     l.tbv_op_latent_prep.argtypes = [c_vp] * 7 + [I] * 11 + [F, F, I, c_vp]
     l.tbv_op_latent_attn_rows.argtypes = [c_vp] * 7 + [I] * 8 + [F, I, c_vp]
     l.tbv_op_latent_gather.argtypes = [c_vp] * 4 + [I] * 3 + [c_vp]

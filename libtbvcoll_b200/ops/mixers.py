@@ -48,16 +48,18 @@ def causal_conv_silu(x, out, taps, bias, conv_state, segs, seg_of_row, positions
     _count()
 
 
-def selective_scan(u, xz, z_off: int, dt, bc, b_off: int, c_off: int, a_log2e, d, ssm, conv_state, out, segs, positions) -> None:
-    """Per channel c and state n: S <- exp2(dt a_log2e) S + dt u B; y = sum_n S C + d u; out = y * silu(z), z at columns z_off.. of xz.
+def selective_scan(u, xz, z_off: int, dt, bc, b_off: int, c_off: int, a_log2e, d, ssm, conv_state, out, segs, positions,
+                   one_token: bool = False) -> None:
+    """Per channel c and state n, dt = softplus of the given values: S <- exp2(dt a_log2e) S + dt u B; y = sum_n S C + d u; out = y * silu(z), z at columns z_off.. of xz.
     a_log2e fp32 [inner, N] (= -exp(A_log) * log2 e); ssm fp32 [slots, inner, N] and conv_state (the convolution's last inputs, from
-    the first columns of xz) are replaced.  ``out`` may be ``u``."""
+    the first columns of xz) are replaced.  ``out`` may be ``u``.
+    ``one_token``: every segment has one row (a decode step)."""
     inner, N = a_log2e.shape
     assert ssm.shape[1:] == (inner, N) and ssm.dtype is torch.float32 and dt.dtype is torch.float32 and bc.dtype is torch.float32
     assert u.dtype is xz.dtype is out.dtype and segs.dtype is torch.int32
     _chk(lib().tbv_op_selective_scan(_p(u), _p(xz), _p(dt), _p(bc), _p(a_log2e), _p(d), _p(ssm), _p(conv_state), _p(out), _p(segs), _p(positions),
                                      segs.shape[0], inner, N, u.stride(0), xz.stride(0), z_off, dt.stride(0), bc.stride(0), b_off, c_off,
-                                     out.stride(0), conv_state.shape[2], conv_state.shape[1] + 1, _is_bf16(u), _st()), "tbv_op_selective_scan")
+                                     out.stride(0), conv_state.shape[2], conv_state.shape[1] + 1, int(one_token), _is_bf16(u), _st()), "tbv_op_selective_scan")
     _count()
 
 
