@@ -199,7 +199,7 @@ def kernel_numbers(size: str, T: int, seqs: int, ctx: int) -> list:
     nr = T if decode else 0
 
     def mk_prep(i):
-        qkv, qa, cache = _w(T, qc), torch.empty(max(nr, 1), H, Dk, dtype=bf, device=dev), _w(nslots, Dk)
+        qkv, qa, cache = _w(T, qc), torch.empty(max(nr, 1), H, Dk + 8, dtype=bf, device=dev), _w(nslots, Dk + 8)
         gm = torch.ones(R, device=dev)
         return lambda: ops.latent_prep(qkv, qa[:nr], cache, gm, freq, 1.0, pos, slots, nr, H * a.dim, H * (a.dim + rot), H * (a.dim + rot) + R, H, R, R, rot, 1e-5)
     k.time("attention", "nubosun rotation + latent norm + cache write", mk_prep, T * (2 * H * rot + 2 * Dk) * 2)
@@ -213,8 +213,8 @@ def kernel_numbers(size: str, T: int, seqs: int, ctx: int) -> list:
         return s
     if decode:
         def mk_rows(i):
-            qa, cache, o = _w(T, H, Dk), _w(nslots, Dk), torch.empty(T, H, R, dtype=bf, device=dev)
-            sp = splits((H + 15) // 16, 1)
+            qa, cache, o = _w(T, H, Dk + 8), _w(nslots, Dk + 8), torch.empty(T, H, R, dtype=bf, device=dev)
+            sp = splits((H + 15) // 16, 0.8)
             return lambda: ops.latent_attention_rows(qa, cache, tables, seq_of_row, ctx_lens, sink, o, R, a.scale, bs, splits=sp)
         k.time("attention", "nubosun latent attention, rows form", mk_rows, seqs * ctx * Dk * 2 + T * H * (Dk + R) * 2, 2.0 * pairs_causal * H * (Dk + R))
 
@@ -229,7 +229,7 @@ def kernel_numbers(size: str, T: int, seqs: int, ctx: int) -> list:
         tl, sl = torch.from_numpy(tl).to(dev), torch.from_numpy(sl).to(dev)
 
         def mk_gather(i):
-            cache, c, kr = _w(nslots, Dk), torch.empty(T, R, dtype=bf, device=dev), torch.empty(T, rot, dtype=bf, device=dev)
+            cache, c, kr = _w(nslots, Dk + 8), torch.empty(T, R, dtype=bf, device=dev), torch.empty(T, rot, dtype=bf, device=dev)
             return lambda: ops.latent_gather(cache, sl, c, kr)
         k.time("attention", "nubosun gather of the latents", mk_gather, 2 * T * Dk * 2)
 

@@ -346,7 +346,9 @@ void gemm_config(int M, int N, int K, int splits_hint, int* bn_out, int* splits_
   } else {
     // a K range per CTA of at least `min_kb` 64-wide blocks (TBV_GEMM_MIN_KB, read once)
     static const int min_kb = [] { const char* e = getenv("TBV_GEMM_MIN_KB"); int v = e ? atoi(e) : 8; return v < 1 ? 1 : v; }();
-    while (splits < 8 && tiles * splits * 2 <= 2 * sms && kb / (splits * 2) >= min_kb) splits *= 2;
+    // fp32 staging of a 256-token tile (128 KB) leaves room for one CTA per SM
+    const int slots = f32_out && bn == 256 ? sms : 2 * sms;
+    while (splits < 8 && tiles * splits * 2 <= slots && kb / (splits * 2) >= min_kb) splits *= 2;
   }
   while (splits > 1 && (kb + splits - 1) / splits * (splits - 1) >= kb) splits /= 2;  // every split gets work
   const int stage_bytes = gemm::kATileBytes + bn * 128;

@@ -1,7 +1,8 @@
 // latent_attn.cu — attention over a compressed (latent) paged cache, with a learned sink per head.
 //
 // A cached token is one row of Dk = Rp + rotp values shared by all heads: the normalised latent c (R values, padded to Rp)
-// and one rotated key part (padded to rotp).  Head h scores it as (q_h . W_uk,h c + q_rot,h . k_rot) * scale and its
+// and one rotated key part (padded to rotp).  Rows of the cache (and of the folded queries) lie kRowPad values apart: the tokens of
+// a block come into shared memory as ONE bulk copy and already have the odd 16-byte pitch that ldmatrix wants.  Head h scores it as (q_h . W_uk,h c + q_rot,h . k_rot) * scale and its
 // value is W_uv,h c.  Two forms of the same sum:
 //   rows form     W_uk is folded into the query (qa_h = W_uk,h^T q_h), the cache rows serve as keys AND as values, and the
 //                 result is a latent per head that W_uv expands afterwards.  The cache is read once for all heads: the
@@ -15,12 +16,15 @@
 #include <stdio.h>
 
 #include "../pdl.cuh"
+#include "ops.h"
+#include "sm100.cuh"
 
 namespace {
 
 constexpr float kNegBig = -1e30f;
 constexpr float kLog2e = 1.4426950408889634f;
 constexpr int kMaxPairs = 512;
+constexpr int kRowPad = 8;
 
 __device__ __forceinline__ float to_f(float v) { return v; }
 __device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
@@ -30,8 +34,8 @@ __device__ __forceinline__ void from_f(__nv_bfloat16& d, float v) { d = __float2
 // ---- rotation, latent norm, cache write ------------------------------------------------------------------------------
 struct PrepParams {
   void* qkv;                // [rows, ldq]: head parts (q_off: rotated parts of all heads), latent (c_off), key part (k_off)
-  void* qa;                 // [n_rows_form, heads, Dk]: rotated query parts of the first n_rows_form rows go to column Rp
-  void* cache;              // [slots, Dk]
+  void* qa;                 // [n_rows_form, heads, Dk + kRowPad]: rotated query parts of the first n_rows_form rows go to column Rp
+  void* cache;              // [slots, Dk + kRowPad]
   const float* gamma;       // [R]
   const float* inv_freq;    // [pairs]
   const int* positions;
@@ -68,7 +72,7 @@ __global__ void __launch_bounds__(256) k_latent_prep(const PrepParams p) {
   const int Dk = p.Rp + p.rotp, half = p.rotp / 2;
   const long long slot = p.slots[row];
   if (slot >= 0) {
-    T* kc = static_cast<T*>(p.cache) + size_t(slot) * Dk;
+    T* kc = static_cast<T*>(p.cache) + size_t(slot) * (Dk + kRowPad);
     for (int i = tid; i < p.Rp; i += 256) from_f(kc[i], i < p.R ? to_f(cv[i]) * r * p.gamma[i] : 0.f);
     const T* kr = q + p.k_off;
     for (int i = tid; i < half; i += 256) {
@@ -84,7 +88,7 @@ __global__ void __launch_bounds__(256) k_latent_prep(const PrepParams p) {
     const int h = j / half, i = j - h * half;
     const float a = to_f(qr[h * p.rotp + 2 * i]), b = to_f(qr[h * p.rotp + 2 * i + 1]);
     const bool rot = i < p.pairs;
-    T* dst = rows_form ? static_cast<T*>(p.qa) + (size_t(row) * p.heads + h) * Dk + p.Rp + 2 * i : qr + h * p.rotp + 2 * i;
+    T* dst = rows_form ? static_cast<T*>(p.qa) + (size_t(row) * p.heads + h) * (Dk + kRowPad) + p.Rp + 2 * i : qr + h * p.rotp + 2 * i;
     from_f(dst[0], rot ? a * cs[i] - b * sn[i] : a);
     from_f(dst[1], rot ? b * cs[i] + a * sn[i] : b);
   }
@@ -92,8 +96,8 @@ __global__ void __launch_bounds__(256) k_latent_prep(const PrepParams p) {
 
 // ---- rows form ---------------------------------------------------------------------------------------------------------
 struct RowsParams {
-  const void* qa;           // [rows, heads, Dk]
-  const void* cache;        // [slots, Dk]
+  const void* qa;           // [rows, heads, Dk + kRowPad]
+  const void* cache;        // [slots, Dk + kRowPad]
   const int* tables;        // [nseq, max_blocks]
   const int* seq_of_row;    // [rows] or null
   const int* ctx_lens;      // [rows]
@@ -101,6 +105,7 @@ struct RowsParams {
   void* out;                // [rows, heads, Rp]
   int heads, R, Rp, rotp, block_size, max_blocks, splits;
   float scale_log2, scale;
+  int* err;                 // device flag: set to 1 if a wait for copies gave up
 };
 
 // fp32: one CTA per (row, head), tiles of 128 keys.  Exponents are taken of differences of natural-unit scores: a score of
@@ -114,7 +119,7 @@ __global__ void __launch_bounds__(128) k_latent_rows_f32(const RowsParams p) {
   float* sq = sm;            // [Dk]
   float* sp = sm + Dk;       // [128]
   int* sl = reinterpret_cast<int*>(sp + 128);
-  const float* qa = static_cast<const float*>(p.qa) + (size_t(row) * p.heads + h) * Dk;
+  const float* qa = static_cast<const float*>(p.qa) + (size_t(row) * p.heads + h) * (Dk + kRowPad);
   for (int i = tid; i < Dk; i += 128) sq[i] = qa[i];
   const float* cache = static_cast<const float*>(p.cache);
   const int ctx = min(p.ctx_lens[row], p.max_blocks * p.block_size);
@@ -131,7 +136,7 @@ __global__ void __launch_bounds__(128) k_latent_rows_f32(const RowsParams p) {
     if (tid < n) {
       const int tok = t0 + tid, slot = bt[tok / p.block_size] * p.block_size + tok % p.block_size;
       sl[tid] = slot;
-      const float4* kr = reinterpret_cast<const float4*>(cache + size_t(slot) * Dk);
+      const float4* kr = reinterpret_cast<const float4*>(cache + size_t(slot) * (Dk + kRowPad));
       const float4* q4 = reinterpret_cast<const float4*>(sq);
       float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
       for (int i = 0; i < Dk / 4; i++) {
@@ -161,7 +166,7 @@ __global__ void __launch_bounds__(128) k_latent_rows_f32(const RowsParams p) {
       const int d = tid + k * 128;
       if (d < p.R) {
         float acc = 0.f;
-        for (int t = 0; t < n; t++) acc = fmaf(sp[t], cache[size_t(sl[t]) * Dk + d], acc);
+        for (int t = 0; t < n; t++) acc = fmaf(sp[t], cache[size_t(sl[t]) * (Dk + kRowPad) + d], acc);
         o[k] = fmaf(o[k], corr, acc);
       }
     }
@@ -224,22 +229,30 @@ __device__ __forceinline__ void cluster_sync() {
   asm volatile("barrier.cluster.arrive.release.aligned;\nbarrier.cluster.wait.acquire.aligned;" ::: "memory");
 }
 
-// bf16: 16 heads of one row per CTA on tensor cores.  Eight warps share tiles of TT cached tokens (two cp.async stages, row
-// pitch Dk * 2 + 16 bytes so that ldmatrix is conflict-free): for the scores warp w takes tokens 8w.. of the tile over all Dk
+// bf16: 16 heads of one row per CTA on tensor cores.  Eight warps share tiles of TT cached tokens (two stages filled by bulk copies): for the scores warp w takes tokens 8w.. of the tile over all Dk
 // columns; for the weighted sum it takes the latent columns of the 16-column blocks w, w + 8, .. (CBW of them).  grid (rows, head tiles,
 // splits), cluster (1, 1, splits): the CTAs of a cluster cover disjoint token ranges and merge in split order.
 constexpr int kRW = 8;
 constexpr int kMaxSplits = 8;
 template <int CBW, int TT>
-__global__ void __launch_bounds__(kRW * 32, 1) k_latent_rows_mma(const RowsParams p) {
+__global__ void __launch_bounds__(kRW * 32 + 32, 1) k_latent_rows_mma(const RowsParams p) {
   extern __shared__ __align__(128) uint8_t dsm[];
   __shared__ float sh_max[kRW][16], sh_l[kRW][16], sh_ml[16][2], sh_fac[kMaxSplits][16], sh_sm[kMaxSplits][16];
   __shared__ __align__(16) uint8_t sh_p[16 * (TT * 2 + 16)];
+  __shared__ unsigned long long full[2];
+  __shared__ int abort_flag;
   pdl::launch_dependents();
+  if (threadIdx.x == 0) {
+    sm100::mbar_init(smem_addr(&full[0]), 1);
+    sm100::mbar_init(smem_addr(&full[1]), 1);
+    abort_flag = 0;
+    sm100::mbar_fence_init();
+  }
+  __syncthreads();
   pdl::grid_dependency_wait();
   const int row = blockIdx.x, h0 = blockIdx.y * 16, sp = blockIdx.z, S = p.splits;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r8 = lane >> 2, quad = lane & 3;
-  const int Dk = p.Rp + p.rotp, chunks = Dk / 8, pitch = Dk * 2 + 16, ksteps = Dk / 16, cblocks = p.Rp / 16;
+  const int Dk = p.Rp + p.rotp, chunks = Dk / 8, pitch = (Dk + kRowPad) * 2, ksteps = Dk / 16, cblocks = p.Rp / 16;
   const uint32_t sq = smem_addr(dsm), sk0 = sq + 16 * pitch, stage = uint32_t(TT) * pitch, spb = smem_addr(sh_p);
   constexpr int kPP = TT * 2 + 16;
   const int ctx = min(p.ctx_lens[row], p.max_blocks * p.block_size);
@@ -249,66 +262,101 @@ __global__ void __launch_bounds__(kRW * 32, 1) k_latent_rows_mma(const RowsParam
   const int t0 = min(ctx, sp * chunk), t1 = min(ctx, t0 + chunk);
   const int ntiles = (t1 - t0 + TT - 1) / TT;
 
-  const __nv_bfloat16* qa = static_cast<const __nv_bfloat16*>(p.qa) + (size_t(row) * p.heads + h0) * Dk;
-  for (int r = warp; r < 16; r += kRW)
-    for (int c = lane; c < chunks; c += 32) {
-      if (h0 + r < p.heads) cp_async16(sq + r * pitch + c * 16, qa + size_t(r) * Dk + c * 8);
-      else st_zero16(sq + r * pitch + c * 16);
-    }
+  const __nv_bfloat16* qa = static_cast<const __nv_bfloat16*>(p.qa) + (size_t(row) * p.heads + h0) * (Dk + kRowPad);
   const __nv_bfloat16* cache = static_cast<const __nv_bfloat16*>(p.cache);
-  auto issue = [&](int i) {
-    if (i < ntiles) {
-      const uint32_t dst = sk0 + (i & 1) * stage;
-      // the warp's TT / kRW table entries with one load, handed out by shuffles
-      const int mt = t0 + i * TT + warp + (lane & (TT / kRW - 1)) * kRW;
-      const int mine = mt < t1 ? bt[mt / p.block_size] * p.block_size + mt % p.block_size : 0;
-#pragma unroll
-      for (int k = 0; k < TT / kRW; k++) {
-        const int r = warp + k * kRW;
-        const int tok = t0 + i * TT + r, slot = __shfl_sync(0xffffffffu, mine, k);
-        if (tok < t1) {
-          const __nv_bfloat16* src = cache + size_t(slot) * Dk;
-          for (int c = lane; c < chunks; c += 32) cp_async16(dst + r * pitch + c * 16, src + c * 8);
-        } else {
-          for (int c = lane; c < chunks; c += 32) st_zero16(dst + r * pitch + c * 16);
-        }
-      }
-    }
-    cp_async_commit();
+  const int nq = min(16, p.heads - h0);
+  for (int r = nq + warp; r < 16; r += kRW + 1)
+    for (int c = lane; c < chunks; c += 32) st_zero16(sq + r * pitch + c * 16);
+  // The ninth warp brings the tiles in.  Tile i: it asks for the tokens, a block (or the part of one inside the tile) per copy, and for the query rows with tile 0.  A
+  // partial tile ends at a multiple of 16 tokens, its missing rows are zeros, so that a weight of zero meets no stale bit pattern.  Table entries are looked up a
+  // tile ahead of their use: table and cache are two memory round trips, and both would otherwise stand between two tiles.
+  const int bs = p.block_size;
+  auto look_up = [&](int i) {
+    const int pg = (t0 + i * TT) / bs + lane;
+    return pg * bs < t1 ? bt[pg] : 0;
   };
+  auto issue = [&](int i, int block) {
+    if (i >= ntiles) return;
+    const uint32_t dst = sk0 + (i & 1) * stage, bar = smem_addr(&full[i & 1]);
+    const int tok0 = t0 + i * TT, n = min(TT, t1 - tok0), pg0 = tok0 / bs;
+    if (lane == 0) {
+      sm100::mbar_expect_tx(bar, uint32_t(n + (i == 0 ? nq : 0)) * uint32_t(pitch));
+      if (i == 0) sm100::bulk_load(sq, qa, uint32_t(nq) * pitch, bar);
+    }
+    __syncwarp();
+    for (int pg = pg0 + lane; pg * bs < tok0 + n; pg += 32) {
+      if (pg >= pg0 + 32) block = bt[pg];      // blocks of one or two tokens only
+      const int a = max(tok0, pg * bs), e = min(tok0 + n, (pg + 1) * bs);
+      sm100::bulk_load(dst + (a - tok0) * pitch, cache + (size_t(block) * bs + (a - pg * bs)) * (Dk + kRowPad), uint32_t(e - a) * pitch, bar);
+    }
+    for (int r = n; r < ((n + 15) & ~15); r++)
+      for (int c = lane; c < chunks; c += 32) st_zero16(dst + r * pitch + c * 16);
+  };
+  const bool producer = warp == kRW;
   float o[CBW][2][4];
 #pragma unroll
   for (int b = 0; b < CBW; b++)
 #pragma unroll
     for (int n = 0; n < 2; n++) o[b][n][0] = o[b][n][1] = o[b][n][2] = o[b][n][3] = 0.f;
   float m_lo = kNegBig, m_hi = kNegBig, l_lo = 0.f, l_hi = 0.f;
-  issue(0);
+  int block = 0;
+  if (producer) {
+    const int block0 = look_up(0), block1 = look_up(1);
+    block = look_up(2);
+    issue(0, block0);
+    issue(1, block1);
+  }
+  __syncthreads();                               // rows of zeros are in place
   for (int i = 0; i < ntiles; i++) {
-    issue(i + 1);
-    cp_async_wait<1>();
-    __syncthreads();
+    if (producer) {                              // keeps step with the barriers below, then refills the stage they released
+      __syncthreads();
+      __syncthreads();
+      __syncthreads();
+      issue(i + 2, block);
+      block = look_up(i + 3);
+      continue;
+    }
+    // zeros for a tile are stored two iterations, hence barriers, before it is read
+    sm100::mbar_wait(smem_addr(&full[i & 1]), uint32_t(i >> 1) & 1u, &abort_flag, 2000000000ull);
+    __syncwarp();
     const uint32_t sk = sk0 + (i & 1) * stage;
     float sc[4] = {0.f, 0.f, 0.f, 0.f}, sd[4] = {0.f, 0.f, 0.f, 0.f};
-    const bool has_s = warp * 8 < TT;
+    const int n16 = (min(TT, t1 - t0 - i * TT) + 15) & ~15;
+    const bool has_s = warp * 8 < n16;
     if (has_s) {
-      // two accumulators: consecutive k steps do not wait for one another
+      // operands of the next two k steps are requested before the products of these two; four accumulators in turn
       const uint32_t qaddr = sq + (lane & 15) * pitch + (lane >> 4) * 16;
       const uint32_t kaddr = sk + (warp * 8 + (lane & 7)) * pitch + (lane >> 3) * 16;
-      int ks = 0;
-      for (; ks + 1 < ksteps; ks += 2) {
-        uint32_t a0[4], a1[4], b[4];
-        ldmatrix_x4(qaddr + ks * 32, a0);
-        ldmatrix_x4(qaddr + ks * 32 + 32, a1);
-        ldmatrix_x4(kaddr + ks * 32, b);
-        mma_bf16(sc, a0, b[0], b[1]);
-        mma_bf16(sd, a1, b[2], b[3]);
+      float se[4] = {0.f, 0.f, 0.f, 0.f}, sf[4] = {0.f, 0.f, 0.f, 0.f};
+      uint32_t a[2][2][4], b[2][4];
+      auto load = [&](int ks, int w) {
+        ldmatrix_x4(kaddr + ks * 32, b[w]);
+        ldmatrix_x4(qaddr + ks * 32, a[w][0]);
+        ldmatrix_x4(qaddr + ks * 32 + 32, a[w][1]);
+      };
+      const int pairs = ksteps / 2;
+      load(0, 0);
+      int k2 = 0;
+      for (; k2 + 1 < pairs; k2 += 2) {
+        load(2 * k2 + 2, 1);
+        mma_bf16(sc, a[0][0], b[0][0], b[0][1]);
+        mma_bf16(sd, a[0][1], b[0][2], b[0][3]);
+        if (k2 + 2 < pairs) load(2 * k2 + 4, 0);
+        mma_bf16(se, a[1][0], b[1][0], b[1][1]);
+        mma_bf16(sf, a[1][1], b[1][2], b[1][3]);
       }
-      if (ks < ksteps) {
-        uint32_t a0[4], b[2];
-        ldmatrix_x4(qaddr + ks * 32, a0);
-        ldmatrix_x2(sk + (warp * 8 + (lane & 7)) * pitch + ((lane >> 3) & 1) * 16 + ks * 32, b);
-        mma_bf16(sc, a0, b[0], b[1]);
+      if (k2 < pairs) {
+        mma_bf16(sc, a[0][0], b[0][0], b[0][1]);
+        mma_bf16(sd, a[0][1], b[0][2], b[0][3]);
       }
+      if (ksteps & 1) {
+        const int ks = ksteps - 1;
+        ldmatrix_x4(qaddr + ks * 32, a[0][0]);
+        ldmatrix_x2(sk + (warp * 8 + (lane & 7)) * pitch + ((lane >> 3) & 1) * 16 + ks * 32, b[0]);
+        mma_bf16(se, a[0][0], b[0][0], b[0][1]);
+      }
+#pragma unroll
+      for (int j = 0; j < 4; j++) sc[j] += se[j], sd[j] += sf[j];
       const int tok = t0 + i * TT + warp * 8 + quad * 2;
 #pragma unroll
       for (int j = 0; j < 4; j++) sc[j] = tok + (j & 1) < t1 ? (sc[j] + sd[j]) * p.scale_log2 : kNegBig;
@@ -318,6 +366,8 @@ __global__ void __launch_bounds__(kRW * 32, 1) k_latent_rows_mma(const RowsParam
       x_hi = fmaxf(x_hi, __shfl_xor_sync(0xffffffffu, x_hi, 1));
       x_hi = fmaxf(x_hi, __shfl_xor_sync(0xffffffffu, x_hi, 2));
       if (quad == 0) { sh_max[warp][r8] = x_lo; sh_max[warp][r8 + 8] = x_hi; }
+    } else if (quad == 0) {
+      sh_max[warp][r8] = sh_max[warp][r8 + 8] = kNegBig;
     }
     __syncthreads();
     float n_lo = m_lo, n_hi = m_hi;
@@ -340,36 +390,46 @@ __global__ void __launch_bounds__(kRW * 32, 1) k_latent_rows_mma(const RowsParam
     for (int b = 0; b < CBW; b++)
 #pragma unroll
       for (int n = 0; n < 2; n++) { o[b][n][0] *= c_lo; o[b][n][1] *= c_lo; o[b][n][2] *= c_hi; o[b][n][3] *= c_hi; }
+    uint32_t pa[2][4], v[2][CBW][4];
+    auto load_v = [&](int ks, int w) {
+      ldmatrix_x4(spb + (lane & 15) * kPP + (lane >> 4) * 16 + ks * 32, pa[w]);
+#pragma unroll
+      for (int b = 0; b < CBW; b++)
+        if (warp + b * kRW < cblocks)
+          ldmatrix_x4_trans(sk + (ks * 16 + (lane & 15)) * pitch + (warp + b * kRW) * 32 + (lane >> 4) * 16, v[w][b]);
+    };
+    load_v(0, 0);
 #pragma unroll
     for (int ks = 0; ks < TT / 16; ks++) {
-      uint32_t a[4];
-      ldmatrix_x4(spb + (lane & 15) * kPP + (lane >> 4) * 16 + ks * 32, a);
+      if (ks * 16 >= n16) break;
+      if (ks + 1 < TT / 16 && ks * 16 + 16 < n16) load_v(ks + 1, (ks + 1) & 1);
 #pragma unroll
-      for (int b = 0; b < CBW; b++) {
-        const int cb = warp + b * kRW;
-        if (cb < cblocks) {
-          uint32_t v[4];
-          ldmatrix_x4_trans(sk + (ks * 16 + (lane & 15)) * pitch + cb * 32 + (lane >> 4) * 16, v);
-          mma_bf16(o[b][0], a, v[0], v[1]);
-          mma_bf16(o[b][1], a, v[2], v[3]);
+      for (int b = 0; b < CBW; b++)
+        if (warp + b * kRW < cblocks) {
+          mma_bf16(o[b][0], pa[ks & 1], v[ks & 1][b][0], v[ks & 1][b][1]);
+          mma_bf16(o[b][1], pa[ks & 1], v[ks & 1][b][2], v[ks & 1][b][3]);
         }
-      }
     }
     __syncthreads();   // this stage may be refilled
   }
-  cp_async_wait<0>();
+  if (abort_flag && tid == 0) {
+    // gave up: let the copies in flight land before this memory goes away, and report
+    for (int k = 0; k < 2; k++)
+      for (int spin = 0; spin < 20000 && ntiles > k && !sm100::mbar_try_wait(smem_addr(&full[k]), uint32_t((ntiles - 1 - k) >> 1) & 1u); spin++) __nanosleep(50);
+    atomicExch(p.err, 1);
+  }
   l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1);
   l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
   l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1);
   l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
-  if (quad == 0) { sh_l[warp][r8] = l_lo; sh_l[warp][r8 + 8] = l_hi; }
+  if (quad == 0 && !producer) { sh_l[warp][r8] = l_lo; sh_l[warp][r8 + 8] = l_hi; }
   if (warp == 0 && quad == 0) { sh_ml[r8][0] = m_lo; sh_ml[r8 + 8][0] = m_hi; }
   __syncthreads();     // also: every warp is done with the tiles, whose space now takes the partial results
   float* so = reinterpret_cast<float*>(dsm);   // [16][Rp]
 #pragma unroll
   for (int b = 0; b < CBW; b++) {
     const int cb = warp + b * kRW;
-    if (cb < cblocks) {
+    if (cb < cblocks && !producer) {
 #pragma unroll
       for (int n = 0; n < 2; n++) {
         const int col = cb * 16 + n * 8 + quad * 2;
@@ -411,7 +471,7 @@ __global__ void __launch_bounds__(kRW * 32, 1) k_latent_rows_mma(const RowsParam
   const int nh = min(16, p.heads - h0), total = nh * p.Rp / 4, per = (total + S - 1) / S;
   __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + (size_t(row) * p.heads + h0) * p.Rp;
   const uint32_t soa = smem_addr(so);
-  for (int i = tid; i < per; i += kRW * 32) {
+  for (int i = tid; i < per; i += kRW * 32 + 32) {
     const int idx = sp * per + i;
     if (idx < total) {
       const int h = idx * 4 / p.Rp;
@@ -443,7 +503,7 @@ __global__ void __launch_bounds__(256) k_latent_gather(const uint4* __restrict__
   pdl::grid_dependency_wait();
   const int w = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (w >= n) return;
-  const uint4* src = cache + size_t(slots[w]) * (cu + ku);
+  const uint4* src = cache + size_t(slots[w]) * (cu + ku + kRowPad / 8);
   for (int i = lane; i < cu + ku; i += 32) {
     const uint4 v = src[i];
     if (i < cu) c[size_t(w) * cu + i] = v;
@@ -633,7 +693,7 @@ template <int CBW, int TT>
 cudaError_t launch_rows(const RowsParams& p, dim3 grid, size_t smem, cudaStream_t st) {
   static bool done = false;
   cudaError_t e = allow_smem(k_latent_rows_mma<CBW, TT>, smem, &done);
-  return e != cudaSuccess ? e : pdl::launch(k_latent_rows_mma<CBW, TT>, grid, dim3(kRW * 32), smem, st, p.splits, p);
+  return e != cudaSuccess ? e : pdl::launch(k_latent_rows_mma<CBW, TT>, grid, dim3(kRW * 32 + 32), smem, st, p.splits, p);
 }
 template <int VT>
 cudaError_t launch_prefill(const PrefillParams& p, dim3 grid, size_t smem, cudaStream_t st) {
@@ -667,7 +727,7 @@ int tbv_op_latent_attn_rows(const void* qa, const void* cache, const void* table
   if (rows <= 0) return 0;
   if (heads <= 0 || R > Rp || (Rp % 16) || (rotp % 16) || block_size <= 0) return -2;
   RowsParams p{qa, cache, static_cast<const int*>(tables), static_cast<const int*>(seq_of_row), static_cast<const int*>(ctx_lens),
-               static_cast<const float*>(sink), out, heads, R, Rp, rotp, block_size, max_blocks, 1, scale * kLog2e, scale};
+               static_cast<const float*>(sink), out, heads, R, Rp, rotp, block_size, max_blocks, 1, scale * kLog2e, scale, tbvops::gemm_err_flag()};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   cudaError_t e;
   if (!bf16) {

@@ -138,7 +138,22 @@ struct ScanParams {
   int inner, N, ldu, ldxz, zoff, lddt, ldbc, boff, coff, ldo, ldc, taps;
 };
 
-__device__ __forceinline__ float softplus(float v) { return v > 20.f ? v : log1pf(expf(v)); }
+// log(1 + e^v), relative error near 2^-21 also where it is tiny.  fp32 models: CUDA's functions.  bf16 models: max(v, 0) + log1p(e^-|v|)
+// with log1p(e) = 2 atanh(e / (2 + e)), whose series in the square of e / (2 + e) <= 1/3 is cut after the 15th power.
+template <typename T> __device__ __forceinline__ float softplus(float v);
+template <> __device__ __forceinline__ float softplus<float>(float v) { return v > 20.f ? v : log1pf(expf(v)); }
+template <> __device__ __forceinline__ float softplus<__nv_bfloat16>(float v) {
+  const float e = __expf(-fabsf(v)), r = __fdividef(e, 2.f + e), q = r * r;
+  float h = 1.f / 15.f;
+  h = fmaf(h, q, 1.f / 13.f);
+  h = fmaf(h, q, 1.f / 11.f);
+  h = fmaf(h, q, 1.f / 9.f);
+  h = fmaf(h, q, 1.f / 7.f);
+  h = fmaf(h, q, 1.f / 5.f);
+  h = fmaf(h, q, 1.f / 3.f);
+  h = fmaf(h, q, 1.f);
+  return fmaxf(v, 0.f) + 2.f * r * h;
+}
 // 2^x: the hardware instruction for bf16 models, CUDA's exp2f for fp32 ones
 template <typename T> __device__ __forceinline__ float pow2(float x);
 template <> __device__ __forceinline__ float pow2<float>(float x) { return exp2f(x); }
@@ -187,45 +202,59 @@ __global__ void __launch_bounds__(128) k_selective_scan(const ScanParams p) {
   const bool fresh = p.positions[first] == 0;
   const T* u = static_cast<const T*>(p.u);
   const T* xz = static_cast<const T*>(p.xz);
-  T* out = static_cast<T*>(p.out);
   float* sp = p.ssm + (size_t(slot) * p.inner + c) * p.N + n0;
 #pragma unroll
   for (int i = 0; i < NPL; i++) s[i] = active && n0 + i < p.N && !fresh ? sp[i] : 0.f;
 
-  float ru[EX], rd[EX], rg[EX], rb[EB], rc[EB];
+  // raw values: nothing here depends on a load before the next tile is staged
+  T ru[EX], rg[EX], zero;
+  from_f(zero, 0.f);
+  float rd[EX], rb[EB], rc[EB];
+  // element e of this thread: row tx + e * kRX of the tile, channel c0 + cx (and row tn + .., state nn + .. of B and C)
+  constexpr int kRX = 128 / kC;
+  const int tx = threadIdx.x / kC, cx = threadIdx.x % kC;
+  const bool cok = c0 + cx < p.inner;
+  const T* pu = u + (size_t(first) + tx) * p.ldu + c0 + cx;
+  const T* pz = xz + (size_t(first) + tx) * p.ldxz + p.zoff + c0 + cx;
+  const float* pd = p.dt + (size_t(first) + tx) * p.lddt + c0 + cx;
+  const float* pb = p.bc + size_t(first) * p.ldbc;
   auto fetch = [&](int t0) {
 #pragma unroll
     for (int e = 0; e < EX; e++) {
-      const int id = threadIdx.x + e * 128, t = id / kC, cc = c0 + id % kC;
-      const bool ok = id < TT * kC && t0 + t < count && cc < p.inner;
-      const size_t row = size_t(first) + t0 + t;
-      ru[e] = ok ? to_f(u[row * p.ldu + cc]) : 0.f;
-      rd[e] = ok ? p.dt[row * p.lddt + cc] : 0.f;
-      rg[e] = ok ? to_f(xz[row * p.ldxz + p.zoff + cc]) : 0.f;
+      const int t = tx + e * kRX;
+      const bool ok = cok && t < TT && t0 + t < count;
+      ru[e] = ok ? pu[e * kRX * p.ldu] : zero;
+      rd[e] = ok ? pd[e * kRX * p.lddt] : 0.f;
+      rg[e] = ok ? pz[e * kRX * p.ldxz] : zero;
     }
 #pragma unroll
     for (int e = 0; e < EB; e++) {
       const int id = threadIdx.x + e * 128, t = id / NP, n = id % NP;
       const bool ok = id < TT * NP && t0 + t < count && n < p.N;
-      const size_t row = size_t(first) + t0 + t;
-      rb[e] = ok ? p.bc[row * p.ldbc + p.boff + n] : 0.f;
-      rc[e] = ok ? p.bc[row * p.ldbc + p.coff + n] : 0.f;
+      rb[e] = ok ? pb[t * p.ldbc + p.boff + n] : 0.f;
+      rc[e] = ok ? pb[t * p.ldbc + p.coff + n] : 0.f;
     }
+    pu += size_t(TT) * p.ldu;
+    pz += size_t(TT) * p.ldxz;
+    pd += size_t(TT) * p.lddt;
+    pb += size_t(TT) * p.ldbc;
   };
+  T* po = static_cast<T*>(p.out) + (size_t(first) + tx) * p.ldo + c0 + cx;
   fetch(0);
   for (int t0 = 0; t0 < count; t0 += TT) {
     const int nt = min(TT, count - t0);
     __syncthreads();
 #pragma unroll
     for (int e = 0; e < EX; e++) {
-      const int id = threadIdx.x + e * 128, t = id / kC, cc = id % kC;
-      if (id < TT * kC) {
+      const int t = tx + e * kRX, cc = cx;
+      if (t < TT) {
         // rows past the end get a zero step: they leave the state as it is
-        const float dt = t < nt ? softplus(rd[e]) : 0.f;
+        const float dt = t < nt ? softplus<T>(rd[e]) : 0.f;
         sdt[cc][t] = dt;
-        sdx[cc][t] = dt * ru[e];
-        su[t][cc] = ru[e];
-        sg[t][cc] = silu(rg[e]);
+        const float uv = to_f(ru[e]);
+        sdx[cc][t] = dt * uv;
+        su[t][cc] = uv;
+        sg[t][cc] = silu(to_f(rg[e]));
       }
     }
 #pragma unroll
@@ -247,6 +276,11 @@ __global__ void __launch_bounds__(128) k_selective_scan(const ScanParams p) {
 #pragma unroll
         for (int j = 0; j < 4; j++) {
           float bv[NPL], cv[NPL];
+          if constexpr (NPL == 2) {
+            const float2 b2 = *reinterpret_cast<const float2*>(&sb[tb + q + j][n0]), c2 = *reinterpret_cast<const float2*>(&sc[tb + q + j][n0]);
+            bv[0] = b2.x; bv[1] = b2.y;
+            cv[0] = c2.x; cv[1] = c2.y;
+          } else
 #pragma unroll
           for (int i = 0; i < NPL; i += 4) {
             const float4 b4 = *reinterpret_cast<const float4*>(&sb[tb + q + j][n0 + i]), c4 = *reinterpret_cast<const float4*>(&sc[tb + q + j][n0 + i]);
@@ -288,10 +322,10 @@ __global__ void __launch_bounds__(128) k_selective_scan(const ScanParams p) {
     __syncthreads();
 #pragma unroll
     for (int e = 0; e < EX; e++) {
-      const int id = threadIdx.x + e * 128, t = id / kC, cc = id % kC;
-      if (id < TT * kC && t < nt && c0 + cc < p.inner)
-        from_f(out[(size_t(first) + t0 + t) * p.ldo + c0 + cc], fmaf(sd[cc], su[t][cc], sy[t][cc]) * sg[t][cc]);
+      const int t = tx + e * kRX;
+      if (t < nt && cok) from_f(po[e * kRX * p.ldo], fmaf(sd[cx], su[t][cx], sy[t][cx]) * sg[t][cx]);
     }
+    po += size_t(TT) * p.ldo;
   }
 #pragma unroll
   for (int i = 0; i < NPL; i++)
@@ -329,7 +363,7 @@ __global__ void __launch_bounds__(128) k_scan_step(const ScanParams p) {
     bv[i] = ok ? bc[p.boff + i] : 0.f;
     cv[i] = ok ? bc[p.coff + i] : 0.f;
   }
-  dt = softplus(dt);
+  dt = softplus<T>(dt);
   float y = 0.f;
 #pragma unroll
   for (int i = 0; i < NPL; i++) {
@@ -352,6 +386,9 @@ cudaError_t launch_scan_t(const ScanParams& p, int nseg, bool one, cudaStream_t 
 }
 template <typename T>
 cudaError_t launch_scan(const ScanParams& p, int nseg, bool one, cudaStream_t st) {
+  // few channels x segments: twice the lanes with half the states each keep more warps in flight
+  const bool thin = !one && (long long)p.inner * nseg * 4 <= 148LL * 512;
+  if (thin && p.N > 8 && p.N <= 16) return launch_scan_t<T, 8, 2>(p, nseg, one, st);
   if (p.N <= 4) return launch_scan_t<T, 1, 4>(p, nseg, one, st);
   if (p.N <= 8) return launch_scan_t<T, 2, 4>(p, nseg, one, st);
   if (p.N <= 16) return launch_scan_t<T, 4, 4>(p, nseg, one, st);

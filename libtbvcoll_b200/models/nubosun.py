@@ -33,7 +33,8 @@ class Nubosun:
     # portions of at most this many tokens take the attention's rows form
     ROWS_FORM_MAX = 32
     uses_state = True
-    attn_ctas_per_sm = 1
+    # one CTA of the rows kernel fills an SM, and clusters of eight find only about four fifths of the SMs (15 of them fit)
+    attn_ctas_per_sm = 0.8
 
     def __init__(self, cfg: NubosunConfig, tp: TPGroup, weights: Dict[str, torch.Tensor], device, max_tokens: int, max_batch: int,
                  num_blocks: int, block_size: int = 16, max_attn_splits: int = 8, dtype: torch.dtype = torch.bfloat16):
@@ -57,7 +58,7 @@ class Nubosun:
             "proj": zeros(T * big([_pad16(m.dt_rank + 2 * m.state) for m in mambas]), dt=f32),
             "proj_h": zeros(T * big([_pad16(m.dt_rank + 2 * m.state) for m in mambas]) if dtype is torch.bfloat16 else 0),
             "dt": zeros(T * big([_pad16(m.inner) for m in mambas]), dt=f32),
-            "qa": zeros(T * big([m.heads * (_pad16(m.kv_rank) + _pad16(m.rot_dim)) for m in latents])),
+            "qa": zeros(T * big([m.heads * self._row(m) for m in latents])),
             "lat": zeros(T * big([m.heads * _pad16(m.kv_rank) for m in latents])),
         }
         self.ones = torch.ones(cfg.streams, dtype=f32, device=dev)
@@ -75,7 +76,7 @@ class Nubosun:
                 self.conv.append(zeros(slots, m.conv - 1, _pad16(m.inner), dt=f32))
                 self.ssm.append(zeros(slots, m.inner, m.state, dt=f32))
             else:
-                self.cache.append(zeros(num_blocks * block_size, _pad16(m.kv_rank) + _pad16(m.rot_dim)))
+                self.cache.append(zeros(num_blocks * block_size, self._row(m)))
                 self.conv.append(None)
                 self.ssm.append(None)
                 if i not in self.rot:
@@ -94,6 +95,10 @@ class Nubosun:
     @staticmethod
     def _qkv_cols(m: LatentSpec) -> int:
         return m.heads * (_pad16(m.dim) + _pad16(m.rot_dim)) + _pad16(m.kv_rank) + _pad16(m.rot_dim)
+
+    @staticmethod
+    def _row(m: LatentSpec) -> int:
+        return ops.latent_row(_pad16(m.kv_rank), _pad16(m.rot_dim))
 
     def _buf(self, name: str, rows: int, *shape: int) -> torch.Tensor:
         n = rows
@@ -137,14 +142,14 @@ class Nubosun:
         q_rot = H * D
         c_off = q_rot + H * rot
         qkv, out = self._buf("wide", T, self._qkv_cols(m)), self._buf("mid", T, H * V)
-        qa, lat = self._buf("qa", n, H, R + rot), self._buf("lat", n, H, R)
+        qa, lat = self._buf("qa", n, H, self._row(m)), self._buf("lat", n, H, R)
         freq, factor = self.rot[i]
         cache = self.cache[run]
         ops.linear(h, w[p + "qkv"], qkv)
         ops.latent_prep(qkv, qa, cache, w[p + "dkv.norm"], freq, factor, b.positions, b.slots, n, q_rot, c_off, c_off + R, H, m.kv_rank, R, rot,
                         self.cfg.rms_eps)
         if n:
-            ops.linear(qkv[:n], w[p + "wabs"], qa.view(n, -1), groups=H, x_group=D, y_group=R + rot)
+            ops.linear(qkv[:n], w[p + "wabs"], qa.view(n, -1), groups=H, x_group=D, y_group=self._row(m))
             ops.latent_attention_rows(qa, cache, b.tables, b.seq_of_row, b.ctx, w[p + "sink"], lat, m.kv_rank, m.scale, self.block_size,
                                       splits=b.attn_splits)
             ops.linear(lat.view(n, -1), w[p + "wuv"], out[:n], groups=H, x_group=R, y_group=V)

@@ -411,4 +411,4 @@ def prefill_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
 
 
 from .mixers import (causal_conv_silu, hyper_embed, hyper_mix, latent_attention_prefill, latent_attention_rows, latent_gather,  # noqa: E402,F401
-                     latent_prefill_fits, latent_prep, selective_scan)
+                     latent_prefill_fits, latent_prep, latent_row, selective_scan)

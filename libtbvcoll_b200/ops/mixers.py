@@ -63,12 +63,21 @@ def selective_scan(u, xz, z_off: int, dt, bc, b_off: int, c_off: int, a_log2e, d
     _count()
 
 
+LATENT_ROW_PAD = 8
+
+
+def latent_row(rank_p: int, rot_p: int) -> int:
+    """Values between two rows of the latent cache (and of the folded queries): latent, rotated part, pad (the pitch the rows
+    kernel wants in shared memory)."""
+    return rank_p + rot_p + LATENT_ROW_PAD
+
+
 def latent_prep(qkv, qa, cache, gamma, inv_freq, mscale: float, positions, slots, n_rows_form: int, q_off: int, c_off: int, k_off: int, heads: int,
                 rank: int, rank_p: int, rot_p: int, eps: float) -> None:
     """Rotates the query parts (columns q_off.., heads x rot_p; interleaved pairs) and writes the cache row: RMSNorm of the latent
-    (c_off..) and the rotated key part (k_off..).  The first n_rows_form rows' query parts go to qa [rows, heads, rank_p + rot_p], the
-    others stay in place.  cos and sin are multiplied by mscale."""
-    assert qkv.dtype is qa.dtype is cache.dtype and cache.shape[1] == rank_p + rot_p and positions.dtype is torch.int32 and slots.dtype is torch.int64
+    (c_off..) and the rotated key part (k_off..).  The first n_rows_form rows' query parts go to qa [rows, heads, row], the
+    others stay in place.  Rows of qa and cache: ``latent_row``.  cos and sin are multiplied by mscale."""
+    assert qkv.dtype is qa.dtype is cache.dtype and cache.shape[1] == latent_row(rank_p, rot_p) and positions.dtype is torch.int32 and slots.dtype is torch.int64
     _chk(lib().tbv_op_latent_prep(_p(qkv), _p(qa), _p(cache), _p(gamma), _p(inv_freq), _p(positions), _p(slots), qkv.shape[0], n_rows_form,
                                   qkv.stride(0), q_off, c_off, k_off, heads, rank, rank_p, rot_p, inv_freq.shape[0], eps, mscale, _is_bf16(qkv), _st()),
          "tbv_op_latent_prep")
@@ -76,11 +85,11 @@ def latent_prep(qkv, qa, cache, gamma, inv_freq, mscale: float, positions, slots
 
 
 def latent_attention_rows(qa, cache, tables, seq_of_row, ctx_lens, sink, out, rank: int, scale: float, block_size: int, splits: int = 1) -> None:
-    """qa [rows, heads, Dk] against the cache rows (keys over all Dk columns, values = the first out.shape[2] columns); softmax with
+    """qa [rows, heads, row] against the cache rows (keys over all columns of ``latent_row`` but the pad, values = the first out.shape[2] columns); softmax with
     exp(sink) in the denominator (sink fp32 [heads] or None)."""
-    rows, H, Dk = qa.shape
-    Rp = out.shape[2]
-    assert qa.is_contiguous() and out.is_contiguous() and cache.shape[1] == Dk and qa.dtype is cache.dtype is out.dtype
+    rows, H, row = qa.shape
+    Rp, Dk = out.shape[2], row - LATENT_ROW_PAD
+    assert qa.is_contiguous() and out.is_contiguous() and cache.shape[1] == row and qa.dtype is cache.dtype is out.dtype
     assert tables.dtype is torch.int32 and ctx_lens.dtype is torch.int32
     _chk(lib().tbv_op_latent_attn_rows(_p(qa), _p(cache), _p(tables), _p(seq_of_row), _p(ctx_lens), _p(sink), _p(out), rows, H, rank, Rp, Dk - Rp,
                                        block_size, tables.shape[1], splits, scale, _is_bf16(qa), _st()), "tbv_op_latent_attn_rows")
