@@ -31,6 +31,23 @@ __device__ __forceinline__ void load8(const __nv_bfloat16* p, float* f) {
   f[4] = __uint_as_float(v.z << 16); f[5] = __uint_as_float(v.z & 0xffff0000u);
   f[6] = __uint_as_float(v.w << 16); f[7] = __uint_as_float(v.w & 0xffff0000u);
 }
+// eight channels as they lie in memory
+template <typename T> struct Raw8;
+template <> struct Raw8<float> {
+  float4 a, b;
+  __device__ __forceinline__ void load(const float* p) { a = *reinterpret_cast<const float4*>(p); b = *reinterpret_cast<const float4*>(p + 4); }
+  __device__ __forceinline__ void unpack(float* f) const { f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w; }
+};
+template <> struct Raw8<__nv_bfloat16> {
+  uint4 v;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { v = *reinterpret_cast<const uint4*>(p); }
+  __device__ __forceinline__ void unpack(float* f) const {
+    f[0] = __uint_as_float(v.x << 16); f[1] = __uint_as_float(v.x & 0xffff0000u);
+    f[2] = __uint_as_float(v.y << 16); f[3] = __uint_as_float(v.y & 0xffff0000u);
+    f[4] = __uint_as_float(v.z << 16); f[5] = __uint_as_float(v.z & 0xffff0000u);
+    f[6] = __uint_as_float(v.w << 16); f[7] = __uint_as_float(v.w & 0xffff0000u);
+  }
+};
 __device__ __forceinline__ void store8(float* p, const float* f) {
   *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
   *reinterpret_cast<float4*>(p + 4) = make_float4(f[4], f[5], f[6], f[7]);
@@ -74,21 +91,24 @@ __global__ void __launch_bounds__(128) k_causal_conv_silu(const ConvParams p) {
   if (c8 >= p.ldc) return;
   const T* x = static_cast<const T*>(p.x);
   const int t0 = blockIdx.y * R;
-  if (R > 1 && TAPS > 0 && t0 + R <= p.rows) {
+  if (R > 1 && TAPS > 0 && t0 >= TAPS - 1 && t0 + R <= p.rows) {
+    // the window is requested before it is known whether the rows share a segment
+    Raw8<T> win[TAPS > 0 ? TAPS + R - 1 : 1];
+#pragma unroll
+    for (int i = 0; i < TAPS + R - 1; i++) win[i].load(x + size_t(t0 - (TAPS - 1) + i) * p.ldx + c8);
     const int sa = p.seg_of_row ? p.seg_of_row[t0] : t0, sb = p.seg_of_row ? p.seg_of_row[t0 + R - 1] : t0 + R - 1;
     if (sa == sb && t0 - p.segs[4 * sa] >= taps - 1) {
-      float win[TAPS > 0 ? TAPS + R - 1 : 1][8];
-#pragma unroll
-      for (int i = 0; i < TAPS + R - 1; i++) load8(x + size_t(t0 - (TAPS - 1) + i) * p.ldx + c8, win[i]);
 #pragma unroll
       for (int r = 0; r < R; r++) {
-        float acc[8];
+        float acc[8], v[8];
 #pragma unroll
         for (int i = 0; i < 8; i++) acc[i] = bias[i];
 #pragma unroll
-        for (int k = 0; k < TAPS; k++)
+        for (int k = 0; k < TAPS; k++) {
+          win[r + k].unpack(v);
 #pragma unroll
-          for (int i = 0; i < 8; i++) acc[i] = fmaf(w[k][i], win[r + k][i], acc[i]);
+          for (int i = 0; i < 8; i++) acc[i] = fmaf(w[k][i], v[i], acc[i]);
+        }
 #pragma unroll
         for (int i = 0; i < 8; i++) acc[i] = silu(acc[i]);
         store8(static_cast<T*>(p.out) + size_t(t0 + r) * p.ldo + c8, acc);

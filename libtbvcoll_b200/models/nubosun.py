@@ -83,7 +83,7 @@ class Nubosun:
                     f, factor = ops.rope_frequencies(m.rot.dims, m.rot.base, m.rot.scaling)
                     self.rot[i] = (f.to(f32).to(dev), factor)
         self.attn_ctas_per_row = max([(m.heads + 15) // 16 for m in latents], default=1)
-        two_forms = dtype is torch.bfloat16 and all(ops.latent_prefill_fits(_pad16(m.dim), _pad16(m.rot_dim), _pad16(m.vdim)) for m in latents)
+        two_forms = bool(latents) and dtype is torch.bfloat16 and all(ops.latent_prefill_fits(_pad16(m.dim), _pad16(m.rot_dim), _pad16(m.vdim)) for m in latents)
         self.rows_form_max = self.ROWS_FORM_MAX if two_forms else 1 << 60
         self._ctx_rows = 0
 

@@ -2,12 +2,21 @@
 
 One function per mechanism, written for whole sequences with ordinary loops and matrix products, in float32 (or float64
 on request), no cache, no state hand-over, no batching, nothing shared with the product code.  ``w`` maps checkpoint tensor names to tensors
-and ``cfg`` is the parsed ``config.json`` dictionary."""
+and ``cfg`` is the parsed ``config.json`` dictionary.  ``r`` rounds what a 16-bit run may keep in 16 bits (inputs and results of matrix
+products, short convolutions, cached rows); it is the identity unless the size of those roundings is wanted."""
 from __future__ import annotations
 
 import math
 
 import torch
+
+
+def exact(x):
+    return x
+
+
+def to_bf16(x):
+    return x.to(torch.bfloat16).to(x.dtype)
 
 
 def rms(x, eps):
@@ -46,16 +55,16 @@ def selective_scan(u, dt, a_log, b, c, d):
     return out
 
 
-def mamba_mixer(h, w, p, m):
+def mamba_mixer(h, w, p, m, r=exact):
     inner, state, rank = m["inner"], m["state"], m["dt_rank"]
-    xz = h @ w[p + "in"].T
+    xz = r(r(h) @ w[p + "in"].T)
     x, z = xz[:, :inner], xz[:, inner:]
-    x = silu(causal_conv(x, w[p + "conv"], w[p + "conv.b"]))
+    x = r(silu(causal_conv(x, w[p + "conv"], w[p + "conv.b"])))
     proj = x @ w[p + "x"].T
-    dt = softplus(proj[:, :rank] @ w[p + "dt"].T + w[p + "dt.b"])
+    dt = softplus(r(proj[:, :rank]) @ w[p + "dt"].T + w[p + "dt.b"])
     b, c = proj[:, rank:rank + state], proj[:, rank + state:]
     y = selective_scan(x, dt, w[p + "A_log"], b, c, w[p + "D"])
-    return (y * silu(z)) @ w[p + "o"].T
+    return r(y * silu(z)) @ w[p + "o"].T
 
 
 def rotary_frequencies(rot):
@@ -97,28 +106,28 @@ def sink_softmax(scores, sink):
     return e / (e.sum(-1, keepdim=True) + torch.exp(sink[:, None, None] - m))
 
 
-def latent_attention_mixer(h, w, p, m, eps, first_position=0):
+def latent_attention_mixer(h, w, p, m, eps, r=exact):
     T = h.shape[0]
     H, dim, rd, vd, R = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
-    pos = torch.arange(T) + first_position
-    q = (h @ w[p + "q"].T).view(T, H, dim + rd)
-    kv = h @ w[p + "dkv"].T
-    c = rms(kv[:, :R], eps) * w[p + "dkv.norm"]
-    kr = rotate_pairs(kv[:, None, R:], pos, m["rot"])[:, 0]
-    qr = rotate_pairs(q[..., dim:], pos, m["rot"])
-    k = (c @ w[p + "uk"].T).view(T, H, dim)
-    v = (c @ w[p + "uv"].T).view(T, H, vd)
+    pos = torch.arange(T)
+    q = r(r(h) @ w[p + "q"].T).view(T, H, dim + rd)
+    kv = r(r(h) @ w[p + "dkv"].T)
+    c = r(rms(kv[:, :R], eps) * w[p + "dkv.norm"])
+    kr = r(rotate_pairs(kv[:, None, R:], pos, m["rot"])[:, 0])
+    qr = r(rotate_pairs(q[..., dim:], pos, m["rot"]))
+    k = r(c @ w[p + "uk"].T).view(T, H, dim)
+    v = r(c @ w[p + "uv"].T).view(T, H, vd)
     s = (torch.einsum("ihd,jhd->hij", q[..., :dim], k) + torch.einsum("ihd,jd->hij", qr, kr)) * m["scale"]
     s = s.masked_fill(torch.ones(T, T, dtype=torch.bool).triu(1)[None], float("-inf"))
-    o = torch.einsum("hij,jhd->ihd", sink_softmax(s, w[p + "sink"]), v)
+    o = r(torch.einsum("hij,jhd->ihd", r(sink_softmax(s, w[p + "sink"])), v))
     return o.reshape(T, H * vd) @ w[p + "o"].T
 
 
-def clamped_glu_mlp(h, w, p, m):
-    lim = m["limit"]
+def clamped_glu_mlp(h, w, p, m, r=exact):
+    lim, h = m["limit"], r(h)
     g = torch.clamp(h @ w[p + "gate"].T, max=lim)
     u = torch.clamp(h @ w[p + "up"].T, -lim, lim)
-    return (g / (1.0 + torch.exp(-1.702 * g)) * (u + 1.0)) @ w[p + "down"].T
+    return r(g / (1.0 + torch.exp(-1.702 * g)) * (u + 1.0)) @ w[p + "down"].T
 
 
 def hyper_sublayer(xs, fn, gamma, scale, hin, hout, hmix, eps):
@@ -137,7 +146,7 @@ def layer_order(cfg):
     return list(range(lp["start"])) + list(range(lp["start"], lp["stop"])) * lp["times"] + list(range(lp["stop"], n))
 
 
-def forward(cfg, w, tokens, dtype=torch.float32, collect=None):
+def forward(cfg, w, tokens, dtype=torch.float32, collect=None, r=exact):
     """Logits [T, vocab] of one sequence; ``collect`` (a list) receives the summed streams after every layer run."""
     w = {k: v.to(dtype) for k, v in w.items()}
     eps = cfg["norm"]["eps"]
@@ -147,17 +156,17 @@ def forward(cfg, w, tokens, dtype=torch.float32, collect=None):
         lay, p = cfg["layers"][i], f"l{i}."
         m = lay["mixer"]
         if lay["type"] == "mamba1":
-            fn = lambda h: mamba_mixer(h, w, p + "mix.", m)
+            fn = lambda h: mamba_mixer(h, w, p + "mix.", m, r)
         elif lay["type"] == "latent_attention":
-            fn = lambda h: latent_attention_mixer(h, w, p + "mix.", m, eps)
+            fn = lambda h: latent_attention_mixer(h, w, p + "mix.", m, eps, r)
         else:
             raise ValueError(lay["type"])
         xs = hyper_sublayer(xs, fn, w[p + "norm1"], w[p + "ls1"], w[p + "hc1.in"], w[p + "hc1.out"], w[p + "hc1.mix"], eps)
         if lay["mlp"] is not None:
-            fn = lambda h: clamped_glu_mlp(h, w, p + "mlp.", lay["mlp"])
+            fn = lambda h: clamped_glu_mlp(h, w, p + "mlp.", lay["mlp"], r)
             xs = hyper_sublayer(xs, fn, w[p + "norm2"], w[p + "ls2"], w[p + "hc2.in"], w[p + "hc2.out"], w[p + "hc2.mix"], eps)
         if collect is not None:
             collect.append(sum(xs))
-    logits = (rms(sum(xs), eps) * w["final.norm"]) @ w["head"].T
+    logits = r(rms(sum(xs), eps) * w["final.norm"]) @ w["head"].T
     cap = cfg["logit_softcap"]
     return cap * torch.tanh(logits / cap)

@@ -1,0 +1,292 @@
+"""Nubosun through the engine: whole prompts, portions, mixed batches, pages and slots used again, decoding, generation, the trace replay
+and the command line, against the plain statement in ``nubosun_oracle``."""
+import json
+import os
+import random
+import subprocess
+import sys
+
+import numpy as np
+import pytest
+import torch
+
+import nubosun_cases as cases
+import nubosun_oracle as oracle
+
+pytestmark = pytest.mark.gpu
+ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+BF, F32 = torch.bfloat16, torch.float32
+
+
+class Expected:
+    """Oracle logits with a limit per position: in bf16 three times the error that rounding to 16 bits alone causes there (never less than
+    the median over the sequence), in fp32 a fixed one."""
+
+    def __init__(self, logits, limits):
+        self.logits, self.limits = logits, limits
+
+    @staticmethod
+    def of(raw, w, toks):
+        logits = oracle.forward(raw, w, toks)
+        e = Expected.error(oracle.forward(raw, w, toks, r=oracle.to_bf16), logits, logits)
+        return Expected(logits, {BF: 3 * torch.maximum(e, e.median()), F32: torch.full_like(e, 2e-4)})
+
+    @staticmethod
+    def error(got, want, whole):
+        """rms over the vocabulary of the mean-free difference, over the rms of the logits"""
+        d = got.double().cpu() - want.double()
+        d = d - d.mean(-1, keepdim=True)
+        return d.pow(2).mean(-1).sqrt() / whole.double().std()
+
+    def check(self, got, dtype):
+        e = Expected.error(got, self.logits, self.logits) / self.limits[dtype]
+        over = int((e > 1).sum())
+        assert float(e.max()) < 1.5 and over <= max(1, len(e) // 50), (float(e.max()), int(e.argmax()), over)
+
+    def __getitem__(self, rows):
+        return Expected(self.logits[rows], {k: v[rows] for k, v in self.limits.items()})
+
+    @staticmethod
+    def stack(parts):
+        """rows [(Expected, position), ..] of several sequences"""
+        return Expected(torch.stack([e.logits[p] for e, p in parts]), {k: torch.stack([e.limits[k][p] for e, p in parts]) for k in (BF, F32)})
+
+
+def engine(raw, w, dtype, **kw):
+    from libtbvcoll_b200.engine.engine import Engine
+    from libtbvcoll_b200.models.config import parse_nubosun_config
+    kw = {"max_batch": 4, "max_seq_len": 512, "prefill_chunk": 256, **kw}
+    return Engine(parse_nubosun_config(raw), device="cuda:0", source=cases.Source(w), dtype=dtype, **kw)
+
+
+def check(got, want, dtype):
+    want.check(got, dtype)
+
+
+_cache = {}
+
+
+def model(name):
+    """(config, weights, {sequence: tokens}, {sequence: Expected}) of a case, computed once."""
+    if name not in _cache:
+        raw = cases.CASES[name]()
+        w = cases.tensors(raw)
+        seqs = {k: cases.tokens(raw, n, seed=n) for k, n in (("long", 210), ("mid", 77), ("short", 19), ("one", 1))}
+        _cache[name] = raw, w, seqs, {k: Expected.of(raw, w, t) for k, t in seqs.items()}
+    return _cache[name]
+
+
+def feed(eng, key, toks, portions):
+    """Runs one request alone in the given portions; logits of every position."""
+    out, at = [], 0
+    for n in portions:
+        n = min(n, len(toks) - at)
+        if n:
+            out.append(eng.step([(key, toks[at: at + n], range(n))], end=[key] if at + n == len(toks) else []))
+        at += n
+    return torch.cat(out)
+
+
+@pytest.mark.parametrize("dtype", [F32, BF])
+@pytest.mark.parametrize("name", sorted(cases.CASES))
+def test_whole_portions_and_single_tokens(name, dtype):
+    raw, w, seqs, want = model(name)
+    eng = engine(raw, w, dtype)
+    for k, t in seqs.items():
+        check(feed(eng, k, t, [len(t)]), want[k], dtype)
+    t = seqs["long"]
+    for portions in ([2] * 105, [3, 13, 15, 1, 16, 17, 31, 33, 64, 17], [1, 33, 2, 100, 1, 1, 72], [63, 65, 82]):
+        check(feed(eng, "p", t, portions), want["long"], dtype)
+    check(feed(eng, "d", seqs["mid"], [1] * 77), want["mid"], dtype)
+
+
+@pytest.mark.parametrize("dtype", [F32, BF])
+def test_streams_after_every_layer_run(dtype):
+    from libtbvcoll_b200.engine.batch import Portion
+    raw, w, seqs, _ = model("odd")
+    t, want, got = seqs["mid"], [], []
+    oracle.forward(raw, w, t, collect=want)
+    eng = engine(raw, w, dtype)
+    r = eng.requests.extend("a", len(t))
+    eng.bm.sync_to_device()
+    eng.model.forward_batch(eng.batch_of([Portion(r.row, 0, t)]), on_layer=lambda i, x: got.append(x.sum(1).cpu()))
+    assert len(got) == len(want) == 8
+    for g, x in zip(got, want):
+        assert float((g - x).norm() / x.norm()) < (3e-2 if dtype is BF else 5e-6)
+
+
+@pytest.mark.parametrize("dtype", [F32, BF])
+@pytest.mark.parametrize("name", ["odd", "wide"])
+def test_mixed_batches_rows_pages_and_slots_used_again(name, dtype):
+    """Random schedules of unequal requests: portions beside single tokens, requests left out of steps, rows, pages and state slots handed on;
+    the pool is just large enough for what is live."""
+    raw, w, seqs, want = model(name)
+    eng = engine(raw, w, dtype, max_batch=3, max_seq_len=224, max_cache_tokens=224 + 80 + 64, prefill_chunk=150)
+    rng = random.Random(5)
+    todo = [(k, i) for i in range(3) for k in ("mid", "short", "one", "short")] + [("long", 0), ("long", 1)]
+    rng.shuffle(todo)
+    live, at, seen = [], {}, {}
+    while todo or live:
+        while todo and len(live) < 3 and not (todo[0][0] == "long" and any(k == "long" for k, _ in live)) \
+                and sum(len(seqs[k]) for k, _ in live + todo[:1]) <= 290:
+            live.append(todo.pop(0))
+        entries, end, rows = [], [], []
+        for r in rng.sample(live, rng.randint(1, len(live))):
+            t, a = seqs[r[0]], at.get(r, 0)
+            n = min(len(t) - a, rng.choice([1, 1, 1, 2, 5, 16, 33, 70]))
+            pick = sorted(rng.sample(range(n), rng.randint(0, n)))
+            entries.append((r, t[a: a + n], pick))
+            rows += [(r[0], a + p) for p in pick]
+            at[r] = a + n
+            if at[r] == len(t):
+                end.append(r)
+        got = eng.step(entries, end=end)
+        live = [r for r in live if r not in end]
+        assert got.shape == (len(rows), raw["vocab"])
+        if rows:
+            check(got, Expected.stack([(want[k], p) for k, p in rows]), dtype)
+    assert len(eng.bm.free) == eng.bm.num_blocks - 1 and sorted(eng.requests.free_rows) == [0, 1, 2]
+
+
+@pytest.mark.parametrize("dtype", [F32, BF])
+def test_a_batch_gives_what_each_request_gives_alone(dtype):
+    raw, w, seqs, want = model("plain")
+    eng = engine(raw, w, dtype)
+    alone = {k: eng.step([(k, t, range(len(t)))], end=[k]) for k, t in seqs.items()}
+    ks = ["mid", "one", "long", "short"]
+    both = eng.step([(k, seqs[k], range(len(seqs[k]))) for k in ks], end=ks)         # longer than a pass: cut inside "long"
+    at = 0
+    for k in ks:
+        n = len(seqs[k])
+        check(both[at: at + n], Expected(alone[k].cpu(), want[k].limits), dtype)
+        at += n
+
+
+def test_far_token_shows_at_the_end():
+    """Attention made so that the last position looks at one early token: changing it must change the last logits the way the oracle says."""
+    raw, w, _, _ = model("plain")
+    toks = cases.tokens(raw, 330, seed=9)
+    w = dict(w)
+    for k in list(w):
+        if k.endswith("mix.q"):
+            w[k] = (w[k].float() * 6).to(BF)                                         # sharp scores: single keys stand out
+    other = list(toks)
+    other[7] = (other[7] + 1) % raw["vocab"]
+    a, b = Expected.of(raw, w, toks), Expected.of(raw, w, other)
+    assert float((a.logits[-1] - b.logits[-1]).std() / a.logits.std()) > 0.1
+    for dtype in (F32, BF):
+        eng = engine(raw, w, dtype)
+        ga = torch.cat([feed(eng, 0, toks, [330])[-1:], feed(eng, 0, toks, [5, 40, 1, 200, 83, 1])[-1:]])
+        gb = feed(eng, 0, other, [300] + [1] * 30)[-1:]
+        check(ga, a[[-1, -1]], dtype)
+        check(gb, b[[-1]], dtype)
+
+
+def test_long_decoding_through_the_captured_step():
+    """300 tokens decoded one by one after a short prompt: the graph-captured serving loop, the device loop and the eager loop agree, and in
+    fp32 every token is the oracle's choice (where the oracle is not undecided)."""
+    raw, w, seqs, _ = model("odd")
+    prompts = [seqs["short"], seqs["mid"], seqs["one"]]
+    eng = engine(raw, w, F32)
+    outs = eng.generate(prompts, 300)
+    for p, o in zip(prompts, outs):
+        full = oracle.forward(raw, w, p + o[:-1])
+        top = full.topk(2, dim=-1)
+        for i, t in enumerate(o):
+            v = top.values[len(p) - 1 + i]
+            assert t == int(top.indices[len(p) - 1 + i, 0]) or float(v[0] - v[1]) < 1e-3
+    for loop, graph in (("host", False), ("device", True), ("device", False)):
+        assert eng.generate(prompts, 300, loop=loop, use_graph=graph) == outs
+    assert eng.generate(prompts, 300) == outs                                          # captured before: state starts afresh
+    half = engine(raw, w, BF)
+    a = half.generate(prompts, 120)
+    assert a == half.generate(prompts, 120, loop="device") == half.generate(prompts, 120, use_graph=False)
+
+
+def test_generation_through_the_scheduler():
+    """More prompts than rows, a pool that cannot hold them all: the scheduler's mixed steps give what static batches give."""
+    raw, w, seqs, _ = model("wide")
+    prompts = [cases.tokens(raw, n, seed=100 + n) for n in (60, 3, 17, 90, 1, 33, 45)]
+    eng = engine(raw, w, F32, max_batch=3, max_seq_len=128, max_cache_tokens=256, prefill_chunk=40)
+    outs = eng.generate(prompts, 12)                                                   # 7 prompts > 3 rows
+    alone = engine(raw, w, F32, max_batch=1, max_seq_len=128)
+    assert outs == [alone.generate([p], 12)[0] for p in prompts]
+    stop = outs[0][4]
+    cut = eng.generate(prompts, 12, eos_id=stop)
+    assert cut == [o[: o.index(stop) + 1] if stop in o else o for o in outs]
+
+
+def test_capture_leaves_no_trace_in_the_state():
+    raw, w, seqs, _ = model("scans")
+    a = engine(raw, w, F32, max_batch=2)
+    first = a.prefill([seqs["short"], seqs["mid"]], 8)
+    before = [s.clone() for s in a.model.ssm + a.model.conv]
+    a._load_decode_inputs(2, first, [len(seqs["short"]), len(seqs["mid"])])
+    a.capture(2, 1, True)
+    torch.cuda.synchronize()
+    for s, b in zip(a.model.ssm + a.model.conv, before):
+        assert torch.equal(s[1:], b[1:])
+
+
+def run_trace(path, out, dtype, steps, n):
+    env = dict(os.environ, HOME=str(out))
+    r = subprocess.run([os.path.join(ROOT, "bin", "trace_run"), "--model", str(path), "--dtype", dtype, "--out", str(out), "--max-tokens", str(n)],
+                       input="".join(json.dumps(s) + "\n" for s in steps), capture_output=True, text=True, timeout=600, env=env)
+    return r
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_trace_replay(tmp_path, dtype):
+    raw, w, seqs, want = model("plain")
+    cases.write_checkpoint(str(tmp_path), raw, w)
+    m, s = seqs["mid"], seqs["short"]
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": m[:40], "want": [0, 39]}], "end": []},
+             {"step": 1, "entries": [{"id": "b", "tokens": s[:2], "want": []}, {"id": "a", "tokens": m[40:41], "want": []}], "end": []},
+             {"step": 2, "entries": [{"id": "a", "tokens": m[41:], "want": [35, 0]}, {"id": "b", "tokens": s[2:], "want": [16]}], "end": ["a"]},
+             {"step": 3, "entries": [{"id": "a", "tokens": s, "want": [18]}], "end": ["a", "b"]}]
+    r = run_trace(tmp_path, tmp_path, dtype, steps, 128)
+    assert r.returncode == 0, r.stderr[-2000:]
+    assert [ln for ln in r.stdout.splitlines() if ln.startswith("done")] == [f"done {i}" for i in range(4)]
+    assert not os.path.exists(tmp_path / "1.f32")
+    read = lambda i: torch.from_numpy(np.fromfile(tmp_path / f"{i}.f32", dtype="<f4").reshape(-1, raw["vocab"]).copy())
+    dt = getattr(torch, dtype)
+    check(read(0), want["mid"][[0, 39]], dt)
+    check(read(2), Expected.stack([(want["mid"], 76), (want["mid"], 41), (want["short"], 18)]), dt)
+    check(read(3), want["short"][[18]], dt)
+
+
+def test_trace_replay_of_a_llama_checkpoint_and_the_refused_dtype(tmp_path):
+    """The replay picks the model by config.json: a Llama-family directory runs the same way, in bf16 only."""
+    from libtbvcoll_b200.engine.engine import Engine
+    from libtbvcoll_b200.models.config import get_config
+    from libtbvcoll_b200.utils.weights import RandomSource, save_hf_checkpoint
+    cfg = get_config("tiny")
+    src = RandomSource(cfg, seed=2)
+    save_hf_checkpoint(src, str(tmp_path))
+    (tmp_path / "config.json").write_text(json.dumps({
+        "model_type": "llama", "hidden_size": cfg.hidden_size, "num_hidden_layers": cfg.num_layers, "num_attention_heads": cfg.num_heads,
+        "num_key_value_heads": cfg.num_kv_heads, "head_dim": cfg.head_dim, "intermediate_size": cfg.intermediate_size, "vocab_size": cfg.vocab_size,
+        "rope_theta": cfg.rope_theta, "rms_norm_eps": cfg.rms_eps, "max_position_embeddings": cfg.max_position}))
+    toks = torch.randint(0, cfg.vocab_size, (50,), generator=torch.Generator().manual_seed(0)).tolist()
+    steps = [{"step": 0, "entries": [{"id": "x", "tokens": toks[:30], "want": list(range(20))}], "end": []},
+             {"step": 1, "entries": [{"id": "x", "tokens": toks[30:], "want": [19]}], "end": ["x"]}]
+    r = run_trace(tmp_path, tmp_path, "bfloat16", steps, 64)
+    assert r.returncode == 0, r.stderr[-2000:]
+    got = np.fromfile(tmp_path / "1.f32", dtype="<f4")
+    eng = Engine(cfg, device="cuda:0", source=src, max_batch=1, max_seq_len=64)
+    eng.prefill([toks], 1)
+    ref = eng.model.logits[0].float().cpu().numpy()
+    assert np.abs(got - ref).max() < 0.05 * np.abs(ref).max() + 0.02
+    assert np.fromfile(tmp_path / "0.f32", dtype="<f4").size == 20 * cfg.vocab_size
+    assert run_trace(tmp_path, tmp_path, "float32", steps, 64).returncode == 3
+
+
+def test_generate_command_line(tmp_path):
+    raw, w, seqs, _ = model("plain")
+    cases.write_checkpoint(str(tmp_path), raw, w)
+    r = subprocess.run([sys.executable, "-m", "libtbvcoll_b200.generate", "--model", str(tmp_path), "--dtype", "float32", "--new", "6",
+                        "--prompt", ",".join(map(str, seqs["short"])), "--prompt", "3"], capture_output=True, text=True, timeout=600, cwd=ROOT)
+    assert r.returncode == 0, r.stderr[-2000:]
+    rows = [json.loads(ln) for ln in r.stdout.splitlines() if ln.startswith("{")]
+    assert [len(x["tokens"]) for x in rows] == [6, 6]
+    assert rows[0]["tokens"] == engine(raw, w, F32).generate([seqs["short"], [3]], 6)[0]
