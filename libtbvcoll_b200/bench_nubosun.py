@@ -6,7 +6,8 @@ throughput through the engine, and every kernel of both at the same shapes again
 
 Random weights, random token ids.  Model numbers: device time of captured decode steps (CUDA events), prefill by events around
 the engine's prefill.  Kernel numbers: ``reps`` distinct sets of operands (more than the L2 in total) cycled inside one CUDA graph; roofline
-time = max(bytes / measured copy bandwidth, FLOPs / measured bf16 rate), fraction = roofline time / measured time."""
+time = max(bytes / measured copy bandwidth, FLOPs / measured bf16 rate, for the scan also exponentials / 16 per clock and SM at 1965 MHz),
+fraction = roofline time / measured time."""
 from __future__ import annotations
 
 import argparse
@@ -76,14 +77,15 @@ class _Kernels:
         from .bench_ops import peaks
         self.hbm, self.tf, self.src = peaks()
         self.rows = []
+        self.sms = torch.cuda.get_device_properties(0).multi_processor_count
 
-    def time(self, group: str, name: str, make, bytes_, flops=0.0):
+    def time(self, group: str, name: str, make, bytes_, flops=0.0, exps=0.0):
         """make(i) -> callable on the i-th set of operands; sets are made until they exceed the L2."""
         from .bench_ops import time_graph
         torch.cuda.empty_cache()
         sets = max(2, min(64, math.ceil(400e6 / max(bytes_, 1.0))))
         us = time_graph([make(i) for i in range(sets)])
-        ideal = max(bytes_ / (self.hbm * 1e3), flops / (self.tf * 1e6))
+        ideal = max(bytes_ / (self.hbm * 1e3), flops / (self.tf * 1e6), exps / (16 * self.sms * 1.965e3))
         self.rows.append({"group": group, "kernel": name, "us": round(us, 2), "roofline_us": round(ideal, 2), "of_measured_peak": round(ideal / us, 3)})
 
 
@@ -113,6 +115,8 @@ def kernel_numbers(size: str, T: int, seqs: int, ctx: int) -> list:
     from . import ops
     from .engine.batch import dense_context
     from .models.config import LatentSpec, MambaSpec, get_config
+    from .models.llama import LlamaTP
+    from .models.nubosun import Nubosun
     nb, ll = (get_config(n) for n in PAIRS[size])
     m = next(l.mixer for l in nb.layers if isinstance(l.mixer, MambaSpec))
     a = next(l.mixer for l in nb.layers if isinstance(l.mixer, LatentSpec))
@@ -190,7 +194,8 @@ def kernel_numbers(size: str, T: int, seqs: int, ctx: int) -> list:
         a2, d = -torch.rand(m.inner, m.state, device=dev), torch.ones(m.inner, device=dev)
         ssm, st = torch.zeros(seqs + 1, m.inner, m.state, device=dev), torch.zeros(seqs + 1, m.conv - 1, ip, device=dev)
         return lambda: ops.selective_scan(u, xz, ip, dt, bc, m.dt_rank, m.dt_rank + m.state, a2, d, ssm, st, u, segs, pos, one_token=decode)
-    k.time("scan", "nubosun selective scan", mk_scan, T * ip * 10 + T * m.state * 8 + seqs * m.inner * m.state * (8 if decode else 4) + m.inner * m.state * 4)
+    k.time("scan", "nubosun selective scan", mk_scan, T * ip * 10 + T * m.state * 8 + seqs * m.inner * m.state * (8 if decode else 4) + m.inner * m.state * 4,
+           exps=float(T) * m.inner * m.state)
 
     # attention
     R, rot, H = _pad16(a.kv_rank), _pad16(a.rot_dim), a.heads
@@ -206,21 +211,21 @@ def kernel_numbers(size: str, T: int, seqs: int, ctx: int) -> list:
     sink = torch.zeros(H, device=dev)
     sms = torch.cuda.get_device_properties(0).multi_processor_count
 
-    def splits(units, per_sm):
+    def splits(units, slots):
         s = 1
-        while s < 8 and seqs * units * s * 2 <= per_sm * sms and ctx // (s * 2) >= 64:
+        while s < 8 and seqs * units * s * 2 <= slots(s * 2, sms) and ctx // (s * 2) >= 64:
             s *= 2
         return s
     if decode:
         def mk_rows(i):
             qa, cache, o = _w(T, H, Dk + 8), _w(nslots, Dk + 8), torch.empty(T, H, R, dtype=bf, device=dev)
-            sp = splits((H + 15) // 16, 0.8)
+            sp = splits((H + 15) // 16, Nubosun.attn_cta_slots)
             return lambda: ops.latent_attention_rows(qa, cache, tables, seq_of_row, ctx_lens, sink, o, R, a.scale, bs, splits=sp)
         k.time("attention", "nubosun latent attention, rows form", mk_rows, seqs * ctx * Dk * 2 + T * H * (Dk + R) * 2, 2.0 * pairs_causal * H * (Dk + R))
 
         def mk_paged(i):
             q, kc, vc, o = _w(T, nq, D), _w(nslots, nkv, D), _w(nslots, nkv, D), torch.empty(T, nq, D, dtype=bf, device=dev)
-            sp = splits(nkv, 2)
+            sp = splits(nkv, LlamaTP.attn_cta_slots)
             return lambda: ops.paged_attention(q, kc, vc, tables, ctx_lens, o, D ** -0.5, bs, splits=sp)
         k.time("attention", "llama paged attention", mk_paged, seqs * ctx * nkv * D * 4 + T * nq * D * 4, 4.0 * pairs_causal * nq * D)
     else:

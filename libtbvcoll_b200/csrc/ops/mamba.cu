@@ -18,7 +18,11 @@ __device__ __forceinline__ float to_f(float v) { return v; }
 __device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
 __device__ __forceinline__ void from_f(float& d, float v) { d = v; }
 __device__ __forceinline__ void from_f(__nv_bfloat16& d, float v) { d = __float2bfloat16_rn(v); }
-__device__ __forceinline__ float silu(float v) { return v / (1.0f + __expf(-v)); }
+__device__ __forceinline__ float silu(float v) { return v / (1.0f + expf(-v)); }
+// SiLU: bf16 models take the fast exponential and division (1 + e^-v may overflow to infinity: the quotient is 0)
+template <typename T> __device__ __forceinline__ float gate(float v);
+template <> __device__ __forceinline__ float gate<float>(float v) { return silu(v); }
+template <> __device__ __forceinline__ float gate<__nv_bfloat16>(float v) { return __fdividef(v, 1.0f + __expf(-v)); }
 
 __device__ __forceinline__ void load8(const float* p, float* f) {
   const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
@@ -110,7 +114,7 @@ __global__ void __launch_bounds__(128) k_causal_conv_silu(const ConvParams p) {
           for (int i = 0; i < 8; i++) acc[i] = fmaf(w[k][i], v[i], acc[i]);
         }
 #pragma unroll
-        for (int i = 0; i < 8; i++) acc[i] = silu(acc[i]);
+        for (int i = 0; i < 8; i++) acc[i] = gate<T>(acc[i]);
         store8(static_cast<T*>(p.out) + size_t(t0 + r) * p.ldo + c8, acc);
       }
       return;
@@ -138,7 +142,7 @@ __global__ void __launch_bounds__(128) k_causal_conv_silu(const ConvParams p) {
       for (int i = 0; i < 8; i++) acc[i] = fmaf(TAPS > 0 ? w[TAPS > 0 ? k : 0][i] : wk[i], none ? 0.f : v[i], acc[i]);
     }
 #pragma unroll
-    for (int i = 0; i < 8; i++) acc[i] = silu(acc[i]);
+    for (int i = 0; i < 8; i++) acc[i] = gate<T>(acc[i]);
     store8(static_cast<T*>(p.out) + size_t(t) * p.ldo + c8, acc);
   }
 }
@@ -183,6 +187,25 @@ template <> __device__ __forceinline__ float pow2<__nv_bfloat16>(float x) {
   return y;
 }
 
+// Two fp32 values in a 64-bit register pair: one instruction does both (each rounded as its scalar form).
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack2(float a, float b) {
+  f32x2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ void unpack2(f32x2 v, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+  f32x2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+
 // Replaces the convolution state of channel c by its last taps - 1 inputs; ascending, so an old entry is read before it is overwritten.
 template <typename T>
 __device__ __forceinline__ void roll_conv_state(const ScanParams& p, const T* xz, int first, int count, int slot, bool fresh, int c) {
@@ -212,9 +235,13 @@ __global__ void __launch_bounds__(128) k_selective_scan(const ScanParams p) {
   pdl::launch_dependents();
   const int c0 = blockIdx.x * kC, cl = threadIdx.x / LPC, c = c0 + cl, lane = threadIdx.x % LPC, n0 = lane * NPL;
   const bool active = c < p.inner;
-  float a[NPL], s[NPL];
+  constexpr int NQ = NPL / 2;
+  f32x2 a[NQ], s[NQ];
 #pragma unroll
-  for (int i = 0; i < NPL; i++) a[i] = active && n0 + i < p.N ? p.a2[size_t(c) * p.N + n0 + i] : 0.f;
+  for (int i = 0; i < NQ; i++) {
+    const float* ap = p.a2 + size_t(c) * p.N + n0 + 2 * i;
+    a[i] = pack2(active && n0 + 2 * i < p.N ? ap[0] : 0.f, active && n0 + 2 * i + 1 < p.N ? ap[1] : 0.f);
+  }
   if (threadIdx.x < kC) sd[threadIdx.x] = c0 + int(threadIdx.x) < p.inner ? p.d[c0 + threadIdx.x] : 0.f;
   pdl::grid_dependency_wait();
   const int* seg = p.segs + 4 * blockIdx.y;
@@ -224,7 +251,8 @@ __global__ void __launch_bounds__(128) k_selective_scan(const ScanParams p) {
   const T* xz = static_cast<const T*>(p.xz);
   float* sp = p.ssm + (size_t(slot) * p.inner + c) * p.N + n0;
 #pragma unroll
-  for (int i = 0; i < NPL; i++) s[i] = active && n0 + i < p.N && !fresh ? sp[i] : 0.f;
+  for (int i = 0; i < NQ; i++)
+    s[i] = pack2(active && n0 + 2 * i < p.N && !fresh ? sp[2 * i] : 0.f, active && n0 + 2 * i + 1 < p.N && !fresh ? sp[2 * i + 1] : 0.f);
 
   // raw values: nothing here depends on a load before the next tile is staged
   T ru[EX], rg[EX], zero;
@@ -274,7 +302,7 @@ __global__ void __launch_bounds__(128) k_selective_scan(const ScanParams p) {
         const float uv = to_f(ru[e]);
         sdx[cc][t] = dt * uv;
         su[t][cc] = uv;
-        sg[t][cc] = silu(to_f(rg[e]));
+        sg[t][cc] = gate<T>(to_f(rg[e]));
       }
     }
 #pragma unroll
@@ -295,24 +323,30 @@ __global__ void __launch_bounds__(128) k_selective_scan(const ScanParams p) {
         const float dts[4] = {dt4.x, dt4.y, dt4.z, dt4.w}, dxs[4] = {dx4.x, dx4.y, dx4.z, dx4.w};
 #pragma unroll
         for (int j = 0; j < 4; j++) {
-          float bv[NPL], cv[NPL];
-          if constexpr (NPL == 2) {
-            const float2 b2 = *reinterpret_cast<const float2*>(&sb[tb + q + j][n0]), c2 = *reinterpret_cast<const float2*>(&sc[tb + q + j][n0]);
-            bv[0] = b2.x; bv[1] = b2.y;
-            cv[0] = c2.x; cv[1] = c2.y;
-          } else
+          f32x2 bv[NQ], cv[NQ];
+          if constexpr (NQ == 1) {
+            bv[0] = *reinterpret_cast<const f32x2*>(&sb[tb + q + j][n0]);
+            cv[0] = *reinterpret_cast<const f32x2*>(&sc[tb + q + j][n0]);
+          } else {
 #pragma unroll
-          for (int i = 0; i < NPL; i += 4) {
-            const float4 b4 = *reinterpret_cast<const float4*>(&sb[tb + q + j][n0 + i]), c4 = *reinterpret_cast<const float4*>(&sc[tb + q + j][n0 + i]);
-            bv[i] = b4.x; bv[i + 1] = b4.y; bv[i + 2] = b4.z; bv[i + 3] = b4.w;
-            cv[i] = c4.x; cv[i + 1] = c4.y; cv[i + 2] = c4.z; cv[i + 3] = c4.w;
+            for (int i = 0; i < NQ; i += 2) {
+              const ulonglong2 b4 = *reinterpret_cast<const ulonglong2*>(&sb[tb + q + j][n0 + 2 * i]), c4 = *reinterpret_cast<const ulonglong2*>(&sc[tb + q + j][n0 + 2 * i]);
+              bv[i] = b4.x; bv[i + 1] = b4.y;
+              cv[i] = c4.x; cv[i + 1] = c4.y;
+            }
           }
-          float acc = 0.f;
+          const f32x2 dt2 = pack2(dts[j], dts[j]), dx2 = pack2(dxs[j], dxs[j]);
+          f32x2 acc2 = 0ull;
 #pragma unroll
-          for (int i = 0; i < NPL; i++) {
-            s[i] = fmaf(pow2<T>(dts[j] * a[i]), s[i], dxs[j] * bv[i]);
-            acc = fmaf(s[i], cv[i], acc);
+          for (int i = 0; i < NQ; i++) {
+            float e0, e1;
+            unpack2(mul2(dt2, a[i]), e0, e1);
+            s[i] = fma2(pack2(pow2<T>(e0), pow2<T>(e1)), s[i], mul2(dx2, bv[i]));
+            acc2 = i == 0 ? mul2(s[0], cv[0]) : fma2(s[i], cv[i], acc2);
           }
+          float acc, acc_hi;
+          unpack2(acc2, acc, acc_hi);
+          acc += acc_hi;
           y[q + j] = acc;
         }
       }
@@ -348,8 +382,12 @@ __global__ void __launch_bounds__(128) k_selective_scan(const ScanParams p) {
     po += size_t(TT) * p.ldo;
   }
 #pragma unroll
-  for (int i = 0; i < NPL; i++)
-    if (active && n0 + i < p.N) sp[i] = s[i];
+  for (int i = 0; i < NQ; i++) {
+    float lo, hi;
+    unpack2(s[i], lo, hi);
+    if (active && n0 + 2 * i < p.N) sp[2 * i] = lo;
+    if (active && n0 + 2 * i + 1 < p.N) sp[2 * i + 1] = hi;
+  }
   if (active && lane == 0) roll_conv_state(p, xz, first, count, slot, fresh, c);
 }
 
@@ -370,7 +408,11 @@ __global__ void __launch_bounds__(128) k_scan_step(const ScanParams p) {
   float* sp = p.ssm + (size_t(slot) * p.inner + c) * p.N + n0;
   const float* bc = p.bc + size_t(row) * p.ldbc + n0;
   const T* xz = static_cast<const T*>(p.xz);
-  float u = 0.f, dt = 0.f, z = 0.f;
+  float u = 0.f, dt = 0.f, z = 0.f, roll = 0.f;
+  // the convolution state moves up by one: lane k brings entry k + 1 (the last one: this token's input), all before any is stored
+  const bool by_lanes = p.taps - 1 <= LPC, mine = active && by_lanes && lane < p.taps - 1;
+  float* cs = p.conv_state + size_t(slot) * (p.taps - 1) * p.ldc + c;
+  if (mine) roll = lane + 1 < p.taps - 1 ? cs[size_t(lane + 1) * p.ldc] : to_f(xz[size_t(row) * p.ldxz + c]);
   if (active) {
     u = to_f(static_cast<const T*>(p.u)[size_t(row) * p.ldu + c]);
     dt = p.dt[size_t(row) * p.lddt + c];
@@ -393,10 +435,10 @@ __global__ void __launch_bounds__(128) k_scan_step(const ScanParams p) {
   }
 #pragma unroll
   for (int o = LPC / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-  if (active && lane == 0) {
-    from_f(static_cast<T*>(p.out)[size_t(row) * p.ldo + c], fmaf(d, u, y) * silu(z));
-    roll_conv_state(p, xz, row, 1, slot, fresh, c);
-  }
+  if (active && lane == 0) from_f(static_cast<T*>(p.out)[size_t(row) * p.ldo + c], fmaf(d, u, y) * gate<T>(z));
+  __syncwarp();
+  if (mine) cs[size_t(lane) * p.ldc] = fresh && lane + 1 < p.taps - 1 ? 0.f : roll;
+  if (active && lane == 0 && !by_lanes) roll_conv_state(p, xz, row, 1, slot, fresh, c);
 }
 
 template <typename T, int LPC, int NPL>

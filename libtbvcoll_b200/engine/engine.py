@@ -234,9 +234,9 @@ class Engine:
     def attn_splits_for(self, B: int, max_ctx: int) -> int:
         sms = torch.cuda.get_device_properties(self.device).multi_processor_count
         # kv splits are the CTAs of one cluster: the largest power of two (<= 8) that keeps the whole
-        # grid in one wave (two CTAs per SM) and leaves at least 64 cached tokens per CTA
+        # grid in one wave and leaves at least 64 cached tokens per CTA
         s = 1
-        while s < 8 and B * self.model.attn_ctas_per_row * s * 2 <= self.model.attn_ctas_per_sm * sms and max_ctx // (s * 2) >= 64:
+        while s < 8 and B * self.model.attn_ctas_per_row * s * 2 <= self.model.attn_cta_slots(s * 2, sms) and max_ctx // (s * 2) >= 64:
             s *= 2
         return min(s, self.model.max_attn_splits)
 

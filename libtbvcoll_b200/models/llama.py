@@ -34,7 +34,11 @@ from .config import ModelConfig
 class LlamaTP:
     rows_form_max = 0          # one attention form: rows of a step keep their order
     uses_state = False         # nothing is carried from token to token besides the KV cache
-    attn_ctas_per_sm = 2
+
+    @staticmethod
+    def attn_cta_slots(splits: int, sms: int) -> int:
+        """Attention CTAs that run at once (two per SM)."""
+        return 2 * sms
 
     def __init__(self, cfg: ModelConfig, tp: TPGroup, weights: Dict[str, torch.Tensor], device, max_tokens: int,
                  max_batch: int, num_blocks: int, block_size: int = 16, max_attn_splits: int = 32, dtype: torch.dtype = torch.bfloat16):

@@ -33,8 +33,11 @@ class Nubosun:
     # portions of at most this many tokens take the attention's rows form
     ROWS_FORM_MAX = 32
     uses_state = True
-    # one CTA of the rows kernel fills an SM, and clusters of eight find only about four fifths of the SMs (15 of them fit)
-    attn_ctas_per_sm = 0.8
+
+    @staticmethod
+    def attn_cta_slots(splits: int, sms: int) -> int:
+        """CTAs of the rows kernel that run at once: one per SM, but clusters of eight find only about four fifths of the SMs."""
+        return sms if splits < 8 else sms * 4 // 5
 
     def __init__(self, cfg: NubosunConfig, tp: TPGroup, weights: Dict[str, torch.Tensor], device, max_tokens: int, max_batch: int,
                  num_blocks: int, block_size: int = 16, max_attn_splits: int = 8, dtype: torch.dtype = torch.bfloat16):
