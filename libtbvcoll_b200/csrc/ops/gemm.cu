@@ -455,6 +455,8 @@ int tbv_op_gemm(const void* w, const void* x, void* y, const void* bias, int M, 
 // sigmoid.  groups > 1: w is [groups * M, K]; group g reads x columns g * x_group .. + K and writes y columns g * y_group .. .
 int tbv_op_gemm_ex(const void* w, const void* x, void* y, void* y2, const void* bias, int M, int N, int K, int ldx, int ldy, int epi,
                    int act, float act_a, float act_b, int groups, int x_group, int y_group, void* stream) {
+  const char* pf_ptr = nullptr;
+  const unsigned long long pf_bytes = tbvops::take_next_prefetch(&pf_ptr, (unsigned long long)(M > 0 ? M : 0) * (unsigned long long)(K > 0 ? K : 0) * 2ull);
   if (M <= 0 || N <= 0 || K <= 0 || (K % 8) || (ldx % 8) || (ldy % 8) || (reinterpret_cast<uintptr_t>(y) & 15u)) return -2;
   if (epi < 0 || epi > 3 || (epi == kEpiClampGlu && (M % 2)) || (y2 && (epi != kEpiF32 || (reinterpret_cast<uintptr_t>(y2) & 7u)))) return -2;
   if (groups > 1 && ((x_group % 8) || (y_group % 8) || bias)) return -2;
@@ -465,6 +467,8 @@ int tbv_op_gemm_ex(const void* w, const void* x, void* y, void* y2, const void* 
   else p.y = static_cast<__nv_bfloat16*>(y);
   p.y2 = static_cast<__nv_bfloat16*>(y2);
   p.act = act; p.act_a = act_a; p.act_b = act_b;
+  p.pf_ptr = pf_ptr;
+  p.pf_bytes = pf_bytes;
   p.groups = groups > 1 ? groups : 1; p.x_group = groups > 1 ? x_group : 0; p.y_group = groups > 1 ? y_group : 0;
   if (groups <= 1 && persist_mode() > 0 && !(reinterpret_cast<uintptr_t>(y) & 31u)) {   // its fp32 stores are 32 bytes wide
     const int th = tbvops::gemm_tok_choose(M, N, K, ldy, epi, persist_mode());

@@ -15,6 +15,7 @@ norm).  Between two of them:
 All buffers of a decode step are preallocated, so the step can be captured in a CUDA graph."""
 from __future__ import annotations
 
+import os
 from typing import Callable, Dict, Optional
 
 import torch
@@ -89,6 +90,7 @@ class Nubosun:
         two_forms = bool(latents) and dtype is torch.bfloat16 and all(ops.latent_prefill_fits(_pad16(m.dim), _pad16(m.rot_dim), _pad16(m.vdim)) for m in latents)
         self.rows_form_max = self.ROWS_FORM_MAX if two_forms else 1 << 60
         self._ctx_rows = 0
+        self.l2_prefetch = os.environ.get("TBV_L2_PREFETCH", "1") != "0"
 
     @staticmethod
     def load_weights(cfg: NubosunConfig, source, tp: TPGroup, device, dtype):
@@ -137,6 +139,7 @@ class Nubosun:
         ops.linear(low[:, :kd], w[p + "dt"], dt, bias=w[p + "dt.b"])
         ops.selective_scan(u, xz, ip, dt, proj, m.dt_rank, m.dt_rank + m.state, w[p + "a2"], w[p + "D"], self.ssm[run], self.conv[run], u, b.segs,
                            b.positions, one_token=b.seg_of_row is None)
+        self._announce_mlp(i, T)
         ops.linear(u, w[p + "o"], y)
 
     def _latent(self, b: StepBatch, run: int, i: int, m: LatentSpec, h, y) -> None:
@@ -162,7 +165,13 @@ class Nubosun:
             ops.latent_gather(cache, b.dense_slots, c, kr)
             ops.linear(c, w[p + "wukv"], kv)
             ops.latent_attention_prefill(qkv, q_rot, kv, kr, b.dense_tiles, w[p + "sink"], out, H, D, V, m.scale)
+        self._announce_mlp(i, T)
         ops.linear(out, w[p + "o"], y)
+
+    def _announce_mlp(self, i: int, T: int) -> None:
+        """Decode: the out-projection asks for the gate / up weights that follow it (ops.prefetch_next)."""
+        if self.l2_prefetch and T <= 64 and self.cfg.layers[i].mlp is not None and self.dtype is torch.bfloat16:
+            ops.prefetch_next(self.w[f"l{i}.mlp.gate_up"])
 
     def _mlp(self, b: StepBatch, i: int, m, h, y) -> None:
         p = f"l{i}.mlp."

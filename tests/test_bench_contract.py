@@ -20,7 +20,7 @@ def test_reference_arm_prints_unavailable_and_exits_zero():
 def test_help_lists_the_driver_flags():
     r = subprocess.run([sys.executable, os.path.join(ROOT, "bench.py"), "--help"], capture_output=True, text=True, timeout=300, cwd=ROOT)
     assert r.returncode == 0
-    for flag in ("--gpus", "--steps", "--warmup", "--impl"):
+    for flag in ("--gpus", "--steps", "--warmup", "--impl", "--compare"):
         assert flag in r.stdout
 
 
