@@ -64,8 +64,8 @@ def _compile(src: Path, force: bool, verbose: bool, hdr_m: float, bounds: bool =
     return obj, p.stderr if verbose else ""
 
 
-def build(force: bool = False, verbose: bool = False) -> Path:
-    """Compile and link; returns the path of the shared object."""
+def build(force: bool = False, verbose: bool = False, executables: bool = True) -> Path:
+    """Compile and link; returns the path of the shared object.  ``executables=False`` leaves out the standalone programs."""
     OBJ.mkdir(exist_ok=True)
     srcs = lib_sources()
     hdr_m = _headers_mtime()
@@ -81,7 +81,7 @@ def build(force: bool = False, verbose: bool = False) -> Path:
         _link(LIB, objs)
     # standalone microbenchmark executable (counterpart of the reference's ar2/armr binaries)
     proto = CSRC / "proto" / "arbench.cu"
-    if proto.exists() and (force or not AR_BENCH.exists() or AR_BENCH.stat().st_mtime < max(proto.stat().st_mtime, LIB.stat().st_mtime)):
+    if executables and proto.exists() and (force or not AR_BENCH.exists() or AR_BENCH.stat().st_mtime < max(proto.stat().st_mtime, LIB.stat().st_mtime)):
         cmd = [nvcc(), *ARCH, *COMMON, str(proto), "-o", str(AR_BENCH), f"-L{PKG}", "-ltbvcoll",
                "-Xlinker", "-rpath,$ORIGIN"]
         p = subprocess.run(cmd, capture_output=True, text=True)
@@ -126,7 +126,7 @@ def ensure_built() -> Path:
     except OSError:
         if LIB.exists():
             return LIB
-    return build()
+    return build(executables=False)
 
 
 if __name__ == "__main__":

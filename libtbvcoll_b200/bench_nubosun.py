@@ -73,7 +73,8 @@ def model_numbers(name: str, batches=(1, 8, 32), prompt: int = 512, long_prompt:
 
 # ---- kernel by kernel -------------------------------------------------------------------------------------------------------
 class _Kernels:
-    def __init__(self):
+    def __init__(self, only: str = ""):
+        self.only = only
         from .bench_ops import peaks
         self.hbm, self.tf, self.src = peaks()
         self.rows = []
@@ -81,6 +82,8 @@ class _Kernels:
 
     def time(self, group: str, name: str, make, bytes_, flops=0.0, exps=0.0):
         """make(i) -> callable on the i-th set of operands; sets are made until they exceed the L2."""
+        if self.only not in name:
+            return
         from .bench_ops import time_graph
         torch.cuda.empty_cache()
         sets = max(2, min(64, math.ceil(400e6 / max(bytes_, 1.0))))
@@ -110,7 +113,7 @@ def _linear(k: _Kernels, group, name, T, M, K, f32=False, glu=None, act=0, copy=
     k.time(group, name, make, T * groups * K * 2 + groups * M * K * 2 + out_bytes, 2.0 * T * groups * M * K)
 
 
-def kernel_numbers(size: str, T: int, seqs: int, ctx: int) -> list:
+def kernel_numbers(size: str, T: int, seqs: int, ctx: int, only: str = "") -> list:
     """T rows in ``seqs`` sequences: T == seqs is a decode step over ``ctx`` cached tokens, otherwise whole prompts."""
     from . import ops
     from .engine.batch import dense_context
@@ -120,7 +123,7 @@ def kernel_numbers(size: str, T: int, seqs: int, ctx: int) -> list:
     nb, ll = (get_config(n) for n in PAIRS[size])
     m = next(l.mixer for l in nb.layers if isinstance(l.mixer, MambaSpec))
     a = next(l.mixer for l in nb.layers if isinstance(l.mixer, LatentSpec))
-    k, W, S, dev = _Kernels(), nb.hidden_size, nb.streams, "cuda"
+    k, W, S, dev = _Kernels(only), nb.hidden_size, nb.streams, "cuda"
     decode = T == seqs
     L = T // seqs
     bf, f32, i32 = torch.bfloat16, torch.float32, torch.int32
@@ -253,16 +256,19 @@ def kernel_numbers(size: str, T: int, seqs: int, ctx: int) -> list:
     return k.rows
 
 
-def run(sizes, kernels=True, models=True) -> dict:
+CASES = {"decode 8 rows, 640 cached tokens": (8, 8, 640), "decode 32 rows, 640 cached tokens": (32, 32, 640),
+         "decode 32 rows, 8192 cached tokens": (32, 32, 8192),
+         "prefill 8 x 512": (4096, 8, 512), "prefill 1 x 4096": (4096, 1, 4096)}
+
+
+def run(sizes, kernels=True, models=True, only="", case="") -> dict:
     out = {"bench": "nubosun beside llama", "data": "synthetic (random token ids, random weights)", "dtype": "bf16", "sizes": {}}
     for s in sizes:
         r = out["sizes"][s] = {}
         if models:
             r["models"] = [model_numbers(n) for n in PAIRS[s]]
         if kernels:
-            r["kernels"] = {"decode 8 rows, 640 cached tokens": kernel_numbers(s, 8, 8, 640),
-                            "decode 32 rows, 640 cached tokens": kernel_numbers(s, 32, 32, 640),
-                            "prefill 8 x 512": kernel_numbers(s, 4096, 8, 512), "prefill 1 x 4096": kernel_numbers(s, 4096, 1, 4096)}
+            r["kernels"] = {c: kernel_numbers(s, *v, only=only) for c, v in CASES.items() if case in c}
     return out
 
 
@@ -271,9 +277,11 @@ def main() -> int:
     ap.add_argument("--sizes", default="2k,8b")
     ap.add_argument("--no-kernels", action="store_true")
     ap.add_argument("--no-models", action="store_true")
+    ap.add_argument("--only", default="", help="kernels whose name contains this")
+    ap.add_argument("--case", default="", help="cases whose name contains this")
     ap.add_argument("--table", action="store_true", help="print kernel rows as text")
     a = ap.parse_args()
-    r = run(a.sizes.split(","), not a.no_kernels, not a.no_models)
+    r = run(a.sizes.split(","), not a.no_kernels, not a.no_models, a.only, a.case)
     if a.table:
         for s, v in r["sizes"].items():
             for m in v.get("models", []):

@@ -94,8 +94,8 @@ def test_padded_weights_compute_the_same_products(name):
 
 def test_rotation_frequencies():
     from libtbvcoll_b200.ops import rope_frequencies
-    for dims, base, sc in ((32, 1e4, None), (64, 5e5, {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}),
-                           (10, 1e4, cases.YARN), (2, 100.0, cases.YARN), (48, 1e6, {"factor": 40.0, "original": 128, "fast": 1.0, "slow": 1.0})):
+    for dims, base, sc in ((36, 1e4, None), (64, 5e5, {"factor": 6.0, "original": 4096, "fast": 30.0, "slow": 1.0}),
+                           (10, 1e4, cases.YARN), (2, 100.0, cases.YARN), (48, 2e6, {"factor": 40.0, "original": 128, "fast": 1.0, "slow": 1.0})):
         f, factor = rope_frequencies(dims, base, sc)
         want, wf = oracle.rotary_frequencies({"dims": dims, "base": base, "scaling": sc})
         assert np.allclose(f.numpy(), want, rtol=1e-12) and abs(factor - wf) < 1e-12
