@@ -229,9 +229,10 @@ __device__ __forceinline__ void cluster_sync() {
   asm volatile("barrier.cluster.arrive.release.aligned;\nbarrier.cluster.wait.acquire.aligned;" ::: "memory");
 }
 
-// bf16: 16 heads of one row per CTA on tensor cores.  Eight warps share tiles of TT cached tokens (two stages filled by bulk copies): for the scores warp w takes tokens 8w.. of the tile over all Dk
-// columns; for the weighted sum it takes the latent columns of the 16-column blocks w, w + 8, .. (CBW of them).  grid (rows, head tiles,
-// splits), cluster (1, 1, splits): the CTAs of a cluster cover disjoint token ranges and merge in split order.
+// bf16: 16 heads of one row per CTA on tensor cores.  Eight warps share tiles of TT cached tokens that a ninth brings into two stages by
+// bulk copies.  Scores: warp w takes tokens 8w.. of the tile over all Dk columns.  Weighted sum: it takes the latent columns of the
+// 16-column blocks w, w + 8, .. (CBW of them).  grid (rows, head tiles, splits), cluster (1, 1, splits): the CTAs of a cluster cover
+// disjoint token ranges and merge in split order.
 constexpr int kRW = 8;
 constexpr int kMaxSplits = 8;
 template <int CBW, int TT>
@@ -267,9 +268,10 @@ __global__ void __launch_bounds__(kRW * 32 + 32, 1) k_latent_rows_mma(const Rows
   const int nq = min(16, p.heads - h0);
   for (int r = nq + warp; r < 16; r += kRW + 1)
     for (int c = lane; c < chunks; c += 32) st_zero16(sq + r * pitch + c * 16);
-  // The ninth warp brings the tiles in.  Tile i: it asks for the tokens, a block (or the part of one inside the tile) per copy, and for the query rows with tile 0.  A
-  // partial tile ends at a multiple of 16 tokens, its missing rows are zeros, so that a weight of zero meets no stale bit pattern.  Table entries are looked up a
-  // tile ahead of their use: table and cache are two memory round trips, and both would otherwise stand between two tiles.
+  // The ninth warp brings the tiles in.  Tile i: its tokens, a block (or the part of one inside the tile) per copy, and the query rows
+  // with tile 0.  A partial tile ends at a multiple of 16 tokens; its missing rows are zeros, so that a weight of zero meets no stale
+  // bit pattern.  Table entries are looked up a tile ahead of their use: table and cache are two memory round trips, and both would
+  // otherwise stand between two tiles.
   const int bs = p.block_size;
   auto look_up = [&](int i) {
     const int pg = (t0 + i * TT) / bs + lane;
