@@ -5,6 +5,7 @@ GQA, SiLU-gated MLP); Qwen2 adds a bias on the q/k/v projections."""
 from __future__ import annotations
 
 import json
+import math
 from dataclasses import dataclass, field
 from typing import List, Optional, Union
 
@@ -209,7 +210,153 @@ def nubosun_like(hidden: int, layers: int, ff: int, heads: int, vocab: int, head
     return NubosunConfig(name=name, vocab_size=vocab, hidden_size=hidden, layers=lay, streams=streams, logit_softcap=30.0)
 
 
+# ---- Tinapel: gated linear attention, WKV and key-as-value attention beside mixtures of experts ------------------------------
+@dataclass
+class GlaSpec:
+    heads: int
+    dim: int                               # key channels per head
+    vdim: int
+    tau: float                             # decay = sigmoid(z)^(1 / tau)
+    decay_rank: Optional[int] = None       # of the low-rank decay projection; None: the checkpoint's tensors tell
+
+
+@dataclass
+class WkvSpec:
+    heads: int
+    dim: int                               # key and value channels per head
+    decay_rank: Optional[int] = None
+
+
+@dataclass
+class SharedKvSpec:
+    """Attention whose values are the keys before their norm: one cached row per token and key head serves as both."""
+    heads: int
+    kv_heads: int
+    dim: int
+    scale: float
+    softcap: Optional[float] = None
+    temp_coef: float = 0.0                 # query factor at position p: 1 + coef * ln(floor((p + 1) / every) + 1)
+    temp_every: float = 1.0
+
+
+@dataclass
+class MoeSpec:
+    experts: int
+    top: int
+    ff: int                                # of an expert
+    scale: float = 1.0                     # on the normalised weights of the chosen experts
+    shared_ff: Optional[int] = None        # of the expert that every token uses
+
+
+@dataclass
+class ParallelLayerSpec:
+    mixer: Union[GlaSpec, WkvSpec, SharedKvSpec]
+    mlp: Optional[MoeSpec] = None
+
+
+@dataclass
+class LoopSpec:
+    start: int
+    stop: int
+    times: int
+
+
+@dataclass
+class TinapelConfig:
+    name: str
+    vocab_size: int
+    hidden_size: int
+    layers: List[ParallelLayerSpec]
+    embedding_scale: float = 1.0
+    rms_eps: float = 1e-6
+    loop: Optional[LoopSpec] = None
+
+    def __post_init__(self):
+        lp = self.loop
+        if lp is not None and not (0 <= lp.start < lp.stop <= len(self.layers) and lp.times >= 0):
+            raise ValueError(f"loop {lp} does not fit {len(self.layers)} layers")
+        for i, lay in enumerate(self.layers):
+            m = lay.mixer
+            if isinstance(m, SharedKvSpec) and m.heads % m.kv_heads:
+                raise ValueError(f"layer {i}: {m.heads} query heads on {m.kv_heads} key heads")
+            if lay.mlp is not None and not 1 <= lay.mlp.top <= lay.mlp.experts:
+                raise ValueError(f"layer {i}: {lay.mlp.top} of {lay.mlp.experts} experts")
+
+    def check_tp(self, tp: int) -> None:
+        if tp != 1:
+            raise ValueError("Tinapel models run on one GPU (no tensor-parallel sharding of the recurrent states and the shared cache rows)")
+
+    @property
+    def schedule(self) -> List[tuple]:
+        """(layer, pass) of every layer run in order; pass = number of the loop's pass that begins right before this run, else None."""
+        n, lp = len(self.layers), self.loop
+        if lp is None:
+            return [(i, None) for i in range(n)]
+        out = [(i, None) for i in range(lp.start)]
+        for t in range(lp.times):
+            out += [(i, t if i == lp.start else None) for i in range(lp.start, lp.stop)]
+        return out + [(i, None) for i in range(lp.stop, n)]
+
+    @property
+    def runs(self) -> List[int]:
+        return [i for i, _ in self.schedule]
+
+    @property
+    def num_layers(self) -> int:
+        return len(self.schedule)
+
+    def param_count(self) -> int:
+        from ..utils.weights import tensor_shapes
+        return sum(math.prod(s) for s in tensor_shapes(self).values())
+
+
+def _parse_moe(i: int, c: Optional[dict]) -> Optional[MoeSpec]:
+    if c is None:
+        return None
+    if c.get("kind") != "moe":
+        raise ValueError(f"layer {i}: unknown feed-forward {c.get('kind')!r}")
+    r, shared = c["router"], c.get("shared")
+    return MoeSpec(experts=r["experts"], top=r["top"], ff=c["expert"]["ff"], scale=float(r.get("scale", 1.0)), shared_ff=shared["ff"] if shared else None)
+
+
+def parse_tinapel_config(c: dict) -> TinapelConfig:
+    """``config.json`` of a Tinapel checkpoint."""
+    layers = []
+    for i, e in enumerate(c["layers"]):
+        m = e["mixer"]
+        if e["type"] == "gla":
+            mixer = GlaSpec(heads=m["heads"], dim=m["dim"], vdim=m["vdim"], tau=float(m["tau"]))
+        elif e["type"] == "wkv":
+            mixer = WkvSpec(heads=m["heads"], dim=m["dim"])
+        elif e["type"] == "attention":
+            if m.get("vdim", m["dim"]) != m["dim"]:
+                raise ValueError(f"layer {i}: values are keys, but have {m['vdim']} channels of {m['dim']}")
+            temp, cap = m.get("q_temp"), m.get("softcap")
+            mixer = SharedKvSpec(heads=m["heads"], kv_heads=m.get("kv_heads", m["heads"]), dim=m["dim"], scale=float(m["scale"]),
+                                 softcap=float(cap) if cap else None, temp_coef=float(temp["coef"]) if temp else 0.0,
+                                 temp_every=float(temp["every"]) if temp else 1.0)
+        else:
+            raise ValueError(f"layer {i}: unknown type {e['type']!r}")
+        layers.append(ParallelLayerSpec(mixer, _parse_moe(i, e.get("mlp"))))
+    lp = c.get("loop")
+    return TinapelConfig(name=c.get("name", "tinapel"), vocab_size=c["vocab"], hidden_size=c["width"], layers=layers,
+                         embedding_scale=float(c.get("embedding", {}).get("scale", 1.0)), rms_eps=float(c["norm"]["eps"]),
+                         loop=LoopSpec(lp["start"], lp["stop"], lp["times"]) if lp and lp["stop"] > lp["start"] else None)
+
+
+def tinapel_like(hidden: int, layers: int, ff: int, heads: int, kv_heads: int, vocab: int, head_dim: int = 128, experts: int = 8, top: int = 2,
+                 name: str = "tinapel") -> TinapelConfig:
+    """A Tinapel of ordinary proportions: layers in turn gated linear attention, WKV and attention; a token uses a shared expert of half of
+    ``ff`` and ``top`` experts that make up the other half, so that it meets as many feed-forward weights as in a dense model of ``ff``."""
+    kinds = (lambda: GlaSpec(heads=heads, dim=head_dim, vdim=head_dim, tau=16.0, decay_rank=64), lambda: WkvSpec(heads=heads, dim=head_dim, decay_rank=64),
+             lambda: SharedKvSpec(heads=heads, kv_heads=kv_heads, dim=head_dim, scale=head_dim ** -0.5, softcap=50.0, temp_coef=0.1, temp_every=4096))
+    lay = [ParallelLayerSpec(kinds[i % 3](), MoeSpec(experts=experts, top=top, ff=ff // (2 * top), scale=1.0, shared_ff=ff // 2)) for i in range(layers)]
+    return TinapelConfig(name=name, vocab_size=vocab, hidden_size=hidden, layers=lay)
+
+
 PRESETS["nubosun-8b"] = nubosun_like(4096, 32, 14336, 32, 128256, name="nubosun-8b")
 PRESETS["nubosun-2k"] = nubosun_like(2048, 16, 7168, 16, 32768, name="nubosun-2k")
 PRESETS["llama3-2k"] = ModelConfig(name="llama3-2k", hidden_size=2048, num_layers=16, num_heads=16, num_kv_heads=4, intermediate_size=7168,
                                    vocab_size=32768)
+PRESETS["tinapel-8b"] = tinapel_like(4096, 32, 14336, 32, 8, 128256, name="tinapel-8b")
+PRESETS["tinapel-2k"] = tinapel_like(2048, 16, 7168, 16, 4, 32768, name="tinapel-2k")

@@ -7,7 +7,7 @@ import os
 from dataclasses import dataclass
 from typing import Callable, Tuple
 
-from .config import ModelConfig, NubosunConfig, from_hf_config, parse_nubosun_config
+from .config import ModelConfig, NubosunConfig, TinapelConfig, from_hf_config, parse_nubosun_config, parse_tinapel_config
 
 
 @dataclass(frozen=True)
@@ -29,9 +29,15 @@ def _nubosun():
     return Nubosun
 
 
+def _tinapel():
+    from .tinapel import Tinapel
+    return Tinapel
+
+
 ARCHITECTURES = {
     "llama": Architecture("llama", ModelConfig, _llama, ("bfloat16",), True),
     "nubosun": Architecture("nubosun", NubosunConfig, _nubosun, ("bfloat16", "float32"), False),
+    "tinapel": Architecture("tinapel", TinapelConfig, _tinapel, ("bfloat16", "float32"), False),
 }
 
 
@@ -50,6 +56,8 @@ def load_config(model_dir: str):
     arch = str(c.get("architecture", "")).lower()
     if arch == "nubosun":
         return parse_nubosun_config(c)
+    if arch == "tinapel":
+        return parse_tinapel_config(c)
     if arch:
         raise ValueError(f"unknown architecture {c['architecture']!r}")
     return from_hf_config(path)            # Llama / Qwen2 families in the HF layout

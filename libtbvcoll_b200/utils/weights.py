@@ -17,7 +17,7 @@ from typing import Callable, Dict, Iterable, Optional
 
 import torch
 
-from ..models.config import LatentSpec, MambaSpec, ModelConfig, NubosunConfig
+from ..models.config import GlaSpec, LatentSpec, MambaSpec, ModelConfig, NubosunConfig, TinapelConfig, WkvSpec
 
 
 def hf_tensor_shapes(cfg: ModelConfig) -> Dict[str, tuple]:
@@ -65,9 +65,64 @@ def nubosun_tensor_shapes(cfg: NubosunConfig) -> Dict[str, tuple]:
     return shapes
 
 
+def tinapel_tensor_shapes(cfg: TinapelConfig) -> Dict[str, tuple]:
+    """A decay rank that the configuration leaves open is 16 here; in a checkpoint its tensors tell."""
+    W = cfg.hidden_size
+    shapes = {"embed": (cfg.vocab_size, W), "final.norm": (W,)}
+    if cfg.loop is not None:
+        shapes["loop.step"] = (cfg.loop.times, W)
+    for i, lay in enumerate(cfg.layers):
+        p, m, f = f"l{i}.", lay.mixer, lay.mlp
+        shapes[p + "norm1"] = (W,)
+        x = p + "mix."
+        if isinstance(m, GlaSpec):
+            K, V, R = m.heads * m.dim, m.heads * m.vdim, m.decay_rank or 16
+            shapes.update({x + "q": (K, W), x + "k": (K, W), x + "v": (V, W), x + "g": (V, W), x + "o": (W, V), x + "norm": (m.vdim,), x + "a1": (R, W),
+                           x + "a2": (K, R), x + "a2.b": (K,)})
+        elif isinstance(m, WkvSpec):
+            K, R = m.heads * m.dim, m.decay_rank or 16
+            shapes.update({x + "mu." + s: (W,) for s in "rkvgw"})
+            shapes.update({x + s: (K, W) for s in "rkvg"})
+            shapes.update({x + "w1": (R, W), x + "w2": (K, R), x + "w0": (K,), x + "u": (m.heads, m.dim), x + "norm": (K,), x + "o": (W, K)})
+        else:
+            shapes.update({x + "q": (m.heads * m.dim, W), x + "k": (m.kv_heads * m.dim, W), x + "q.norm": (m.dim,), x + "k.norm": (m.dim,),
+                           x + "o": (W, m.heads * m.dim)})
+        if f is not None:
+            shapes[p + "norm2"] = (W,)
+            shapes[p + "mlp.router"] = (f.experts, W)
+            ffs = {f"e{e}.": f.ff for e in range(f.experts)}
+            if f.shared_ff:
+                ffs["shared."] = f.shared_ff
+            for e, n in ffs.items():
+                shapes.update({p + "mlp." + e + "gate": (n, W), p + "mlp." + e + "up": (n, W), p + "mlp." + e + "down": (W, n)})
+    return shapes
+
+
 def tensor_shapes(cfg) -> Dict[str, tuple]:
     """Checkpoint tensor names and shapes of a configuration of any architecture."""
-    return nubosun_tensor_shapes(cfg) if isinstance(cfg, NubosunConfig) else hf_tensor_shapes(cfg)
+    for kind, shapes in ((NubosunConfig, nubosun_tensor_shapes), (TinapelConfig, tinapel_tensor_shapes)):
+        if isinstance(cfg, kind):
+            return shapes(cfg)
+    return hf_tensor_shapes(cfg)
+
+
+def _tinapel_random(name: str, shape: tuple, g: torch.Generator, device) -> torch.Tensor:
+    """Random values that keep a Tinapel's activations near unit size: decays over many time scales, norms near one."""
+    leaf = name.split(".", 1)[1] if name.startswith("l") and "." in name else name
+    n = lambda: torch.randn(shape, generator=g, device=device, dtype=torch.float32)
+    if leaf in ("norm1", "norm2", "final.norm"):
+        return 0.1 * n()                              # norms are stored around zero
+    if leaf in ("mix.norm", "mix.q.norm", "mix.k.norm"):
+        return 1.0 + 0.1 * n()
+    if leaf.startswith("mix.mu."):
+        return torch.rand(shape, generator=g, device=device, dtype=torch.float32)
+    if leaf == "mix.w0":
+        return -3.0 + 1.5 * n()                       # decays exp(-exp(.)): memories of a few to a few hundred tokens
+    if leaf == "mix.a2.b":
+        return 1.0 + n()
+    if leaf in ("mix.u", "step"):
+        return 0.3 * n()
+    return n() if leaf == "embed" else n() / shape[1] ** 0.5
 
 
 def _nubosun_random(name: str, shape: tuple, g: torch.Generator, device) -> torch.Tensor:
@@ -114,6 +169,8 @@ class RandomSource:
         g = torch.Generator(device=self.device).manual_seed((self.seed * 1000003 + zlib.crc32(name.encode())) & 0x7FFFFFFF)
         if isinstance(self.cfg, NubosunConfig):
             t = _nubosun_random(name, shape, g, self.device)
+        elif isinstance(self.cfg, TinapelConfig):
+            t = _tinapel_random(name, shape, g, self.device)
         elif name.endswith("layernorm.weight") or name.endswith("norm.weight"):
             t = 1.0 + 0.1 * torch.randn(shape, generator=g, device=self.device, dtype=torch.float32)
         elif name.endswith(".bias"):
@@ -279,6 +336,98 @@ def load_nubosun(cfg: NubosunConfig, source, device, dtype=torch.bfloat16) -> Di
             g, u = _padded(get(x + "gate"), fp, Wp), _padded(get(x + "up"), fp, Wp)
             put(x + "gate_up", torch.stack((g, u), 1).reshape(2 * fp, Wp))
             put(x + "down", _padded(get(x + "down"), Wp, fp))
+    return out
+
+
+def load_tinapel(cfg: TinapelConfig, source, device, dtype=torch.bfloat16) -> Dict[str, torch.Tensor]:
+    """Tensors the way the kernels consume them; dimensions of matrix products and heads are zero-padded to multiples of 16, parameters that
+    act in 32-bit are fp32.
+
+    ``embed`` serves as the head too (rows padded).  GLA: ``in`` stacks q, k, v, g and the first decay projection.  WKV: ``in`` stacks r, k, v,
+    g and the first decay projection, each for a mix of its own; ``mu`` [5, width] in the same order.  Attention: ``in`` stacks q and k; ``fold`` =
+    query norm * key norm * scale (what is left of a key is one factor per token).  Experts: ``gate_up`` [experts * 2 ff, width], rows
+    interleaved, and ``down`` [experts * width, ff].  Norm weights hold 1 + w."""
+    dev, out, f32 = torch.device(device), {}, torch.float32
+    W, Wp = cfg.hidden_size, _pad16(cfg.hidden_size)
+    want = tinapel_tensor_shapes(cfg)
+
+    def get(name, open_dim=None):
+        t = source.get(name)
+        shape = list(want[name])
+        if open_dim is not None:
+            shape[open_dim] = t.shape[open_dim]
+        if list(t.shape) != shape:
+            raise ValueError(f"{name}: shape {tuple(t.shape)}, expected {tuple(shape)}")
+        return t
+
+    def put(name, t, as_dtype=dtype):
+        out[name] = t.to(as_dtype).to(dev).contiguous()
+
+    def heads_padded(t, heads, dim):          # [heads * dim, K] -> [heads * pad16(dim), Wp or K]
+        return _pad_heads(t, heads, dim, _pad16(dim))
+
+    def vector(t, heads, dim):                # [heads * dim] -> [heads * pad16(dim)]
+        return _pad_heads(t.reshape(-1, 1), heads, dim, _pad16(dim)).reshape(-1)
+
+    def out_proj(t, heads, dim):              # [W, heads * dim] -> [Wp, heads * pad16(dim)]
+        return _padded(_pad_heads(t.t(), heads, dim, _pad16(dim)).t(), Wp, heads * _pad16(dim))
+
+    def gate_up(gate, up, ff):
+        fp = _pad16(ff)
+        return torch.stack((_padded(gate, fp, Wp), _padded(up, fp, Wp)), 1).reshape(2 * fp, Wp)
+
+    put("embed", _padded(get("embed"), _pad16(cfg.vocab_size), Wp))
+    put("final.norm", _padded(1.0 + get("final.norm").float(), Wp), f32)
+    if cfg.loop is not None:
+        put("loop.step", _padded(get("loop.step"), cfg.loop.times, Wp), f32)
+    for i, lay in enumerate(cfg.layers):
+        p, m, f = f"l{i}.", lay.mixer, lay.mlp
+        x = p + "mix."
+        put(p + "norm1", _padded(1.0 + get(p + "norm1").float(), Wp), f32)
+        if isinstance(m, GlaSpec):
+            H, D, V = m.heads, m.dim, m.vdim
+            a1 = get(x + "a1", 0)
+            R = _pad16(a1.shape[0])
+            rows = torch.cat((heads_padded(get(x + "q"), H, D), heads_padded(get(x + "k"), H, D), heads_padded(get(x + "v"), H, V),
+                              heads_padded(get(x + "g"), H, V), _padded(a1, R, W)))
+            put(x + "in", _padded(rows, rows.shape[0], Wp))
+            put(x + "decay", _padded(heads_padded(get(x + "a2", 1), H, D), H * _pad16(D), R))
+            put(x + "decay.b", vector(get(x + "a2.b"), H, D))
+            put(x + "norm", vector(get(x + "norm").repeat(H), H, V), f32)
+            put(x + "o", out_proj(get(x + "o"), H, V))
+        elif isinstance(m, WkvSpec):
+            H, D = m.heads, m.dim
+            w1 = get(x + "w1", 0)
+            R = _pad16(w1.shape[0])
+            rows = torch.cat([heads_padded(get(x + s), H, D) for s in "rkvg"] + [_padded(w1, R, W)])
+            put(x + "in", _padded(rows, rows.shape[0], Wp))
+            put(x + "mu", torch.stack([_padded(get(x + "mu." + s), Wp) for s in "rkvgw"]), f32)
+            put(x + "decay", _padded(heads_padded(get(x + "w2", 1), H, D), H * _pad16(D), R))
+            put(x + "decay.b", vector(get(x + "w0"), H, D))
+            put(x + "u", vector(get(x + "u").reshape(-1), H, D), f32)
+            put(x + "norm", vector(get(x + "norm"), H, D), f32)
+            put(x + "o", out_proj(get(x + "o"), H, D))
+        else:
+            H, G, D = m.heads, m.kv_heads, m.dim
+            rows = torch.cat((heads_padded(get(x + "q"), H, D), heads_padded(get(x + "k"), G, D)))
+            put(x + "in", _padded(rows, rows.shape[0], Wp))
+            put(x + "fold", _padded(get(x + "q.norm").float() * get(x + "k.norm").float() * m.scale, _pad16(D)), f32)
+            put(x + "o", out_proj(get(x + "o"), H, D))
+        if f is not None:
+            x = p + "mlp."
+            put(p + "norm2", _padded(1.0 + get(p + "norm2").float(), Wp), f32)
+            put(x + "router", _padded(get(x + "router"), _pad16(f.experts), Wp))
+            fp = _pad16(f.ff)
+            gu = torch.empty(f.experts * 2 * fp, Wp, dtype=dtype, device=dev)
+            down = torch.empty(f.experts * Wp, fp, dtype=dtype, device=dev)
+            for e in range(f.experts):
+                q = f"{x}e{e}."
+                gu[e * 2 * fp: (e + 1) * 2 * fp] = gate_up(get(q + "gate"), get(q + "up"), f.ff)
+                down[e * Wp: (e + 1) * Wp] = _padded(get(q + "down"), Wp, fp)
+            out[x + "gate_up"], out[x + "down"] = gu, down
+            if f.shared_ff:
+                put(x + "shared.gate_up", gate_up(get(x + "shared.gate"), get(x + "shared.up"), f.shared_ff))
+                put(x + "shared.down", _padded(get(x + "shared.down"), Wp, _pad16(f.shared_ff)))
     return out
 
 
