@@ -42,15 +42,15 @@ __device__ __forceinline__ float silu_mul_bf16(float g, float u) {
 template <>
 __device__ __forceinline__ float glu_pair<kEpiSiluMul>(const Params& p, float g, float u) { return silu_mul_bf16(g, u); }
 template <>
-__device__ __forceinline__ float glu_pair<kEpiClampGlu>(const Params& p, float g, float u) { return gemm::clamp_glu(g, u, p.act_a, p.act_b); }
+__device__ __forceinline__ float glu_pair<kEpiClampGlu>(const Params& p, float g, float u) { return gemm::clamp_glu(g, u, p.act_a, p.act_b, p.act_c); }
 
 // four consecutive fp32 features of one token: activation, store, optional bf16 copy
-__device__ __forceinline__ void store_f32x4(const Params& p, size_t off, int m, float4 v) {
+__device__ __forceinline__ void store_f32x4(const Params& p, int M, size_t off, int m, float4 v) {
   v.x = gemm::apply_act(v.x, p.act, p.act_a);
   v.y = gemm::apply_act(v.y, p.act, p.act_a);
   v.z = gemm::apply_act(v.z, p.act, p.act_a);
   v.w = gemm::apply_act(v.w, p.act, p.act_a);
-  if (m + 4 <= p.M) {
+  if (m + 4 <= M) {
     *reinterpret_cast<float4*>(p.yf + off) = v;
     if (p.y2) {
       __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
@@ -61,7 +61,7 @@ __device__ __forceinline__ void store_f32x4(const Params& p, size_t off, int m, 
     }
   } else {
     const float a4[4] = {v.x, v.y, v.z, v.w};
-    for (int e = 0; e < 4 && m + e < p.M; e++) {
+    for (int e = 0; e < 4 && m + e < M; e++) {
       p.yf[off + e] = a4[e];
       if (p.y2) p.y2[off + e] = __float2bfloat16_rn(a4[e]);
     }
@@ -78,12 +78,20 @@ k_gemm(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensor
   // must run together, so that the weights stream from HBM once and the activations stay in L2.
   constexpr bool kGlu = EPI == kEpiSiluMul || EPI == kEpiClampGlu;
   int m0 = (p.raster ? blockIdx.y : blockIdx.x) * gemm::kBM;
-  const int n0 = (p.raster ? blockIdx.x : blockIdx.y) * p.bn;
+  int n0 = (p.raster ? blockIdx.x : blockIdx.y) * p.bn, M = p.M, nend = p.N;
   int grp = 0;                                   // group of a grouped problem; m0 becomes the feature inside the group
-  if (p.groups > 1) {
+  if (p.groups > 1 || p.m_last) {
     const int mt = (p.M + gemm::kBM - 1) / gemm::kBM;
     grp = (m0 / gemm::kBM) / mt;
+    if (p.m_last && grp >= p.groups) { grp = p.groups; M = p.m_last; }
     m0 -= grp * mt * gemm::kBM;
+  }
+  if (p.row_off) {                               // rows of this group; CTAs (whole clusters) beyond them have nothing to do
+    pdl::grid_dependency_wait();
+    const int first = p.row_off[grp], end = p.row_off[grp + 1];
+    if (n0 >= end - first) return;
+    n0 += first;
+    nend = end;
   }
   const size_t ycol = size_t(grp) * p.y_group;
   const int S = p.splits;
@@ -95,7 +103,7 @@ k_gemm(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensor
 
   uint8_t* sm = gemm::mainloop(&tmA, &tmB, p, s, smem_raw, grp * p.M + m0, n0, kb0, nkb, grp * p.x_group);
   volatile int* abortp = &s.abort_flag;
-  const int rows = (p.N - n0 < p.bn) ? (p.N - n0) : p.bn;  // valid tokens in this tile
+  const int rows = (nend - n0 < p.bn) ? (nend - n0) : p.bn;  // valid tokens in this tile
   constexpr int OUTW = kGlu ? 64 : 128;       // output features per tile
 
   if (warp >= 2) {
@@ -106,7 +114,7 @@ k_gemm(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensor
     // (.sync.aligned) TMEM loads, and make the decision to load warp-uniform
     ok = __all_sync(0xffffffffu, ok);
     tc_fence_after();
-    const float bias = (p.bias && m0 + ml < p.M) ? __bfloat162float(p.bias[m0 + ml]) : 0.f;
+    const float bias = (p.bias && m0 + ml < M) ? __bfloat162float(p.bias[m0 + ml]) : 0.f;
     float* stage_f = reinterpret_cast<float*>(sm);
     __nv_bfloat16* stage_h = reinterpret_cast<__nv_bfloat16*>(sm);
     for (int c = 0; c < p.bn; c += 16) {
@@ -145,8 +153,8 @@ k_gemm(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensor
       const int te = threadIdx.x - 64;
       for (int idx = te; idx < rows * 32; idx += 128) {
         const int t = idx >> 5, m = m0 + (idx & 31) * 4;
-        if (m < p.M)
-          store_f32x4(p, size_t(n0 + t) * p.ldy + ycol + m, m, *reinterpret_cast<const float4*>(stage_f + t * 128 + (idx & 31) * 4));
+        if (m < M)
+          store_f32x4(p, M, size_t(n0 + t) * p.ldy + ycol + m, m, *reinterpret_cast<const float4*>(stage_f + t * 128 + (idx & 31) * 4));
       }
     } else if (S == 1) {
       // coalesced copy-out of the staged tile: 16-byte pieces, OUTW features per token row
@@ -154,7 +162,7 @@ k_gemm(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensor
       const int te = threadIdx.x - 64;
       constexpr int PPR = OUTW / 8;  // 16-byte pieces per row
       const int out_m0 = kGlu ? (m0 >> 1) : m0;
-      const int out_M = kGlu ? (p.M >> 1) : p.M;
+      const int out_M = kGlu ? (M >> 1) : M;
       for (int idx = te; idx < rows * PPR; idx += 128) {
         const int t = idx / PPR, pc = idx % PPR;
         const int m = out_m0 + pc * 8;
@@ -182,19 +190,19 @@ k_gemm(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensor
         float4 acc = dsmem_sum_f32x4(stage_addr + uint32_t((t * 128 + f) * 4), S);
         const int m = m0 + f;
         if (p.bias) {
-          if (m + 0 < p.M) acc.x += __bfloat162float(p.bias[m + 0]);
-          if (m + 1 < p.M) acc.y += __bfloat162float(p.bias[m + 1]);
-          if (m + 2 < p.M) acc.z += __bfloat162float(p.bias[m + 2]);
-          if (m + 3 < p.M) acc.w += __bfloat162float(p.bias[m + 3]);
+          if (m + 0 < M) acc.x += __bfloat162float(p.bias[m + 0]);
+          if (m + 1 < M) acc.y += __bfloat162float(p.bias[m + 1]);
+          if (m + 2 < M) acc.z += __bfloat162float(p.bias[m + 2]);
+          if (m + 3 < M) acc.w += __bfloat162float(p.bias[m + 3]);
         }
         if (EPI == kEpiF32) {
-          if (m < p.M) store_f32x4(p, size_t(n0 + t) * p.ldy + ycol + m, m, acc);
+          if (m < M) store_f32x4(p, M, size_t(n0 + t) * p.ldy + ycol + m, m, acc);
         } else if (kGlu) {
           __nv_bfloat162 o = __floats2bfloat162_rn(glu_pair<kGlu ? EPI : kEpiSiluMul>(p, acc.x, acc.y), glu_pair<kGlu ? EPI : kEpiSiluMul>(p, acc.z, acc.w));
-          if (m + 4 <= p.M) *reinterpret_cast<__nv_bfloat162*>(p.y + size_t(n0 + t) * p.ldy + ycol + (m >> 1)) = o;
+          if (m + 4 <= M) *reinterpret_cast<__nv_bfloat162*>(p.y + size_t(n0 + t) * p.ldy + ycol + (m >> 1)) = o;
         } else {
           __nv_bfloat16* dst = p.y + size_t(n0 + t) * p.ldy + ycol + m;
-          if (m + 4 <= p.M) {
+          if (m + 4 <= M) {
             __nv_bfloat162 lo = __floats2bfloat162_rn(acc.x, acc.y), hi = __floats2bfloat162_rn(acc.z, acc.w);
             uint2 pk;
             pk.x = *reinterpret_cast<uint32_t*>(&lo);
@@ -202,7 +210,7 @@ k_gemm(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensor
             *reinterpret_cast<uint2*>(dst) = pk;
           } else {
             float a4[4] = {acc.x, acc.y, acc.z, acc.w};
-            for (int e = 0; e < 4 && m + e < p.M; e++) dst[e] = __float2bfloat16_rn(a4[e]);
+            for (int e = 0; e < 4 && m + e < M; e++) dst[e] = __float2bfloat16_rn(a4[e]);
           }
         }
       }
@@ -367,10 +375,17 @@ namespace {
 int launch_decode_form(const void* w, const void* x, int ldx, Params& p, int epi, int splits_hint, cudaStream_t st) {
   const int M = p.M, N = p.N, K = p.K, G = p.groups > 1 ? p.groups : 1;
   int bn, splits, stages;
-  tbvops::gemm_config(M, N, K, splits_hint, &bn, &splits, &stages, G, epi == kEpiF32);
+  if (p.row_off) {
+    // tiles for twice the average number of rows (a longer group takes several); K is split by the groups that can have rows at all
+    const int avg = (p.x_rows + G - 1) / G, want = N < 2 * avg + 8 ? N : 2 * avg + 8;
+    tbvops::gemm_config(M, want < 128 ? want : 128, K, splits_hint, &bn, &splits, &stages, G < p.x_rows ? G : p.x_rows, epi == kEpiF32);
+  } else {
+    tbvops::gemm_config(M, N, K, splits_hint, &bn, &splits, &stages, G, epi == kEpiF32);
+  }
   CUtensorMap tmA, tmB;
-  if (tbvops::make_tensor_map_bf16(&tmA, w, (unsigned long long)G * M, K, K, 128) != 0) return -3;
-  if (tbvops::make_tensor_map_bf16(&tmB, x, N, (unsigned long long)(G - 1) * p.x_group + K, ldx, bn) != 0) return -3;
+  const int xg = G - 1 + (p.m_last > 0);
+  if (tbvops::make_tensor_map_bf16(&tmA, w, (unsigned long long)G * M + p.m_last, K, K, 128) != 0) return -3;
+  if (tbvops::make_tensor_map_bf16(&tmB, x, p.row_off ? p.x_rows : N, (unsigned long long)xg * p.x_group + K, ldx, bn) != 0) return -3;
   p.bn = bn; p.splits = splits; p.stages = stages;
   p.kb_total = (K + 63) / 64;
   p.limit_ns = 2000000000ull;
@@ -389,7 +404,7 @@ int launch_decode_form(const void* w, const void* x, int ldx, Params& p, int epi
       }
     g_attr_done = true;
   }
-  const int mt = G * ((M + 127) / 128), nt = (N + bn - 1) / bn;
+  const int mt = G * ((M + 127) / 128) + (p.m_last + 127) / 128, nt = (N + bn - 1) / bn;
   p.raster = nt > 1 ? 1 : 0;
   const dim3 grid(p.raster ? nt : mt, p.raster ? mt : nt, splits), blk(gemm::kThreads);
   cudaError_t e;
@@ -451,10 +466,11 @@ int tbv_op_gemm(const void* w, const void* x, void* y, const void* bias, int M, 
 
 // The GEMM with the wider set of epilogues: fp32 output with an activation, clamped gated unit, grouped weights.
 // y: fp32 [N, ldy] for epi 2, bf16 otherwise; y2: optional bf16 copy of an fp32 result (same ldy).  act (epi 2): 0 none,
-// 1 softplus, 2 act_a * tanh(v / act_a).  epi 3: rows of w interleaved (gate_i, up_i), act_a = clamp limit, act_b = slope of the
-// sigmoid.  groups > 1: w is [groups * M, K]; group g reads x columns g * x_group .. + K and writes y columns g * y_group .. .
+// 1 softplus, 2 act_a * tanh(v / act_a), 3 tanh.  epi 3: rows of w interleaved (gate_i, up_i), act_a = clamp limit, act_b = slope of the
+// sigmoid, act_c = what is added to u.  groups > 1: w is [groups * M (+ m_last), K]; group g reads x columns g * x_group .. + K and writes y
+// columns g * y_group ..; m_last > 0 is one more group with that many features.
 int tbv_op_gemm_ex(const void* w, const void* x, void* y, void* y2, const void* bias, int M, int N, int K, int ldx, int ldy, int epi,
-                   int act, float act_a, float act_b, int groups, int x_group, int y_group, void* stream) {
+                   int act, float act_a, float act_b, float act_c, int groups, int x_group, int y_group, int m_last, void* stream) {
   const char* pf_ptr = nullptr;
   const unsigned long long pf_bytes = tbvops::take_next_prefetch(&pf_ptr, (unsigned long long)(M > 0 ? M : 0) * (unsigned long long)(K > 0 ? K : 0) * 2ull);
   if (M <= 0 || N <= 0 || K <= 0 || (K % 8) || (ldx % 8) || (ldy % 8) || (reinterpret_cast<uintptr_t>(y) & 15u)) return -2;
@@ -466,7 +482,7 @@ int tbv_op_gemm_ex(const void* w, const void* x, void* y, void* y2, const void* 
   if (epi == kEpiF32) p.yf = static_cast<float*>(y);
   else p.y = static_cast<__nv_bfloat16*>(y);
   p.y2 = static_cast<__nv_bfloat16*>(y2);
-  p.act = act; p.act_a = act_a; p.act_b = act_b;
+  p.act = act; p.act_a = act_a; p.act_b = act_b; p.act_c = act_c; p.m_last = groups > 1 ? m_last : 0;
   p.pf_ptr = pf_ptr;
   p.pf_bytes = pf_bytes;
   p.groups = groups > 1 ? groups : 1; p.x_group = groups > 1 ? x_group : 0; p.y_group = groups > 1 ? y_group : 0;
@@ -474,6 +490,22 @@ int tbv_op_gemm_ex(const void* w, const void* x, void* y, void* y2, const void* 
     const int th = tbvops::gemm_tok_choose(M, N, K, ldy, epi, persist_mode());
     if (th > 0) return tbvops::gemm_tok_launch_p(w, x, p, ldx, epi, th, stream);
   }
+  return launch_decode_form(w, x, ldx, p, epi, 0, static_cast<cudaStream_t>(stream));
+}
+
+// Row-grouped GEMM: rows row_off[g] .. row_off[g + 1] - 1 of x (x_rows in all, at most max_rows of one group) times rows g * M .. of w.  epi 0
+// stores bf16, 3 is the gated unit (arguments as above).
+int tbv_op_gemm_rows(const void* w, const void* x, void* y, const void* row_off, int groups, int M, int x_rows, int max_rows, int K, int ldx,
+                     int ldy, int epi, float act_a, float act_b, float act_c, void* stream) {
+  if (M <= 0 || x_rows <= 0 || max_rows <= 0 || K <= 0 || groups <= 0 || (K % 8) || (ldx % 8) || (ldy % 8) || (reinterpret_cast<uintptr_t>(y) & 15u) || !row_off) return -2;
+  if ((epi != kEpiStore && epi != kEpiClampGlu) || (epi == kEpiClampGlu && (M % 2))) return -2;
+  Params p{};
+  p.M = M; p.N = max_rows; p.K = K; p.ldy = ldy;
+  p.y = static_cast<__nv_bfloat16*>(y);
+  p.act_a = act_a; p.act_b = act_b; p.act_c = act_c;
+  p.groups = groups; p.row_off = static_cast<const int*>(row_off); p.x_rows = x_rows;
+  const int th = persist_mode() > 0 ? tbvops::gemm_tok_rows_choose(M, x_rows, groups) : 0;
+  if (th > 0) return tbvops::gemm_tok_launch_p(w, x, p, ldx, epi, th, stream);
   return launch_decode_form(w, x, ldx, p, epi, 0, static_cast<cudaStream_t>(stream));
 }
 

@@ -38,10 +38,15 @@ struct Params {
   float* yf;
   __nv_bfloat16* y2;
   int act;             // Act below
-  float act_a, act_b;  // softcap: limit; clamped GLU: limit, slope of the sigmoid
+  float act_a, act_b, act_c;  // softcap: limit; gated unit: limit, slope of the sigmoid, what is added to u
   // grouped form (decode-form kernel): `groups` problems of M features side by side; group g multiplies rows g * M .. of w
   // with columns g * x_group .. of x and writes at column g * y_group.  groups <= 1: one plain problem.
   int groups, x_group, y_group;
+  int m_last;          // > 0: one more group after the others, with this many features
+  // row-grouped form (a mixture of experts): group g owns rows row_off[g] .. row_off[g + 1] - 1 of x and y (device memory, read after the
+  // dependency wait) and rows g * M .. of w; N bounds the rows of one group, x_rows counts them all
+  const int* row_off;
+  int x_rows;
   unsigned long long limit_ns;  // bound on every barrier wait
   int* err;                     // device flag: set to 1 if a wait gave up
   const char* pf_ptr;           // weights of the GEMM that runs next (or null): see the producer's last step
@@ -49,18 +54,19 @@ struct Params {
 };
 
 enum Epi : int { kEpiStore = 0, kEpiSiluMul = 1, kEpiF32 = 2, kEpiClampGlu = 3 };
-enum Act : int { kActNone = 0, kActSoftplus = 1, kActSoftcap = 2 };
+enum Act : int { kActNone = 0, kActSoftplus = 1, kActSoftcap = 2, kActTanh = 3 };
 
 __device__ __forceinline__ float apply_act(float v, int act, float a) {
   if (act == kActSoftplus) return v > 20.f ? v : log1pf(expf(v));
   if (act == kActSoftcap) return a * tanhf(v / a);
+  if (act == kActTanh) return tanhf(v);
   return v;
 }
-// clamped gated unit: g = min(g, limit), u = clamp(u, -limit, limit); g * sigmoid(slope * g) * (u + 1), all in fp32
-__device__ __forceinline__ float clamp_glu(float g, float u, float limit, float slope) {
+// gated unit: g = min(g, limit), u = clamp(u, -limit, limit); g * sigmoid(slope * g) * (u + shift), all in fp32
+__device__ __forceinline__ float clamp_glu(float g, float u, float limit, float slope, float shift) {
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
-  return g / (1.0f + __expf(-slope * g)) * (u + 1.0f);
+  return g / (1.0f + __expf(-slope * g)) * (u + shift);
 }
 
 struct Smem {  // static shared state of one CTA

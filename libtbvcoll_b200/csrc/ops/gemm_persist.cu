@@ -27,6 +27,8 @@
 #include <cuda_runtime.h>
 #include <stdio.h>
 
+#include <type_traits>
+
 #include "gemm.cuh"
 #include "ops.h"
 
@@ -53,6 +55,14 @@ template <int TH> struct Shape {
 constexpr double kEffDecode[2] = {0.59, 0.43};   // decode-form kernel: store / SiLU-mul epilogue
 constexpr double kEffTok1 = 0.62;                // 128-token tiles: gate_up 4096 x 28672 x 4096 in 25 rounds, 722 us
 constexpr double kEffTok2 = 0.69;                // 256-token tiles: 0.66 (K 4096, SiLU-mul) .. 0.75 (K 14336) per round
+
+constexpr int kMaxRowGroups = 512;
+
+// Where a tile of a row-grouped problem lies: tiles are numbered group after group, inside a group token tile fastest.
+struct RowGroups {
+  int off[kMaxRowGroups + 1];      // first row of every group
+  int tile[kMaxRowGroups + 1];     // first tile of every group
+};
 
 struct PSmem {
   unsigned long long full[kMaxStages], empty[kMaxStages], acc_full[2], acc_empty[2];
@@ -108,7 +118,7 @@ __device__ __forceinline__ void store16(const gemm::Params& p, int n, int f, con
   } else if (EPI == gemm::kEpiClampGlu) {
     float o[8];
 #pragma unroll
-    for (int j = 0; j < 8; j++) o[j] = gemm::clamp_glu(v[2 * j], v[2 * j + 1], p.act_a, p.act_b);
+    for (int j = 0; j < 8; j++) o[j] = gemm::clamp_glu(v[2 * j], v[2 * j + 1], p.act_a, p.act_b, p.act_c);
     *reinterpret_cast<uint4*>(p.y + size_t(n) * p.ldy + (f >> 1)) =
         make_uint4(pack_bf16(o[0], o[1]), pack_bf16(o[2], o[3]), pack_bf16(o[4], o[5]), pack_bf16(o[6], o[7]));
   } else if (EPI == 1) {
@@ -130,7 +140,8 @@ __device__ __forceinline__ void store16(const gemm::Params& p, int n, int f, con
 
 // EPI 0: store (+bias); 1: SiLU-mul over interleaved gate/up features (output has M / 2 features); 2: fp32 store with
 // an activation; 3: clamped gated unit over interleaved gate/up features.
-template <int EPI, int TH>
+// ROWS: row-grouped problem (p.row_off).
+template <int EPI, int TH, bool ROWS>
 __global__ void __launch_bounds__(Shape<TH>::kThreads, 1)
 k_gemm_tok(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUtensorMap tmW, const gemm::Params p) {
   using S = Shape<TH>;
@@ -140,9 +151,8 @@ k_gemm_tok(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUte
   const uint32_t raw = smem_u32(smem_raw);
   const uint32_t base = (raw + 1023u) & ~1023u;
   const int tok_tiles = (p.N + S::kTok - 1) / S::kTok, feat_tiles = (p.M + kFeatTile - 1) / kFeatTile;
-  const int tiles = tok_tiles * feat_tiles;
   const int nkb = p.kb_total;
-  const int my_tiles = int(blockIdx.x) < tiles ? (tiles - int(blockIdx.x) + int(gridDim.x) - 1) / int(gridDim.x) : 0;
+  __shared__ typename std::conditional<ROWS, RowGroups, int>::type groups;
 
   if (threadIdx.x == 0) {
     for (int i = 0; i < S::kStages; i++) {
@@ -168,6 +178,48 @@ k_gemm_tok(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUte
   __syncthreads();
   tc_fence_after();
   pdl::launch_dependents();
+  int tiles = tok_tiles * feat_tiles;
+  if constexpr (ROWS) {
+    // the groups' rows were counted on the device by a kernel before this one
+    pdl::grid_dependency_wait();
+    for (int g = threadIdx.x; g <= p.groups; g += S::kThreads) groups.off[g] = p.row_off[g];
+    __syncthreads();
+    if (warp == 0) {
+      const int per = (p.groups + 31) / 32, a = min(p.groups, lane * per), b = min(p.groups, a + per);
+      auto count = [&](int g) { return (groups.off[g + 1] - groups.off[g] + S::kTok - 1) / S::kTok * feat_tiles; };
+      int sum = 0;
+      for (int g = a; g < b; g++) sum += count(g);
+      int inc = sum;
+      for (int o = 1; o < 32; o <<= 1) {
+        const int v = __shfl_up_sync(0xffffffffu, inc, o);
+        if (lane >= o) inc += v;
+      }
+      int run = inc - sum;
+      for (int g = a; g < b; g++) { groups.tile[g] = run; run += count(g); }
+      if (lane == 31) groups.tile[p.groups] = inc;
+    }
+    __syncthreads();
+    tiles = groups.tile[p.groups];
+  }
+  const int my_tiles = int(blockIdx.x) < tiles ? (tiles - int(blockIdx.x) + int(gridDim.x) - 1) / int(gridDim.x) : 0;
+  // first token row, end of the rows, first feature and its weight row of a tile
+  struct At { int n0, nend, f0, w0; };
+  auto locate = [&](int tile) -> At {
+    if constexpr (ROWS) {
+      int lo = 0, hi = p.groups - 1;               // the last group whose first tile is not beyond `tile`; empty groups are passed over
+      while (lo < hi) {
+        const int mid = (lo + hi + 1) >> 1;
+        if (groups.tile[mid] <= tile) lo = mid;
+        else hi = mid - 1;
+      }
+      const int local = tile - groups.tile[lo], tt = (groups.off[lo + 1] - groups.off[lo] + S::kTok - 1) / S::kTok;
+      const int f0 = local / tt * kFeatTile;
+      return At{groups.off[lo] + local % tt * S::kTok, groups.off[lo + 1], f0, lo * p.M + f0};
+    } else {
+      const int f0 = tile / tok_tiles * kFeatTile;
+      return At{tile % tok_tiles * S::kTok, p.N, f0, f0};
+    }
+  };
   const uint32_t tmem0 = s.tmem_base;
   volatile int* abortp = &s.abort_flag;
 
@@ -183,23 +235,26 @@ k_gemm_tok(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUte
       const int tile = int(blockIdx.x) + (i / nkb) * int(gridDim.x), kb = i % nkb;
       const uint32_t fb = smem_u32(&s.full[i]);
       mbar_expect_tx(fb, S::kStageBytes);
-      tma_load_2d(base + i * S::kStageBytes + S::kXBytes, &tmW, kb * gemm::kBK, (tile / tok_tiles) * kFeatTile, fb);
+      tma_load_2d(base + i * S::kStageBytes + S::kXBytes, &tmW, kb * gemm::kBK, locate(tile).w0, fb);
     }
     pdl::grid_dependency_wait();
     for (int i = 0; i < pre; i++) {
       const int tile = int(blockIdx.x) + (i / nkb) * int(gridDim.x), kb = i % nkb;
-      tma_load_2d_hint(base + i * S::kStageBytes, &tmX, kb * gemm::kBK, (tile % tok_tiles) * S::kTok, smem_u32(&s.full[i]), pol_x);
+      tma_load_2d_hint(base + i * S::kStageBytes, &tmX, kb * gemm::kBK, locate(tile).n0, smem_u32(&s.full[i]), pol_x);
     }
     issued = pre;
+    int cur = -1;
+    At at{};
     for (long i = pre; i < total; i++) {
       const int st = int(i % S::kStages);
       const uint32_t ph = uint32_t(i / S::kStages) & 1u;
       if (!mbar_wait(smem_u32(&s.empty[st]), ph ^ 1u, abortp, p.limit_ns)) break;
       const int tile = int(blockIdx.x) + int(i / nkb) * int(gridDim.x), kb = int(i % nkb);
+      if (tile != cur) at = locate(cur = tile);
       const uint32_t fb = smem_u32(&s.full[st]);
       mbar_expect_tx(fb, S::kStageBytes);
-      tma_load_2d_hint(base + st * S::kStageBytes, &tmX, kb * gemm::kBK, (tile % tok_tiles) * S::kTok, fb, pol_x);
-      tma_load_2d(base + st * S::kStageBytes + S::kXBytes, &tmW, kb * gemm::kBK, (tile / tok_tiles) * kFeatTile, fb);
+      tma_load_2d_hint(base + st * S::kStageBytes, &tmX, kb * gemm::kBK, at.n0, fb, pol_x);
+      tma_load_2d(base + st * S::kStageBytes + S::kXBytes, &tmW, kb * gemm::kBK, at.w0, fb);
       issued = i + 1;
     }
     if (*abortp) {
@@ -248,10 +303,11 @@ k_gemm_tok(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUte
       if (!ok) break;
       tc_fence_after();
       const int tile = int(blockIdx.x) + t * int(gridDim.x);
-      const int n = (tile % tok_tiles) * S::kTok + half * 128 + quarter * 32 + lane;   // token row
-      const int f0 = (tile / tok_tiles) * kFeatTile;
+      const At at = locate(tile);
+      const int n = at.n0 + half * 128 + quarter * 32 + lane;   // token row
+      const int f0 = at.f0;
       const uint32_t trow = tmem0 + (uint32_t(quarter * 32) << 16) + uint32_t((TH == 1 ? buf : half) * kFeatTile);
-      const bool row_ok = n < p.N;
+      const bool row_ok = n < at.nend;
       for (int c = 0; c < kFeatTile; c += 32) {
         uint32_t r[32];
         __syncwarp();   // rows past the end skip the stores below: reconverge before the warp-wide load
@@ -283,19 +339,20 @@ k_gemm_tok(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUte
 
 bool g_attr = false;
 
-template <int EPI, int TH>
+template <int EPI, int TH, bool ROWS = false>
 cudaError_t launch(const void* w, const void* x, const gemm::Params& p, int ldx, cudaStream_t st, int* map_rc) {
   using S = Shape<TH>;
   CUtensorMap tmX, tmW;
   *map_rc = 0;
-  if (tbvops::make_tensor_map_bf16(&tmX, x, p.N, p.K, ldx, S::kTok) != 0 || tbvops::make_tensor_map_bf16(&tmW, w, p.M, p.K, p.K, kFeatTile) != 0) {
+  if (tbvops::make_tensor_map_bf16(&tmX, x, ROWS ? p.x_rows : p.N, p.K, ldx, S::kTok) != 0 ||
+      tbvops::make_tensor_map_bf16(&tmW, w, (unsigned long long)(ROWS ? p.groups : 1) * p.M, p.K, p.K, kFeatTile) != 0) {
     *map_rc = -3;
     return cudaSuccess;
   }
-  const int tiles = ((p.N + S::kTok - 1) / S::kTok) * ((p.M + kFeatTile - 1) / kFeatTile);
+  const int tiles = ((ROWS ? p.x_rows / S::kTok + p.groups : (p.N + S::kTok - 1) / S::kTok)) * ((p.M + kFeatTile - 1) / kFeatTile);   // ROWS: at most
   const int sms = tbvops::sm_count();
   const size_t smem = size_t(S::kStages) * S::kStageBytes + 1024;
-  return pdl::launch(k_gemm_tok<EPI, TH>, dim3(tiles < sms ? tiles : sms), dim3(S::kThreads), smem, st, 1, tmX, tmW, p);
+  return pdl::launch(k_gemm_tok<EPI, TH, ROWS>, dim3(tiles < sms ? tiles : sms), dim3(S::kThreads), smem, st, 1, tmX, tmW, p);
 }
 
 }  // namespace
@@ -324,6 +381,13 @@ int gemm_tok_choose(int M, int N, int K, int ldy, int epi, int mode) {
   return e1 <= e2 ? 1 : 2;
 }
 
+// Row-grouped: the decode form re-reads a group's weights for every tile of up to 128 rows; this form wastes what a group's last tile lacks.
+int gemm_tok_rows_choose(int M, int x_rows, int groups) {
+  if ((M % 16) || groups > kMaxRowGroups) return 0;
+  const int avg = x_rows / groups;
+  return avg >= 384 ? 2 : (avg >= 64 ? 1 : 0);
+}
+
 int gemm_tok_launch(const void* w, const void* x, void* y, const void* bias, int M, int N, int K, int ldx, int ldy, int epi, int th,
                     void* stream) {
   gemm::Params p{};
@@ -339,14 +403,18 @@ int gemm_tok_launch_p(const void* w, const void* x, gemm::Params& p, int ldx, in
   p.limit_ns = 2000000000ull;
   p.err = gemm_err_flag();
   if (!g_attr) {
-    cudaError_t a[8] = {cudaFuncSetAttribute(k_gemm_tok<0, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
-                        cudaFuncSetAttribute(k_gemm_tok<1, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
-                        cudaFuncSetAttribute(k_gemm_tok<2, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
-                        cudaFuncSetAttribute(k_gemm_tok<3, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
-                        cudaFuncSetAttribute(k_gemm_tok<0, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
-                        cudaFuncSetAttribute(k_gemm_tok<1, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
-                        cudaFuncSetAttribute(k_gemm_tok<2, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
-                        cudaFuncSetAttribute(k_gemm_tok<3, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024)};
+    cudaError_t a[12] = {cudaFuncSetAttribute(k_gemm_tok<0, 1, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
+                        cudaFuncSetAttribute(k_gemm_tok<1, 1, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
+                        cudaFuncSetAttribute(k_gemm_tok<2, 1, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
+                        cudaFuncSetAttribute(k_gemm_tok<3, 1, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
+                        cudaFuncSetAttribute(k_gemm_tok<0, 2, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
+                        cudaFuncSetAttribute(k_gemm_tok<1, 2, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
+                        cudaFuncSetAttribute(k_gemm_tok<2, 2, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
+                        cudaFuncSetAttribute(k_gemm_tok<3, 2, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024),
+                         cudaFuncSetAttribute(k_gemm_tok<0, 1, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024),
+                         cudaFuncSetAttribute(k_gemm_tok<0, 2, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024),
+                         cudaFuncSetAttribute(k_gemm_tok<3, 1, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024),
+                         cudaFuncSetAttribute(k_gemm_tok<3, 2, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)};
     for (cudaError_t e : a)
       if (e != cudaSuccess) return -1;
     g_attr = true;
@@ -354,7 +422,10 @@ int gemm_tok_launch_p(const void* w, const void* x, gemm::Params& p, int ldx, in
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   int map_rc = 0;
   cudaError_t e;
-  switch (epi * 2 + (th == 2 ? 1 : 0)) {
+  if (p.row_off) {
+    if (epi == gemm::kEpiClampGlu) e = th == 2 ? launch<3, 2, true>(w, x, p, ldx, st, &map_rc) : launch<3, 1, true>(w, x, p, ldx, st, &map_rc);
+    else e = th == 2 ? launch<0, 2, true>(w, x, p, ldx, st, &map_rc) : launch<0, 1, true>(w, x, p, ldx, st, &map_rc);
+  } else switch (epi * 2 + (th == 2 ? 1 : 0)) {
     case 1: e = launch<0, 2>(w, x, p, ldx, st, &map_rc); break;
     case 2: e = launch<1, 1>(w, x, p, ldx, st, &map_rc); break;
     case 3: e = launch<1, 2>(w, x, p, ldx, st, &map_rc); break;

@@ -10,26 +10,28 @@
 //   prefill form  keys and values of the visible context are expanded once into dense rows and many query rows share
 //                 them: a third of the arithmetic per (query, key) pair.
 // Scores, softmax and sums are fp32; the denominator contains exp(sink_h) once.
+//
+// The rows form also serves attention whose values are the unnormalised keys (template KS; shared_attn.cu): kv_heads rows per token, each used by
+// heads / kv_heads query heads, with one fp32 factor per row (kept in the row's pad) on its scores, and an optional soft cap.
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
 #include <stdio.h>
 
 #include "../pdl.cuh"
+#include "attn_mma.cuh"
 #include "ops.h"
 #include "sm100.cuh"
+#include "vec.cuh"
+
+using namespace attn_mma;
+using vec::from_f;
+using vec::to_f;
 
 namespace {
 
-constexpr float kNegBig = -1e30f;
-constexpr float kLog2e = 1.4426950408889634f;
 constexpr int kMaxPairs = 512;
 constexpr int kRowPad = 8;
-
-__device__ __forceinline__ float to_f(float v) { return v; }
-__device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
-__device__ __forceinline__ void from_f(float& d, float v) { d = v; }
-__device__ __forceinline__ void from_f(__nv_bfloat16& d, float v) { d = __float2bfloat16_rn(v); }
 
 // ---- rotation, latent norm, cache write ------------------------------------------------------------------------------
 struct PrepParams {
@@ -104,12 +106,15 @@ struct RowsParams {
   const float* sink;        // [heads] or null
   void* out;                // [rows, heads, Rp]
   int heads, R, Rp, rotp, block_size, max_blocks, splits;
+  int kv_heads;             // cache rows per token: block b, head g and place t of a block at row (b * kv_heads + g) * block_size + t
   float scale_log2, scale;
+  float softcap;            // 0: none (KS form only)
   int* err;                 // device flag: set to 1 if a wait for copies gave up
 };
 
 // fp32: one CTA per (row, head), tiles of 128 keys.  Exponents are taken of differences of natural-unit scores: a score of
 // hundreds loses nothing to a multiplication by log2 e.
+template <bool KS>
 __global__ void __launch_bounds__(128) k_latent_rows_f32(const RowsParams p) {
   extern __shared__ float sm[];
   __shared__ float red[4];
@@ -124,6 +129,7 @@ __global__ void __launch_bounds__(128) k_latent_rows_f32(const RowsParams p) {
   const float* cache = static_cast<const float*>(p.cache);
   const int ctx = min(p.ctx_lens[row], p.max_blocks * p.block_size);
   const int* bt = p.tables + size_t(p.seq_of_row ? p.seq_of_row[row] : row) * p.max_blocks;
+  const int G = p.kv_heads, g = h / (p.heads / G);
   constexpr int kAcc = 16;   // Rp <= 2048
   float o[kAcc];
 #pragma unroll
@@ -134,7 +140,7 @@ __global__ void __launch_bounds__(128) k_latent_rows_f32(const RowsParams p) {
     __syncthreads();
     float s = kNegBig;
     if (tid < n) {
-      const int tok = t0 + tid, slot = bt[tok / p.block_size] * p.block_size + tok % p.block_size;
+      const int tok = t0 + tid, slot = (bt[tok / p.block_size] * G + g) * p.block_size + tok % p.block_size;
       sl[tid] = slot;
       const float4* kr = reinterpret_cast<const float4*>(cache + size_t(slot) * (Dk + kRowPad));
       const float4* q4 = reinterpret_cast<const float4*>(sq);
@@ -144,6 +150,10 @@ __global__ void __launch_bounds__(128) k_latent_rows_f32(const RowsParams p) {
         a.x = fmaf(q.x, k.x, a.x); a.y = fmaf(q.y, k.y, a.y); a.z = fmaf(q.z, k.z, a.z); a.w = fmaf(q.w, k.w, a.w);
       }
       s = ((a.x + a.y) + (a.z + a.w)) * p.scale;
+      if (KS) {
+        s *= cache[size_t(slot) * (Dk + kRowPad) + Dk];
+        if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
+      }
     }
     float mx = s;
 #pragma unroll
@@ -185,57 +195,13 @@ __global__ void __launch_bounds__(128) k_latent_rows_f32(const RowsParams p) {
   }
 }
 
-__device__ __forceinline__ uint32_t smem_addr(const void* p) { return static_cast<uint32_t>(__cvta_generic_to_shared(p)); }
-__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-__device__ __forceinline__ void st_zero16(uint32_t dst) { asm volatile("st.shared.v4.u32 [%0], {%1,%1,%1,%1};" ::"r"(dst), "r"(0u) : "memory"); }
-__device__ __forceinline__ void ldmatrix_x4(uint32_t addr, uint32_t* r) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ldmatrix_x2(uint32_t addr, uint32_t* r) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(addr));
-}
-__device__ __forceinline__ void ldmatrix_x4_trans(uint32_t addr, uint32_t* r) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void mma_bf16(float* d, const uint32_t* a, uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
-  __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
-  return *reinterpret_cast<uint32_t*>(&v);
-}
-__device__ __forceinline__ float ld_cluster_f32(uint32_t addr, uint32_t rank) {
-  uint32_t r;
-  float v;
-  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(addr), "r"(rank));
-  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(r) : "memory");
-  return v;
-}
-__device__ __forceinline__ float4 ld_cluster_f32x4(uint32_t addr, uint32_t rank) {
-  uint32_t r;
-  float4 v;
-  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(addr), "r"(rank));
-  asm volatile("ld.shared::cluster.v4.f32 {%0,%1,%2,%3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(r) : "memory");
-  return v;
-}
-__device__ __forceinline__ void cluster_sync() {
-  asm volatile("barrier.cluster.arrive.release.aligned;\nbarrier.cluster.wait.acquire.aligned;" ::: "memory");
-}
-
 // bf16: 16 heads of one row per CTA on tensor cores.  Eight warps share tiles of TT cached tokens that a ninth brings into two stages by
 // bulk copies.  Scores: warp w takes tokens 8w.. of the tile over all Dk columns.  Weighted sum: it takes the latent columns of the
 // 16-column blocks w, w + 8, .. (CBW of them).  grid (rows, head tiles, splits), cluster (1, 1, splits): the CTAs of a cluster cover
 // disjoint token ranges and merge in split order.
 constexpr int kRW = 8;
 constexpr int kMaxSplits = 8;
-template <int CBW, int TT>
+template <int CBW, int TT, bool KS>
 __global__ void __launch_bounds__(kRW * 32 + 32, 1) k_latent_rows_mma(const RowsParams p) {
   extern __shared__ __align__(128) uint8_t dsm[];
   __shared__ float sh_max[kRW][16], sh_l[kRW][16], sh_ml[16][2], sh_fac[kMaxSplits][16], sh_sm[kMaxSplits][16];
@@ -251,7 +217,10 @@ __global__ void __launch_bounds__(kRW * 32 + 32, 1) k_latent_rows_mma(const Rows
   }
   __syncthreads();
   pdl::grid_dependency_wait();
-  const int row = blockIdx.x, h0 = blockIdx.y * 16, sp = blockIdx.z, S = p.splits;
+  const int row = blockIdx.x, sp = blockIdx.z, S = p.splits;
+  // head tile: 16 query heads of one cache head g
+  const int G = KS ? p.kv_heads : 1, hpk = p.heads / G, tpg = (hpk + 15) / 16, g = KS ? blockIdx.y / tpg : 0;
+  const int h0 = g * hpk + (blockIdx.y - g * tpg) * 16;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r8 = lane >> 2, quad = lane & 3;
   const int Dk = p.Rp + p.rotp, chunks = Dk / 8, pitch = (Dk + kRowPad) * 2, ksteps = Dk / 16, cblocks = p.Rp / 16;
   const uint32_t sq = smem_addr(dsm), sk0 = sq + 16 * pitch, stage = uint32_t(TT) * pitch, spb = smem_addr(sh_p);
@@ -265,7 +234,7 @@ __global__ void __launch_bounds__(kRW * 32 + 32, 1) k_latent_rows_mma(const Rows
 
   const __nv_bfloat16* qa = static_cast<const __nv_bfloat16*>(p.qa) + (size_t(row) * p.heads + h0) * (Dk + kRowPad);
   const __nv_bfloat16* cache = static_cast<const __nv_bfloat16*>(p.cache);
-  const int nq = min(16, p.heads - h0);
+  const int nq = min(16, (g + 1) * hpk - h0);
   for (int r = nq + warp; r < 16; r += kRW + 1)
     for (int c = lane; c < chunks; c += 32) st_zero16(sq + r * pitch + c * 16);
   // The ninth warp brings the tiles in.  Tile i: its tokens, a block (or the part of one inside the tile) per copy, and the query rows
@@ -289,7 +258,7 @@ __global__ void __launch_bounds__(kRW * 32 + 32, 1) k_latent_rows_mma(const Rows
     for (int pg = pg0 + lane; pg * bs < tok0 + n; pg += 32) {
       if (pg >= pg0 + 32) block = bt[pg];      // blocks of one or two tokens only
       const int a = max(tok0, pg * bs), e = min(tok0 + n, (pg + 1) * bs);
-      sm100::bulk_load(dst + (a - tok0) * pitch, cache + (size_t(block) * bs + (a - pg * bs)) * (Dk + kRowPad), uint32_t(e - a) * pitch, bar);
+      sm100::bulk_load(dst + (a - tok0) * pitch, cache + ((size_t(block) * G + g) * bs + (a - pg * bs)) * (Dk + kRowPad), uint32_t(e - a) * pitch, bar);
     }
     for (int r = n; r < ((n + 15) & ~15); r++)
       for (int c = lane; c < chunks; c += 32) st_zero16(dst + r * pitch + c * 16);
@@ -360,8 +329,16 @@ __global__ void __launch_bounds__(kRW * 32 + 32, 1) k_latent_rows_mma(const Rows
 #pragma unroll
       for (int j = 0; j < 4; j++) sc[j] += se[j], sd[j] += sf[j];
       const int tok = t0 + i * TT + warp * 8 + quad * 2;
+      if constexpr (KS) {
+        float f[2];            // the two tokens' factors (stale past the end: masked below)
 #pragma unroll
-      for (int j = 0; j < 4; j++) sc[j] = tok + (j & 1) < t1 ? (sc[j] + sd[j]) * p.scale_log2 : kNegBig;
+        for (int j = 0; j < 2; j++) asm volatile("ld.shared.f32 %0, [%1];" : "=f"(f[j]) : "r"(sk + (warp * 8 + quad * 2 + j) * pitch + Dk * 2) : "memory");
+#pragma unroll
+        for (int j = 0; j < 4; j++) sc[j] = tok + (j & 1) < t1 ? capped_log2((sc[j] + sd[j]) * (f[j & 1] * p.scale), p.softcap) : kNegBig;
+      } else {
+#pragma unroll
+        for (int j = 0; j < 4; j++) sc[j] = tok + (j & 1) < t1 ? (sc[j] + sd[j]) * p.scale_log2 : kNegBig;
+      }
       float x_lo = fmaxf(sc[0], sc[1]), x_hi = fmaxf(sc[2], sc[3]);
       x_lo = fmaxf(x_lo, __shfl_xor_sync(0xffffffffu, x_lo, 1));
       x_lo = fmaxf(x_lo, __shfl_xor_sync(0xffffffffu, x_lo, 2));
@@ -462,7 +439,7 @@ __global__ void __launch_bounds__(kRW * 32 + 32, 1) k_latent_rows_mma(const Rows
   }
   __syncthreads();
   if (tid < 16) {
-    const float sk = p.sink && h0 + tid < p.heads ? p.sink[h0 + tid] * kLog2e : kNegBig;
+    const float sk = p.sink && tid < nq ? p.sink[h0 + tid] * kLog2e : kNegBig;
     float mx = sk, l = 0.f;
     for (int r = 0; r < S; r++) mx = fmaxf(mx, sh_sm[r][tid]);
     for (int r = 0; r < S; r++) l = fmaf(sh_fac[r][tid], exp2f(sh_sm[r][tid] - mx), l);
@@ -470,7 +447,7 @@ __global__ void __launch_bounds__(kRW * 32 + 32, 1) k_latent_rows_mma(const Rows
     for (int r = 0; r < S; r++) sh_fac[r][tid] = l > 0.f ? exp2f(sh_sm[r][tid] - mx) / l : 0.f;
   }
   __syncthreads();
-  const int nh = min(16, p.heads - h0), total = nh * p.Rp / 4, per = (total + S - 1) / S;
+  const int total = nq * p.Rp / 4, per = (total + S - 1) / S;
   __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + (size_t(row) * p.heads + h0) * p.Rp;
   const uint32_t soa = smem_addr(so);
   for (int i = tid; i < per; i += kRW * 32 + 32) {
@@ -678,24 +655,11 @@ __global__ void __launch_bounds__(128, 2) k_latent_prefill_mma(const PrefillPara
   }
 }
 
-constexpr size_t kMaxSmem = 226 * 1024;
-
-template <typename K>
-cudaError_t allow_smem(K kern, size_t bytes, bool* done) {
-  if (*done || bytes <= 32 * 1024) return cudaSuccess;   // up to 48 KB with the static part needs no opt-in
-  cudaFuncAttributes a;
-  cudaError_t e = cudaFuncGetAttributes(&a, kern);
-  if (e != cudaSuccess) return e;
-  e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, int(227 * 1024 - a.sharedSizeBytes));   // static + dynamic: 227 KB
-  if (e == cudaSuccess) *done = true;
-  return e;
-}
-
-template <int CBW, int TT>
+template <int CBW, int TT, bool KS>
 cudaError_t launch_rows(const RowsParams& p, dim3 grid, size_t smem, cudaStream_t st) {
   static bool done = false;
-  cudaError_t e = allow_smem(k_latent_rows_mma<CBW, TT>, smem, &done);
-  return e != cudaSuccess ? e : pdl::launch(k_latent_rows_mma<CBW, TT>, grid, dim3(kRW * 32 + 32), smem, st, p.splits, p);
+  cudaError_t e = allow_smem(k_latent_rows_mma<CBW, TT, KS>, smem, &done);
+  return e != cudaSuccess ? e : pdl::launch(k_latent_rows_mma<CBW, TT, KS>, grid, dim3(kRW * 32 + 32), smem, st, p.splits, p);
 }
 template <int VT>
 cudaError_t launch_prefill(const PrefillParams& p, dim3 grid, size_t smem, cudaStream_t st) {
@@ -705,6 +669,31 @@ cudaError_t launch_prefill(const PrefillParams& p, dim3 grid, size_t smem, cudaS
 }
 size_t rows_smem(int Dk, int TT) { return size_t(16 + 2 * TT) * (Dk * 2 + 16); }
 size_t prefill_smem(int Dq, int vdp) { return size_t(64 + 2 * kPK) * (Dq * 2 + 16) + size_t(2) * kPK * (vdp * 2 + 16); }
+
+template <bool KS>
+int rows_form(RowsParams& p, int rows, int bf16, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (p.heads <= 0 || p.block_size <= 0) return -2;
+  p.err = tbvops::gemm_err_flag();
+  cudaError_t e;
+  if (!bf16) {
+    p.splits = 1;
+    if (p.Rp > 2048) return -2;
+    e = pdl::launch(k_latent_rows_f32<KS>, dim3(rows, p.heads), dim3(128), size_t(p.Rp + p.rotp + 256) * 4, st, 1, p);
+    return e == cudaSuccess ? 0 : -1;
+  }
+  p.splits = p.splits < 1 ? 1 : (p.splits > kMaxSplits ? kMaxSplits : p.splits);
+  const int Dk = p.Rp + p.rotp;
+  const dim3 grid(rows, p.kv_heads * ((p.heads / p.kv_heads + 15) / 16), p.splits);
+  const size_t s64 = rows_smem(Dk, 64), s32 = rows_smem(Dk, 32);   // either holds the [16][Rp] fp32 partials too
+  if (p.Rp <= 128) e = launch_rows<1, 64, KS>(p, grid, s64, st);
+  else if (p.Rp <= 256) e = launch_rows<2, 64, KS>(p, grid, s64, st);
+  else if (p.Rp <= 512 && s64 <= kMaxSmem - 8192) e = launch_rows<4, 64, KS>(p, grid, s64, st);
+  else if (p.Rp <= 1024 && s32 <= kMaxSmem - 8192) e = launch_rows<8, 32, KS>(p, grid, s32, st);
+  else return -2;
+  if (e != cudaSuccess) fprintf(stderr, "[tbvops] latent attention launch failed: %s\n", cudaGetErrorString(e));
+  return e == cudaSuccess ? 0 : -1;
+}
 
 }  // namespace
 
@@ -726,28 +715,21 @@ int tbv_op_latent_prep(void* qkv, void* qa, void* cache, const void* gamma, cons
 int tbv_op_latent_attn_rows(const void* qa, const void* cache, const void* tables, const void* seq_of_row, const void* ctx_lens,
                             const void* sink, void* out, int rows, int heads, int R, int Rp, int rotp, int block_size, int max_blocks,
                             int splits, float scale, int bf16, void* stream) {
-  if (rows <= 0) return 0;
-  if (heads <= 0 || R > Rp || (Rp % 16) || (rotp % 16) || block_size <= 0) return -2;
+  if (R > Rp || (Rp % 16) || (rotp % 16)) return -2;
   RowsParams p{qa, cache, static_cast<const int*>(tables), static_cast<const int*>(seq_of_row), static_cast<const int*>(ctx_lens),
-               static_cast<const float*>(sink), out, heads, R, Rp, rotp, block_size, max_blocks, 1, scale * kLog2e, scale, tbvops::gemm_err_flag()};
-  cudaStream_t st = static_cast<cudaStream_t>(stream);
-  cudaError_t e;
-  if (!bf16) {
-    if (Rp > 2048) return -2;
-    e = pdl::launch(k_latent_rows_f32, dim3(rows, heads), dim3(128), size_t(Rp + rotp + 256) * 4, st, 1, p);
-    return e == cudaSuccess ? 0 : -1;
-  }
-  p.splits = splits < 1 ? 1 : (splits > kMaxSplits ? kMaxSplits : splits);
-  const int Dk = Rp + rotp;
-  const dim3 grid(rows, (heads + 15) / 16, p.splits);
-  const size_t s64 = rows_smem(Dk, 64), s32 = rows_smem(Dk, 32);   // either holds the [16][Rp] fp32 partials too
-  if (Rp <= 128) e = launch_rows<1, 64>(p, grid, s64, st);
-  else if (Rp <= 256) e = launch_rows<2, 64>(p, grid, s64, st);
-  else if (Rp <= 512 && s64 <= kMaxSmem - 8192) e = launch_rows<4, 64>(p, grid, s64, st);
-  else if (Rp <= 1024 && s32 <= kMaxSmem - 8192) e = launch_rows<8, 32>(p, grid, s32, st);
-  else return -2;
-  if (e != cudaSuccess) fprintf(stderr, "[tbvops] latent attention launch failed: %s\n", cudaGetErrorString(e));
-  return e == cudaSuccess ? 0 : -1;
+               static_cast<const float*>(sink), out, heads, R, Rp, rotp, block_size, max_blocks, splits, 1, scale * kLog2e, scale, 0.f, nullptr};
+  return rows_form<false>(p, rows, bf16, static_cast<cudaStream_t>(stream));
+}
+
+// Keys that are values (see shared_attn.cu): qa [rows, heads, Dp + pad], cache [blocks, kv_heads, block_size, Dp + pad] with the row's score
+// factor as fp32 in the first pad places; softcap 0 = none.
+int tbv_op_shared_attn_rows(const void* qa, const void* cache, const void* tables, const void* seq_of_row, const void* ctx_lens, void* out,
+                            int rows, int heads, int kv_heads, int Dp, int block_size, int max_blocks, int splits, float softcap, int bf16,
+                            void* stream) {
+  if ((Dp % 16) || kv_heads <= 0 || heads % kv_heads) return -2;
+  RowsParams p{qa, cache, static_cast<const int*>(tables), static_cast<const int*>(seq_of_row), static_cast<const int*>(ctx_lens),
+               nullptr, out, heads, Dp, Dp, 0, block_size, max_blocks, splits, kv_heads, kLog2e, 1.f, softcap, nullptr};
+  return rows_form<true>(p, rows, bf16, static_cast<cudaStream_t>(stream));
 }
 
 int tbv_op_latent_gather(const void* cache, const void* slots, void* c, void* kr, int n, int Rp, int rotp, void* stream) {

@@ -22,6 +22,8 @@ int gemm_tok_launch(const void* w, const void* x, void* y, const void* bias, int
                     void* stream);
 // the same for a filled parameter block (M, N, K, ldy, outputs, epilogue arguments)
 int gemm_tok_launch_p(const void* w, const void* x, gemm::Params& p, int ldx, int epi, int th, void* stream);
+// the same choice for row-grouped problems (x_rows rows over `groups` groups)
+int gemm_tok_rows_choose(int M, int x_rows, int groups);
 // evenly-split (stream-K) decode GEMM, gemm_streamk.cu
 bool gemm_streamk_wants(int M, int N, int K, int epi, int splits_hint, bool w_not_constant);
 int gemm_streamk_launch(const void* w, const void* x, void* y, const void* bias, int M, int N, int K, int ldx, int ldy, int epi,

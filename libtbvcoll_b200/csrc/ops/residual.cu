@@ -1,0 +1,257 @@
+// residual.cu — one fp32 residual stream with parallel branches: what lies between two layers in one kernel.
+//
+// A layer is x <- x + mixer(norm1(x)) + ff(norm2(x)).  The kernel that ends it adds the branches' results and starts the next layer:
+//   x  <- x + y1 + y2 + sum_j weight_j * routed[place_j]        (each term optional; the last is a mixture of experts)
+//   x  <- x + x0 + step                                           (optional: a loop's pass begins; x0 is the stream as the embedding left it)
+//   h1 = norm(x) * gamma1,  h2 = norm(x) * gamma2                 (both norms are of the same x: one root mean square)
+// or, for the embedding, x = table[id] * scale + position vector.  Sine and cosine come from turns = position * frequency / 2 pi in two
+// fp32 pieces, reduced before they are rounded.  For layers that mix every token with the one before, h1 stays fp32; when every
+// sequence has one row (a decode step) the mixes are written here, with the previous token's h1 from the carried state; otherwise
+// k_token_shift writes them from h1.
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <stdint.h>
+
+#include "../pdl.cuh"
+#include "vec.cuh"
+
+using vec::from_f;
+using vec::to_f;
+
+namespace {
+
+constexpr int kThreads = 512;
+constexpr int kMaxUnits = 16;       // float4 units of a row per thread: width <= 512 * 16 * 4
+constexpr int kMaxTop = 64;
+
+struct ResidualParams {
+  // embedding
+  const long long* ids;
+  const void* table;                // [vocab, ld] in the activation type
+  const float2* freq;               // [ceil(width / 2)]: turns per position, high and low part
+  const int* positions;
+  float embed_scale;
+  long long vocab;
+  // branches
+  float* x;                         // [rows, ld]
+  float* x0;                        // embedding: stored if given; otherwise added if given
+  const float *y1, *y2, *step;      // [rows, ld], [rows, ld], [ld]
+  const void* routed;               // [places, ld] in the activation type
+  const int* place;                 // [rows, top]
+  const float* weight;              // [rows, top]
+  int top;
+  // norms
+  const float *g1, *g2;
+  void *h1, *h2;                    // [rows, ldh]
+  int h1_f32;
+  const long long* rows;            // last: source row of every output row (null = identity); x is not written
+  int last;
+  // mixes with the previous token (one row per sequence)
+  const float* mu;                  // [nmix, ld]
+  void* mixes;                      // [rows, nmix, ld]
+  float* shift;                     // [slots, ld]
+  const int* segs;
+  int nmix;
+  int width, ld, ldh;
+  float eps;
+};
+
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xffff0000u));
+}
+__device__ __forceinline__ void store4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, const float4& v) {
+  __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+}
+__device__ __forceinline__ void add4(float4& a, const float4& b) { a.x += b.x; a.y += b.y; a.z += b.z; a.w += b.w; }
+__device__ __forceinline__ void fma4(float4& a, float s, const float4& b) { a.x = fmaf(s, b.x, a.x); a.y = fmaf(s, b.y, a.y); a.z = fmaf(s, b.z, a.z); a.w = fmaf(s, b.w, a.w); }
+__device__ __forceinline__ float4 mix4(const float4& h, const float4& prev, const float4& mu) {
+  return make_float4(fmaf(prev.x - h.x, mu.x, h.x), fmaf(prev.y - h.y, mu.y, h.y), fmaf(prev.z - h.z, mu.z, h.z), fmaf(prev.w - h.w, mu.w, h.w));
+}
+// sine and cosine of position * 2 pi * f, f = hi + lo turns per position
+__device__ __forceinline__ void sincos_turns(float pos, float2 f, float* s, float* c) {
+  const float t = pos * f.x, e = fmaf(pos, f.x, -t);      // t + e is the exact product
+  const float frac = (t - rintf(t)) + fmaf(pos, f.y, e);
+  sincospif(2.0f * frac, s, c);
+}
+
+template <typename T, bool EMBED, int U>
+__global__ void __launch_bounds__(kThreads) k_residual(const ResidualParams p) {
+  __shared__ float red[32], sw[kMaxTop];
+  __shared__ int sp[kMaxTop];
+  pdl::launch_dependents();
+  pdl::grid_dependency_wait();
+  const int units = p.ld / 4;
+  const size_t row = p.last && p.rows ? size_t(p.rows[blockIdx.x]) : blockIdx.x;
+  if (!EMBED && p.routed) {
+    if (threadIdx.x < p.top) {
+      sp[threadIdx.x] = p.place[row * p.top + threadIdx.x];
+      sw[threadIdx.x] = p.weight[row * p.top + threadIdx.x];
+    }
+    __syncthreads();
+  }
+  float* xr = p.x + row * p.ld;
+  float4 u[U];
+  float ss = 0.f;
+  const T* erow = nullptr;
+  float pos = 0.f;
+  if (EMBED) {
+    const long long id = p.ids[row];
+    erow = static_cast<const T*>(p.table) + size_t(id < 0 ? 0 : (id >= p.vocab ? p.vocab - 1 : id)) * p.ld;
+    pos = float(p.positions[row]);
+  }
+#pragma unroll
+  for (int k = 0; k < U; k++) {
+    const int i = threadIdx.x + k * blockDim.x;
+    u[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < units) {
+      if (EMBED) {
+        const float4 e = load4(erow + i * 4);
+        float pv[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int j = 0; j < 2; j++) {
+          const int c = i * 4 + 2 * j;
+          if (c < p.width) {
+            float s, co;
+            sincos_turns(pos, p.freq[c / 2], &s, &co);
+            pv[2 * j] = s;
+            if (c + 1 < p.width) pv[2 * j + 1] = co;
+          }
+        }
+        u[k] = make_float4(fmaf(e.x, p.embed_scale, pv[0]), fmaf(e.y, p.embed_scale, pv[1]), fmaf(e.z, p.embed_scale, pv[2]), fmaf(e.w, p.embed_scale, pv[3]));
+        if (p.x0) store4(p.x0 + row * p.ld + i * 4, u[k]);
+      } else {
+        u[k] = load4(xr + i * 4);
+        float4 b = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (p.y1) b = load4(p.y1 + row * p.ld + i * 4);
+        if (p.y2) add4(b, load4(p.y2 + row * p.ld + i * 4));
+        if (p.routed) {
+          const T* ro = static_cast<const T*>(p.routed) + i * 4;
+#pragma unroll 4
+          for (int j = 0; j < p.top; j++) fma4(b, sw[j], load4(ro + size_t(sp[j]) * p.ld));
+        }
+        add4(u[k], b);
+        if (p.x0) add4(u[k], load4(p.x0 + row * p.ld + i * 4));
+      }
+      if (p.step) add4(u[k], load4(p.step + i * 4));
+      if (!p.last) store4(xr + i * 4, u[k]);
+      ss += u[k].x * u[k].x + u[k].y * u[k].y + u[k].z * u[k].z + u[k].w * u[k].w;   // pad columns hold zeros
+    }
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  float tot = 0.f;
+  for (int w = 0; w < int(blockDim.x + 31) / 32; w++) tot += red[w];
+  const float r = 1.0f / sqrtf(tot / float(p.width) + p.eps);
+  float* shift = nullptr;
+  bool fresh = true;
+  if (p.mu) {
+    shift = p.shift + size_t(p.segs[4 * blockIdx.x + 2]) * p.ld;
+    fresh = p.positions[row] == 0;
+  }
+#pragma unroll
+  for (int k = 0; k < U; k++) {
+    const int i = threadIdx.x + k * blockDim.x;
+    if (i < units) {
+      const float4 g = load4(p.g1 + i * 4);
+      const float4 v = make_float4(u[k].x * r * g.x, u[k].y * r * g.y, u[k].z * r * g.z, u[k].w * r * g.w);
+      const size_t off = size_t(blockIdx.x) * p.ldh + i * 4;
+      if (p.mu) {
+        const float4 prev = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : load4(shift + i * 4);
+        store4(shift + i * 4, v);
+        for (int s = 0; s < p.nmix; s++)
+          store4(static_cast<T*>(p.mixes) + (row * p.nmix + s) * p.ld + i * 4, mix4(v, prev, load4(p.mu + size_t(s) * p.ld + i * 4)));
+      } else if (p.h1_f32) {
+        store4(static_cast<float*>(p.h1) + off, v);
+      } else {
+        store4(static_cast<T*>(p.h1) + off, v);
+      }
+      if (p.g2) {
+        const float4 g2 = load4(p.g2 + i * 4);
+        store4(static_cast<T*>(p.h2) + off, make_float4(u[k].x * r * g2.x, u[k].y * r * g2.y, u[k].z * r * g2.z, u[k].w * r * g2.w));
+      }
+    }
+  }
+}
+
+// mixes[t][s] = h_t + (h_{t-1} - h_t) * mu_s; the row before a segment's first comes from the state (zeros at a sequence's start).  The state is
+// read only: the recurrence of the layer, which runs later, replaces it.
+template <typename T>
+__global__ void __launch_bounds__(256) k_token_shift(const float* __restrict__ h, const float* __restrict__ mu, const float* __restrict__ shift,
+                                                     T* __restrict__ mixes, const int* __restrict__ segs, const int* __restrict__ seg_of_row,
+                                                     const int* __restrict__ positions, int ld, int nmix) {
+  pdl::launch_dependents();
+  pdl::grid_dependency_wait();
+  const int row = blockIdx.x, i = (blockIdx.y * 256 + threadIdx.x) * 4;
+  if (i >= ld) return;
+  const int* sg = segs + 4 * (seg_of_row ? seg_of_row[row] : row);
+  const float4 v = load4(h + size_t(row) * ld + i);
+  float4 prev = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (row > sg[0]) prev = load4(h + size_t(row - 1) * ld + i);
+  else if (positions[row] != 0) prev = load4(shift + size_t(sg[2]) * ld + i);
+  for (int s = 0; s < nmix; s++) store4(mixes + (size_t(row) * nmix + s) * ld + i, mix4(v, prev, load4(mu + size_t(s) * ld + i)));
+}
+
+template <typename T, bool EMBED>
+cudaError_t launch_u(const ResidualParams& p, int rows, cudaStream_t st) {
+  const int units = p.ld / 4;
+  const int per = units <= 64 ? 1 : (units <= kThreads * 2 ? 2 : (units <= kThreads * 4 ? 4 : (units <= kThreads * 8 ? 8 : 16)));
+  int threads = ((units + per - 1) / per + 31) / 32 * 32;
+  if (threads > kThreads) return cudaErrorInvalidValue;
+  if (threads < kMaxTop) threads = kMaxTop;
+  const dim3 grid(rows), blk(threads);
+  switch (per) {
+    case 1: return pdl::launch(k_residual<T, EMBED, 1>, grid, blk, 0, st, 1, p);
+    case 2: return pdl::launch(k_residual<T, EMBED, 2>, grid, blk, 0, st, 1, p);
+    case 4: return pdl::launch(k_residual<T, EMBED, 4>, grid, blk, 0, st, 1, p);
+    case 8: return pdl::launch(k_residual<T, EMBED, 8>, grid, blk, 0, st, 1, p);
+    default: return pdl::launch(k_residual<T, EMBED, 16>, grid, blk, 0, st, 1, p);
+  }
+}
+
+}  // namespace
+
+extern "C" {
+
+// See the top of the file.  ids != null: the embedding (y1, y2, routed ignored).  mu != null: the mixes are written instead of h1.
+int tbv_op_residual(const void* ids, const void* table, const void* freq, const void* positions, float embed_scale, long long vocab, void* x,
+                    void* x0, const void* y1, const void* y2, const void* step, const void* routed, const void* place, const void* weight, int top,
+                    const void* g1, const void* g2, void* h1, void* h2, int h1_f32, const void* row_map, int last, const void* mu, void* mixes,
+                    void* shift, const void* segs, int nmix, int rows, int width, int ld, int ldh, float eps, int bf16, void* stream) {
+  if (rows <= 0) return 0;
+  if (width <= 0 || width > ld || (ld % 4) || (ldh % 4) || ld > kThreads * 4 * kMaxUnits || ldh < ld || (routed && (top < 1 || top > kMaxTop))) return -2;
+  if (mu && (last || !segs || !positions || !shift || !mixes)) return -2;
+  ResidualParams p{};
+  p.ids = static_cast<const long long*>(ids); p.table = table; p.freq = static_cast<const float2*>(freq); p.positions = static_cast<const int*>(positions);
+  p.embed_scale = embed_scale; p.vocab = vocab;
+  p.x = static_cast<float*>(x); p.x0 = static_cast<float*>(x0); p.y1 = static_cast<const float*>(y1); p.y2 = static_cast<const float*>(y2);
+  p.step = static_cast<const float*>(step); p.routed = routed; p.place = static_cast<const int*>(place); p.weight = static_cast<const float*>(weight); p.top = top;
+  p.g1 = static_cast<const float*>(g1); p.g2 = static_cast<const float*>(g2); p.h1 = h1; p.h2 = h2; p.h1_f32 = h1_f32;
+  p.rows = static_cast<const long long*>(row_map); p.last = last; p.mu = static_cast<const float*>(mu); p.mixes = mixes; p.shift = static_cast<float*>(shift);
+  p.segs = static_cast<const int*>(segs); p.nmix = nmix; p.width = width; p.ld = ld; p.ldh = ldh; p.eps = eps;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  cudaError_t e = ids ? (bf16 ? launch_u<__nv_bfloat16, true>(p, rows, st) : launch_u<float, true>(p, rows, st))
+                      : (bf16 ? launch_u<__nv_bfloat16, false>(p, rows, st) : launch_u<float, false>(p, rows, st));
+  return e == cudaSuccess ? 0 : -1;
+}
+
+// h fp32 [rows, ld] -> mixes [rows, nmix, ld]
+int tbv_op_token_shift(const void* h, const void* mu, const void* shift, void* mixes, const void* segs, const void* seg_of_row, const void* positions,
+                       int rows, int ld, int nmix, int bf16, void* stream) {
+  if (rows <= 0) return 0;
+  if (ld % 4) return -2;
+  const dim3 grid(rows, (ld / 4 + 255) / 256);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const float *hf = static_cast<const float*>(h), *m = static_cast<const float*>(mu), *s = static_cast<const float*>(shift);
+  const int *sg = static_cast<const int*>(segs), *so = static_cast<const int*>(seg_of_row), *po = static_cast<const int*>(positions);
+  cudaError_t e = bf16 ? pdl::launch(k_token_shift<__nv_bfloat16>, grid, dim3(256), 0, st, 1, hf, m, s, static_cast<__nv_bfloat16*>(mixes), sg, so, po, ld, nmix)
+                       : pdl::launch(k_token_shift<float>, grid, dim3(256), 0, st, 1, hf, m, s, static_cast<float*>(mixes), sg, so, po, ld, nmix);
+  return e == cudaSuccess ? 0 : -1;
+}
+
+}  // extern "C"

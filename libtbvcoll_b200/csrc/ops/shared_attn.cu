@@ -1,0 +1,270 @@
+// shared_attn.cu — grouped-query attention whose values are the keys before their norm, with a query temperature that grows with the position
+// and soft-capped scores.
+//
+// A key is its value times one factor (the reciprocal root mean square over the head) times a weight per channel.  The weight and the
+// score scale are folded into the query, so ONE cached row per token and key head serves as key and as value:
+//   row = dim values | fp32 factor | pad          (dim padded to 16; eight places behind it, as in the latent cache)
+//   score(i, j) = cap * tanh((q'_i . row_j) * factor_j / cap),  q' = norm(q) * temperature * fold
+// Rows of a block lie together per key head ([blocks, kv_heads, block_size, dim + 8]), so that the rows form (latent_attn.cu, template KS)
+// brings a block in with one bulk copy.  Here: the kernel that normalises queries and writes cache rows, and the prefill form.
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <stdint.h>
+#include <stdio.h>
+
+#include "../pdl.cuh"
+#include "attn_mma.cuh"
+#include "vec.cuh"
+
+using namespace attn_mma;
+using vec::from_f;
+using vec::to_f;
+
+namespace {
+
+constexpr int kRowPad = 8;
+
+struct PrepParams {
+  void* qk;                 // [rows, ldq]: heads * Dp query columns, kv_heads * Dp key columns
+  void* qa;                 // [n_rows_form, heads, Dp + pad]; the queries of later rows stay in place
+  void* cache;
+  const float* fold;        // [Dp]
+  const int* positions;
+  const long long* slots;
+  int rows, ldq, heads, kv_heads, dim, Dp, n_rows_form, block_size;
+  float eps, temp_coef;
+  double temp_every;
+};
+
+// one warp per (row, head); heads of keys come after those of queries
+template <typename T>
+__global__ void __launch_bounds__(256) k_shared_prep(const PrepParams p) {
+  pdl::launch_dependents();
+  pdl::grid_dependency_wait();
+  const int lane = threadIdx.x & 31, nh = p.heads + p.kv_heads;
+  const long long w = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (w >= (long long)p.rows * nh) return;
+  const int row = int(w / nh), h = int(w - (long long)row * nh);
+  T* src = static_cast<T*>(p.qk) + size_t(row) * p.ldq + size_t(h) * p.Dp;
+  float ss = 0.f;
+  for (int i = lane; i < p.dim; i += 32) { const float v = to_f(src[i]); ss = fmaf(v, v, ss); }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  const float r = 1.0f / sqrtf(ss / float(p.dim) + p.eps);
+  if (h < p.heads) {
+    const double turns = floor((double(p.positions[row]) + 1.0) / p.temp_every);
+    const float f = r * (1.0f + p.temp_coef * logf(float(turns) + 1.0f));
+    T* dst = row < p.n_rows_form ? static_cast<T*>(p.qa) + (size_t(row) * p.heads + h) * (p.Dp + kRowPad) : src;
+    for (int i = lane; i < p.Dp; i += 32) from_f(dst[i], to_f(src[i]) * f * p.fold[i]);
+  } else {
+    const long long slot = p.slots[row];
+    if (slot < 0) return;
+    const size_t at = size_t((slot / p.block_size * p.kv_heads + (h - p.heads)) * p.block_size + slot % p.block_size);
+    T* dst = static_cast<T*>(p.cache) + at * (p.Dp + kRowPad);
+    for (int i = lane; i < p.Dp; i += 32) dst[i] = src[i];
+    if (lane == 0) *reinterpret_cast<float*>(dst + p.Dp) = r;
+  }
+}
+
+struct PrefillParams {
+  const __nv_bfloat16* q;   // [rows, ldq], head h at h * Dp
+  const __nv_bfloat16* cache;
+  __nv_bfloat16* out;       // [rows, ldo], head h at h * Dp
+  const int* tiles;         // [ntiles, 4]: first query row, rows (<= 64), unused, keys the first row sees
+  const int* seq_of_row;    // table row of a query row
+  const int* tables;
+  int ldq, ldo, heads, kv_heads, Dp, block_size, max_blocks;
+  float softcap;
+};
+
+// 64 query rows of one sequence and one head per CTA, four warps of 16 rows; tiles of 64 cached rows, keys and values at once, in two
+// cp.async stages.
+constexpr int kPK = 64;
+template <int VT>
+__global__ void __launch_bounds__(128, VT > 8 ? 2 : 3) k_shared_prefill_mma(const PrefillParams p) {
+  extern __shared__ __align__(128) uint8_t dsm[];
+  pdl::launch_dependents();
+  pdl::grid_dependency_wait();
+  const int* tl = p.tiles + 4 * blockIdx.y;
+  const int row0 = tl[0], nrows = tl[1], see0 = tl[3], h = blockIdx.x, g = h / (p.heads / p.kv_heads);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r8 = lane >> 2, quad = lane & 3;
+  const int ksteps = p.Dp / 16, pitch = (p.Dp + kRowPad) * 2, vblocks = p.Dp / 16, nch = p.Dp / 8;
+  const uint32_t sq = smem_addr(dsm), sk0 = sq + 64 * pitch;
+  const int* bt = p.tables + size_t(p.seq_of_row[row0]) * p.max_blocks;
+  const int nkeys = min(see0 + nrows - 1, p.max_blocks * p.block_size), ntiles = (nkeys + kPK - 1) / kPK;
+
+  // rows are copied by groups of lanes: 4 rows per warp pass, 8 lanes per row
+  const int g8 = lane >> 3, l8 = lane & 7;
+  for (int r = warp * 4 + g8; r < 64; r += 16) {
+    const uint32_t d = sq + r * pitch;
+    const __nv_bfloat16* src = p.q + size_t(row0 + r) * p.ldq + size_t(h) * p.Dp;
+    for (int c = l8; c < nch; c += 8) {
+      if (r < nrows) cp_async16(d + c * 16, src + c * 8);
+      else st_zero16(d + c * 16);
+    }
+  }
+  auto issue = [&](int i) {
+    if (i < ntiles) {
+      const uint32_t kb = sk0 + (i & 1) * kPK * pitch;
+      for (int r = warp * 4 + g8; r < kPK; r += 16) {
+        const int tok = i * kPK + r;
+        const uint32_t kd = kb + r * pitch;
+        if (tok < nkeys) {
+          const int pg = tok / p.block_size;
+          const __nv_bfloat16* src = p.cache + ((size_t(bt[pg]) * p.kv_heads + g) * p.block_size + (tok - pg * p.block_size)) * (p.Dp + kRowPad);
+          for (int c = l8; c <= nch; c += 8) cp_async16(kd + c * 16, src + c * 8);   // the last piece holds the factor
+        } else {
+          for (int c = l8; c <= nch; c += 8) st_zero16(kd + c * 16);
+        }
+      }
+    }
+    cp_async_commit();
+  };
+  float o[VT * 2][4];
+#pragma unroll
+  for (int n = 0; n < VT * 2; n++) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
+  float m_lo = kNegBig, m_hi = kNegBig, l_lo = 0.f, l_hi = 0.f;
+  const int see_lo = see0 + warp * 16 + r8, see_hi = see_lo + 8;   // keys visible to this lane's two rows
+  issue(0);
+  for (int i = 0; i < ntiles; i++) {
+    issue(i + 1);
+    cp_async_wait<1>();
+    __syncthreads();
+    const int tok0 = i * kPK;
+    if (tok0 < see0 + warp * 16 + 15) {          // otherwise every key of the tile is hidden from this warp's rows
+      const uint32_t sk = sk0 + (i & 1) * kPK * pitch;
+      float s[kPK / 8][4];
+#pragma unroll
+      for (int n = 0; n < kPK / 8; n++) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
+      const uint32_t qaddr = sq + (warp * 16 + (lane & 15)) * pitch + (lane >> 4) * 16;
+      const uint32_t kaddr = sk + ((lane & 7) + ((lane >> 4) << 3)) * pitch + ((lane >> 3) & 1) * 16;
+      for (int ks = 0; ks < ksteps; ks++) {
+        uint32_t a[4];
+        ldmatrix_x4(qaddr + ks * 32, a);
+#pragma unroll
+        for (int n = 0; n < kPK / 16; n++) {
+          uint32_t b[4];
+          ldmatrix_x4(kaddr + n * 16 * pitch + ks * 32, b);
+          mma_bf16(s[2 * n], a, b[0], b[1]);
+          mma_bf16(s[2 * n + 1], a, b[2], b[3]);
+        }
+      }
+      const bool diagonal = tok0 + kPK > see0 + warp * 16;
+      float x_lo = m_lo, x_hi = m_hi;
+#pragma unroll
+      for (int n = 0; n < kPK / 8; n++)
+#pragma unroll
+        for (int j = 0; j < 2; j++) {
+          float f;
+          asm volatile("ld.shared.f32 %0, [%1];" : "=f"(f) : "r"(sk + (n * 8 + quad * 2 + j) * pitch + p.Dp * 2) : "memory");
+          s[n][j] = capped_log2(s[n][j] * f, p.softcap);
+          s[n][2 + j] = capped_log2(s[n][2 + j] * f, p.softcap);
+          if (diagonal) {
+            const int tok = tok0 + n * 8 + quad * 2 + j;
+            if (tok >= see_lo) s[n][j] = kNegBig;
+            if (tok >= see_hi) s[n][2 + j] = kNegBig;
+          }
+        }
+#pragma unroll
+      for (int n = 0; n < kPK / 8; n++) { x_lo = fmaxf(x_lo, fmaxf(s[n][0], s[n][1])); x_hi = fmaxf(x_hi, fmaxf(s[n][2], s[n][3])); }
+      x_lo = fmaxf(x_lo, __shfl_xor_sync(0xffffffffu, x_lo, 1));
+      x_lo = fmaxf(x_lo, __shfl_xor_sync(0xffffffffu, x_lo, 2));
+      x_hi = fmaxf(x_hi, __shfl_xor_sync(0xffffffffu, x_hi, 1));
+      x_hi = fmaxf(x_hi, __shfl_xor_sync(0xffffffffu, x_hi, 2));
+      const float c_lo = exp2f(m_lo - x_lo), c_hi = exp2f(m_hi - x_hi);
+      m_lo = x_lo;
+      m_hi = x_hi;
+      float t_lo = 0.f, t_hi = 0.f;
+      uint32_t pa[kPK / 16][4];
+#pragma unroll
+      for (int n = 0; n < kPK / 8; n++) {
+        const float p0 = exp2f(s[n][0] - x_lo), p1 = exp2f(s[n][1] - x_lo), p2 = exp2f(s[n][2] - x_hi), p3 = exp2f(s[n][3] - x_hi);
+        t_lo += p0 + p1;
+        t_hi += p2 + p3;
+        pa[n >> 1][(n & 1) * 2] = pack_bf16(p0, p1);
+        pa[n >> 1][(n & 1) * 2 + 1] = pack_bf16(p2, p3);
+      }
+      l_lo = l_lo * c_lo + t_lo;
+      l_hi = l_hi * c_hi + t_hi;
+#pragma unroll
+      for (int n = 0; n < VT * 2; n++) { o[n][0] *= c_lo; o[n][1] *= c_lo; o[n][2] *= c_hi; o[n][3] *= c_hi; }
+#pragma unroll
+      for (int b = 0; b < VT; b++) {
+        if (b < vblocks) {
+#pragma unroll
+          for (int ks = 0; ks < kPK / 16; ks++) {
+            uint32_t v[4];
+            ldmatrix_x4_trans(sk + (ks * 16 + (lane & 15)) * pitch + b * 32 + (lane >> 4) * 16, v);
+            mma_bf16(o[2 * b], pa[ks], v[0], v[1]);
+            mma_bf16(o[2 * b + 1], pa[ks], v[2], v[3]);
+          }
+        }
+      }
+    }
+    __syncthreads();
+  }
+  cp_async_wait<0>();
+  l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1);
+  l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
+  l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1);
+  l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
+  const float f_lo = l_lo > 0.f ? 1.f / l_lo : 0.f, f_hi = l_hi > 0.f ? 1.f / l_hi : 0.f;
+  const int rl = warp * 16 + r8, rh = rl + 8;
+#pragma unroll
+  for (int n = 0; n < VT * 2; n++) {
+    if (n < vblocks * 2) {
+      const int col = h * p.Dp + n * 8 + quad * 2;
+      if (rl < nrows) *reinterpret_cast<uint32_t*>(p.out + size_t(row0 + rl) * p.ldo + col) = pack_bf16(o[n][0] * f_lo, o[n][1] * f_lo);
+      if (rh < nrows) *reinterpret_cast<uint32_t*>(p.out + size_t(row0 + rh) * p.ldo + col) = pack_bf16(o[n][2] * f_hi, o[n][3] * f_hi);
+    }
+  }
+}
+
+template <int VT>
+cudaError_t launch_prefill(const PrefillParams& p, dim3 grid, size_t smem, cudaStream_t st) {
+  static bool done = false;
+  cudaError_t e = allow_smem(k_shared_prefill_mma<VT>, smem, &done);
+  return e != cudaSuccess ? e : pdl::launch(k_shared_prefill_mma<VT>, grid, dim3(128), smem, st, 1, p);
+}
+
+}  // namespace
+
+extern "C" {
+
+int tbv_op_shared_attn_prep(void* qk, void* qa, void* cache, const void* fold, const void* positions, const void* slots, int rows,
+                            int n_rows_form, int ldq, int heads, int kv_heads, int dim, int Dp, int block_size, float eps, float temp_coef,
+                            double temp_every, int bf16, void* stream) {
+  if (rows <= 0) return 0;
+  if (dim > Dp || dim <= 0 || (Dp % 16) || kv_heads <= 0 || heads % kv_heads || n_rows_form > rows || block_size <= 0 || !(temp_every > 0)) return -2;
+  PrepParams p{qk, qa, cache, static_cast<const float*>(fold), static_cast<const int*>(positions), static_cast<const long long*>(slots),
+               rows, ldq, heads, kv_heads, dim, Dp, n_rows_form, block_size, eps, temp_coef, temp_every};
+  const dim3 grid(unsigned(((long long)rows * (heads + kv_heads) + 7) / 8));
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  cudaError_t e = bf16 ? pdl::launch(k_shared_prep<__nv_bfloat16>, grid, dim3(256), 0, st, 1, p) : pdl::launch(k_shared_prep<float>, grid, dim3(256), 0, st, 1, p);
+  return e == cudaSuccess ? 0 : -1;
+}
+
+// head sizes (padded) that the prefill form takes
+int tbv_op_shared_prefill_max_dim(void) { return 256; }
+
+int tbv_op_shared_attn_prefill(const void* q, const void* cache, const void* tables, const void* seq_of_row, const void* tiles, void* out,
+                               int ntiles, int ldq, int ldo, int heads, int kv_heads, int Dp, int block_size, int max_blocks, float softcap,
+                               void* stream) {
+  if (ntiles <= 0) return 0;
+  if ((Dp % 16) || Dp > 256 || (ldq % 8) || (ldo % 8) || kv_heads <= 0 || heads % kv_heads || ntiles > 65535 || !seq_of_row) return -2;
+  PrefillParams p{static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(cache), static_cast<__nv_bfloat16*>(out),
+                  static_cast<const int*>(tiles), static_cast<const int*>(seq_of_row), static_cast<const int*>(tables),
+                  ldq, ldo, heads, kv_heads, Dp, block_size, max_blocks, softcap};
+  const size_t smem = size_t(64 + 2 * kPK) * (Dp + kRowPad) * 2;
+  const dim3 grid(heads, ntiles);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  cudaError_t e;
+  if (Dp <= 32) e = launch_prefill<2>(p, grid, smem, st);
+  else if (Dp <= 64) e = launch_prefill<4>(p, grid, smem, st);
+  else if (Dp <= 128) e = launch_prefill<8>(p, grid, smem, st);
+  else e = launch_prefill<16>(p, grid, smem, st);
+  if (e != cudaSuccess) fprintf(stderr, "[tbvops] shared-row prefill launch failed: %s\n", cudaGetErrorString(e));
+  return e == cudaSuccess ? 0 : -1;
+}
+
+}  // extern "C"

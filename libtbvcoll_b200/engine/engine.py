@@ -188,7 +188,9 @@ class Engine:
             if hb.n_rows_form:
                 b.attn_splits = self.attn_splits_for(hb.n_rows_form, int(hb.pos[: hb.n_rows_form].max()) + 1)
             if hb.n_rows_form < T:
-                b.dense_tiles, b.dense_slots = put(hb.dense_tiles, np.int32), put(hb.dense_slots, np.int64)
+                b.dense_tiles = put(hb.dense_tiles, np.int32)
+                if m.expands_context:
+                    b.dense_slots = put(hb.dense_slots, np.int64)
         elif self.tiled_prefill_attention:
             b.tiles = ops.prefill_tiles(torch.from_numpy(hb.seq.astype(np.int32)), m.nq // m.nkv).to(dev)
         return b

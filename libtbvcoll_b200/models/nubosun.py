@@ -34,6 +34,7 @@ class Nubosun:
     # portions of at most this many tokens take the attention's rows form
     ROWS_FORM_MAX = 32
     uses_state = True
+    expands_context = True
 
     @staticmethod
     def attn_cta_slots(splits: int, sms: int) -> int:

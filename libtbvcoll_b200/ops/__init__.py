@@ -33,8 +33,17 @@ def lib():
     I, F, LL, SZ = ctypes.c_int, ctypes.c_float, ctypes.c_longlong, ctypes.c_size_t
     l.tbv_op_gemm.argtypes = [c_vp, c_vp, c_vp, c_vp, I, I, I, I, I, I, I, c_vp]
     l.tbv_op_gemm_error.restype = I
-    l.tbv_op_gemm_ex.argtypes = [c_vp, c_vp, c_vp, c_vp, c_vp, I, I, I, I, I, I, I, F, F, I, I, I, c_vp]
-    l.tbv_op_gemm_f32.argtypes = [c_vp, c_vp, c_vp, c_vp, I, I, I, I, I, I, I, F, F, I, I, I, c_vp]
+    l.tbv_op_gemm_ex.argtypes = [c_vp, c_vp, c_vp, c_vp, c_vp, I, I, I, I, I, I, I, F, F, F, I, I, I, I, c_vp]
+    l.tbv_op_gemm_f32.argtypes = [c_vp, c_vp, c_vp, c_vp, I, I, I, I, I, I, I, F, F, F, I, I, I, I, c_vp]
+    l.tbv_op_gemm_rows.argtypes = l.tbv_op_gemm_rows_f32.argtypes = [c_vp] * 4 + [I] * 8 + [F, F, F, c_vp]
+    l.tbv_op_residual.argtypes = [c_vp] * 4 + [F, LL] + [c_vp] * 8 + [I] + [c_vp] * 4 + [I, c_vp, I] + [c_vp] * 4 + [I] * 5 + [F, I, c_vp]
+    l.tbv_op_token_shift.argtypes = [c_vp] * 7 + [I] * 4 + [c_vp]
+    l.tbv_op_moe_route.argtypes = [c_vp] * 8 + [I] * 4 + [F, I, c_vp]
+    l.tbv_op_decay_scan.argtypes = [c_vp] * 14 + [I] * 10 + [F, F, F, I, c_vp]
+    l.tbv_op_decay_step.argtypes = [c_vp] * 13 + [I] * 9 + [F, F, F, I, c_vp]
+    l.tbv_op_shared_attn_prep.argtypes = [c_vp] * 6 + [I] * 8 + [F, F, ctypes.c_double, I, c_vp]
+    l.tbv_op_shared_attn_rows.argtypes = [c_vp] * 6 + [I] * 7 + [F, I, c_vp]
+    l.tbv_op_shared_attn_prefill.argtypes = [c_vp] * 6 + [I] * 8 + [F, c_vp]
     l.tbv_op_argmax_f32.argtypes = [c_vp, I, I, I, LL, c_vp, c_vp, c_vp, c_vp]
     l.tbv_op_hyper_embed.argtypes = [c_vp, c_vp, LL, F, c_vp, c_vp, c_vp, c_vp, I, I, I, I, I, F, I, c_vp]
     l.tbv_op_hyper_mix.argtypes = [c_vp, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp, I, I, I, I, I, I, F, I, c_vp]
@@ -115,7 +124,8 @@ def _count(n=1):
 
 
 EPI_STORE, EPI_SILU_MUL, EPI_F32, EPI_CLAMP_GLU = 0, 1, 2, 3
-ACT_NONE, ACT_SOFTPLUS, ACT_SOFTCAP = 0, 1, 2
+ACT_NONE, ACT_SOFTPLUS, ACT_SOFTCAP, ACT_TANH = 0, 1, 2, 3
+SILU_GLU = (math.inf, 1.0, 0.0)           # ``glu`` of ``linear``: silu(gate) * up
 
 
 def gemm(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None,
@@ -143,30 +153,49 @@ def gemm(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, b
 
 
 def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[torch.Tensor] = None, act: int = ACT_NONE, act_arg: float = 0.0,
-           glu: Optional[tuple] = None, copy: Optional[torch.Tensor] = None, groups: int = 1, x_group: int = 0, y_group: int = 0) -> torch.Tensor:
+           glu: Optional[tuple] = None, copy: Optional[torch.Tensor] = None, groups: int = 1, x_group: int = 0, y_group: int = 0,
+           last: int = 0) -> torch.Tensor:
     """out[N, M] = epilogue(x[N, K] @ w[M, K]^T + bias) for bf16 operands (tcgen05) or fp32 operands (CUDA cores, full 32-bit).
 
-    The output dtype is ``out``'s: fp32 results take an activation (``ACT_SOFTPLUS``, ``ACT_SOFTCAP`` with its limit in ``act_arg``)
-    and, from bf16 operands, an optional bf16 ``copy`` with the same row stride.  ``glu=(limit, slope)``: ``w`` holds gate / up rows
-    interleaved and out[N, M/2] = g * sigmoid(slope * g) * (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit).
-    ``groups`` > 1: w is [groups * M, K]; group g multiplies columns g * x_group .. of x and writes columns g * y_group .. of out."""
+    The output dtype is ``out``'s: fp32 results take an activation (``ACT_SOFTPLUS``, ``ACT_TANH``, ``ACT_SOFTCAP`` with its limit in ``act_arg``)
+    and, from bf16 operands, an optional bf16 ``copy`` with the same row stride.  ``glu=(limit, slope[, shift = 1])``: ``w`` holds gate / up rows
+    interleaved and out[N, M/2] = g * sigmoid(slope * g) * (u + shift) with g = min(gate, limit), u = clamp(up, -limit, limit).
+    ``groups`` > 1: w is [groups * M + last, K]; group g multiplies columns g * x_group .. of x and writes columns g * y_group .. of out; ``last``
+    features (0 = none) form one more group."""
     assert x.is_cuda and x.dtype is w.dtype and x.stride(1) == 1 and w.is_contiguous() and out.stride(1) == 1 and x.shape[0] == out.shape[0]
     N, K = x.shape[0], w.shape[1]
-    M = w.shape[0] // groups
+    assert groups > 1 or last == 0
+    M = (w.shape[0] - last) // groups
     assert x.shape[1] >= (groups - 1) * x_group + K and out.shape[1] >= (groups - 1) * y_group + (M // 2 if glu else M)
+    assert last == 0 or (x.shape[1] >= groups * x_group + K and out.shape[1] >= groups * y_group + last)
     if N == 0:
         return out
-    limit, slope = glu if glu else (act_arg, 0.0)
+    limit, slope, shift = (*glu, 1.0)[:3] if glu else (act_arg, 0.0, 0.0)
     if x.dtype is torch.float32:
         assert out.dtype is torch.float32 and copy is None and (bias is None or bias.dtype is torch.float32)
         _chk(lib().tbv_op_gemm_f32(_p(w), _p(x), _p(out), _p(bias), M, N, K, x.stride(0), out.stride(0), EPI_CLAMP_GLU if glu else EPI_F32, act,
-                                   limit, slope, groups, x_group, y_group, _st()), "tbv_op_gemm_f32")
+                                   limit, slope, shift, groups, x_group, y_group, last, _st()), "tbv_op_gemm_f32")
     else:
         epi = EPI_CLAMP_GLU if glu else (EPI_F32 if out.dtype is torch.float32 else EPI_STORE)
         assert x.dtype is torch.bfloat16 and (bias is None or bias.dtype is torch.bfloat16) and (epi == EPI_F32 or (act == ACT_NONE and copy is None))
         assert copy is None or (copy.dtype is torch.bfloat16 and copy.stride(0) == out.stride(0))
-        _chk(lib().tbv_op_gemm_ex(_p(w), _p(x), _p(out), _p(copy), _p(bias), M, N, K, x.stride(0), out.stride(0), epi, act, limit, slope,
-                                  groups, x_group, y_group, _st()), "tbv_op_gemm_ex")
+        _chk(lib().tbv_op_gemm_ex(_p(w), _p(x), _p(out), _p(copy), _p(bias), M, N, K, x.stride(0), out.stride(0), epi, act, limit, slope, shift,
+                                  groups, x_group, y_group, last, _st()), "tbv_op_gemm_ex")
+    _count()
+    return out
+
+
+def linear_rows(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, row_off: torch.Tensor, groups: int, max_rows: int,
+                glu: Optional[tuple] = None) -> torch.Tensor:
+    """Row-grouped product: rows row_off[g] .. row_off[g + 1] - 1 of x [R, K] (device int32 [groups + 1], at most max_rows per group) times rows
+    g * M .. of w [groups * M, K]; out [R, M], or the gated unit of ``linear`` [R, M / 2]."""
+    assert x.is_cuda and x.dtype is w.dtype is out.dtype and x.stride(1) == 1 and w.is_contiguous() and out.stride(1) == 1 and row_off.dtype is torch.int32
+    M, K = w.shape[0] // groups, w.shape[1]
+    assert x.shape[1] == K and x.shape[0] == out.shape[0] and out.shape[1] >= (M // 2 if glu else M) and row_off.shape[0] == groups + 1
+    limit, slope, shift = (*glu, 1.0)[:3] if glu else (0.0, 0.0, 0.0)
+    fn = lib().tbv_op_gemm_rows_f32 if x.dtype is torch.float32 else lib().tbv_op_gemm_rows
+    _chk(fn(_p(w), _p(x), _p(out), _p(row_off), groups, M, x.shape[0], max_rows, K, x.stride(0), out.stride(0), EPI_CLAMP_GLU if glu else EPI_STORE,
+            limit, slope, shift, _st()), "tbv_op_gemm_rows")
     _count()
     return out
 
@@ -410,5 +439,6 @@ def prefill_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
     return out
 
 
-from .mixers import (causal_conv_silu, hyper_embed, hyper_mix, latent_attention_prefill, latent_attention_rows, latent_gather,  # noqa: E402,F401
-                     latent_prefill_fits, latent_prep, latent_row, selective_scan)
+from .mixers import (SHARED_PREFILL_MAX_DIM, causal_conv_silu, decay_scan, decay_step, hyper_embed, hyper_mix,  # noqa: E402,F401
+                     latent_attention_prefill, latent_attention_rows, latent_gather, latent_prefill_fits, latent_prep, latent_row, moe_route,
+                     position_turns, residual, selective_scan, shared_attention_prefill, shared_attention_prep, shared_attention_rows, token_shift)

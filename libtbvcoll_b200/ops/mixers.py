@@ -1,11 +1,13 @@
-"""Entry points of the mixer operators: residual streams with hyper-connections, short convolution + selective scan over
-carried state, and attention over a compressed (latent) paged cache.  bf16 or fp32 activations; what enters a softmax, a
+"""Entry points of the mixer operators: residual streams with hyper-connections, one residual stream with parallel branches, short
+convolution + selective scan and linear recurrences over carried state, attention over a compressed (latent) paged cache and over
+a cache whose rows are keys and values at once, and the routing of a mixture of experts.  bf16 or fp32 activations; what enters a softmax, a
 norm, a recurrence or the residual sum is fp32 in both.
 
 ``segs`` is the device int32 [nseg, 4] list of a ragged batch: (first row, rows, state slot, 0) per sequence, rows of a
 sequence consecutive and in position order."""
 from __future__ import annotations
 
+import math
 from typing import Optional
 
 import torch
@@ -114,3 +116,128 @@ def latent_attention_prefill(qkv, q_rot_off: int, kv, kr, tiles, sink, out, head
     _chk(lib().tbv_op_latent_prefill(_p(qkv), _p(kv), _p(kr), _p(tiles), _p(sink), _p(out), tiles.shape[0], heads, qkv.stride(0), q_rot_off,
                                      kv.stride(0), heads * dim_p, out.stride(0), dim_p, kr.shape[1], v_p, scale, _st()), "tbv_op_latent_prefill")
     _count()
+
+
+# ---- one residual stream with parallel branches -----------------------------------------------------------------------------
+def position_turns(width: int, device, base: float = 10000.0) -> torch.Tensor:
+    """fp32 [ceil(width / 2), 2]: turns per position of every sine / cosine pair of the position vector, as high and low part."""
+    f = base ** (-2.0 * torch.arange((width + 1) // 2, dtype=torch.float64) / width) / (2.0 * math.pi)
+    hi = f.to(torch.float32)
+    return torch.stack((hi, (f - hi.double()).to(torch.float32)), 1).contiguous().to(device)
+
+
+def residual(x, g1, h1, width: int, eps: float, g2=None, h2=None, embed=None, positions=None, y1=None, y2=None, routed=None, x0=None, step=None,
+             rows: Optional[torch.Tensor] = None, last: bool = False, mix=None) -> None:
+    """x <- x + y1 + y2 + sum_j weight_j * routed_j (+ x0 + step);  h1 := RMSNorm(x) * g1,  h2 := RMSNorm(x) * g2.
+
+    x, y1, y2, x0 fp32 [rows, ld].  ``routed`` = (rows of the experts' results, place int32 [rows, top], weight fp32 [rows, top]).
+    ``embed`` = (ids, table, scale, turns): x := table[ids] * scale + position vector instead, kept in ``x0`` as well if that is given.
+    h1 may be fp32 beside bf16 activations.  ``last``: only the rows listed in ``rows`` (None = all) give an h1, packed, and x is not written.
+    ``mix`` = (mu fp32 [n, ld], mixes [rows, n * ld], shift fp32 [slots, ld], segs): one row per segment; instead of h1 its mixes
+    h1 + (previous h1 - h1) * mu_s are written, and shift is replaced."""
+    ld = x.shape[1]
+    n = h1.shape[0] if last else x.shape[0]
+    assert x.dtype is torch.float32 and x.is_contiguous() and (h2 is None or h2.stride(0) == h1.stride(0)) and (rows is None or (last and rows.dtype is torch.int64))
+    for t in (y1, y2, x0):
+        assert t is None or (t.dtype is torch.float32 and t.stride(0) == ld)
+    ids, table, scale, turns = embed if embed is not None else (None, None, 0.0, None)
+    ro, place, weight = routed if routed is not None else (None, None, None)
+    mu, mixes, shift, segs = mix if mix is not None else (None, None, None, None)
+    act = [t.dtype for t in (table, ro, h2, mixes) if t is not None] or [h1.dtype]
+    assert all(d is act[0] for d in act) and (h1.dtype is act[0] or h1.dtype is torch.float32)
+    assert ro is None or (ro.stride(0) == ld and place.dtype is torch.int32 and weight.dtype is torch.float32 and place.is_contiguous())
+    assert mu is None or (mixes.shape[1] == mu.shape[0] * ld and shift.shape[1] == ld and shift.dtype is torch.float32)
+    _chk(lib().tbv_op_residual(_p(ids), _p(table), _p(turns), _p(positions), scale, table.shape[0] if table is not None else 0, _p(x), _p(x0), _p(y1), _p(y2),
+                               _p(step), _p(ro), _p(place), _p(weight), place.shape[1] if place is not None else 0, _p(g1), _p(g2), _p(h1), _p(h2),
+                               int(h1.dtype is torch.float32), _p(rows), int(last), _p(mu), _p(mixes), _p(shift), _p(segs),
+                               mu.shape[0] if mu is not None else 0, n, width, ld, h1.stride(0), eps, int(act[0] is torch.bfloat16), _st()), "tbv_op_residual")
+    _count()
+
+
+def token_shift(h, mu, shift, mixes, segs, seg_of_row, positions) -> None:
+    """mixes[t] = n mixes of h_t (fp32 [rows, ld]) with h_{t-1}: h_t + (h_{t-1} - h_t) * mu_s; the row before a segment's first is shift[slot] (zeros at a
+    sequence's start).  shift is left as it is (``decay_scan`` replaces it)."""
+    n, ld = mu.shape
+    assert h.dtype is mu.dtype is shift.dtype is torch.float32 and h.is_contiguous() and mixes.is_contiguous() and mixes.shape[1] == n * ld
+    _chk(lib().tbv_op_token_shift(_p(h), _p(mu), _p(shift), _p(mixes), _p(segs), _p(seg_of_row), _p(positions), h.shape[0], ld, n, _is_bf16(mixes), _st()),
+         "tbv_op_token_shift")
+    _count()
+
+
+# ---- linear recurrences with a matrix state -----------------------------------------------------------------------------------
+def decay_scan(q, k, v, g, z, norm, state, o, out, segs, positions, vdim: int, eps: float, qscale: float = 1.0, tau: float = 1.0, u=None,
+               shift=None) -> None:
+    """Per head S_t = diag(a_t) S_{t-1} + k_t v_t^T over the rows of every segment, then out = RMSNorm(o) * norm * silu(g).
+    u None (gated linear attention): a = sigmoid(z)^(1 / tau), o_t = S_t^T (qscale q_t).  u fp32 [heads * Dp] (WKV): a = exp(-exp(z)),
+    o_t = (S_{t-1} + diag(u) k_t v_t^T)^T q_t.
+
+    q, k, v, g: column views [rows, heads * size] of one buffer; z fp32 [rows, heads * Dp]; state fp32 [slots, heads, Dp, Vp] is replaced;
+    o: fp32 scratch [rows, heads * Vp]; ``shift`` = (h fp32 [rows, ld], shift fp32 [slots, ld]): every segment's last row of h is kept."""
+    _, H, Dp, Vp = state.shape
+    rows = q.shape[0]
+    assert state.dtype is torch.float32 and z.dtype is torch.float32 and o.dtype is torch.float32 and o.numel() >= rows * H * Vp and q.dtype is out.dtype
+    assert q.stride(0) == k.stride(0) == v.stride(0) == g.stride(0) and q.shape[1] == k.shape[1] == H * Dp and v.shape[1] == g.shape[1] == H * Vp
+    h1, sh = shift if shift is not None else (None, None)
+    _chk(lib().tbv_op_decay_scan(_p(q), _p(k), _p(v), _p(g), _p(z), _p(u), _p(norm), _p(state), _p(o), _p(out), _p(h1), _p(sh), _p(segs), _p(positions),
+                                 rows, segs.shape[0], H, Dp, Vp, vdim, q.stride(0), z.stride(0), out.stride(0), h1.shape[1] if h1 is not None else 0,
+                                 qscale, tau, eps, _is_bf16(q), _st()), "tbv_op_decay_scan")
+    _count(2)
+
+
+def decay_step(q, k, v, g, low, w2, b2, norm, state, out, segs, positions, vdim: int, eps: float, qscale: float = 1.0, tau: float = 1.0, u=None) -> None:
+    """``decay_scan`` for one row per segment, with z = act(low) @ w2^T + b2 computed inside (act = tanh for WKV)."""
+    _, H, Dp, Vp = state.shape
+    rank = w2.shape[1]
+    assert state.dtype is torch.float32 and q.dtype is low.dtype is w2.dtype is b2.dtype is out.dtype and w2.shape[0] == H * Dp and low.shape[1] == rank
+    assert q.stride(0) == k.stride(0) == v.stride(0) == g.stride(0) and q.shape[1] == k.shape[1] == H * Dp and v.shape[1] == g.shape[1] == H * Vp
+    _chk(lib().tbv_op_decay_step(_p(q), _p(k), _p(v), _p(g), _p(low), _p(w2), _p(b2), _p(u), _p(norm), _p(state), _p(out), _p(segs), _p(positions),
+                                 segs.shape[0], H, Dp, Vp, vdim, q.stride(0), low.stride(0), rank, out.stride(0), qscale, tau, eps, _is_bf16(q), _st()),
+         "tbv_op_decay_step")
+    _count()
+
+
+# ---- attention whose cached rows are keys and values at once --------------------------------------------------------------------
+SHARED_PREFILL_MAX_DIM = 256          # padded head size that the prefill form takes
+
+
+def shared_attention_prep(qk, qa, cache, fold, positions, slots, n_rows_form: int, heads: int, kv_heads: int, dim: int, block_size: int, eps: float,
+                          temp_coef: float = 0.0, temp_every: float = 1.0) -> None:
+    """qk [rows, (heads + kv_heads) * Dp]: queries := RMSNorm(q) * (1 + coef * ln(floor((p + 1) / every) + 1)) * fold, to qa [n, heads, Dp + 8] for the first
+    n_rows_form rows and in place for the others; cache [blocks * kv_heads * block_size, Dp + 8] takes the key rows and their fp32 factor."""
+    Dp = fold.shape[0]
+    assert qk.dtype is qa.dtype is cache.dtype and cache.shape[1] == Dp + LATENT_ROW_PAD and slots.dtype is torch.int64 and positions.dtype is torch.int32
+    _chk(lib().tbv_op_shared_attn_prep(_p(qk), _p(qa), _p(cache), _p(fold), _p(positions), _p(slots), qk.shape[0], n_rows_form, qk.stride(0), heads, kv_heads,
+                                       dim, Dp, block_size, eps, temp_coef, temp_every, _is_bf16(qk), _st()), "tbv_op_shared_attn_prep")
+    _count()
+
+
+def shared_attention_rows(qa, cache, tables, seq_of_row, ctx_lens, out, kv_heads: int, block_size: int, softcap: float = 0.0, splits: int = 1) -> None:
+    """qa [rows, heads, Dp + 8] against the cached rows of each row's sequence; out [rows, heads, Dp]."""
+    rows, H, row = qa.shape
+    Dp = row - LATENT_ROW_PAD
+    assert qa.is_contiguous() and out.is_contiguous() and cache.shape[1] == row and qa.dtype is cache.dtype is out.dtype and out.shape[-1] * out.shape[-2] == H * Dp
+    assert tables.dtype is torch.int32 and ctx_lens.dtype is torch.int32
+    _chk(lib().tbv_op_shared_attn_rows(_p(qa), _p(cache), _p(tables), _p(seq_of_row), _p(ctx_lens), _p(out), rows, H, kv_heads, Dp, block_size,
+                                       tables.shape[1], splits, softcap, _is_bf16(qa), _st()), "tbv_op_shared_attn_rows")
+    _count()
+
+
+def shared_attention_prefill(q, cache, tables, seq_of_row, tiles, out, heads: int, kv_heads: int, block_size: int, softcap: float = 0.0) -> None:
+    """Many query rows q [rows, heads * Dp ..] in tiles int32 [n, 4] = (first row, rows <= 64, -, keys the first row sees); bf16."""
+    Dp = cache.shape[1] - LATENT_ROW_PAD
+    assert q.dtype is cache.dtype is out.dtype is torch.bfloat16 and tiles.dtype is torch.int32 and seq_of_row.dtype is torch.int32
+    _chk(lib().tbv_op_shared_attn_prefill(_p(q), _p(cache), _p(tables), _p(seq_of_row), _p(tiles), _p(out), tiles.shape[0], q.stride(0), out.stride(0), heads,
+                                          kv_heads, Dp, block_size, tables.shape[1], softcap, _st()), "tbv_op_shared_attn_prefill")
+    _count()
+
+
+# ---- mixture of experts -----------------------------------------------------------------------------------------------------------
+def moe_route(logits, h, xp, place, weight, offsets, counts, choice, experts: int, scale: float) -> None:
+    """Softmax over the first ``experts`` columns of logits (fp32 [T, ..]), the place.shape[1] largest chosen, their scores / (sum + 1e-20) * scale
+    to weight; h's rows copied to xp [T * top, ld], expert after expert: place int32 [T, top], offsets int32 [experts + 1].
+    counts [experts] and choice [T * top * 2] are int32 scratch."""
+    T, top = place.shape
+    assert logits.dtype is torch.float32 and h.is_contiguous() and xp.is_contiguous() and h.dtype is xp.dtype and h.shape[1] == xp.shape[1] and xp.shape[0] >= T * top
+    _chk(lib().tbv_op_moe_route(_p(logits), _p(h), _p(xp), _p(place), _p(weight), _p(offsets), _p(counts), _p(choice), T, experts, logits.stride(0), top, scale,
+                                h.shape[1] * h.element_size(), _st()), "tbv_op_moe_route")
+    _count(1 if T <= lib().tbv_op_moe_small() else 2)
