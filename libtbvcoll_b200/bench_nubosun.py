@@ -80,15 +80,16 @@ class _Kernels:
         self.rows = []
         self.sms = torch.cuda.get_device_properties(0).multi_processor_count
 
-    def time(self, group: str, name: str, make, bytes_, flops=0.0, exps=0.0):
-        """make(i) -> callable on the i-th set of operands; sets are made until they exceed the L2."""
+    def time(self, group: str, name: str, make, bytes_, flops=0.0, exps=0.0, fp32=0.0):
+        """make(i) -> callable on the i-th set of operands; sets are made until they exceed the L2.  ``exps`` run at 16, ``fp32`` instructions (FMA or
+        other) at 128 per clock and SM."""
         if self.only not in name:
             return
         from .bench_ops import time_graph
         torch.cuda.empty_cache()
         sets = max(2, min(64, math.ceil(400e6 / max(bytes_, 1.0))))
         us = time_graph([make(i) for i in range(sets)])
-        ideal = max(bytes_ / (self.hbm * 1e3), flops / (self.tf * 1e6), exps / (16 * self.sms * 1.965e3))
+        ideal = max(bytes_ / (self.hbm * 1e3), flops / (self.tf * 1e6), exps / (16 * self.sms * 1.965e3), fp32 / (128 * self.sms * 1.965e3))
         self.rows.append({"group": group, "kernel": name, "us": round(us, 2), "roofline_us": round(ideal, 2), "of_measured_peak": round(ideal / us, 3)})
 
 
@@ -272,8 +273,8 @@ def run(sizes, kernels=True, models=True, only="", case="") -> dict:
     return out
 
 
-def main() -> int:
-    ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
+def main(run=run, doc=__doc__) -> int:
+    ap = argparse.ArgumentParser(description=doc, formatter_class=argparse.RawDescriptionHelpFormatter)
     ap.add_argument("--sizes", default="2k,8b")
     ap.add_argument("--no-kernels", action="store_true")
     ap.add_argument("--no-models", action="store_true")

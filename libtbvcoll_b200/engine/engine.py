@@ -183,7 +183,9 @@ class Engine:
                       ctx=put(hb.pos + 1, np.int32), n_logits=int(hb.want_rows.size), seq_of_row=put(hb.seq, np.int32),
                       logit_rows=put(hb.want_rows, np.int64), out_tokens=out_tokens, logits_out=logits_out, n_rows_form=hb.n_rows_form)
         if m.uses_state:
-            b.segs, b.seg_of_row = put(hb.segs, np.int32), put(hb.seg, np.int32)
+            b.segs = put(hb.segs, np.int32)
+            if T > len(hb.segs):                   # otherwise one row per sequence: the models' one-token forms
+                b.seg_of_row = put(hb.seg, np.int32)
         if m.rows_form_max:
             if hb.n_rows_form:
                 b.attn_splits = self.attn_splits_for(hb.n_rows_form, int(hb.pos[: hb.n_rows_form].max()) + 1)
