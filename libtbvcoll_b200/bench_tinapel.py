@@ -19,7 +19,7 @@ TRIPLES = {"2k": ("tinapel-2k", "nubosun-2k", "llama3-2k"), "8b": ("tinapel-8b",
 def kernel_numbers(size: str, T: int, seqs: int, ctx: int, only: str = "") -> list:
     """T rows in ``seqs`` sequences: T == seqs is a decode step over ``ctx`` cached tokens, otherwise whole prompts."""
     from . import ops
-    from .engine.batch import dense_context
+    from .engine.batch import dense_context, scan_groups
     from .models.config import GlaSpec, SharedKvSpec, get_config
     from .models.tinapel import Tinapel
     cfg = get_config(TRIPLES[size][0])
@@ -76,8 +76,13 @@ def kernel_numbers(size: str, T: int, seqs: int, ctx: int, only: str = "") -> li
             if decode:
                 w2, b2 = _w(K, R), _w(K)
                 return lambda: ops.decay_step(q, kk, v, g, low, w2, b2, norm, st, out, segs, pos, vdim=r.vdim, eps=1e-5, tau=16.0, u=u)
+            model = Tinapel.__new__(Tinapel)           # its choice of groups only
+            model.dtype, model.scan_heads, model.device = bf, r.heads, dev
+            gr = scan_groups(segs.cpu().numpy(), model.scan_group_rows(segs[:, 1].cpu().numpy()))
+            cut, gr = len(gr) > seqs, torch.from_numpy(gr).to(dev)
+            scratch = (torch.empty(len(gr) * K * _pad16(r.vdim), device=dev), torch.empty(len(gr) * K, device=dev)) if cut else None
             z, o = torch.randn(T, K, device=dev), torch.empty(T, V, device=dev)
-            return lambda: ops.decay_scan(q, kk, v, g, z, norm, st, o, out, segs, pos, vdim=r.vdim, eps=1e-5, tau=16.0, u=u)
+            return lambda: ops.decay_scan(q, kk, v, g, z, norm, st, o, out, segs, pos, vdim=r.vdim, eps=1e-5, tau=16.0, u=u, groups=gr, scratch=scratch)
         state = seqs * K * r.vdim * 4
         if decode:
             k.time("scan", f"tinapel {name} step (decay product, norm, gate)", mk_rec, 2 * state + T * (2 * K + 3 * V + R) * 2 + K * R * 2)

@@ -1,0 +1,39 @@
+// decay.cuh — parameters and decays shared by the kernels of linear recurrences with a matrix state (decay_scan.cu, chunk_scan.cu).
+#pragma once
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+
+namespace decay_ops {
+
+struct ScanParams {
+  const void *q, *k, *v, *g;   // [rows, ld]: column h * Dp (q, k) or h * Vp (v, g) of each pointer
+  const float* z;              // [rows, ldz] decay inputs (many rows)
+  const void *low, *w2, *b2;   // one row: z = low . w2 + b2, low [rows, ldlow], w2 [heads * Dp, rank], b2 [heads * Dp]
+  const float* u;              // [heads * Dp]: WKV (null: gated linear attention)
+  const float* norm;           // [heads * Vp]
+  float* state;
+  float* o;                    // [rows, heads * Vp] (many rows)
+  void* out;                   // [rows, ldo]
+  const float* h1;             // [rows, ldh] inputs whose last row per segment goes to shift [slots, ldh] (null: none)
+  float* shift;
+  const int *segs, *positions;
+  int heads, Dp, Vp, vdim, ld, ldz, ldlow, rank, ldo, ldh;
+  float qscale, inv_tau, eps;
+};
+
+// decay of one key channel; bf16 models take the fast exponential and logarithm (1 + e^-|z| lies in 1 .. 2: absolute error about 1e-7)
+template <typename T> __device__ __forceinline__ float decay(float z, bool wkv, float inv_tau);
+template <> __device__ __forceinline__ float decay<float>(float z, bool wkv, float inv_tau) {
+  if (wkv) return expf(-expf(z));
+  return expf(-(fmaxf(-z, 0.f) + log1pf(expf(-fabsf(z)))) * inv_tau);
+}
+template <> __device__ __forceinline__ float decay<__nv_bfloat16>(float z, bool wkv, float inv_tau) {
+  if (wkv) return __expf(-__expf(z));
+  return __expf(-(fmaxf(-z, 0.f) + __logf(1.f + __expf(-fabsf(z)))) * inv_tau);
+}
+
+// chunk_scan.cu: the recurrence of a bf16 model over many rows.  groups [ngroups, 4]: (first row, rows, state slot, flags: 1 = a group of the same
+// segment precedes, 2 = one follows).
+cudaError_t chunk_scan(const ScanParams& p, const int* groups, int ngroups, bool multi, float* starts, float* totals, cudaStream_t st);
+
+}  // namespace decay_ops

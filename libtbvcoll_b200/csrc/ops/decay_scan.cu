@@ -8,6 +8,7 @@
 // and per head  out = o / rms(o) * weight * silu(gate).  A segment (first row, rows, state slot) may be a whole prompt, a portion or one
 // token; positions[first row] == 0 starts from zero whatever the slot holds.  State fp32 [slots, heads, Dp, Vp]; all of it is fp32 arithmetic.
 //
+//   chunk_scan.cu  many rows of bf16 models, on tensor cores; k_decay_scan is its 32-bit counterpart
 //   k_decay_scan   many rows: a CTA walks one segment for one head and a block of value columns.  A thread keeps KT keys x VT columns of S
 //                  in registers (packed pairs of keys); rows come in chunks whose decays are made once per chunk in shared memory.  The sums
 //                  over keys cross KG lanes by halving.  o goes to memory in fp32 and k_head_norm_gate finishes it.
@@ -20,39 +21,15 @@
 
 #include "../pdl.cuh"
 #include "attn_mma.cuh"
+#include "decay.cuh"
 #include "ops.h"
 #include "vec.cuh"
 
 using namespace vec;
+using decay_ops::decay;
+using decay_ops::ScanParams;
 
 namespace {
-
-struct ScanParams {
-  const void *q, *k, *v, *g;   // [rows, ld]: column h * Dp (q, k) or h * Vp (v, g) of each pointer
-  const float* z;              // [rows, ldz] decay inputs (many rows)
-  const void *low, *w2, *b2;   // one row: z = low . w2 + b2, low [rows, ldlow], w2 [heads * Dp, rank], b2 [heads * Dp]
-  const float* u;              // [heads * Dp]: WKV (null: gated linear attention)
-  const float* norm;           // [heads * Vp]
-  float* state;
-  float* o;                    // [rows, heads * Vp] (many rows)
-  void* out;                   // [rows, ldo]
-  const float* h1;             // [rows, ldh] inputs whose last row per segment goes to shift [slots, ldh] (null: none)
-  float* shift;
-  const int *segs, *positions;
-  int heads, Dp, Vp, vdim, ld, ldz, ldlow, rank, ldo, ldh;
-  float qscale, inv_tau, eps;
-};
-
-// decay of one key channel; bf16 models take the fast exponential and logarithm (1 + e^-|z| lies in 1 .. 2: absolute error about 1e-7)
-template <typename T> __device__ __forceinline__ float decay(float z, bool wkv, float inv_tau);
-template <> __device__ __forceinline__ float decay<float>(float z, bool wkv, float inv_tau) {
-  if (wkv) return expf(-expf(z));
-  return expf(-(fmaxf(-z, 0.f) + log1pf(expf(-fabsf(z)))) * inv_tau);
-}
-template <> __device__ __forceinline__ float decay<__nv_bfloat16>(float z, bool wkv, float inv_tau) {
-  if (wkv) return __expf(-__expf(z));
-  return __expf(-(fmaxf(-z, 0.f) + __logf(1.f + __expf(-fabsf(z)))) * inv_tau);
-}
 
 template <int DK, int COLS>
 struct ScanShape {
@@ -411,8 +388,11 @@ bool sizes_ok(int heads, int Dp, int Vp, int vdim) { return heads > 0 && heads <
 extern "C" {
 
 // Many rows per segment: recurrence (o fp32 scratch [rows, heads * Vp]), then head norm and gate.  u != null: WKV.  h1 / shift: see the top.
+// groups (bf16; null: the sequential kernel): the segments cut for the chunked kernels (chunk_scan.cu), [ngroups, 4]; `multi` tells whether any segment
+// has several; starts [ngroups, heads, Dp, Vp] and totals [ngroups, heads, Dp] fp32 are their scratch.
 int tbv_op_decay_scan(const void* q, const void* k, const void* v, const void* g, const void* z, const void* u, const void* norm, void* state,
-                      void* o, void* out, const void* h1, void* shift, const void* segs, const void* positions, int rows, int nseg, int heads, int Dp,
+                      void* o, void* out, const void* h1, void* shift, const void* segs, const void* positions, const void* groups, int ngroups, int multi,
+                      void* starts, void* totals, int rows, int nseg, int heads, int Dp,
                       int Vp, int vdim, int ld, int ldz, int ldo, int ldh, float qscale, float tau, float eps, int bf16, void* stream) {
   if (rows <= 0 || nseg <= 0) return 0;
   if (!sizes_ok(heads, Dp, Vp, vdim) || nseg > 65535 || (ld % 8) || (ldz % 8) || (ldo % 8) || !(tau > 0.f)) return -2;
@@ -423,7 +403,9 @@ int tbv_op_decay_scan(const void* q, const void* k, const void* v, const void* g
   p.heads = heads; p.Dp = Dp; p.Vp = Vp; p.vdim = vdim; p.ld = ld; p.ldz = ldz; p.ldo = ldo; p.ldh = ldh;
   p.qscale = qscale; p.inv_tau = 1.0f / tau; p.eps = eps;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  cudaError_t e = bf16 ? scan<__nv_bfloat16>(p, nseg, st) : scan<float>(p, nseg, st);
+  cudaError_t e;
+  if (bf16 && groups) e = decay_ops::chunk_scan(p, static_cast<const int*>(groups), ngroups, multi, static_cast<float*>(starts), static_cast<float*>(totals), st);
+  else e = bf16 ? scan<__nv_bfloat16>(p, nseg, st) : scan<float>(p, nseg, st);
   if (e == cudaSuccess) {
     const dim3 grid(unsigned(((long long)rows * heads + 7) / 8));
     e = bf16 ? pdl::launch(k_head_norm_gate<__nv_bfloat16>, grid, dim3(256), 0, st, 1, p, rows) : pdl::launch(k_head_norm_gate<float>, grid, dim3(256), 0, st, 1, p, rows);

@@ -40,6 +40,10 @@ class StepBatch:
     # models with carried state: int32 [nseg, 4] (first row, rows, state slot, 0) and the segment of every row (None: identity)
     segs: Optional[torch.Tensor] = None
     seg_of_row: Optional[torch.Tensor] = None
+    # the segments cut for chunked recurrences: int32 [n, 4] (first row, rows, state slot, flags: 1 = a group of the segment precedes, 2 = one
+    # follows); scan_cut: some segment has several
+    scan_groups: Optional[torch.Tensor] = None
+    scan_cut: bool = False
     # two-form attention: rows [0, n_rows_form) take the few-row form; the context of the others is expanded
     n_rows_form: int = 0
     dense_tiles: Optional[torch.Tensor] = None     # int32 [n, 4] (first row, rows <= 64, first context row, keys of the first row)
@@ -60,6 +64,15 @@ def dense_context(first_rows, counts, starts, rows, tables_host: np.ndarray, blo
     t = np.asarray(tiles, dtype=np.int32).reshape(-1, 4)
     t = t[np.argsort(-(t[:, 3] + t[:, 1]), kind="stable")]
     return t, np.concatenate(slots) if slots else np.zeros(0, dtype=np.int64)
+
+
+def scan_groups(segs: np.ndarray, group_rows: int) -> np.ndarray:
+    """Segments (first row, rows, slot, 0) cut into groups of at most ``group_rows`` rows (a multiple of the recurrences' chunk)."""
+    out = []
+    for first, n, slot, _ in segs.tolist():
+        for at in range(0, n, group_rows):
+            out.append((first + at, min(group_rows, n - at), slot, (1 if at else 0) | (2 if at + group_rows < n else 0)))
+    return np.asarray(out, dtype=np.int32).reshape(-1, 4)
 
 
 @dataclass

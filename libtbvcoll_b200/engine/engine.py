@@ -30,7 +30,7 @@ from .. import ops
 from ..models.registry import architecture_of
 from ..parallel.tp import TPGroup
 from ..utils.weights import RandomSource
-from .batch import Portion, StepBatch, lay_out
+from .batch import Portion, StepBatch, lay_out, scan_groups
 from .kv_cache import BlockManager, RequestTable
 
 
@@ -186,6 +186,10 @@ class Engine:
             b.segs = put(hb.segs, np.int32)
             if T > len(hb.segs):                   # otherwise one row per sequence: the models' one-token forms
                 b.seg_of_row = put(hb.seg, np.int32)
+                rows = m.scan_group_rows(hb.segs[:, 1])
+                if rows:
+                    groups = scan_groups(hb.segs, rows)
+                    b.scan_groups, b.scan_cut = put(groups, np.int32), len(groups) > len(hb.segs)
         if m.rows_form_max:
             if hb.n_rows_form:
                 b.attn_splits = self.attn_splits_for(hb.n_rows_form, int(hb.pos[: hb.n_rows_form].max()) + 1)

@@ -94,6 +94,11 @@ class Nubosun:
         self.l2_prefetch = os.environ.get("TBV_L2_PREFETCH", "1") != "0"
 
     @staticmethod
+    def scan_group_rows(rows) -> int:
+        """The selective scan takes whole segments."""
+        return 0
+
+    @staticmethod
     def load_weights(cfg: NubosunConfig, source, tp: TPGroup, device, dtype):
         from ..utils.weights import load_nubosun
         return load_nubosun(cfg, source, device, dtype)

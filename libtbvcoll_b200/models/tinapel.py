@@ -95,8 +95,29 @@ class Tinapel:
             self.state.append(None if attn else zeros(slots, m.heads, _pad16(m.dim), _pad16(getattr(m, "vdim", m.dim)), dt=f32))
             self.shift.append(zeros(slots, self.Wp, dt=f32) if isinstance(m, WkvSpec) else None)
         self.attn_ctas_per_row = max([m.kv_heads * ((m.heads // m.kv_heads + 15) // 16) for m in attns], default=1)
+        self.scan_heads = min([m.heads for _, m in recurrent], default=0)
+        self._groups = 0
         two_forms = bool(attns) and dtype is torch.bfloat16 and all(_pad16(m.dim) <= ops.SHARED_PREFILL_MAX_DIM for m in attns)
         self.rows_form_max = self.ROWS_FORM_MAX if two_forms else 1 << 60
+
+    def scan_group_rows(self, rows) -> int:
+        """Rows per group of the chunked recurrence for segments of the given lengths; 0: the sequential (32-bit) kernel.  Cutting a segment costs a
+        second pass over its keys and values, so it is done only as far as the GPU would otherwise be short of CTAs."""
+        if self.dtype is not torch.bfloat16 or not self.scan_heads:
+            return 0
+        sms = torch.cuda.get_device_properties(self.device).multi_processor_count
+        fair = max(256, -(-int(rows.sum()) * self.scan_heads // (2 * sms * 16)) * 16)
+        longest = -(-int(rows.max()) // 16) * 16
+        return longest if 2 * longest <= 3 * fair else fair
+
+    def _group_scratch(self, groups: int) -> tuple:
+        """(states, decay totals) of the groups of cut segments, grown on demand (never inside a captured step)."""
+        if groups > self._groups:
+            sizes = [(m.heads * _pad16(m.dim), _pad16(getattr(m, "vdim", m.dim))) for m in (l.mixer for l in self.cfg.layers) if not isinstance(m, SharedKvSpec)]
+            self._flat["starts"] = torch.empty(groups * max(k * v for k, v in sizes), dtype=torch.float32, device=self.device)
+            self._flat["totals"] = torch.empty(groups * max(k for k, _ in sizes), dtype=torch.float32, device=self.device)
+            self._groups = groups
+        return self._flat["starts"], self._flat["totals"]
 
     @staticmethod
     def load_weights(cfg: TinapelConfig, source, tp: TPGroup, device, dtype):
@@ -108,6 +129,11 @@ class Tinapel:
         for s in shape:
             n *= s
         return self._flat[name][:n].view(rows, *shape)
+
+    def _groups_of(self, b: StepBatch) -> dict:
+        if b.scan_groups is None:
+            return {}
+        return {"groups": b.scan_groups, "scratch": self._group_scratch(b.scan_groups.shape[0]) if b.scan_cut else None}
 
     # -- branches of a layer -------------------------------------------------------------------------
     def _gla(self, b: StepBatch, run: int, i: int, m: GlaSpec, y) -> None:
@@ -122,7 +148,7 @@ class Tinapel:
         else:
             z = self._buf("z", T, K)
             ops.linear(low, w[p + "decay"], z, bias=w[p + "decay.b"])
-            ops.decay_scan(q, k, v, g, z, w[p + "norm"], self.state[run], self._buf("o", T, V), out, b.segs, b.positions, **args)
+            ops.decay_scan(q, k, v, g, z, w[p + "norm"], self.state[run], self._buf("o", T, V), out, b.segs, b.positions, **args, **self._groups_of(b))
         ops.linear(out, w[p + "o"], y)
 
     def _wkv(self, b: StepBatch, run: int, i: int, m: WkvSpec, y) -> None:
@@ -146,7 +172,7 @@ class Tinapel:
             ops.linear(mixes[:, 4 * Wp:], w[p + "in"][4 * K:], lf, act=ops.ACT_TANH, copy=lh)
             ops.linear(lf if lh is None else lh, w[p + "decay"], z, bias=w[p + "decay.b"])
             ops.decay_scan(r, k, v, g, z, w[p + "norm"], self.state[run], self._buf("o", T, K), out, b.segs, b.positions,
-                           shift=(self.h1f[:T], self.shift[run]), **args)
+                           shift=(self.h1f[:T], self.shift[run]), **args, **self._groups_of(b))
         ops.linear(out, w[p + "o"], y)
 
     def _attention(self, b: StepBatch, run: int, i: int, m: SharedKvSpec, y) -> None:

@@ -39,7 +39,7 @@ def lib():
     l.tbv_op_residual.argtypes = [c_vp] * 4 + [F, LL] + [c_vp] * 8 + [I] + [c_vp] * 4 + [I, c_vp, I] + [c_vp] * 4 + [I] * 5 + [F, I, c_vp]
     l.tbv_op_token_shift.argtypes = [c_vp] * 7 + [I] * 4 + [c_vp]
     l.tbv_op_moe_route.argtypes = [c_vp] * 8 + [I] * 4 + [F, I, c_vp]
-    l.tbv_op_decay_scan.argtypes = [c_vp] * 14 + [I] * 10 + [F, F, F, I, c_vp]
+    l.tbv_op_decay_scan.argtypes = [c_vp] * 15 + [I, I, c_vp, c_vp] + [I] * 10 + [F, F, F, I, c_vp]
     l.tbv_op_decay_step.argtypes = [c_vp] * 13 + [I] * 9 + [F, F, F, I, c_vp]
     l.tbv_op_shared_attn_prep.argtypes = [c_vp] * 6 + [I] * 8 + [F, F, ctypes.c_double, I, c_vp]
     l.tbv_op_shared_attn_rows.argtypes = [c_vp] * 6 + [I] * 7 + [F, I, c_vp]
