@@ -697,6 +697,14 @@ int rows_form(RowsParams& p, int rows, int bf16, cudaStream_t st) {
 
 }  // namespace
 
+namespace tbvops {
+int shared_attn_rows_any(const void* qa, const void* cache, const int* tables, const int* seq_of_row, const int* ctx_lens, void* out, int rows,
+                         int heads, int kv_heads, int Dp, int block_size, int max_blocks, int splits, float softcap, int bf16, cudaStream_t st) {
+  RowsParams p{qa, cache, tables, seq_of_row, ctx_lens, nullptr, out, heads, Dp, Dp, 0, block_size, max_blocks, splits, kv_heads, kLog2e, 1.f, softcap, nullptr};
+  return rows_form<true>(p, rows, bf16, st);
+}
+}  // namespace tbvops
+
 extern "C" {
 
 int tbv_op_latent_prep(void* qkv, void* qa, void* cache, const void* gamma, const void* inv_freq, const void* positions, const void* slots,
@@ -719,17 +727,6 @@ int tbv_op_latent_attn_rows(const void* qa, const void* cache, const void* table
   RowsParams p{qa, cache, static_cast<const int*>(tables), static_cast<const int*>(seq_of_row), static_cast<const int*>(ctx_lens),
                static_cast<const float*>(sink), out, heads, R, Rp, rotp, block_size, max_blocks, splits, 1, scale * kLog2e, scale, 0.f, nullptr};
   return rows_form<false>(p, rows, bf16, static_cast<cudaStream_t>(stream));
-}
-
-// Keys that are values (see shared_attn.cu): qa [rows, heads, Dp + pad], cache [blocks, kv_heads, block_size, Dp + pad] with the row's score
-// factor as fp32 in the first pad places; softcap 0 = none.
-int tbv_op_shared_attn_rows(const void* qa, const void* cache, const void* tables, const void* seq_of_row, const void* ctx_lens, void* out,
-                            int rows, int heads, int kv_heads, int Dp, int block_size, int max_blocks, int splits, float softcap, int bf16,
-                            void* stream) {
-  if ((Dp % 16) || kv_heads <= 0 || heads % kv_heads) return -2;
-  RowsParams p{qa, cache, static_cast<const int*>(tables), static_cast<const int*>(seq_of_row), static_cast<const int*>(ctx_lens),
-               nullptr, out, heads, Dp, Dp, 0, block_size, max_blocks, splits, kv_heads, kLog2e, 1.f, softcap, nullptr};
-  return rows_form<true>(p, rows, bf16, static_cast<cudaStream_t>(stream));
 }
 
 int tbv_op_latent_gather(const void* cache, const void* slots, void* c, void* kr, int n, int Rp, int rotp, void* stream) {

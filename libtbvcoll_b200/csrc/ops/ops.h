@@ -1,6 +1,7 @@
 // ops.h — internal declarations shared by the operator translation units.
 #pragma once
 #include <cuda.h>
+#include <cuda_runtime.h>
 
 namespace gemm { struct Params; }
 
@@ -28,6 +29,9 @@ int gemm_tok_rows_choose(int M, int x_rows, int groups);
 bool gemm_streamk_wants(int M, int N, int K, int epi, int splits_hint, bool w_not_constant);
 int gemm_streamk_launch(const void* w, const void* x, void* y, const void* bias, int M, int N, int K, int ldx, int ldy, int epi,
                         void* stream);
+// rows form of attention over rows that are keys and values, any size and type (latent_attn.cu)
+int shared_attn_rows_any(const void* qa, const void* cache, const int* tables, const int* seq_of_row, const int* ctx_lens, void* out, int rows,
+                         int heads, int kv_heads, int Dp, int block_size, int max_blocks, int splits, float softcap, int bf16, cudaStream_t st);
 // threads per CTA for the row-normalisation kernels; the fused collective uses the same
 // mapping so that both produce identical bits
 inline int norm_threads(int hidden) {

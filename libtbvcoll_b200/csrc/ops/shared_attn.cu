@@ -6,7 +6,9 @@
 //   row = dim values | fp32 factor | pad          (dim padded to 16; eight places behind it, as in the latent cache)
 //   score(i, j) = cap * tanh((q'_i . row_j) * factor_j / cap),  q' = norm(q) * temperature * fold
 // Rows of a block lie together per key head ([blocks, kv_heads, block_size, dim + 8]), so that the rows form (latent_attn.cu, template KS)
-// brings a block in with one bulk copy.  Here: the kernel that normalises queries and writes cache rows, and the prefill form.
+// brings a block in with one bulk copy.  Here: the kernel that normalises queries and writes cache rows, the prefill form, and a rows form for heads
+// of up to 128 channels in which every warp walks blocks of its own: a row is small, so that the barriers of a CTA-wide tile would cost
+// more than its work.
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
@@ -14,6 +16,8 @@
 
 #include "../pdl.cuh"
 #include "attn_mma.cuh"
+#include "ops.h"
+#include "sm100.cuh"
 #include "vec.cuh"
 
 using namespace attn_mma;
@@ -66,6 +70,258 @@ __global__ void __launch_bounds__(256) k_shared_prep(const PrepParams p) {
   }
 }
 
+// ---- rows form ---------------------------------------------------------------------------------------------------------
+struct RowsParams {
+  const __nv_bfloat16 *qa, *cache;
+  __nv_bfloat16* out;       // [rows, heads, Dp]
+  const int *tables, *seq_of_row, *ctx_lens;
+  int heads, kv_heads, Dp, block_size, max_blocks, splits;
+  float softcap;
+  int* err;
+};
+
+// One row and up to 16 query heads of a key head per CTA; grid (rows, head tiles, splits), cluster (1, 1, splits).  Warp w takes the 32-token
+// units w, w + kWarps, .. of the CTA's token range through a ring of its own, filled by bulk copies of 16 tokens, with a running maximum of its own;
+// the warps' results are merged at the end, then those of the cluster, in fixed order.
+constexpr int kWarps = 4, kStages = 3, kMaxSplits = 8, kTok = 32;
+template <int NK>           // k steps of 16 channels (at most)
+__global__ void __launch_bounds__(kWarps * 32, 2) k_shared_rows(const RowsParams p) {
+  extern __shared__ __align__(128) uint8_t dsm[];
+  __shared__ unsigned long long full[kWarps][kStages];
+  __shared__ float sh_m[kWarps][16], sh_l[kWarps][16], sh_ml[16][2], sh_fac[kMaxSplits][16], sh_sm[kMaxSplits][16];
+  __shared__ int abort_flag;
+  pdl::launch_dependents();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r8 = lane >> 2, quad = lane & 3;
+  if (lane == 0) {
+    for (int s = 0; s < kStages; s++) sm100::mbar_init(smem_addr(&full[warp][s]), 1);
+    if (warp == 0) abort_flag = 0;
+    sm100::mbar_fence_init();
+  }
+  __syncthreads();
+  pdl::grid_dependency_wait();
+  const int row = blockIdx.x, sp = blockIdx.z, S = p.splits;
+  const int G = p.kv_heads, hpk = p.heads / G, tpg = (hpk + 15) / 16, g = blockIdx.y / tpg;
+  const int h0 = g * hpk + (blockIdx.y - g * tpg) * 16, nq = min(16, (g + 1) * hpk - h0);
+  const int ksteps = p.Dp / 16, rowlen = p.Dp + kRowPad, pitch = rowlen * 2;
+  const int ctx = min(p.ctx_lens[row], p.max_blocks * p.block_size);
+  const int* bt = p.tables + size_t(p.seq_of_row ? p.seq_of_row[row] : row) * p.max_blocks;
+  int chunk = (ctx + S - 1) / S;
+  chunk = (chunk + kTok - 1) / kTok * kTok;
+  const int t0 = min(ctx, sp * chunk), t1 = min(ctx, t0 + chunk);
+  const int units = (t1 - t0 + kTok - 1) / kTok, mine = units > warp ? (units - warp + kWarps - 1) / kWarps : 0;
+
+  // blocks of this warp's unit i: looked up for 16 units at a time, a lane per half unit
+  int entry = 0;
+  auto look_up = [&](int i0) {
+    const int tok = t0 + (warp + kWarps * (i0 + (lane >> 1))) * kTok + (lane & 1) * 16;
+    return tok < t1 ? bt[tok / p.block_size] : 0;
+  };
+  const uint32_t ring = smem_addr(dsm) + uint32_t(warp) * kStages * kTok * pitch;
+  auto issue = [&](int i) {               // whole warp; unit i of this warp into its stage
+    if (i >= mine) return;
+    if ((i & 15) == 0) entry = look_up(i);
+    const int block = __shfl_sync(0xffffffffu, entry, (i & 15) * 2 + (lane & 1));
+    const int tok = t0 + (warp + kWarps * i) * kTok, n = min(kTok, t1 - tok);
+    const uint32_t bar = smem_addr(&full[warp][i % kStages]);
+    if (lane == 0) sm100::mbar_expect_tx(bar, uint32_t(n) * pitch);
+    __syncwarp();
+    if (lane * 16 < n) {                   // lanes 0 and 1
+      const int tk = tok + lane * 16;
+      sm100::bulk_load(ring + ((i % kStages) * kTok + lane * 16) * pitch, p.cache + ((size_t(block) * G + g) * p.block_size + tk % p.block_size) * rowlen,
+                       uint32_t(min(16, n - lane * 16)) * pitch, bar);
+    }
+  };
+#pragma unroll
+  for (int i = 0; i < kStages; i++) issue(i);
+
+  uint32_t qf[NK][4];
+  const __nv_bfloat16* qa = p.qa + (size_t(row) * p.heads + h0) * rowlen + quad * 2;
+#pragma unroll
+  for (int k = 0; k < NK; k++)
+#pragma unroll
+    for (int j = 0; j < 4; j++) {
+      const int r = r8 + (j & 1) * 8;
+      qf[k][j] = k < ksteps && r < nq ? *reinterpret_cast<const uint32_t*>(qa + size_t(r) * rowlen + k * 16 + (j >> 1) * 8) : 0u;
+    }
+  float o[NK * 2][4];
+#pragma unroll
+  for (int n = 0; n < NK * 2; n++) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
+  float m_lo = kNegBig, m_hi = kNegBig, l_lo = 0.f, l_hi = 0.f;
+
+  int done = 0;
+  for (; done < mine; done++) {
+    const int i = done, n = min(kTok, t1 - t0 - (warp + kWarps * i) * kTok);
+    const uint32_t sk = ring + (i % kStages) * kTok * pitch;
+    if (!__all_sync(0xffffffffu, sm100::mbar_wait(smem_addr(&full[warp][i % kStages]), uint32_t(i / kStages) & 1u, &abort_flag, 2000000000ull))) break;
+    if (n < kTok) {                        // missing rows: a weight of zero must not meet a stale bit pattern
+      for (int r = n; r < kTok; r++)
+        for (int c = lane; c <= p.Dp / 8; c += 32) st_zero16(sk + r * pitch + c * 16);
+      __syncwarp();
+    }
+    float s[kTok / 8][4] = {};
+#pragma unroll
+    for (int k = 0; k < NK; k++)
+      if (k < ksteps) {
+#pragma unroll
+        for (int t = 0; t < kTok / 16; t++) {
+          uint32_t b[4];
+          ldmatrix_x4(sk + (t * 16 + (lane & 7) + ((lane >> 4) << 3)) * pitch + ((lane >> 3) & 1) * 16 + k * 32, b);
+          mma_bf16(s[2 * t], qf[k], b[0], b[1]);
+          mma_bf16(s[2 * t + 1], qf[k], b[2], b[3]);
+        }
+      }
+    float x_lo = m_lo, x_hi = m_hi;
+#pragma unroll
+    for (int t = 0; t < kTok / 8; t++)
+#pragma unroll
+      for (int j = 0; j < 2; j++) {
+        const int tok = t * 8 + quad * 2 + j;
+        float f;
+        asm volatile("ld.shared.f32 %0, [%1];" : "=f"(f) : "r"(sk + tok * pitch + p.Dp * 2) : "memory");
+        s[t][j] = tok < n ? capped_log2(s[t][j] * f, p.softcap) : kNegBig;
+        s[t][2 + j] = tok < n ? capped_log2(s[t][2 + j] * f, p.softcap) : kNegBig;
+        x_lo = fmaxf(x_lo, s[t][j]);
+        x_hi = fmaxf(x_hi, s[t][2 + j]);
+      }
+    x_lo = fmaxf(x_lo, __shfl_xor_sync(0xffffffffu, x_lo, 1));
+    x_lo = fmaxf(x_lo, __shfl_xor_sync(0xffffffffu, x_lo, 2));
+    x_hi = fmaxf(x_hi, __shfl_xor_sync(0xffffffffu, x_hi, 1));
+    x_hi = fmaxf(x_hi, __shfl_xor_sync(0xffffffffu, x_hi, 2));
+    if (__any_sync(0xffffffffu, x_lo > m_lo || x_hi > m_hi)) {
+      const float c_lo = exp2f(m_lo - x_lo), c_hi = exp2f(m_hi - x_hi);
+      m_lo = x_lo;
+      m_hi = x_hi;
+      l_lo *= c_lo;
+      l_hi *= c_hi;
+#pragma unroll
+      for (int d = 0; d < NK * 2; d++) { o[d][0] *= c_lo; o[d][1] *= c_lo; o[d][2] *= c_hi; o[d][3] *= c_hi; }
+    }
+    uint32_t pa[kTok / 16][4];
+#pragma unroll
+    for (int t = 0; t < kTok / 8; t++) {
+      const float p0 = exp2f(s[t][0] - m_lo), p1 = exp2f(s[t][1] - m_lo), p2 = exp2f(s[t][2] - m_hi), p3 = exp2f(s[t][3] - m_hi);
+      l_lo += p0 + p1;
+      l_hi += p2 + p3;
+      pa[t >> 1][(t & 1) * 2] = pack_bf16(p0, p1);
+      pa[t >> 1][(t & 1) * 2 + 1] = pack_bf16(p2, p3);
+    }
+#pragma unroll
+    for (int d = 0; d < NK; d++)
+      if (d < ksteps) {
+#pragma unroll
+        for (int t = 0; t < kTok / 16; t++) {
+          uint32_t v[4];
+          ldmatrix_x4_trans(sk + (t * 16 + (lane & 15)) * pitch + d * 32 + (lane >> 4) * 16, v);
+          mma_bf16(o[2 * d], pa[t], v[0], v[1]);
+          mma_bf16(o[2 * d + 1], pa[t], v[2], v[3]);
+        }
+      }
+    __syncwarp();
+    issue(i + kStages);
+  }
+  if (done < mine) {
+    // gave up: let the copies in flight land before this memory goes away, and report
+    for (int i = done; i < mine && i < done + kStages; i++)
+      for (int spin = 0; spin < 20000 && !sm100::mbar_try_wait(smem_addr(&full[warp][i % kStages]), uint32_t(i / kStages) & 1u); spin++) __nanosleep(50);
+    if (lane == 0) atomicExch(p.err, 1);
+  }
+  l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1);
+  l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
+  l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1);
+  l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
+  if (quad == 0) {
+    sh_m[warp][r8] = m_lo; sh_m[warp][r8 + 8] = m_hi;
+    sh_l[warp][r8] = l_lo; sh_l[warp][r8 + 8] = l_hi;
+  }
+  __syncthreads();                          // the rings are free: their space takes the warps' sums [warps][16][Dp]
+  float* so = reinterpret_cast<float*>(dsm);
+#pragma unroll
+  for (int d = 0; d < NK * 2; d++)
+    if (d < ksteps * 2) {
+      const int col = d * 8 + quad * 2;
+      if (r8 < nq) *reinterpret_cast<float2*>(so + (warp * 16 + r8) * p.Dp + col) = make_float2(o[d][0], o[d][1]);
+      if (r8 + 8 < nq) *reinterpret_cast<float2*>(so + (warp * 16 + r8 + 8) * p.Dp + col) = make_float2(o[d][2], o[d][3]);
+    }
+  if (tid < 16) {
+    float m = kNegBig, l = 0.f;
+#pragma unroll
+    for (int w = 0; w < kWarps; w++) m = fmaxf(m, sh_m[w][tid]);
+#pragma unroll
+    for (int w = 0; w < kWarps; w++) {
+      const float f = exp2f(sh_m[w][tid] - m);
+      l = fmaf(sh_l[w][tid], f, l);
+      sh_m[w][tid] = f;                     // factor of the warp from here on
+    }
+    sh_ml[tid][0] = m;
+    sh_ml[tid][1] = l;
+  }
+  __syncthreads();
+  __nv_bfloat16* out = p.out + (size_t(row) * p.heads + h0) * p.Dp;
+  const int total = nq * p.Dp / 4;
+  for (int i = tid; i < total; i += kWarps * 32) {
+    const int h = i * 4 / p.Dp;
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int w = 0; w < kWarps; w++) {
+      const float4 v = *reinterpret_cast<const float4*>(so + w * 16 * p.Dp + i * 4);
+      const float f = sh_m[w][h];
+      a.x = fmaf(v.x, f, a.x); a.y = fmaf(v.y, f, a.y); a.z = fmaf(v.z, f, a.z); a.w = fmaf(v.w, f, a.w);
+    }
+    if (S == 1) {
+      const float l = sh_ml[h][1], f = l > 0.f ? 1.f / l : 0.f;
+      *reinterpret_cast<uint2*>(out + i * 4) = make_uint2(pack_bf16(a.x * f, a.y * f), pack_bf16(a.z * f, a.w * f));
+    } else {
+      *reinterpret_cast<float4*>(so + i * 4) = a;
+    }
+  }
+  if (S == 1) return;
+  cluster_sync();
+  if (tid < 16 * kMaxSplits) {              // as many as there are threads
+    const int r = tid >> 4, h = tid & 15;
+    const uint32_t a = smem_addr(&sh_ml[h][0]);
+    sh_sm[r][h] = r < S ? ld_cluster_f32(a, r) : kNegBig;
+    sh_fac[r][h] = r < S ? ld_cluster_f32(a + 4, r) : 0.f;
+  }
+  __syncthreads();
+  if (tid < 16) {
+    float mx = kNegBig, l = 0.f;
+    for (int r = 0; r < S; r++) mx = fmaxf(mx, sh_sm[r][tid]);
+    for (int r = 0; r < S; r++) l = fmaf(sh_fac[r][tid], exp2f(sh_sm[r][tid] - mx), l);
+    for (int r = 0; r < S; r++) sh_fac[r][tid] = l > 0.f ? exp2f(sh_sm[r][tid] - mx) / l : 0.f;
+  }
+  __syncthreads();
+  const int per = (total + S - 1) / S;
+  const uint32_t soa = smem_addr(so);
+  for (int i = tid; i < per; i += kWarps * 32) {
+    const int idx = sp * per + i;
+    if (idx >= total) break;
+    const int h = idx * 4 / p.Dp;
+    float4 v[kMaxSplits], a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int r = 0; r < kMaxSplits; r++)
+      if (r < S) v[r] = ld_cluster_f32x4(soa + idx * 16, r);
+#pragma unroll
+    for (int r = 0; r < kMaxSplits; r++)
+      if (r < S) {
+        const float f = sh_fac[r][h];
+        a.x = fmaf(v[r].x, f, a.x); a.y = fmaf(v[r].y, f, a.y); a.z = fmaf(v[r].z, f, a.z); a.w = fmaf(v[r].w, f, a.w);
+      }
+    *reinterpret_cast<uint2*>(out + idx * 4) = make_uint2(pack_bf16(a.x, a.y), pack_bf16(a.z, a.w));
+  }
+  cluster_sync();                           // nobody leaves while a peer may still read its shared memory
+}
+
+template <int NK>
+cudaError_t launch_rows(const RowsParams& p, int rows, cudaStream_t st) {
+  static bool done = false;
+  const int pitch = (p.Dp + kRowPad) * 2;
+  const size_t ring = size_t(kWarps) * kStages * kTok * pitch, sums = size_t(kWarps) * 16 * p.Dp * 4, smem = ring > sums ? ring : sums;
+  cudaError_t e = allow_smem(k_shared_rows<NK>, smem, &done);
+  const dim3 grid(rows, p.kv_heads * ((p.heads / p.kv_heads + 15) / 16), p.splits);
+  return e != cudaSuccess ? e : pdl::launch(k_shared_rows<NK>, grid, dim3(kWarps * 32), smem, st, p.splits, p);
+}
+
+// ---- prefill form --------------------------------------------------------------------------------------------------------
 struct PrefillParams {
   const __nv_bfloat16* q;   // [rows, ldq], head h at h * Dp
   const __nv_bfloat16* cache;
@@ -241,6 +497,23 @@ int tbv_op_shared_attn_prep(void* qk, void* qa, void* cache, const void* fold, c
   const dim3 grid(unsigned(((long long)rows * (heads + kv_heads) + 7) / 8));
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   cudaError_t e = bf16 ? pdl::launch(k_shared_prep<__nv_bfloat16>, grid, dim3(256), 0, st, 1, p) : pdl::launch(k_shared_prep<float>, grid, dim3(256), 0, st, 1, p);
+  return e == cudaSuccess ? 0 : -1;
+}
+
+// qa [rows, heads, Dp + pad], cache [blocks, kv_heads, block_size, Dp + pad], softcap 0 = none; a row sees the first ctx_lens[row] tokens.
+int tbv_op_shared_attn_rows(const void* qa, const void* cache, const void* tables, const void* seq_of_row, const void* ctx_lens, void* out,
+                            int rows, int heads, int kv_heads, int Dp, int block_size, int max_blocks, int splits, float softcap, int bf16,
+                            void* stream) {
+  if (rows <= 0) return 0;
+  if ((Dp % 16) || Dp <= 0 || kv_heads <= 0 || heads % kv_heads || block_size <= 0) return -2;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const int *tb = static_cast<const int*>(tables), *sq = static_cast<const int*>(seq_of_row), *cl = static_cast<const int*>(ctx_lens);
+  if (!bf16 || Dp > 128 || (block_size % 16))
+    return tbvops::shared_attn_rows_any(qa, cache, tb, sq, cl, out, rows, heads, kv_heads, Dp, block_size, max_blocks, splits, softcap, bf16, st);
+  RowsParams p{static_cast<const __nv_bfloat16*>(qa), static_cast<const __nv_bfloat16*>(cache), static_cast<__nv_bfloat16*>(out), tb, sq, cl,
+               heads, kv_heads, Dp, block_size, max_blocks, splits < 1 ? 1 : (splits > kMaxSplits ? kMaxSplits : splits), softcap, tbvops::gemm_err_flag()};
+  cudaError_t e = Dp <= 32 ? launch_rows<2>(p, rows, st) : (Dp <= 64 ? launch_rows<4>(p, rows, st) : launch_rows<8>(p, rows, st));
+  if (e != cudaSuccess) fprintf(stderr, "[tbvops] shared-row attention launch failed: %s\n", cudaGetErrorString(e));
   return e == cudaSuccess ? 0 : -1;
 }
 

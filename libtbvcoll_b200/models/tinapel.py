@@ -38,8 +38,8 @@ class Tinapel:
 
     @staticmethod
     def attn_cta_slots(splits: int, sms: int) -> int:
-        """CTAs of the rows kernel that run at once: one per SM, but clusters of eight find only about four fifths of the SMs."""
-        return sms if splits < 8 else sms * 4 // 5
+        """CTAs of the rows kernel that run at once: two per SM, but clusters of eight find only about four fifths of the places."""
+        return 2 * sms if splits < 8 else 2 * sms * 4 // 5
 
     def __init__(self, cfg: TinapelConfig, tp: TPGroup, weights: Dict[str, torch.Tensor], device, max_tokens: int, max_batch: int,
                  num_blocks: int, block_size: int = 16, max_attn_splits: int = 8, dtype: torch.dtype = torch.bfloat16):
