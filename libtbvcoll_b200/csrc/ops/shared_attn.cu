@@ -82,9 +82,10 @@ struct RowsParams {
 
 // One row and up to 16 query heads of a key head per CTA; grid (rows, head tiles, splits), cluster (1, 1, splits).  Warp w takes the 32-token
 // units w, w + kWarps, .. of the CTA's token range through a ring of its own, filled by bulk copies of 16 tokens, with a running maximum of its own;
-// the warps' results are merged at the end, then those of the cluster, in fixed order.
+// the warps' results are merged at the end, then those of the cluster, in fixed order.  Tokens (scores) and channels (sums) sit on the M side of the
+// products and heads on the N side, eight at a time (NH times): four query heads per key head leave half of the columns idle, not three quarters.
 constexpr int kWarps = 4, kStages = 3, kMaxSplits = 8, kTok = 32;
-template <int NK>           // k steps of 16 channels (at most)
+template <int NK, int NH>   // k steps of 16 channels (at most), tiles of 8 heads
 __global__ void __launch_bounds__(kWarps * 32, 2) k_shared_rows(const RowsParams p) {
   extern __shared__ __align__(128) uint8_t dsm[];
   __shared__ unsigned long long full[kWarps][kStages];
@@ -134,19 +135,24 @@ __global__ void __launch_bounds__(kWarps * 32, 2) k_shared_rows(const RowsParams
 #pragma unroll
   for (int i = 0; i < kStages; i++) issue(i);
 
-  uint32_t qf[NK][4];
+  // right operand of the scores: q^T, channels x heads
+  uint32_t qf[NK][NH][2];
   const __nv_bfloat16* qa = p.qa + (size_t(row) * p.heads + h0) * rowlen + quad * 2;
 #pragma unroll
   for (int k = 0; k < NK; k++)
 #pragma unroll
-    for (int j = 0; j < 4; j++) {
-      const int r = r8 + (j & 1) * 8;
-      qf[k][j] = k < ksteps && r < nq ? *reinterpret_cast<const uint32_t*>(qa + size_t(r) * rowlen + k * 16 + (j >> 1) * 8) : 0u;
-    }
-  float o[NK * 2][4];
+    for (int t = 0; t < NH; t++)
 #pragma unroll
-  for (int n = 0; n < NK * 2; n++) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
-  float m_lo = kNegBig, m_hi = kNegBig, l_lo = 0.f, l_hi = 0.f;
+      for (int j = 0; j < 2; j++)
+        qf[k][t][j] = k < ksteps && t * 8 + r8 < nq ? *reinterpret_cast<const uint32_t*>(qa + size_t(t * 8 + r8) * rowlen + k * 16 + j * 8) : 0u;
+  float o[NK][NH][4];         // channels 16 k + r8 (+ 8), heads 8 t + 2 quad (+ 1)
+#pragma unroll
+  for (int k = 0; k < NK; k++)
+#pragma unroll
+    for (int t = 0; t < NH; t++) o[k][t][0] = o[k][t][1] = o[k][t][2] = o[k][t][3] = 0.f;
+  float m[NH][2], l[NH][2];
+#pragma unroll
+  for (int t = 0; t < NH; t++) { m[t][0] = m[t][1] = kNegBig; l[t][0] = l[t][1] = 0.f; }
 
   int done = 0;
   for (; done < mine; done++) {
@@ -158,62 +164,81 @@ __global__ void __launch_bounds__(kWarps * 32, 2) k_shared_rows(const RowsParams
         for (int c = lane; c <= p.Dp / 8; c += 32) st_zero16(sk + r * pitch + c * 16);
       __syncwarp();
     }
-    float s[kTok / 8][4] = {};
+    float s[kTok / 16][NH][4] = {};       // tokens 16 x + r8 (+ 8), heads as in o
 #pragma unroll
     for (int k = 0; k < NK; k++)
       if (k < ksteps) {
 #pragma unroll
-        for (int t = 0; t < kTok / 16; t++) {
-          uint32_t b[4];
-          ldmatrix_x4(sk + (t * 16 + (lane & 7) + ((lane >> 4) << 3)) * pitch + ((lane >> 3) & 1) * 16 + k * 32, b);
-          mma_bf16(s[2 * t], qf[k], b[0], b[1]);
-          mma_bf16(s[2 * t + 1], qf[k], b[2], b[3]);
+        for (int x = 0; x < kTok / 16; x++) {
+          uint32_t a[4];
+          ldmatrix_x4(sk + (x * 16 + (lane & 15)) * pitch + (lane >> 4) * 16 + k * 32, a);
+#pragma unroll
+          for (int t = 0; t < NH; t++) mma_bf16(s[x][t], a, qf[k][t][0], qf[k][t][1]);
         }
       }
-    float x_lo = m_lo, x_hi = m_hi;
+    float mx[NH][2];
 #pragma unroll
-    for (int t = 0; t < kTok / 8; t++)
+    for (int t = 0; t < NH; t++) { mx[t][0] = m[t][0]; mx[t][1] = m[t][1]; }
 #pragma unroll
-      for (int j = 0; j < 2; j++) {
-        const int tok = t * 8 + quad * 2 + j;
+    for (int x = 0; x < kTok / 16; x++)
+#pragma unroll
+      for (int r = 0; r < 2; r++) {
+        const int tok = x * 16 + r * 8 + r8;
         float f;
         asm volatile("ld.shared.f32 %0, [%1];" : "=f"(f) : "r"(sk + tok * pitch + p.Dp * 2) : "memory");
-        s[t][j] = tok < n ? capped_log2(s[t][j] * f, p.softcap) : kNegBig;
-        s[t][2 + j] = tok < n ? capped_log2(s[t][2 + j] * f, p.softcap) : kNegBig;
-        x_lo = fmaxf(x_lo, s[t][j]);
-        x_hi = fmaxf(x_hi, s[t][2 + j]);
+#pragma unroll
+        for (int t = 0; t < NH; t++)
+#pragma unroll
+          for (int j = 0; j < 2; j++) {
+            float& v = s[x][t][2 * r + j];
+            v = tok < n ? capped_log2(v * f, p.softcap) : kNegBig;
+            mx[t][j] = fmaxf(mx[t][j], v);
+          }
       }
-    x_lo = fmaxf(x_lo, __shfl_xor_sync(0xffffffffu, x_lo, 1));
-    x_lo = fmaxf(x_lo, __shfl_xor_sync(0xffffffffu, x_lo, 2));
-    x_hi = fmaxf(x_hi, __shfl_xor_sync(0xffffffffu, x_hi, 1));
-    x_hi = fmaxf(x_hi, __shfl_xor_sync(0xffffffffu, x_hi, 2));
-    if (__any_sync(0xffffffffu, x_lo > m_lo || x_hi > m_hi)) {
-      const float c_lo = exp2f(m_lo - x_lo), c_hi = exp2f(m_hi - x_hi);
-      m_lo = x_lo;
-      m_hi = x_hi;
-      l_lo *= c_lo;
-      l_hi *= c_hi;
+    bool grew = false;
 #pragma unroll
-      for (int d = 0; d < NK * 2; d++) { o[d][0] *= c_lo; o[d][1] *= c_lo; o[d][2] *= c_hi; o[d][3] *= c_hi; }
+    for (int t = 0; t < NH; t++)
+#pragma unroll
+      for (int j = 0; j < 2; j++) {
+        mx[t][j] = fmaxf(mx[t][j], __shfl_xor_sync(0xffffffffu, mx[t][j], 4));
+        mx[t][j] = fmaxf(mx[t][j], __shfl_xor_sync(0xffffffffu, mx[t][j], 8));
+        mx[t][j] = fmaxf(mx[t][j], __shfl_xor_sync(0xffffffffu, mx[t][j], 16));
+        grew |= mx[t][j] > m[t][j];
+      }
+    if (__any_sync(0xffffffffu, grew)) {
+#pragma unroll
+      for (int t = 0; t < NH; t++)
+#pragma unroll
+        for (int j = 0; j < 2; j++) {
+          const float c = exp2f(m[t][j] - mx[t][j]);
+          m[t][j] = mx[t][j];
+          l[t][j] *= c;
+#pragma unroll
+          for (int k = 0; k < NK; k++) { o[k][t][j] *= c; o[k][t][2 + j] *= c; }
+        }
     }
-    uint32_t pa[kTok / 16][4];
+    // weights as the right operand of the sums (tokens x heads): the accumulator tiles transposed
+    uint32_t w[kTok / 16][NH][2];
 #pragma unroll
-    for (int t = 0; t < kTok / 8; t++) {
-      const float p0 = exp2f(s[t][0] - m_lo), p1 = exp2f(s[t][1] - m_lo), p2 = exp2f(s[t][2] - m_hi), p3 = exp2f(s[t][3] - m_hi);
-      l_lo += p0 + p1;
-      l_hi += p2 + p3;
-      pa[t >> 1][(t & 1) * 2] = pack_bf16(p0, p1);
-      pa[t >> 1][(t & 1) * 2 + 1] = pack_bf16(p2, p3);
-    }
+    for (int x = 0; x < kTok / 16; x++)
 #pragma unroll
-    for (int d = 0; d < NK; d++)
-      if (d < ksteps) {
+      for (int t = 0; t < NH; t++)
 #pragma unroll
-        for (int t = 0; t < kTok / 16; t++) {
-          uint32_t v[4];
-          ldmatrix_x4_trans(sk + (t * 16 + (lane & 15)) * pitch + d * 32 + (lane >> 4) * 16, v);
-          mma_bf16(o[2 * d], pa[t], v[0], v[1]);
-          mma_bf16(o[2 * d + 1], pa[t], v[2], v[3]);
+        for (int r = 0; r < 2; r++) {
+          const float p0 = exp2f(s[x][t][2 * r] - m[t][0]), p1 = exp2f(s[x][t][2 * r + 1] - m[t][1]);
+          l[t][0] += p0;
+          l[t][1] += p1;
+          w[x][t][r] = transpose_8x8(pack_bf16(p0, p1));
+        }
+#pragma unroll
+    for (int k = 0; k < NK; k++)
+      if (k < ksteps) {
+#pragma unroll
+        for (int x = 0; x < kTok / 16; x++) {
+          uint32_t a[4];               // values transposed: channels x tokens
+          ldmatrix_x4_trans(sk + (x * 16 + (lane & 7) + ((lane >> 4) << 3)) * pitch + k * 32 + ((lane >> 3) & 1) * 16, a);
+#pragma unroll
+          for (int t = 0; t < NH; t++) mma_bf16(o[k][t], a, w[x][t][0], w[x][t][1]);
         }
       }
     __syncwarp();
@@ -225,24 +250,32 @@ __global__ void __launch_bounds__(kWarps * 32, 2) k_shared_rows(const RowsParams
       for (int spin = 0; spin < 20000 && !sm100::mbar_try_wait(smem_addr(&full[warp][i % kStages]), uint32_t(i / kStages) & 1u); spin++) __nanosleep(50);
     if (lane == 0) atomicExch(p.err, 1);
   }
-  l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1);
-  l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
-  l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1);
-  l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
-  if (quad == 0) {
-    sh_m[warp][r8] = m_lo; sh_m[warp][r8 + 8] = m_hi;
-    sh_l[warp][r8] = l_lo; sh_l[warp][r8 + 8] = l_hi;
-  }
+#pragma unroll
+  for (int t = 0; t < NH; t++)
+#pragma unroll
+    for (int j = 0; j < 2; j++) {
+      l[t][j] += __shfl_xor_sync(0xffffffffu, l[t][j], 4);
+      l[t][j] += __shfl_xor_sync(0xffffffffu, l[t][j], 8);
+      l[t][j] += __shfl_xor_sync(0xffffffffu, l[t][j], 16);
+      if (r8 == 0) {
+        sh_m[warp][t * 8 + quad * 2 + j] = m[t][j];
+        sh_l[warp][t * 8 + quad * 2 + j] = l[t][j];
+      }
+    }
   __syncthreads();                          // the rings are free: their space takes the warps' sums [warps][16][Dp]
   float* so = reinterpret_cast<float*>(dsm);
 #pragma unroll
-  for (int d = 0; d < NK * 2; d++)
-    if (d < ksteps * 2) {
-      const int col = d * 8 + quad * 2;
-      if (r8 < nq) *reinterpret_cast<float2*>(so + (warp * 16 + r8) * p.Dp + col) = make_float2(o[d][0], o[d][1]);
-      if (r8 + 8 < nq) *reinterpret_cast<float2*>(so + (warp * 16 + r8 + 8) * p.Dp + col) = make_float2(o[d][2], o[d][3]);
+  for (int k = 0; k < NK; k++)
+    if (k < ksteps) {
+#pragma unroll
+      for (int t = 0; t < NH; t++)
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+          const int h = t * 8 + quad * 2 + (j & 1);
+          if (h < nq) so[(warp * 16 + h) * p.Dp + k * 16 + r8 + (j >> 1) * 8] = o[k][t][j];
+        }
     }
-  if (tid < 16) {
+  if (tid < NH * 8) {
     float m = kNegBig, l = 0.f;
 #pragma unroll
     for (int w = 0; w < kWarps; w++) m = fmaxf(m, sh_m[w][tid]);
@@ -279,8 +312,8 @@ __global__ void __launch_bounds__(kWarps * 32, 2) k_shared_rows(const RowsParams
   if (tid < 16 * kMaxSplits) {              // as many as there are threads
     const int r = tid >> 4, h = tid & 15;
     const uint32_t a = smem_addr(&sh_ml[h][0]);
-    sh_sm[r][h] = r < S ? ld_cluster_f32(a, r) : kNegBig;
-    sh_fac[r][h] = r < S ? ld_cluster_f32(a + 4, r) : 0.f;
+    sh_sm[r][h] = r < S && h < nq ? ld_cluster_f32(a, r) : kNegBig;
+    sh_fac[r][h] = r < S && h < nq ? ld_cluster_f32(a + 4, r) : 0.f;
   }
   __syncthreads();
   if (tid < 16) {
@@ -311,14 +344,14 @@ __global__ void __launch_bounds__(kWarps * 32, 2) k_shared_rows(const RowsParams
   cluster_sync();                           // nobody leaves while a peer may still read its shared memory
 }
 
-template <int NK>
+template <int NK, int NH>
 cudaError_t launch_rows(const RowsParams& p, int rows, cudaStream_t st) {
   static bool done = false;
   const int pitch = (p.Dp + kRowPad) * 2;
   const size_t ring = size_t(kWarps) * kStages * kTok * pitch, sums = size_t(kWarps) * 16 * p.Dp * 4, smem = ring > sums ? ring : sums;
-  cudaError_t e = allow_smem(k_shared_rows<NK>, smem, &done);
+  cudaError_t e = allow_smem(k_shared_rows<NK, NH>, smem, &done);
   const dim3 grid(rows, p.kv_heads * ((p.heads / p.kv_heads + 15) / 16), p.splits);
-  return e != cudaSuccess ? e : pdl::launch(k_shared_rows<NK>, grid, dim3(kWarps * 32), smem, st, p.splits, p);
+  return e != cudaSuccess ? e : pdl::launch(k_shared_rows<NK, NH>, grid, dim3(kWarps * 32), smem, st, p.splits, p);
 }
 
 // ---- prefill form --------------------------------------------------------------------------------------------------------
@@ -512,7 +545,9 @@ int tbv_op_shared_attn_rows(const void* qa, const void* cache, const void* table
     return tbvops::shared_attn_rows_any(qa, cache, tb, sq, cl, out, rows, heads, kv_heads, Dp, block_size, max_blocks, splits, softcap, bf16, st);
   RowsParams p{static_cast<const __nv_bfloat16*>(qa), static_cast<const __nv_bfloat16*>(cache), static_cast<__nv_bfloat16*>(out), tb, sq, cl,
                heads, kv_heads, Dp, block_size, max_blocks, splits < 1 ? 1 : (splits > kMaxSplits ? kMaxSplits : splits), softcap, tbvops::gemm_err_flag()};
-  cudaError_t e = Dp <= 32 ? launch_rows<2>(p, rows, st) : (Dp <= 64 ? launch_rows<4>(p, rows, st) : launch_rows<8>(p, rows, st));
+  cudaError_t e;
+  if (heads / kv_heads <= 8) e = Dp <= 32 ? launch_rows<2, 1>(p, rows, st) : (Dp <= 64 ? launch_rows<4, 1>(p, rows, st) : launch_rows<8, 1>(p, rows, st));
+  else e = Dp <= 32 ? launch_rows<2, 2>(p, rows, st) : (Dp <= 64 ? launch_rows<4, 2>(p, rows, st) : launch_rows<8, 2>(p, rows, st));
   if (e != cudaSuccess) fprintf(stderr, "[tbvops] shared-row attention launch failed: %s\n", cudaGetErrorString(e));
   return e == cudaSuccess ? 0 : -1;
 }
