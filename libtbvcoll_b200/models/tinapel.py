@@ -14,6 +14,7 @@ norms of the next layer, in a decode step also its mixes with the previous token
 All buffers of a decode step are preallocated, so the step can be captured in a CUDA graph."""
 from __future__ import annotations
 
+import os
 from typing import Callable, Dict, Optional
 
 import torch
@@ -97,6 +98,7 @@ class Tinapel:
         self.attn_ctas_per_row = max([m.kv_heads * ((m.heads // m.kv_heads + 15) // 16) for m in attns], default=1)
         self.scan_heads = min([m.heads for _, m in recurrent], default=0)
         self._groups = 0
+        self.side = [torch.cuda.Stream(device=dev) for _ in range(2)] if os.environ.get("TBV_BRANCH_STREAMS", "1") != "0" and dev.type == "cuda" else []
         two_forms = bool(attns) and dtype is torch.bfloat16 and all(_pad16(m.dim) <= ops.SHARED_PREFILL_MAX_DIM for m in attns)
         self.rows_form_max = self.ROWS_FORM_MAX if two_forms else 1 << 60
 
@@ -188,8 +190,8 @@ class Tinapel:
             ops.shared_attention_prefill(qk, cache, b.tables, b.seq_of_row, b.dense_tiles, out, H, G, self.block_size, cap)
         ops.linear(out, w[p + "o"], y)
 
-    def _moe(self, b: StepBatch, i: int, f: MoeSpec, y):
-        """Shared expert -> y (None without one); returns the routed experts' results as ``ops.residual`` takes them."""
+    def _moe(self, b: StepBatch, i: int, f: MoeSpec) -> tuple:
+        """The routed experts' results as ``ops.residual`` takes them."""
         w, p, T, h = self.w, f"l{i}.mlp.", b.T, self.h2[: b.T]
         P, fp = T * f.top, _pad16(f.ff)
         logits = self._buf("router", T, _pad16(f.experts))
@@ -199,21 +201,38 @@ class Tinapel:
         ops.moe_route(logits, h, xp, place, weight, off, self.counts, self._flat["choice"], f.experts, f.scale)
         ops.linear_rows(xp, w[p + "gate_up"], act, off, f.experts, T, glu=ops.SILU_GLU)
         ops.linear_rows(act, w[p + "down"], routed, off, f.experts, T)
-        if f.shared_ff:
-            sh = self._buf("shared", T, _pad16(f.shared_ff))
-            ops.linear(h, w[p + "shared.gate_up"], sh, glu=ops.SILU_GLU)
-            ops.linear(sh, w[p + "shared.down"], y)
         return routed, place, weight
 
+    def _shared(self, b: StepBatch, i: int, f: MoeSpec, y) -> None:
+        p, sh = f"l{i}.mlp.shared.", self._buf("shared", b.T, _pad16(f.shared_ff))
+        ops.linear(self.h2[: b.T], self.w[p + "gate_up"], sh, glu=ops.SILU_GLU)
+        ops.linear(sh, self.w[p + "down"], y)
+
     def _layer(self, b: StepBatch, run: int, i: int) -> dict:
-        """Runs the branches of layer ``i``; returns their results as arguments of ``ops.residual``."""
+        """Runs the branches of layer ``i``; returns their results as arguments of ``ops.residual``.  In a captured step the branches are
+        parallel branches of the graph: each is a chain of kernels too small to fill the GPU."""
         lay, y1, y2 = self.cfg.layers[i], self.y1[: b.T], self.y2[: b.T]
         mixer = {GlaSpec: self._gla, WkvSpec: self._wkv, SharedKvSpec: self._attention}[type(lay.mixer)]
-        mixer(b, run, i, lay.mixer, y1)
-        if lay.mlp is None:
-            return dict(y1=y1)
-        routed = self._moe(b, i, lay.mlp, y2)
-        return dict(y1=y1, y2=y2 if lay.mlp.shared_ff else None, routed=routed)
+        out, branches = dict(y1=y1), []
+        if lay.mlp is not None:
+            branches.append(lambda: out.update(routed=self._moe(b, i, lay.mlp)))
+            if lay.mlp.shared_ff:
+                out["y2"] = y2
+                branches.append(lambda: self._shared(b, i, lay.mlp, y2))
+        if self.side and branches and torch.cuda.is_current_stream_capturing():
+            main = torch.cuda.current_stream(self.device)
+            for s, fn in zip(self.side, branches):
+                s.wait_stream(main)
+                with torch.cuda.stream(s):
+                    fn()
+            mixer(b, run, i, lay.mixer, y1)
+            for s, _ in zip(self.side, branches):
+                main.wait_stream(s)
+        else:
+            mixer(b, run, i, lay.mixer, y1)
+            for fn in branches:
+                fn()
+        return out
 
     # -- between layers --------------------------------------------------------------------------------
     def _enter(self, b: StepBatch, run: int, **terms) -> None:
