@@ -58,7 +58,6 @@ def kernel_numbers(size: str, T: int, seqs: int, ctx: int, only: str = "") -> li
     else:
         _linear(k, "gemm", "tinapel wkv r / k / v / gate, each", T, K, W)
         _linear(k, "gemm", "tinapel decay first (tanh, fp32 + copy)", T, R, W, f32=True, act=ops.ACT_TANH, copy=True)
-        _linear(k, "gemm", "tinapel decay second (fp32)", T, K, R, f32=True)
     _linear(k, "gemm", "tinapel attention q + k", T, (a.heads + a.kv_heads) * a.dim, W)
     _linear(k, "gemm", "tinapel mixer out (fp32)", T, W, V, f32=True)
     _linear(k, "gemm", "tinapel head (fp32)", min(T, seqs), _pad16(cfg.vocab_size), W, f32=True)
@@ -81,13 +80,13 @@ def kernel_numbers(size: str, T: int, seqs: int, ctx: int, only: str = "") -> li
             gr = scan_groups(segs.cpu().numpy(), model.scan_group_rows(segs[:, 1].cpu().numpy()))
             cut, gr = len(gr) > seqs, torch.from_numpy(gr).to(dev)
             scratch = (torch.empty(len(gr) * K * _pad16(r.vdim), device=dev), torch.empty(len(gr) * K, device=dev)) if cut else None
-            z, o = torch.randn(T, K, device=dev), torch.empty(T, V, device=dev)
-            return lambda: ops.decay_scan(q, kk, v, g, z, norm, st, o, out, segs, pos, vdim=r.vdim, eps=1e-5, tau=16.0, u=u, groups=gr, scratch=scratch)
+            w2, b2, o = _w(K, R), _w(K), torch.empty(T, V, device=dev)
+            return lambda: ops.decay_scan(q, kk, v, g, None, norm, st, o, out, segs, pos, vdim=r.vdim, eps=1e-5, tau=16.0, u=u, groups=gr, scratch=scratch, low=(low, w2, b2))
         state = seqs * K * r.vdim * 4
         if decode:
             k.time("scan", f"tinapel {name} step (decay product, norm, gate)", mk_rec, 2 * state + T * (2 * K + 3 * V + R) * 2 + K * R * 2)
         else:
-            k.time("scan", f"tinapel {name} recurrence + norm, gate", mk_rec, state + T * (2 * K + 3 * V) * 2 + T * K * 4, fp32=3.0 * T * K * r.vdim)
+            k.time("scan", f"tinapel {name} recurrence (decay product, norm, gate)", mk_rec, state + T * (2 * K + 3 * V + R) * 2 + K * R * 2, fp32=3.0 * T * K * r.vdim)
 
     # attention
     H, G, D = a.heads, a.kv_heads, _pad16(a.dim)

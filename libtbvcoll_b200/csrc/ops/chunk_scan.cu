@@ -11,6 +11,9 @@
 // also the left operand of the readout.  v is bf16 as it stands.  fp32 operands are carried as sums of bf16 numbers: k_s R_s as three (24 bits: the
 // state is updated as in fp32), q_t P_t, S and A as two for the readout, whose result is rounded to bf16 behind the head norm.
 //
+// The decay inputs come from memory (p.z) or from the low-rank product itself: z = low . w2^T + b2 for a chunk is a few products per warp with w2's
+// rows of the head in shared memory.  If a CTA owns all value columns of its head, head norm, weight and gate follow here as well.
+//
 // A CTA alternates between making a chunk's operands (elementwise, shared memory) and its products; two CTAs per SM overlap the two.
 // Long segments are cut into groups that run in parallel: states of all groups but a segment's last from zero (k_chunk_scan<true>), then the
 // states they start from (k_group_starts), then all outputs.
@@ -21,6 +24,7 @@
 #include "../pdl.cuh"
 #include "attn_mma.cuh"
 #include "decay.cuh"
+#include "vec.cuh"
 
 using namespace attn_mma;
 using decay_ops::decay;
@@ -51,7 +55,11 @@ struct Shape {
   static constexpr int oE = oRk + kC * DK * 2;                     // P_16                [DK] fp32
   static constexpr int oTri = oE + DK * 4;                         // triangles           [2 chunks][item warps][2][36] fp32
   static constexpr int oOff = oTri + 2 * kItemWarps * 72 * 4;      // the block between the halves [warps][64] fp32
-  static constexpr int kBytes = oOff + NW * 64 * 4;
+  static constexpr int kOPitch = NW * 16 + 4;                      // floats
+  static constexpr int oO = oOff + NW * 64 * 4;                    // o                   [16][opitch] fp32
+  static constexpr int oG = oO + kC * kOPitch * 4;                 // gates               [16][vpitch] bf16
+  static constexpr int oLow = oG + kC * kVPitch;                   // low                 [2 chunks][16][rank pitch], then w2 [DK][rank pitch]
+  static constexpr int bytes(int rank) { return oLow + (rank ? (2 * kC + DK) * (rank * 2 + 16) : 0); }
 };
 
 __device__ __forceinline__ float bf16_to_f(uint32_t bits) { return __uint_as_float(bits << 16); }
@@ -75,8 +83,8 @@ __device__ __forceinline__ void pack_split(float x, float y, uint32_t& hi, uint3
   lo = pack_bf16(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xffff0000u));
 }
 
-template <int DK, bool STATE_ONLY>
-__global__ void __launch_bounds__(Shape<DK>::NW * 32, DK > 128 ? 1 : 2) k_chunk_scan(const ScanParams p, const int* groups, float* starts, float* totals) {
+template <int DK, bool STATE_ONLY, bool LOW>
+__global__ void __launch_bounds__(Shape<DK>::NW * 32, DK > 128 ? 1 : (DK > 64 ? 2 : 3)) k_chunk_scan(const ScanParams p, const int* groups, float* starts, float* totals) {
   using S = Shape<DK>;
   constexpr int NW = S::NW, NI = S::NI, NT = NW * 32;
   extern __shared__ __align__(16) uint8_t sm[];
@@ -99,7 +107,7 @@ __global__ void __launch_bounds__(Shape<DK>::NW * 32, DK > 128 ? 1 : 2) k_chunk_
   // rows of chunk c on their way to shared memory; missing rows of v are zeros, the others' are left out when they are used
   auto issue = [&](int c) {
     const int at = c * kC, nt = min(kC, n - at), dch = p.Dp / 8, vch = min(NW * 16, p.Vp - vb) / 8;
-    for (int i = tid; i < nt * dch * 2; i += NT) {
+    if (!LOW) for (int i = tid; i < nt * dch * 2; i += NT) {
       const int t = i / (dch * 2), x = i - t * dch * 2;
       cp_async16(base + S::oZ + (t * DK + x * 4) * 4, zg + size_t(first + at + t) * p.ldz + x * 4);
     }
@@ -114,7 +122,70 @@ __global__ void __launch_bounds__(Shape<DK>::NW * 32, DK > 128 ? 1 : 2) k_chunk_
       if (t < nt) cp_async16(vbuf + t * S::kVPitch + x * 16, vg + size_t(first + at + t) * p.ld + x * 8);
       else st_zero16(vbuf + t * S::kVPitch + x * 16);
     }
-    cp_async_commit();
+  };
+  const int lpitch = p.rank * 2 + 16;
+  const uint32_t w2s = base + S::oLow + 2 * kC * lpitch;
+  auto issue_low = [&](int c) {
+    const int at = c * kC, nt = min(kC, n - at), ch = p.rank / 8;
+    for (int i = tid; i < nt * ch; i += NT) {
+      const int t = i / ch, x = i - t * ch;
+      cp_async16(base + S::oLow + ((c & 1) * kC + t) * lpitch + x * 16, static_cast<const __nv_bfloat16*>(p.low) + size_t(first + at + t) * p.ldlow + x * 8);
+    }
+  };
+  // decay inputs of chunk c: tokens x channels, 16 channels per warp and item
+  auto decay_product = [&](int c) {
+#pragma unroll
+    for (int it = 0; it < NI; it++) {
+      const int d0 = (warp + it * NW) * 16;
+      float acc[2][4] = {};
+      for (int ks = 0; ks < p.rank / 16; ks++) {
+        uint32_t a[4], b[4];
+        ldmatrix_x4(base + S::oLow + ((c & 1) * kC + (lane & 15)) * lpitch + (lane >> 4) * 16 + ks * 32, a);
+        ldmatrix_x4(w2s + (d0 + (lane & 7) + ((lane >> 4) << 3)) * lpitch + ((lane >> 3) & 1) * 16 + ks * 32, b);
+        mma_bf16(acc[0], a, b[0], b[1]);
+        mma_bf16(acc[1], a, b[2], b[3]);
+      }
+#pragma unroll
+      for (int i = 0; i < 2; i++) {
+        const int d = d0 + i * 8 + quad * 2;
+        float2 b = make_float2(0.f, 0.f);
+        if (d < p.Dp) b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(static_cast<const __nv_bfloat16*>(p.b2) + size_t(h) * p.Dp + d));
+        float* z = reinterpret_cast<float*>(sm + S::oZ) + r8 * DK + d;
+        *reinterpret_cast<float2*>(z) = make_float2(acc[i][0] + b.x, acc[i][1] + b.y);
+        *reinterpret_cast<float2*>(z + 8 * DK) = make_float2(acc[i][2] + b.x, acc[i][3] + b.y);
+      }
+    }
+  };
+  // head norm, weight and gate of chunk c, whose o lies in shared memory; a row per 2 NW lanes, 8 columns per lane
+  const bool fused = !STATE_ONLY && p.o == nullptr;
+  auto issue_gates = [&](int c) {
+    const int at = c * kC, nt = min(kC, n - at), vch = p.Vp / 8;
+    for (int i = tid; i < nt * vch; i += NT) {
+      const int t = i / vch, x = i - t * vch;
+      cp_async16(base + S::oG + t * S::kVPitch + x * 16, static_cast<const __nv_bfloat16*>(p.g) + size_t(first + at + t) * p.ld + size_t(h) * p.Vp + x * 8);
+    }
+  };
+  auto emit = [&](int c) {
+    const int t = tid / (2 * NW), v = tid % (2 * NW) * 8;
+    float f[8], ss = 0.f;
+    vec::load8(reinterpret_cast<const float*>(sm + S::oO) + t * S::kOPitch + v, f);
+    if (v >= p.Vp) {
+#pragma unroll
+      for (int e = 0; e < 8; e++) f[e] = 0.f;
+    }
+#pragma unroll
+    for (int e = 0; e < 8; e++) ss = fmaf(f[e], f[e], ss);
+#pragma unroll
+    for (int o = NW; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (c * kC + t < n && v < p.Vp) {
+      const float r = 1.0f / sqrtf(ss / float(p.vdim) + p.eps);
+      float g[8], w[8];
+      vec::load8(reinterpret_cast<const __nv_bfloat16*>(sm + S::oG + t * S::kVPitch) + v, g);
+      vec::load8(p.norm + size_t(h) * p.Vp + v, w);
+#pragma unroll
+      for (int e = 0; e < 8; e++) f[e] = f[e] * r * w[e] * vec::gate<__nv_bfloat16>(g[e]);
+      vec::store8(static_cast<__nv_bfloat16*>(p.out) + size_t(first + c * kC + t) * p.ldo + size_t(h) * p.Vp + v, f);
+    }
   };
 
   float etot[NI];
@@ -271,19 +342,38 @@ __global__ void __launch_bounds__(Shape<DK>::NW * 32, DK > 128 ? 1 : 2) k_chunk_
     for (int i = 0; i < 2; i++)
 #pragma unroll
       for (int j = 0; j < 4; j++) {
-        const int t = at + i * 8 + quad * 2 + (j & 1);
-        if (t < n) p.o[(size_t(first + t) * p.heads + h) * p.Vp + v0 + r8 + (j >> 1) * 8] = o[i][j];
+        const int t = i * 8 + quad * 2 + (j & 1), v = r8 + (j >> 1) * 8;
+        if (fused) reinterpret_cast<float*>(sm + S::oO)[t * S::kOPitch + warp * 16 + v] = o[i][j];
+        else if (at + t < n) p.o[(size_t(first + at + t) * p.heads + h) * p.Vp + v0 + v] = o[i][j];
       }
   };
 
   const int nc = (n + kC - 1) / kC;
+  if (LOW) {
+    const int ch = p.rank / 8;
+    for (int i = tid; i < p.Dp * ch; i += NT) {
+      const int d = i / ch, x = i - d * ch;
+      cp_async16(w2s + d * lpitch + x * 16, static_cast<const __nv_bfloat16*>(p.w2) + (size_t(h) * p.Dp + d) * p.rank + x * 8);
+    }
+    issue_low(0);
+    if (nc > 1) issue_low(1);
+  }
   issue(0);
+  cp_async_commit();
   cp_async_wait<0>();
   __syncthreads();
+  if (LOW) {
+    decay_product(0);
+    __syncthreads();
+  }
   prepare(0);
   __syncthreads();
   for (int c = 0; c < nc; c++) {
     if (c + 1 < nc) issue(c + 1);
+    if (LOW && c + 2 < nc) issue_low(c + 2);
+    if (fused && c > 0) issue_gates(c - 1);
+    cp_async_commit();
+    if (LOW && c + 1 < nc) decay_product(c + 1);
     if (mma_warp) {
       if (!STATE_ONLY) {
         if (c > 0) finish(c - 1);
@@ -345,11 +435,21 @@ __global__ void __launch_bounds__(Shape<DK>::NW * 32, DK > 128 ? 1 : 2) k_chunk_
     cp_async_wait<0>();
     __syncthreads();
     if (!STATE_ONLY) assemble(c);
+    if (fused && c > 0) emit(c - 1);
     if (c + 1 < nc) prepare(c + 1);
     __syncthreads();
   }
+  if (fused) {
+    issue_gates(nc - 1);
+    cp_async_commit();
+  }
+  if (mma_warp && !STATE_ONLY) finish(nc - 1);
+  if (fused) {
+    cp_async_wait<0>();
+    __syncthreads();
+    emit(nc - 1);
+  }
   if (mma_warp) {
-    if (!STATE_ONLY) finish(nc - 1);
     float* to = STATE_ONLY ? starts + (size_t(gi + 1) * p.heads + h) * hs : p.state + (size_t(slot) * p.heads + h) * hs;
     if (STATE_ONLY || !(flags & 2)) {
 #pragma unroll
@@ -399,34 +499,40 @@ __global__ void __launch_bounds__(256) k_group_starts(const ScanParams p, const 
   }
 }
 
-template <int DK, bool STATE_ONLY>
+template <int DK, bool STATE_ONLY, bool LOW>
 cudaError_t launch(const ScanParams& p, const int* groups, int ngroups, float* starts, float* totals, cudaStream_t st) {
   using S = Shape<DK>;
   static bool done = false;
-  cudaError_t e = allow_smem(k_chunk_scan<DK, STATE_ONLY>, S::kBytes, &done);
-  return e != cudaSuccess ? e : pdl::launch(k_chunk_scan<DK, STATE_ONLY>, dim3(ngroups, p.heads, (p.Vp / 16 + S::NW - 1) / S::NW), dim3(S::NW * 32), size_t(S::kBytes), st, 1, p,
+  const size_t smem = size_t(S::bytes(LOW ? p.rank : 0));
+  cudaError_t e = allow_smem(k_chunk_scan<DK, STATE_ONLY, LOW>, smem, &done);
+  return e != cudaSuccess ? e : pdl::launch(k_chunk_scan<DK, STATE_ONLY, LOW>, dim3(ngroups, p.heads, (p.Vp / 16 + S::NW - 1) / S::NW), dim3(S::NW * 32), smem, st, 1, p,
                                             groups, starts, totals);
 }
-template <int DK>
-cudaError_t run(const ScanParams& p, const int* groups, int ngroups, bool multi, float* starts, float* totals, cudaStream_t st) {
+template <int DK, bool LOW>
+cudaError_t run(ScanParams p, const int* groups, int ngroups, bool multi, float* starts, float* totals, bool* finished, cudaStream_t st) {
+  *finished = p.Vp <= Shape<DK>::NW * 16;
+  if (*finished) p.o = nullptr;
   cudaError_t e = cudaSuccess;
   if (multi) {
-    e = launch<DK, true>(p, groups, ngroups, starts, totals, st);
+    e = launch<DK, true, LOW>(p, groups, ngroups, starts, totals, st);
     if (e == cudaSuccess) e = pdl::launch(k_group_starts, dim3(ngroups, p.heads, (p.Dp * p.Vp / 4 + 255) / 256), dim3(256), 0, st, 1, p, groups, starts, static_cast<const float*>(totals));
   }
-  return e != cudaSuccess ? e : launch<DK, false>(p, groups, ngroups, starts, totals, st);
+  return e != cudaSuccess ? e : launch<DK, false, LOW>(p, groups, ngroups, starts, totals, st);
+}
+template <int DK>
+cudaError_t run(const ScanParams& p, const int* groups, int ngroups, bool multi, float* starts, float* totals, bool* finished, cudaStream_t st) {
+  return p.z ? run<DK, false>(p, groups, ngroups, multi, starts, totals, finished, st) : run<DK, true>(p, groups, ngroups, multi, starts, totals, finished, st);
 }
 
 }  // namespace
 
 namespace decay_ops {
 
-cudaError_t chunk_scan(const ScanParams& p, const int* groups, int ngroups, bool multi, float* starts, float* totals, cudaStream_t st) {
-  if (p.Dp <= 32) return run<32>(p, groups, ngroups, multi, starts, totals, st);
-  if (p.Dp <= 64) return run<64>(p, groups, ngroups, multi, starts, totals, st);
-  if (p.Dp <= 96) return run<96>(p, groups, ngroups, multi, starts, totals, st);
-  if (p.Dp <= 128) return run<128>(p, groups, ngroups, multi, starts, totals, st);
-  return run<256>(p, groups, ngroups, multi, starts, totals, st);
+cudaError_t chunk_scan(const ScanParams& p, const int* groups, int ngroups, bool multi, float* starts, float* totals, bool* finished, cudaStream_t st) {
+  if (p.Dp <= 32) return run<32>(p, groups, ngroups, multi, starts, totals, finished, st);
+  if (p.Dp <= 64) return run<64>(p, groups, ngroups, multi, starts, totals, finished, st);
+  if (p.Dp <= 128) return run<128>(p, groups, ngroups, multi, starts, totals, finished, st);
+  return run<256>(p, groups, ngroups, multi, starts, totals, finished, st);
 }
 
 }  // namespace decay_ops

@@ -8,7 +8,7 @@ namespace decay_ops {
 struct ScanParams {
   const void *q, *k, *v, *g;   // [rows, ld]: column h * Dp (q, k) or h * Vp (v, g) of each pointer
   const float* z;              // [rows, ldz] decay inputs (many rows)
-  const void *low, *w2, *b2;   // one row: z = low . w2 + b2, low [rows, ldlow], w2 [heads * Dp, rank], b2 [heads * Dp]
+  const void *low, *w2, *b2;   // or z = low . w2 + b2, low [rows, ldlow], w2 [heads * Dp, rank], b2 [heads * Dp]
   const float* u;              // [heads * Dp]: WKV (null: gated linear attention)
   const float* norm;           // [heads * Vp]
   float* state;
@@ -33,7 +33,9 @@ template <> __device__ __forceinline__ float decay<__nv_bfloat16>(float z, bool 
 }
 
 // chunk_scan.cu: the recurrence of a bf16 model over many rows.  groups [ngroups, 4]: (first row, rows, state slot, flags: 1 = a group of the same
-// segment precedes, 2 = one follows).
-cudaError_t chunk_scan(const ScanParams& p, const int* groups, int ngroups, bool multi, float* starts, float* totals, cudaStream_t st);
+// segment precedes, 2 = one follows).  p.z null: decay inputs from p.low, p.w2, p.b2 (p.low as it enters the product).  *finished: head norm and gate
+// are done too (p.out), otherwise o is left in p.o.
+constexpr int kMaxRank = 128;     // of the fused decay product
+cudaError_t chunk_scan(const ScanParams& p, const int* groups, int ngroups, bool multi, float* starts, float* totals, bool* finished, cudaStream_t st);
 
 }  // namespace decay_ops

@@ -389,24 +389,28 @@ extern "C" {
 
 // Many rows per segment: recurrence (o fp32 scratch [rows, heads * Vp]), then head norm and gate.  u != null: WKV.  h1 / shift: see the top.
 // groups (bf16; null: the sequential kernel): the segments cut for the chunked kernels (chunk_scan.cu), [ngroups, 4]; `multi` tells whether any segment
-// has several; starts [ngroups, heads, Dp, Vp] and totals [ngroups, heads, Dp] fp32 are their scratch.
+// has several; starts [ngroups, heads, Dp, Vp] and totals [ngroups, heads, Dp] fp32 are their scratch.  With groups, z may be null: then
+// z = low . w2 + b2 inside (low [rows, ldlow] as it enters the product, w2 [heads * Dp, rank], rank a multiple of 16 and at most 128).
 int tbv_op_decay_scan(const void* q, const void* k, const void* v, const void* g, const void* z, const void* u, const void* norm, void* state,
                       void* o, void* out, const void* h1, void* shift, const void* segs, const void* positions, const void* groups, int ngroups, int multi,
-                      void* starts, void* totals, int rows, int nseg, int heads, int Dp,
+                      void* starts, void* totals, const void* low, const void* w2, const void* b2, int ldlow, int rank, int rows, int nseg, int heads, int Dp,
                       int Vp, int vdim, int ld, int ldz, int ldo, int ldh, float qscale, float tau, float eps, int bf16, void* stream) {
   if (rows <= 0 || nseg <= 0) return 0;
   if (!sizes_ok(heads, Dp, Vp, vdim) || nseg > 65535 || (ld % 8) || (ldz % 8) || (ldo % 8) || !(tau > 0.f)) return -2;
+  if (!z && (!bf16 || !groups || rank <= 0 || (rank % 16) || rank > decay_ops::kMaxRank || (ldlow % 8))) return -2;
   ScanParams p{};
   p.q = q; p.k = k; p.v = v; p.g = g; p.z = static_cast<const float*>(z); p.u = static_cast<const float*>(u); p.norm = static_cast<const float*>(norm);
   p.state = static_cast<float*>(state); p.o = static_cast<float*>(o); p.out = out; p.h1 = static_cast<const float*>(h1); p.shift = static_cast<float*>(shift);
   p.segs = static_cast<const int*>(segs); p.positions = static_cast<const int*>(positions);
   p.heads = heads; p.Dp = Dp; p.Vp = Vp; p.vdim = vdim; p.ld = ld; p.ldz = ldz; p.ldo = ldo; p.ldh = ldh;
+  p.low = low; p.w2 = w2; p.b2 = b2; p.ldlow = ldlow; p.rank = rank;
   p.qscale = qscale; p.inv_tau = 1.0f / tau; p.eps = eps;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   cudaError_t e;
-  if (bf16 && groups) e = decay_ops::chunk_scan(p, static_cast<const int*>(groups), ngroups, multi, static_cast<float*>(starts), static_cast<float*>(totals), st);
+  bool finished = false;
+  if (bf16 && groups) e = decay_ops::chunk_scan(p, static_cast<const int*>(groups), ngroups, multi, static_cast<float*>(starts), static_cast<float*>(totals), &finished, st);
   else e = bf16 ? scan<__nv_bfloat16>(p, nseg, st) : scan<float>(p, nseg, st);
-  if (e == cudaSuccess) {
+  if (e == cudaSuccess && !finished) {
     const dim3 grid(unsigned(((long long)rows * heads + 7) / 8));
     e = bf16 ? pdl::launch(k_head_norm_gate<__nv_bfloat16>, grid, dim3(256), 0, st, 1, p, rows) : pdl::launch(k_head_norm_gate<float>, grid, dim3(256), 0, st, 1, p, rows);
   }

@@ -132,10 +132,17 @@ class Tinapel:
             n *= s
         return self._flat[name][:n].view(rows, *shape)
 
-    def _groups_of(self, b: StepBatch) -> dict:
-        if b.scan_groups is None:
-            return {}
-        return {"groups": b.scan_groups, "scratch": self._group_scratch(b.scan_groups.shape[0]) if b.scan_cut else None}
+    def _scan(self, b: StepBatch, run: int, p: str, q, k, v, g, low, V: int, out, args: dict) -> None:
+        """Recurrence over many rows; ``low`` is what enters the second decay product, which the chunked kernels do themselves."""
+        w, z = self.w, None
+        if b.scan_groups is not None:
+            args = {**args, "groups": b.scan_groups, "scratch": self._group_scratch(b.scan_groups.shape[0]) if b.scan_cut else None}
+        if b.scan_groups is not None and low.shape[1] <= ops.DECAY_RANK_MAX:
+            args["low"] = (low, w[p + "decay"], w[p + "decay.b"])
+        else:
+            z = self._buf("z", b.T, w[p + "decay"].shape[0])
+            ops.linear(low, w[p + "decay"], z, bias=w[p + "decay.b"])
+        ops.decay_scan(q, k, v, g, z, w[p + "norm"], self.state[run], self._buf("o", b.T, V), out, b.segs, b.positions, **args)
 
     # -- branches of a layer -------------------------------------------------------------------------
     def _gla(self, b: StepBatch, run: int, i: int, m: GlaSpec, y) -> None:
@@ -148,9 +155,7 @@ class Tinapel:
         if b.seg_of_row is None:
             ops.decay_step(q, k, v, g, low, w[p + "decay"], w[p + "decay.b"], w[p + "norm"], self.state[run], out, b.segs, b.positions, **args)
         else:
-            z = self._buf("z", T, K)
-            ops.linear(low, w[p + "decay"], z, bias=w[p + "decay.b"])
-            ops.decay_scan(q, k, v, g, z, w[p + "norm"], self.state[run], self._buf("o", T, V), out, b.segs, b.positions, **args, **self._groups_of(b))
+            self._scan(b, run, p, q, k, v, g, low, V, out, args)
         ops.linear(out, w[p + "o"], y)
 
     def _wkv(self, b: StepBatch, run: int, i: int, m: WkvSpec, y) -> None:
@@ -169,12 +174,10 @@ class Tinapel:
             else:
                 for s, t in enumerate((r, k, v, g)):
                     ops.linear(mixes[:, s * Wp: (s + 1) * Wp], w[p + "in"][s * K: (s + 1) * K], t)
-            lf, z = self._buf("low", T, R), self._buf("z", T, K)
+            lf = self._buf("low", T, R)
             lh = self._buf("low_h", T, R) if self.dtype is torch.bfloat16 else None
             ops.linear(mixes[:, 4 * Wp:], w[p + "in"][4 * K:], lf, act=ops.ACT_TANH, copy=lh)
-            ops.linear(lf if lh is None else lh, w[p + "decay"], z, bias=w[p + "decay.b"])
-            ops.decay_scan(r, k, v, g, z, w[p + "norm"], self.state[run], self._buf("o", T, K), out, b.segs, b.positions,
-                           shift=(self.h1f[:T], self.shift[run]), **args, **self._groups_of(b))
+            self._scan(b, run, p, r, k, v, g, lf if lh is None else lh, K, out, {**args, "shift": (self.h1f[:T], self.shift[run])})
         ops.linear(out, w[p + "o"], y)
 
     def _attention(self, b: StepBatch, run: int, i: int, m: SharedKvSpec, y) -> None:

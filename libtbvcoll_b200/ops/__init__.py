@@ -39,7 +39,7 @@ def lib():
     l.tbv_op_residual.argtypes = [c_vp] * 4 + [F, LL] + [c_vp] * 8 + [I] + [c_vp] * 4 + [I, c_vp, I] + [c_vp] * 4 + [I] * 5 + [F, I, c_vp]
     l.tbv_op_token_shift.argtypes = [c_vp] * 7 + [I] * 4 + [c_vp]
     l.tbv_op_moe_route.argtypes = [c_vp] * 8 + [I] * 4 + [F, I, c_vp]
-    l.tbv_op_decay_scan.argtypes = [c_vp] * 15 + [I, I, c_vp, c_vp] + [I] * 10 + [F, F, F, I, c_vp]
+    l.tbv_op_decay_scan.argtypes = [c_vp] * 15 + [I, I, c_vp, c_vp, c_vp, c_vp, c_vp] + [I] * 12 + [F, F, F, I, c_vp]
     l.tbv_op_decay_step.argtypes = [c_vp] * 13 + [I] * 9 + [F, F, F, I, c_vp]
     l.tbv_op_shared_attn_prep.argtypes = [c_vp] * 6 + [I] * 8 + [F, F, ctypes.c_double, I, c_vp]
     l.tbv_op_shared_attn_rows.argtypes = [c_vp] * 6 + [I] * 7 + [F, I, c_vp]
@@ -439,6 +439,6 @@ def prefill_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
     return out
 
 
-from .mixers import (SHARED_PREFILL_MAX_DIM, causal_conv_silu, decay_scan, decay_step, hyper_embed, hyper_mix,  # noqa: E402,F401
+from .mixers import (DECAY_RANK_MAX, SHARED_PREFILL_MAX_DIM, causal_conv_silu, decay_scan, decay_step, hyper_embed, hyper_mix,  # noqa: E402,F401
                      latent_attention_prefill, latent_attention_rows, latent_gather, latent_prefill_fits, latent_prep, latent_row, moe_route,
                      position_turns, residual, selective_scan, shared_attention_prefill, shared_attention_prep, shared_attention_rows, token_shift)

@@ -165,8 +165,11 @@ def token_shift(h, mu, shift, mixes, segs, seg_of_row, positions) -> None:
 
 
 # ---- linear recurrences with a matrix state -----------------------------------------------------------------------------------
+DECAY_RANK_MAX = 128                  # of the decay product inside decay_scan
+
+
 def decay_scan(q, k, v, g, z, norm, state, o, out, segs, positions, vdim: int, eps: float, qscale: float = 1.0, tau: float = 1.0, u=None,
-               shift=None, groups=None, scratch=None) -> None:
+               shift=None, groups=None, scratch=None, low=None) -> None:
     """Per head S_t = diag(a_t) S_{t-1} + k_t v_t^T over the rows of every segment, then out = RMSNorm(o) * norm * silu(g).
     u None (gated linear attention): a = sigmoid(z)^(1 / tau), o_t = S_t^T (qscale q_t).  u fp32 [heads * Dp] (WKV): a = exp(-exp(z)),
     o_t = (S_{t-1} + diag(u) k_t v_t^T)^T q_t.
@@ -174,10 +177,15 @@ def decay_scan(q, k, v, g, z, norm, state, o, out, segs, positions, vdim: int, e
     q, k, v, g: column views [rows, heads * size] of one buffer; z fp32 [rows, heads * Dp]; state fp32 [slots, heads, Dp, Vp] is replaced;
     ``groups`` (bf16; None: the sequential kernel): the segments cut into groups of rows, int32 [n, 4] (engine.batch.scan_groups), for the chunked
     tensor-core kernels; ``scratch`` = fp32 (states of n * heads * Dp * Vp, totals of n * heads * Dp) if a segment has several groups, else None.
+    ``low`` (with groups) = (low [rows, rank], w2 [heads * Dp, rank], b2 [heads * Dp]) instead of z: z = low @ w2^T + b2 computed inside,
+    rank at most ``DECAY_RANK_MAX``.
     o: fp32 scratch [rows, heads * Vp]; ``shift`` = (h fp32 [rows, ld], shift fp32 [slots, ld]): every segment's last row of h is kept."""
     _, H, Dp, Vp = state.shape
     rows = q.shape[0]
-    assert state.dtype is torch.float32 and z.dtype is torch.float32 and o.dtype is torch.float32 and o.numel() >= rows * H * Vp and q.dtype is out.dtype
+    assert state.dtype is torch.float32 and o.dtype is torch.float32 and o.numel() >= rows * H * Vp and q.dtype is out.dtype
+    assert (z is None) == (low is not None) and (z is None or z.dtype is torch.float32)
+    lo, w2, b2 = low if low is not None else (None, None, None)
+    assert lo is None or (lo.dtype is w2.dtype is b2.dtype is torch.bfloat16 and w2.is_contiguous() and lo.shape[1] == w2.shape[1])
     assert q.stride(0) == k.stride(0) == v.stride(0) == g.stride(0) and q.shape[1] == k.shape[1] == H * Dp and v.shape[1] == g.shape[1] == H * Vp
     h1, sh = shift if shift is not None else (None, None)
     n = 0 if groups is None else groups.shape[0]
@@ -185,7 +193,8 @@ def decay_scan(q, k, v, g, z, norm, state, o, out, segs, positions, vdim: int, e
     assert groups is None or (q.dtype is torch.bfloat16 and groups.dtype is torch.int32)
     assert scratch is None or (starts.numel() >= n * H * Dp * Vp and totals.numel() >= n * H * Dp and starts.dtype is totals.dtype is torch.float32)
     _chk(lib().tbv_op_decay_scan(_p(q), _p(k), _p(v), _p(g), _p(z), _p(u), _p(norm), _p(state), _p(o), _p(out), _p(h1), _p(sh), _p(segs), _p(positions),
-                                 _p(groups), n, int(scratch is not None), _p(starts), _p(totals), rows, segs.shape[0], H, Dp, Vp, vdim, q.stride(0), z.stride(0), out.stride(0), h1.shape[1] if h1 is not None else 0,
+                                 _p(groups), n, int(scratch is not None), _p(starts), _p(totals), _p(lo), _p(w2), _p(b2), lo.stride(0) if lo is not None else 0,
+                                 w2.shape[1] if w2 is not None else 0, rows, segs.shape[0], H, Dp, Vp, vdim, q.stride(0), z.stride(0) if z is not None else 0, out.stride(0), h1.shape[1] if h1 is not None else 0,
                                  qscale, tau, eps, _is_bf16(q), _st()), "tbv_op_decay_scan")
     _count(4 if scratch is not None else 2)
 

@@ -164,7 +164,7 @@ class Recurrence:
         return a if self.kind == "wkv" else {**a, "qscale": self.D ** -0.5, "tau": self.tau}
 
 
-def run_recurrence(seqs, portions, state, slots, dtype, group_rows=None, step_form=False):
+def run_recurrence(seqs, portions, state, slots, dtype, group_rows=None, step_form=False, low_form=False):
     """The next ``portions[i]`` = (start, end) of every sequence as one batch; outputs [rows, H, V] per sequence."""
     from libtbvcoll_b200 import ops
     from libtbvcoll_b200.engine.batch import scan_groups
@@ -191,7 +191,12 @@ def run_recurrence(seqs, portions, state, slots, dtype, group_rows=None, step_fo
             groups = torch.from_numpy(gr).to(DEV)
             if len(gr) > len(segs):
                 scratch = (torch.full((len(gr) * K * pad16(V),), 9.0, device=DEV), torch.full((len(gr) * K,), 9.0, device=DEV))
-        ops.decay_scan(q, k, v, g, z, norm, state, torch.empty(at * Vw, device=DEV), out, sd, pos, groups=groups, scratch=scratch, **s0.args())
+        lo = None
+        if low_form:                                         # the decay product inside
+            act = torch.cat([padded(torch.tanh(s.low[a:b]) if s.kind == "wkv" else s.low[a:b], R, dtype) for s, (a, b) in zip(seqs, portions)])
+            z, lo = None, (act, padded(padded(s0.w2.view(H, D, -1).transpose(1, 2), pad16(D), dtype).transpose(1, 2), R, dtype).reshape(K, R).contiguous(),
+                           pad_heads(s0.b2.view(1, H, D), dtype)[0])
+        ops.decay_scan(q, k, v, g, z, norm, state, torch.empty(at * Vw, device=DEV), out, sd, pos, groups=groups, scratch=scratch, low=lo, **s0.args())
     out = out.view(at, H, pad16(V))
     assert not out[..., V:].any()
     return [out[f: f + n, :, :V] for f, n, _, _ in segs]
@@ -202,13 +207,13 @@ SIZES = [(3, 24, 20), (2, 32, 64), (5, 36, 48), (2, 96, 144), (1, 128, 128), (2,
 
 @pytest.mark.parametrize("kind", ["gla", "wkv"])
 @pytest.mark.parametrize("size", SIZES)
-@pytest.mark.parametrize("form", ["sequential f32", "sequential", "chunks", "groups"])
+@pytest.mark.parametrize("form", ["sequential f32", "sequential", "chunks", "groups", "chunks, low", "groups, low"])
 def test_recurrence_over_portions(kind, size, form):
     """Whole sequences and portions down to one token, of unequal sequences in one batch, slots that held something else: the same outputs and the
     same final state as one plain pass."""
     H, D, V = size if kind == "gla" else (size[0], min(size[1], 160), min(size[1], 160))
     dtype = F32 if form == "sequential f32" else BF
-    rows = {"chunks": 512, "groups": 32}.get(form)
+    rows, low = {"chunks": 512, "groups": 32}.get(form.split(",")[0]), form.endswith("low")
     seqs = [Recurrence(kind, n, H, D, V, seed=n + 1, dtype=dtype) for n in (97, 33, 150)]
     for s in seqs:                                          # one set of weights
         s.norm, s.u, s.w2, s.b2 = seqs[0].norm, seqs[0].u, seqs[0].w2, seqs[0].b2
@@ -219,7 +224,7 @@ def test_recurrence_over_portions(kind, size, form):
             oracle.gated_linear_attention(s.q.double() / D ** 0.5, s.k.double(), s.v.double(), oracle.sigmoid(zz) ** (1 / s.tau))
         s.want = (oracle.rms(s.o, s.eps).flatten(1) * s.norm * oracle.silu(s.g.double())).view(s.T, H, V)
     state = torch.full((6, H, pad16(D), pad16(V)), 5.0, device=DEV)
-    outs = run_recurrence(seqs, [(0, s.T) for s in seqs], state, (2, 5, 1), dtype, rows)
+    outs = run_recurrence(seqs, [(0, s.T) for s in seqs], state, (2, 5, 1), dtype, rows, low_form=low)
     for s, o in zip(seqs, outs):
         close(o, s.want, dtype)
     whole = state[[2, 5, 1]].clone()
@@ -228,11 +233,11 @@ def test_recurrence_over_portions(kind, size, form):
     cuts = [(0, 2, 3, 19, 35, 67, 68, 97), (0, 1, 15, 16, 17, 30, 32, 33), (0, 16, 32, 33, 64, 100, 149, 150)]
     at = [[] for _ in seqs]
     for j in range(7):
-        for i, o in enumerate(run_recurrence(seqs, [(c[j], c[j + 1]) for c in cuts], state, (3, 2, 4), dtype, rows)):
+        for i, o in enumerate(run_recurrence(seqs, [(c[j], c[j + 1]) for c in cuts], state, (3, 2, 4), dtype, rows, low_form=low)):
             at[i].append(o)
     for s, o in zip(seqs, at):
         close(torch.cat(o), s.want, dtype)
-    close(state[[3, 2, 4]], whole, dtype, 2e-5 if dtype is F32 or rows is None else 4e-5)      # the state is 32-bit in every form
+    close(state[[3, 2, 4]], whole, dtype, 2e-5 if dtype is F32 or rows is None else 4e-5)      # carried in 32-bit in every form
 
 
 @pytest.mark.parametrize("kind", ["gla", "wkv"])
