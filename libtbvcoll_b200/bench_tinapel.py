@@ -57,7 +57,7 @@ def kernel_numbers(size: str, T: int, seqs: int, ctx: int, only: str = "") -> li
         k.time("gemm", "tinapel wkv r, k, v, gate, decay (grouped)", mk_mix_gemm, (T * 5 * W + (4 * K + R) * W + T * (4 * K + R)) * 2, 2.0 * T * (4 * K + R) * W)
     else:
         _linear(k, "gemm", "tinapel wkv r / k / v / gate, each", T, K, W)
-        _linear(k, "gemm", "tinapel decay first (tanh, fp32 + copy)", T, R, W, f32=True, act=ops.ACT_TANH, copy=True)
+        _linear(k, "gemm", "tinapel decay first (tanh, fp32 + copy)", T, R, W, f32=True, act=ops.ACT_SOFTCAP, copy=True)
     _linear(k, "gemm", "tinapel attention q + k", T, (a.heads + a.kv_heads) * a.dim, W)
     _linear(k, "gemm", "tinapel mixer out (fp32)", T, W, V, f32=True)
     _linear(k, "gemm", "tinapel head (fp32)", min(T, seqs), _pad16(cfg.vocab_size), W, f32=True)

@@ -54,12 +54,11 @@ struct Params {
 };
 
 enum Epi : int { kEpiStore = 0, kEpiSiluMul = 1, kEpiF32 = 2, kEpiClampGlu = 3 };
-enum Act : int { kActNone = 0, kActSoftplus = 1, kActSoftcap = 2, kActTanh = 3 };
+enum Act : int { kActNone = 0, kActSoftplus = 1, kActSoftcap = 2 };
 
 __device__ __forceinline__ float apply_act(float v, int act, float a) {
   if (act == kActSoftplus) return v > 20.f ? v : log1pf(expf(v));
   if (act == kActSoftcap) return a * tanhf(v / a);
-  if (act == kActTanh) return tanhf(v);
   return v;
 }
 // gated unit: g = min(g, limit), u = clamp(u, -limit, limit); g * sigmoid(slope * g) * (u + shift), all in fp32

@@ -176,7 +176,7 @@ class Tinapel:
                     ops.linear(mixes[:, s * Wp: (s + 1) * Wp], w[p + "in"][s * K: (s + 1) * K], t)
             lf = self._buf("low", T, R)
             lh = self._buf("low_h", T, R) if self.dtype is torch.bfloat16 else None
-            ops.linear(mixes[:, 4 * Wp:], w[p + "in"][4 * K:], lf, act=ops.ACT_TANH, copy=lh)
+            ops.linear(mixes[:, 4 * Wp:], w[p + "in"][4 * K:], lf, act=ops.ACT_SOFTCAP, act_arg=1.0, copy=lh)          # tanh
             self._scan(b, run, p, r, k, v, g, lf if lh is None else lh, K, out, {**args, "shift": (self.h1f[:T], self.shift[run])})
         ops.linear(out, w[p + "o"], y)
 

@@ -124,7 +124,7 @@ def _count(n=1):
 
 
 EPI_STORE, EPI_SILU_MUL, EPI_F32, EPI_CLAMP_GLU = 0, 1, 2, 3
-ACT_NONE, ACT_SOFTPLUS, ACT_SOFTCAP, ACT_TANH = 0, 1, 2, 3
+ACT_NONE, ACT_SOFTPLUS, ACT_SOFTCAP = 0, 1, 2          # a soft cap of 1 is tanh
 SILU_GLU = (math.inf, 1.0, 0.0)           # ``glu`` of ``linear``: silu(gate) * up
 
 
@@ -157,7 +157,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[t
            last: int = 0) -> torch.Tensor:
     """out[N, M] = epilogue(x[N, K] @ w[M, K]^T + bias) for bf16 operands (tcgen05) or fp32 operands (CUDA cores, full 32-bit).
 
-    The output dtype is ``out``'s: fp32 results take an activation (``ACT_SOFTPLUS``, ``ACT_TANH``, ``ACT_SOFTCAP`` with its limit in ``act_arg``)
+    The output dtype is ``out``'s: fp32 results take an activation (``ACT_SOFTPLUS``, ``ACT_SOFTCAP`` with its limit in ``act_arg``)
     and, from bf16 operands, an optional bf16 ``copy`` with the same row stride.  ``glu=(limit, slope[, shift = 1])``: ``w`` holds gate / up rows
     interleaved and out[N, M/2] = g * sigmoid(slope * g) * (u + shift) with g = min(gate, limit), u = clamp(up, -limit, limit).
     ``groups`` > 1: w is [groups * M + last, K]; group g multiplies columns g * x_group .. of x and writes columns g * y_group .. of out; ``last``
