@@ -46,10 +46,12 @@ __device__ __forceinline__ float glu_pair<kEpiClampGlu>(const Params& p, float g
 
 // four consecutive fp32 features of one token: activation, store, optional bf16 copy
 __device__ __forceinline__ void store_f32x4(const Params& p, int M, size_t off, int m, float4 v) {
-  v.x = gemm::apply_act(v.x, p.act, p.act_a);
-  v.y = gemm::apply_act(v.y, p.act, p.act_a);
-  v.z = gemm::apply_act(v.z, p.act, p.act_a);
-  v.w = gemm::apply_act(v.w, p.act, p.act_a);
+  if (p.act != gemm::kActNone) {                    // one branch, not one per value
+    v.x = gemm::apply_act(v.x, p.act, p.act_a);
+    v.y = gemm::apply_act(v.y, p.act, p.act_a);
+    v.z = gemm::apply_act(v.z, p.act, p.act_a);
+    v.w = gemm::apply_act(v.w, p.act, p.act_a);
+  }
   if (m + 4 <= M) {
     *reinterpret_cast<float4*>(p.yf + off) = v;
     if (p.y2) {

@@ -64,6 +64,26 @@ struct RowGroups {
   int tile[kMaxRowGroups + 1];     // first tile of every group
 };
 
+// first token row, end of the rows, first feature and its weight row of a tile
+struct At { int n0, nend, f0, w0; };
+template <bool ROWS, int TOK, typename G>
+__device__ __forceinline__ At find_tile(const G& groups, int tile, int tok_tiles, int ngroups, int M, int N) {
+  if constexpr (ROWS) {
+    int lo = 0, hi = ngroups - 1;                  // the last group whose first tile is not beyond `tile`; empty groups are passed over
+    while (lo < hi) {
+      const int mid = (lo + hi + 1) >> 1;
+      if (groups.tile[mid] <= tile) lo = mid;
+      else hi = mid - 1;
+    }
+    const int local = tile - groups.tile[lo], tt = (groups.off[lo + 1] - groups.off[lo] + TOK - 1) / TOK;
+    const int f0 = local / tt * kFeatTile;
+    return At{groups.off[lo] + local % tt * TOK, groups.off[lo + 1], f0, lo * M + f0};
+  } else {
+    const int f0 = tile / tok_tiles * kFeatTile;
+    return At{tile % tok_tiles * TOK, N, f0, f0};
+  }
+}
+
 struct PSmem {
   unsigned long long full[kMaxStages], empty[kMaxStages], acc_full[2], acc_empty[2];
   uint32_t tmem_base;
@@ -105,8 +125,10 @@ __device__ __forceinline__ void store16(const gemm::Params& p, int n, int f, con
     for (int j = 0; j < 16; j++) v[j] += __bfloat162float(p.bias[f + j]);
   }
   if (EPI == gemm::kEpiF32) {
+    if (p.act != gemm::kActNone) {                  // one branch, not one per value
 #pragma unroll
-    for (int j = 0; j < 16; j++) v[j] = gemm::apply_act(v[j], p.act, p.act_a);
+      for (int j = 0; j < 16; j++) v[j] = gemm::apply_act(v[j], p.act, p.act_a);
+    }
     float* dst = p.yf + size_t(n) * p.ldy + f;      // 64-byte aligned rows: M and ldy are multiples of 16 and 8
     st_global_f32x8(dst, v);
     st_global_f32x8(dst + 8, v + 8);
@@ -143,7 +165,7 @@ __device__ __forceinline__ void store16(const gemm::Params& p, int n, int f, con
 // ROWS: row-grouped problem (p.row_off).
 template <int EPI, int TH, bool ROWS>
 __global__ void __launch_bounds__(Shape<TH>::kThreads, 1)
-k_gemm_tok(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUtensorMap tmW, const gemm::Params p) {
+k_gemm_tok(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUtensorMap tmW, const __grid_constant__ gemm::Params p) {
   using S = Shape<TH>;
   extern __shared__ uint8_t smem_raw[];
   __shared__ PSmem s;
@@ -202,24 +224,9 @@ k_gemm_tok(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUte
     tiles = groups.tile[p.groups];
   }
   const int my_tiles = int(blockIdx.x) < tiles ? (tiles - int(blockIdx.x) + int(gridDim.x) - 1) / int(gridDim.x) : 0;
-  // first token row, end of the rows, first feature and its weight row of a tile
-  struct At { int n0, nend, f0, w0; };
-  auto locate = [&](int tile) -> At {
-    if constexpr (ROWS) {
-      int lo = 0, hi = p.groups - 1;               // the last group whose first tile is not beyond `tile`; empty groups are passed over
-      while (lo < hi) {
-        const int mid = (lo + hi + 1) >> 1;
-        if (groups.tile[mid] <= tile) lo = mid;
-        else hi = mid - 1;
-      }
-      const int local = tile - groups.tile[lo], tt = (groups.off[lo + 1] - groups.off[lo] + S::kTok - 1) / S::kTok;
-      const int f0 = local / tt * kFeatTile;
-      return At{groups.off[lo] + local % tt * S::kTok, groups.off[lo + 1], f0, lo * p.M + f0};
-    } else {
-      const int f0 = tile / tok_tiles * kFeatTile;
-      return At{tile % tok_tiles * S::kTok, p.N, f0, f0};
-    }
-  };
+  const int ngroups = p.groups, feats = p.M, all_rows = p.N;
+  // (by value: a capture of the parameter block would put it in local memory)
+  auto locate = [=](int tile) -> At { return find_tile<ROWS, S::kTok>(groups, tile, tok_tiles, ngroups, feats, all_rows); };
   const uint32_t tmem0 = s.tmem_base;
   volatile int* abortp = &s.abort_flag;
 
