@@ -1,5 +1,5 @@
 // attn_mma.cuh — pieces shared by the attention kernels built on warp-level tensor-core products: cp.async, ldmatrix, mma.sync, cluster
-// reads, and the opt-in to large shared memory.
+// reads, soft cap, limits of what a row sees, and the opt-in to large shared memory.
 #pragma once
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
@@ -42,6 +42,10 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<uint32_t*>(&v);
 }
+__device__ __forceinline__ float4 load_bf16x4(const __nv_bfloat16* p) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xffff0000u));
+}
 __device__ __forceinline__ float ld_cluster_f32(uint32_t addr, uint32_t rank) {
   uint32_t r;
   float v;
@@ -64,6 +68,13 @@ __device__ __forceinline__ void cluster_sync() {
 __device__ __forceinline__ float capped_log2(float s, float cap) {
   if (cap <= 0.f) return s * kLog2e;
   return cap * kLog2e * (1.f - __fdividef(2.f, 1.f + exp2f(s * (2.f * kLog2e / cap))));
+}
+
+// first key that a row sees which causally sees `ctx` of them: all, the last `window`, or those of its own chunk of `chunk` positions (0: no such limit)
+__device__ __forceinline__ int first_visible(int ctx, int window, int chunk) {
+  if (window > 0) return max(0, ctx - window);
+  if (chunk > 0) return max(0, ctx - 1) / chunk * chunk;
+  return 0;
 }
 
 constexpr size_t kMaxSmem = 226 * 1024;

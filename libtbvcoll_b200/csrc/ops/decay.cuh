@@ -1,4 +1,4 @@
-// decay.cuh — parameters and decays shared by the kernels of linear recurrences with a matrix state (decay_scan.cu, chunk_scan.cu).
+// decay.cuh — parameters and decays shared by the kernels of linear recurrences with a matrix state (decay_scan.cu, chunk_scan.cu, fixed_decay.cu).
 #pragma once
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
@@ -19,6 +19,8 @@ struct ScanParams {
   const int *segs, *positions;
   int heads, Dp, Vp, vdim, ld, ldz, ldlow, rank, ldo, ldh;
   float qscale, inv_tau, eps;
+  const float* fixed;          // one constant decay per head instead of z, at fixed[h * fixed_ld] (32-bit sequential kernel only)
+  int fixed_ld;
 };
 
 // decay of one key channel; bf16 models take the fast exponential and logarithm (1 + e^-|z| lies in 1 .. 2: absolute error about 1e-7)
@@ -32,6 +34,10 @@ template <> __device__ __forceinline__ float decay<__nv_bfloat16>(float z, bool 
   return __expf(-(fmaxf(-z, 0.f) + __logf(1.f + __expf(-fabsf(z)))) * inv_tau);
 }
 
+inline bool sizes_ok(int heads, int Dp, int Vp) { return heads > 0 && heads <= 65535 && Dp > 0 && Dp <= 256 && (Dp % 16) == 0 && Vp > 0 && Vp <= 1024 && (Vp % 16) == 0; }
+
+// decay_scan.cu: q, k, v and decays -> o (p.o), token by token in fp32
+cudaError_t sequential_scan_f32(const ScanParams& p, int nseg, cudaStream_t st);
 // chunk_scan.cu: the recurrence of a bf16 model over many rows.  groups [ngroups, 4]: (first row, rows, state slot, flags: 1 = a group of the same
 // segment precedes, 2 = one follows).  p.z null: decay inputs from p.low, p.w2, p.b2 (p.low as it enters the product).  *finished: head norm and gate
 // are done too (p.out), otherwise o is left in p.o.

@@ -53,6 +53,7 @@ __global__ void __launch_bounds__(128) k_decay_scan(const ScanParams p) {
   const int* seg = p.segs + 4 * blockIdx.z;
   const int first = seg[0], n = seg[1], slot = seg[2];
   const bool fresh = p.positions[first] == 0, wkv = p.u != nullptr;
+  const float fixed = p.fixed ? p.fixed[h * p.fixed_ld] : 0.f;
   const T* qp = static_cast<const T*>(p.q) + size_t(h) * p.Dp;
   const T* kp = static_cast<const T*>(p.k) + size_t(h) * p.Dp;
   const T* vp = static_cast<const T*>(p.v) + size_t(h) * p.Vp + c0;
@@ -68,7 +69,7 @@ __global__ void __launch_bounds__(128) k_decay_scan(const ScanParams p) {
         const size_t r = size_t(first + at + t);
         rq[i].load(qp + r * p.ld + d);
         rk[i].load(kp + r * p.ld + d);
-        rz[i].load(p.z + r * p.ldz + size_t(h) * p.Dp + d);
+        if (!p.fixed) rz[i].load(p.z + r * p.ldz + size_t(h) * p.Dp + d);
       }
     }
 #pragma unroll
@@ -102,10 +103,10 @@ __global__ void __launch_bounds__(128) k_decay_scan(const ScanParams p) {
           float z[8];
           rq[i].unpack(q);
           rk[i].unpack(k);
-          rz[i].unpack(z);
+          if (!p.fixed) rz[i].unpack(z);
 #pragma unroll
           for (int e = 0; e < 8; e++) {
-            a[e] = decay<T>(z[e], wkv, p.inv_tau);
+            a[e] = p.fixed ? fixed : decay<T>(z[e], wkv, p.inv_tau);
             if (wkv) {
               s = fmaf(q[e] * p.u[h * p.Dp + d + e], k[e], s);
             } else {
@@ -381,9 +382,13 @@ cudaError_t scan(const ScanParams& p, int nseg, cudaStream_t st) {
   if (p.Dp <= 128) return scan_columns<T, 16, 8>(p, nseg, st);
   return scan_columns<T, 32, 8>(p, nseg, st);
 }
-bool sizes_ok(int heads, int Dp, int Vp, int vdim) { return heads > 0 && heads <= 65535 && Dp > 0 && Dp <= 256 && (Dp % 16) == 0 && Vp > 0 && Vp <= 1024 && (Vp % 16) == 0 && vdim <= Vp; }
+bool sizes_ok(int heads, int Dp, int Vp, int vdim) { return decay_ops::sizes_ok(heads, Dp, Vp) && vdim <= Vp; }
 
 }  // namespace
+
+namespace decay_ops {
+cudaError_t sequential_scan_f32(const ScanParams& p, int nseg, cudaStream_t st) { return scan<float>(p, nseg, st); }
+}  // namespace decay_ops
 
 extern "C" {
 

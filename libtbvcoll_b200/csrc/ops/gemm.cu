@@ -121,6 +121,7 @@ k_gemm(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensor
     __nv_bfloat16* stage_h = reinterpret_cast<__nv_bfloat16*>(sm);
     for (int c = 0; c < p.bn; c += 16) {
       uint32_t r[16];
+      __syncwarp();                                // an activation may act on some of the warp's features only
       if (ok && nkb > 0) {
         tmem_ld16(s.tmem_base + (uint32_t(quarter * 32) << 16) + uint32_t(c), r);
         tmem_ld_wait();
@@ -145,6 +146,9 @@ k_gemm(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensor
           const float o = (lane & 1) ? glu_pair<kGlu ? EPI : kEpiSiluMul>(p, recv, v1) : glu_pair<kGlu ? EPI : kEpiSiluMul>(p, v0, recv);
           stage_h[(c + j + (lane & 1)) * 64 + (ml >> 1)] = __float2bfloat16_rn(o);
         }
+      } else if (p.act != gemm::kActNone && m0 + ml < p.act_m) {
+#pragma unroll
+        for (int j = 0; j < 16; j++) stage_h[(c + j) * 128 + ml] = __float2bfloat16_rn(gemm::apply_act(__uint_as_float(r[j]) + bias, p.act, p.act_a));
       } else {
 #pragma unroll
         for (int j = 0; j < 16; j++) stage_h[(c + j) * 128 + ml] = __float2bfloat16_rn(__uint_as_float(r[j]) + bias);
@@ -204,6 +208,12 @@ k_gemm(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensor
           if (m + 4 <= M) *reinterpret_cast<__nv_bfloat162*>(p.y + size_t(n0 + t) * p.ldy + ycol + (m >> 1)) = o;
         } else {
           __nv_bfloat16* dst = p.y + size_t(n0 + t) * p.ldy + ycol + m;
+          if (p.act != gemm::kActNone && m < p.act_m) {
+            acc.x = gemm::apply_act(acc.x, p.act, p.act_a);
+            acc.y = gemm::apply_act(acc.y, p.act, p.act_a);
+            acc.z = gemm::apply_act(acc.z, p.act, p.act_a);
+            acc.w = gemm::apply_act(acc.w, p.act, p.act_a);
+          }
           if (m + 4 <= M) {
             __nv_bfloat162 lo = __floats2bfloat162_rn(acc.x, acc.y), hi = __floats2bfloat162_rn(acc.z, acc.w);
             uint2 pk;
@@ -468,15 +478,16 @@ int tbv_op_gemm(const void* w, const void* x, void* y, const void* bias, int M, 
 
 // The GEMM with the wider set of epilogues: fp32 output with an activation, clamped gated unit, grouped weights.
 // y: fp32 [N, ldy] for epi 2, bf16 otherwise; y2: optional bf16 copy of an fp32 result (same ldy).  act (epi 2): 0 none,
-// 1 softplus, 2 act_a * tanh(v / act_a).  epi 3: rows of w interleaved (gate_i, up_i), act_a = clamp limit, act_b = slope of the
+// 1 softplus, 2 act_a * tanh(v / act_a), 3 SiLU; with epi 0 act acts on the first act_m features (a multiple of 16; plain problems only).  epi 3: rows of w interleaved (gate_i, up_i), act_a = clamp limit, act_b = slope of the
 // sigmoid, act_c = what is added to u.  groups > 1: w is [groups * M (+ m_last), K]; group g reads x columns g * x_group .. + K and writes y
 // columns g * y_group ..; m_last > 0 is one more group with that many features.
 int tbv_op_gemm_ex(const void* w, const void* x, void* y, void* y2, const void* bias, int M, int N, int K, int ldx, int ldy, int epi,
-                   int act, float act_a, float act_b, float act_c, int groups, int x_group, int y_group, int m_last, void* stream) {
+                   int act, float act_a, float act_b, float act_c, int act_m, int groups, int x_group, int y_group, int m_last, void* stream) {
   const char* pf_ptr = nullptr;
   const unsigned long long pf_bytes = tbvops::take_next_prefetch(&pf_ptr, (unsigned long long)(M > 0 ? M : 0) * (unsigned long long)(K > 0 ? K : 0) * 2ull);
   if (M <= 0 || N <= 0 || K <= 0 || (K % 8) || (ldx % 8) || (ldy % 8) || (reinterpret_cast<uintptr_t>(y) & 15u)) return -2;
   if (epi < 0 || epi > 3 || (epi == kEpiClampGlu && (M % 2)) || (y2 && (epi != kEpiF32 || (reinterpret_cast<uintptr_t>(y2) & 7u)))) return -2;
+  if (epi == kEpiStore && act != gemm::kActNone && (groups > 1 || (act_m % 16))) return -2;
   if (groups > 1 && ((x_group % 8) || (y_group % 8) || bias)) return -2;
   Params p{};
   p.M = M; p.N = N; p.K = K; p.ldy = ldy;
@@ -484,7 +495,7 @@ int tbv_op_gemm_ex(const void* w, const void* x, void* y, void* y2, const void* 
   if (epi == kEpiF32) p.yf = static_cast<float*>(y);
   else p.y = static_cast<__nv_bfloat16*>(y);
   p.y2 = static_cast<__nv_bfloat16*>(y2);
-  p.act = act; p.act_a = act_a; p.act_b = act_b; p.act_c = act_c; p.m_last = groups > 1 ? m_last : 0;
+  p.act = act; p.act_a = act_a; p.act_b = act_b; p.act_c = act_c; p.act_m = act_m; p.m_last = groups > 1 ? m_last : 0;
   p.pf_ptr = pf_ptr;
   p.pf_bytes = pf_bytes;
   p.groups = groups > 1 ? groups : 1; p.x_group = groups > 1 ? x_group : 0; p.y_group = groups > 1 ? y_group : 0;

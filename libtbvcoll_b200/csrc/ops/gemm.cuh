@@ -37,7 +37,8 @@ struct Params {
   // fp32 output (kEpiF32): activation after the bias, and an optional bf16 copy of the result under the same indexing
   float* yf;
   __nv_bfloat16* y2;
-  int act;             // Act below
+  int act;             // Act below (bf16 stores: on the first act_m features, a multiple of 16; fp32 stores: on all)
+  int act_m;
   float act_a, act_b, act_c;  // softcap: limit; gated unit: limit, slope of the sigmoid, what is added to u
   // grouped form (decode-form kernel): `groups` problems of M features side by side; group g multiplies rows g * M .. of w
   // with columns g * x_group .. of x and writes at column g * y_group.  groups <= 1: one plain problem.
@@ -54,17 +55,19 @@ struct Params {
 };
 
 enum Epi : int { kEpiStore = 0, kEpiSiluMul = 1, kEpiF32 = 2, kEpiClampGlu = 3 };
-enum Act : int { kActNone = 0, kActSoftplus = 1, kActSoftcap = 2 };
+enum Act : int { kActNone = 0, kActSoftplus = 1, kActSoftcap = 2, kActSilu = 3 };
 
 __device__ __forceinline__ float apply_act(float v, int act, float a) {
   if (act == kActSoftplus) return v > 20.f ? v : log1pf(expf(v));
   if (act == kActSoftcap) return a * tanhf(v / a);
+  if (act == kActSilu) return __fdividef(v, 1.0f + __expf(-v));   // an infinite denominator gives 0
   return v;
 }
-// gated unit: g = min(g, limit), u = clamp(u, -limit, limit); g * sigmoid(slope * g) * (u + shift), all in fp32
+// gated unit: g = min(g, limit), u = clamp(u, -limit, limit); g * sigmoid(slope * g) * (u + shift), all in fp32.  An infinite slope makes it a ReLU.
 __device__ __forceinline__ float clamp_glu(float g, float u, float limit, float slope, float shift) {
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
+  if (isinf(slope)) return fmaxf(g, 0.f) * (u + shift);
   return g / (1.0f + __expf(-slope * g)) * (u + shift);
 }
 

@@ -19,6 +19,7 @@ struct F32Params {
   int M, N, K, ldx, ldy, epi, act, groups, x_group, y_group;
   float act_a, act_b, act_c;
   int m_last;             // > 0: one more group with this many features
+  int act_m;              // the activation acts on the first act_m features
   const int* row_off;     // row-grouped form: group g owns rows row_off[g] .. row_off[g + 1] - 1
 };
 
@@ -74,13 +75,16 @@ __global__ void __launch_bounds__(256) k_gemm_f32(const F32Params p) {
       for (int j = 0; j < 4; j += 2) {
         if (m0 + tm + j + 1 < M) {
           const float g = fminf(v[j], p.act_a), u = fminf(fmaxf(v[j + 1], -p.act_a), p.act_a);
-          y[size_t(n) * p.ldy + (m0 + tm + j) / 2] = g / (1.0f + expf(-p.act_b * g)) * (u + p.act_c);
+          y[size_t(n) * p.ldy + (m0 + tm + j) / 2] = (isinf(p.act_b) ? fmaxf(g, 0.f) : g / (1.0f + expf(-p.act_b * g))) * (u + p.act_c);
         }
       }
     } else {
 #pragma unroll
       for (int j = 0; j < 4; j++)
-        if (m0 + tm + j < M) y[size_t(n) * p.ldy + m0 + tm + j] = gemm::apply_act(v[j], p.act, p.act_a);
+        if (m0 + tm + j < M) {
+          if (p.act && m0 + tm + j < p.act_m) v[j] = p.act == gemm::kActSilu ? v[j] / (1.0f + expf(-v[j])) : gemm::apply_act(v[j], p.act, p.act_a);
+          y[size_t(n) * p.ldy + m0 + tm + j] = v[j];
+        }
     }
   }
 }
@@ -91,10 +95,10 @@ extern "C" {
 
 // Arguments as tbv_op_gemm_ex, everything fp32; epi 0 / 2 store (act applies), 3 clamped gated unit.
 int tbv_op_gemm_f32(const void* w, const void* x, void* y, const void* bias, int M, int N, int K, int ldx, int ldy, int epi, int act,
-                    float act_a, float act_b, float act_c, int groups, int x_group, int y_group, int m_last, void* stream) {
+                    float act_a, float act_b, float act_c, int act_m, int groups, int x_group, int y_group, int m_last, void* stream) {
   if (M <= 0 || N <= 0 || K <= 0 || (epi != 0 && epi != 2 && epi != 3) || (epi == 3 && (M % 2)) || (groups > 1 && bias)) return -2;
   F32Params p{static_cast<const float*>(w), static_cast<const float*>(x), static_cast<const float*>(bias), static_cast<float*>(y),
-              M, N, K, ldx, ldy, epi, act, groups > 1 ? groups : 1, x_group, y_group, act_a, act_b, act_c, groups > 1 ? m_last : 0, nullptr};
+              M, N, K, ldx, ldy, epi, act, groups > 1 ? groups : 1, x_group, y_group, act_a, act_b, act_c, groups > 1 ? m_last : 0, act_m, nullptr};
   const dim3 grid(p.groups * ((M + kT - 1) / kT) + (p.m_last + kT - 1) / kT, (N + kT - 1) / kT);
   return pdl::launch(k_gemm_f32, grid, dim3(256), 0, static_cast<cudaStream_t>(stream), 1, p) == cudaSuccess ? 0 : -1;
 }
@@ -104,7 +108,7 @@ int tbv_op_gemm_rows_f32(const void* w, const void* x, void* y, const void* row_
                          int ldy, int epi, float act_a, float act_b, float act_c, void* stream) {
   if (M <= 0 || x_rows <= 0 || max_rows <= 0 || K <= 0 || groups <= 0 || (epi != 0 && epi != 3) || (epi == 3 && (M % 2)) || !row_off) return -2;
   F32Params p{static_cast<const float*>(w), static_cast<const float*>(x), nullptr, static_cast<float*>(y),
-              M, max_rows, K, ldx, ldy, epi, 0, groups, 0, 0, act_a, act_b, act_c, 0, static_cast<const int*>(row_off)};
+              M, max_rows, K, ldx, ldy, epi, 0, groups, 0, 0, act_a, act_b, act_c, 0, 0, static_cast<const int*>(row_off)};
   const dim3 grid(groups * ((M + kT - 1) / kT), (max_rows + kT - 1) / kT);
   return pdl::launch(k_gemm_f32, grid, dim3(256), 0, static_cast<cudaStream_t>(stream), 1, p) == cudaSuccess ? 0 : -1;
 }

@@ -151,6 +151,10 @@ __device__ __forceinline__ void store16(const gemm::Params& p, int n, int f, con
     o.w = pack_bf16(silu_mul_bf16(v[12], v[13]), silu_mul_bf16(v[14], v[15]));
     *reinterpret_cast<uint4*>(p.y + size_t(n) * p.ldy + (f >> 1)) = o;
   } else {
+    if (p.act != gemm::kActNone && f < p.act_m) {   // act_m is a multiple of 16
+#pragma unroll
+      for (int j = 0; j < 16; j++) v[j] = gemm::apply_act(v[j], p.act, p.act_a);
+    }
     uint4 o0, o1;
     o0.x = pack_bf16(v[0], v[1]);   o0.y = pack_bf16(v[2], v[3]);   o0.z = pack_bf16(v[4], v[5]);   o0.w = pack_bf16(v[6], v[7]);
     o1.x = pack_bf16(v[8], v[9]);   o1.y = pack_bf16(v[10], v[11]); o1.z = pack_bf16(v[12], v[13]); o1.w = pack_bf16(v[14], v[15]);

@@ -12,7 +12,8 @@
 // Scores, softmax and sums are fp32; the denominator contains exp(sink_h) once.
 //
 // The rows form also serves attention whose values are the unnormalised keys (template KS; shared_attn.cu): kv_heads rows per token, each used by
-// heads / kv_heads query heads, with one fp32 factor per row (kept in the row's pad) on its scores, and an optional soft cap.
+// heads / kv_heads query heads, with one fp32 factor per row (kept in the row's pad) on its scores, and an optional soft cap.  And attention over rows that
+// hold key and value side by side (kPaired; shared_attn.cu as well), with a window or chunks and a gate on the result.
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
@@ -108,24 +109,30 @@ struct RowsParams {
   int heads, R, Rp, rotp, block_size, max_blocks, splits;
   int kv_heads;             // cache rows per token: block b, head g and place t of a block at row (b * kv_heads + g) * block_size + t
   float scale_log2, scale;
-  float softcap;            // 0: none (KS form only)
+  float softcap;            // 0: none (not in the latent form)
   int* err;                 // device flag: set to 1 if a wait for copies gave up
+  // paired rows: rotp = key columns (first), Rp = value columns (behind them)
+  int window, chunk;        // attn_mma::first_visible
+  const void* gate;         // [rows, ldg] or null: results are multiplied by sigmoid of column h * Rp ..
+  int ldg;
 };
+enum RowKind { kLatent, kShared, kPaired };
 
 // fp32: one CTA per (row, head), tiles of 128 keys.  Exponents are taken of differences of natural-unit scores: a score of
 // hundreds loses nothing to a multiplication by log2 e.
-template <bool KS>
+template <RowKind KIND>
 __global__ void __launch_bounds__(128) k_latent_rows_f32(const RowsParams p) {
   extern __shared__ float sm[];
   __shared__ float red[4];
   pdl::launch_dependents();
   pdl::grid_dependency_wait();
   const int row = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, Dk = p.Rp + p.rotp;
-  float* sq = sm;            // [Dk]
-  float* sp = sm + Dk;       // [128]
+  const int kd = KIND == kPaired ? p.rotp : Dk, voff = KIND == kPaired ? p.rotp : 0;   // columns of the scores, first one of the values
+  float* sq = sm;            // [kd]
+  float* sp = sm + kd;       // [128]
   int* sl = reinterpret_cast<int*>(sp + 128);
-  const float* qa = static_cast<const float*>(p.qa) + (size_t(row) * p.heads + h) * (Dk + kRowPad);
-  for (int i = tid; i < Dk; i += 128) sq[i] = qa[i];
+  const float* qa = static_cast<const float*>(p.qa) + (size_t(row) * p.heads + h) * (kd + kRowPad);
+  for (int i = tid; i < kd; i += 128) sq[i] = qa[i];
   const float* cache = static_cast<const float*>(p.cache);
   const int ctx = min(p.ctx_lens[row], p.max_blocks * p.block_size);
   const int* bt = p.tables + size_t(p.seq_of_row ? p.seq_of_row[row] : row) * p.max_blocks;
@@ -135,7 +142,7 @@ __global__ void __launch_bounds__(128) k_latent_rows_f32(const RowsParams p) {
 #pragma unroll
   for (int k = 0; k < kAcc; k++) o[k] = 0.f;
   float m = kNegBig, l = 0.f;
-  for (int t0 = 0; t0 < ctx; t0 += 128) {
+  for (int t0 = KIND == kPaired ? first_visible(ctx, p.window, p.chunk) : 0; t0 < ctx; t0 += 128) {
     const int n = min(128, ctx - t0);
     __syncthreads();
     float s = kNegBig;
@@ -145,15 +152,13 @@ __global__ void __launch_bounds__(128) k_latent_rows_f32(const RowsParams p) {
       const float4* kr = reinterpret_cast<const float4*>(cache + size_t(slot) * (Dk + kRowPad));
       const float4* q4 = reinterpret_cast<const float4*>(sq);
       float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-      for (int i = 0; i < Dk / 4; i++) {
+      for (int i = 0; i < kd / 4; i++) {
         const float4 k = kr[i], q = q4[i];
         a.x = fmaf(q.x, k.x, a.x); a.y = fmaf(q.y, k.y, a.y); a.z = fmaf(q.z, k.z, a.z); a.w = fmaf(q.w, k.w, a.w);
       }
       s = ((a.x + a.y) + (a.z + a.w)) * p.scale;
-      if (KS) {
-        s *= cache[size_t(slot) * (Dk + kRowPad) + Dk];
-        if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
-      }
+      if (KIND == kShared) s *= cache[size_t(slot) * (Dk + kRowPad) + Dk];
+      if (KIND != kLatent && p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
     }
     float mx = s;
 #pragma unroll
@@ -176,7 +181,7 @@ __global__ void __launch_bounds__(128) k_latent_rows_f32(const RowsParams p) {
       const int d = tid + k * 128;
       if (d < p.R) {
         float acc = 0.f;
-        for (int t = 0; t < n; t++) acc = fmaf(sp[t], cache[size_t(sl[t]) * (Dk + kRowPad) + d], acc);
+        for (int t = 0; t < n; t++) acc = fmaf(sp[t], cache[size_t(sl[t]) * (Dk + kRowPad) + voff + d], acc);
         o[k] = fmaf(o[k], corr, acc);
       }
     }
@@ -191,7 +196,11 @@ __global__ void __launch_bounds__(128) k_latent_rows_f32(const RowsParams p) {
 #pragma unroll
   for (int k = 0; k < kAcc; k++) {
     const int d = tid + k * 128;
-    if (d < p.Rp) out[d] = d < p.R && l > 0.f ? o[k] * c / l : 0.f;
+    if (d < p.Rp) {
+      float v = d < p.R && l > 0.f ? o[k] * c / l : 0.f;
+      if (KIND == kPaired && p.gate) v *= vec::sigmoid<float>(static_cast<const float*>(p.gate)[size_t(row) * p.ldg + size_t(h) * p.Rp + d]);
+      out[d] = v;
+    }
   }
 }
 
@@ -201,7 +210,7 @@ __global__ void __launch_bounds__(128) k_latent_rows_f32(const RowsParams p) {
 // disjoint token ranges and merge in split order.
 constexpr int kRW = 8;
 constexpr int kMaxSplits = 8;
-template <int CBW, int TT, bool KS>
+template <int CBW, int TT, RowKind KIND>
 __global__ void __launch_bounds__(kRW * 32 + 32, 1) k_latent_rows_mma(const RowsParams p) {
   extern __shared__ __align__(128) uint8_t dsm[];
   __shared__ float sh_max[kRW][16], sh_l[kRW][16], sh_ml[16][2], sh_fac[kMaxSplits][16], sh_sm[kMaxSplits][16];
@@ -219,24 +228,27 @@ __global__ void __launch_bounds__(kRW * 32 + 32, 1) k_latent_rows_mma(const Rows
   pdl::grid_dependency_wait();
   const int row = blockIdx.x, sp = blockIdx.z, S = p.splits;
   // head tile: 16 query heads of one cache head g
-  const int G = KS ? p.kv_heads : 1, hpk = p.heads / G, tpg = (hpk + 15) / 16, g = KS ? blockIdx.y / tpg : 0;
+  constexpr bool HEADS = KIND != kLatent;
+  const int G = HEADS ? p.kv_heads : 1, hpk = p.heads / G, tpg = (hpk + 15) / 16, g = HEADS ? blockIdx.y / tpg : 0;
   const int h0 = g * hpk + (blockIdx.y - g * tpg) * 16;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r8 = lane >> 2, quad = lane & 3;
-  const int Dk = p.Rp + p.rotp, chunks = Dk / 8, pitch = (Dk + kRowPad) * 2, ksteps = Dk / 16, cblocks = p.Rp / 16;
+  const int Dk = p.Rp + p.rotp, kd = KIND == kPaired ? p.rotp : Dk, voff = KIND == kPaired ? p.rotp : 0;   // columns: all, of the scores, before the values
+  const int chunks = Dk / 8, pitch = (Dk + kRowPad) * 2, qpitch = (kd + kRowPad) * 2, ksteps = kd / 16, cblocks = p.Rp / 16;
   const uint32_t sq = smem_addr(dsm), sk0 = sq + 16 * pitch, stage = uint32_t(TT) * pitch, spb = smem_addr(sh_p);
   constexpr int kPP = TT * 2 + 16;
   const int ctx = min(p.ctx_lens[row], p.max_blocks * p.block_size);
   const int* bt = p.tables + size_t(p.seq_of_row ? p.seq_of_row[row] : row) * p.max_blocks;
-  int chunk = (ctx + S - 1) / S;
+  const int lo = KIND == kPaired ? first_visible(ctx, p.window, p.chunk) : 0, from = lo & ~15;
+  int chunk = (ctx - from + S - 1) / S;
   chunk = (chunk + 15) / 16 * 16;
-  const int t0 = min(ctx, sp * chunk), t1 = min(ctx, t0 + chunk);
+  const int t0 = min(ctx, from + sp * chunk), t1 = min(ctx, t0 + chunk);
   const int ntiles = (t1 - t0 + TT - 1) / TT;
 
-  const __nv_bfloat16* qa = static_cast<const __nv_bfloat16*>(p.qa) + (size_t(row) * p.heads + h0) * (Dk + kRowPad);
+  const __nv_bfloat16* qa = static_cast<const __nv_bfloat16*>(p.qa) + (size_t(row) * p.heads + h0) * (kd + kRowPad);
   const __nv_bfloat16* cache = static_cast<const __nv_bfloat16*>(p.cache);
   const int nq = min(16, (g + 1) * hpk - h0);
   for (int r = nq + warp; r < 16; r += kRW + 1)
-    for (int c = lane; c < chunks; c += 32) st_zero16(sq + r * pitch + c * 16);
+    for (int c = lane; c < kd / 8; c += 32) st_zero16(sq + r * qpitch + c * 16);
   // The ninth warp brings the tiles in.  Tile i: its tokens, a block (or the part of one inside the tile) per copy, and the query rows
   // with tile 0.  A partial tile ends at a multiple of 16 tokens; its missing rows are zeros, so that a weight of zero meets no stale
   // bit pattern.  Table entries are looked up a tile ahead of their use: table and cache are two memory round trips, and both would
@@ -251,8 +263,8 @@ __global__ void __launch_bounds__(kRW * 32 + 32, 1) k_latent_rows_mma(const Rows
     const uint32_t dst = sk0 + (i & 1) * stage, bar = smem_addr(&full[i & 1]);
     const int tok0 = t0 + i * TT, n = min(TT, t1 - tok0), pg0 = tok0 / bs;
     if (lane == 0) {
-      sm100::mbar_expect_tx(bar, uint32_t(n + (i == 0 ? nq : 0)) * uint32_t(pitch));
-      if (i == 0) sm100::bulk_load(sq, qa, uint32_t(nq) * pitch, bar);
+      sm100::mbar_expect_tx(bar, uint32_t(n) * uint32_t(pitch) + (i == 0 ? uint32_t(nq) * uint32_t(qpitch) : 0u));
+      if (i == 0) sm100::bulk_load(sq, qa, uint32_t(nq) * qpitch, bar);
     }
     __syncwarp();
     for (int pg = pg0 + lane; pg * bs < tok0 + n; pg += 32) {
@@ -296,7 +308,7 @@ __global__ void __launch_bounds__(kRW * 32 + 32, 1) k_latent_rows_mma(const Rows
     const bool has_s = warp * 8 < n16;
     if (has_s) {
       // operands of the next two k steps are requested before the products of these two; four accumulators in turn
-      const uint32_t qaddr = sq + (lane & 15) * pitch + (lane >> 4) * 16;
+      const uint32_t qaddr = sq + (lane & 15) * qpitch + (lane >> 4) * 16;
       const uint32_t kaddr = sk + (warp * 8 + (lane & 7)) * pitch + (lane >> 3) * 16;
       float se[4] = {0.f, 0.f, 0.f, 0.f}, sf[4] = {0.f, 0.f, 0.f, 0.f};
       uint32_t a[2][2][4], b[2][4];
@@ -306,7 +318,7 @@ __global__ void __launch_bounds__(kRW * 32 + 32, 1) k_latent_rows_mma(const Rows
         ldmatrix_x4(qaddr + ks * 32 + 32, a[w][1]);
       };
       const int pairs = ksteps / 2;
-      load(0, 0);
+      if (pairs > 0) load(0, 0);
       int k2 = 0;
       for (; k2 + 1 < pairs; k2 += 2) {
         load(2 * k2 + 2, 1);
@@ -329,7 +341,10 @@ __global__ void __launch_bounds__(kRW * 32 + 32, 1) k_latent_rows_mma(const Rows
 #pragma unroll
       for (int j = 0; j < 4; j++) sc[j] += se[j], sd[j] += sf[j];
       const int tok = t0 + i * TT + warp * 8 + quad * 2;
-      if constexpr (KS) {
+      if constexpr (KIND == kPaired) {
+#pragma unroll
+        for (int j = 0; j < 4; j++) sc[j] = tok + (j & 1) < t1 && tok + (j & 1) >= lo ? capped_log2(sc[j] + sd[j], p.softcap) : kNegBig;
+      } else if constexpr (KIND == kShared) {
         float f[2];            // the two tokens' factors (stale past the end: masked below)
 #pragma unroll
         for (int j = 0; j < 2; j++) asm volatile("ld.shared.f32 %0, [%1];" : "=f"(f[j]) : "r"(sk + (warp * 8 + quad * 2 + j) * pitch + Dk * 2) : "memory");
@@ -375,7 +390,7 @@ __global__ void __launch_bounds__(kRW * 32 + 32, 1) k_latent_rows_mma(const Rows
 #pragma unroll
       for (int b = 0; b < CBW; b++)
         if (warp + b * kRW < cblocks)
-          ldmatrix_x4_trans(sk + (ks * 16 + (lane & 15)) * pitch + (warp + b * kRW) * 32 + (lane >> 4) * 16, v[w][b]);
+          ldmatrix_x4_trans(sk + (ks * 16 + (lane & 15)) * pitch + (warp + b * kRW) * 32 + voff * 2 + (lane >> 4) * 16, v[w][b]);
     };
     load_v(0, 0);
 #pragma unroll
@@ -468,6 +483,11 @@ __global__ void __launch_bounds__(kRW * 32 + 32, 1) k_latent_rows_mma(const Rows
           const float f = sh_fac[r][h];
           a.x = fmaf(v[r].x, f, a.x); a.y = fmaf(v[r].y, f, a.y); a.z = fmaf(v[r].z, f, a.z); a.w = fmaf(v[r].w, f, a.w);
         }
+      if (KIND == kPaired && p.gate) {
+        const float4 gt = load_bf16x4(static_cast<const __nv_bfloat16*>(p.gate) + size_t(row) * p.ldg + size_t(h0) * p.Rp + idx * 4);
+        a.x *= vec::sigmoid<__nv_bfloat16>(gt.x); a.y *= vec::sigmoid<__nv_bfloat16>(gt.y);
+        a.z *= vec::sigmoid<__nv_bfloat16>(gt.z); a.w *= vec::sigmoid<__nv_bfloat16>(gt.w);
+      }
       *reinterpret_cast<uint2*>(out + idx * 4) = make_uint2(pack_bf16(a.x, a.y), pack_bf16(a.z, a.w));
     }
   }
@@ -655,11 +675,11 @@ __global__ void __launch_bounds__(128, 2) k_latent_prefill_mma(const PrefillPara
   }
 }
 
-template <int CBW, int TT, bool KS>
+template <int CBW, int TT, RowKind KIND>
 cudaError_t launch_rows(const RowsParams& p, dim3 grid, size_t smem, cudaStream_t st) {
   static bool done = false;
-  cudaError_t e = allow_smem(k_latent_rows_mma<CBW, TT, KS>, smem, &done);
-  return e != cudaSuccess ? e : pdl::launch(k_latent_rows_mma<CBW, TT, KS>, grid, dim3(kRW * 32 + 32), smem, st, p.splits, p);
+  cudaError_t e = allow_smem(k_latent_rows_mma<CBW, TT, KIND>, smem, &done);
+  return e != cudaSuccess ? e : pdl::launch(k_latent_rows_mma<CBW, TT, KIND>, grid, dim3(kRW * 32 + 32), smem, st, p.splits, p);
 }
 template <int VT>
 cudaError_t launch_prefill(const PrefillParams& p, dim3 grid, size_t smem, cudaStream_t st) {
@@ -670,7 +690,7 @@ cudaError_t launch_prefill(const PrefillParams& p, dim3 grid, size_t smem, cudaS
 size_t rows_smem(int Dk, int TT) { return size_t(16 + 2 * TT) * (Dk * 2 + 16); }
 size_t prefill_smem(int Dq, int vdp) { return size_t(64 + 2 * kPK) * (Dq * 2 + 16) + size_t(2) * kPK * (vdp * 2 + 16); }
 
-template <bool KS>
+template <RowKind KIND>
 int rows_form(RowsParams& p, int rows, int bf16, cudaStream_t st) {
   if (rows <= 0) return 0;
   if (p.heads <= 0 || p.block_size <= 0) return -2;
@@ -679,17 +699,17 @@ int rows_form(RowsParams& p, int rows, int bf16, cudaStream_t st) {
   if (!bf16) {
     p.splits = 1;
     if (p.Rp > 2048) return -2;
-    e = pdl::launch(k_latent_rows_f32<KS>, dim3(rows, p.heads), dim3(128), size_t(p.Rp + p.rotp + 256) * 4, st, 1, p);
+    e = pdl::launch(k_latent_rows_f32<KIND>, dim3(rows, p.heads), dim3(128), size_t(p.Rp + p.rotp + 256) * 4, st, 1, p);
     return e == cudaSuccess ? 0 : -1;
   }
   p.splits = p.splits < 1 ? 1 : (p.splits > kMaxSplits ? kMaxSplits : p.splits);
   const int Dk = p.Rp + p.rotp;
   const dim3 grid(rows, p.kv_heads * ((p.heads / p.kv_heads + 15) / 16), p.splits);
   const size_t s64 = rows_smem(Dk, 64), s32 = rows_smem(Dk, 32);   // either holds the [16][Rp] fp32 partials too
-  if (p.Rp <= 128) e = launch_rows<1, 64, KS>(p, grid, s64, st);
-  else if (p.Rp <= 256) e = launch_rows<2, 64, KS>(p, grid, s64, st);
-  else if (p.Rp <= 512 && s64 <= kMaxSmem - 8192) e = launch_rows<4, 64, KS>(p, grid, s64, st);
-  else if (p.Rp <= 1024 && s32 <= kMaxSmem - 8192) e = launch_rows<8, 32, KS>(p, grid, s32, st);
+  if (p.Rp <= 128) e = launch_rows<1, 64, KIND>(p, grid, s64, st);
+  else if (p.Rp <= 256) e = launch_rows<2, 64, KIND>(p, grid, s64, st);
+  else if (p.Rp <= 512 && s64 <= kMaxSmem - 8192) e = launch_rows<4, 64, KIND>(p, grid, s64, st);
+  else if (p.Rp <= 1024 && s32 <= kMaxSmem - 8192) e = launch_rows<8, 32, KIND>(p, grid, s32, st);
   else return -2;
   if (e != cudaSuccess) fprintf(stderr, "[tbvops] latent attention launch failed: %s\n", cudaGetErrorString(e));
   return e == cudaSuccess ? 0 : -1;
@@ -700,8 +720,15 @@ int rows_form(RowsParams& p, int rows, int bf16, cudaStream_t st) {
 namespace tbvops {
 int shared_attn_rows_any(const void* qa, const void* cache, const int* tables, const int* seq_of_row, const int* ctx_lens, void* out, int rows,
                          int heads, int kv_heads, int Dp, int block_size, int max_blocks, int splits, float softcap, int bf16, cudaStream_t st) {
-  RowsParams p{qa, cache, tables, seq_of_row, ctx_lens, nullptr, out, heads, Dp, Dp, 0, block_size, max_blocks, splits, kv_heads, kLog2e, 1.f, softcap, nullptr};
-  return rows_form<true>(p, rows, bf16, st);
+  RowsParams p{qa, cache, tables, seq_of_row, ctx_lens, nullptr, out, heads, Dp, Dp, 0, block_size, max_blocks, splits, kv_heads, kLog2e, 1.f, softcap, nullptr, 0, 0, nullptr, 0};
+  return rows_form<kShared>(p, rows, bf16, st);
+}
+int paired_attn_rows_any(const void* qa, const void* cache, const int* tables, const int* seq_of_row, const int* ctx_lens, const void* gate, void* out, int rows,
+                         int heads, int kv_heads, int Dp, int Vp, int ldg, int block_size, int max_blocks, int splits, float softcap, int window, int chunk, int bf16,
+                         cudaStream_t st) {
+  RowsParams p{qa, cache, tables, seq_of_row, ctx_lens, nullptr, out, heads, Vp, Vp, Dp, block_size, max_blocks, splits, kv_heads, kLog2e, 1.f, softcap, nullptr,
+               window, chunk, gate, ldg};
+  return rows_form<kPaired>(p, rows, bf16, st);
 }
 }  // namespace tbvops
 
@@ -725,8 +752,8 @@ int tbv_op_latent_attn_rows(const void* qa, const void* cache, const void* table
                             int splits, float scale, int bf16, void* stream) {
   if (R > Rp || (Rp % 16) || (rotp % 16)) return -2;
   RowsParams p{qa, cache, static_cast<const int*>(tables), static_cast<const int*>(seq_of_row), static_cast<const int*>(ctx_lens),
-               static_cast<const float*>(sink), out, heads, R, Rp, rotp, block_size, max_blocks, splits, 1, scale * kLog2e, scale, 0.f, nullptr};
-  return rows_form<false>(p, rows, bf16, static_cast<cudaStream_t>(stream));
+               static_cast<const float*>(sink), out, heads, R, Rp, rotp, block_size, max_blocks, splits, 1, scale * kLog2e, scale, 0.f, nullptr, 0, 0, nullptr, 0};
+  return rows_form<kLatent>(p, rows, bf16, static_cast<cudaStream_t>(stream));
 }
 
 int tbv_op_latent_gather(const void* cache, const void* slots, void* c, void* kr, int n, int Rp, int rotp, void* stream) {

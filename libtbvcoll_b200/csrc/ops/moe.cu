@@ -7,6 +7,9 @@
 //
 // Up to kSmall tokens: one kernel, in which every CTA routes all tokens and moves one.  More: k_route (a warp per token; ranks from atomic
 // counters, so that the order inside an expert is not fixed — no row's result depends on it), then k_dispatch.
+//
+// Where a table gives every token id its experts there is no router: places depend on the ids alone, so one launch lays out all such layers of a model at
+// the start of a step (k_place_table, a CTA per layer), and whoever makes the rows writes them to their places.
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
@@ -166,6 +169,35 @@ __global__ void __launch_bounds__(256) k_dispatch(const RouteParams p) {
   }
 }
 
+// One layer's table and results; as laid out in device memory by the caller.
+struct TableLayer {
+  const int* table;      // [vocab, top]: the experts of every token id, all different
+  int* place;            // [T, top]
+  int* offsets;          // [E + 1]
+  int E, top;
+};
+
+__global__ void __launch_bounds__(1024) k_place_table(const long long* __restrict__ ids, const TableLayer* __restrict__ layers, int T, long long vocab) {
+  __shared__ int cnt[kMaxExperts], off[kMaxExperts + 1];
+  pdl::launch_dependents();
+  const TableLayer l = layers[blockIdx.x];
+  for (int e = threadIdx.x; e < l.E; e += 1024) cnt[e] = 0;
+  __syncthreads();
+  pdl::grid_dependency_wait();
+  const int n = T * l.top;
+  auto expert = [&](int i) {
+    const long long id = ids[i / l.top];
+    const int e = l.table[size_t(id < 0 ? 0 : (id >= vocab ? vocab - 1 : id)) * l.top + i % l.top];
+    return e < 0 ? 0 : (e >= l.E ? l.E - 1 : e);
+  };
+  for (int i = threadIdx.x; i < n; i += 1024) l.place[i] = atomicAdd(&cnt[expert(i)], 1);
+  __syncthreads();
+  if (threadIdx.x < 32) warp_prefix(cnt, off, l.E);
+  __syncthreads();
+  for (int e = threadIdx.x; e <= l.E; e += 1024) l.offsets[e] = off[e];
+  for (int i = threadIdx.x; i < n; i += 1024) l.place[i] += off[expert(i)];
+}
+
 }  // namespace
 
 extern "C" {
@@ -190,6 +222,15 @@ int tbv_op_moe_route(const void* logits, const void* h, void* xp, void* place, v
     if (e == cudaSuccess) e = pdl::launch(k_dispatch, dim3((T + 7) / 8), dim3(256), 0, st, 1, p);
   }
   return e == cudaSuccess ? 0 : -1;
+}
+
+// Places and offsets of `nlayers` layers whose experts come from tables (TableLayer records in device memory: three pointers, experts, top; at most
+// max_experts experts).  ids int64 [T].
+int tbv_op_moe_place_table(const void* ids, const void* layers, int nlayers, int max_experts, int T, long long vocab, void* stream) {
+  if (T <= 0 || nlayers <= 0) return 0;
+  if (max_experts < 1 || max_experts > kMaxExperts || vocab < 1) return -2;
+  return pdl::launch(k_place_table, dim3(nlayers), dim3(1024), 0, static_cast<cudaStream_t>(stream), 1, static_cast<const long long*>(ids),
+                     static_cast<const TableLayer*>(layers), T, vocab) == cudaSuccess ? 0 : -1;
 }
 
 }  // extern "C"

@@ -32,6 +32,10 @@ int gemm_streamk_launch(const void* w, const void* x, void* y, const void* bias,
 // rows form of attention over rows that are keys and values, any size and type (latent_attn.cu)
 int shared_attn_rows_any(const void* qa, const void* cache, const int* tables, const int* seq_of_row, const int* ctx_lens, void* out, int rows,
                          int heads, int kv_heads, int Dp, int block_size, int max_blocks, int splits, float softcap, int bf16, cudaStream_t st);
+// the same over rows that hold a key (Dp columns) and a value (Vp) side by side, with a window or chunks (0: none) and a gate (null: none) on the result
+int paired_attn_rows_any(const void* qa, const void* cache, const int* tables, const int* seq_of_row, const int* ctx_lens, const void* gate, void* out, int rows,
+                         int heads, int kv_heads, int Dp, int Vp, int ldg, int block_size, int max_blocks, int splits, float softcap, int window, int chunk, int bf16,
+                         cudaStream_t st);
 // threads per CTA for the row-normalisation kernels; the fused collective uses the same
 // mapping so that both produce identical bits
 inline int norm_threads(int hidden) {

@@ -8,6 +8,11 @@
 // fp32 pieces, reduced before they are rounded.  For layers that mix every token with the one before, h1 stays fp32; when every
 // sequence has one row (a decode step) the mixes are written here, with the previous token's h1 from the carried state; otherwise
 // k_token_shift writes them from h1.
+//
+// Layers with a norm before and behind every sublayer, x <- x + norm_b(f(norm_a(x))), use the same kernel with a second reduction (POST): the
+// branches' sum goes through a norm of its own before it is added.  If what entered the branch's last product was still to be divided by a root mean
+// square of its row (the joint norm of a recurrence's heads), its square sums come along (`sums`) and the product is divided here.  h1 may
+// go straight to the rows of a row-grouped product (`out_place`) instead of to its own row.
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
@@ -15,8 +20,7 @@
 #include "../pdl.cuh"
 #include "vec.cuh"
 
-using vec::from_f;
-using vec::to_f;
+using vec::sincos_turns;
 
 namespace {
 
@@ -28,7 +32,7 @@ struct ResidualParams {
   // embedding
   const long long* ids;
   const void* table;                // [vocab, ld] in the activation type
-  const float2* freq;               // [ceil(width / 2)]: turns per position, high and low part
+  const float2* freq;               // [ceil(width / 2)]: turns per position, high and low part (null: no position vector)
   const int* positions;
   float embed_scale;
   long long vocab;
@@ -38,11 +42,17 @@ struct ResidualParams {
   const float *y1, *y2, *step;      // [rows, ld], [rows, ld], [ld]
   const void* routed;               // [places, ld] in the activation type
   const int* place;                 // [rows, top]
-  const float* weight;              // [rows, top]
+  const float* weight;              // [rows, top]; null: every weight is `weight_const`
+  float weight_const;
   int top;
+  const float* post;                // POST: [ld] weight of the branches' norm
+  const float* sums;                // POST: [rows, nsum] square sums, or null: the branches are divided by sqrt(their sum / sum_width + eps)
+  int nsum, sum_width;
   // norms
   const float *g1, *g2;
   void *h1, *h2;                    // [rows, ldh]
+  const int* out_place;             // [rows, out_top]: h1 goes to these rows (null: to its own)
+  int out_top;
   int h1_f32;
   const long long* rows;            // last: source row of every output row (null = identity); x is not written
   int last;
@@ -71,42 +81,88 @@ __device__ __forceinline__ void fma4(float4& a, float s, const float4& b) { a.x 
 __device__ __forceinline__ float4 mix4(const float4& h, const float4& prev, const float4& mu) {
   return make_float4(fmaf(prev.x - h.x, mu.x, h.x), fmaf(prev.y - h.y, mu.y, h.y), fmaf(prev.z - h.z, mu.z, h.z), fmaf(prev.w - h.w, mu.w, h.w));
 }
-// sine and cosine of position * 2 pi * f, f = hi + lo turns per position
-__device__ __forceinline__ void sincos_turns(float pos, float2 f, float* s, float* c) {
-  const float t = pos * f.x, e = fmaf(pos, f.x, -t);      // t + e is the exact product
-  const float frac = (t - rintf(t)) + fmaf(pos, f.y, e);
-  sincospif(2.0f * frac, s, c);
+// sums over the block; `red` = 32 floats of shared memory per value
+__device__ __forceinline__ float block_sum(float v, float* red) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float tot = 0.f;
+  for (int w = 0; w < int(blockDim.x + 31) / 32; w++) tot += red[w];
+  return tot;
 }
 
-template <typename T, bool EMBED, int U>
+template <typename T, bool EMBED, bool POST, int U>
 __global__ void __launch_bounds__(kThreads) k_residual(const ResidualParams p) {
-  __shared__ float red[32], sw[kMaxTop];
-  __shared__ int sp[kMaxTop];
+  __shared__ float red[32], red_b[32], red_s[32], sw[kMaxTop];
+  __shared__ int sp[kMaxTop], so[kMaxTop];
   pdl::launch_dependents();
   pdl::grid_dependency_wait();
   const int units = p.ld / 4;
   const size_t row = p.last && p.rows ? size_t(p.rows[blockIdx.x]) : blockIdx.x;
+  if (p.out_place && threadIdx.x < p.out_top) so[threadIdx.x] = p.out_place[row * p.out_top + threadIdx.x];   // read behind a reduction's barrier
   if (!EMBED && p.routed) {
     if (threadIdx.x < p.top) {
       sp[threadIdx.x] = p.place[row * p.top + threadIdx.x];
-      sw[threadIdx.x] = p.weight[row * p.top + threadIdx.x];
+      sw[threadIdx.x] = p.weight ? p.weight[row * p.top + threadIdx.x] : p.weight_const;
     }
     __syncthreads();
   }
   float* xr = p.x + row * p.ld;
-  float4 u[U];
+  float4 u[U], b[POST ? U : 1];
+  if constexpr (POST) {
+    float sb = 0.f, sq = 0.f;
+    if (p.sums)
+      for (int i = threadIdx.x; i < p.nsum; i += blockDim.x) sq += p.sums[row * p.nsum + i];
+#pragma unroll
+    for (int k = 0; k < U; k++) {
+      const int i = threadIdx.x + k * blockDim.x;
+      b[k] = u[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (i < units) {
+        u[k] = load4(xr + i * 4);
+        if (p.y1) b[k] = load4(p.y1 + row * p.ld + i * 4);
+        if (p.routed) {
+          const T* ro = static_cast<const T*>(p.routed) + i * 4;
+#pragma unroll 4
+          for (int j = 0; j < p.top; j++) fma4(b[k], sw[j], load4(ro + size_t(sp[j]) * p.ld));
+        }
+        sb += b[k].x * b[k].x + b[k].y * b[k].y + b[k].z * b[k].z + b[k].w * b[k].w;
+      }
+    }
+    if (p.sums) {
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+      if ((threadIdx.x & 31) == 0) red_s[threadIdx.x >> 5] = sq;
+    }
+    const float tot = block_sum(sb, red_b);
+    float f = 1.f;
+    if (p.sums) {
+      float t = 0.f;
+      for (int w = 0; w < int(blockDim.x + 31) / 32; w++) t += red_s[w];
+      f = 1.0f / sqrtf(t / float(p.sum_width) + p.eps);
+    }
+    f /= sqrtf(tot * f * f / float(p.width) + p.eps);
+#pragma unroll
+    for (int k = 0; k < U; k++) {
+      const int i = threadIdx.x + k * blockDim.x;
+      if (i < units) {
+        const float4 g = load4(p.post + i * 4);
+        b[k] = make_float4(b[k].x * f * g.x, b[k].y * f * g.y, b[k].z * f * g.z, b[k].w * f * g.w);
+      }
+    }
+  }
   float ss = 0.f;
   const T* erow = nullptr;
   float pos = 0.f;
   if (EMBED) {
     const long long id = p.ids[row];
     erow = static_cast<const T*>(p.table) + size_t(id < 0 ? 0 : (id >= p.vocab ? p.vocab - 1 : id)) * p.ld;
-    pos = float(p.positions[row]);
+    if (p.freq) pos = float(p.positions[row]);
   }
 #pragma unroll
   for (int k = 0; k < U; k++) {
     const int i = threadIdx.x + k * blockDim.x;
-    u[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (!POST) u[k] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (i < units) {
       if (EMBED) {
         const float4 e = load4(erow + i * 4);
@@ -114,7 +170,7 @@ __global__ void __launch_bounds__(kThreads) k_residual(const ResidualParams p) {
 #pragma unroll
         for (int j = 0; j < 2; j++) {
           const int c = i * 4 + 2 * j;
-          if (c < p.width) {
+          if (p.freq && c < p.width) {
             float s, co;
             sincos_turns(pos, p.freq[c / 2], &s, &co);
             pv[2 * j] = s;
@@ -123,6 +179,8 @@ __global__ void __launch_bounds__(kThreads) k_residual(const ResidualParams p) {
         }
         u[k] = make_float4(fmaf(e.x, p.embed_scale, pv[0]), fmaf(e.y, p.embed_scale, pv[1]), fmaf(e.z, p.embed_scale, pv[2]), fmaf(e.w, p.embed_scale, pv[3]));
         if (p.x0) store4(p.x0 + row * p.ld + i * 4, u[k]);
+      } else if (POST) {
+        add4(u[k], b[POST ? k : 0]);
       } else {
         u[k] = load4(xr + i * 4);
         float4 b = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -141,13 +199,7 @@ __global__ void __launch_bounds__(kThreads) k_residual(const ResidualParams p) {
       ss += u[k].x * u[k].x + u[k].y * u[k].y + u[k].z * u[k].z + u[k].w * u[k].w;   // pad columns hold zeros
     }
   }
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
-  __syncthreads();
-  float tot = 0.f;
-  for (int w = 0; w < int(blockDim.x + 31) / 32; w++) tot += red[w];
-  const float r = 1.0f / sqrtf(tot / float(p.width) + p.eps);
+  const float r = 1.0f / sqrtf(block_sum(ss, red) / float(p.width) + p.eps);
   float* shift = nullptr;
   bool fresh = true;
   if (p.mu) {
@@ -166,6 +218,8 @@ __global__ void __launch_bounds__(kThreads) k_residual(const ResidualParams p) {
         store4(shift + i * 4, v);
         for (int s = 0; s < p.nmix; s++)
           store4(static_cast<T*>(p.mixes) + (row * p.nmix + s) * p.ld + i * 4, mix4(v, prev, load4(p.mu + size_t(s) * p.ld + i * 4)));
+      } else if (p.out_place) {
+        for (int j = 0; j < p.out_top; j++) store4(static_cast<T*>(p.h1) + size_t(so[j]) * p.ldh + i * 4, v);
       } else if (p.h1_f32) {
         store4(static_cast<float*>(p.h1) + off, v);
       } else {
@@ -197,7 +251,7 @@ __global__ void __launch_bounds__(256) k_token_shift(const float* __restrict__ h
   for (int s = 0; s < nmix; s++) store4(mixes + (size_t(row) * nmix + s) * ld + i, mix4(v, prev, load4(mu + size_t(s) * ld + i)));
 }
 
-template <typename T, bool EMBED>
+template <typename T, bool EMBED, bool POST>
 cudaError_t launch_u(const ResidualParams& p, int rows, cudaStream_t st) {
   const int units = p.ld / 4;
   const int per = units <= 64 ? 1 : (units <= kThreads * 2 ? 2 : (units <= kThreads * 4 ? 4 : (units <= kThreads * 8 ? 8 : 16)));
@@ -206,37 +260,47 @@ cudaError_t launch_u(const ResidualParams& p, int rows, cudaStream_t st) {
   if (threads < kMaxTop) threads = kMaxTop;
   const dim3 grid(rows), blk(threads);
   switch (per) {
-    case 1: return pdl::launch(k_residual<T, EMBED, 1>, grid, blk, 0, st, 1, p);
-    case 2: return pdl::launch(k_residual<T, EMBED, 2>, grid, blk, 0, st, 1, p);
-    case 4: return pdl::launch(k_residual<T, EMBED, 4>, grid, blk, 0, st, 1, p);
-    case 8: return pdl::launch(k_residual<T, EMBED, 8>, grid, blk, 0, st, 1, p);
-    default: return pdl::launch(k_residual<T, EMBED, 16>, grid, blk, 0, st, 1, p);
+    case 1: return pdl::launch(k_residual<T, EMBED, POST, 1>, grid, blk, 0, st, 1, p);
+    case 2: return pdl::launch(k_residual<T, EMBED, POST, 2>, grid, blk, 0, st, 1, p);
+    case 4: return pdl::launch(k_residual<T, EMBED, POST, 4>, grid, blk, 0, st, 1, p);
+    case 8: return pdl::launch(k_residual<T, EMBED, POST, 8>, grid, blk, 0, st, 1, p);
+    default: return pdl::launch(k_residual<T, EMBED, POST, 16>, grid, blk, 0, st, 1, p);
   }
+}
+template <typename T>
+cudaError_t launch_t(const ResidualParams& p, int rows, cudaStream_t st) {
+  if (p.ids) return launch_u<T, true, false>(p, rows, st);
+  return p.post ? launch_u<T, false, true>(p, rows, st) : launch_u<T, false, false>(p, rows, st);
 }
 
 }  // namespace
 
 extern "C" {
 
-// See the top of the file.  ids != null: the embedding (y1, y2, routed ignored).  mu != null: the mixes are written instead of h1.
+// See the top of the file.  ids != null: the embedding (y1, y2, routed ignored; freq null: no position vector).  mu != null: the mixes are written
+// instead of h1.  post != null: the branches' norm (y2, x0, step and mixes do not go with it).  weight null: every weight is weight_const.
 int tbv_op_residual(const void* ids, const void* table, const void* freq, const void* positions, float embed_scale, long long vocab, void* x,
                     void* x0, const void* y1, const void* y2, const void* step, const void* routed, const void* place, const void* weight, int top,
                     const void* g1, const void* g2, void* h1, void* h2, int h1_f32, const void* row_map, int last, const void* mu, void* mixes,
-                    void* shift, const void* segs, int nmix, int rows, int width, int ld, int ldh, float eps, int bf16, void* stream) {
+                    void* shift, const void* segs, int nmix, const void* post, const void* sums, int nsum, int sum_width, float weight_const, const void* out_place,
+                    int out_top, int rows, int width, int ld, int ldh, float eps, int bf16, void* stream) {
   if (rows <= 0) return 0;
   if (width <= 0 || width > ld || (ld % 4) || (ldh % 4) || ld > kThreads * 4 * kMaxUnits || ldh < ld || (routed && (top < 1 || top > kMaxTop))) return -2;
+  if (post && (ids || y2 || x0 || step || mu)) return -2;
+  if ((sums && (!post || nsum <= 0 || sum_width <= 0)) || (out_place && (last || (h1_f32 && bf16) || mu || out_top < 1 || out_top > kMaxTop))) return -2;
   if (mu && (last || !segs || !positions || !shift || !mixes)) return -2;
   ResidualParams p{};
   p.ids = static_cast<const long long*>(ids); p.table = table; p.freq = static_cast<const float2*>(freq); p.positions = static_cast<const int*>(positions);
   p.embed_scale = embed_scale; p.vocab = vocab;
   p.x = static_cast<float*>(x); p.x0 = static_cast<float*>(x0); p.y1 = static_cast<const float*>(y1); p.y2 = static_cast<const float*>(y2);
-  p.step = static_cast<const float*>(step); p.routed = routed; p.place = static_cast<const int*>(place); p.weight = static_cast<const float*>(weight); p.top = top;
+  p.step = static_cast<const float*>(step); p.routed = routed; p.place = static_cast<const int*>(place); p.weight = static_cast<const float*>(weight); p.weight_const = weight_const; p.top = top;
+  p.post = static_cast<const float*>(post); p.sums = static_cast<const float*>(sums); p.nsum = nsum; p.sum_width = sum_width;
+  p.out_place = static_cast<const int*>(out_place); p.out_top = out_top;
   p.g1 = static_cast<const float*>(g1); p.g2 = static_cast<const float*>(g2); p.h1 = h1; p.h2 = h2; p.h1_f32 = h1_f32;
   p.rows = static_cast<const long long*>(row_map); p.last = last; p.mu = static_cast<const float*>(mu); p.mixes = mixes; p.shift = static_cast<float*>(shift);
   p.segs = static_cast<const int*>(segs); p.nmix = nmix; p.width = width; p.ld = ld; p.ldh = ldh; p.eps = eps;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  cudaError_t e = ids ? (bf16 ? launch_u<__nv_bfloat16, true>(p, rows, st) : launch_u<float, true>(p, rows, st))
-                      : (bf16 ? launch_u<__nv_bfloat16, false>(p, rows, st) : launch_u<float, false>(p, rows, st));
+  cudaError_t e = bf16 ? launch_t<__nv_bfloat16>(p, rows, st) : launch_t<float>(p, rows, st);
   return e == cudaSuccess ? 0 : -1;
 }
 

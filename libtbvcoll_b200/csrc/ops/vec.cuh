@@ -1,5 +1,5 @@
-// vec.cuh — small helpers of the kernels that run on bf16 or fp32 activations: conversions, eight-wide loads and stores, SiLU, and
-// packed pairs of fp32 values.
+// vec.cuh — small helpers of the kernels that run on bf16 or fp32 activations: conversions, eight-wide loads and stores, SiLU, sigmoid,
+// angles, and packed pairs of fp32 values.
 #pragma once
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
@@ -17,6 +17,10 @@ template <typename T> __device__ __forceinline__ float gate(float v);
 template <> __device__ __forceinline__ float gate<float>(float v) { return silu(v); }
 template <> __device__ __forceinline__ float gate<__nv_bfloat16>(float v) { return __fdividef(v, 1.0f + __expf(-v)); }
 
+template <typename T> __device__ __forceinline__ float sigmoid(float v);
+template <> __device__ __forceinline__ float sigmoid<float>(float v) { return 1.0f / (1.0f + expf(-v)); }
+template <> __device__ __forceinline__ float sigmoid<__nv_bfloat16>(float v) { return __fdividef(1.0f, 1.0f + __expf(-v)); }
+
 __device__ __forceinline__ void load8(const float* p, float* f) {
   const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
   f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
@@ -32,11 +36,13 @@ __device__ __forceinline__ void load8(const __nv_bfloat16* p, float* f) {
 template <typename T> struct Raw8;
 template <> struct Raw8<float> {
   float4 a, b;
+  __device__ __forceinline__ void store(float* p) const { *reinterpret_cast<float4*>(p) = a; *reinterpret_cast<float4*>(p + 4) = b; }
   __device__ __forceinline__ void load(const float* p) { a = *reinterpret_cast<const float4*>(p); b = *reinterpret_cast<const float4*>(p + 4); }
   __device__ __forceinline__ void unpack(float* f) const { f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w; }
 };
 template <> struct Raw8<__nv_bfloat16> {
   uint4 v;
+  __device__ __forceinline__ void store(__nv_bfloat16* p) const { *reinterpret_cast<uint4*>(p) = v; }
   __device__ __forceinline__ void load(const __nv_bfloat16* p) { v = *reinterpret_cast<const uint4*>(p); }
   __device__ __forceinline__ void unpack(float* f) const {
     f[0] = __uint_as_float(v.x << 16); f[1] = __uint_as_float(v.x & 0xffff0000u);
@@ -57,6 +63,13 @@ __device__ __forceinline__ void store8(__nv_bfloat16* p, const float* f) {
     w[i] = *reinterpret_cast<uint32_t*>(&v);
   }
   *reinterpret_cast<uint4*>(p) = make_uint4(w[0], w[1], w[2], w[3]);
+}
+
+// sine and cosine of position * 2 pi * f, f = hi + lo turns per position; the angle is reduced before it is rounded
+__device__ __forceinline__ void sincos_turns(float pos, float2 f, float* s, float* c) {
+  const float t = pos * f.x, e = fmaf(pos, f.x, -t);      // t + e is the exact product
+  const float frac = (t - rintf(t)) + fmaf(pos, f.y, e);
+  sincospif(2.0f * frac, s, c);
 }
 
 // Two fp32 values in a 64-bit register pair: one instruction does both (each rounded as its scalar form).

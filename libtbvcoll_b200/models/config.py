@@ -354,9 +354,146 @@ def tinapel_like(hidden: int, layers: int, ff: int, heads: int, kv_heads: int, v
     return TinapelConfig(name=name, vocab_size=vocab, hidden_size=hidden, layers=lay)
 
 
+# ---- Bobarax: fixed-decay recurrences, windowed and chunked attention, a norm before and behind every sublayer -----------------------
+@dataclass
+class LightningSpec:
+    heads: int
+    dim: int                               # key channels per head
+    vdim: int
+    decay: List[float] = field(default_factory=list)   # one constant per head
+
+
+@dataclass
+class PairedAttentionSpec:
+    """Grouped-query attention with one cached row (key, value) per token and key head; queries and keys are normed over the whole projection."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    softcap: Optional[float] = None
+    window: int = 0                        # a position sees itself and the window - 1 before it (0: no such limit)
+    chunk: int = 0                         # a position sees its own chunk of positions only (0: no such limit)
+    rot: Optional[RotationSpec] = None     # None: positions do not enter the scores
+    gated: bool = False                    # sigmoid gate on the result
+    kv_from: Optional[int] = None          # keys and values of that layer instead of its own
+
+
+@dataclass
+class GatedMlpSpec:
+    ff: int                                # relu(gate) * up
+
+
+@dataclass
+class TableMoeSpec:
+    """Mixture of experts without a router: a table gives every token id its experts, equally weighted."""
+    experts: int
+    top: int
+    ff: int
+    limit: float                           # of the experts' clamped gated unit
+    slope: float = 1.702
+
+
+@dataclass
+class SandwichLayerSpec:
+    mixer: Union[LightningSpec, PairedAttentionSpec]
+    mlp: Optional[Union[GatedMlpSpec, TableMoeSpec]] = None
+
+
+@dataclass
+class BobaraxConfig:
+    name: str
+    vocab_size: int
+    hidden_size: int
+    layers: List[SandwichLayerSpec]
+    residual_mult: float = 1.0
+    logit_scale: float = 1.0
+    rms_eps: float = 1e-5
+
+    def __post_init__(self):
+        for i, lay in enumerate(self.layers):
+            m, f = lay.mixer, lay.mlp
+            if isinstance(m, LightningSpec):
+                if len(m.decay) != m.heads or not all(0.0 <= a <= 1.0 for a in m.decay):
+                    raise ValueError(f"layer {i}: {len(m.decay)} decays (each 0 to 1) for {m.heads} heads")
+            else:
+                if m.kv_heads < 1 or m.heads % m.kv_heads:
+                    raise ValueError(f"layer {i}: {m.heads} query heads on {m.kv_heads} key heads")
+                if m.window < 0 or m.chunk < 0 or (m.window and m.chunk):
+                    raise ValueError(f"layer {i}: a window of {m.window} and chunks of {m.chunk} positions")
+                if m.rot is not None and (m.rot.dims % 2 or not 0 <= m.rot.dims <= m.dim):
+                    raise ValueError(f"layer {i}: {m.rot.dims} rotated dimensions of {m.dim}")
+                if m.kv_from is not None:
+                    j = m.kv_from
+                    s = self.layers[j].mixer if 0 <= j < i else None
+                    if not isinstance(s, PairedAttentionSpec) or s.kv_from is not None or (s.kv_heads, s.dim, s.vdim, s.rot) != (m.kv_heads, m.dim, m.vdim, m.rot):
+                        raise ValueError(f"layer {i}: layer {j} has no keys and values that fit")
+            if isinstance(f, TableMoeSpec) and not 1 <= f.top <= f.experts:
+                raise ValueError(f"layer {i}: {f.top} of {f.experts} experts")
+
+    def check_tp(self, tp: int) -> None:
+        if tp != 1:
+            raise ValueError("Bobarax models run on one GPU (no tensor-parallel sharding of the recurrent states and the paired cache rows)")
+
+    @property
+    def num_layers(self) -> int:
+        return len(self.layers)
+
+    def param_count(self) -> int:
+        from ..utils.weights import tensor_shapes
+        return sum(math.prod(s) for s in tensor_shapes(self).values())
+
+
+def parse_bobarax_config(c: dict) -> BobaraxConfig:
+    """``config.json`` of a Bobarax checkpoint."""
+    layers = []
+    for i, e in enumerate(c["layers"]):
+        m, f, kind = e["mixer"], e.get("mlp"), e["type"]
+        if kind == "lightning":
+            mixer = LightningSpec(heads=m["heads"], dim=m["dim"], vdim=m["vdim"], decay=[float(a) for a in m["decay"]])
+        elif kind in ("attention", "attention_2"):
+            rot, cap, mask = m.get("rot") if kind == "attention_2" else None, m.get("softcap"), m.get("mask") or {"size": 0}
+            mixer = PairedAttentionSpec(heads=m["heads"], kv_heads=m.get("kv_heads", m["heads"]), dim=m["dim"], vdim=m.get("vdim", m["dim"]), scale=float(m["scale"]),
+                                        softcap=float(cap) if cap else None, window=mask["size"] if kind == "attention_2" else 0,
+                                        chunk=mask["size"] if kind == "attention" else 0, rot=RotationSpec(rot["dims"], float(rot["base"])) if rot else None,
+                                        gated=kind == "attention_2", kv_from=m.get("kv_from"))
+        else:
+            raise ValueError(f"layer {i}: unknown type {kind!r}")
+        if f is None:
+            mlp = None
+        elif f.get("kind") == "dense":
+            mlp = GatedMlpSpec(ff=f["ff"])
+        elif f.get("kind") == "moe":
+            mlp = TableMoeSpec(experts=f["router"]["experts"], top=f["router"]["top"], ff=f["expert"]["ff"], limit=float(f["expert"]["limit"]))
+        else:
+            raise ValueError(f"layer {i}: unknown feed-forward {f.get('kind')!r}")
+        layers.append(SandwichLayerSpec(mixer, mlp))
+    return BobaraxConfig(name=c.get("name", "bobarax"), vocab_size=c["vocab"], hidden_size=c["width"], layers=layers, residual_mult=float(c.get("residual_mult", 1.0)),
+                         logit_scale=float(c.get("logit_scale", 1.0)), rms_eps=float(c["norm"]["eps"]))
+
+
+def bobarax_like(hidden: int, layers: int, ff: int, heads: int, kv_heads: int, vocab: int, head_dim: int = 128, experts: int = 8, top: int = 2,
+                 window: int = 4096, chunk: int = 8192, name: str = "bobarax") -> BobaraxConfig:
+    """A Bobarax of ordinary proportions: layers in turn lightning, windowed attention, lightning, chunked attention, every fourth windowed layer with the keys
+    and values of the one before; every other feed-forward a mixture of experts of which a token meets ``ff`` in all, the others dense."""
+    lay = []
+    for i in range(layers):
+        if i % 2 == 0:
+            mixer = LightningSpec(heads, head_dim, head_dim, [math.exp(-2.0 ** (-0.5 - 8.0 * h / heads)) for h in range(heads)])
+        elif i % 4 == 1:
+            mixer = PairedAttentionSpec(heads, kv_heads, head_dim, head_dim, head_dim ** -0.5, window=window, rot=RotationSpec(head_dim // 2, 5e5), gated=True,
+                                        kv_from=i - 4 if i % 16 == 13 else None)
+        else:
+            mixer = PairedAttentionSpec(heads, kv_heads, head_dim, head_dim, head_dim ** -0.5, softcap=50.0, chunk=chunk)
+        lay.append(SandwichLayerSpec(mixer, TableMoeSpec(experts, top, ff // top, 7.0) if i // 2 % 2 else GatedMlpSpec(ff)))
+    return BobaraxConfig(name=name, vocab_size=vocab, hidden_size=hidden, layers=lay, residual_mult=0.8, logit_scale=hidden ** -0.5)
+
+
 PRESETS["nubosun-8b"] = nubosun_like(4096, 32, 14336, 32, 128256, name="nubosun-8b")
 PRESETS["nubosun-2k"] = nubosun_like(2048, 16, 7168, 16, 32768, name="nubosun-2k")
 PRESETS["llama3-2k"] = ModelConfig(name="llama3-2k", hidden_size=2048, num_layers=16, num_heads=16, num_kv_heads=4, intermediate_size=7168,
                                    vocab_size=32768)
 PRESETS["tinapel-8b"] = tinapel_like(4096, 32, 14336, 32, 8, 128256, name="tinapel-8b")
 PRESETS["tinapel-2k"] = tinapel_like(2048, 16, 7168, 16, 4, 32768, name="tinapel-2k")
+PRESETS["bobarax-8b"] = bobarax_like(4096, 32, 14336, 32, 8, 128256, name="bobarax-8b")
+PRESETS["bobarax-2k"] = bobarax_like(2048, 16, 7168, 16, 4, 32768, name="bobarax-2k")

@@ -5,9 +5,10 @@ from __future__ import annotations
 import json
 import os
 from dataclasses import dataclass
-from typing import Callable, Tuple
+from typing import Callable, Optional, Tuple
 
-from .config import ModelConfig, NubosunConfig, TinapelConfig, from_hf_config, parse_nubosun_config, parse_tinapel_config
+from .config import (BobaraxConfig, ModelConfig, NubosunConfig, TinapelConfig, from_hf_config, parse_bobarax_config, parse_nubosun_config,
+                     parse_tinapel_config)
 
 
 @dataclass(frozen=True)
@@ -17,6 +18,7 @@ class Architecture:
     model: Callable[[], type]              # imported on use: the model modules need the native library
     dtypes: Tuple[str, ...]                # compute types the model runs in
     tensor_parallel: bool
+    parse: Optional[Callable[[dict], object]] = None   # config.json that names this architecture (None: the HF layout)
 
 
 def _llama():
@@ -34,10 +36,16 @@ def _tinapel():
     return Tinapel
 
 
+def _bobarax():
+    from .bobarax import Bobarax
+    return Bobarax
+
+
 ARCHITECTURES = {
     "llama": Architecture("llama", ModelConfig, _llama, ("bfloat16",), True),
-    "nubosun": Architecture("nubosun", NubosunConfig, _nubosun, ("bfloat16", "float32"), False),
-    "tinapel": Architecture("tinapel", TinapelConfig, _tinapel, ("bfloat16", "float32"), False),
+    "nubosun": Architecture("nubosun", NubosunConfig, _nubosun, ("bfloat16", "float32"), False, parse_nubosun_config),
+    "tinapel": Architecture("tinapel", TinapelConfig, _tinapel, ("bfloat16", "float32"), False, parse_tinapel_config),
+    "bobarax": Architecture("bobarax", BobaraxConfig, _bobarax, ("bfloat16", "float32"), False, parse_bobarax_config),
 }
 
 
@@ -54,10 +62,8 @@ def load_config(model_dir: str):
     with open(path) as f:
         c = json.load(f)
     arch = str(c.get("architecture", "")).lower()
-    if arch == "nubosun":
-        return parse_nubosun_config(c)
-    if arch == "tinapel":
-        return parse_tinapel_config(c)
+    if arch in ARCHITECTURES and ARCHITECTURES[arch].parse is not None:
+        return ARCHITECTURES[arch].parse(c)
     if arch:
         raise ValueError(f"unknown architecture {c['architecture']!r}")
     return from_hf_config(path)            # Llama / Qwen2 families in the HF layout

@@ -23,24 +23,12 @@ from .. import ops
 from ..engine.batch import StepBatch
 from ..parallel.tp import TPGroup
 from .config import GlaSpec, MoeSpec, SharedKvSpec, TinapelConfig, WkvSpec
+from .decoder import StreamDecoder, pad16 as _pad16
 
 
-def _pad16(n: int) -> int:
-    return (n + 15) // 16 * 16
-
-
-class Tinapel:
-    # portions of at most this many tokens take the attention's rows form
-    ROWS_FORM_MAX = 32
+class Tinapel(StreamDecoder):
     # from this many rows on, the mixes of a WKV layer go through separate many-token products instead of the grouped one
     GROUPED_MAX = 384
-    uses_state = True
-    expands_context = False
-
-    @staticmethod
-    def attn_cta_slots(splits: int, sms: int) -> int:
-        """CTAs of the rows kernel that run at once: two per SM, but clusters of eight find only about four fifths of the places."""
-        return 2 * sms if splits < 8 else 2 * sms * 4 // 5
 
     def __init__(self, cfg: TinapelConfig, tp: TPGroup, weights: Dict[str, torch.Tensor], device, max_tokens: int, max_batch: int,
                  num_blocks: int, block_size: int = 16, max_attn_splits: int = 8, dtype: torch.dtype = torch.bfloat16):
@@ -48,7 +36,7 @@ class Tinapel:
         self.cfg, self.w, self.device, self.dtype = cfg, weights, torch.device(device), dtype
         self.block_size, self.num_blocks, self.max_tokens, self.max_batch, self.max_attn_splits = block_size, num_blocks, max_tokens, max_batch, max_attn_splits
         dev, f32, T = self.device, torch.float32, max_tokens
-        self.W, self.Wp, self.Vp = cfg.hidden_size, _pad16(cfg.hidden_size), _pad16(cfg.vocab_size)
+        self.W, self.Wp = cfg.hidden_size, _pad16(cfg.hidden_size)
         zeros = lambda *shape, dt=dtype: torch.zeros(*shape, dtype=dt, device=dev)
         big = lambda sizes: max(sizes, default=0)
         mixers = [(i, l.mixer) for i, l in enumerate(cfg.layers)]
@@ -82,10 +70,7 @@ class Tinapel:
         }
         self.offsets = zeros(big([f.experts for f in moes]) + 1, dt=torch.int32)
         self.counts = zeros(big([f.experts for f in moes]), dt=torch.int32)
-        self.hl = zeros(max_batch, self.Wp)
-        self.logits = zeros(max_batch, self.Vp, dt=f32)
-        self.argmax_ws = ops.argmax_workspace(max_batch, dev)
-        self.argmax_val = zeros(max_batch, dt=f32)
+        self._init_head()
         # cache and state, one per layer run (a looped layer has one per pass); slot 0 of the state is never a sequence's
         self.cache, self.state, self.shift = [], [], []
         slots = max_batch + 1
@@ -102,16 +87,6 @@ class Tinapel:
         two_forms = bool(attns) and dtype is torch.bfloat16 and all(_pad16(m.dim) <= ops.SHARED_PREFILL_MAX_DIM for m in attns)
         self.rows_form_max = self.ROWS_FORM_MAX if two_forms else 1 << 60
 
-    def scan_group_rows(self, rows) -> int:
-        """Rows per group of the chunked recurrence for segments of the given lengths; 0: the sequential (32-bit) kernel.  Cutting a segment costs a
-        second pass over its keys and values, so it is done only as far as the GPU would otherwise be short of CTAs."""
-        if self.dtype is not torch.bfloat16 or not self.scan_heads:
-            return 0
-        sms = torch.cuda.get_device_properties(self.device).multi_processor_count
-        fair = max(256, -(-int(rows.sum()) * self.scan_heads // (2 * sms * 16)) * 16)
-        longest = -(-int(rows.max()) // 16) * 16
-        return longest if 2 * longest <= 3 * fair else fair
-
     def _group_scratch(self, groups: int) -> tuple:
         """(states, decay totals) of the groups of cut segments, grown on demand (never inside a captured step)."""
         if groups > self._groups:
@@ -125,12 +100,6 @@ class Tinapel:
     def load_weights(cfg: TinapelConfig, source, tp: TPGroup, device, dtype):
         from ..utils.weights import load_tinapel
         return load_tinapel(cfg, source, device, dtype)
-
-    def _buf(self, name: str, rows: int, *shape: int) -> torch.Tensor:
-        n = rows
-        for s in shape:
-            n *= s
-        return self._flat[name][:n].view(rows, *shape)
 
     def _scan(self, b: StepBatch, run: int, p: str, q, k, v, g, low, V: int, out, args: dict) -> None:
         """Recurrence over many rows; ``low`` is what enters the second decay product, which the chunked kernels do themselves."""
@@ -270,7 +239,7 @@ class Tinapel:
         layer_end = len(schedule) if layer_end is None else layer_end
         assert 0 < T <= self.max_tokens
         n = b.n_logits
-        hl = self.hl[:n] if n <= self.max_batch else torch.empty(n, self.Wp, dtype=self.dtype, device=self.device)
+        hl = self._head_rows(n)
         if layer_begin == 0:
             embed = (b.ids, w["embed"][: cfg.vocab_size], cfg.embedding_scale, self.turns)
             x0 = {} if self.x0 is None else {"x0": self.x0[:T]}
@@ -291,10 +260,4 @@ class Tinapel:
                 self._leave(b, hl, **terms)
         if layer_end < len(schedule) or not n:
             return
-        logits = self.logits[:n] if n <= self.max_batch else torch.empty(n, self.Vp, dtype=torch.float32, device=self.device)
-        ops.linear(hl, w["embed"], logits)
-        if b.logits_out is not None:
-            b.logits_out.copy_(logits[:, : cfg.vocab_size])
-        if b.out_tokens is not None:
-            assert n <= self.max_batch
-            ops.argmax(logits[:, : cfg.vocab_size], self.argmax_ws, 0, self.argmax_val[:n], b.out_tokens[:n])
+        self._head(b, hl)

@@ -33,12 +33,20 @@ def lib():
     I, F, LL, SZ = ctypes.c_int, ctypes.c_float, ctypes.c_longlong, ctypes.c_size_t
     l.tbv_op_gemm.argtypes = [c_vp, c_vp, c_vp, c_vp, I, I, I, I, I, I, I, c_vp]
     l.tbv_op_gemm_error.restype = I
-    l.tbv_op_gemm_ex.argtypes = [c_vp, c_vp, c_vp, c_vp, c_vp, I, I, I, I, I, I, I, F, F, F, I, I, I, I, c_vp]
-    l.tbv_op_gemm_f32.argtypes = [c_vp, c_vp, c_vp, c_vp, I, I, I, I, I, I, I, F, F, F, I, I, I, I, c_vp]
+    l.tbv_op_gemm_ex.argtypes = [c_vp, c_vp, c_vp, c_vp, c_vp, I, I, I, I, I, I, I, F, F, F, I, I, I, I, I, c_vp]
+    l.tbv_op_gemm_f32.argtypes = [c_vp, c_vp, c_vp, c_vp, I, I, I, I, I, I, I, F, F, F, I, I, I, I, I, c_vp]
     l.tbv_op_gemm_rows.argtypes = l.tbv_op_gemm_rows_f32.argtypes = [c_vp] * 4 + [I] * 8 + [F, F, F, c_vp]
-    l.tbv_op_residual.argtypes = [c_vp] * 4 + [F, LL] + [c_vp] * 8 + [I] + [c_vp] * 4 + [I, c_vp, I] + [c_vp] * 4 + [I] * 5 + [F, I, c_vp]
+    l.tbv_op_residual.argtypes = [c_vp] * 4 + [F, LL] + [c_vp] * 8 + [I] + [c_vp] * 4 + [I, c_vp, I] + [c_vp] * 4 + [I, c_vp, c_vp, I, I, F, c_vp] + [I] * 5 + [F, I, c_vp]
     l.tbv_op_token_shift.argtypes = [c_vp] * 7 + [I] * 4 + [c_vp]
     l.tbv_op_moe_route.argtypes = [c_vp] * 8 + [I] * 4 + [F, I, c_vp]
+    l.tbv_op_moe_place_table.argtypes = [c_vp, c_vp, I, I, I, LL, c_vp]
+    l.tbv_op_fixed_decay_scan.argtypes = [c_vp] * 13 + [I, I, c_vp] + [I] * 8 + [c_vp]
+    l.tbv_op_fixed_decay_step.argtypes = [c_vp] * 11 + [I] * 7 + [c_vp]
+    l.tbv_op_fixed_decay_sums.argtypes = [I, I, I]
+    l.tbv_op_paired_attn_prep.argtypes = [c_vp] * 8 + [I] * 10 + [F, I, c_vp]
+    l.tbv_op_paired_attn_rows.argtypes = [c_vp] * 7 + [I] * 9 + [F, I, I, I, c_vp]
+    l.tbv_op_paired_attn_prefill.argtypes = [c_vp] * 7 + [I] * 10 + [F, I, I, c_vp]
+    l.tbv_op_paired_prefill_fits.argtypes = [I, I]
     l.tbv_op_decay_scan.argtypes = [c_vp] * 15 + [I, I, c_vp, c_vp, c_vp, c_vp, c_vp] + [I] * 12 + [F, F, F, I, c_vp]
     l.tbv_op_decay_step.argtypes = [c_vp] * 13 + [I] * 9 + [F, F, F, I, c_vp]
     l.tbv_op_shared_attn_prep.argtypes = [c_vp] * 6 + [I] * 8 + [F, F, ctypes.c_double, I, c_vp]
@@ -124,8 +132,9 @@ def _count(n=1):
 
 
 EPI_STORE, EPI_SILU_MUL, EPI_F32, EPI_CLAMP_GLU = 0, 1, 2, 3
-ACT_NONE, ACT_SOFTPLUS, ACT_SOFTCAP = 0, 1, 2          # a soft cap of 1 is tanh
+ACT_NONE, ACT_SOFTPLUS, ACT_SOFTCAP, ACT_SILU = 0, 1, 2, 3          # a soft cap of 1 is tanh
 SILU_GLU = (math.inf, 1.0, 0.0)           # ``glu`` of ``linear``: silu(gate) * up
+RELU_GLU = (math.inf, math.inf, 0.0)      # relu(gate) * up
 
 
 def gemm(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None,
@@ -154,11 +163,12 @@ def gemm(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, b
 
 def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[torch.Tensor] = None, act: int = ACT_NONE, act_arg: float = 0.0,
            glu: Optional[tuple] = None, copy: Optional[torch.Tensor] = None, groups: int = 1, x_group: int = 0, y_group: int = 0,
-           last: int = 0) -> torch.Tensor:
+           last: int = 0, act_cols: int = 0) -> torch.Tensor:
     """out[N, M] = epilogue(x[N, K] @ w[M, K]^T + bias) for bf16 operands (tcgen05) or fp32 operands (CUDA cores, full 32-bit).
 
-    The output dtype is ``out``'s: fp32 results take an activation (``ACT_SOFTPLUS``, ``ACT_SOFTCAP`` with its limit in ``act_arg``)
-    and, from bf16 operands, an optional bf16 ``copy`` with the same row stride.  ``glu=(limit, slope[, shift = 1])``: ``w`` holds gate / up rows
+    The output dtype is ``out``'s: fp32 results take an activation (``ACT_SOFTPLUS``, ``ACT_SOFTCAP`` with its limit in ``act_arg``, ``ACT_SILU``)
+    and, from bf16 operands, an optional bf16 ``copy`` with the same row stride; ``act_cols`` > 0 (a multiple of 16; results of the operands' dtype): the
+    activation acts on that many leading columns.  ``glu=(limit, slope[, shift = 1])``: ``w`` holds gate / up rows
     interleaved and out[N, M/2] = g * sigmoid(slope * g) * (u + shift) with g = min(gate, limit), u = clamp(up, -limit, limit).
     ``groups`` > 1: w is [groups * M + last, K]; group g multiplies columns g * x_group .. of x and writes columns g * y_group .. of out; ``last``
     features (0 = none) form one more group."""
@@ -171,16 +181,18 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[t
     if N == 0:
         return out
     limit, slope, shift = (*glu, 1.0)[:3] if glu else (act_arg, 0.0, 0.0)
+    act_m = act_cols or 1 << 30
+    assert act_cols % 16 == 0 and (not act_cols or (out.dtype is x.dtype and glu is None and groups == 1))
     if x.dtype is torch.float32:
         assert out.dtype is torch.float32 and copy is None and (bias is None or bias.dtype is torch.float32)
         _chk(lib().tbv_op_gemm_f32(_p(w), _p(x), _p(out), _p(bias), M, N, K, x.stride(0), out.stride(0), EPI_CLAMP_GLU if glu else EPI_F32, act,
-                                   limit, slope, shift, groups, x_group, y_group, last, _st()), "tbv_op_gemm_f32")
+                                   limit, slope, shift, act_m, groups, x_group, y_group, last, _st()), "tbv_op_gemm_f32")
     else:
         epi = EPI_CLAMP_GLU if glu else (EPI_F32 if out.dtype is torch.float32 else EPI_STORE)
-        assert x.dtype is torch.bfloat16 and (bias is None or bias.dtype is torch.bfloat16) and (epi == EPI_F32 or (act == ACT_NONE and copy is None))
+        assert x.dtype is torch.bfloat16 and (bias is None or bias.dtype is torch.bfloat16) and (epi == EPI_F32 or ((act == ACT_NONE or act_cols) and copy is None))
         assert copy is None or (copy.dtype is torch.bfloat16 and copy.stride(0) == out.stride(0))
         _chk(lib().tbv_op_gemm_ex(_p(w), _p(x), _p(out), _p(copy), _p(bias), M, N, K, x.stride(0), out.stride(0), epi, act, limit, slope, shift,
-                                  groups, x_group, y_group, last, _st()), "tbv_op_gemm_ex")
+                                  act_m, groups, x_group, y_group, last, _st()), "tbv_op_gemm_ex")
     _count()
     return out
 
@@ -439,6 +451,8 @@ def prefill_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
     return out
 
 
-from .mixers import (DECAY_RANK_MAX, SHARED_PREFILL_MAX_DIM, causal_conv_silu, decay_scan, decay_step, hyper_embed, hyper_mix,  # noqa: E402,F401
-                     latent_attention_prefill, latent_attention_rows, latent_gather, latent_prefill_fits, latent_prep, latent_row, moe_route,
-                     position_turns, residual, selective_scan, shared_attention_prefill, shared_attention_prep, shared_attention_rows, token_shift)
+from .mixers import (DECAY_RANK_MAX, SHARED_PREFILL_MAX_DIM, causal_conv_silu, decay_powers, decay_scan, decay_step, fixed_decay_scan,  # noqa: E402,F401
+                     fixed_decay_step, fixed_decay_sums, hyper_embed, hyper_mix, latent_attention_prefill, latent_attention_rows, latent_gather,
+                     latent_prefill_fits, latent_prep, latent_row, moe_place_table, moe_route, moe_table_layers, paired_attention_prefill, paired_attention_prep,
+                     paired_attention_rows, paired_prefill_fits, position_turns, residual, rotation_turns, selective_scan, shared_attention_prefill,
+                     shared_attention_prep, shared_attention_rows, token_shift)

@@ -1,6 +1,6 @@
 """Entry points of the mixer operators: residual streams with hyper-connections, one residual stream with parallel branches, short
-convolution + selective scan and linear recurrences over carried state, attention over a compressed (latent) paged cache and over
-a cache whose rows are keys and values at once, and the routing of a mixture of experts.  bf16 or fp32 activations; what enters a softmax, a
+convolution + selective scan and linear recurrences over carried state, attention over a compressed (latent) paged cache, over
+a cache whose rows are keys and values at once and over one with both side by side, and the routing of a mixture of experts.  bf16 or fp32 activations; what enters a softmax, a
 norm, a recurrence or the residual sum is fp32 in both.
 
 ``segs`` is the device int32 [nseg, 4] list of a ragged batch: (first row, rows, state slot, 0) per sequence, rows of a
@@ -121,36 +121,55 @@ def latent_attention_prefill(qkv, q_rot_off: int, kv, kr, tiles, sink, out, head
 # ---- one residual stream with parallel branches -----------------------------------------------------------------------------
 def position_turns(width: int, device, base: float = 10000.0) -> torch.Tensor:
     """fp32 [ceil(width / 2), 2]: turns per position of every sine / cosine pair of the position vector, as high and low part."""
-    f = base ** (-2.0 * torch.arange((width + 1) // 2, dtype=torch.float64) / width) / (2.0 * math.pi)
+    return _turns(base ** (-2.0 * torch.arange((width + 1) // 2, dtype=torch.float64) / width), device)
+
+
+def rotation_turns(dims: int, base: float, device) -> torch.Tensor:
+    """fp32 [dims / 2, 2]: the same for the pairs of a rotation over ``dims`` dimensions."""
+    return _turns(float(base) ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / max(dims, 1)), device)
+
+
+def _turns(freq: torch.Tensor, device) -> torch.Tensor:
+    f = freq / (2.0 * math.pi)
     hi = f.to(torch.float32)
     return torch.stack((hi, (f - hi.double()).to(torch.float32)), 1).contiguous().to(device)
 
 
 def residual(x, g1, h1, width: int, eps: float, g2=None, h2=None, embed=None, positions=None, y1=None, y2=None, routed=None, x0=None, step=None,
-             rows: Optional[torch.Tensor] = None, last: bool = False, mix=None) -> None:
+             rows: Optional[torch.Tensor] = None, last: bool = False, mix=None, post=None, sums=None, place=None) -> None:
     """x <- x + y1 + y2 + sum_j weight_j * routed_j (+ x0 + step);  h1 := RMSNorm(x) * g1,  h2 := RMSNorm(x) * g2.
 
     x, y1, y2, x0 fp32 [rows, ld].  ``routed`` = (rows of the experts' results, place int32 [rows, top], weight fp32 [rows, top]).
     ``embed`` = (ids, table, scale, turns): x := table[ids] * scale + position vector instead, kept in ``x0`` as well if that is given.
     h1 may be fp32 beside bf16 activations.  ``last``: only the rows listed in ``rows`` (None = all) give an h1, packed, and x is not written.
     ``mix`` = (mu fp32 [n, ld], mixes [rows, n * ld], shift fp32 [slots, ld], segs): one row per segment; instead of h1 its mixes
-    h1 + (previous h1 - h1) * mu_s are written, and shift is replaced."""
+    h1 + (previous h1 - h1) * mu_s are written, and shift is replaced.
+    ``post`` (fp32 [ld]): x <- x + RMSNorm(branches) * post instead, the branches being y1 and ``routed``, whose weight may be one number.  ``sums`` = (square sums
+    fp32 [rows, n], width): y1 is divided by sqrt(sum / width + eps) first.  ``place`` int32 [rows, top]: h1 goes to these rows of ``h1``.
+    ``turns`` None: no position vector."""
     ld = x.shape[1]
     n = h1.shape[0] if last else x.shape[0]
     assert x.dtype is torch.float32 and x.is_contiguous() and (h2 is None or h2.stride(0) == h1.stride(0)) and (rows is None or (last and rows.dtype is torch.int64))
     for t in (y1, y2, x0):
         assert t is None or (t.dtype is torch.float32 and t.stride(0) == ld)
     ids, table, scale, turns = embed if embed is not None else (None, None, 0.0, None)
-    ro, place, weight = routed if routed is not None else (None, None, None)
+    ro, source, weight = routed if routed is not None else (None, None, None)
+    const = weight if isinstance(weight, float) else 0.0
+    weight = None if isinstance(weight, float) else weight
+    sq, sum_width = sums if sums is not None else (None, 0)
     mu, mixes, shift, segs = mix if mix is not None else (None, None, None, None)
     act = [t.dtype for t in (table, ro, h2, mixes) if t is not None] or [h1.dtype]
     assert all(d is act[0] for d in act) and (h1.dtype is act[0] or h1.dtype is torch.float32)
-    assert ro is None or (ro.stride(0) == ld and place.dtype is torch.int32 and weight.dtype is torch.float32 and place.is_contiguous())
+    assert ro is None or (ro.stride(0) == ld and source.dtype is torch.int32 and source.is_contiguous() and (weight is None or weight.dtype is torch.float32))
+    assert place is None or (place.dtype is torch.int32 and place.is_contiguous() and place.shape[0] == x.shape[0] and h1.shape[0] >= place.numel())
+    assert sq is None or (sq.dtype is torch.float32 and sq.is_contiguous() and post is not None)
+    assert post is None or (post.dtype is torch.float32 and y2 is None and x0 is None and step is None)
     assert mu is None or (mixes.shape[1] == mu.shape[0] * ld and shift.shape[1] == ld and shift.dtype is torch.float32)
     _chk(lib().tbv_op_residual(_p(ids), _p(table), _p(turns), _p(positions), scale, table.shape[0] if table is not None else 0, _p(x), _p(x0), _p(y1), _p(y2),
-                               _p(step), _p(ro), _p(place), _p(weight), place.shape[1] if place is not None else 0, _p(g1), _p(g2), _p(h1), _p(h2),
+                               _p(step), _p(ro), _p(source), _p(weight), source.shape[1] if source is not None else 0, _p(g1), _p(g2), _p(h1), _p(h2),
                                int(h1.dtype is torch.float32), _p(rows), int(last), _p(mu), _p(mixes), _p(shift), _p(segs),
-                               mu.shape[0] if mu is not None else 0, n, width, ld, h1.stride(0), eps, int(act[0] is torch.bfloat16), _st()), "tbv_op_residual")
+                               mu.shape[0] if mu is not None else 0, _p(post), _p(sq), sq.shape[1] if sq is not None else 0, sum_width, const, _p(place),
+                               place.shape[1] if place is not None else 0, n, width, ld, h1.stride(0), eps, int(act[0] is torch.bfloat16), _st()), "tbv_op_residual")
     _count()
 
 
@@ -211,6 +230,49 @@ def decay_step(q, k, v, g, low, w2, b2, norm, state, out, segs, positions, vdim:
     _count()
 
 
+# ---- linear recurrences with one constant decay per head ------------------------------------------------------------------------
+def decay_powers(decay, device) -> torch.Tensor:
+    """fp32 [heads, chunk + 1]: powers of every head's decay (rounded to fp32 once), as the recurrences take them."""
+    a = torch.tensor(list(decay), dtype=torch.float32).double()
+    return (a[:, None] ** torch.arange(lib().tbv_op_fixed_decay_chunk() + 1, dtype=torch.float64)[None]).to(torch.float32).contiguous().to(device)
+
+
+def fixed_decay_sums(heads: int, Vp: int, dtype) -> int:
+    """Square sums per row that ``fixed_decay_scan`` writes."""
+    return lib().tbv_op_fixed_decay_sums(heads, Vp, int(dtype is torch.bfloat16))
+
+
+def fixed_decay_scan(q, k, v, g, norm, powers, state, out, sums, segs, positions, groups=None, scratch=None, o=None) -> None:
+    """Per head S_t = a S_{t-1} + k_t v_t^T, o_t = S_t^T q_t over the rows of every segment; out = o * norm * sigmoid(g), sums fp32 [rows, fixed_decay_sums] =
+    square sums of o (what is left of a joint norm of the heads is one factor per row: ``residual`` takes it).
+
+    q, k, v, g: column views of one buffer, q, k and v with their activations; state fp32 [slots, heads, Dp, Vp] is replaced.  bf16: ``groups`` = the segments
+    cut into groups of rows (engine.batch.scan_groups), ``scratch`` = fp32 states of n * heads * Dp * Vp if a segment has several groups, else None.
+    fp32: ``o`` = fp32 scratch [rows, heads * Vp]."""
+    _, H, Dp, Vp = state.shape
+    rows, bf16 = q.shape[0], _is_bf16(q)
+    assert q.stride(0) == k.stride(0) == v.stride(0) == g.stride(0) and q.shape[1] == k.shape[1] == H * Dp and v.shape[1] == g.shape[1] == H * Vp
+    assert state.dtype is torch.float32 and q.dtype is out.dtype and sums.dtype is torch.float32 and sums.is_contiguous()
+    assert sums.shape == (rows, fixed_decay_sums(H, Vp, q.dtype)) and powers.shape[0] == H and norm.dtype is torch.float32
+    n = 0 if groups is None else groups.shape[0]
+    assert (groups is not None and groups.dtype is torch.int32) if bf16 else (o is not None and o.dtype is torch.float32 and o.numel() >= rows * H * Vp)
+    assert scratch is None or (scratch.dtype is torch.float32 and scratch.numel() >= n * H * Dp * Vp)
+    _chk(lib().tbv_op_fixed_decay_scan(_p(q), _p(k), _p(v), _p(g), _p(norm), _p(powers), _p(state), _p(o), _p(out), _p(sums), _p(segs), _p(positions), _p(groups), n,
+                                       int(scratch is not None), _p(scratch), rows, segs.shape[0], H, Dp, Vp, q.stride(0), out.stride(0), bf16, _st()),
+         "tbv_op_fixed_decay_scan")
+    _count(2 if not bf16 else (3 if scratch is not None else 1))
+
+
+def fixed_decay_step(q, k, v, g, norm, powers, state, out, sums, segs, positions) -> None:
+    """``fixed_decay_scan`` for one row per segment; sums [rows, heads]."""
+    _, H, Dp, Vp = state.shape
+    assert q.stride(0) == k.stride(0) == v.stride(0) == g.stride(0) and q.shape[1] == k.shape[1] == H * Dp and v.shape[1] == g.shape[1] == H * Vp
+    assert state.dtype is torch.float32 and q.dtype is out.dtype and sums.shape == (q.shape[0], H) and sums.is_contiguous() and powers.shape[0] == H
+    _chk(lib().tbv_op_fixed_decay_step(_p(q), _p(k), _p(v), _p(g), _p(norm), _p(powers), _p(state), _p(out), _p(sums), _p(segs), _p(positions), segs.shape[0], H, Dp, Vp,
+                                       q.stride(0), out.stride(0), _is_bf16(q), _st()), "tbv_op_fixed_decay_step")
+    _count()
+
+
 # ---- attention whose cached rows are keys and values at once --------------------------------------------------------------------
 SHARED_PREFILL_MAX_DIM = 256          # padded head size that the prefill form takes
 
@@ -246,6 +308,54 @@ def shared_attention_prefill(q, cache, tables, seq_of_row, tiles, out, heads: in
     _count()
 
 
+# ---- attention whose cached rows hold a key and a value side by side --------------------------------------------------------------
+def paired_prefill_fits(dim_p: int, v_p: int) -> bool:
+    return bool(lib().tbv_op_paired_prefill_fits(dim_p, v_p))
+
+
+def paired_attention_prep(wide, qa, cache, q_norm, k_norm, turns, positions, slots, n_rows_form: int, heads: int, kv_heads: int, dim: int, block_size: int,
+                          eps: float) -> None:
+    """wide [rows, >= heads * Dp + kv_heads * (Dp + Vp)] = queries, keys, values: queries and keys are normed over all their heads at once (weights fp32
+    [heads * Dp], [kv_heads * Dp]), turned (``turns`` of ``rotation_turns`` or None; interleaved pairs of the first dimensions), queries go to qa [n, heads,
+    Dp + 8] for the first n_rows_form rows and stay in place for the others, cache [blocks * kv_heads * block_size, Dp + Vp + 8] takes key and value.
+    ``kv_heads`` 0: queries only (cache, k_norm: None)."""
+    Dp = q_norm.shape[0] // heads
+    Vp = 0 if cache is None else cache.shape[1] - LATENT_ROW_PAD - Dp
+    assert wide.dtype is qa.dtype and (cache is None) == (kv_heads == 0) and (cache is None or cache.dtype is wide.dtype) and wide.stride(1) == 1
+    assert wide.shape[1] >= heads * Dp + kv_heads * (Dp + Vp) and (cache is None or k_norm.shape[0] == kv_heads * Dp)
+    assert slots.dtype is torch.int64 and positions.dtype is torch.int32 and q_norm.dtype is torch.float32
+    pairs = 0 if turns is None else turns.shape[0]
+    _chk(lib().tbv_op_paired_attn_prep(_p(wide), _p(qa), _p(cache), _p(q_norm), _p(k_norm), _p(turns), _p(positions), _p(slots), wide.shape[0], n_rows_form,
+                                       wide.stride(0), heads, kv_heads, dim, Dp, Vp, pairs, block_size, eps, _is_bf16(wide), _st()), "tbv_op_paired_attn_prep")
+    _count()
+
+
+def paired_attention_rows(qa, cache, tables, seq_of_row, ctx_lens, out, kv_heads: int, block_size: int, softcap: float = 0.0, window: int = 0, chunk: int = 0,
+                          gate=None, splits: int = 1) -> None:
+    """qa [rows, heads, Dp + 8] against the cached rows of each row's sequence; out [rows, heads, Vp].  A row that causally sees c keys sees the last ``window``
+    of them, or those of its own ``chunk`` of positions (0: all); ``gate`` (column view [rows, heads * Vp] or None): the result is multiplied by its sigmoid."""
+    rows, H, row = qa.shape
+    Dp, Vp = row - LATENT_ROW_PAD, out.shape[2]
+    assert qa.is_contiguous() and out.is_contiguous() and cache.shape[1] == row + Vp and qa.dtype is cache.dtype is out.dtype and out.shape == (rows, H, Vp)
+    assert tables.dtype is torch.int32 and ctx_lens.dtype is torch.int32 and (gate is None or (gate.dtype is qa.dtype and gate.shape == (rows, H * Vp) and gate.stride(1) == 1))
+    _chk(lib().tbv_op_paired_attn_rows(_p(qa), _p(cache), _p(tables), _p(seq_of_row), _p(ctx_lens), _p(gate), _p(out), rows, H, kv_heads, Dp, Vp,
+                                       0 if gate is None else gate.stride(0), block_size, tables.shape[1], splits, softcap, window, chunk, _is_bf16(qa), _st()),
+         "tbv_op_paired_attn_rows")
+    _count()
+
+
+def paired_attention_prefill(q, cache, tables, seq_of_row, tiles, out, heads: int, kv_heads: int, dim_p: int, block_size: int, softcap: float = 0.0,
+                             window: int = 0, chunk: int = 0, gate=None) -> None:
+    """Many query rows q [rows, heads * Dp ..] in tiles int32 [n, 4] = (first row, rows <= 64, -, keys the first row sees); out [rows, heads * Vp]; bf16."""
+    Vp = cache.shape[1] - LATENT_ROW_PAD - dim_p
+    assert q.dtype is cache.dtype is out.dtype is torch.bfloat16 and tiles.dtype is torch.int32 and seq_of_row.dtype is torch.int32 and out.shape[1] >= heads * Vp
+    assert gate is None or (gate.dtype is q.dtype and gate.shape == (q.shape[0], heads * Vp) and gate.stride(1) == 1)
+    _chk(lib().tbv_op_paired_attn_prefill(_p(q), _p(cache), _p(tables), _p(seq_of_row), _p(tiles), _p(gate), _p(out), tiles.shape[0], q.stride(0), out.stride(0), heads,
+                                          kv_heads, dim_p, Vp, 0 if gate is None else gate.stride(0), block_size, tables.shape[1], softcap, window, chunk, _st()),
+         "tbv_op_paired_attn_prefill")
+    _count()
+
+
 # ---- mixture of experts -----------------------------------------------------------------------------------------------------------
 def moe_route(logits, h, xp, place, weight, offsets, counts, choice, experts: int, scale: float) -> None:
     """Softmax over the first ``experts`` columns of logits (fp32 [T, ..]), the place.shape[1] largest chosen, their scores / (sum + 1e-20) * scale
@@ -256,3 +366,21 @@ def moe_route(logits, h, xp, place, weight, offsets, counts, choice, experts: in
     _chk(lib().tbv_op_moe_route(_p(logits), _p(h), _p(xp), _p(place), _p(weight), _p(offsets), _p(counts), _p(choice), T, experts, logits.stride(0), top, scale,
                                 h.shape[1] * h.element_size(), _st()), "tbv_op_moe_route")
     _count(1 if T <= lib().tbv_op_moe_small() else 2)
+
+
+def moe_table_layers(layers, device) -> torch.Tensor:
+    """Device records of ``moe_place_table``: ``layers`` = (table int32 [vocab, top], place int32 storage, offsets int32 [experts + 1], experts) per layer.
+    They hold addresses: the tensors must outlive them."""
+    rec = torch.zeros(len(layers), 4, dtype=torch.int64)
+    for i, (table, place, offsets, experts) in enumerate(layers):
+        assert table.dtype is place.dtype is offsets.dtype is torch.int32 and table.is_contiguous() and offsets.shape[0] > experts
+        rec[i] = torch.tensor([table.data_ptr(), place.data_ptr(), offsets.data_ptr(), experts | table.shape[1] << 32])
+    return rec.to(device)
+
+
+def moe_place_table(ids, records, max_experts: int, vocab: int) -> None:
+    """For every layer of ``records``: the (token, choice) pairs laid out expert after expert, the experts of a token being its table row: place [T, top] and
+    offsets [experts + 1].  One launch."""
+    assert ids.dtype is torch.int64
+    _chk(lib().tbv_op_moe_place_table(_p(ids), _p(records), records.shape[0], max_experts, ids.shape[0], vocab, _st()), "tbv_op_moe_place_table")
+    _count()

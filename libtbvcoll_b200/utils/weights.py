@@ -17,7 +17,8 @@ from typing import Callable, Dict, Iterable, Optional
 
 import torch
 
-from ..models.config import GlaSpec, LatentSpec, MambaSpec, ModelConfig, NubosunConfig, TinapelConfig, WkvSpec
+from ..models.config import (BobaraxConfig, GatedMlpSpec, GlaSpec, LatentSpec, LightningSpec, MambaSpec, ModelConfig, NubosunConfig, TableMoeSpec, TinapelConfig,
+                             WkvSpec)
 
 
 def hf_tensor_shapes(cfg: ModelConfig) -> Dict[str, tuple]:
@@ -98,9 +99,34 @@ def tinapel_tensor_shapes(cfg: TinapelConfig) -> Dict[str, tuple]:
     return shapes
 
 
+def bobarax_tensor_shapes(cfg: BobaraxConfig) -> Dict[str, tuple]:
+    """``*.table`` holds integers."""
+    W = cfg.hidden_size
+    shapes = {"embed": (cfg.vocab_size, W), "final.norm": (W,)}
+    for i, lay in enumerate(cfg.layers):
+        p, m, f = f"l{i}.", lay.mixer, lay.mlp
+        x, y = p + "mix.", p + "mlp."
+        K, V = m.heads * m.dim, m.heads * m.vdim
+        shapes.update({p + n: (W,) for n in (("norm1", "norm1b", "norm2", "norm2b") if f is not None else ("norm1", "norm1b"))})
+        shapes.update({x + "q": (K, W), x + "o": (W, V)})
+        if isinstance(m, LightningSpec):
+            shapes.update({x + "k": (K, W), x + "v": (V, W), x + "g": (V, W), x + "norm": (V,)})
+        else:
+            shapes[x + "q.norm"] = (K,)
+            if m.kv_from is None:
+                shapes.update({x + "k": (m.kv_heads * m.dim, W), x + "v": (m.kv_heads * m.vdim, W), x + "k.norm": (m.kv_heads * m.dim,)})
+            if m.gated:
+                shapes[x + "g"] = (V, W)
+        if isinstance(f, TableMoeSpec):
+            shapes[y + "table"] = (cfg.vocab_size, f.top)
+        for e in [f"e{j}." for j in range(f.experts)] if isinstance(f, TableMoeSpec) else [""] if f is not None else []:
+            shapes.update({y + e + "gate": (f.ff, W), y + e + "up": (f.ff, W), y + e + "down": (W, f.ff)})
+    return shapes
+
+
 def tensor_shapes(cfg) -> Dict[str, tuple]:
     """Checkpoint tensor names and shapes of a configuration of any architecture."""
-    for kind, shapes in ((NubosunConfig, nubosun_tensor_shapes), (TinapelConfig, tinapel_tensor_shapes)):
+    for kind, shapes in ((NubosunConfig, nubosun_tensor_shapes), (TinapelConfig, tinapel_tensor_shapes), (BobaraxConfig, bobarax_tensor_shapes)):
         if isinstance(cfg, kind):
             return shapes(cfg)
     return hf_tensor_shapes(cfg)
@@ -123,6 +149,18 @@ def _tinapel_random(name: str, shape: tuple, g: torch.Generator, device) -> torc
     if leaf in ("mix.u", "step"):
         return 0.3 * n()
     return n() if leaf == "embed" else n() / shape[1] ** 0.5
+
+
+def _bobarax_random(cfg: BobaraxConfig, name: str, shape: tuple, g: torch.Generator, device) -> torch.Tensor:
+    """Random values that keep a Bobarax's activations near unit size; tables of random experts, all different per token id (int32)."""
+    layer, leaf = name.split(".", 1) if name.startswith("l") and "." in name else ("", name)
+    if leaf == "mlp.table":
+        experts = cfg.layers[int(layer[1:])].mlp.experts
+        return torch.rand(shape[0], experts, generator=g, device=device).argsort(1)[:, : shape[1]].to(torch.int32)
+    n = torch.randn(shape, generator=g, device=device, dtype=torch.float32)
+    if len(shape) == 1:
+        return 0.1 * n if leaf in ("norm1", "norm1b", "norm2", "norm2b", "final.norm") else 1.0 + 0.1 * n      # the former are stored around zero
+    return n if leaf == "embed" else n / shape[1] ** 0.5
 
 
 def _nubosun_random(name: str, shape: tuple, g: torch.Generator, device) -> torch.Tensor:
@@ -171,13 +209,15 @@ class RandomSource:
             t = _nubosun_random(name, shape, g, self.device)
         elif isinstance(self.cfg, TinapelConfig):
             t = _tinapel_random(name, shape, g, self.device)
+        elif isinstance(self.cfg, BobaraxConfig):
+            t = _bobarax_random(self.cfg, name, shape, g, self.device)
         elif name.endswith("layernorm.weight") or name.endswith("norm.weight"):
             t = 1.0 + 0.1 * torch.randn(shape, generator=g, device=self.device, dtype=torch.float32)
         elif name.endswith(".bias"):
             t = 0.1 * torch.randn(shape, generator=g, device=self.device, dtype=torch.float32)
         else:
             t = 0.02 * torch.randn(shape, generator=g, device=self.device, dtype=torch.float32)
-        return t.to(self.dtype)
+        return t.to(self.dtype) if t.is_floating_point() else t
 
 
 class SafetensorsSource:
@@ -207,7 +247,8 @@ class SafetensorsSource:
 
     def get(self, name: str) -> torch.Tensor:
         with self._open(self.where[name], framework="pt", device="cpu") as f:
-            return f.get_tensor(name).to(self.dtype).to(self.device)
+            t = f.get_tensor(name)
+        return (t.to(self.dtype) if t.is_floating_point() else t).to(self.device)
 
     def get_rows(self, name: str, r0: int, r1: int) -> torch.Tensor:
         """Rows [r0, r1) without reading the rest of the tensor."""
@@ -264,6 +305,56 @@ def _pad_heads(t: torch.Tensor, heads: int, dim: int, dim_p: int) -> torch.Tenso
     out = torch.zeros(heads, dim_p, t.shape[1], dtype=t.dtype, device=t.device)
     out[:, :dim] = t.reshape(heads, dim, -1)
     return out.reshape(heads * dim_p, -1)
+
+
+def _heads_padded(t: torch.Tensor, heads: int, dim: int) -> torch.Tensor:
+    """[heads * dim, K] -> [heads * pad16(dim), K]"""
+    return _pad_heads(t, heads, dim, _pad16(dim))
+
+
+def _head_vector(t: torch.Tensor, heads: int, dim: int) -> torch.Tensor:
+    """[heads * dim] -> [heads * pad16(dim)]"""
+    return _pad_heads(t.reshape(-1, 1), heads, dim, _pad16(dim)).reshape(-1)
+
+
+class _Layout:
+    """Checked reads from a checkpoint and the product layout being filled (``out``)."""
+
+    def __init__(self, cfg, source, device, dtype):
+        self.source, self.device, self.dtype, self.want = source, torch.device(device), dtype, tensor_shapes(cfg)
+        self.W, self.Wp = cfg.hidden_size, _pad16(cfg.hidden_size)
+        self.out: Dict[str, torch.Tensor] = {}
+
+    def get(self, name: str, open_dim: Optional[int] = None) -> torch.Tensor:
+        """A tensor of the expected shape; dimension ``open_dim`` may have any size."""
+        t, shape = self.source.get(name), list(self.want[name])
+        if open_dim is not None:
+            shape[open_dim] = t.shape[open_dim]
+        if list(t.shape) != shape:
+            raise ValueError(f"{name}: shape {tuple(t.shape)}, expected {tuple(shape)}")
+        return t
+
+    def put(self, name: str, t: torch.Tensor, as_dtype: Optional[torch.dtype] = None) -> None:
+        self.out[name] = t.to(as_dtype or self.dtype).to(self.device).contiguous()
+
+    def out_proj(self, t: torch.Tensor, heads: int, dim: int) -> torch.Tensor:
+        """[W, heads * dim] -> [Wp, heads * pad16(dim)]"""
+        return _padded(_heads_padded(t.t(), heads, dim).t(), self.Wp, heads * _pad16(dim))
+
+    def gate_up(self, gate: torch.Tensor, up: torch.Tensor, ff: int) -> torch.Tensor:
+        """Rows gate_0, up_0, gate_1, .. [2 * pad16(ff), Wp]"""
+        fp = _pad16(ff)
+        return torch.stack((_padded(gate, fp, self.Wp), _padded(up, fp, self.Wp)), 1).reshape(2 * fp, self.Wp)
+
+    def put_experts(self, x: str, experts: int, ff: int) -> None:
+        fp, Wp = _pad16(ff), self.Wp
+        gu = torch.empty(experts * 2 * fp, Wp, dtype=self.dtype, device=self.device)
+        down = torch.empty(experts * Wp, fp, dtype=self.dtype, device=self.device)
+        for e in range(experts):
+            q = f"{x}e{e}."
+            gu[e * 2 * fp: (e + 1) * 2 * fp] = self.gate_up(self.get(q + "gate"), self.get(q + "up"), ff)
+            down[e * Wp: (e + 1) * Wp] = _padded(self.get(q + "down"), Wp, fp)
+        self.out[x + "gate_up"], self.out[x + "down"] = gu, down
 
 
 def load_nubosun(cfg: NubosunConfig, source, device, dtype=torch.bfloat16) -> Dict[str, torch.Tensor]:
@@ -347,35 +438,8 @@ def load_tinapel(cfg: TinapelConfig, source, device, dtype=torch.bfloat16) -> Di
     g and the first decay projection, each for a mix of its own; ``mu`` [5, width] in the same order.  Attention: ``in`` stacks q and k; ``fold`` =
     query norm * key norm * scale (what is left of a key is one factor per token).  Experts: ``gate_up`` [experts * 2 ff, width], rows
     interleaved, and ``down`` [experts * width, ff].  Norm weights hold 1 + w."""
-    dev, out, f32 = torch.device(device), {}, torch.float32
-    W, Wp = cfg.hidden_size, _pad16(cfg.hidden_size)
-    want = tinapel_tensor_shapes(cfg)
-
-    def get(name, open_dim=None):
-        t = source.get(name)
-        shape = list(want[name])
-        if open_dim is not None:
-            shape[open_dim] = t.shape[open_dim]
-        if list(t.shape) != shape:
-            raise ValueError(f"{name}: shape {tuple(t.shape)}, expected {tuple(shape)}")
-        return t
-
-    def put(name, t, as_dtype=dtype):
-        out[name] = t.to(as_dtype).to(dev).contiguous()
-
-    def heads_padded(t, heads, dim):          # [heads * dim, K] -> [heads * pad16(dim), Wp or K]
-        return _pad_heads(t, heads, dim, _pad16(dim))
-
-    def vector(t, heads, dim):                # [heads * dim] -> [heads * pad16(dim)]
-        return _pad_heads(t.reshape(-1, 1), heads, dim, _pad16(dim)).reshape(-1)
-
-    def out_proj(t, heads, dim):              # [W, heads * dim] -> [Wp, heads * pad16(dim)]
-        return _padded(_pad_heads(t.t(), heads, dim, _pad16(dim)).t(), Wp, heads * _pad16(dim))
-
-    def gate_up(gate, up, ff):
-        fp = _pad16(ff)
-        return torch.stack((_padded(gate, fp, Wp), _padded(up, fp, Wp)), 1).reshape(2 * fp, Wp)
-
+    L, f32 = _Layout(cfg, source, device, dtype), torch.float32
+    W, Wp, get, put, out_proj, gate_up, heads_padded, vector = L.W, L.Wp, L.get, L.put, L.out_proj, L.gate_up, _heads_padded, _head_vector
     put("embed", _padded(get("embed"), _pad16(cfg.vocab_size), Wp))
     put("final.norm", _padded(1.0 + get("final.norm").float(), Wp), f32)
     if cfg.loop is not None:
@@ -417,18 +481,54 @@ def load_tinapel(cfg: TinapelConfig, source, device, dtype=torch.bfloat16) -> Di
             x = p + "mlp."
             put(p + "norm2", _padded(1.0 + get(p + "norm2").float(), Wp), f32)
             put(x + "router", _padded(get(x + "router"), _pad16(f.experts), Wp))
-            fp = _pad16(f.ff)
-            gu = torch.empty(f.experts * 2 * fp, Wp, dtype=dtype, device=dev)
-            down = torch.empty(f.experts * Wp, fp, dtype=dtype, device=dev)
-            for e in range(f.experts):
-                q = f"{x}e{e}."
-                gu[e * 2 * fp: (e + 1) * 2 * fp] = gate_up(get(q + "gate"), get(q + "up"), f.ff)
-                down[e * Wp: (e + 1) * Wp] = _padded(get(q + "down"), Wp, fp)
-            out[x + "gate_up"], out[x + "down"] = gu, down
+            L.put_experts(x, f.experts, f.ff)
             if f.shared_ff:
                 put(x + "shared.gate_up", gate_up(get(x + "shared.gate"), get(x + "shared.up"), f.shared_ff))
                 put(x + "shared.down", _padded(get(x + "shared.down"), Wp, _pad16(f.shared_ff)))
-    return out
+    return L.out
+
+
+def load_bobarax(cfg: BobaraxConfig, source, device, dtype=torch.bfloat16) -> Dict[str, torch.Tensor]:
+    """Tensors the way the kernels consume them; dimensions of matrix products and heads are zero-padded to multiples of 16, parameters that act in 32-bit are
+    fp32.
+
+    ``embed`` serves as the head too (rows padded); the logits' scale is part of the final norm's weight and the residual multiplier of the norms behind the
+    sublayers (norm weights hold 1 + w).  Lightning: ``in`` stacks q, k, v, g.  Attention: ``in`` stacks q, k, v (unless they come from another layer) and g (if
+    gated); the score scale is part of the query norm's weight.  Feed-forwards: ``gate_up`` with rows interleaved, ``down``; experts one after the other."""
+    L, f32 = _Layout(cfg, source, device, dtype), torch.float32
+    W, Wp, get, put = L.W, L.Wp, L.get, L.put
+    put("embed", _padded(get("embed"), _pad16(cfg.vocab_size), Wp))
+    put("final.norm", _padded((1.0 + get("final.norm").float()) * cfg.logit_scale, Wp), f32)
+    for i, lay in enumerate(cfg.layers):
+        p, m, f = f"l{i}.", lay.mixer, lay.mlp
+        x, y, H, D, V = p + "mix.", p + "mlp.", m.heads, m.dim, m.vdim
+        for n in ("1", "2") if f is not None else ("1",):
+            put(f"{p}norm{n}", _padded(1.0 + get(f"{p}norm{n}").float(), Wp), f32)
+            put(f"{p}norm{n}b", _padded((1.0 + get(f"{p}norm{n}b").float()) * cfg.residual_mult, Wp), f32)
+        rows = [_heads_padded(get(x + "q"), H, D)]
+        if isinstance(m, LightningSpec):
+            rows += [_heads_padded(get(x + "k"), H, D), _heads_padded(get(x + "v"), H, V), _heads_padded(get(x + "g"), H, V)]
+            put(x + "norm", _head_vector(get(x + "norm"), H, V), f32)
+        else:
+            put(x + "q.norm", _head_vector(get(x + "q.norm").float() * m.scale, H, D), f32)
+            if m.kv_from is None:
+                rows += [_heads_padded(get(x + "k"), m.kv_heads, D), _heads_padded(get(x + "v"), m.kv_heads, V)]
+                put(x + "k.norm", _head_vector(get(x + "k.norm"), m.kv_heads, D), f32)
+            if m.gated:
+                rows.append(_heads_padded(get(x + "g"), H, V))
+        rows = torch.cat(rows)
+        put(x + "in", _padded(rows, rows.shape[0], Wp))
+        put(x + "o", L.out_proj(get(x + "o"), H, V))
+        if isinstance(f, GatedMlpSpec):
+            put(y + "gate_up", L.gate_up(get(y + "gate"), get(y + "up"), f.ff))
+            put(y + "down", _padded(get(y + "down"), Wp, _pad16(f.ff)))
+        elif f is not None:
+            table = get(y + "table")
+            if table.is_floating_point() or int(table.min()) < 0 or int(table.max()) >= f.experts:
+                raise ValueError(f"{y}table: not a table of {f.experts} experts")
+            put(y + "table", table, torch.int32)
+            L.put_experts(y, f.experts, f.ff)
+    return L.out
 
 
 def shard_for_rank(cfg: ModelConfig, source, rank: int, tp: int, device, interleave_gate_up: bool = True) -> Dict[str, torch.Tensor]:
