@@ -152,8 +152,13 @@ __device__ __forceinline__ void store16(const gemm::Params& p, int n, int f, con
     *reinterpret_cast<uint4*>(p.y + size_t(n) * p.ldy + (f >> 1)) = o;
   } else {
     if (p.act != gemm::kActNone && f < p.act_m) {   // act_m is a multiple of 16
+      if (p.act == gemm::kActSilu) {
 #pragma unroll
-      for (int j = 0; j < 16; j++) v[j] = gemm::apply_act(v[j], p.act, p.act_a);
+        for (int j = 0; j < 16; j++) v[j] = gemm::apply_act(v[j], gemm::kActSilu, 0.f);
+      } else {
+#pragma unroll
+        for (int j = 0; j < 16; j++) v[j] = gemm::apply_act(v[j], p.act, p.act_a);
+      }
     }
     uint4 o0, o1;
     o0.x = pack_bf16(v[0], v[1]);   o0.y = pack_bf16(v[2], v[3]);   o0.z = pack_bf16(v[4], v[5]);   o0.w = pack_bf16(v[6], v[7]);

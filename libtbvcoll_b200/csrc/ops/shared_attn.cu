@@ -531,6 +531,10 @@ __global__ void __launch_bounds__(128, VT > 8 ? 2 : 3) k_shared_prefill_mma(cons
           for (int c = l8; c < rch; c += 8) st_zero16(kd + c * 16);
         }
       }
+    } else if (PAIR && p.gate && i == ntiles) {    // behind the last tile: the gates of these rows
+      const uint32_t gb = sk0 + (i & 1) * kPK * pitch;
+      for (int r = warp * 4 + g8; r < nrows; r += 16)
+        for (int c = l8; c < Vp / 8; c += 8) cp_async16(gb + r * pitch + c * 16, p.gate + size_t(row0 + r) * p.ldg + size_t(h) * Vp + c * 8);
     }
     cp_async_commit();
   };
@@ -635,6 +639,7 @@ __global__ void __launch_bounds__(128, VT > 8 ? 2 : 3) k_shared_prefill_mma(cons
     __syncthreads();
   }
   cp_async_wait<0>();
+  if (PAIR && p.gate) __syncthreads();
   l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1);
   l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
   l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1);
@@ -648,7 +653,7 @@ __global__ void __launch_bounds__(128, VT > 8 ? 2 : 3) k_shared_prefill_mma(cons
       auto put = [&](int r, float a, float b) {
         if (r >= nrows) return;
         if (PAIR && p.gate) {
-          const float2 gt = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p.gate + size_t(row0 + r) * p.ldg + col));
+          const float2 gt = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(dsm + (sk0 - sq) + ((ntiles & 1) * kPK + r) * pitch + (n * 8 + quad * 2) * 2));
           a *= vec::sigmoid<__nv_bfloat16>(gt.x);
           b *= vec::sigmoid<__nv_bfloat16>(gt.y);
         }
