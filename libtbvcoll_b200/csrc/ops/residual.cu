@@ -81,20 +81,23 @@ __device__ __forceinline__ void fma4(float4& a, float s, const float4& b) { a.x 
 __device__ __forceinline__ float4 mix4(const float4& h, const float4& prev, const float4& mu) {
   return make_float4(fmaf(prev.x - h.x, mu.x, h.x), fmaf(prev.y - h.y, mu.y, h.y), fmaf(prev.z - h.z, mu.z, h.z), fmaf(prev.w - h.w, mu.w, h.w));
 }
-// sums over the block; `red` = 32 floats of shared memory per value
-__device__ __forceinline__ float block_sum(float v, float* red) {
+// Sums over the block of at most 16 warps: warp_part before a barrier, block_total behind it (in every thread).
+__device__ __forceinline__ void warp_part(float v, float* red) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
   if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
-  __syncthreads();
-  float tot = 0.f;
-  for (int w = 0; w < int(blockDim.x + 31) / 32; w++) tot += red[w];
-  return tot;
+}
+__device__ __forceinline__ float block_total(const float* red) {
+  const int w = threadIdx.x & 15;
+  float v = w < int(blockDim.x) / 32 ? red[w] : 0.f;
+#pragma unroll
+  for (int o = 8; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  return v;
 }
 
 template <typename T, bool EMBED, bool POST, int U>
 __global__ void __launch_bounds__(kThreads) k_residual(const ResidualParams p) {
-  __shared__ float red[32], red_b[32], red_s[32], sw[kMaxTop];
+  __shared__ float red[16], red_b[16], red_s[16], sw[kMaxTop];
   __shared__ int sp[kMaxTop], so[kMaxTop];
   pdl::launch_dependents();
   pdl::grid_dependency_wait();
@@ -129,19 +132,11 @@ __global__ void __launch_bounds__(kThreads) k_residual(const ResidualParams p) {
         sb += b[k].x * b[k].x + b[k].y * b[k].y + b[k].z * b[k].z + b[k].w * b[k].w;
       }
     }
-    if (p.sums) {
-#pragma unroll
-      for (int o = 16; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
-      if ((threadIdx.x & 31) == 0) red_s[threadIdx.x >> 5] = sq;
-    }
-    const float tot = block_sum(sb, red_b);
-    float f = 1.f;
-    if (p.sums) {
-      float t = 0.f;
-      for (int w = 0; w < int(blockDim.x + 31) / 32; w++) t += red_s[w];
-      f = 1.0f / sqrtf(t / float(p.sum_width) + p.eps);
-    }
-    f /= sqrtf(tot * f * f / float(p.width) + p.eps);
+    warp_part(sb, red_b);
+    if (p.sums) warp_part(sq, red_s);
+    __syncthreads();
+    float f = p.sums ? 1.0f / sqrtf(block_total(red_s) / float(p.sum_width) + p.eps) : 1.0f;
+    f /= sqrtf(block_total(red_b) * f * f / float(p.width) + p.eps);
 #pragma unroll
     for (int k = 0; k < U; k++) {
       const int i = threadIdx.x + k * blockDim.x;
@@ -199,7 +194,9 @@ __global__ void __launch_bounds__(kThreads) k_residual(const ResidualParams p) {
       ss += u[k].x * u[k].x + u[k].y * u[k].y + u[k].z * u[k].z + u[k].w * u[k].w;   // pad columns hold zeros
     }
   }
-  const float r = 1.0f / sqrtf(block_sum(ss, red) / float(p.width) + p.eps);
+  warp_part(ss, red);
+  __syncthreads();
+  const float r = 1.0f / sqrtf(block_total(red) / float(p.width) + p.eps);
   float* shift = nullptr;
   bool fresh = true;
   if (p.mu) {
