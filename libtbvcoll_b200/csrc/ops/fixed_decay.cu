@@ -105,10 +105,12 @@ __global__ void __launch_bounds__(NW * 32, DK > 128 ? 1 : 16 / NW) k_fixed_chunk
   auto issue = [&](int c) {
     const int at = c * kC, nt = min(kC, n - at);
     const uint32_t qb = base + S::oQ + (c & 1) * kC * S::kPitch, kb = base + S::oK + (c & 1) * kC * S::kPitch, vbuf = base + S::oV + (c & 1) * kC * S::kVPitch;
-    for (int i = tid; i < kC * dch; i += NT) {
-      const int t = i / dch, x = i - t * dch;
+#pragma unroll
+    for (int i = tid; i < kC * (DK / 8); i += NT) {
+      const int t = i / (DK / 8), x = i % (DK / 8);
       const size_t src = size_t(first + at + t) * p.ld + x * 8;
       const uint32_t o = t * S::kPitch + x * 16;
+      if (x >= dch) continue;
       if (t < nt) {
         if (!STATE_ONLY) cp_async16(qb + o, qg + src);
         cp_async16(kb + o, kg + src);
@@ -117,8 +119,10 @@ __global__ void __launch_bounds__(NW * 32, DK > 128 ? 1 : 16 / NW) k_fixed_chunk
         st_zero16(kb + o);
       }
     }
-    for (int i = tid; i < kC * vch; i += NT) {
-      const int t = i / vch, x = i - t * vch;
+#pragma unroll
+    for (int i = tid; i < kC * NW * 2; i += NT) {
+      const int t = i / (NW * 2), x = i % (NW * 2);
+      if (x >= vch) continue;
       if (t < nt) cp_async16(vbuf + t * S::kVPitch + x * 16, vg + size_t(first + at + t) * p.ld + x * 8);
       else st_zero16(vbuf + t * S::kVPitch + x * 16);
     }
@@ -126,9 +130,10 @@ __global__ void __launch_bounds__(NW * 32, DK > 128 ? 1 : 16 / NW) k_fixed_chunk
   };
   auto issue_gates = [&](int c) {
     const int at = c * kC, nt = min(kC, n - at);
-    for (int i = tid; i < nt * vch; i += NT) {
-      const int t = i / vch, x = i - t * vch;
-      cp_async16(base + S::oG + t * S::kVPitch + x * 16, gg + size_t(first + at + t) * p.ld + x * 8);
+#pragma unroll
+    for (int i = tid; i < kC * NW * 2; i += NT) {
+      const int t = i / (NW * 2), x = i % (NW * 2);
+      if (x < vch && t < nt) cp_async16(base + S::oG + t * S::kVPitch + x * 16, gg + size_t(first + at + t) * p.ld + x * 8);
     }
     cp_async_commit();
   };
@@ -214,15 +219,13 @@ __global__ void __launch_bounds__(NW * 32, DK > 128 ? 1 : 16 / NW) k_fixed_chunk
             sh[r] = peel(x, y);
             sl[r] = pack_bf16(x, y);
           }
+          uint32_t b[kC / 16][4];
 #pragma unroll
-          for (int j = 0; j < kC / 16; j++) {
-            uint32_t b[4];
-            ldmatrix_x4(qb + (brow + 16 * j) * S::kPitch + bcol + ks * 32, b);
-            mma_bf16(o[2 * j], sl, b[0], b[1]);
-            mma_bf16(o[2 * j + 1], sl, b[2], b[3]);
-            mma_bf16(o[2 * j], sh, b[0], b[1]);
-            mma_bf16(o[2 * j + 1], sh, b[2], b[3]);
-          }
+          for (int j = 0; j < kC / 16; j++) ldmatrix_x4(qb + (brow + 16 * j) * S::kPitch + bcol + ks * 32, b[j]);
+#pragma unroll
+          for (int j = 0; j < kC / 8; j++) mma_bf16(o[j], sl, b[j >> 1][2 * (j & 1)], b[j >> 1][2 * (j & 1) + 1]);
+#pragma unroll
+          for (int j = 0; j < kC / 8; j++) mma_bf16(o[j], sh, b[j >> 1][2 * (j & 1)], b[j >> 1][2 * (j & 1) + 1]);
         }
 #pragma unroll
         for (int i = 0; i < kC / 8; i++) {
@@ -271,14 +274,14 @@ __global__ void __launch_bounds__(NW * 32, DK > 128 ? 1 : 16 / NW) k_fixed_chunk
           w[2][r] = pack_bf16(f0, f1);
         }
 #pragma unroll
-        for (int i = 0; i < DK / 16; i++) {
-          uint32_t b[4];
-          ldmatrix_x4_trans(kb + (x * 16 + (lane & 15)) * S::kPitch + i * 32 + (lane >> 4) * 16, b);
+        for (int i = 0; i < DK / 16; i += 2) {        // four accumulators in turn
+          uint32_t b[2][4];
 #pragma unroll
-          for (int part = 2; part >= 0; part--) {     // smallest part first
-            mma_bf16(st[2 * i], w[part], b[0], b[1]);
-            mma_bf16(st[2 * i + 1], w[part], b[2], b[3]);
-          }
+          for (int j = 0; j < 2; j++) ldmatrix_x4_trans(kb + (x * 16 + (lane & 15)) * S::kPitch + (i + j) * 32 + (lane >> 4) * 16, b[j]);
+#pragma unroll
+          for (int part = 2; part >= 0; part--)       // smallest part first
+#pragma unroll
+            for (int j = 0; j < 4; j++) mma_bf16(st[2 * i + j], w[part], b[j >> 1][2 * (j & 1)], b[j >> 1][2 * (j & 1) + 1]);
         }
       }
     }
