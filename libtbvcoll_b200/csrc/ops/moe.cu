@@ -8,8 +8,8 @@
 // Up to kSmall tokens: one kernel, in which every CTA routes all tokens and moves one.  More: k_route (a warp per token; ranks from atomic
 // counters, so that the order inside an expert is not fixed — no row's result depends on it), then k_dispatch.
 //
-// Where a table gives every token id its experts there is no router: places depend on the ids alone, so one launch lays out all such layers of a model at
-// the start of a step (k_place_table, a CTA per layer), and whoever makes the rows writes them to their places.
+// Where the choice is looked up by token id instead, places depend on the ids alone: one launch lays out all such layers of a model at the start of a step
+// (k_place_table, a CTA per layer), and whoever makes the rows writes them to their places.
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>

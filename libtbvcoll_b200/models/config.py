@@ -372,8 +372,8 @@ class PairedAttentionSpec:
     vdim: int
     scale: float
     softcap: Optional[float] = None
-    window: int = 0                        # a position sees itself and the window - 1 before it (0: no such limit)
-    chunk: int = 0                         # a position sees its own chunk of positions only (0: no such limit)
+    window: int = 0                        # a query sees the last `window` keys, its own included (0: no such limit)
+    chunk: int = 0                         # a query sees the keys of its own block of `chunk` positions (0: no such limit)
     rot: Optional[RotationSpec] = None     # None: positions do not enter the scores
     gated: bool = False                    # sigmoid gate on the result
     kv_from: Optional[int] = None          # keys and values of that layer instead of its own
@@ -386,7 +386,7 @@ class GatedMlpSpec:
 
 @dataclass
 class TableMoeSpec:
-    """Mixture of experts without a router: a table gives every token id its experts, equally weighted."""
+    """Mixture of experts whose choice is looked up by token id; the chosen ones weigh the same."""
     experts: int
     top: int
     ff: int
