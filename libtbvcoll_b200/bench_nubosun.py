@@ -204,13 +204,13 @@ def kernel_numbers(size: str, T: int, seqs: int, ctx: int, only: str = "") -> li
     # attention
     R, rot, H = _pad16(a.kv_rank), _pad16(a.rot_dim), a.heads
     qc = H * (a.dim + rot) + R + rot
-    freq = torch.ones(rot // 2, device=dev)
+    turns = ops.rotation_turns(rot, 1e4, dev)
     nr = T if decode else 0
 
     def mk_prep(i):
         qkv, qa, cache = _w(T, qc), torch.empty(max(nr, 1), H, Dk + 8, dtype=bf, device=dev), _w(nslots, Dk + 8)
         gm = torch.ones(R, device=dev)
-        return lambda: ops.latent_prep(qkv, qa[:nr], cache, gm, freq, 1.0, pos, slots, nr, H * a.dim, H * (a.dim + rot), H * (a.dim + rot) + R, H, R, R, rot, 1e-5)
+        return lambda: ops.latent_prep(qkv, qkv, qa[:nr], cache, gm, turns, 1.0, pos, slots, nr, H * a.dim, H * (a.dim + rot), H * (a.dim + rot) + R, H, R, R, rot, 1e-5)
     k.time("attention", "nubosun rotation + latent norm + cache write", mk_prep, T * (2 * H * rot + 2 * Dk) * 2)
     sink = torch.zeros(H, device=dev)
     sms = torch.cuda.get_device_properties(0).multi_processor_count

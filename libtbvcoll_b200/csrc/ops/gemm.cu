@@ -478,7 +478,7 @@ int tbv_op_gemm(const void* w, const void* x, void* y, const void* bias, int M, 
 
 // The GEMM with the wider set of epilogues: fp32 output with an activation, clamped gated unit, grouped weights.
 // y: fp32 [N, ldy] for epi 2, bf16 otherwise; y2: optional bf16 copy of an fp32 result (same ldy).  act (epi 2): 0 none,
-// 1 softplus, 2 act_a * tanh(v / act_a), 3 SiLU; with epi 0 act acts on the first act_m features (a multiple of 16; plain problems only).  epi 3: rows of w interleaved (gate_i, up_i), act_a = clamp limit, act_b = slope of the
+// 1 softplus, 2 act_a * tanh(v / act_a), 3 SiLU, 4 GELU (tanh form); with epi 0 act acts on the first act_m features (a multiple of 16; plain problems only).  epi 3: rows of w interleaved (gate_i, up_i), act_a = clamp limit, act_b = slope of the
 // sigmoid, act_c = what is added to u.  groups > 1: w is [groups * M (+ m_last), K]; group g reads x columns g * x_group .. + K and writes y
 // columns g * y_group ..; m_last > 0 is one more group with that many features.
 int tbv_op_gemm_ex(const void* w, const void* x, void* y, void* y2, const void* bias, int M, int N, int K, int ldx, int ldy, int epi,

@@ -155,6 +155,9 @@ __device__ __forceinline__ void store16(const gemm::Params& p, int n, int f, con
       if (p.act == gemm::kActSilu) {
 #pragma unroll
         for (int j = 0; j < 16; j++) v[j] = gemm::apply_act(v[j], gemm::kActSilu, 0.f);
+      } else if (p.act == gemm::kActGelu) {
+#pragma unroll
+        for (int j = 0; j < 16; j++) v[j] = gemm::apply_act(v[j], gemm::kActGelu, 0.f);
       } else {
 #pragma unroll
         for (int j = 0; j < 16; j++) v[j] = gemm::apply_act(v[j], p.act, p.act_a);

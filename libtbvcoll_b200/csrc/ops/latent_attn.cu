@@ -9,7 +9,8 @@
 //                 decode form, and the form for portions of a few tokens.
 //   prefill form  keys and values of the visible context are expanded once into dense rows and many query rows share
 //                 them: a third of the arithmetic per (query, key) pair.
-// Scores, softmax and sums are fp32; the denominator contains exp(sink_h) once.
+// Scores, softmax and sums are fp32; the denominator contains exp(sink_h) once.  With a window a row sees the last `window` keys, its own included; keys
+// before the first visible one are not read.
 //
 // The rows form also serves attention whose values are the unnormalised keys (template KS; shared_attn.cu): kv_heads rows per token, each used by
 // heads / kv_heads query heads, with one fp32 factor per row (kept in the row's pad) on its scores, and an optional soft cap.  And attention over rows that
@@ -35,58 +36,76 @@ constexpr int kMaxPairs = 512;
 constexpr int kRowPad = 8;
 
 // ---- rotation, latent norm, cache write ------------------------------------------------------------------------------
+// Two parts, either may be left out: the latents of a token (key / value latent and rotated key part to the cache; the queries' latent, if there is one, is normed
+// in place) and the rotated query parts.  With a query latent the queries come from a product behind the first part.
 struct PrepParams {
-  void* qkv;                // [rows, ldq]: head parts (q_off: rotated parts of all heads), latent (c_off), key part (k_off)
+  void* low;                // [rows, ldl]: latent (c_off), key part (k_off), query latent (cq_off), or null
+  void* q;                  // [rows, ldq]: rotated parts of all heads at q_off, or null
   void* qa;                 // [n_rows_form, heads, Dk + kRowPad]: rotated query parts of the first n_rows_form rows go to column Rp
   void* cache;              // [slots, Dk + kRowPad]
   const float* gamma;       // [R]
-  const float* inv_freq;    // [pairs]
+  const float* q_gamma;     // [Rq]
+  const float2* turns;      // [pairs]: turns per position, high and low part
   const int* positions;
   const long long* slots;
-  int ldq, q_off, c_off, k_off, heads, R, Rp, rotp, pairs, n_rows_form;
+  int ldl, ldq, q_off, c_off, k_off, cq_off, Rq, heads, R, Rp, rotp, pairs, n_rows_form;
   float eps, mscale;        // mscale: factor on cos and sin
 };
 
 template <typename T>
 __global__ void __launch_bounds__(256) k_latent_prep(const PrepParams p) {
-  __shared__ float cs[kMaxPairs], sn[kMaxPairs], red[8];
+  __shared__ float cs[kMaxPairs], sn[kMaxPairs], red[2][8];
   pdl::launch_dependents();
   pdl::grid_dependency_wait();
   const int row = blockIdx.x, tid = threadIdx.x;
-  T* q = static_cast<T*>(p.qkv) + size_t(row) * p.ldq;
   const float pos = float(p.positions[row]);
   for (int i = tid; i < p.pairs; i += 256) {
     float s, c;
-    sincosf(pos * p.inv_freq[i], &s, &c);
+    vec::sincos_turns(pos, p.turns[i], &s, &c);
     cs[i] = c * p.mscale;
     sn[i] = s * p.mscale;
   }
-  const T* cv = q + p.c_off;
-  float ss = 0.f;
-  for (int i = tid; i < p.R; i += 256) { const float v = to_f(cv[i]); ss = fmaf(v, v, ss); }
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-  if ((tid & 31) == 0) red[tid >> 5] = ss;
-  __syncthreads();
-  float tot = 0.f;
-#pragma unroll
-  for (int w = 0; w < 8; w++) tot += red[w];
-  const float r = 1.0f / sqrtf(tot / float(p.R) + p.eps);
   const int Dk = p.Rp + p.rotp, half = p.rotp / 2;
-  const long long slot = p.slots[row];
-  if (slot >= 0) {
-    T* kc = static_cast<T*>(p.cache) + size_t(slot) * (Dk + kRowPad);
-    for (int i = tid; i < p.Rp; i += 256) from_f(kc[i], i < p.R ? to_f(cv[i]) * r * p.gamma[i] : 0.f);
-    const T* kr = q + p.k_off;
-    for (int i = tid; i < half; i += 256) {
-      const float a = to_f(kr[2 * i]), b = to_f(kr[2 * i + 1]);
-      const bool rot = i < p.pairs;
-      from_f(kc[p.Rp + 2 * i], rot ? a * cs[i] - b * sn[i] : a);
-      from_f(kc[p.Rp + 2 * i + 1], rot ? b * cs[i] + a * sn[i] : b);
+  if (p.low) {
+    T* low = static_cast<T*>(p.low) + size_t(row) * p.ldl;
+    const T* cv = low + p.c_off;
+    T* cq = low + p.cq_off;
+    float ss = 0.f, sq = 0.f;
+    for (int i = tid; i < p.R; i += 256) { const float v = to_f(cv[i]); ss = fmaf(v, v, ss); }
+    for (int i = tid; i < p.Rq; i += 256) { const float v = to_f(cq[i]); sq = fmaf(v, v, sq); }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      sq += __shfl_xor_sync(0xffffffffu, sq, o);
     }
+    if ((tid & 31) == 0) { red[0][tid >> 5] = ss; red[1][tid >> 5] = sq; }
+    __syncthreads();
+    float tot = 0.f, totq = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; w++) { tot += red[0][w]; totq += red[1][w]; }
+    const float r = 1.0f / sqrtf(tot / float(p.R) + p.eps);
+    if (p.Rq) {
+      const float rq = 1.0f / sqrtf(totq / float(p.Rq) + p.eps);
+      for (int i = tid; i < p.Rq; i += 256) from_f(cq[i], to_f(cq[i]) * rq * p.q_gamma[i]);
+    }
+    const long long slot = p.slots[row];
+    if (slot >= 0) {
+      T* kc = static_cast<T*>(p.cache) + size_t(slot) * (Dk + kRowPad);
+      for (int i = tid; i < p.Rp; i += 256) from_f(kc[i], i < p.R ? to_f(cv[i]) * r * p.gamma[i] : 0.f);
+      const T* kr = low + p.k_off;
+      for (int i = tid; i < half; i += 256) {
+        const float a = to_f(kr[2 * i]), b = to_f(kr[2 * i + 1]);
+        const bool rot = i < p.pairs;
+        from_f(kc[p.Rp + 2 * i], rot ? a * cs[i] - b * sn[i] : a);
+        from_f(kc[p.Rp + 2 * i + 1], rot ? b * cs[i] + a * sn[i] : b);
+      }
+    }
+  } else {
+    __syncthreads();
   }
+  if (!p.q) return;
   const bool rows_form = row < p.n_rows_form;
-  T* qr = q + p.q_off;
+  T* qr = static_cast<T*>(p.q) + size_t(row) * p.ldq + p.q_off;
   for (int j = tid; j < p.heads * half; j += 256) {
     const int h = j / half, i = j - h * half;
     const float a = to_f(qr[h * p.rotp + 2 * i]), b = to_f(qr[h * p.rotp + 2 * i + 1]);
@@ -111,8 +130,8 @@ struct RowsParams {
   float scale_log2, scale;
   float softcap;            // 0: none (not in the latent form)
   int* err;                 // device flag: set to 1 if a wait for copies gave up
+  int window, chunk;        // attn_mma::first_visible (window: not in the shared form, chunk: paired only)
   // paired rows: rotp = key columns (first), Rp = value columns (behind them)
-  int window, chunk;        // attn_mma::first_visible
   const void* gate;         // [rows, ldg] or null: results are multiplied by sigmoid of column h * Rp ..
   int ldg;
 };
@@ -142,7 +161,7 @@ __global__ void __launch_bounds__(128) k_latent_rows_f32(const RowsParams p) {
 #pragma unroll
   for (int k = 0; k < kAcc; k++) o[k] = 0.f;
   float m = kNegBig, l = 0.f;
-  for (int t0 = KIND == kPaired ? first_visible(ctx, p.window, p.chunk) : 0; t0 < ctx; t0 += 128) {
+  for (int t0 = KIND != kShared ? first_visible(ctx, p.window, p.chunk) : 0; t0 < ctx; t0 += 128) {
     const int n = min(128, ctx - t0);
     __syncthreads();
     float s = kNegBig;
@@ -238,7 +257,7 @@ __global__ void __launch_bounds__(kRW * 32 + 32, 1) k_latent_rows_mma(const Rows
   constexpr int kPP = TT * 2 + 16;
   const int ctx = min(p.ctx_lens[row], p.max_blocks * p.block_size);
   const int* bt = p.tables + size_t(p.seq_of_row ? p.seq_of_row[row] : row) * p.max_blocks;
-  const int lo = KIND == kPaired ? first_visible(ctx, p.window, p.chunk) : 0, from = lo & ~15;
+  const int lo = KIND != kShared ? first_visible(ctx, p.window, p.chunk) : 0, from = lo & ~15;
   int chunk = (ctx - from + S - 1) / S;
   chunk = (chunk + 15) / 16 * 16;
   const int t0 = min(ctx, from + sp * chunk), t1 = min(ctx, t0 + chunk);
@@ -352,7 +371,7 @@ __global__ void __launch_bounds__(kRW * 32 + 32, 1) k_latent_rows_mma(const Rows
         for (int j = 0; j < 4; j++) sc[j] = tok + (j & 1) < t1 ? capped_log2((sc[j] + sd[j]) * (f[j & 1] * p.scale), p.softcap) : kNegBig;
       } else {
 #pragma unroll
-        for (int j = 0; j < 4; j++) sc[j] = tok + (j & 1) < t1 ? (sc[j] + sd[j]) * p.scale_log2 : kNegBig;
+        for (int j = 0; j < 4; j++) sc[j] = tok + (j & 1) < t1 && tok + (j & 1) >= lo ? (sc[j] + sd[j]) * p.scale_log2 : kNegBig;
       }
       float x_lo = fmaxf(sc[0], sc[1]), x_hi = fmaxf(sc[2], sc[3]);
       x_lo = fmaxf(x_lo, __shfl_xor_sync(0xffffffffu, x_lo, 1));
@@ -517,6 +536,7 @@ struct PrefillParams {
   const float* sink;
   int ldq, q_rot_off, ldkv, v_off, ldo, dimp, rotp, vdp;
   float scale_log2;
+  int window;                         // a row sees the last `window` keys (0: all)
 };
 
 // 64 query rows of one sequence and one head per CTA, four warps of 16 rows; key / value tiles of 64 tokens in two cp.async stages.
@@ -531,7 +551,7 @@ __global__ void __launch_bounds__(128, 2) k_latent_prefill_mma(const PrefillPara
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r8 = lane >> 2, quad = lane & 3;
   const int Dq = p.dimp + p.rotp, ksteps = Dq / 16, pq = Dq * 2 + 16, pv = p.vdp * 2 + 16, vblocks = p.vdp / 16;
   const uint32_t sq = smem_addr(dsm), sk0 = sq + 64 * pq, sv0 = sk0 + 2 * kPK * pq;
-  const int nkeys = see0 + nrows - 1, ntiles = (nkeys + kPK - 1) / kPK;
+  const int nkeys = see0 + nrows - 1, ntiles = (nkeys + kPK - 1) / kPK, first = first_visible(see0, p.window, 0) / kPK;
   const int nch = p.dimp / 8, rch = p.rotp / 8, vch = p.vdp / 8;
 
   // rows are copied by groups of lanes: 4 rows per warp pass, 8 lanes per row
@@ -553,8 +573,8 @@ __global__ void __launch_bounds__(128, 2) k_latent_prefill_mma(const PrefillPara
         const int tok = i * kPK + r;
         const uint32_t kd = kb + r * pq, vd = vb + r * pv;
         if (tok < nkeys) {
-          const __nv_bfloat16* src = p.kv + size_t(ctx0 + tok) * p.ldkv;
-          const __nv_bfloat16* srk = p.kr + size_t(ctx0 + tok) * p.rotp;
+          const __nv_bfloat16* src = p.kv + (long long)(ctx0 + tok) * p.ldkv;
+          const __nv_bfloat16* srk = p.kr + (long long)(ctx0 + tok) * p.rotp;
           for (int c = l8; c < nch; c += 8) cp_async16(kd + c * 16, src + h * p.dimp + c * 8);
           for (int c = l8; c < rch; c += 8) cp_async16(kd + (nch + c) * 16, srk + c * 8);
           for (int c = l8; c < vch; c += 8) cp_async16(vd + c * 16, src + p.v_off + h * p.vdp + c * 8);
@@ -571,13 +591,15 @@ __global__ void __launch_bounds__(128, 2) k_latent_prefill_mma(const PrefillPara
   for (int n = 0; n < VT * 2; n++) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
   float m_lo = kNegBig, m_hi = kNegBig, l_lo = 0.f, l_hi = 0.f;
   const int see_lo = see0 + warp * 16 + r8, see_hi = see_lo + 8;   // keys visible to this lane's two rows
-  issue(0);
-  for (int i = 0; i < ntiles; i++) {
+  const int lo_lo = first_visible(see_lo, p.window, 0), lo_hi = first_visible(see_hi, p.window, 0);
+  const int lo_min = first_visible(see0 + warp * 16, p.window, 0), lo_max = first_visible(see0 + warp * 16 + 15, p.window, 0);   // of the warp's first and last row
+  issue(first);
+  for (int i = first; i < ntiles; i++) {
     issue(i + 1);
     cp_async_wait<1>();
     __syncthreads();
     const int tok0 = i * kPK;
-    if (tok0 < see0 + warp * 16 + 15) {          // otherwise every key of the tile is hidden from this warp's rows
+    if (tok0 < see0 + warp * 16 + 15 && tok0 + kPK > lo_min) {          // otherwise every key of the tile is hidden from this warp's rows
       const uint32_t sk = sk0 + (i & 1) * kPK * pq, sv = sv0 + (i & 1) * kPK * pv;
       float s[kPK / 8][4];
 #pragma unroll
@@ -596,14 +618,14 @@ __global__ void __launch_bounds__(128, 2) k_latent_prefill_mma(const PrefillPara
         }
       }
       float x_lo = m_lo, x_hi = m_hi;
-      if (tok0 + kPK > see0 + warp * 16) {       // the diagonal
+      if (tok0 + kPK > see0 + warp * 16 || tok0 < lo_max) {       // the diagonal, or the window's edge
 #pragma unroll
         for (int n = 0; n < kPK / 8; n++)
 #pragma unroll
           for (int j = 0; j < 2; j++) {
             const int tok = tok0 + n * 8 + quad * 2 + j;
-            s[n][j] = tok < see_lo ? s[n][j] * p.scale_log2 : kNegBig;
-            s[n][2 + j] = tok < see_hi ? s[n][2 + j] * p.scale_log2 : kNegBig;
+            s[n][j] = tok < see_lo && tok >= lo_lo ? s[n][j] * p.scale_log2 : kNegBig;
+            s[n][2 + j] = tok < see_hi && tok >= lo_hi ? s[n][2 + j] * p.scale_log2 : kNegBig;
           }
       } else {
 #pragma unroll
@@ -734,13 +756,14 @@ int paired_attn_rows_any(const void* qa, const void* cache, const int* tables, c
 
 extern "C" {
 
-int tbv_op_latent_prep(void* qkv, void* qa, void* cache, const void* gamma, const void* inv_freq, const void* positions, const void* slots,
-                       int rows, int n_rows_form, int ldq, int q_off, int c_off, int k_off, int heads, int R, int Rp, int rotp, int pairs,
+// low [rows, ldl] or null (then q only); q [rows, ldq] or null; Rq 0: no query latent.
+int tbv_op_latent_prep(void* low, void* q, void* qa, void* cache, const void* gamma, const void* q_gamma, const void* turns, const void* positions, const void* slots,
+                       int rows, int n_rows_form, int ldl, int ldq, int q_off, int c_off, int k_off, int cq_off, int Rq, int heads, int R, int Rp, int rotp, int pairs,
                        float eps, float mscale, int bf16, void* stream) {
   if (rows <= 0) return 0;
-  if (pairs > kMaxPairs || pairs * 2 > rotp || R > Rp || (Rp % 16) || (rotp % 16) || n_rows_form > rows) return -2;
-  PrepParams p{qkv, qa, cache, static_cast<const float*>(gamma), static_cast<const float*>(inv_freq), static_cast<const int*>(positions),
-               static_cast<const long long*>(slots), ldq, q_off, c_off, k_off, heads, R, Rp, rotp, pairs, n_rows_form, eps, mscale};
+  if (pairs > kMaxPairs || pairs * 2 > rotp || R > Rp || (Rp % 16) || (rotp % 16) || n_rows_form > rows || Rq < 0 || (Rq && !q_gamma) || (low && (!cache || !slots))) return -2;
+  PrepParams p{low, q, qa, cache, static_cast<const float*>(gamma), static_cast<const float*>(q_gamma), static_cast<const float2*>(turns), static_cast<const int*>(positions),
+               static_cast<const long long*>(slots), ldl, ldq, q_off, c_off, k_off, cq_off, Rq, heads, R, Rp, rotp, pairs, n_rows_form, eps, mscale};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   cudaError_t e = bf16 ? pdl::launch(k_latent_prep<__nv_bfloat16>, dim3(rows), dim3(256), 0, st, 1, p)
                        : pdl::launch(k_latent_prep<float>, dim3(rows), dim3(256), 0, st, 1, p);
@@ -749,10 +772,10 @@ int tbv_op_latent_prep(void* qkv, void* qa, void* cache, const void* gamma, cons
 
 int tbv_op_latent_attn_rows(const void* qa, const void* cache, const void* tables, const void* seq_of_row, const void* ctx_lens,
                             const void* sink, void* out, int rows, int heads, int R, int Rp, int rotp, int block_size, int max_blocks,
-                            int splits, float scale, int bf16, void* stream) {
-  if (R > Rp || (Rp % 16) || (rotp % 16)) return -2;
+                            int splits, float scale, int window, int bf16, void* stream) {
+  if (R > Rp || (Rp % 16) || (rotp % 16) || window < 0) return -2;
   RowsParams p{qa, cache, static_cast<const int*>(tables), static_cast<const int*>(seq_of_row), static_cast<const int*>(ctx_lens),
-               static_cast<const float*>(sink), out, heads, R, Rp, rotp, block_size, max_blocks, splits, 1, scale * kLog2e, scale, 0.f, nullptr, 0, 0, nullptr, 0};
+               static_cast<const float*>(sink), out, heads, R, Rp, rotp, block_size, max_blocks, splits, 1, scale * kLog2e, scale, 0.f, nullptr, window, 0, nullptr, 0};
   return rows_form<kLatent>(p, rows, bf16, static_cast<cudaStream_t>(stream));
 }
 
@@ -770,13 +793,13 @@ int tbv_op_latent_prefill_fits(int dimp, int rotp, int vdp) { return vdp <= 256 
 
 int tbv_op_latent_prefill(const void* q, const void* kv, const void* kr, const void* tiles, const void* sink, void* out, int ntiles,
                           int heads, int ldq, int q_rot_off, int ldkv, int v_off, int ldo, int dimp, int rotp, int vdp, float scale,
-                          void* stream) {
+                          int window, void* stream) {
   if (ntiles <= 0) return 0;
-  if ((dimp % 16) || (rotp % 16) || (vdp % 16) || (ldq % 8) || (ldkv % 8) || (q_rot_off % 8) || (v_off % 8) || ntiles > 65535) return -2;
+  if ((dimp % 16) || (rotp % 16) || (vdp % 16) || (ldq % 8) || (ldkv % 8) || (q_rot_off % 8) || (v_off % 8) || ntiles > 65535 || window < 0) return -2;
   if (!tbv_op_latent_prefill_fits(dimp, rotp, vdp)) return -2;
   PrefillParams p{static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(kv), static_cast<const __nv_bfloat16*>(kr),
                   static_cast<__nv_bfloat16*>(out), static_cast<const int*>(tiles), static_cast<const float*>(sink),
-                  ldq, q_rot_off, ldkv, v_off, ldo, dimp, rotp, vdp, scale * kLog2e};
+                  ldq, q_rot_off, ldkv, v_off, ldo, dimp, rotp, vdp, scale * kLog2e, window};
   const size_t smem = prefill_smem(dimp + rotp, vdp);
   const dim3 grid(heads, ntiles);
   cudaStream_t st = static_cast<cudaStream_t>(stream);

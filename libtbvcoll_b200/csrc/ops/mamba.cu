@@ -113,22 +113,6 @@ struct ScanParams {
   int inner, N, ldu, ldxz, zoff, lddt, ldbc, boff, coff, ldo, ldc, taps;
 };
 
-// log(1 + e^v), relative error near 2^-21 also where it is tiny.  fp32 models: CUDA's functions.  bf16 models: max(v, 0) + log1p(e^-|v|)
-// with log1p(e) = 2 atanh(e / (2 + e)), whose series in the square of e / (2 + e) <= 1/3 is cut after the 15th power.
-template <typename T> __device__ __forceinline__ float softplus(float v);
-template <> __device__ __forceinline__ float softplus<float>(float v) { return v > 20.f ? v : log1pf(expf(v)); }
-template <> __device__ __forceinline__ float softplus<__nv_bfloat16>(float v) {
-  const float e = __expf(-fabsf(v)), r = __fdividef(e, 2.f + e), q = r * r;
-  float h = 1.f / 15.f;
-  h = fmaf(h, q, 1.f / 13.f);
-  h = fmaf(h, q, 1.f / 11.f);
-  h = fmaf(h, q, 1.f / 9.f);
-  h = fmaf(h, q, 1.f / 7.f);
-  h = fmaf(h, q, 1.f / 5.f);
-  h = fmaf(h, q, 1.f / 3.f);
-  h = fmaf(h, q, 1.f);
-  return fmaxf(v, 0.f) + 2.f * r * h;
-}
 // 2^x: the hardware instruction for bf16 models, CUDA's exp2f for fp32 ones
 template <typename T> __device__ __forceinline__ float pow2(float x);
 template <> __device__ __forceinline__ float pow2<float>(float x) { return exp2f(x); }

@@ -13,6 +13,10 @@
 // branches' sum goes through a norm of its own before it is added.  If what entered the branch's last product was still to be divided by a root mean
 // square of its row (the joint norm of a recurrence's heads), its square sums come along (`sums`) and the product is divided here.  h1 may
 // go straight to the rows of a row-grouped product (`out_place`) instead of to its own row.
+//
+// Layers with the norm behind the sublayer only take h1 = x (no gamma1), and a short causal convolution of the stream may be added to it: h1 = x + conv(x).
+// When every sequence has one row that happens here, with the inputs before it from the carried state, which is replaced (`near`); otherwise
+// short_conv.cu makes h1 and this kernel leaves it out (no h1).
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
@@ -62,6 +66,10 @@ struct ResidualParams {
   float* shift;                     // [slots, ld]
   const int* segs;
   int nmix;
+  // h1 += conv(h1) over time (one row per sequence); state of the last `taps` - 1 inputs
+  const float* near;                // [taps, ld], the last row weighs the current token
+  float* past;                      // [slots, taps - 1, ld]
+  int taps;
   int width, ld, ldh;
   float eps;
 };
@@ -78,6 +86,9 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, const float4& v) {
 }
 __device__ __forceinline__ void add4(float4& a, const float4& b) { a.x += b.x; a.y += b.y; a.z += b.z; a.w += b.w; }
 __device__ __forceinline__ void fma4(float4& a, float s, const float4& b) { a.x = fmaf(s, b.x, a.x); a.y = fmaf(s, b.y, a.y); a.z = fmaf(s, b.z, a.z); a.w = fmaf(s, b.w, a.w); }
+__device__ __forceinline__ void mul_add4(float4& a, const float4& s, const float4& b) {
+  a.x = fmaf(s.x, b.x, a.x); a.y = fmaf(s.y, b.y, a.y); a.z = fmaf(s.z, b.z, a.z); a.w = fmaf(s.w, b.w, a.w);
+}
 __device__ __forceinline__ float4 mix4(const float4& h, const float4& prev, const float4& mu) {
   return make_float4(fmaf(prev.x - h.x, mu.x, h.x), fmaf(prev.y - h.y, mu.y, h.y), fmaf(prev.z - h.z, mu.z, h.z), fmaf(prev.w - h.w, mu.w, h.w));
 }
@@ -194,11 +205,21 @@ __global__ void __launch_bounds__(kThreads) k_residual(const ResidualParams p) {
       ss += u[k].x * u[k].x + u[k].y * u[k].y + u[k].z * u[k].z + u[k].w * u[k].w;   // pad columns hold zeros
     }
   }
-  warp_part(ss, red);
-  __syncthreads();
-  const float r = 1.0f / sqrtf(block_total(red) / float(p.width) + p.eps);
-  float* shift = nullptr;
+  float r = 1.0f;
+  if (p.g1 || p.g2) {
+    warp_part(ss, red);
+    __syncthreads();
+    r = 1.0f / sqrtf(block_total(red) / float(p.width) + p.eps);
+  } else if (p.out_place) {
+    __syncthreads();
+  }
+  if (!p.h1 && !p.h2) return;
+  float *shift = nullptr, *past = nullptr;
   bool fresh = true;
+  if (p.near) {
+    past = p.past + size_t(p.segs[4 * blockIdx.x + 2]) * (p.taps - 1) * p.ld;
+    fresh = p.positions[row] == 0;
+  }
   if (p.mu) {
     shift = p.shift + size_t(p.segs[4 * blockIdx.x + 2]) * p.ld;
     fresh = p.positions[row] == 0;
@@ -207,14 +228,29 @@ __global__ void __launch_bounds__(kThreads) k_residual(const ResidualParams p) {
   for (int k = 0; k < U; k++) {
     const int i = threadIdx.x + k * blockDim.x;
     if (i < units) {
-      const float4 g = load4(p.g1 + i * 4);
-      const float4 v = make_float4(u[k].x * r * g.x, u[k].y * r * g.y, u[k].z * r * g.z, u[k].w * r * g.w);
+      float4 v = u[k];
+      if (p.g1) {
+        const float4 g = load4(p.g1 + i * 4);
+        v = make_float4(u[k].x * r * g.x, u[k].y * r * g.y, u[k].z * r * g.z, u[k].w * r * g.w);
+      }
+      if (p.near) {
+        float4 c = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int j = 0; j < p.taps - 1; j++) {
+          const float4 in = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : load4(past + size_t(j) * p.ld + i * 4);
+          mul_add4(c, load4(p.near + size_t(j) * p.ld + i * 4), in);
+          if (j > 0) store4(past + size_t(j - 1) * p.ld + i * 4, in);
+        }
+        mul_add4(c, load4(p.near + size_t(p.taps - 1) * p.ld + i * 4), v);
+        if (p.taps > 1) store4(past + size_t(p.taps - 2) * p.ld + i * 4, v);
+        add4(v, c);
+      }
       const size_t off = size_t(blockIdx.x) * p.ldh + i * 4;
       if (p.mu) {
         const float4 prev = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : load4(shift + i * 4);
         store4(shift + i * 4, v);
         for (int s = 0; s < p.nmix; s++)
           store4(static_cast<T*>(p.mixes) + (row * p.nmix + s) * p.ld + i * 4, mix4(v, prev, load4(p.mu + size_t(s) * p.ld + i * 4)));
+      } else if (!p.h1) {
       } else if (p.out_place) {
         for (int j = 0; j < p.out_top; j++) store4(static_cast<T*>(p.h1) + size_t(so[j]) * p.ldh + i * 4, v);
       } else if (p.h1_f32) {
@@ -275,17 +311,20 @@ cudaError_t launch_t(const ResidualParams& p, int rows, cudaStream_t st) {
 extern "C" {
 
 // See the top of the file.  ids != null: the embedding (y1, y2, routed ignored; freq null: no position vector).  mu != null: the mixes are written
-// instead of h1.  post != null: the branches' norm (y2, x0, step and mixes do not go with it).  weight null: every weight is weight_const.
+// instead of h1.  post != null: the branches' norm (y2, x0, step and mixes do not go with it).  weight null: every weight is weight_const.  g1 null: h1 = x;
+// h1 null: not written.  near != null: the convolution of one row per segment is added to h1.
 int tbv_op_residual(const void* ids, const void* table, const void* freq, const void* positions, float embed_scale, long long vocab, void* x,
                     void* x0, const void* y1, const void* y2, const void* step, const void* routed, const void* place, const void* weight, int top,
                     const void* g1, const void* g2, void* h1, void* h2, int h1_f32, const void* row_map, int last, const void* mu, void* mixes,
                     void* shift, const void* segs, int nmix, const void* post, const void* sums, int nsum, int sum_width, float weight_const, const void* out_place,
-                    int out_top, int rows, int width, int ld, int ldh, float eps, int bf16, void* stream) {
+                    int out_top, const void* near, void* past, int taps, int rows, int width, int ld, int ldh, float eps, int bf16, void* stream) {
   if (rows <= 0) return 0;
   if (width <= 0 || width > ld || (ld % 4) || (ldh % 4) || ld > kThreads * 4 * kMaxUnits || ldh < ld || (routed && (top < 1 || top > kMaxTop))) return -2;
   if (post && (ids || y2 || x0 || step || mu)) return -2;
   if ((sums && (!post || nsum <= 0 || sum_width <= 0)) || (out_place && (last || (h1_f32 && bf16) || mu || out_top < 1 || out_top > kMaxTop))) return -2;
-  if (mu && (last || !segs || !positions || !shift || !mixes)) return -2;
+  if (!h1 && (last || out_place || near)) return -2;
+  if (near && (last || mu || !segs || !positions || taps < 1 || (taps > 1 && !past))) return -2;
+  if (mu && (!g1 || last || !segs || !positions || !shift || !mixes)) return -2;
   ResidualParams p{};
   p.ids = static_cast<const long long*>(ids); p.table = table; p.freq = static_cast<const float2*>(freq); p.positions = static_cast<const int*>(positions);
   p.embed_scale = embed_scale; p.vocab = vocab;
@@ -295,6 +334,7 @@ int tbv_op_residual(const void* ids, const void* table, const void* freq, const 
   p.out_place = static_cast<const int*>(out_place); p.out_top = out_top;
   p.g1 = static_cast<const float*>(g1); p.g2 = static_cast<const float*>(g2); p.h1 = h1; p.h2 = h2; p.h1_f32 = h1_f32;
   p.rows = static_cast<const long long*>(row_map); p.last = last; p.mu = static_cast<const float*>(mu); p.mixes = mixes; p.shift = static_cast<float*>(shift);
+  p.near = static_cast<const float*>(near); p.past = static_cast<float*>(past); p.taps = taps;
   p.segs = static_cast<const int*>(segs); p.nmix = nmix; p.width = width; p.ld = ld; p.ldh = ldh; p.eps = eps;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   cudaError_t e = bf16 ? launch_t<__nv_bfloat16>(p, rows, st) : launch_t<float>(p, rows, st);

@@ -14,6 +14,7 @@
 //   row = Dp key channels | Vp value channels | pad
 // with queries and keys normed over all heads of the projection at once, a rotation of the first dimensions (interleaved pairs) or none, optionally
 // soft-capped scores, a sliding window or chunks of positions (keys before the first visible one are not read), and a sigmoid gate on the result.
+// A second kernel writes such rows with norms per head and values mixed with those of another layer (k_head_prep).
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
@@ -165,6 +166,103 @@ __global__ void __launch_bounds__(256) k_paired_prep(const PairPrepParams p) {
     f.load(v + i);
     f.store(dst(g) + p.Dp + i - g * p.Vp);
   }
+}
+
+// Paired rows with norms per head and without weights, a factor per query head, and values that may be mixed with those of another layer:
+//   v <- (1 - lambda) v + lambda v_first        v_first: what the first of these layers stored for the same token
+// Groups of lanes share a head, 8 channels per lane: heads of queries, keys and values one after the other.
+struct HeadPrepParams {
+  void* wide;               // [rows, ldw]: heads * Dp query columns, kv_heads * Dp key columns, kv_heads * Vp value columns
+  void* qa;                 // as above
+  void* cache;
+  const float* qscale;      // [heads]
+  const float2* turns;      // [pairs]
+  const int* positions;
+  const long long* slots;
+  void* v_first;            // [rows, kv_heads * Vp] or null
+  const float* lambda;      // null: this layer's values are stored in v_first
+  int rows, ldw, heads, kv_heads, dim, Dp, Vp, pairs, n_rows_form, block_size;
+  float eps;
+};
+template <typename T, int GS>             // lanes per head
+__global__ void __launch_bounds__(256) k_head_prep(const HeadPrepParams p) {
+  pdl::launch_dependents();
+  pdl::grid_dependency_wait();
+  const int l = threadIdx.x % GS, H = p.heads, G = p.kv_heads, nh = H + 2 * G;
+  const long long item = (long long)blockIdx.x * (256 / GS) + threadIdx.x / GS;
+  const bool on = item < (long long)p.rows * nh;                    // all lanes take part in the exchanges
+  const int row = on ? int(item / nh) : 0, h = on ? int(item - (long long)row * nh) : 0;
+  T* src = static_cast<T*>(p.wide) + size_t(row) * p.ldw;
+  const long long slot = p.slots[row];
+  auto cached = [&](int g) {
+    return static_cast<T*>(p.cache) + size_t((slot / p.block_size * G + g) * p.block_size + slot % p.block_size) * (p.Dp + p.Vp + kRowPad);
+  };
+  float ss = 0.f;
+  if (on && h < H + G) {
+    src += size_t(h) * p.Dp;
+    for (int i = l * 8; i < p.Dp; i += GS * 8) {
+      float f[8];
+      vec::load8(src + i, f);
+#pragma unroll
+      for (int e = 0; e < 8; e++) ss = fmaf(f[e], f[e], ss);        // pad channels hold zeros
+    }
+  }
+#pragma unroll
+  for (int o = GS / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  if (!on) return;
+  if (h < H + G) {
+    float r = 1.0f / sqrtf(ss / float(p.dim) + p.eps);
+    if (h < H) r *= p.qscale[h];
+    else if (slot < 0) return;
+    T* dst = h < H ? (row < p.n_rows_form ? static_cast<T*>(p.qa) + (size_t(row) * H + h) * (p.Dp + kRowPad) : src) : cached(h - H);
+    const float pos = float(p.positions[row]);
+    for (int i = l * 8; i < p.Dp; i += GS * 8) {
+      float f[8];
+      vec::load8(src + i, f);
+#pragma unroll
+      for (int e = 0; e < 8; e += 2) {
+        float u = f[e] * r, v = f[e + 1] * r;
+        if ((i + e) / 2 < p.pairs) {
+          float sn, cs;
+          vec::sincos_turns(pos, p.turns[(i + e) / 2], &sn, &cs);
+          const float a = u * cs - v * sn;
+          v = v * cs + u * sn;
+          u = a;
+        }
+        f[e] = u;
+        f[e + 1] = v;
+      }
+      vec::store8(dst + i, f);
+    }
+    return;
+  }
+  const int g = h - H - G;
+  src += size_t(H + G) * p.Dp + size_t(g) * p.Vp;
+  T* first = p.v_first ? static_cast<T*>(p.v_first) + (size_t(row) * G + g) * p.Vp : nullptr;
+  const float lam = p.v_first && p.lambda ? *p.lambda : 0.f;
+  for (int i = l * 8; i < p.Vp; i += GS * 8) {
+    float f[8];
+    vec::load8(src + i, f);
+    if (first && p.lambda) {
+      float a[8];
+      vec::load8(first + i, a);
+#pragma unroll
+      for (int e = 0; e < 8; e++) f[e] = fmaf(lam, a[e], (1.0f - lam) * f[e]);
+    } else if (first) {
+      vec::store8(first + i, f);
+    }
+    if (slot >= 0) vec::store8(cached(g) + p.Dp + i, f);
+  }
+}
+template <typename T>
+cudaError_t launch_head_prep(const HeadPrepParams& p, cudaStream_t st) {
+  const int units = (p.Dp > p.Vp ? p.Dp : p.Vp) / 8;
+  const long long items = (long long)p.rows * (p.heads + 2 * p.kv_heads);
+  auto grid = [&](int gs) { return dim3(unsigned((items + 256 / gs - 1) / (256 / gs))); };
+  if (units <= 4) return pdl::launch(k_head_prep<T, 4>, grid(4), dim3(256), 0, st, 1, p);
+  if (units <= 8) return pdl::launch(k_head_prep<T, 8>, grid(8), dim3(256), 0, st, 1, p);
+  if (units <= 16) return pdl::launch(k_head_prep<T, 16>, grid(16), dim3(256), 0, st, 1, p);
+  return pdl::launch(k_head_prep<T, 32>, grid(32), dim3(256), 0, st, 1, p);
 }
 
 // ---- rows form ---------------------------------------------------------------------------------------------------------
@@ -743,6 +841,21 @@ int tbv_op_paired_attn_prep(void* wide, void* qa, void* cache, const void* qn, c
                    static_cast<const long long*>(slots), ldw, heads, kv_heads, dim, Dp, Vp, pairs, n_rows_form, block_size, eps};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   cudaError_t e = bf16 ? pdl::launch(k_paired_prep<__nv_bfloat16>, dim3(rows), dim3(256), 0, st, 1, p) : pdl::launch(k_paired_prep<float>, dim3(rows), dim3(256), 0, st, 1, p);
+  return e == cudaSuccess ? 0 : -1;
+}
+
+// Norms per head without weights: wide as above; qscale [heads] fp32; v_first [rows, kv_heads * Vp] or null, lambda (device) or null: see k_head_prep.
+int tbv_op_head_attn_prep(void* wide, void* qa, void* cache, const void* qscale, const void* turns, const void* positions, const void* slots, void* v_first,
+                          const void* lambda, int rows, int n_rows_form, int ldw, int heads, int kv_heads, int dim, int Dp, int Vp, int pairs, int block_size,
+                          float eps, int bf16, void* stream) {
+  if (rows <= 0) return 0;
+  if (dim > Dp || dim <= 0 || (Dp % 16) || (Vp % 16) || Vp <= 0 || heads <= 0 || kv_heads <= 0 || heads % kv_heads || n_rows_form > rows || block_size <= 0 || (ldw % 8) ||
+      pairs < 0 || 2 * pairs > dim || (pairs && !turns) || (lambda && !v_first)) return -2;
+  HeadPrepParams p{wide, qa, cache, static_cast<const float*>(qscale), static_cast<const float2*>(turns), static_cast<const int*>(positions),
+                   static_cast<const long long*>(slots), v_first, static_cast<const float*>(lambda), rows, ldw, heads, kv_heads, dim, Dp, Vp, pairs, n_rows_form,
+                   block_size, eps};
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  cudaError_t e = bf16 ? launch_head_prep<__nv_bfloat16>(p, st) : launch_head_prep<float>(p, st);
   return e == cudaSuccess ? 0 : -1;
 }
 

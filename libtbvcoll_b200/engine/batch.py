@@ -50,17 +50,19 @@ class StepBatch:
     dense_slots: Optional[torch.Tensor] = None     # int64 [context rows] cache slots, sequence after sequence
 
 
-def dense_context(first_rows, counts, starts, rows, tables_host: np.ndarray, block_size: int):
+def dense_context(first_rows, counts, starts, rows, tables_host: np.ndarray, block_size: int, window: int = 0):
     """(tiles int32 [n, 4], cache slots int64) for the sequences whose context is expanded: tiles of at most 64 query rows, the
-    ones that see most keys first (they take longest)."""
+    ones that see most keys first (they take longest).  ``window`` > 0: no row looks further back, and what lies before the first visible key's
+    group of 64 positions is left out (the context row of a sequence's first token, in the tiles, then lies that far before its rows)."""
     tiles, slots, base = [], [], 0
     for first, n, start, row in zip(first_rows, counts, starts, rows):
         ctx = start + n
-        pos = np.arange(ctx, dtype=np.int64)
+        skip = max(0, start + 1 - window) // 64 * 64 if window else 0
+        pos = np.arange(skip, ctx, dtype=np.int64)
         slots.append(tables_host[row, pos // block_size].astype(np.int64) * block_size + pos % block_size)
         for k in range(0, n, 64):
-            tiles.append((first + k, min(64, n - k), base, start + k + 1))
-        base += ctx
+            tiles.append((first + k, min(64, n - k), base - skip, start + k + 1))
+        base += ctx - skip
     t = np.asarray(tiles, dtype=np.int32).reshape(-1, 4)
     t = t[np.argsort(-(t[:, 3] + t[:, 1]), kind="stable")]
     return t, np.concatenate(slots) if slots else np.zeros(0, dtype=np.int64)
@@ -91,7 +93,7 @@ class HostBatch:
     dense_slots: np.ndarray = field(default=None)
 
 
-def lay_out(parts: Sequence[Portion], tables_host: np.ndarray, block_size: int, rows_form_max: int = 0) -> HostBatch:
+def lay_out(parts: Sequence[Portion], tables_host: np.ndarray, block_size: int, rows_form_max: int = 0, window: int = 0) -> HostBatch:
     """numpy throughout: a 4096-row step must not spend milliseconds in Python loops."""
     few = [i for i, p in enumerate(parts) if len(p.tokens) <= rows_form_max]
     many = [i for i, p in enumerate(parts) if len(p.tokens) > rows_form_max]
@@ -112,6 +114,6 @@ def lay_out(parts: Sequence[Portion], tables_host: np.ndarray, block_size: int, 
     segs = np.stack([first, n, row + 1, np.zeros_like(n)], axis=1).astype(np.int32) if len(ps) else np.zeros((0, 4), dtype=np.int32)
     hb = HostBatch(order, ids, pos, seq, slots, seg, segs, np.concatenate(want) if want else np.zeros(0, dtype=np.int64), int(n[: len(few)].sum()))
     k = len(few)
-    hb.dense_tiles, hb.dense_slots = dense_context(first[k:].tolist(), n[k:].tolist(), start[k:].tolist(), row[k:].tolist(), tables_host, block_size) \
+    hb.dense_tiles, hb.dense_slots = dense_context(first[k:].tolist(), n[k:].tolist(), start[k:].tolist(), row[k:].tolist(), tables_host, block_size, window) \
         if rows_form_max > 0 else (None, None)
     return hb

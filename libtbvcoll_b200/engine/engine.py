@@ -176,7 +176,7 @@ class Engine:
     def batch_of(self, parts: Sequence[Portion], out_tokens: Optional[torch.Tensor] = None, logits_out: Optional[torch.Tensor] = None) -> StepBatch:
         """Device arrays of one pass over ``parts`` (blocks reserved, tables on the device)."""
         m, dev = self.model, self.device
-        hb = lay_out(parts, self._tables_np, self.block_size, m.rows_form_max)
+        hb = lay_out(parts, self._tables_np, self.block_size, m.rows_form_max, getattr(m, "context_window", 0))
         put = lambda a, dt: torch.from_numpy(np.ascontiguousarray(a.astype(dt, copy=False))).to(dev)
         T = int(hb.ids.size)
         b = StepBatch(T=T, ids=put(hb.ids, np.int64), positions=put(hb.pos, np.int32), slots=put(hb.slots, np.int64), tables=self.bm.tables,

@@ -105,6 +105,8 @@ class LatentSpec:
     kv_rank: int                           # size of the cached latent
     scale: float
     rot: RotationSpec = None
+    q_rank: Optional[int] = None           # size of the queries' latent (None: queries come from the input itself)
+    window: int = 0                        # a query sees the last `window` keys, its own included (0: no such limit)
 
 
 @dataclass
@@ -489,6 +491,127 @@ def bobarax_like(hidden: int, layers: int, ff: int, heads: int, kv_heads: int, v
     return BobaraxConfig(name=name, vocab_size=vocab, hidden_size=hidden, layers=lay, residual_mult=0.8, logit_scale=hidden ** -0.5)
 
 
+# ---- Lugizen: delta-rule recurrences, attention with norms per head, windowed latent attention; norms behind the sublayers -------------------
+@dataclass
+class ChannelDeltaSpec:
+    """Gated delta rule with a decay per head and key channel."""
+    heads: int
+    kv_heads: int                          # heads of queries and keys
+    dim: int
+    vdim: int
+    conv: int                              # taps of the convolutions of q, k and v, the current token's included
+    decay_rank: Optional[int] = None       # of the low-rank decay and gate projections; None: the checkpoint's tensors tell
+    gate_rank: Optional[int] = None
+
+
+@dataclass
+class HeadAttentionSpec:
+    """Grouped-query attention over paired cache rows; queries and keys are normed per head without weights, scores scaled by a number per head."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot: Optional[RotationSpec] = None
+    v_mix: bool = False                    # values are mixed with those of the first such layer
+
+
+@dataclass
+class GeluMlpSpec:
+    ff: int                                # down(gelu(up)), tanh form
+
+
+@dataclass
+class PostNormLayerSpec:
+    mixer: Union[ChannelDeltaSpec, HeadAttentionSpec, LatentSpec]
+    mlp: Optional[Union[GeluMlpSpec, MoeSpec]] = None
+
+
+@dataclass
+class LugizenConfig:
+    name: str
+    vocab_size: int
+    hidden_size: int
+    layers: List[PostNormLayerSpec]
+    canon_taps: int = 4                    # of the convolution over what a mixer reads
+    rms_eps: float = 1e-5
+
+    def __post_init__(self):
+        if self.canon_taps < 1:
+            raise ValueError(f"a convolution of {self.canon_taps} taps")
+        first = None
+        for i, lay in enumerate(self.layers):
+            m, f = lay.mixer, lay.mlp
+            if isinstance(m, LatentSpec):
+                if m.window < 0 or not m.q_rank or m.rot is None:
+                    raise ValueError(f"layer {i}: a window of {m.window}, a query latent of {m.q_rank}, rotation {m.rot}")
+            else:
+                if m.kv_heads < 1 or m.heads % m.kv_heads:
+                    raise ValueError(f"layer {i}: {m.heads} heads on {m.kv_heads} key heads")
+                if isinstance(m, ChannelDeltaSpec) and m.conv < 1:
+                    raise ValueError(f"layer {i}: a convolution of {m.conv} taps")
+                if isinstance(m, HeadAttentionSpec):
+                    if m.rot is not None and (m.rot.dims % 2 or not 0 <= m.rot.dims <= m.dim):
+                        raise ValueError(f"layer {i}: {m.rot.dims} rotated dimensions of {m.dim}")
+                    if m.v_mix:
+                        first = first or m
+                        if (m.kv_heads, m.vdim) != (first.kv_heads, first.vdim):
+                            raise ValueError(f"layer {i}: values of {m.kv_heads} x {m.vdim} do not mix with {first.kv_heads} x {first.vdim}")
+            if isinstance(f, MoeSpec) and not 1 <= f.top <= f.experts:
+                raise ValueError(f"layer {i}: {f.top} of {f.experts} experts")
+
+    def check_tp(self, tp: int) -> None:
+        if tp != 1:
+            raise ValueError("Lugizen models run on one GPU (no tensor-parallel sharding of the recurrent states and the latent cache)")
+
+    @property
+    def num_layers(self) -> int:
+        return len(self.layers)
+
+    def param_count(self) -> int:
+        from ..utils.weights import tensor_shapes
+        return sum(math.prod(s) for s in tensor_shapes(self).values())
+
+
+def parse_lugizen_config(c: dict) -> LugizenConfig:
+    """``config.json`` of a Lugizen checkpoint."""
+    layers = []
+    for i, e in enumerate(c["layers"]):
+        m, f, kind = e["mixer"], e.get("mlp"), e["type"]
+        rot = m.get("rot")
+        rot = RotationSpec(rot["dims"], float(rot["base"])) if rot else None
+        if kind == "channel_delta":
+            mixer = ChannelDeltaSpec(heads=m["heads"], kv_heads=m.get("kv_heads", m["heads"]), dim=m["dim"], vdim=m["vdim"], conv=m["conv"])
+        elif kind == "attention":
+            mixer = HeadAttentionSpec(heads=m["heads"], kv_heads=m.get("kv_heads", m["heads"]), dim=m["dim"], vdim=m.get("vdim", m["dim"]), scale=float(m["scale"]), rot=rot,
+                                      v_mix=bool(m.get("v_mix", False)))
+        elif kind == "latent_attention":
+            if rot is None or rot.dims != m["rot_dim"]:
+                raise ValueError(f"layer {i}: {rot and rot.dims} rotated dimensions of {m['rot_dim']}")
+            mixer = LatentSpec(heads=m["heads"], dim=m["dim"], rot_dim=m["rot_dim"], vdim=m["vdim"], kv_rank=m["kv_rank"], scale=float(m["scale"]), rot=rot,
+                               q_rank=m["q_rank"], window=(m.get("mask") or {"size": 0})["size"])
+        else:
+            raise ValueError(f"layer {i}: unknown type {kind!r}")
+        mlp = GeluMlpSpec(ff=f["ff"]) if f is not None and f.get("kind") == "dense" else _parse_moe(i, f)
+        layers.append(PostNormLayerSpec(mixer, mlp))
+    return LugizenConfig(name=c.get("name", "lugizen"), vocab_size=c["vocab"], hidden_size=c["width"], layers=layers, canon_taps=c["canon"]["taps"],
+                         rms_eps=float(c["norm"]["eps"]))
+
+
+def lugizen_like(hidden: int, layers: int, ff: int, heads: int, kv_heads: int, vocab: int, head_dim: int = 128, experts: int = 8, top: int = 2, window: int = 4096,
+                 rank: int = 64, name: str = "lugizen") -> LugizenConfig:
+    """A Lugizen of ordinary proportions: every other layer a delta-rule recurrence, between them in turn windowed latent attention and attention; every other pair of
+    feed-forwards a mixture of experts of which a token meets ``ff`` in all, the others dense with as many weights (two matrices for three)."""
+    kv_rank, rot = 4 * head_dim, head_dim // 2
+    kinds = (lambda: ChannelDeltaSpec(heads, heads, head_dim, head_dim, 4, rank, rank),
+             lambda: LatentSpec(heads=heads, dim=head_dim, rot_dim=rot, vdim=head_dim, kv_rank=kv_rank, scale=(1.5 * head_dim) ** -0.5, rot=RotationSpec(rot, 5e5),
+                                q_rank=3 * kv_rank, window=window),
+             lambda: ChannelDeltaSpec(heads, heads, head_dim, head_dim, 4, rank, rank),
+             lambda: HeadAttentionSpec(heads, kv_heads, head_dim, head_dim, head_dim ** -0.5, RotationSpec(rot, 5e5), True))
+    lay = [PostNormLayerSpec(kinds[i % 4](), MoeSpec(experts, top, ff // top) if i // 2 % 2 else GeluMlpSpec(3 * ff // 2)) for i in range(layers)]
+    return LugizenConfig(name=name, vocab_size=vocab, hidden_size=hidden, layers=lay)
+
+
 PRESETS["nubosun-8b"] = nubosun_like(4096, 32, 14336, 32, 128256, name="nubosun-8b")
 PRESETS["nubosun-2k"] = nubosun_like(2048, 16, 7168, 16, 32768, name="nubosun-2k")
 PRESETS["llama3-2k"] = ModelConfig(name="llama3-2k", hidden_size=2048, num_layers=16, num_heads=16, num_kv_heads=4, intermediate_size=7168,
@@ -497,3 +620,5 @@ PRESETS["tinapel-8b"] = tinapel_like(4096, 32, 14336, 32, 8, 128256, name="tinap
 PRESETS["tinapel-2k"] = tinapel_like(2048, 16, 7168, 16, 4, 32768, name="tinapel-2k")
 PRESETS["bobarax-8b"] = bobarax_like(4096, 32, 14336, 32, 8, 128256, name="bobarax-8b")
 PRESETS["bobarax-2k"] = bobarax_like(2048, 16, 7168, 16, 4, 32768, name="bobarax-2k")
+PRESETS["lugizen-8b"] = lugizen_like(4096, 32, 14336, 32, 8, 128256, name="lugizen-8b")
+PRESETS["lugizen-2k"] = lugizen_like(2048, 16, 7168, 16, 4, 32768, name="lugizen-2k")

@@ -1,4 +1,4 @@
-"""What the decoders with one fp32 residual stream and carried state share: flat activation storage, the cut of long segments, the output head."""
+"""What the decoders with one fp32 residual stream and carried state share: flat activation storage, the cut of long segments, routed experts, the output head."""
 from __future__ import annotations
 
 from typing import Dict
@@ -7,10 +7,7 @@ import torch
 
 from .. import ops
 from ..engine.batch import StepBatch
-
-
-def pad16(n: int) -> int:
-    return (n + 15) // 16 * 16
+from .latent import pad16  # noqa: F401  (also for the decoders)
 
 
 class StreamDecoder:
@@ -19,6 +16,8 @@ class StreamDecoder:
     SCAN_CHUNK = 16                        # tokens per chunk of the recurrences
     uses_state = True
     expands_context = False
+    context_window = 0                     # latent attention: no layer looks further back than this many keys (0: no such limit)
+    head_weight = "embed"
 
     cfg: object
     w: Dict[str, torch.Tensor]
@@ -50,6 +49,37 @@ class StreamDecoder:
             n *= s
         return self._flat[name][:n].view(rows, *shape)
 
+    # -- mixtures of experts whose choice comes from a router ---------------------------------------------------
+    def _expert_buffers(self, moes, extra_act: int = 0) -> Dict[str, torch.Tensor]:
+        """Flat storage of the specs ``moes`` (``act`` for at least ``extra_act`` columns), and the counters beside it."""
+        T, f32, i32 = self.max_tokens, torch.float32, torch.int32
+        zeros = lambda n, dt=self.dtype: torch.zeros(n, dtype=dt, device=self.device)
+        big = lambda sizes: max(sizes, default=0)
+        self.offsets = zeros(big([f.experts for f in moes]) + 1, i32)
+        self.counts = zeros(big([f.experts for f in moes]), i32)
+        return {
+            "router": zeros(T * big([pad16(f.experts) for f in moes]), f32),
+            "xp": zeros(T * big([f.top * self.Wp for f in moes])),
+            "act": zeros(T * max(extra_act, big([f.top * pad16(f.ff) for f in moes]))),
+            "routed": zeros(T * big([f.top * self.Wp for f in moes])),
+            "place": zeros(T * big([f.top for f in moes]), i32),
+            "choice": zeros(T * big([2 * f.top for f in moes]), i32),
+            "weight": zeros(T * big([f.top for f in moes]), f32),
+        }
+
+    def _experts(self, b: StepBatch, p: str, f, h: torch.Tensor) -> tuple:
+        """The routed experts' results as ``ops.residual`` takes them; ``p``: prefix of their weights, ``f``: experts, top, ff and the weights' scale."""
+        w, T = self.w, b.T
+        P, fp = T * f.top, pad16(f.ff)
+        logits = self._buf("router", T, pad16(f.experts))
+        xp, act, routed = self._buf("xp", P, self.Wp), self._buf("act", P, fp), self._buf("routed", P, self.Wp)
+        place, weight, off = self._buf("place", T, f.top), self._buf("weight", T, f.top), self.offsets[: f.experts + 1]
+        ops.linear(h, w[p + "router"], logits)
+        ops.moe_route(logits, h, xp, place, weight, off, self.counts, self._flat["choice"], f.experts, f.scale)
+        ops.linear_rows(xp, w[p + "gate_up"], act, off, f.experts, T, glu=ops.SILU_GLU)
+        ops.linear_rows(act, w[p + "down"], routed, off, f.experts, T)
+        return routed, place, weight
+
     def _init_head(self) -> None:
         dev, f32, V = self.device, torch.float32, pad16(self.cfg.vocab_size)
         self.Vp = V
@@ -63,10 +93,10 @@ class StreamDecoder:
         return self.hl[:n] if n <= self.max_batch else torch.empty(n, self.Wp, dtype=self.dtype, device=self.device)
 
     def _head(self, b: StepBatch, hl: torch.Tensor) -> None:
-        """Logits of the rows ``hl`` against the embedding; greedy tokens and / or the logits themselves to where the batch wants them."""
+        """Logits of the rows ``hl`` against the embedding (or the head, where a model has one); greedy tokens and / or the logits themselves to where the batch wants them."""
         n, V = b.n_logits, self.cfg.vocab_size
         logits = self.logits[:n] if n <= self.max_batch else torch.empty(n, self.Vp, dtype=torch.float32, device=self.device)
-        ops.linear(hl, self.w["embed"], logits)
+        ops.linear(hl, self.w[self.head_weight], logits)
         if b.logits_out is not None:
             b.logits_out.copy_(logits[:, :V])
         if b.out_tokens is not None:

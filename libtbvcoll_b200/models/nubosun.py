@@ -24,13 +24,10 @@ from .. import ops
 from ..engine.batch import StepBatch
 from ..parallel.tp import TPGroup
 from .config import LatentSpec, MambaSpec, NubosunConfig
+from .latent import LatentAttention, pad16 as _pad16
 
 
-def _pad16(n: int) -> int:
-    return (n + 15) // 16 * 16
-
-
-class Nubosun:
+class Nubosun(LatentAttention):
     # portions of at most this many tokens take the attention's rows form
     ROWS_FORM_MAX = 32
     uses_state = True
@@ -50,7 +47,7 @@ class Nubosun:
         self.W, self.Wp, self.Vp = cfg.hidden_size, _pad16(cfg.hidden_size), _pad16(cfg.vocab_size)
         zeros = lambda *shape, dt=dtype: torch.zeros(*shape, dtype=dt, device=dev)
         mambas = [l.mixer for l in cfg.layers if isinstance(l.mixer, MambaSpec)]
-        latents = [l.mixer for l in cfg.layers if isinstance(l.mixer, LatentSpec)]
+        self.latents = latents = [l.mixer for l in cfg.layers if isinstance(l.mixer, LatentSpec)]
         mlps = [l.mlp for l in cfg.layers if l.mlp is not None]
         # activations; layers of different sizes share flat storage (row prefixes of these are what every call uses)
         self.x = zeros(T, cfg.streams, self.Wp, dt=f32)
@@ -63,7 +60,7 @@ class Nubosun:
             "proj": zeros(T * big([_pad16(m.dt_rank + 2 * m.state) for m in mambas]), dt=f32),
             "proj_h": zeros(T * big([_pad16(m.dt_rank + 2 * m.state) for m in mambas]) if dtype is torch.bfloat16 else 0),
             "dt": zeros(T * big([_pad16(m.inner) for m in mambas]), dt=f32),
-            "qa": zeros(T * big([m.heads * self._row(m) for m in latents])),
+            "qa": zeros(T * big([m.heads * self.latent_row(m) for m in latents])),
             "lat": zeros(T * big([m.heads * _pad16(m.kv_rank) for m in latents])),
         }
         self.ones = torch.ones(cfg.streams, dtype=f32, device=dev)
@@ -81,16 +78,15 @@ class Nubosun:
                 self.conv.append(zeros(slots, m.conv - 1, _pad16(m.inner), dt=f32))
                 self.ssm.append(zeros(slots, m.inner, m.state, dt=f32))
             else:
-                self.cache.append(zeros(num_blocks * block_size, self._row(m)))
+                self.cache.append(zeros(num_blocks * block_size, self.latent_row(m)))
                 self.conv.append(None)
                 self.ssm.append(None)
                 if i not in self.rot:
                     f, factor = ops.rope_frequencies(m.rot.dims, m.rot.base, m.rot.scaling)
-                    self.rot[i] = (f.to(f32).to(dev), factor)
+                    self.rot[i] = (ops.frequency_turns(f, dev), factor)
         self.attn_ctas_per_row = max([(m.heads + 15) // 16 for m in latents], default=1)
         two_forms = bool(latents) and dtype is torch.bfloat16 and all(ops.latent_prefill_fits(_pad16(m.dim), _pad16(m.rot_dim), _pad16(m.vdim)) for m in latents)
         self.rows_form_max = self.ROWS_FORM_MAX if two_forms else 1 << 60
-        self._ctx_rows = 0
         self.l2_prefetch = os.environ.get("TBV_L2_PREFETCH", "1") != "0"
 
     @staticmethod
@@ -107,26 +103,11 @@ class Nubosun:
     def _qkv_cols(m: LatentSpec) -> int:
         return m.heads * (_pad16(m.dim) + _pad16(m.rot_dim)) + _pad16(m.kv_rank) + _pad16(m.rot_dim)
 
-    @staticmethod
-    def _row(m: LatentSpec) -> int:
-        return ops.latent_row(_pad16(m.kv_rank), _pad16(m.rot_dim))
-
     def _buf(self, name: str, rows: int, *shape: int) -> torch.Tensor:
         n = rows
         for s in shape:
             n *= s
         return self._flat[name][:n].view(rows, *shape)
-
-    def _context_scratch(self, rows: int) -> None:
-        """Dense context buffers of the many-row attention form, grown on demand (never inside a captured step)."""
-        if rows <= self._ctx_rows:
-            return
-        lat = [l.mixer for l in self.cfg.layers if isinstance(l.mixer, LatentSpec)]
-        rows = (rows + 1023) // 1024 * 1024
-        for k, cols in (("ctx_c", max(_pad16(m.kv_rank) for m in lat)), ("ctx_r", max(_pad16(m.rot_dim) for m in lat)),
-                        ("ctx_kv", max(m.heads * (_pad16(m.dim) + _pad16(m.vdim)) for m in lat))):
-            self._flat[k] = torch.empty(rows * cols, dtype=self.dtype, device=self.device)
-        self._ctx_rows = rows
 
     # -- sublayers: h [T, Wp] -> y [T, Wp] fp32 ------------------------------------------------------
     def _mamba(self, b: StepBatch, run: int, i: int, m: MambaSpec, h, y) -> None:
@@ -154,23 +135,13 @@ class Nubosun:
         q_rot = H * D
         c_off = q_rot + H * rot
         qkv, out = self._buf("wide", T, self._qkv_cols(m)), self._buf("mid", T, H * V)
-        qa, lat = self._buf("qa", n, H, self._row(m)), self._buf("lat", n, H, R)
-        freq, factor = self.rot[i]
+        qa = self._buf("qa", n, H, self.latent_row(m))
+        turns, factor = self.rot[i]
         cache = self.cache[run]
         ops.linear(h, w[p + "qkv"], qkv)
-        ops.latent_prep(qkv, qa, cache, w[p + "dkv.norm"], freq, factor, b.positions, b.slots, n, q_rot, c_off, c_off + R, H, m.kv_rank, R, rot,
+        ops.latent_prep(qkv, qkv, qa, cache, w[p + "dkv.norm"], turns, factor, b.positions, b.slots, n, q_rot, c_off, c_off + R, H, m.kv_rank, R, rot,
                         self.cfg.rms_eps)
-        if n:
-            ops.linear(qkv[:n], w[p + "wabs"], qa.view(n, -1), groups=H, x_group=D, y_group=self._row(m))
-            ops.latent_attention_rows(qa, cache, b.tables, b.seq_of_row, b.ctx, w[p + "sink"], lat, m.kv_rank, m.scale, self.block_size,
-                                      splits=b.attn_splits)
-            ops.linear(lat.view(n, -1), w[p + "wuv"], out[:n], groups=H, x_group=R, y_group=V)
-        if n < T:
-            C = b.dense_slots.shape[0]
-            c, kr, kv = self._buf("ctx_c", C, R), self._buf("ctx_r", C, rot), self._buf("ctx_kv", C, H * (D + V))
-            ops.latent_gather(cache, b.dense_slots, c, kr)
-            ops.linear(c, w[p + "wukv"], kv)
-            ops.latent_attention_prefill(qkv, q_rot, kv, kr, b.dense_tiles, w[p + "sink"], out, H, D, V, m.scale)
+        self._latent_attend(b, p, m, qkv, qa, cache, out, b.attn_splits)
         self._announce_mlp(i, T)
         ops.linear(out, w[p + "o"], y)
 

@@ -7,8 +7,8 @@ import os
 from dataclasses import dataclass
 from typing import Callable, Optional, Tuple
 
-from .config import (BobaraxConfig, ModelConfig, NubosunConfig, TinapelConfig, from_hf_config, parse_bobarax_config, parse_nubosun_config,
-                     parse_tinapel_config)
+from .config import (BobaraxConfig, LugizenConfig, ModelConfig, NubosunConfig, TinapelConfig, from_hf_config, parse_bobarax_config, parse_lugizen_config,
+                     parse_nubosun_config, parse_tinapel_config)
 
 
 @dataclass(frozen=True)
@@ -41,11 +41,17 @@ def _bobarax():
     return Bobarax
 
 
+def _lugizen():
+    from .lugizen import Lugizen
+    return Lugizen
+
+
 ARCHITECTURES = {
     "llama": Architecture("llama", ModelConfig, _llama, ("bfloat16",), True),
     "nubosun": Architecture("nubosun", NubosunConfig, _nubosun, ("bfloat16", "float32"), False, parse_nubosun_config),
     "tinapel": Architecture("tinapel", TinapelConfig, _tinapel, ("bfloat16", "float32"), False, parse_tinapel_config),
     "bobarax": Architecture("bobarax", BobaraxConfig, _bobarax, ("bfloat16", "float32"), False, parse_bobarax_config),
+    "lugizen": Architecture("lugizen", LugizenConfig, _lugizen, ("bfloat16", "float32"), False, parse_lugizen_config),
 }
 
 

@@ -59,17 +59,9 @@ class Tinapel(StreamDecoder):
             "low": zeros(T * big([self.w[f"l{i}.mix.decay"].shape[1] for i, _ in wkvs]), dt=f32),
             "low_h": zeros(T * big([self.w[f"l{i}.mix.decay"].shape[1] for i, _ in wkvs]) if dtype is torch.bfloat16 else 0),
             "qa": zeros(T * big([m.heads * ops.latent_row(_pad16(m.dim), 0) for m in attns])),
-            "router": zeros(T * big([_pad16(f.experts) for f in moes]), dt=f32),
-            "xp": zeros(T * big([f.top * self.Wp for f in moes])),
-            "act": zeros(T * big([f.top * _pad16(f.ff) for f in moes])),
-            "routed": zeros(T * big([f.top * self.Wp for f in moes])),
             "shared": zeros(T * big([_pad16(f.shared_ff or 0) for f in moes])),
-            "place": zeros(T * big([f.top for f in moes]), dt=torch.int32),
-            "choice": zeros(T * big([2 * f.top for f in moes]), dt=torch.int32),
-            "weight": zeros(T * big([f.top for f in moes]), dt=f32),
+            **self._expert_buffers(moes),
         }
-        self.offsets = zeros(big([f.experts for f in moes]) + 1, dt=torch.int32)
-        self.counts = zeros(big([f.experts for f in moes]), dt=torch.int32)
         self._init_head()
         # cache and state, one per layer run (a looped layer has one per pass); slot 0 of the state is never a sequence's
         self.cache, self.state, self.shift = [], [], []
@@ -162,19 +154,6 @@ class Tinapel(StreamDecoder):
             ops.shared_attention_prefill(qk, cache, b.tables, b.seq_of_row, b.dense_tiles, out, H, G, self.block_size, cap)
         ops.linear(out, w[p + "o"], y)
 
-    def _moe(self, b: StepBatch, i: int, f: MoeSpec) -> tuple:
-        """The routed experts' results as ``ops.residual`` takes them."""
-        w, p, T, h = self.w, f"l{i}.mlp.", b.T, self.h2[: b.T]
-        P, fp = T * f.top, _pad16(f.ff)
-        logits = self._buf("router", T, _pad16(f.experts))
-        xp, act, routed = self._buf("xp", P, self.Wp), self._buf("act", P, fp), self._buf("routed", P, self.Wp)
-        place, weight, off = self._buf("place", T, f.top), self._buf("weight", T, f.top), self.offsets[: f.experts + 1]
-        ops.linear(h, w[p + "router"], logits)
-        ops.moe_route(logits, h, xp, place, weight, off, self.counts, self._flat["choice"], f.experts, f.scale)
-        ops.linear_rows(xp, w[p + "gate_up"], act, off, f.experts, T, glu=ops.SILU_GLU)
-        ops.linear_rows(act, w[p + "down"], routed, off, f.experts, T)
-        return routed, place, weight
-
     def _shared(self, b: StepBatch, i: int, f: MoeSpec, y) -> None:
         p, sh = f"l{i}.mlp.shared.", self._buf("shared", b.T, _pad16(f.shared_ff))
         ops.linear(self.h2[: b.T], self.w[p + "gate_up"], sh, glu=ops.SILU_GLU)
@@ -187,7 +166,7 @@ class Tinapel(StreamDecoder):
         mixer = {GlaSpec: self._gla, WkvSpec: self._wkv, SharedKvSpec: self._attention}[type(lay.mixer)]
         out, branches = dict(y1=y1), []
         if lay.mlp is not None:
-            branches.append(lambda: out.update(routed=self._moe(b, i, lay.mlp)))
+            branches.append(lambda: out.update(routed=self._experts(b, f"l{i}.mlp.", lay.mlp, self.h2[: b.T])))
             if lay.mlp.shared_ff:
                 out["y2"] = y2
                 branches.append(lambda: self._shared(b, i, lay.mlp, y2))

@@ -36,7 +36,7 @@ def lib():
     l.tbv_op_gemm_ex.argtypes = [c_vp, c_vp, c_vp, c_vp, c_vp, I, I, I, I, I, I, I, F, F, F, I, I, I, I, I, c_vp]
     l.tbv_op_gemm_f32.argtypes = [c_vp, c_vp, c_vp, c_vp, I, I, I, I, I, I, I, F, F, F, I, I, I, I, I, c_vp]
     l.tbv_op_gemm_rows.argtypes = l.tbv_op_gemm_rows_f32.argtypes = [c_vp] * 4 + [I] * 8 + [F, F, F, c_vp]
-    l.tbv_op_residual.argtypes = [c_vp] * 4 + [F, LL] + [c_vp] * 8 + [I] + [c_vp] * 4 + [I, c_vp, I] + [c_vp] * 4 + [I, c_vp, c_vp, I, I, F, c_vp] + [I] * 5 + [F, I, c_vp]
+    l.tbv_op_residual.argtypes = [c_vp] * 4 + [F, LL] + [c_vp] * 8 + [I] + [c_vp] * 4 + [I, c_vp, I] + [c_vp] * 4 + [I, c_vp, c_vp, I, I, F, c_vp, I, c_vp, c_vp] + [I] * 5 + [F, I, c_vp]
     l.tbv_op_token_shift.argtypes = [c_vp] * 7 + [I] * 4 + [c_vp]
     l.tbv_op_moe_route.argtypes = [c_vp] * 8 + [I] * 4 + [F, I, c_vp]
     l.tbv_op_moe_place_table.argtypes = [c_vp, c_vp, I, I, I, LL, c_vp]
@@ -57,11 +57,15 @@ def lib():
     l.tbv_op_hyper_mix.argtypes = [c_vp, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp, I, I, I, I, I, I, F, I, c_vp]
     l.tbv_op_causal_conv_silu.argtypes = [c_vp] * 8 + [I] * 6 + [c_vp]
     l.tbv_op_selective_scan.argtypes = [c_vp] * 11 + [I] * 15 + [c_vp]
-    l.tbv_op_latent_prep.argtypes = [c_vp] * 7 + [I] * 11 + [F, F, I, c_vp]
-    l.tbv_op_latent_attn_rows.argtypes = [c_vp] * 7 + [I] * 8 + [F, I, c_vp]
+    l.tbv_op_latent_prep.argtypes = [c_vp] * 9 + [I] * 14 + [F, F, I, c_vp]
+    l.tbv_op_latent_attn_rows.argtypes = [c_vp] * 7 + [I] * 8 + [F, I, I, c_vp]
+    l.tbv_op_short_conv.argtypes = [c_vp] * 7 + [I] * 7 + [c_vp]
+    l.tbv_op_delta_scan.argtypes = [c_vp] * 14 + [I] * 14 + [F, I, c_vp]
+    l.tbv_op_delta_step.argtypes = [c_vp] * 17 + [I] * 12 + [F, I, c_vp]
+    l.tbv_op_head_attn_prep.argtypes = [c_vp] * 9 + [I] * 10 + [F, I, c_vp]
     l.tbv_op_latent_gather.argtypes = [c_vp] * 4 + [I] * 3 + [c_vp]
     l.tbv_op_latent_prefill_fits.argtypes = [I, I, I]
-    l.tbv_op_latent_prefill.argtypes = [c_vp] * 6 + [I] * 10 + [F, c_vp]
+    l.tbv_op_latent_prefill.argtypes = [c_vp] * 6 + [I] * 10 + [F, I, c_vp]
     l.tbv_op_gemm_persist_mode.argtypes = [I]
     l.tbv_op_gemm_persist_mode.restype = None
     l.tbv_op_gemm_streamk_min_bytes.argtypes = [ctypes.c_long]
@@ -132,7 +136,7 @@ def _count(n=1):
 
 
 EPI_STORE, EPI_SILU_MUL, EPI_F32, EPI_CLAMP_GLU = 0, 1, 2, 3
-ACT_NONE, ACT_SOFTPLUS, ACT_SOFTCAP, ACT_SILU = 0, 1, 2, 3          # a soft cap of 1 is tanh
+ACT_NONE, ACT_SOFTPLUS, ACT_SOFTCAP, ACT_SILU, ACT_GELU = 0, 1, 2, 3, 4          # a soft cap of 1 is tanh; GELU in its tanh form
 SILU_GLU = (math.inf, 1.0, 0.0)           # ``glu`` of ``linear``: silu(gate) * up
 RELU_GLU = (math.inf, math.inf, 0.0)      # relu(gate) * up
 
@@ -166,7 +170,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[t
            last: int = 0, act_cols: int = 0) -> torch.Tensor:
     """out[N, M] = epilogue(x[N, K] @ w[M, K]^T + bias) for bf16 operands (tcgen05) or fp32 operands (CUDA cores, full 32-bit).
 
-    The output dtype is ``out``'s: fp32 results take an activation (``ACT_SOFTPLUS``, ``ACT_SOFTCAP`` with its limit in ``act_arg``, ``ACT_SILU``)
+    The output dtype is ``out``'s: fp32 results take an activation (``ACT_SOFTPLUS``, ``ACT_SOFTCAP`` with its limit in ``act_arg``, ``ACT_SILU``, ``ACT_GELU``)
     and, from bf16 operands, an optional bf16 ``copy`` with the same row stride; ``act_cols`` > 0 (a multiple of 16; results of the operands' dtype): the
     activation acts on that many leading columns.  ``glu=(limit, slope[, shift = 1])``: ``w`` holds gate / up rows
     interleaved and out[N, M/2] = g * sigmoid(slope * g) * (u + shift) with g = min(gate, limit), u = clamp(up, -limit, limit).
@@ -451,8 +455,8 @@ def prefill_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
     return out
 
 
-from .mixers import (DECAY_RANK_MAX, SHARED_PREFILL_MAX_DIM, causal_conv_silu, decay_powers, decay_scan, decay_step, fixed_decay_scan,  # noqa: E402,F401
-                     fixed_decay_step, fixed_decay_sums, hyper_embed, hyper_mix, latent_attention_prefill, latent_attention_rows, latent_gather,
-                     latent_prefill_fits, latent_prep, latent_row, moe_place_table, moe_route, moe_table_layers, paired_attention_prefill, paired_attention_prep,
-                     paired_attention_rows, paired_prefill_fits, position_turns, residual, rotation_turns, selective_scan, shared_attention_prefill,
-                     shared_attention_prep, shared_attention_rows, token_shift)
+from .mixers import (DECAY_RANK_MAX, SHARED_PREFILL_MAX_DIM, causal_conv_silu, decay_powers, decay_scan, decay_step, delta_scan, delta_step,  # noqa: E402,F401
+                     fixed_decay_scan, fixed_decay_step, fixed_decay_sums, frequency_turns, head_attention_prep, hyper_embed, hyper_mix,
+                     latent_attention_prefill, latent_attention_rows, latent_gather, latent_prefill_fits, latent_prep, latent_row, moe_place_table, moe_route,
+                     moe_table_layers, paired_attention_prefill, paired_attention_prep, paired_attention_rows, paired_prefill_fits, position_turns, residual,
+                     rotation_turns, selective_scan, shared_attention_prefill, shared_attention_prep, shared_attention_rows, short_conv, token_shift)

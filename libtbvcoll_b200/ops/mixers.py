@@ -65,6 +65,16 @@ def selective_scan(u, xz, z_off: int, dt, bc, b_off: int, c_off: int, a_log2e, d
     _count()
 
 
+def short_conv(x, out, taps, state, segs, seg_of_row, positions, add: bool = False) -> None:
+    """out = silu(conv(x)), or x + conv(x) with ``add`` (x fp32 then): causal depthwise convolution over time of the first taps.shape[1] columns of x; taps fp32
+    [K, C] with the last row weighing the current token.  state fp32 [slots, K - 1, C] holds the inputs before a segment's first row and is replaced by its last ones."""
+    K, C = taps.shape
+    assert state.shape[1:] == (K - 1, C) and state.dtype is taps.dtype is torch.float32 and (x.dtype is out.dtype or (add and x.dtype is torch.float32))
+    _chk(lib().tbv_op_short_conv(_p(x), _p(out), _p(taps), _p(state), _p(segs), _p(seg_of_row), _p(positions), x.shape[0], x.stride(0), out.stride(0), C, K, int(add),
+                                 _is_bf16(out), _st()), "tbv_op_short_conv")
+    _count()
+
+
 LATENT_ROW_PAD = 8
 
 
@@ -74,27 +84,31 @@ def latent_row(rank_p: int, rot_p: int) -> int:
     return rank_p + rot_p + LATENT_ROW_PAD
 
 
-def latent_prep(qkv, qa, cache, gamma, inv_freq, mscale: float, positions, slots, n_rows_form: int, q_off: int, c_off: int, k_off: int, heads: int,
-                rank: int, rank_p: int, rot_p: int, eps: float) -> None:
-    """Rotates the query parts (columns q_off.., heads x rot_p; interleaved pairs) and writes the cache row: RMSNorm of the latent
-    (c_off..) and the rotated key part (k_off..).  The first n_rows_form rows' query parts go to qa [rows, heads, row], the
-    others stay in place.  Rows of qa and cache: ``latent_row``.  cos and sin are multiplied by mscale."""
-    assert qkv.dtype is qa.dtype is cache.dtype and cache.shape[1] == latent_row(rank_p, rot_p) and positions.dtype is torch.int32 and slots.dtype is torch.int64
-    _chk(lib().tbv_op_latent_prep(_p(qkv), _p(qa), _p(cache), _p(gamma), _p(inv_freq), _p(positions), _p(slots), qkv.shape[0], n_rows_form,
-                                  qkv.stride(0), q_off, c_off, k_off, heads, rank, rank_p, rot_p, inv_freq.shape[0], eps, mscale, _is_bf16(qkv), _st()),
-         "tbv_op_latent_prep")
+def latent_prep(low, q, qa, cache, gamma, turns, mscale: float, positions, slots, n_rows_form: int, q_off: int, c_off: int, k_off: int, heads: int,
+                rank: int, rank_p: int, rot_p: int, eps: float, query_latent=None) -> None:
+    """Rotates the query parts of q (columns q_off.., heads x rot_p; interleaved pairs) and writes the cache row: RMSNorm of the latent of low
+    (c_off..) and its rotated key part (k_off..).  The first n_rows_form rows' query parts go to qa [rows, heads, row], the
+    others stay in place.  Rows of qa and cache: ``latent_row``.  ``turns`` of ``rotation_turns``; cos and sin are multiplied by mscale.  ``query_latent`` =
+    (column, size, weight fp32): that part of low is RMS-normed in place.  low or q may be None (then its part is left out)."""
+    act = low if low is not None else q
+    assert act.dtype is cache.dtype and cache.shape[1] == latent_row(rank_p, rot_p) and positions.dtype is torch.int32 and turns.dtype is torch.float32
+    assert (q is None or (qa.dtype is q.dtype and q.stride(1) == 1)) and (low is None or (slots.dtype is torch.int64 and gamma.dtype is torch.float32))
+    col, size, weight = query_latent if query_latent is not None else (0, 0, None)
+    _chk(lib().tbv_op_latent_prep(_p(low), _p(q), _p(qa), _p(cache), _p(gamma), _p(weight), _p(turns), _p(positions), _p(slots), act.shape[0], n_rows_form,
+                                  low.stride(0) if low is not None else 0, q.stride(0) if q is not None else 0, q_off, c_off, k_off, col, size, heads, rank, rank_p,
+                                  rot_p, turns.shape[0], eps, mscale, _is_bf16(act), _st()), "tbv_op_latent_prep")
     _count()
 
 
-def latent_attention_rows(qa, cache, tables, seq_of_row, ctx_lens, sink, out, rank: int, scale: float, block_size: int, splits: int = 1) -> None:
+def latent_attention_rows(qa, cache, tables, seq_of_row, ctx_lens, sink, out, rank: int, scale: float, block_size: int, splits: int = 1, window: int = 0) -> None:
     """qa [rows, heads, row] against the cache rows (keys over all columns of ``latent_row`` but the pad, values = the first out.shape[2] columns); softmax with
-    exp(sink) in the denominator (sink fp32 [heads] or None)."""
+    exp(sink) in the denominator (sink fp32 [heads] or None); a row sees the last ``window`` keys (0: all)."""
     rows, H, row = qa.shape
     Rp, Dk = out.shape[2], row - LATENT_ROW_PAD
     assert qa.is_contiguous() and out.is_contiguous() and cache.shape[1] == row and qa.dtype is cache.dtype is out.dtype
     assert tables.dtype is torch.int32 and ctx_lens.dtype is torch.int32
     _chk(lib().tbv_op_latent_attn_rows(_p(qa), _p(cache), _p(tables), _p(seq_of_row), _p(ctx_lens), _p(sink), _p(out), rows, H, rank, Rp, Dk - Rp,
-                                       block_size, tables.shape[1], splits, scale, _is_bf16(qa), _st()), "tbv_op_latent_attn_rows")
+                                       block_size, tables.shape[1], splits, scale, window, _is_bf16(qa), _st()), "tbv_op_latent_attn_rows")
     _count()
 
 
@@ -109,34 +123,36 @@ def latent_prefill_fits(dim_p: int, rot_p: int, v_p: int) -> bool:
     return bool(lib().tbv_op_latent_prefill_fits(dim_p, rot_p, v_p))
 
 
-def latent_attention_prefill(qkv, q_rot_off: int, kv, kr, tiles, sink, out, heads: int, dim_p: int, v_p: int, scale: float) -> None:
+def latent_attention_prefill(qkv, q_rot_off: int, kv, kr, tiles, sink, out, heads: int, dim_p: int, v_p: int, scale: float, window: int = 0) -> None:
     """Many query rows against expanded keys / values: kv [ctx rows, heads * dim_p | heads * v_p], rotated key parts kr [ctx rows, rot_p];
-    tiles int32 [n, 4] = (first query row, rows <= 64, first ctx row of the sequence, keys the first row sees)."""
+    tiles int32 [n, 4] = (first query row, rows <= 64, ctx row of the sequence's first token, keys the first row sees).  With a ``window`` rows before the first
+    visible key's tile of 64 positions are not read (and need not be there: that ctx row may lie before the first one)."""
     assert qkv.dtype is kv.dtype is kr.dtype is out.dtype is torch.bfloat16 and tiles.dtype is torch.int32
     _chk(lib().tbv_op_latent_prefill(_p(qkv), _p(kv), _p(kr), _p(tiles), _p(sink), _p(out), tiles.shape[0], heads, qkv.stride(0), q_rot_off,
-                                     kv.stride(0), heads * dim_p, out.stride(0), dim_p, kr.shape[1], v_p, scale, _st()), "tbv_op_latent_prefill")
+                                     kv.stride(0), heads * dim_p, out.stride(0), dim_p, kr.shape[1], v_p, scale, window, _st()), "tbv_op_latent_prefill")
     _count()
 
 
 # ---- one residual stream with parallel branches -----------------------------------------------------------------------------
 def position_turns(width: int, device, base: float = 10000.0) -> torch.Tensor:
     """fp32 [ceil(width / 2), 2]: turns per position of every sine / cosine pair of the position vector, as high and low part."""
-    return _turns(base ** (-2.0 * torch.arange((width + 1) // 2, dtype=torch.float64) / width), device)
+    return frequency_turns(base ** (-2.0 * torch.arange((width + 1) // 2, dtype=torch.float64) / width), device)
 
 
 def rotation_turns(dims: int, base: float, device) -> torch.Tensor:
     """fp32 [dims / 2, 2]: the same for the pairs of a rotation over ``dims`` dimensions."""
-    return _turns(float(base) ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / max(dims, 1)), device)
+    return frequency_turns(float(base) ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / max(dims, 1)), device)
 
 
-def _turns(freq: torch.Tensor, device) -> torch.Tensor:
+def frequency_turns(freq: torch.Tensor, device) -> torch.Tensor:
+    """fp32 [n, 2]: turns per position of the angular frequencies ``freq`` (float64), as high and low part."""
     f = freq / (2.0 * math.pi)
     hi = f.to(torch.float32)
     return torch.stack((hi, (f - hi.double()).to(torch.float32)), 1).contiguous().to(device)
 
 
 def residual(x, g1, h1, width: int, eps: float, g2=None, h2=None, embed=None, positions=None, y1=None, y2=None, routed=None, x0=None, step=None,
-             rows: Optional[torch.Tensor] = None, last: bool = False, mix=None, post=None, sums=None, place=None) -> None:
+             rows: Optional[torch.Tensor] = None, last: bool = False, mix=None, post=None, sums=None, place=None, conv=None) -> None:
     """x <- x + y1 + y2 + sum_j weight_j * routed_j (+ x0 + step);  h1 := RMSNorm(x) * g1,  h2 := RMSNorm(x) * g2.
 
     x, y1, y2, x0 fp32 [rows, ld].  ``routed`` = (rows of the experts' results, place int32 [rows, top], weight fp32 [rows, top]).
@@ -146,9 +162,13 @@ def residual(x, g1, h1, width: int, eps: float, g2=None, h2=None, embed=None, po
     h1 + (previous h1 - h1) * mu_s are written, and shift is replaced.
     ``post`` (fp32 [ld]): x <- x + RMSNorm(branches) * post instead, the branches being y1 and ``routed``, whose weight may be one number.  ``sums`` = (square sums
     fp32 [rows, n], width): y1 is divided by sqrt(sum / width + eps) first.  ``place`` int32 [rows, top]: h1 goes to these rows of ``h1``.
-    ``turns`` None: no position vector."""
+    ``turns`` None: no position vector.
+    g1 None: h1 := x.  h1 None: only x is written.  ``conv`` = (taps fp32 [k, ld], past fp32 [slots, k - 1, ld], segs): one row per segment; the causal
+    convolution of h1 over time is added to it, past is replaced (``short_conv`` for many rows)."""
     ld = x.shape[1]
     n = h1.shape[0] if last else x.shape[0]
+    taps, past, conv_segs = conv if conv is not None else (None, None, None)
+    assert taps is None or (taps.shape[1] == ld and taps.dtype is past.dtype is torch.float32 and past.shape[1:] == (taps.shape[0] - 1, ld) and mix is None)
     assert x.dtype is torch.float32 and x.is_contiguous() and (h2 is None or h2.stride(0) == h1.stride(0)) and (rows is None or (last and rows.dtype is torch.int64))
     for t in (y1, y2, x0):
         assert t is None or (t.dtype is torch.float32 and t.stride(0) == ld)
@@ -158,8 +178,10 @@ def residual(x, g1, h1, width: int, eps: float, g2=None, h2=None, embed=None, po
     weight = None if isinstance(weight, float) else weight
     sq, sum_width = sums if sums is not None else (None, 0)
     mu, mixes, shift, segs = mix if mix is not None else (None, None, None, None)
-    act = [t.dtype for t in (table, ro, h2, mixes) if t is not None] or [h1.dtype]
-    assert all(d is act[0] for d in act) and (h1.dtype is act[0] or h1.dtype is torch.float32)
+    act = [t.dtype for t in (table, ro, h2, mixes, h1) if t is not None] or [torch.float32]
+    h1_f32 = h1 is not None and h1.dtype is torch.float32
+    assert all(d is act[0] for d in act[:-1]) and (h1 is None or h1.dtype is act[0] or h1_f32)
+    segs = conv_segs if segs is None else segs
     assert ro is None or (ro.stride(0) == ld and source.dtype is torch.int32 and source.is_contiguous() and (weight is None or weight.dtype is torch.float32))
     assert place is None or (place.dtype is torch.int32 and place.is_contiguous() and place.shape[0] == x.shape[0] and h1.shape[0] >= place.numel())
     assert sq is None or (sq.dtype is torch.float32 and sq.is_contiguous() and post is not None)
@@ -167,9 +189,10 @@ def residual(x, g1, h1, width: int, eps: float, g2=None, h2=None, embed=None, po
     assert mu is None or (mixes.shape[1] == mu.shape[0] * ld and shift.shape[1] == ld and shift.dtype is torch.float32)
     _chk(lib().tbv_op_residual(_p(ids), _p(table), _p(turns), _p(positions), scale, table.shape[0] if table is not None else 0, _p(x), _p(x0), _p(y1), _p(y2),
                                _p(step), _p(ro), _p(source), _p(weight), source.shape[1] if source is not None else 0, _p(g1), _p(g2), _p(h1), _p(h2),
-                               int(h1.dtype is torch.float32), _p(rows), int(last), _p(mu), _p(mixes), _p(shift), _p(segs),
+                               int(h1_f32), _p(rows), int(last), _p(mu), _p(mixes), _p(shift), _p(segs),
                                mu.shape[0] if mu is not None else 0, _p(post), _p(sq), sq.shape[1] if sq is not None else 0, sum_width, const, _p(place),
-                               place.shape[1] if place is not None else 0, n, width, ld, h1.stride(0), eps, int(act[0] is torch.bfloat16), _st()), "tbv_op_residual")
+                               place.shape[1] if place is not None else 0, _p(taps), _p(past), taps.shape[0] if taps is not None else 0, n, width, ld,
+                               h1.stride(0) if h1 is not None else ld, eps, int(act[0] is torch.bfloat16), _st()), "tbv_op_residual")
     _count()
 
 
@@ -273,6 +296,42 @@ def fixed_decay_step(q, k, v, g, norm, powers, state, out, sums, segs, positions
     _count()
 
 
+# ---- gated delta rule with a decay per key channel -----------------------------------------------------------------------------------
+def delta_scan(q, k, v, beta, z, gate, rate, norm, state, o, out, segs, positions, kv_heads: int, dim: int, vdim: int, eps: float, groups=None) -> None:
+    """Per head, q and k of its key head made unit vectors (q times dim^-0.5), S' = diag(exp(-rate softplus(z_t))) S_{t-1}, u = sigmoid(beta_t) (v_t - S'^T k_t),
+    S_t = S' + k_t u^T over the rows of every segment; out = RMSNorm(S_t^T q_t) * norm * sigmoid(gate).
+
+    q, k [rows, kv_heads * Dp] and v [rows, heads * Vp]: column views of one buffer, behind convolution and SiLU; beta [rows, >= heads], gate [rows, heads * Vp] in the
+    activation type; z fp32 [rows, heads * Dp], rate fp32 [heads], norm fp32 [Vp]; state fp32 [slots, heads, Dp, Vp] is replaced; o fp32 scratch [rows, heads * Vp].
+    ``groups`` (bf16): the segments, int32 [n, 4] (engine.batch.scan_groups), for the chunked tensor-core kernel where the sizes allow."""
+    _, H, Dp, Vp = state.shape
+    rows = q.shape[0]
+    assert q.stride(0) == k.stride(0) == v.stride(0) and q.shape[1] == k.shape[1] == kv_heads * Dp and v.shape[1] == gate.shape[1] == H * Vp and z.shape[1] == H * Dp
+    assert state.dtype is z.dtype is rate.dtype is norm.dtype is o.dtype is torch.float32 and o.numel() >= rows * H * Vp and norm.shape[0] == Vp and rate.shape[0] == H
+    assert q.dtype is beta.dtype is gate.dtype is out.dtype and beta.shape[1] >= H and (groups is None or (q.dtype is torch.bfloat16 and groups.dtype is torch.int32))
+    _chk(lib().tbv_op_delta_scan(_p(q), _p(k), _p(v), _p(beta), _p(z), _p(gate), _p(rate), _p(norm), _p(state), _p(o), _p(out), _p(segs), _p(positions), _p(groups),
+                                 0 if groups is None else groups.shape[0], rows, segs.shape[0], H, kv_heads, Dp, Vp, dim, vdim, q.stride(0), beta.stride(0), z.stride(0),
+                                 gate.stride(0), out.stride(0), eps, _is_bf16(q), _st()), "tbv_op_delta_scan")
+    _count(2)
+
+
+def delta_step(q, k, v, beta, low_a, low_g, w_a, b_a, w_g, rate, norm, state, out, segs, positions, kv_heads: int, dim: int, vdim: int, eps: float, conv=None) -> None:
+    """``delta_scan`` for one row per segment, with z = low_a @ w_a^T + b_a and gate = low_g @ w_g^T computed inside.  ``conv`` = (taps fp32 [K, C], state fp32
+    [slots, K - 1, C]), for kv_heads = heads: q, k and v are taken before convolution and SiLU, and that state is replaced."""
+    _, H, Dp, Vp = state.shape
+    taps, past = conv if conv is not None else (None, None)
+    rank = w_a.shape[1]
+    assert q.stride(0) == k.stride(0) == v.stride(0) and q.shape[1] == k.shape[1] == kv_heads * Dp and v.shape[1] == H * Vp
+    assert beta.stride(0) == low_a.stride(0) == low_g.stride(0) and beta.shape[1] >= H and low_a.shape[1] == low_g.shape[1] == w_g.shape[1] == rank
+    assert w_a.shape[0] == b_a.shape[0] == H * Dp and w_g.shape[0] == H * Vp and w_a.is_contiguous() and w_g.is_contiguous()
+    assert state.dtype is rate.dtype is norm.dtype is torch.float32 and q.dtype is beta.dtype is low_a.dtype is w_a.dtype is b_a.dtype is w_g.dtype is out.dtype
+    assert taps is None or (taps.dtype is past.dtype is torch.float32 and kv_heads == H and taps.shape[1] == H * (2 * Dp + Vp) and past.shape[1:] == (taps.shape[0] - 1, taps.shape[1]))
+    _chk(lib().tbv_op_delta_step(_p(q), _p(k), _p(v), _p(beta), _p(low_a), _p(low_g), _p(w_a), _p(b_a), _p(w_g), _p(rate), _p(norm), _p(state), _p(out), _p(taps), _p(past),
+                                 _p(segs), _p(positions), segs.shape[0], H, kv_heads, Dp, Vp, dim, vdim, q.stride(0), beta.stride(0), rank,
+                                 taps.shape[0] if taps is not None else 0, out.stride(0), eps, _is_bf16(q), _st()), "tbv_op_delta_step")
+    _count()
+
+
 # ---- attention whose cached rows are keys and values at once --------------------------------------------------------------------
 SHARED_PREFILL_MAX_DIM = 256          # padded head size that the prefill form takes
 
@@ -327,6 +386,20 @@ def paired_attention_prep(wide, qa, cache, q_norm, k_norm, turns, positions, slo
     pairs = 0 if turns is None else turns.shape[0]
     _chk(lib().tbv_op_paired_attn_prep(_p(wide), _p(qa), _p(cache), _p(q_norm), _p(k_norm), _p(turns), _p(positions), _p(slots), wide.shape[0], n_rows_form,
                                        wide.stride(0), heads, kv_heads, dim, Dp, Vp, pairs, block_size, eps, _is_bf16(wide), _st()), "tbv_op_paired_attn_prep")
+    _count()
+
+
+def head_attention_prep(wide, qa, cache, qscale, turns, positions, slots, n_rows_form: int, heads: int, kv_heads: int, dim: int, dim_p: int, block_size: int, eps: float,
+                        v_first=None, mix=None) -> None:
+    """As ``paired_attention_prep``, with norms per head and without weights, and a factor per query head (qscale fp32 [heads]).  ``v_first`` [rows, kv_heads * Vp]:
+    takes this layer's values, or with ``mix`` (fp32, one number) is mixed into them: (1 - mix) v + mix v_first."""
+    Vp = cache.shape[1] - LATENT_ROW_PAD - dim_p
+    assert wide.dtype is qa.dtype is cache.dtype and wide.stride(1) == 1 and wide.shape[1] >= (heads + kv_heads) * dim_p + kv_heads * Vp and qscale.shape[0] == heads
+    assert slots.dtype is torch.int64 and positions.dtype is torch.int32 and qscale.dtype is torch.float32 and (mix is None or (mix.dtype is torch.float32 and v_first is not None))
+    assert v_first is None or (v_first.dtype is wide.dtype and v_first.is_contiguous() and v_first.shape == (wide.shape[0], kv_heads * Vp))
+    _chk(lib().tbv_op_head_attn_prep(_p(wide), _p(qa), _p(cache), _p(qscale), _p(turns), _p(positions), _p(slots), _p(v_first), _p(mix), wide.shape[0], n_rows_form,
+                                     wide.stride(0), heads, kv_heads, dim, dim_p, Vp, 0 if turns is None else turns.shape[0], block_size, eps, _is_bf16(wide), _st()),
+         "tbv_op_head_attn_prep")
     _count()
 
 

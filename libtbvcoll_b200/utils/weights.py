@@ -17,8 +17,8 @@ from typing import Callable, Dict, Iterable, Optional
 
 import torch
 
-from ..models.config import (BobaraxConfig, GatedMlpSpec, GlaSpec, LatentSpec, LightningSpec, MambaSpec, ModelConfig, NubosunConfig, TableMoeSpec, TinapelConfig,
-                             WkvSpec)
+from ..models.config import (BobaraxConfig, ChannelDeltaSpec, GatedMlpSpec, GlaSpec, LatentSpec, LightningSpec, LugizenConfig, MambaSpec, ModelConfig, MoeSpec,
+                             NubosunConfig, TableMoeSpec, TinapelConfig, WkvSpec)
 
 
 def hf_tensor_shapes(cfg: ModelConfig) -> Dict[str, tuple]:
@@ -124,9 +124,42 @@ def bobarax_tensor_shapes(cfg: BobaraxConfig) -> Dict[str, tuple]:
     return shapes
 
 
+def lugizen_tensor_shapes(cfg: LugizenConfig) -> Dict[str, tuple]:
+    """Ranks that the configuration leaves open are 16 here; in a checkpoint its tensors tell.  Norm weights of shape () are one number."""
+    W = cfg.hidden_size
+    shapes = {"embed": (cfg.vocab_size, W), "head": (cfg.vocab_size, W), "final.norm": ()}
+    for i, lay in enumerate(cfg.layers):
+        p, m, f = f"l{i}.", lay.mixer, lay.mlp
+        x, y, H, D, V = p + "mix.", p + "mlp.", m.heads, m.dim, m.vdim
+        shapes.update({p + "norm1": (), p + "canon1": (W, cfg.canon_taps), x + "o": (W, H * V)})
+        if isinstance(m, ChannelDeltaSpec):
+            K, Ra, Rg = m.kv_heads * D, m.decay_rank or 16, m.gate_rank or 16
+            for s, n in (("q", K), ("k", K), ("v", H * V)):
+                shapes.update({x + s: (n, W), x + s + ".conv": (n, m.conv)})
+            shapes.update({x + "b": (H, W), x + "A_log": (H,), x + "norm": (V,), x + "a1": (Ra, W), x + "a2": (H * D, Ra), x + "dt_bias": (H * D,), x + "g1": (Rg, W),
+                           x + "g2": (H * V, Rg)})
+        elif isinstance(m, LatentSpec):
+            shapes.update({x + "dq": (m.q_rank, W), x + "dq.norm": (m.q_rank,), x + "uq": (H * (D + m.rot_dim), m.q_rank), x + "dkv": (m.kv_rank + m.rot_dim, W),
+                           x + "dkv.norm": (m.kv_rank,), x + "uk": (H * D, m.kv_rank), x + "uv": (H * V, m.kv_rank)})
+        else:
+            shapes.update({x + "q": (H * D, W), x + "k": (m.kv_heads * D, W), x + "v": (m.kv_heads * V, W), x + "temp": (H,)})
+            if m.v_mix:
+                shapes[x + "vmix"] = ()
+        if f is not None:
+            shapes[p + "norm2"] = ()
+        if isinstance(f, MoeSpec):
+            shapes[y + "router"] = (f.experts, W)
+            for e in range(f.experts):
+                shapes.update({f"{y}e{e}.gate": (f.ff, W), f"{y}e{e}.up": (f.ff, W), f"{y}e{e}.down": (W, f.ff)})
+        elif f is not None:
+            shapes.update({y + "up": (f.ff, W), y + "down": (W, f.ff)})
+    return shapes
+
+
 def tensor_shapes(cfg) -> Dict[str, tuple]:
     """Checkpoint tensor names and shapes of a configuration of any architecture."""
-    for kind, shapes in ((NubosunConfig, nubosun_tensor_shapes), (TinapelConfig, tinapel_tensor_shapes), (BobaraxConfig, bobarax_tensor_shapes)):
+    for kind, shapes in ((NubosunConfig, nubosun_tensor_shapes), (TinapelConfig, tinapel_tensor_shapes), (BobaraxConfig, bobarax_tensor_shapes),
+                         (LugizenConfig, lugizen_tensor_shapes)):
         if isinstance(cfg, kind):
             return shapes(cfg)
     return hf_tensor_shapes(cfg)
@@ -160,6 +193,24 @@ def _bobarax_random(cfg: BobaraxConfig, name: str, shape: tuple, g: torch.Genera
     n = torch.randn(shape, generator=g, device=device, dtype=torch.float32)
     if len(shape) == 1:
         return 0.1 * n if leaf in ("norm1", "norm1b", "norm2", "norm2b", "final.norm") else 1.0 + 0.1 * n      # the former are stored around zero
+    return n if leaf == "embed" else n / shape[1] ** 0.5
+
+
+def _lugizen_random(name: str, shape: tuple, g: torch.Generator, device) -> torch.Tensor:
+    """Random values that keep a Lugizen's activations near unit size: decays over many time scales."""
+    leaf = name.split(".", 1)[1] if name.startswith("l") and "." in name else name
+    n = torch.randn(shape, generator=g, device=device, dtype=torch.float32)
+    u = lambda: torch.rand(shape, generator=g, device=device, dtype=torch.float32)
+    if len(shape) == 0:
+        return 0.5 + 0.1 * n if leaf == "mix.vmix" else 1.0 + 0.1 * n
+    if leaf == "mix.A_log":
+        return torch.log(1.0 + 15.0 * u())
+    if leaf == "mix.dt_bias":
+        return -7.0 + 5.0 * u()                       # softplus: steps of 0.001 .. 0.1
+    if len(shape) == 1:
+        return 1.0 + 0.1 * n
+    if leaf == "canon1":
+        return 0.3 * n
     return n if leaf == "embed" else n / shape[1] ** 0.5
 
 
@@ -211,6 +262,8 @@ class RandomSource:
             t = _tinapel_random(name, shape, g, self.device)
         elif isinstance(self.cfg, BobaraxConfig):
             t = _bobarax_random(self.cfg, name, shape, g, self.device)
+        elif isinstance(self.cfg, LugizenConfig):
+            t = _lugizen_random(name, shape, g, self.device)
         elif name.endswith("layernorm.weight") or name.endswith("norm.weight"):
             t = 1.0 + 0.1 * torch.randn(shape, generator=g, device=self.device, dtype=torch.float32)
         elif name.endswith(".bias"):
@@ -317,6 +370,28 @@ def _head_vector(t: torch.Tensor, heads: int, dim: int) -> torch.Tensor:
     return _pad_heads(t.reshape(-1, 1), heads, dim, _pad16(dim)).reshape(-1)
 
 
+def _pairs_together(t: torch.Tensor, heads: int, dims: int) -> torch.Tensor:
+    """Rows of every head reordered so that dimensions i and i + dims / 2 of the first ``dims`` become neighbours 2i and 2i + 1 (a rotation of such pairs, norms and
+    products between rows in this order do not notice)."""
+    t = t.reshape(heads, -1, t.shape[1])
+    order = torch.arange(t.shape[1], device=t.device)
+    order[:dims] = torch.arange(dims, device=t.device).view(2, -1).t().reshape(-1)
+    return t[:, order].reshape(-1, t.shape[2])
+
+
+def _latent_products(uk: torch.Tensor, uv: torch.Tensor, m: LatentSpec, dtype) -> Dict[str, torch.Tensor]:
+    """The forms in which latent attention takes W_uk and W_uv: ``wabs`` [heads * rank, dim] folds W_uk into the query, ``wuv`` [heads * vdim, rank] expands a latent,
+    ``wukv`` [heads * (dim + vdim), rank] gives keys then values (bf16 only)."""
+    H, D, V, R = m.heads, _pad16(m.dim), _pad16(m.vdim), _pad16(m.kv_rank)
+    wabs = torch.zeros(H, R, D, dtype=uk.dtype, device=uk.device)
+    wabs[:, : m.kv_rank, : m.dim] = uk.reshape(H, m.dim, m.kv_rank).transpose(1, 2)
+    wuv = _padded(_pad_heads(uv, H, m.vdim, V), H * V, R)
+    out = {"wabs": wabs.reshape(H * R, D), "wuv": wuv}
+    if dtype is torch.bfloat16:
+        out["wukv"] = torch.cat((_padded(_pad_heads(uk, H, m.dim, D), H * D, R), wuv))
+    return out
+
+
 class _Layout:
     """Checked reads from a checkpoint and the product layout being filled (``out``)."""
 
@@ -411,17 +486,9 @@ def load_nubosun(cfg: NubosunConfig, source, device, dtype=torch.bfloat16) -> Di
             put(x + "qkv", _padded(rows, rows.shape[0], Wp))
             put(x + "dkv.norm", get(x + "dkv.norm"), f32)
             put(x + "sink", get(x + "sink"), f32)
-            uk, uv = get(x + "uk"), get(x + "uv")
-            wabs = torch.zeros(H, R, D, dtype=uk.dtype, device=uk.device)
-            wabs[:, : m.kv_rank, : m.dim] = uk.reshape(H, m.dim, m.kv_rank).transpose(1, 2)
-            put(x + "wabs", wabs.reshape(H * R, D))
-            wuv = _padded(_pad_heads(uv, H, m.vdim, V), H * V, R)
-            put(x + "wuv", wuv)
-            if dtype is torch.bfloat16:
-                put(x + "wukv", torch.cat((_padded(_pad_heads(uk, H, m.dim, D), H * D, R), wuv)))
-            o = torch.zeros(Wp, H, V, dtype=uv.dtype, device=uv.device)
-            o[: cfg.hidden_size, :, : m.vdim] = get(x + "o").reshape(cfg.hidden_size, H, m.vdim)
-            put(x + "o", o.reshape(Wp, H * V))
+            for k, t in _latent_products(get(x + "uk"), get(x + "uv"), m, dtype).items():
+                put(x + k, t)
+            put(x + "o", _padded(_heads_padded(get(x + "o").t(), H, m.vdim).t(), Wp, H * V))
         if lay.mlp is not None:
             x, fp = p + "mlp.", _pad16(lay.mlp.ff)
             g, u = _padded(get(x + "gate"), fp, Wp), _padded(get(x + "up"), fp, Wp)
@@ -528,6 +595,67 @@ def load_bobarax(cfg: BobaraxConfig, source, device, dtype=torch.bfloat16) -> Di
                 raise ValueError(f"{y}table: not a table of {f.experts} experts")
             put(y + "table", table, torch.int32)
             L.put_experts(y, f.experts, f.ff)
+    return L.out
+
+
+def load_lugizen(cfg: LugizenConfig, source, device, dtype=torch.bfloat16) -> Dict[str, torch.Tensor]:
+    """Tensors the way the kernels consume them; dimensions of matrix products and heads are zero-padded to multiples of 16, parameters that act in 32-bit are
+    fp32; norms of one number are spread over the width; convolutions are transposed to [taps, channels].
+
+    Delta rule: ``in`` stacks q, k, v, both first low-rank projections (padded to one rank) and the step sizes; ``conv`` covers q, k, v; ``rate`` = exp(A_log).
+    Attention: ``in`` stacks q, k, v; rotated pairs lie next to each other; ``qscale`` = score scale times the head's number.  Latent attention: ``down`` stacks the
+    queries' latent, the latent and the rotated key part, ``uq`` the heads' unrotated rows, then their rotated ones (pairs next to each other)."""
+    L, f32 = _Layout(cfg, source, device, dtype), torch.float32
+    W, Wp, get, put = L.W, L.Wp, L.get, L.put
+    spread = lambda name: put(name, _padded(get(name).float().reshape(1).expand(W), Wp), f32)
+    put("embed", _padded(get("embed"), cfg.vocab_size, Wp))
+    put("head", _padded(get("head"), _pad16(cfg.vocab_size), Wp))
+    spread("final.norm")
+    for i, lay in enumerate(cfg.layers):
+        p, m, f = f"l{i}.", lay.mixer, lay.mlp
+        x, y, H, D, V = p + "mix.", p + "mlp.", m.heads, m.dim, m.vdim
+        spread(p + "norm1")
+        put(p + "canon1", _padded(get(p + "canon1").t(), cfg.canon_taps, Wp), f32)
+        put(x + "o", L.out_proj(get(x + "o"), H, V))
+        if isinstance(m, ChannelDeltaSpec):
+            G, a1, g1 = m.kv_heads, get(x + "a1", 0), get(x + "g1", 0)
+            R = _pad16(max(a1.shape[0], g1.shape[0]))
+            parts = (("q", G, D), ("k", G, D), ("v", H, V))
+            rows = torch.cat([_heads_padded(get(x + s), n, d) for s, n, d in parts] + [_padded(a1, R, W), _padded(g1, R, W), _padded(get(x + "b"), _pad16(H), W)])
+            put(x + "in", _padded(rows, rows.shape[0], Wp))
+            put(x + "conv", torch.cat([_heads_padded(get(x + s + ".conv"), n, d) for s, n, d in parts]).t(), f32)
+            put(x + "a2", _padded(_heads_padded(get(x + "a2", 1), H, D), H * _pad16(D), R))
+            put(x + "dt_bias", _head_vector(get(x + "dt_bias"), H, D))
+            put(x + "g2", _padded(_heads_padded(get(x + "g2", 1), H, V), H * _pad16(V), R))
+            put(x + "rate", torch.exp(get(x + "A_log").float()), f32)
+            put(x + "norm", _padded(get(x + "norm"), _pad16(V)), f32)
+        elif isinstance(m, LatentSpec):
+            R, Rq, rot = _pad16(m.kv_rank), _pad16(m.q_rank), _pad16(m.rot_dim)
+            q, kv = get(x + "uq").reshape(H, D + m.rot_dim, -1), get(x + "dkv")
+            rows = torch.cat((_padded(get(x + "dq"), Rq, W), _padded(kv[: m.kv_rank], R, W), _padded(_pairs_together(kv[m.kv_rank:], 1, m.rot.dims), rot, W)))
+            put(x + "down", _padded(rows, rows.shape[0], Wp))
+            rows = torch.cat((_heads_padded(q[:, :D].reshape(H * D, -1), H, D), _heads_padded(_pairs_together(q[:, D:].reshape(H * m.rot_dim, -1), H, m.rot.dims), H, m.rot_dim)))
+            put(x + "uq", _padded(rows, rows.shape[0], Rq))
+            put(x + "dq.norm", get(x + "dq.norm"), f32)
+            put(x + "dkv.norm", get(x + "dkv.norm"), f32)
+            for k, t in _latent_products(get(x + "uk"), get(x + "uv"), m, dtype).items():
+                put(x + k, t)
+        else:
+            G, dims = m.kv_heads, m.rot.dims if m.rot is not None else 0
+            rows = torch.cat((_heads_padded(_pairs_together(get(x + "q"), H, dims), H, D), _heads_padded(_pairs_together(get(x + "k"), G, dims), G, D),
+                              _heads_padded(get(x + "v"), G, V)))
+            put(x + "in", _padded(rows, rows.shape[0], Wp))
+            put(x + "qscale", get(x + "temp").float() * m.scale, f32)
+            if m.v_mix:
+                put(x + "vmix", get(x + "vmix").reshape(1), f32)
+        if f is not None:
+            spread(p + "norm2")
+        if isinstance(f, MoeSpec):
+            put(y + "router", _padded(get(y + "router"), _pad16(f.experts), Wp))
+            L.put_experts(y, f.experts, f.ff)
+        elif f is not None:
+            put(y + "up", _padded(get(y + "up"), _pad16(f.ff), Wp))
+            put(y + "down", _padded(get(y + "down"), Wp, _pad16(f.ff)))
     return L.out
 
 

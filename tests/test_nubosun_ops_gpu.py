@@ -345,9 +345,9 @@ def test_latent_prep_rotates_norms_and_writes_the_cache(dtype, H, dim, rot, R, d
     row = ops.latent_row(Rp, rp)
     qa, cache = torch.zeros(nf, H, row, dtype=dtype, device=DEV), torch.full((40, row), 4.0, dtype=dtype, device=DEV)
     slots = torch.tensor([33, 2, 3, 17, 18, 19, 30, 1, 39])
-    ops.latent_prep(qkv, qa, cache, gam.to(DEV), freq.float().to(DEV), factor, pos.to(DEV), slots.to(DEV), nf, H * Dp, co, co + Rp, H, R, Rp, rp, eps)
-    # angles in 32-bit, as the model defines them
-    ang = (pos.float()[:, None] * freq.float()[None]).double()
+    ops.latent_prep(qkv, qkv, qa, cache, gam.to(DEV), ops.frequency_turns(freq, DEV), factor, pos.to(DEV), slots.to(DEV), nf, H * Dp, co, co + Rp, H, R, Rp, rp, eps)
+    # angles, factor aside
+    ang = pos.double()[:, None] * freq[None]
     cos, sin = torch.cos(ang) * factor, torch.sin(ang) * factor
 
     def turn(x):
