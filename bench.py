@@ -20,7 +20,8 @@ Rank 0 prints ONE JSON line.  With 2 or more GPUs the line of ``--impl ours`` al
                      device time of calls captured in one CUDA graph, max over ranks, bit-exactness asserted.
 ``--compare nubosun`` (one GPU): instead of the headline, prefill and decode throughput and every kernel's roofline fraction of the
 Nubosun design beside a Llama of equal width, depth, feed-forward, heads and vocabulary (``--sizes 2k,8b``); one JSON line.
-``--compare tinapel`` does the same for the Tinapel design beside Nubosun and Llama, ``--compare bobarax`` for Bobarax beside Tinapel and Llama.
+``--compare tinapel`` does the same for the Tinapel design beside Nubosun and Llama, ``--compare bobarax`` for Bobarax beside Tinapel and Llama,
+``--compare lugizen`` for Lugizen beside Tinapel, Nubosun and Llama.
 ``--shard-of N`` (one GPU): rank 0's shard of a TP=N model with every collective replaced by its local
 arithmetic — no communication, wrong values; it exists to attribute the compute part of a TP=N step.
 """
@@ -51,7 +52,7 @@ def parse():
     ap.add_argument("--layers", type=int, default=0, help="debug only: override the layer count (marks the line INVALID)")
     ap.add_argument("--repeats", type=int, default=0, help="timed regions of --steps steps each (0 = enough for about 0.5 s in total, at most 12)")
     ap.add_argument("--shard-of", type=int, default=0, help="attribution only (marks the line INVALID): one GPU runs one rank's shard of a TP=N model, collectives replaced by local arithmetic")
-    ap.add_argument("--compare", default=None, choices=["nubosun", "tinapel", "bobarax"], help="another design beside the closest model at equal sizes, instead of the headline")
+    ap.add_argument("--compare", default=None, choices=["nubosun", "tinapel", "bobarax", "lugizen"], help="another design beside the closest model at equal sizes, instead of the headline")
     ap.add_argument("--sizes", default="2k,8b", help="sizes of --compare")
     ap.add_argument("--no-extras", action="store_true", help="skip the same-engine NCCL arm and the all-reduce latencies")
     return ap.parse_args()

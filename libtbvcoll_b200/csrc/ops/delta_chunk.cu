@@ -13,8 +13,9 @@
 // fp32 numbers carried as sums of kParts bf16 numbers, products of parts kept down to the kParts-th order (three parts: 24 bits, as fp32); what only enters the output,
 // which is rounded to bf16 behind the head norm, in two.
 //
-// A CTA alternates between making a chunk's operands (elementwise, shared memory) and its products; two CTAs per SM overlap the two.  If a CTA owns all
-// value columns of its head, head norm, weight and gate follow here as well.
+// Eight warps of a CTA make the chunks' operands (they do not depend on the state), eight others take them through the products, one or two chunks behind; two sets
+// of operands pass between them.  The two groups meet in named barriers only: `full` (operands of a set are there) and `empty` (its products are done).  If a
+// CTA owns all value columns of its head, head norm, weight and gate follow here as well.
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
@@ -32,7 +33,7 @@ using vec::unpack2;
 
 namespace {
 
-constexpr int kC = 16, kNW = 8, kNT = kNW * 32, kCols = kNW * 16;    // tokens of a chunk, warps, threads, value columns of a CTA
+constexpr int kC = 16, kNW = 8, kNT = kNW * 32, kCols = kNW * 16;    // tokens of a chunk, warps and threads of a group, value columns of a CTA
 constexpr int kParts = 3;
 
 template <int DK>
@@ -42,27 +43,34 @@ struct Shape {
   static constexpr int kVPitch = kCols * 2 + 16;
   static constexpr int kAPitch = kC * 2 + 16;
   static constexpr int kOPitch = kCols + 4;                        // floats
-  // byte offsets of dynamic shared memory
+  // a set of operands, byte offsets in it
   static constexpr int oQ = 0;                                     // q P                 [2][16][pitch]
   static constexpr int oK = oQ + 2 * kC * kPitch;                  // k P                 [parts][16][pitch]
   static constexpr int oR = oK + kParts * kC * kPitch;             // k R                 [parts][16][pitch]
-  static constexpr int oTa = oR + kParts * kC * kPitch;            // blocks: left rows   [parts][2 kinds][16][pitch]  (8 of q, 8 of k)
+  static constexpr int oV = oR + kParts * kC * kPitch;             // v                   [16][vpitch]
+  static constexpr int oA = oV + kC * kVPitch;                     // A                   [2][16][apitch]
+  static constexpr int oT = oA + 2 * kC * kAPitch;                 // T                   [parts][16][apitch]
+  static constexpr int oE = oT + kParts * kC * kAPitch;            // P_16                [DK] fp32
+  static constexpr int kSet = oE + DK * 4;
+  // dynamic shared memory: two sets, then what one of the groups has for itself
+  static constexpr int oTa = 2 * kSet;                             // blocks: left rows   [parts][2 kinds][16][pitch]  (8 of q, 8 of k)
   static constexpr int oTb = oTa + kParts * 32 * kPitch;           //         right rows  [parts][2 kinds][8][pitch]
-  static constexpr int oV = oTb + kParts * 16 * kPitch;            // v                   [2 chunks][16][vpitch]
-  static constexpr int oZ = oV + 2 * kC * kVPitch;                 // raw decay inputs    [16][DK] fp32
+  static constexpr int oZ = oTb + kParts * 16 * kPitch;            // raw decay inputs    [16][DK] fp32
   static constexpr int oRq = oZ + kC * DK * 4;                     // raw q, k            [16][DK] bf16 each
   static constexpr int oRk = oRq + kC * DK * 2;
-  static constexpr int oE = oRk + kC * DK * 2;                     // P_16                [DK] fp32
-  static constexpr int oF = oE + DK * 4;                           // factors of q, of k, step sizes [3][16] fp32
-  static constexpr int oTri = oF + 3 * kC * 4;                     // diagonal blocks     [items][4 quarters][16] fp32; then an inverse [16][17], a product [8][17]
-  static constexpr int kTri = kItems * 256 > 24 * 17 * 4 ? kItems * 256 : 24 * 17 * 4;
-  static constexpr int oA = oTri + kTri;                           // A                   [2][16][apitch]
-  static constexpr int oT = oA + 2 * kC * kAPitch;                 // T                   [parts][16][apitch]
-  static constexpr int oL = oT + kParts * kC * kAPitch;            // diag(beta) B        [16][17] fp32
-  static constexpr int oO = oL + 16 * 17 * 4;   // o                 [16][opitch] fp32; before that the blocks' sums [warps][2][16][8]
+  static constexpr int oF = oRk + kC * DK * 2;                     // factors of q, of k, step sizes [2 chunks][3][16] fp32
+  static constexpr int oTri = oF + 6 * kC * 4;                     // diagonal blocks     [items][4 quarters][16] fp32
+  static constexpr int oOff = oTri + (kItems + 1) * 256;           // the other blocks' sums [warps][2][16][8] fp32
+  static constexpr int oL = oOff + kNW * 1024;                     // diag(beta) B [16][17] fp32, its inverse [16][17], a product [8][17]
+  static constexpr int oO = oL + 40 * 17 * 4;                      // o                   [16][opitch] fp32
   static constexpr int kBytes = oO + kC * kOPitch * 4;
-  static_assert(oO % 16 == 0 && kBytes <= 113 * 1024, "two CTAs per SM");
+  static_assert(kSet % 16 == 0 && oO % 16 == 0 && kBytes <= int(kMaxSmem), "shared memory");
 };
+
+// Named barriers (0 is __syncthreads): one inside each group, `full` and `empty` of each set of operands.
+enum Bar : int { kMakers = 1, kProducts = 2, kFull = 3, kEmpty = 5 };
+__device__ __forceinline__ void bar_sync(int id, int threads) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
+__device__ __forceinline__ void bar_arrive(int id, int threads) { asm volatile("bar.arrive %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
 
 __device__ __forceinline__ void st_shared(uint32_t addr, uint32_t v) { asm volatile("st.shared.b32 [%0], %1;" ::"r"(addr), "r"(v) : "memory"); }
 __device__ __forceinline__ float2 of2(f32x2 v) {
@@ -103,50 +111,45 @@ __device__ __forceinline__ void as_left(const float (*v)[4], uint32_t (*a)[4]) {
   }
 }
 
-template <int DK>
-__global__ void __launch_bounds__(kNT, 2) k_delta_chunk(const Params p, const int* groups) {
-  using S = Shape<DK>;
-  extern __shared__ __align__(16) uint8_t sm[];
-  pdl::launch_dependents();
-  pdl::grid_dependency_wait();
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r8 = lane >> 2, quad = lane & 3;
-  const int h = blockIdx.y, g = h / (p.heads / p.kv_heads);
-  const int first = groups[4 * blockIdx.x], n = groups[4 * blockIdx.x + 1], slot = groups[4 * blockIdx.x + 2];
-  const bool fresh = p.positions[first] == 0;
-  const int vb = blockIdx.z * kCols, v0 = vb + warp * 16;           // first value column of the CTA, of the warp
-  const bool mma_warp = v0 < p.Vp, fused = p.o == nullptr;
-  const uint32_t base = smem_addr(sm);
-  const float rate = p.rate[h], qscale = rsqrtf(float(p.dim));
-  const __nv_bfloat16* qg = static_cast<const __nv_bfloat16*>(p.q) + size_t(g) * p.Dp;
-  const __nv_bfloat16* kg = static_cast<const __nv_bfloat16*>(p.k) + size_t(g) * p.Dp;
-  const __nv_bfloat16* vg = static_cast<const __nv_bfloat16*>(p.v) + size_t(h) * p.Vp + vb;
-  const float* zg = p.z + size_t(h) * p.Dp;
-  float* factors = reinterpret_cast<float*>(sm + S::oF);
+struct Job {                        // what one CTA works on, and where a thread stands in its group
+  int h, g, first, n, nc, slot, vb;
+  int tid, warp, lane, row16, l16;  // 16 lanes per row of a chunk
+};
 
-  // rows of chunk c on their way to shared memory, 16 lanes per row; missing rows of v are zeros, the others' are left out when they are used
-  const int row16 = tid >> 4, l16 = tid & 15;
+// ---- the makers -----------------------------------------------------------------------------------------------------------
+template <int DK>
+__device__ __forceinline__ void make_operands(const Params& p, uint8_t* sm, const Job& w) {
+  using S = Shape<DK>;
+  const int tid = w.tid, warp = w.warp, lane = w.lane, r8 = lane >> 2, quad = lane & 3, row16 = w.row16, l16 = w.l16, n = w.n;
+  const uint32_t base = smem_addr(sm);
+  const float rate = p.rate[w.h], qscale = rsqrtf(float(p.dim));
+  const __nv_bfloat16* qg = static_cast<const __nv_bfloat16*>(p.q) + size_t(w.g) * p.Dp;
+  const __nv_bfloat16* kg = static_cast<const __nv_bfloat16*>(p.k) + size_t(w.g) * p.Dp;
+  const __nv_bfloat16* vg = static_cast<const __nv_bfloat16*>(p.v) + size_t(w.h) * p.Vp + w.vb;
+  const float* zg = p.z + size_t(w.h) * p.Dp;
+
+  // rows of chunk c on their way to shared memory (missing rows: whatever the buffer holds, left out when they are used)
   auto issue = [&](int c) {
-    const int at = c * kC, nt = min(kC, n - at), vch = min(kCols, p.Vp - vb) / 8;
-    const size_t r = size_t(first + at + row16);
-    if (row16 < nt) {
-      for (int x = l16; x < p.Dp / 4; x += 16) cp_async16(base + S::oZ + (row16 * DK + x * 4) * 4, zg + r * p.ldz + x * 4);
-      for (int x = l16; x < p.Dp / 8; x += 16) {
-        cp_async16(base + S::oRq + (row16 * DK + x * 8) * 2, qg + r * p.ld + x * 8);
-        cp_async16(base + S::oRk + (row16 * DK + x * 8) * 2, kg + r * p.ld + x * 8);
-      }
+    const size_t r = size_t(w.first + c * kC + row16);
+    if (c * kC + row16 >= n) return;
+    for (int x = l16; x < p.Dp / 4; x += 16) cp_async16(base + S::oZ + (row16 * DK + x * 4) * 4, zg + r * p.ldz + x * 4);
+    for (int x = l16; x < p.Dp / 8; x += 16) {
+      cp_async16(base + S::oRq + (row16 * DK + x * 8) * 2, qg + r * p.ld + x * 8);
+      cp_async16(base + S::oRk + (row16 * DK + x * 8) * 2, kg + r * p.ld + x * 8);
     }
-    const uint32_t vbuf = base + S::oV + ((c & 1) * kC + row16) * S::kVPitch;
-    if (l16 < vch) {
-      if (row16 < nt) cp_async16(vbuf + l16 * 16, vg + r * p.ld + l16 * 8);
-      else st_zero16(vbuf + l16 * 16);
-    }
+  };
+  auto issue_v = [&](int c, uint32_t set) {                         // missing rows are zeros
+    const uint32_t dst = set + S::oV + row16 * S::kVPitch + l16 * 16;
+    if (l16 >= min(kCols, p.Vp - w.vb) / 8) return;
+    if (c * kC + row16 < n) cp_async16(dst, vg + size_t(w.first + c * kC + row16) * p.ld + l16 * 8);
+    else st_zero16(dst);
   };
   __nv_bfloat16 beta_next = __float2bfloat16_rn(0.f);               // step size of row `tid` of the chunk on its way
   auto fetch_beta = [&](int c) {
-    if (tid < kC && c * kC + tid < n) beta_next = static_cast<const __nv_bfloat16*>(p.beta)[size_t(first + c * kC + tid) * p.ldx + h];
+    if (tid < kC && c * kC + tid < n) beta_next = static_cast<const __nv_bfloat16*>(p.beta)[size_t(w.first + c * kC + tid) * p.ldx + w.h];
   };
-  // factors that make rows of q and k unit vectors (missing rows: whatever the buffer holds, never used), step sizes
-  auto norms = [&]() {
+  // factors that make rows of q and k unit vectors, step sizes
+  auto norms = [&](float* factors) {
     float sq = 0.f, sk = 0.f;
     for (int x = l16; x < p.Dp / 8; x += 16) {
       float f[8], k[8];
@@ -166,9 +169,8 @@ __global__ void __launch_bounds__(kNT, 2) k_delta_chunk(const Params p, const in
     }
     if (tid < kC) factors[2 * kC + tid] = vec::sigmoid<__nv_bfloat16>(__bfloat162float(beta_next));
   };
-
   // operands of a chunk of nt rows: a warp takes 16 channels, a lane two of them over four tokens (a quarter of the chunk)
-  auto prepare = [&](int nt) {
+  auto prepare = [&](int nt, uint32_t set, uint8_t* set_p, const float* factors) {
     if (warp * 16 >= p.Dp) return;
     const int quarter = lane >> 3, d = warp * 16 + (lane & 7) * 2;
     f32x2 a[4], q[4], k[4];
@@ -184,15 +186,15 @@ __global__ void __launch_bounds__(kNT, 2) k_delta_chunk(const Params p, const in
       q[j] = ok ? pack2(__uint_as_float(qr << 16) * fq, __uint_as_float(qr & 0xffff0000u) * fq) : 0ull;
       k[j] = ok ? pack2(__uint_as_float(kr << 16) * fk, __uint_as_float(kr & 0xffff0000u) * fk) : 0ull;
     }
-    // products over quarters: t1, t2, t3 of the lanes' neighbours (quarter ^ 1, 2, 3)
+    // products over quarters: t1 of quarter ^ 1, t23 of the two others
     const f32x2 tot = mul2(mul2(a[0], a[1]), mul2(a[2], a[3]));
     const f32x2 t1 = __shfl_xor_sync(0xffffffffu, tot, 8), both = mul2(tot, t1), t23 = __shfl_xor_sync(0xffffffffu, both, 16), one = pack2(1.f, 1.f);
     const bool odd = quarter & 1, late = quarter & 2;
     const f32x2 before = mul2(odd ? t1 : one, late ? t23 : one), after = mul2(odd ? one : t1, late ? one : t23);
     const f32x2 half = odd == late ? t1 : one;                      // to (quarters 0, 1) and from (2, 3) the middle of the chunk: over quarter 1, over quarter 2
-    if (quarter == 0) *reinterpret_cast<float2*>(sm + S::oE + d * 4) = of2(mul2(both, t23));
+    if (quarter == 0) *reinterpret_cast<float2*>(set_p + S::oE + d * 4) = of2(mul2(both, t23));
     constexpr uint32_t kp = kC * S::kPitch, ka = 32 * S::kPitch, kb = 16 * S::kPitch;
-    const uint32_t col = d * 2, own = base + quarter * 4 * S::kPitch + col;
+    const uint32_t col = d * 2, own = set + quarter * 4 * S::kPitch + col;
     f32x2 kc[4], run = one;
 #pragma unroll
     for (int j = 3; j >= 0; j--) {                                  // k times the decays behind it, in its quarter
@@ -227,49 +229,53 @@ __global__ void __launch_bounds__(kNT, 2) k_delta_chunk(const Params p, const in
         const float2 v = of2(mul2(q[t], k[s]));
         val[t * (t + 1) / 2 + s] = v.x + v.y;
         if (s < t) {
-          const float2 w = of2(mul2(k[t], k[s]));
-          val[10 + t * (t - 1) / 2 + s] = w.x + w.y;
+          const float2 x = of2(mul2(k[t], k[s]));
+          val[10 + t * (t - 1) / 2 + s] = x.x + x.y;
         }
       }
     }
     int idx = 0;
 #pragma unroll
-    for (int w = 8; w >= 2; w >>= 1) {
-      const int off = w / 2;
+    for (int c = 8; c >= 2; c >>= 1) {
+      const int off = c / 2;
       const bool up = lane & off;
 #pragma unroll
       for (int j = 0; j < 8; j++)
-        if (j < w) {
-          const float send = up ? val[j] : val[j + w], keep = up ? val[j + w] : val[j];
+        if (j < c) {
+          const float send = up ? val[j] : val[j + c], keep = up ? val[j + c] : val[j];
           val[j] = keep + __shfl_xor_sync(0xffffffffu, send, off);
         }
-      idx += up ? w : 0;
+      idx += up ? c : 0;
     }
     *reinterpret_cast<float2*>(sm + S::oTri + ((warp * 4 + quarter) * 16 + idx) * 4) = make_float2(val[0], val[1]);
   };
   // the blocks between quarters and halves: left rows against right rows, k steps shared out over the warps
   auto blocks = [&]() {
     if (warp * 16 >= p.Dp) return;
+    float acc[2][4] = {};
+    uint32_t a[2][kParts][4], b[2][kParts][2];
 #pragma unroll
-    for (int kind = 0; kind < 2; kind++) {
-      float acc[4] = {0.f, 0.f, 0.f, 0.f};
-      uint32_t a[kParts][4], b[kParts][2];
+    for (int kind = 0; kind < 2; kind++)
 #pragma unroll
       for (int i = 0; i < kParts; i++) {
-        ldmatrix_x4(base + S::oTa + (i * 32 + kind * 16 + (lane & 15)) * S::kPitch + warp * 32 + (lane >> 4) * 16, a[i]);
-        ldmatrix_x2(base + S::oTb + (i * 16 + kind * 8 + (lane & 7)) * S::kPitch + warp * 32 + ((lane >> 3) & 1) * 16, b[i]);
+        ldmatrix_x4(base + S::oTa + (i * 32 + kind * 16 + (lane & 15)) * S::kPitch + warp * 32 + (lane >> 4) * 16, a[kind][i]);
+        ldmatrix_x2(base + S::oTb + (i * 16 + kind * 8 + (lane & 7)) * S::kPitch + warp * 32 + ((lane >> 3) & 1) * 16, b[kind][i]);
       }
 #pragma unroll
-      for (int i = kParts - 1; i >= 0; i--)
+    for (int i = kParts - 1; i >= 0; i--)
 #pragma unroll
-        for (int j = kParts - 1 - i; j >= 0; j--) mma_bf16(acc, a[i], b[j][0], b[j][1]);
-      float* off = reinterpret_cast<float*>(sm + S::oO) + (warp * 2 + kind) * 128;
-      *reinterpret_cast<float2*>(off + r8 * 8 + quad * 2) = make_float2(acc[0], acc[1]);
-      *reinterpret_cast<float2*>(off + (r8 + 8) * 8 + quad * 2) = make_float2(acc[2], acc[3]);
+      for (int j = kParts - 1 - i; j >= 0; j--)
+#pragma unroll
+        for (int kind = 0; kind < 2; kind++) mma_bf16(acc[kind], a[kind][i], b[kind][j][0], b[kind][j][1]);
+#pragma unroll
+    for (int kind = 0; kind < 2; kind++) {
+      float* off = reinterpret_cast<float*>(sm + S::oOff) + (warp * 2 + kind) * 128;
+      *reinterpret_cast<float2*>(off + r8 * 8 + quad * 2) = make_float2(acc[kind][0], acc[kind][1]);
+      *reinterpret_cast<float2*>(off + (r8 + 8) * 8 + quad * 2) = make_float2(acc[kind][2], acc[kind][3]);
     }
   };
   // A and diag(beta) B from their pieces, an element per thread
-  auto assemble = [&]() {
+  auto assemble = [&](uint8_t* set_p, const float* factors) {
     const int t = tid >> 4, s = tid & 15, qt = t >> 2, qs = s >> 2, items = p.Dp / 16;
     float vq = 0.f, vk = 0.f;
     if (s <= t) {
@@ -278,25 +284,27 @@ __global__ void __launch_bounds__(kNT, 2) k_delta_chunk(const Params p, const in
       if (qt == qs) {
         const int tt = t & 3, ss = s & 3;
         at = reinterpret_cast<const float*>(sm + S::oTri) + qt * 16 + tt * (tt + 1) / 2 + ss;
-        ak = reinterpret_cast<const float*>(sm + S::oTri) + qt * 16 + 10 + max(0, tt * (tt - 1) / 2 + ss);
+        ak = reinterpret_cast<const float*>(sm + S::oTri) + qt * 16 + 10 + tt * (tt - 1) / 2 + ss;     // (s = t: not used)
         step = 64;
       } else {
         const bool far = (qt ^ qs) & 2;
-        at = reinterpret_cast<const float*>(sm + S::oO) + (far ? 128 + (t - 8) * 8 + s : ((qt >> 1) * 4 + (t & 3)) * 8 + (qs >> 1) * 4 + (s & 3));
+        at = reinterpret_cast<const float*>(sm + S::oOff) + (far ? 128 + (t - 8) * 8 + s : ((qt >> 1) * 4 + (t & 3)) * 8 + (qs >> 1) * 4 + (s & 3));
         ak = at + 64;
         step = 256;
       }
-      for (int w = 0; w < items; w++) { vq += at[w * step]; vk += ak[w * step]; }
+#pragma unroll
+      for (int i = 0; i < S::kItems; i++)
+        if (i < items) { vq += at[i * step]; vk += ak[i * step]; }
     }
     const __nv_bfloat16 hi = __float2bfloat16_rn(vq);
-    reinterpret_cast<__nv_bfloat16*>(sm + S::oA + t * S::kAPitch)[s] = hi;
-    reinterpret_cast<__nv_bfloat16*>(sm + S::oA + (kC + t) * S::kAPitch)[s] = __float2bfloat16_rn(vq - __bfloat162float(hi));
+    reinterpret_cast<__nv_bfloat16*>(set_p + S::oA + t * S::kAPitch)[s] = hi;
+    reinterpret_cast<__nv_bfloat16*>(set_p + S::oA + (kC + t) * S::kAPitch)[s] = __float2bfloat16_rn(vq - __bfloat162float(hi));
     reinterpret_cast<float*>(sm + S::oL)[t * 17 + s] = s < t ? vk * factors[2 * kC + t] : 0.f;
   };
   // T, by one warp
-  auto invert = [&]() {
+  auto invert = [&](uint32_t set, const float* beta) {
     const float* L = reinterpret_cast<const float*>(sm + S::oL);
-    float *I = reinterpret_cast<float*>(sm + S::oTri), *M = I + 16 * 17;
+    float *I = reinterpret_cast<float*>(sm + S::oL) + 16 * 17, *M = I + 16 * 17;
     const int b8 = lane & 8, j = lane & 7;                          // lanes 16 .. 31 repeat the others
     float x[8];
 #pragma unroll
@@ -330,20 +338,174 @@ __global__ void __launch_bounds__(kNT, 2) k_delta_chunk(const Params p, const in
       m1 = fmaf(-l, M[s * 17 + c + 1], m1);
     }
     // rows r8 and 8 + r8, columns c, c + 1 of both halves
-    const float* beta = factors + 2 * kC;
     auto out = [&](int t, int s, float v0, float v1) {
       uint32_t part[kParts];
       split<kParts>(v0 * beta[s], v1 * beta[s + 1], part);
 #pragma unroll
-      for (int i = 0; i < kParts; i++) st_shared(base + S::oT + (i * kC + t) * S::kAPitch + s * 2, part[i]);
+      for (int i = 0; i < kParts; i++) st_shared(set + S::oT + (i * kC + t) * S::kAPitch + s * 2, part[i]);
     };
     out(r8, c, I[r8 * 17 + c], I[r8 * 17 + c + 1]);
     out(r8, 8 + c, 0.f, 0.f);
     out(8 + r8, c, m0, m1);
     out(8 + r8, 8 + c, I[(8 + r8) * 17 + 8 + c], I[(8 + r8) * 17 + 8 + c + 1]);
   };
-  // head norm, weight and gate of chunk c, whose o lies in shared memory; a row per 16 lanes, 8 columns per lane
-  auto emit = [&](int c, const vec::Raw8<__nv_bfloat16>& gate) {
+
+  issue(0);
+  cp_async_commit();
+  fetch_beta(0);
+  for (int i = tid; i < S::oZ / 16; i += kNT) st_zero16(base + i * 16);     // operand rows of channels beyond Dp stay zero
+  for (int c = 0; c < w.nc; c++) {
+    const int b = c & 1;
+    uint8_t* set_p = sm + b * S::kSet;
+    const uint32_t set = base + b * S::kSet;
+    float* factors = reinterpret_cast<float*>(sm + S::oF) + b * 3 * kC;   // two of them: one warp may still be at the chunk before
+    cp_async_wait<0>();
+    norms(factors);                                                 // of rows that this thread's own copies brought
+    bar_sync(kMakers, kNT);                                         // all raw rows of chunk c are there
+    if (c >= 2) bar_sync(kEmpty + b, 2 * kNT);                      // the products of chunk c - 2 are done
+    issue_v(c, set);
+    cp_async_commit();
+    prepare(min(kC, n - c * kC), set, set_p, factors);
+    bar_sync(kMakers, kNT);
+    if (c + 1 < w.nc) {
+      issue(c + 1);
+      fetch_beta(c + 1);
+    }
+    cp_async_commit();
+    blocks();
+    bar_sync(kMakers, kNT);
+    assemble(set_p, factors);
+    bar_sync(kMakers, kNT);
+    if (warp == 0) invert(set, factors + 2 * kC);
+    cp_async_wait<1>();                                             // v
+    bar_arrive(kFull + b, 2 * kNT);
+  }
+  cp_async_wait<0>();
+}
+
+// ---- the products -----------------------------------------------------------------------------------------------------------
+template <int DK>
+__device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job& w) {
+  using S = Shape<DK>;
+  const int lane = w.lane, r8 = lane >> 2, quad = lane & 3, row16 = w.row16, l16 = w.l16, n = w.n;
+  const uint32_t base = smem_addr(sm);
+  const bool fresh = p.positions[w.first] == 0, fused = p.o == nullptr;
+  const int v0 = w.vb + w.warp * 16;                                // first value column of the warp
+  const bool mma_warp = v0 < p.Vp;
+  float st[DK / 8][4];      // S^T: value column v0 + r8 (+ 8), channels 8 i + 2 quad (+ 1)
+  float* state = p.state + (size_t(w.slot) * p.heads + w.h) * p.Dp * p.Vp;
+#pragma unroll
+  for (int i = 0; i < DK / 8; i++)
+#pragma unroll
+    for (int j = 0; j < 4; j++) {
+      const int d = i * 8 + quad * 2 + (j & 1), v = v0 + r8 + (j >> 1) * 8;
+      st[i][j] = !mma_warp || fresh || d >= p.Dp ? 0.f : state[size_t(d) * p.Vp + v];
+    }
+  const uint32_t brow = (lane & 7) + ((lane >> 4) << 3), bcol = ((lane >> 3) & 1) * 16;    // right operands stored [n][k]
+  for (int c = 0; c < w.nc; c++) {
+    const int b = c & 1, at = c * kC;
+    const uint32_t set = base + b * S::kSet;
+    vec::Raw8<__nv_bfloat16> gate;
+    if (fused && at + row16 < n && l16 * 8 < p.Vp)
+      gate.load(static_cast<const __nv_bfloat16*>(p.gate) + size_t(w.first + at + row16) * p.ldg + size_t(w.h) * p.Vp + l16 * 8);
+    bar_sync(kFull + b, 2 * kNT);
+    if (mma_warp) {
+      // (q P) S and (k P) S, two sums each for even and odd k steps: value column as above, tokens 8 i + 2 quad (+ 1)
+      float o[2][2][4] = {}, x[2][2][4] = {};
+#pragma unroll
+      for (int ks = 0; ks < DK / 16; ks += 2) {
+        uint32_t s[2][kParts][4], f[2][4];
+        as_left<kParts>(st + 2 * ks, s[0]);
+        as_left<kParts>(st + 2 * ks + 2, s[1]);
+#pragma unroll
+        for (int j = kParts - 1; j >= 0; j--) {
+#pragma unroll
+          for (int e = 0; e < 2; e++) ldmatrix_x4(set + S::oK + (j * kC + brow) * S::kPitch + bcol + (ks + e) * 32, f[e]);
+#pragma unroll
+          for (int i = kParts - 1 - j; i >= 0; i--)
+#pragma unroll
+            for (int e = 0; e < 2; e++) {
+              mma_bf16(x[e][0], s[e][i], f[e][0], f[e][1]);
+              mma_bf16(x[e][1], s[e][i], f[e][2], f[e][3]);
+            }
+        }
+#pragma unroll
+        for (int j = 1; j >= 0; j--) {
+#pragma unroll
+          for (int e = 0; e < 2; e++) ldmatrix_x4(set + S::oQ + (j * kC + brow) * S::kPitch + bcol + (ks + e) * 32, f[e]);
+#pragma unroll
+          for (int i = 1 - j; i >= 0; i--)
+#pragma unroll
+            for (int e = 0; e < 2; e++) {
+              mma_bf16(o[e][0], s[e][i], f[e][0], f[e][1]);
+              mma_bf16(o[e][1], s[e][i], f[e][2], f[e][3]);
+            }
+        }
+      }
+      uint32_t l[kParts][4], f[4];
+      ldmatrix_x4_trans(set + S::oV + brow * S::kVPitch + w.warp * 32 + bcol, f);      // v^T: stored [token][column]
+#pragma unroll
+      for (int j = 0; j < 4; j++) {
+        float* y = &x[0][j >> 1][(j & 1) * 2];
+        const float* z = &x[1][j >> 1][(j & 1) * 2];
+        y[0] = __uint_as_float(f[j] << 16) - (y[0] + z[0]);
+        y[1] = __uint_as_float(f[j] & 0xffff0000u) - (y[1] + z[1]);
+      }
+      float u[2][4] = {};
+      as_left<kParts>(x[0], l);
+#pragma unroll
+      for (int j = kParts - 1; j >= 0; j--) {
+        ldmatrix_x4(set + S::oT + (j * kC + brow) * S::kAPitch + bcol, f);
+#pragma unroll
+        for (int i = kParts - 1 - j; i >= 0; i--) {
+          mma_bf16(u[0], l[i], f[0], f[1]);
+          mma_bf16(u[1], l[i], f[2], f[3]);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < DK / 8; i++) {
+        const float2 e = *reinterpret_cast<const float2*>(sm + b * S::kSet + S::oE + (i * 8 + quad * 2) * 4);
+        st[i][0] *= e.x; st[i][1] *= e.y; st[i][2] *= e.x; st[i][3] *= e.y;
+      }
+      as_left<kParts>(u, l);
+#pragma unroll
+      for (int j = 1; j >= 0; j--) {
+        ldmatrix_x4(set + S::oA + (j * kC + brow) * S::kAPitch + bcol, f);
+#pragma unroll
+        for (int i = 1 - j; i >= 0; i--) {
+          mma_bf16(o[i][0], l[i], f[0], f[1]);
+          mma_bf16(o[i][1], l[i], f[2], f[3]);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < DK / 16; i += 2)
+#pragma unroll
+        for (int j = kParts - 1; j >= 0; j--) {                     // smallest part first
+          uint32_t r[2][4];
+#pragma unroll
+          for (int e = 0; e < 2; e++) ldmatrix_x4_trans(set + S::oR + (j * kC + (lane & 15)) * S::kPitch + (i + e) * 32 + (lane >> 4) * 16, r[e]);
+#pragma unroll
+          for (int y = kParts - 1 - j; y >= 0; y--)
+#pragma unroll
+            for (int e = 0; e < 2; e++) {
+              mma_bf16(st[2 * (i + e)], l[y], r[e][0], r[e][1]);
+              mma_bf16(st[2 * (i + e) + 1], l[y], r[e][2], r[e][3]);
+            }
+        }
+#pragma unroll
+      for (int i = 0; i < 2; i++)
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+          const int t = i * 8 + quad * 2 + (j & 1), v = r8 + (j >> 1) * 8;
+          const float y = o[0][i][j] + o[1][i][j];
+          if (fused) reinterpret_cast<float*>(sm + S::oO)[t * S::kOPitch + w.warp * 16 + v] = y;
+          else if (at + t < n) p.o[(size_t(w.first + at + t) * p.heads + w.h) * p.Vp + v0 + v] = y;
+        }
+    }
+    if (c + 2 < w.nc) bar_arrive(kEmpty + b, 2 * kNT);
+    if (!fused) continue;
+    // head norm, weight and gate; a row per 16 lanes, 8 columns per lane.  (The next chunk's o is written behind its `full`, which waits for all of these warps.)
+    bar_sync(kProducts, kNT);
     const int v = l16 * 8;
     float f[8], ss = 0.f;
     vec::load8(reinterpret_cast<const float*>(sm + S::oO) + row16 * S::kOPitch + v, f);
@@ -355,145 +517,15 @@ __global__ void __launch_bounds__(kNT, 2) k_delta_chunk(const Params p, const in
     for (int e = 0; e < 8; e++) ss = fmaf(f[e], f[e], ss);
 #pragma unroll
     for (int o = 8; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-    if (c * kC + row16 < n && v < p.Vp) {
+    if (at + row16 < n && v < p.Vp) {
       const float r = 1.0f / sqrtf(ss / float(p.vdim) + p.eps);
-      float gt[8], w[8];
+      float gt[8], wt[8];
       gate.unpack(gt);
-      vec::load8(p.norm + v, w);
+      vec::load8(p.norm + v, wt);
 #pragma unroll
-      for (int e = 0; e < 8; e++) f[e] = f[e] * r * w[e] * vec::sigmoid<__nv_bfloat16>(gt[e]);
-      vec::store8(static_cast<__nv_bfloat16*>(p.out) + size_t(first + c * kC + row16) * p.ldo + size_t(h) * p.Vp + v, f);
+      for (int e = 0; e < 8; e++) f[e] = f[e] * r * wt[e] * vec::sigmoid<__nv_bfloat16>(gt[e]);
+      vec::store8(static_cast<__nv_bfloat16*>(p.out) + size_t(w.first + at + row16) * p.ldo + size_t(w.h) * p.Vp + v, f);
     }
-  };
-
-  float st[DK / 8][4];      // S^T: value column v0 + r8 (+ 8), channels 8 i + 2 quad (+ 1)
-  float* state = p.state + (size_t(slot) * p.heads + h) * p.Dp * p.Vp;
-#pragma unroll
-  for (int i = 0; i < DK / 8; i++)
-#pragma unroll
-    for (int j = 0; j < 4; j++) {
-      const int d = i * 8 + quad * 2 + (j & 1), v = v0 + r8 + (j >> 1) * 8;
-      st[i][j] = !mma_warp || fresh || d >= p.Dp ? 0.f : state[size_t(d) * p.Vp + v];
-    }
-  // operand rows of channels beyond Dp stay zero
-  for (int i = tid; i < (S::oV - S::oQ) / 16; i += kNT) st_zero16(base + S::oQ + i * 16);
-  for (int i = tid; i < DK; i += kNT) reinterpret_cast<float*>(sm + S::oE)[i] = 0.f;
-
-  const uint32_t brow = (lane & 7) + ((lane >> 4) << 3), bcol = ((lane >> 3) & 1) * 16;    // right operands stored [n][k]
-  const int nc = (n + kC - 1) / kC;
-  issue(0);
-  cp_async_commit();
-  fetch_beta(0);
-  cp_async_wait<0>();
-  __syncthreads();
-  norms();
-  __syncthreads();
-  for (int c = 0; c < nc; c++) {
-    // the raw rows of chunk c are there, its factors too
-    prepare(min(kC, n - c * kC));
-    __syncthreads();
-    if (c + 1 < nc) {
-      issue(c + 1);
-      fetch_beta(c + 1);
-    }
-    cp_async_commit();
-    blocks();
-    __syncthreads();
-    assemble();
-    vec::Raw8<__nv_bfloat16> gate;
-    if (fused && c * kC + row16 < n && l16 * 8 < p.Vp)
-      gate.load(static_cast<const __nv_bfloat16*>(p.gate) + size_t(first + c * kC + row16) * p.ldg + size_t(h) * p.Vp + l16 * 8);
-    __syncthreads();
-    if (warp == 0) invert();
-    float o[2][4] = {}, w[2][4] = {};                               // (q P) S and (k P) S: value column as above, tokens 8 i + 2 quad (+ 1)
-    if (mma_warp) {
-#pragma unroll
-      for (int ks = 0; ks < DK / 16; ks++) {
-        uint32_t s[kParts][4], b[4];
-        as_left<kParts>(st + 2 * ks, s);
-#pragma unroll
-        for (int j = kParts - 1; j >= 0; j--) {
-          ldmatrix_x4(base + S::oK + (j * kC + brow) * S::kPitch + bcol + ks * 32, b);
-#pragma unroll
-          for (int i = kParts - 1 - j; i >= 0; i--) {
-            mma_bf16(w[0], s[i], b[0], b[1]);
-            mma_bf16(w[1], s[i], b[2], b[3]);
-          }
-        }
-#pragma unroll
-        for (int j = 1; j >= 0; j--) {
-          ldmatrix_x4(base + S::oQ + (j * kC + brow) * S::kPitch + bcol + ks * 32, b);
-#pragma unroll
-          for (int i = 1 - j; i >= 0; i--) {
-            mma_bf16(o[0], s[i], b[0], b[1]);
-            mma_bf16(o[1], s[i], b[2], b[3]);
-          }
-        }
-      }
-      uint32_t vf[4];                                               // v^T: stored [token][column]
-      ldmatrix_x4_trans(base + S::oV + (c & 1) * kC * S::kVPitch + brow * S::kVPitch + warp * 32 + bcol, vf);
-#pragma unroll
-      for (int j = 0; j < 4; j++) {
-        float* x = &w[j >> 1][(j & 1) * 2];
-        x[0] = __uint_as_float(vf[j] << 16) - x[0];
-        x[1] = __uint_as_float(vf[j] & 0xffff0000u) - x[1];
-      }
-    }
-    __syncthreads();                                                // T is there
-    if (mma_warp) {
-      float u[2][4] = {};
-      uint32_t l[kParts][4], b[4];
-      as_left<kParts>(w, l);
-#pragma unroll
-      for (int j = kParts - 1; j >= 0; j--) {
-        ldmatrix_x4(base + S::oT + (j * kC + brow) * S::kAPitch + bcol, b);
-#pragma unroll
-        for (int i = kParts - 1 - j; i >= 0; i--) {
-          mma_bf16(u[0], l[i], b[0], b[1]);
-          mma_bf16(u[1], l[i], b[2], b[3]);
-        }
-      }
-      as_left<kParts>(u, l);
-#pragma unroll
-      for (int j = 1; j >= 0; j--) {
-        ldmatrix_x4(base + S::oA + (j * kC + brow) * S::kAPitch + bcol, b);
-#pragma unroll
-        for (int i = 1 - j; i >= 0; i--) {
-          mma_bf16(o[0], l[i], b[0], b[1]);
-          mma_bf16(o[1], l[i], b[2], b[3]);
-        }
-      }
-      const int at = c * kC;
-#pragma unroll
-      for (int i = 0; i < 2; i++)
-#pragma unroll
-        for (int j = 0; j < 4; j++) {
-          const int t = i * 8 + quad * 2 + (j & 1), v = r8 + (j >> 1) * 8;
-          if (fused) reinterpret_cast<float*>(sm + S::oO)[t * S::kOPitch + warp * 16 + v] = o[i][j];
-          else if (at + t < n) p.o[(size_t(first + at + t) * p.heads + h) * p.Vp + v0 + v] = o[i][j];
-        }
-#pragma unroll
-      for (int i = 0; i < DK / 8; i++) {
-        const float2 e = *reinterpret_cast<const float2*>(sm + S::oE + (i * 8 + quad * 2) * 4);
-        st[i][0] *= e.x; st[i][1] *= e.y; st[i][2] *= e.x; st[i][3] *= e.y;
-      }
-#pragma unroll
-      for (int i = 0; i < DK / 16; i++)
-#pragma unroll
-        for (int j = kParts - 1; j >= 0; j--) {                     // smallest part first
-          ldmatrix_x4_trans(base + S::oR + (j * kC + (lane & 15)) * S::kPitch + i * 32 + (lane >> 4) * 16, b);
-#pragma unroll
-          for (int x = kParts - 1 - j; x >= 0; x--) {
-            mma_bf16(st[2 * i], l[x], b[0], b[1]);
-            mma_bf16(st[2 * i + 1], l[x], b[2], b[3]);
-          }
-        }
-    }
-    cp_async_wait<0>();
-    __syncthreads();
-    if (fused) emit(c, gate);
-    if (c + 1 < nc) norms();
-    __syncthreads();
   }
   if (mma_warp) {
 #pragma unroll
@@ -507,12 +539,40 @@ __global__ void __launch_bounds__(kNT, 2) k_delta_chunk(const Params p, const in
 }
 
 template <int DK>
+__global__ void __launch_bounds__(2 * kNT, 1) k_delta_chunk(const Params p, const int* groups) {
+  extern __shared__ __align__(16) uint8_t sm[];
+  pdl::launch_dependents();
+  pdl::grid_dependency_wait();
+  Job w;
+  w.h = blockIdx.y;
+  w.g = w.h / (p.heads / p.kv_heads);
+  w.first = groups[4 * blockIdx.x];
+  w.n = groups[4 * blockIdx.x + 1];
+  w.slot = groups[4 * blockIdx.x + 2];
+  w.nc = (w.n + kC - 1) / kC;
+  w.vb = blockIdx.z * kCols;
+  w.tid = threadIdx.x % kNT;
+  w.warp = w.tid >> 5;
+  w.lane = w.tid & 31;
+  w.row16 = w.tid >> 4;
+  w.l16 = w.tid & 15;
+  // registers of the launch, 128 per thread, shared out anew
+  if (threadIdx.x < kNT) {
+    asm volatile("setmaxnreg.inc.sync.aligned.u32 152;");
+    multiply<DK>(p, sm, w);
+  } else {
+    asm volatile("setmaxnreg.dec.sync.aligned.u32 104;");
+    make_operands<DK>(p, sm, w);
+  }
+}
+
+template <int DK>
 cudaError_t launch(Params p, const int* groups, int ngroups, bool* finished, cudaStream_t st) {
   static bool done = false;
   *finished = p.Vp <= kCols;
   if (*finished) p.o = nullptr;
   cudaError_t e = allow_smem(k_delta_chunk<DK>, Shape<DK>::kBytes, &done);
-  return e != cudaSuccess ? e : pdl::launch(k_delta_chunk<DK>, dim3(ngroups, p.heads, (p.Vp + kCols - 1) / kCols), dim3(kNT), Shape<DK>::kBytes, st, 1, p, groups);
+  return e != cudaSuccess ? e : pdl::launch(k_delta_chunk<DK>, dim3(ngroups, p.heads, (p.Vp + kCols - 1) / kCols), dim3(2 * kNT), Shape<DK>::kBytes, st, 1, p, groups);
 }
 
 }  // namespace

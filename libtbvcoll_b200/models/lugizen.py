@@ -84,7 +84,7 @@ class Lugizen(StreamDecoder, LatentAttention):
                 self.cache.append(zeros(num_blocks * m.kv_heads * block_size, ops.latent_row(pad16(m.dim), pad16(m.vdim))))
         self.expands_context = bool(self.latents)
         self.context_window = max(m.window for m in self.latents) if self.latents and all(m.window for m in self.latents) else 0
-        self.attn_ctas_per_row = max([m.kv_heads * ((m.heads // m.kv_heads + 15) // 16) for m in attns] + [(m.heads + 15) // 16 for m in self.latents], default=1)
+        self.attn_ctas_per_row = 0                             # the engine's choice follows the context alone; layer_splits knows each layer's CTAs
         self.scan_heads = min([m.heads for _, m in deltas], default=0)
         two_forms = bool(attns or self.latents) and dtype is torch.bfloat16 and all(ops.paired_prefill_fits(pad16(m.dim), pad16(m.vdim)) for m in attns) \
             and all(ops.latent_prefill_fits(pad16(m.dim), pad16(m.rot_dim), pad16(m.vdim)) for m in self.latents)
@@ -103,10 +103,12 @@ class Lugizen(StreamDecoder, LatentAttention):
             return 0
         return -(-int(rows.max()) // self.SCAN_CHUNK) * self.SCAN_CHUNK
 
-    def latent_splits(self, m: LatentSpec, rows: int, splits: int) -> int:
-        """CTAs per row of a latent layer: one CTA fits an SM, and a row that sees at most a window needs at least 64 keys for each."""
-        units = rows * ((m.heads + 15) // 16)
-        while splits > 1 and (units * splits > (self.sms if splits < 8 else self.sms * 4 // 5) or (m.window and m.window // splits < 64)):
+    def layer_splits(self, m, rows: int, splits: int) -> int:
+        """CTAs per row of an attention layer, at most ``splits``: what runs at once (an SM holds two CTAs of the kernel over paired rows, one over latents), and at
+        least 64 visible keys for each."""
+        latent = isinstance(m, LatentSpec)
+        units = rows * ((m.heads + 15) // 16 if latent else m.kv_heads * ((m.heads // m.kv_heads + 15) // 16))
+        while splits > 1 and (units * splits > self.attn_cta_slots(splits, self.sms) // (2 if latent else 1) or (latent and m.window and m.window // splits < 64)):
             splits //= 2
         return splits
 
@@ -143,7 +145,7 @@ class Lugizen(StreamDecoder, LatentAttention):
         ops.head_attention_prep(wide, qa, cache, w[p + "qscale"], self.turns[i], b.positions, b.slots, n, H, G, m.dim, D, self.block_size, self.cfg.rms_eps,
                                 v_first=self._buf("first", T, G * V) if m.v_mix else None, mix=w[p + "vmix"] if m.v_mix and i != self.first_values else None)
         if n:
-            ops.paired_attention_rows(qa, cache, b.tables, b.seq_of_row, b.ctx, out[:n].view(n, H, V), G, self.block_size, splits=b.attn_splits)
+            ops.paired_attention_rows(qa, cache, b.tables, b.seq_of_row, b.ctx, out[:n].view(n, H, V), G, self.block_size, splits=self.layer_splits(m, n, b.attn_splits))
         if n < T:
             ops.paired_attention_prefill(wide, cache, b.tables, b.seq_of_row, b.dense_tiles, out, H, G, D, self.block_size)
         return self._project(b, i, out)
@@ -159,7 +161,7 @@ class Lugizen(StreamDecoder, LatentAttention):
         prep(low, None, w[p + "dkv.norm"], (0, m.q_rank, w[p + "dq.norm"]))
         ops.linear(low[:, :Rq], w[p + "uq"], q)
         prep(None, q, None, None)
-        self._latent_attend(b, p, m, q, qa, cache, out, self.latent_splits(m, n, b.attn_splits))
+        self._latent_attend(b, p, m, q, qa, cache, out, self.layer_splits(m, n, b.attn_splits))
         return self._project(b, i, out)
 
     def _project(self, b: StepBatch, i: int, out: torch.Tensor) -> dict:
