@@ -23,6 +23,7 @@
 #include "../pdl.cuh"
 #include "attn_mma.cuh"
 #include "delta.cuh"
+#include "ops.h"
 
 using namespace attn_mma;
 using delta_ops::Params;
@@ -55,10 +56,9 @@ struct Shape {
   // dynamic shared memory: two sets, then what one of the groups has for itself
   static constexpr int oTa = 2 * kSet;                             // blocks: left rows   [parts][2 kinds][16][pitch]  (8 of q, 8 of k)
   static constexpr int oTb = oTa + kParts * 32 * kPitch;           //         right rows  [parts][2 kinds][8][pitch]
-  static constexpr int oZ = oTb + kParts * 16 * kPitch;            // raw decay inputs    [16][DK] fp32
-  static constexpr int oRq = oZ + kC * DK * 4;                     // raw q, k            [16][DK] bf16 each
-  static constexpr int oRk = oRq + kC * DK * 2;
-  static constexpr int oF = oRk + kC * DK * 2;                     // factors of q, of k, step sizes [2 chunks][3][16] fp32
+  static constexpr int oZ = oTb + kParts * 16 * kPitch;            // raw decay inputs [16][DK] fp32, q and k [16][DK] bf16 each; two chunks
+  static constexpr int kRq = kC * DK * 4, kRk = kRq + kC * DK * 2, kRaw = kRk + kC * DK * 2;
+  static constexpr int oF = oZ + 2 * kRaw;                         // factors of q, of k, step sizes [2 chunks][3][16] fp32
   static constexpr int oTri = oF + 6 * kC * 4;                     // diagonal blocks     [items][4 quarters][16] fp32
   static constexpr int oOff = oTri + (kItems + 1) * 256;           // the other blocks' sums [warps][2][16][8] fp32
   static constexpr int oL = oOff + kNW * 1024;                     // diag(beta) B [16][17] fp32, its inverse [16][17], a product [8][17]
@@ -112,7 +112,7 @@ __device__ __forceinline__ void as_left(const float (*v)[4], uint32_t (*a)[4]) {
 }
 
 struct Job {                        // what one CTA works on, and where a thread stands in its group
-  int h, g, first, n, nc, slot, vb;
+  int h, g, first, n, nc, slot, vb, cols;  // vb: first of its value columns
   int tid, warp, lane, row16, l16;  // 16 lanes per row of a chunk
 };
 
@@ -131,16 +131,17 @@ __device__ __forceinline__ void make_operands(const Params& p, uint8_t* sm, cons
   // rows of chunk c on their way to shared memory (missing rows: whatever the buffer holds, left out when they are used)
   auto issue = [&](int c) {
     const size_t r = size_t(w.first + c * kC + row16);
+    const uint32_t raw = base + S::oZ + (c & 1) * S::kRaw;
     if (c * kC + row16 >= n) return;
-    for (int x = l16; x < p.Dp / 4; x += 16) cp_async16(base + S::oZ + (row16 * DK + x * 4) * 4, zg + r * p.ldz + x * 4);
+    for (int x = l16; x < p.Dp / 4; x += 16) cp_async16(raw + (row16 * DK + x * 4) * 4, zg + r * p.ldz + x * 4);
     for (int x = l16; x < p.Dp / 8; x += 16) {
-      cp_async16(base + S::oRq + (row16 * DK + x * 8) * 2, qg + r * p.ld + x * 8);
-      cp_async16(base + S::oRk + (row16 * DK + x * 8) * 2, kg + r * p.ld + x * 8);
+      cp_async16(raw + S::kRq + (row16 * DK + x * 8) * 2, qg + r * p.ld + x * 8);
+      cp_async16(raw + S::kRk + (row16 * DK + x * 8) * 2, kg + r * p.ld + x * 8);
     }
   };
   auto issue_v = [&](int c, uint32_t set) {                         // missing rows are zeros
     const uint32_t dst = set + S::oV + row16 * S::kVPitch + l16 * 16;
-    if (l16 >= min(kCols, p.Vp - w.vb) / 8) return;
+    if (l16 >= min(w.cols, p.Vp - w.vb) / 8) return;
     if (c * kC + row16 < n) cp_async16(dst, vg + size_t(w.first + c * kC + row16) * p.ld + l16 * 8);
     else st_zero16(dst);
   };
@@ -148,13 +149,15 @@ __device__ __forceinline__ void make_operands(const Params& p, uint8_t* sm, cons
   auto fetch_beta = [&](int c) {
     if (tid < kC && c * kC + tid < n) beta_next = static_cast<const __nv_bfloat16*>(p.beta)[size_t(w.first + c * kC + tid) * p.ldx + w.h];
   };
-  // factors that make rows of q and k unit vectors, step sizes
-  auto norms = [&](float* factors) {
-    float sq = 0.f, sk = 0.f;
+  // factors that make rows of q and k unit vectors (of rows that this thread's own copies brought), step sizes
+  auto factors_of = [&](int c) { return reinterpret_cast<float*>(sm + S::oF) + (c & 1) * 3 * kC; };
+  auto norms = [&](int c) {
+    const uint8_t* raw = sm + S::oZ + (c & 1) * S::kRaw;
+    float *factors = factors_of(c), sq = 0.f, sk = 0.f;
     for (int x = l16; x < p.Dp / 8; x += 16) {
       float f[8], k[8];
-      vec::load8(reinterpret_cast<const __nv_bfloat16*>(sm + S::oRq) + row16 * DK + x * 8, f);
-      vec::load8(reinterpret_cast<const __nv_bfloat16*>(sm + S::oRk) + row16 * DK + x * 8, k);
+      vec::load8(reinterpret_cast<const __nv_bfloat16*>(raw + S::kRq) + row16 * DK + x * 8, f);
+      vec::load8(reinterpret_cast<const __nv_bfloat16*>(raw + S::kRk) + row16 * DK + x * 8, k);
 #pragma unroll
       for (int e = 0; e < 8; e++) { sq = fmaf(f[e], f[e], sq); sk = fmaf(k[e], k[e], sk); }
     }
@@ -169,54 +172,59 @@ __device__ __forceinline__ void make_operands(const Params& p, uint8_t* sm, cons
     }
     if (tid < kC) factors[2 * kC + tid] = vec::sigmoid<__nv_bfloat16>(__bfloat162float(beta_next));
   };
-  // operands of a chunk of nt rows: a warp takes 16 channels, a lane two of them over four tokens (a quarter of the chunk)
-  auto prepare = [&](int nt, uint32_t set, uint8_t* set_p, const float* factors) {
-    if (warp * 16 >= p.Dp) return;
-    const int quarter = lane >> 3, d = warp * 16 + (lane & 7) * 2;
+  // Operands of chunk c, a warp takes 16 channels, a lane two of them over four tokens (a quarter of the chunk).  First what the scores of a chunk are made of;
+  // the operands of the state's products, which need their set free, are left in registers: q and k times the decays from their quarter's start (their own
+  // included), k times those behind it in its quarter, products of the decays over the quarters before and after.
+  f32x2 qr[4], kr[4], kc[4], before = 0ull, after = 0ull, all = 0ull;
+  const int quarter = lane >> 3, d = warp * 16 + (lane & 7) * 2;
+  const bool odd = quarter & 1, late = quarter & 2, item = warp * 16 < p.Dp;
+  auto scores = [&](int c) {
+    if (!item) return;
+    const int nt = min(kC, n - c * kC);
+    const uint8_t* raw = sm + S::oZ + (c & 1) * S::kRaw;
+    const float* factors = factors_of(c);
     f32x2 a[4], q[4], k[4];
 #pragma unroll
     for (int j = 0; j < 4; j++) {
       const int t = quarter * 4 + j;
       const bool ok = t < nt;
-      const float2 z = *reinterpret_cast<const float2*>(sm + S::oZ + (t * DK + d) * 4);
-      const uint32_t qr = *reinterpret_cast<const uint32_t*>(sm + S::oRq + (t * DK + d) * 2), kr = *reinterpret_cast<const uint32_t*>(sm + S::oRk + (t * DK + d) * 2);
+      const float2 z = *reinterpret_cast<const float2*>(raw + (t * DK + d) * 4);
+      const uint32_t qb = *reinterpret_cast<const uint32_t*>(raw + S::kRq + (t * DK + d) * 2), kb = *reinterpret_cast<const uint32_t*>(raw + S::kRk + (t * DK + d) * 2);
       const float fq = factors[t], fk = factors[kC + t];
       const float a0 = delta_ops::decay<__nv_bfloat16>(z.x, rate), a1 = delta_ops::decay<__nv_bfloat16>(z.y, rate);
       a[j] = ok ? pack2(a0, a1) : pack2(1.f, 1.f);
-      q[j] = ok ? pack2(__uint_as_float(qr << 16) * fq, __uint_as_float(qr & 0xffff0000u) * fq) : 0ull;
-      k[j] = ok ? pack2(__uint_as_float(kr << 16) * fk, __uint_as_float(kr & 0xffff0000u) * fk) : 0ull;
+      q[j] = ok ? pack2(__uint_as_float(qb << 16) * fq, __uint_as_float(qb & 0xffff0000u) * fq) : 0ull;
+      k[j] = ok ? pack2(__uint_as_float(kb << 16) * fk, __uint_as_float(kb & 0xffff0000u) * fk) : 0ull;
     }
     // products over quarters: t1 of quarter ^ 1, t23 of the two others
     const f32x2 tot = mul2(mul2(a[0], a[1]), mul2(a[2], a[3]));
     const f32x2 t1 = __shfl_xor_sync(0xffffffffu, tot, 8), both = mul2(tot, t1), t23 = __shfl_xor_sync(0xffffffffu, both, 16), one = pack2(1.f, 1.f);
-    const bool odd = quarter & 1, late = quarter & 2;
-    const f32x2 before = mul2(odd ? t1 : one, late ? t23 : one), after = mul2(odd ? one : t1, late ? one : t23);
+    before = mul2(odd ? t1 : one, late ? t23 : one);
+    after = mul2(odd ? one : t1, late ? one : t23);
+    all = mul2(both, t23);
     const f32x2 half = odd == late ? t1 : one;                      // to (quarters 0, 1) and from (2, 3) the middle of the chunk: over quarter 1, over quarter 2
-    if (quarter == 0) *reinterpret_cast<float2*>(set_p + S::oE + d * 4) = of2(mul2(both, t23));
-    constexpr uint32_t kp = kC * S::kPitch, ka = 32 * S::kPitch, kb = 16 * S::kPitch;
-    const uint32_t col = d * 2, own = set + quarter * 4 * S::kPitch + col;
-    f32x2 kc[4], run = one;
+    constexpr uint32_t ka = 32 * S::kPitch, kb = 16 * S::kPitch;
+    const uint32_t col = base + d * 2;
+    f32x2 run = one;
 #pragma unroll
-    for (int j = 3; j >= 0; j--) {                                  // k times the decays behind it, in its quarter
+    for (int j = 3; j >= 0; j--) {
       kc[j] = mul2(k[j], run);
-      put<kParts>(mul2(kc[j], after), own + S::oR + j * S::kPitch, kp);
       run = mul2(run, a[j]);
     }
     run = one;
-    const uint32_t ta = base + S::oTa + (late ? 4 : 0) * S::kPitch + col, tb = base + S::oTb + (late ? 4 : 0) * S::kPitch + col;
-    const uint32_t ua = base + S::oTa + (16 + (odd ? 4 : 0)) * S::kPitch + col, ub = base + S::oTb + (8 + (odd ? 4 : 0)) * S::kPitch + col;
+    const uint32_t ta = col + S::oTa + (late ? 4 : 0) * S::kPitch, tb = col + S::oTb + (late ? 4 : 0) * S::kPitch;
+    const uint32_t ua = col + S::oTa + (16 + (odd ? 4 : 0)) * S::kPitch, ub = col + S::oTb + (8 + (odd ? 4 : 0)) * S::kPitch;
 #pragma unroll
-    for (int j = 0; j < 4; j++) {                                   // q and k times the decays from their quarter's start, their own included
+    for (int j = 0; j < 4; j++) {
       run = mul2(run, a[j]);
-      const f32x2 qr = mul2(q[j], run), kr = mul2(k[j], run);
-      put<2>(mul2(qr, before), own + S::oQ + j * S::kPitch, kp);
-      put<kParts>(mul2(kr, before), own + S::oK + j * S::kPitch, kp);
+      qr[j] = mul2(q[j], run);
+      kr[j] = mul2(k[j], run);
       // between neighbouring quarters: rows of quarters 1 and 3 against those of 0 and 2
-      put<kParts>(odd ? qr : kc[j], (odd ? ta : tb) + j * S::kPitch, odd ? ka : kb);
-      if (odd) put<kParts>(kr, ta + (8 + j) * S::kPitch, ka);
+      put<kParts>(odd ? qr[j] : kc[j], (odd ? ta : tb) + j * S::kPitch, odd ? ka : kb);
+      if (odd) put<kParts>(kr[j], ta + (8 + j) * S::kPitch, ka);
       // between the halves
-      put<kParts>(mul2(late ? qr : kc[j], half), (late ? ua : ub) + j * S::kPitch, late ? ka : kb);
-      if (late) put<kParts>(mul2(kr, half), ua + (8 + j) * S::kPitch, ka);
+      put<kParts>(mul2(late ? qr[j] : kc[j], half), (late ? ua : ub) + j * S::kPitch, late ? ka : kb);
+      if (late) put<kParts>(mul2(kr[j], half), ua + (8 + j) * S::kPitch, ka);
     }
     // the diagonal block of this quarter: (t, s <= t) for q, then (t, s < t) for k, summed over the 8 lanes that share it
     float val[16];
@@ -249,9 +257,21 @@ __device__ __forceinline__ void make_operands(const Params& p, uint8_t* sm, cons
     }
     *reinterpret_cast<float2*>(sm + S::oTri + ((warp * 4 + quarter) * 16 + idx) * 4) = make_float2(val[0], val[1]);
   };
+  auto operands = [&](uint32_t set, uint8_t* set_p) {
+    if (!item) return;
+    constexpr uint32_t kp = kC * S::kPitch;
+    const uint32_t own = set + quarter * 4 * S::kPitch + d * 2;
+    if (quarter == 0) *reinterpret_cast<float2*>(set_p + S::oE + d * 4) = of2(all);
+#pragma unroll
+    for (int j = 0; j < 4; j++) {
+      put<2>(mul2(qr[j], before), own + S::oQ + j * S::kPitch, kp);
+      put<kParts>(mul2(kr[j], before), own + S::oK + j * S::kPitch, kp);
+      put<kParts>(mul2(kc[j], after), own + S::oR + j * S::kPitch, kp);
+    }
+  };
   // the blocks between quarters and halves: left rows against right rows, k steps shared out over the warps
   auto blocks = [&]() {
-    if (warp * 16 >= p.Dp) return;
+    if (!item) return;
     float acc[2][4] = {};
     uint32_t a[2][kParts][4], b[2][kParts][2];
 #pragma unroll
@@ -354,33 +374,36 @@ __device__ __forceinline__ void make_operands(const Params& p, uint8_t* sm, cons
   cp_async_commit();
   fetch_beta(0);
   for (int i = tid; i < S::oZ / 16; i += kNT) st_zero16(base + i * 16);     // operand rows of channels beyond Dp stay zero
-  for (int c = 0; c < w.nc; c++) {
+  cp_async_wait<0>();
+  norms(0);
+  bar_sync(kMakers, kNT);
+  for (int c = 0; c < w.nc; c++) {                                  // the raw rows of chunk c are there, and their factors
     const int b = c & 1;
     uint8_t* set_p = sm + b * S::kSet;
     const uint32_t set = base + b * S::kSet;
-    float* factors = reinterpret_cast<float*>(sm + S::oF) + b * 3 * kC;   // two of them: one warp may still be at the chunk before
-    cp_async_wait<0>();
-    norms(factors);                                                 // of rows that this thread's own copies brought
-    bar_sync(kMakers, kNT);                                         // all raw rows of chunk c are there
-    if (c >= 2) bar_sync(kEmpty + b, 2 * kNT);                      // the products of chunk c - 2 are done
-    issue_v(c, set);
-    cp_async_commit();
-    prepare(min(kC, n - c * kC), set, set_p, factors);
-    bar_sync(kMakers, kNT);
     if (c + 1 < w.nc) {
       issue(c + 1);
       fetch_beta(c + 1);
     }
     cp_async_commit();
+    scores(c);
+    bar_sync(kMakers, kNT);
+    if (c >= 2) bar_sync(kEmpty + b, 2 * kNT);                      // the products of chunk c - 2 are done
+    issue_v(c, set);
+    cp_async_commit();
     blocks();
+    operands(set, set_p);
     bar_sync(kMakers, kNT);
-    assemble(set_p, factors);
+    assemble(set_p, factors_of(c));
+    if (c + 1 < w.nc) {
+      cp_async_wait<1>();
+      norms(c + 1);
+    }
     bar_sync(kMakers, kNT);
-    if (warp == 0) invert(set, factors + 2 * kC);
-    cp_async_wait<1>();                                             // v
+    if (warp == 0) invert(set, factors_of(c) + 2 * kC);             // the others go on
+    cp_async_wait<0>();                                             // v
     bar_arrive(kFull + b, 2 * kNT);
   }
-  cp_async_wait<0>();
 }
 
 // ---- the products -----------------------------------------------------------------------------------------------------------
@@ -391,7 +414,7 @@ __device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job
   const uint32_t base = smem_addr(sm);
   const bool fresh = p.positions[w.first] == 0, fused = p.o == nullptr;
   const int v0 = w.vb + w.warp * 16;                                // first value column of the warp
-  const bool mma_warp = v0 < p.Vp;
+  const bool mma_warp = w.warp * 16 < w.cols && v0 < p.Vp;
   float st[DK / 8][4];      // S^T: value column v0 + r8 (+ 8), channels 8 i + 2 quad (+ 1)
   float* state = p.state + (size_t(w.slot) * p.heads + w.h) * p.Dp * p.Vp;
 #pragma unroll
@@ -539,7 +562,7 @@ __device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job
 }
 
 template <int DK>
-__global__ void __launch_bounds__(2 * kNT, 1) k_delta_chunk(const Params p, const int* groups) {
+__global__ void __launch_bounds__(2 * kNT, 1) k_delta_chunk(const Params p, const int* groups, int cols) {
   extern __shared__ __align__(16) uint8_t sm[];
   pdl::launch_dependents();
   pdl::grid_dependency_wait();
@@ -550,7 +573,8 @@ __global__ void __launch_bounds__(2 * kNT, 1) k_delta_chunk(const Params p, cons
   w.n = groups[4 * blockIdx.x + 1];
   w.slot = groups[4 * blockIdx.x + 2];
   w.nc = (w.n + kC - 1) / kC;
-  w.vb = blockIdx.z * kCols;
+  w.vb = blockIdx.z * cols;
+  w.cols = cols;
   w.tid = threadIdx.x % kNT;
   w.warp = w.tid >> 5;
   w.lane = w.tid & 31;
@@ -569,10 +593,13 @@ __global__ void __launch_bounds__(2 * kNT, 1) k_delta_chunk(const Params p, cons
 template <int DK>
 cudaError_t launch(Params p, const int* groups, int ngroups, bool* finished, cudaStream_t st) {
   static bool done = false;
-  *finished = p.Vp <= kCols;
+  // few CTAs: the value columns of a head are shared out (every CTA makes the operands), and the head norm becomes a kernel of its own
+  int cols = kCols;
+  while (cols > 32 && cols / 2 < p.Vp && 2 * ngroups * p.heads * ((p.Vp + cols - 1) / cols) <= tbvops::sm_count()) cols /= 2;
+  *finished = p.Vp <= cols;
   if (*finished) p.o = nullptr;
   cudaError_t e = allow_smem(k_delta_chunk<DK>, Shape<DK>::kBytes, &done);
-  return e != cudaSuccess ? e : pdl::launch(k_delta_chunk<DK>, dim3(ngroups, p.heads, (p.Vp + kCols - 1) / kCols), dim3(2 * kNT), Shape<DK>::kBytes, st, 1, p, groups);
+  return e != cudaSuccess ? e : pdl::launch(k_delta_chunk<DK>, dim3(ngroups, p.heads, (p.Vp + cols - 1) / cols), dim3(2 * kNT), Shape<DK>::kBytes, st, 1, p, groups, cols);
 }
 
 }  // namespace
