@@ -75,7 +75,7 @@ def kernel_numbers(size: str, T: int, seqs: int, ctx: int, only: str = "") -> li
     X = C + 2 * R + _pad16(H)
     _linear(k, "gemm", "lugizen delta q, k, v, decay, gate, step", T, X, W)
     if not decode:
-        _linear(k, "gemm", "lugizen decay second (fp32)", T, H * D, R, f32=True)
+        _linear(k, "gemm", "lugizen decay second (softplus, fp32)", T, H * D, R, f32=True, act=ops.ACT_SOFTPLUS)
         _linear(k, "gemm", "lugizen gate second", T, H * V, R)
     Da, Va = _pad16(a.dim), _pad16(a.vdim)
     _linear(k, "gemm", "lugizen attention q, k, v", T, (a.heads + a.kv_heads) * Da + a.kv_heads * Va, W)
@@ -111,7 +111,7 @@ def kernel_numbers(size: str, T: int, seqs: int, ctx: int, only: str = "") -> li
             q, kk, v, low_a, low_g, beta = wide.split((K, K, H * V, R, R, _pad16(H)), 1)
             return lambda: ops.delta_step(q, kk, v, beta, low_a, low_g, w_a, b_a, w_g, rate, norm, st, out, segs, pos, conv=(w, past), **args)
         q, kk, v = _w(T, C).split((K, K, H * V), 1)
-        z, gate, o, beta = torch.randn(T, H * D, device=dev) - 3, _w(T, H * V), zeros(T, H * V), wide[:, C + 2 * R:]
+        z, gate, o, beta = torch.rand(T, H * D, device=dev) * 0.1, _w(T, H * V), zeros(T, H * V), wide[:, C + 2 * R:]
         gr = torch.from_numpy(scan_groups(segs.cpu().numpy(), model.scan_group_rows(segs[:, 1].cpu().numpy()))).to(dev)
         return lambda: ops.delta_scan(q, kk, v, beta, z, gate, rate, norm, st, o, out, segs, pos, groups=gr, **args)
     matrix = seqs * H * D * V * 4

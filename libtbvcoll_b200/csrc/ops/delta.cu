@@ -246,7 +246,7 @@ __global__ void __launch_bounds__(kStepThreads) k_delta_step(const Params p) {
 #pragma unroll
       for (int e = 0; e < 8; e++) s = fmaf(low[r + e], w[e], s);
     }
-    if (dec) as[at] = decay<T>(s, rate);
+    if (dec) as[at] = decay<T>(softplus<T>(s), rate);
     else gs[at] = sigmoid<T>(s);
   }
   for (int d = tid; d < p.Dp; d += kStepThreads) {
@@ -351,7 +351,7 @@ cudaError_t scan(const Params& p, int nseg, cudaStream_t st) {
 
 extern "C" {
 
-// Many rows per segment: q, k, v [rows, ld] behind convolution and SiLU, beta [rows, ldb], z fp32 [rows, ldz], gate [rows, ldg]; o fp32 scratch [rows, heads * Vp].
+// Many rows per segment: q, k, v [rows, ld] behind convolution and SiLU, beta [rows, ldb], z fp32 [rows, ldz] = softplus of the decay inputs, gate [rows, ldg]; o fp32 scratch [rows, heads * Vp].
 // groups (bf16; null: the sequential kernel): the segments as the chunked kernel takes them, [ngroups, 4].
 int tbv_op_delta_scan(const void* q, const void* k, const void* v, const void* beta, const void* z, const void* gate, const void* rate, const void* norm,
                       void* state, void* o, void* out, const void* segs, const void* positions, const void* groups, int ngroups, int rows, int nseg, int heads,

@@ -12,7 +12,7 @@ struct Params {
   const void* beta;            // [rows, ldx]: logits, column h
   const void *low_a, *low_g;   // [rows, ldx]: what enters the second products of decays and gates (one-row form)
   const void *w_a, *b_a, *w_g; // [heads * Dp, rank], [heads * Dp], [heads * Vp, rank] (one-row form)
-  const float* z;              // [rows, heads * Dp]: decay inputs, bias included (many-row form)
+  const float* z;              // [rows, heads * Dp]: softplus of the decay inputs (many-row form)
   const void* gate;            // [rows, ldg]: gate logits (many-row form)
   const float* rate;           // [heads]: exp(A_log)
   const float* norm;           // [Vp]
@@ -28,10 +28,10 @@ struct Params {
 
 constexpr float kUnitEps = 1e-6f;      // inside the root of the unit vectors' norm
 
-// e^(-rate * softplus(z)): decay of one key channel
-template <typename T> __device__ __forceinline__ float decay(float z, float rate);
-template <> __device__ __forceinline__ float decay<float>(float z, float rate) { return expf(-rate * vec::softplus<float>(z)); }
-template <> __device__ __forceinline__ float decay<__nv_bfloat16>(float z, float rate) { return __expf(-rate * vec::softplus<__nv_bfloat16>(z)); }
+// e^(-rate * s), s = softplus of the decay input: decay of one key channel
+template <typename T> __device__ __forceinline__ float decay(float s, float rate);
+template <> __device__ __forceinline__ float decay<float>(float s, float rate) { return expf(-rate * s); }
+template <> __device__ __forceinline__ float decay<__nv_bfloat16>(float s, float rate) { return __expf(-rate * s); }
 
 inline bool sizes_ok(const Params& p) {
   return p.heads > 0 && p.heads <= 65535 && p.kv_heads > 0 && p.heads % p.kv_heads == 0 && p.Dp > 0 && p.Dp <= 256 && p.Dp % 16 == 0 && p.Vp > 0 && p.Vp <= 1024 &&

@@ -52,7 +52,9 @@ struct Shape {
   static constexpr int oA = oV + kC * kVPitch;                     // A                   [2][16][apitch]
   static constexpr int oT = oA + 2 * kC * kAPitch;                 // T                   [parts][16][apitch]
   static constexpr int oE = oT + kParts * kC * kAPitch;            // P_16                [DK] fp32
-  static constexpr int kSet = oE + DK * 4;
+  static constexpr int oL = oE + DK * 4;                           // diag(beta) B        [16][17] fp32
+  static constexpr int oB = oL + 16 * 17 * 4;                      // step sizes          [16] fp32
+  static constexpr int kSet = oB + kC * 4;
   // dynamic shared memory: two sets, then what one of the groups has for itself
   static constexpr int oTa = 2 * kSet;                             // blocks: left rows   [parts][2 kinds][16][pitch]  (8 of q, 8 of k)
   static constexpr int oTb = oTa + kParts * 32 * kPitch;           //         right rows  [parts][2 kinds][8][pitch]
@@ -61,8 +63,8 @@ struct Shape {
   static constexpr int oF = oZ + 2 * kRaw;                         // factors of q, of k, step sizes [2 chunks][3][16] fp32
   static constexpr int oTri = oF + 6 * kC * 4;                     // diagonal blocks     [items][4 quarters][16] fp32
   static constexpr int oOff = oTri + (kItems + 1) * 256;           // the other blocks' sums [warps][2][16][8] fp32
-  static constexpr int oL = oOff + kNW * 1024;                     // diag(beta) B [16][17] fp32, its inverse [16][17], a product [8][17]
-  static constexpr int oO = oL + 40 * 17 * 4;                      // o                   [16][opitch] fp32
+  static constexpr int oI = oOff + kNW * 1024;                     // I + diag(beta) B inverted [16][17] fp32, a product [8][17]
+  static constexpr int oO = oI + 24 * 17 * 4;                      // o                   [16][opitch] fp32
   static constexpr int kBytes = oO + kC * kOPitch * 4;
   static_assert(kSet % 16 == 0 && oO % 16 == 0 && kBytes <= int(kMaxSmem), "shared memory");
 };
@@ -78,17 +80,17 @@ __device__ __forceinline__ float2 of2(f32x2 v) {
   unpack2(v, r.x, r.y);
   return r;
 }
-// (x, y) as sums of N bf16 pairs
+// (x, y) as sums of N bf16 pairs: all but the last are cut off behind eight bits, so that what is left is exact
 template <int N>
 __device__ __forceinline__ void split(float x, float y, uint32_t* part) {
 #pragma unroll
-  for (int i = 0; i < N; i++) {
-    part[i] = pack_bf16(x, y);
-    if (i + 1 < N) {
-      x -= __uint_as_float(part[i] << 16);
-      y -= __uint_as_float(part[i] & 0xffff0000u);
-    }
+  for (int i = 0; i + 1 < N; i++) {
+    const uint32_t u = __float_as_uint(x), v = __float_as_uint(y);
+    part[i] = __byte_perm(u, v, 0x7632);
+    x -= __uint_as_float(u & 0xffff0000u);
+    y -= __uint_as_float(v & 0xffff0000u);
   }
+  part[N - 1] = pack_bf16(x, y);
 }
 // two neighbouring channels to `addr`, their parts `stride` bytes apart
 template <int N>
@@ -319,12 +321,67 @@ __device__ __forceinline__ void make_operands(const Params& p, uint8_t* sm, cons
     const __nv_bfloat16 hi = __float2bfloat16_rn(vq);
     reinterpret_cast<__nv_bfloat16*>(set_p + S::oA + t * S::kAPitch)[s] = hi;
     reinterpret_cast<__nv_bfloat16*>(set_p + S::oA + (kC + t) * S::kAPitch)[s] = __float2bfloat16_rn(vq - __bfloat162float(hi));
-    reinterpret_cast<float*>(sm + S::oL)[t * 17 + s] = s < t ? vk * factors[2 * kC + t] : 0.f;
+    reinterpret_cast<float*>(set_p + S::oL)[t * 17 + s] = s < t ? vk * factors[2 * kC + t] : 0.f;
+    if (tid < kC) reinterpret_cast<float*>(set_p + S::oB)[tid] = factors[2 * kC + tid];
   };
-  // T, by one warp
-  auto invert = [&](uint32_t set, const float* beta) {
-    const float* L = reinterpret_cast<const float*>(sm + S::oL);
-    float *I = reinterpret_cast<float*>(sm + S::oL) + 16 * 17, *M = I + 16 * 17;
+  issue(0);
+  cp_async_commit();
+  fetch_beta(0);
+  for (int i = tid; i < S::oZ / 16; i += kNT) st_zero16(base + i * 16);     // operand rows of channels beyond Dp stay zero
+  cp_async_wait<0>();
+  norms(0);
+  bar_sync(kMakers, kNT);
+  for (int c = 0; c < w.nc; c++) {                                  // the raw rows of chunk c are there, and their factors
+    const int b = c & 1;
+    uint8_t* set_p = sm + b * S::kSet;
+    const uint32_t set = base + b * S::kSet;
+    if (c + 1 < w.nc) {
+      issue(c + 1);
+      fetch_beta(c + 1);
+    }
+    cp_async_commit();
+    scores(c);
+    bar_sync(kMakers, kNT);
+    if (c >= 2) bar_sync(kEmpty + b, 2 * kNT);                      // the products of chunk c - 2 are done
+    issue_v(c, set);
+    cp_async_commit();
+    blocks();
+    operands(set, set_p);
+    bar_sync(kMakers, kNT);
+    assemble(set_p, factors_of(c));
+    if (c + 1 < w.nc) {
+      cp_async_wait<1>();
+      norms(c + 1);
+    }
+    bar_sync(kMakers, kNT);
+    cp_async_wait<0>();                                             // v
+    bar_arrive(kFull + b, 2 * kNT);
+  }
+}
+
+// ---- the products -----------------------------------------------------------------------------------------------------------
+template <int DK>
+__device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job& w) {
+  using S = Shape<DK>;
+  const int lane = w.lane, r8 = lane >> 2, quad = lane & 3, row16 = w.row16, l16 = w.l16, n = w.n;
+  const uint32_t base = smem_addr(sm);
+  const bool fresh = p.positions[w.first] == 0, fused = p.o == nullptr;
+  const int v0 = w.vb + w.warp * 16;                                // first value column of the warp
+  const bool mma_warp = w.warp * 16 < w.cols && v0 < p.Vp;
+  float st[DK / 8][4];      // S^T: value column v0 + r8 (+ 8), channels 8 i + 2 quad (+ 1)
+  float* state = p.state + (size_t(w.slot) * p.heads + w.h) * p.Dp * p.Vp;
+#pragma unroll
+  for (int i = 0; i < DK / 8; i++)
+#pragma unroll
+    for (int j = 0; j < 4; j++) {
+      const int d = i * 8 + quad * 2 + (j & 1), v = v0 + r8 + (j >> 1) * 8;
+      st[i][j] = !mma_warp || fresh || d >= p.Dp ? 0.f : state[size_t(d) * p.Vp + v];
+    }
+  const uint32_t brow = (lane & 7) + ((lane >> 4) << 3), bcol = ((lane >> 3) & 1) * 16;    // right operands stored [n][k]
+  // T, by one warp (the last one, which has no columns of its own where they are shared out)
+  auto invert = [&](uint32_t set, const uint8_t* set_p) {
+    const float *L = reinterpret_cast<const float*>(set_p + S::oL), *beta = reinterpret_cast<const float*>(set_p + S::oB);
+    float *I = reinterpret_cast<float*>(sm + S::oI), *M = I + 16 * 17;
     const int b8 = lane & 8, j = lane & 7;                          // lanes 16 .. 31 repeat the others
     float x[8];
 #pragma unroll
@@ -369,62 +426,6 @@ __device__ __forceinline__ void make_operands(const Params& p, uint8_t* sm, cons
     out(8 + r8, c, m0, m1);
     out(8 + r8, 8 + c, I[(8 + r8) * 17 + 8 + c], I[(8 + r8) * 17 + 8 + c + 1]);
   };
-
-  issue(0);
-  cp_async_commit();
-  fetch_beta(0);
-  for (int i = tid; i < S::oZ / 16; i += kNT) st_zero16(base + i * 16);     // operand rows of channels beyond Dp stay zero
-  cp_async_wait<0>();
-  norms(0);
-  bar_sync(kMakers, kNT);
-  for (int c = 0; c < w.nc; c++) {                                  // the raw rows of chunk c are there, and their factors
-    const int b = c & 1;
-    uint8_t* set_p = sm + b * S::kSet;
-    const uint32_t set = base + b * S::kSet;
-    if (c + 1 < w.nc) {
-      issue(c + 1);
-      fetch_beta(c + 1);
-    }
-    cp_async_commit();
-    scores(c);
-    bar_sync(kMakers, kNT);
-    if (c >= 2) bar_sync(kEmpty + b, 2 * kNT);                      // the products of chunk c - 2 are done
-    issue_v(c, set);
-    cp_async_commit();
-    blocks();
-    operands(set, set_p);
-    bar_sync(kMakers, kNT);
-    assemble(set_p, factors_of(c));
-    if (c + 1 < w.nc) {
-      cp_async_wait<1>();
-      norms(c + 1);
-    }
-    bar_sync(kMakers, kNT);
-    if (warp == 0) invert(set, factors_of(c) + 2 * kC);             // the others go on
-    cp_async_wait<0>();                                             // v
-    bar_arrive(kFull + b, 2 * kNT);
-  }
-}
-
-// ---- the products -----------------------------------------------------------------------------------------------------------
-template <int DK>
-__device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job& w) {
-  using S = Shape<DK>;
-  const int lane = w.lane, r8 = lane >> 2, quad = lane & 3, row16 = w.row16, l16 = w.l16, n = w.n;
-  const uint32_t base = smem_addr(sm);
-  const bool fresh = p.positions[w.first] == 0, fused = p.o == nullptr;
-  const int v0 = w.vb + w.warp * 16;                                // first value column of the warp
-  const bool mma_warp = w.warp * 16 < w.cols && v0 < p.Vp;
-  float st[DK / 8][4];      // S^T: value column v0 + r8 (+ 8), channels 8 i + 2 quad (+ 1)
-  float* state = p.state + (size_t(w.slot) * p.heads + w.h) * p.Dp * p.Vp;
-#pragma unroll
-  for (int i = 0; i < DK / 8; i++)
-#pragma unroll
-    for (int j = 0; j < 4; j++) {
-      const int d = i * 8 + quad * 2 + (j & 1), v = v0 + r8 + (j >> 1) * 8;
-      st[i][j] = !mma_warp || fresh || d >= p.Dp ? 0.f : state[size_t(d) * p.Vp + v];
-    }
-  const uint32_t brow = (lane & 7) + ((lane >> 4) << 3), bcol = ((lane >> 3) & 1) * 16;    // right operands stored [n][k]
   for (int c = 0; c < w.nc; c++) {
     const int b = c & 1, at = c * kC;
     const uint32_t set = base + b * S::kSet;
@@ -432,40 +433,42 @@ __device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job
     if (fused && at + row16 < n && l16 * 8 < p.Vp)
       gate.load(static_cast<const __nv_bfloat16*>(p.gate) + size_t(w.first + at + row16) * p.ldg + size_t(w.h) * p.Vp + l16 * 8);
     bar_sync(kFull + b, 2 * kNT);
+    if (w.warp == kNW - 1) invert(set, sm + b * S::kSet);
+    uint32_t l[kParts][4], f[4];
+    float o[2][2][4] = {};
     if (mma_warp) {
       // (q P) S and (k P) S, two sums each for even and odd k steps: value column as above, tokens 8 i + 2 quad (+ 1)
-      float o[2][2][4] = {}, x[2][2][4] = {};
+      float x[2][2][4] = {};
 #pragma unroll
       for (int ks = 0; ks < DK / 16; ks += 2) {
-        uint32_t s[2][kParts][4], f[2][4];
+        uint32_t s[2][kParts][4], r[2][4];
         as_left<kParts>(st + 2 * ks, s[0]);
         as_left<kParts>(st + 2 * ks + 2, s[1]);
 #pragma unroll
         for (int j = kParts - 1; j >= 0; j--) {
 #pragma unroll
-          for (int e = 0; e < 2; e++) ldmatrix_x4(set + S::oK + (j * kC + brow) * S::kPitch + bcol + (ks + e) * 32, f[e]);
+          for (int e = 0; e < 2; e++) ldmatrix_x4(set + S::oK + (j * kC + brow) * S::kPitch + bcol + (ks + e) * 32, r[e]);
 #pragma unroll
           for (int i = kParts - 1 - j; i >= 0; i--)
 #pragma unroll
             for (int e = 0; e < 2; e++) {
-              mma_bf16(x[e][0], s[e][i], f[e][0], f[e][1]);
-              mma_bf16(x[e][1], s[e][i], f[e][2], f[e][3]);
+              mma_bf16(x[e][0], s[e][i], r[e][0], r[e][1]);
+              mma_bf16(x[e][1], s[e][i], r[e][2], r[e][3]);
             }
         }
 #pragma unroll
         for (int j = 1; j >= 0; j--) {
 #pragma unroll
-          for (int e = 0; e < 2; e++) ldmatrix_x4(set + S::oQ + (j * kC + brow) * S::kPitch + bcol + (ks + e) * 32, f[e]);
+          for (int e = 0; e < 2; e++) ldmatrix_x4(set + S::oQ + (j * kC + brow) * S::kPitch + bcol + (ks + e) * 32, r[e]);
 #pragma unroll
           for (int i = 1 - j; i >= 0; i--)
 #pragma unroll
             for (int e = 0; e < 2; e++) {
-              mma_bf16(o[e][0], s[e][i], f[e][0], f[e][1]);
-              mma_bf16(o[e][1], s[e][i], f[e][2], f[e][3]);
+              mma_bf16(o[e][0], s[e][i], r[e][0], r[e][1]);
+              mma_bf16(o[e][1], s[e][i], r[e][2], r[e][3]);
             }
         }
       }
-      uint32_t l[kParts][4], f[4];
       ldmatrix_x4_trans(set + S::oV + brow * S::kVPitch + w.warp * 32 + bcol, f);      // v^T: stored [token][column]
 #pragma unroll
       for (int j = 0; j < 4; j++) {
@@ -474,8 +477,11 @@ __device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job
         y[0] = __uint_as_float(f[j] << 16) - (y[0] + z[0]);
         y[1] = __uint_as_float(f[j] & 0xffff0000u) - (y[1] + z[1]);
       }
-      float u[2][4] = {};
       as_left<kParts>(x[0], l);
+    }
+    bar_sync(kProducts, kNT);                                       // T is there
+    if (mma_warp) {
+      float u[2][4] = {};
 #pragma unroll
       for (int j = kParts - 1; j >= 0; j--) {
         ldmatrix_x4(set + S::oT + (j * kC + brow) * S::kAPitch + bcol, f);
@@ -530,14 +536,14 @@ __device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job
     // head norm, weight and gate; a row per 16 lanes, 8 columns per lane.  (The next chunk's o is written behind its `full`, which waits for all of these warps.)
     bar_sync(kProducts, kNT);
     const int v = l16 * 8;
-    float f[8], ss = 0.f;
-    vec::load8(reinterpret_cast<const float*>(sm + S::oO) + row16 * S::kOPitch + v, f);
+    float y[8], ss = 0.f;
+    vec::load8(reinterpret_cast<const float*>(sm + S::oO) + row16 * S::kOPitch + v, y);
     if (v >= p.Vp) {
 #pragma unroll
-      for (int e = 0; e < 8; e++) f[e] = 0.f;
+      for (int e = 0; e < 8; e++) y[e] = 0.f;
     }
 #pragma unroll
-    for (int e = 0; e < 8; e++) ss = fmaf(f[e], f[e], ss);
+    for (int e = 0; e < 8; e++) ss = fmaf(y[e], y[e], ss);
 #pragma unroll
     for (int o = 8; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
     if (at + row16 < n && v < p.Vp) {
@@ -546,8 +552,8 @@ __device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job
       gate.unpack(gt);
       vec::load8(p.norm + v, wt);
 #pragma unroll
-      for (int e = 0; e < 8; e++) f[e] = f[e] * r * wt[e] * vec::sigmoid<__nv_bfloat16>(gt[e]);
-      vec::store8(static_cast<__nv_bfloat16*>(p.out) + size_t(w.first + at + row16) * p.ldo + size_t(w.h) * p.Vp + v, f);
+      for (int e = 0; e < 8; e++) y[e] = y[e] * r * wt[e] * vec::sigmoid<__nv_bfloat16>(gt[e]);
+      vec::store8(static_cast<__nv_bfloat16*>(p.out) + size_t(w.first + at + row16) * p.ldo + size_t(w.h) * p.Vp + v, y);
     }
   }
   if (mma_warp) {

@@ -14,6 +14,7 @@
 #pragma once
 #include "../pdl.cuh"
 #include "sm100.cuh"
+#include "vec.cuh"
 
 namespace gemm {
 
@@ -60,7 +61,7 @@ enum Act : int { kActNone = 0, kActSoftplus = 1, kActSoftcap = 2, kActSilu = 3, 
 // tanh form of gelu: v / 2 * (1 + tanh(s / 2)) = v * sigmoid(s), s = 2 sqrt(2 / pi) (v + 0.044715 v^3)
 __device__ __forceinline__ float gelu_slope(float v) { return 1.5957691216057308f * fmaf(0.044715f * v * v, v, v); }
 __device__ __forceinline__ float apply_act(float v, int act, float a) {
-  if (act == kActSoftplus) return v > 20.f ? v : log1pf(expf(v));
+  if (act == kActSoftplus) return vec::softplus<__nv_bfloat16>(v);
   if (act == kActSoftcap) return a * tanhf(v / a);
   if (act == kActSilu) return __fdividef(v, 1.0f + __expf(-v));   // an infinite denominator gives 0
   if (act == kActGelu) return __fdividef(v, 1.0f + __expf(-gelu_slope(v)));

@@ -84,7 +84,7 @@ __global__ void __launch_bounds__(256) k_gemm_f32(const F32Params p) {
         if (m0 + tm + j < M) {
           if (p.act && m0 + tm + j < p.act_m) {
             if (p.act == gemm::kActSilu || p.act == gemm::kActGelu) v[j] = v[j] / (1.0f + expf(p.act == gemm::kActSilu ? -v[j] : -gemm::gelu_slope(v[j])));
-            else v[j] = gemm::apply_act(v[j], p.act, p.act_a);
+            else v[j] = p.act == gemm::kActSoftplus ? vec::softplus<float>(v[j]) : gemm::apply_act(v[j], p.act, p.act_a);
           }
           y[size_t(n) * p.ldy + m0 + tm + j] = v[j];
         }

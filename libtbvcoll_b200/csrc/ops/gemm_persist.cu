@@ -125,7 +125,10 @@ __device__ __forceinline__ void store16(const gemm::Params& p, int n, int f, con
     for (int j = 0; j < 16; j++) v[j] += __bfloat162float(p.bias[f + j]);
   }
   if (EPI == gemm::kEpiF32) {
-    if (p.act != gemm::kActNone) {                  // one branch, not one per value
+    if (p.act == gemm::kActSoftplus) {              // one branch, not one per value
+#pragma unroll
+      for (int j = 0; j < 16; j++) v[j] = gemm::apply_act(v[j], gemm::kActSoftplus, 0.f);
+    } else if (p.act != gemm::kActNone) {
 #pragma unroll
       for (int j = 0; j < 16; j++) v[j] = gemm::apply_act(v[j], p.act, p.act_a);
     }

@@ -4,7 +4,7 @@ attention; dense GELU feed-forwards or mixtures of experts; one norm behind ever
 What lies between two sublayers is ONE kernel (``ops.residual`` with ``post``: norm of the branch, residual sum and, when every sequence has one row, the next
 layer's convolution; otherwise ``ops.short_conv`` follows).  Feed-forwards read the residual stream itself.
 
-    delta       q, k, v, low-rank decay and gate, step size GEMM -> [convolution + SiLU -> decay GEMM (fp32), gate GEMM -> recurrence with unit norms, head norm and
+    delta       q, k, v, low-rank decay and gate, step size GEMM -> [convolution + SiLU -> decay GEMM (fp32, softplus inside), gate GEMM -> recurrence with unit norms, head norm and
                 gate] -> out-projection GEMM (fp32); in brackets: one kernel when every sequence has one row
     attention   q, k, v GEMM -> norms, rotation, value mix, cache write -> rows kernel over the cache (few rows) or tiled kernel (many) -> out-projection GEMM (fp32)
     latent      query latent, latent, rotated key GEMM -> norms, rotation, cache write -> query GEMM -> rotation -> latent attention with a window ->
@@ -132,7 +132,7 @@ class Lugizen(StreamDecoder, LatentAttention):
                            conv=(w[p + "conv"], self.conv[i]) if inside else None, **args)
         else:
             z, gate = self._buf("z", T, w[p + "a2"].shape[0]), self._buf("gate", T, V)
-            ops.linear(low_a, w[p + "a2"], z, bias=w[p + "dt_bias"])
+            ops.linear(low_a, w[p + "a2"], z, bias=w[p + "dt_bias"], act=ops.ACT_SOFTPLUS)
             ops.linear(low_g, w[p + "g2"], gate)
             ops.delta_scan(q, k, v, beta, z, gate, w[p + "rate"], w[p + "norm"], self.state[i], self._buf("o", T, V), out, b.segs, b.positions, groups=b.scan_groups, **args)
         return self._project(b, i, out)

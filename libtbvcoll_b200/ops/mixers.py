@@ -298,11 +298,11 @@ def fixed_decay_step(q, k, v, g, norm, powers, state, out, sums, segs, positions
 
 # ---- gated delta rule with a decay per key channel -----------------------------------------------------------------------------------
 def delta_scan(q, k, v, beta, z, gate, rate, norm, state, o, out, segs, positions, kv_heads: int, dim: int, vdim: int, eps: float, groups=None) -> None:
-    """Per head, q and k of its key head made unit vectors (q times dim^-0.5), S' = diag(exp(-rate softplus(z_t))) S_{t-1}, u = sigmoid(beta_t) (v_t - S'^T k_t),
+    """Per head, q and k of its key head made unit vectors (q times dim^-0.5), S' = diag(exp(-rate z_t)) S_{t-1}, u = sigmoid(beta_t) (v_t - S'^T k_t),
     S_t = S' + k_t u^T over the rows of every segment; out = RMSNorm(S_t^T q_t) * norm * sigmoid(gate).
 
     q, k [rows, kv_heads * Dp] and v [rows, heads * Vp]: column views of one buffer, behind convolution and SiLU; beta [rows, >= heads], gate [rows, heads * Vp] in the
-    activation type; z fp32 [rows, heads * Dp], rate fp32 [heads], norm fp32 [Vp]; state fp32 [slots, heads, Dp, Vp] is replaced; o fp32 scratch [rows, heads * Vp].
+    activation type; z fp32 [rows, heads * Dp] (softplus of the decay inputs), rate fp32 [heads], norm fp32 [Vp]; state fp32 [slots, heads, Dp, Vp] is replaced; o fp32 scratch [rows, heads * Vp].
     ``groups`` (bf16): the segments, int32 [n, 4] (engine.batch.scan_groups), for the chunked tensor-core kernel where the sizes allow."""
     _, H, Dp, Vp = state.shape
     rows = q.shape[0]
@@ -316,7 +316,7 @@ def delta_scan(q, k, v, beta, z, gate, rate, norm, state, o, out, segs, position
 
 
 def delta_step(q, k, v, beta, low_a, low_g, w_a, b_a, w_g, rate, norm, state, out, segs, positions, kv_heads: int, dim: int, vdim: int, eps: float, conv=None) -> None:
-    """``delta_scan`` for one row per segment, with z = low_a @ w_a^T + b_a and gate = low_g @ w_g^T computed inside.  ``conv`` = (taps fp32 [K, C], state fp32
+    """``delta_scan`` for one row per segment, with z = softplus(low_a @ w_a^T + b_a) and gate = low_g @ w_g^T computed inside.  ``conv`` = (taps fp32 [K, C], state fp32
     [slots, K - 1, C]), for kv_heads = heads: q, k and v are taken before convolution and SiLU, and that state is replaced."""
     _, H, Dp, Vp = state.shape
     taps, past = conv if conv is not None else (None, None)
