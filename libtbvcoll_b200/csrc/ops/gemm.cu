@@ -372,7 +372,8 @@ void gemm_config(int M, int N, int K, int splits_hint, int* bn_out, int* splits_
   }
   while (splits > 1 && (kb + splits - 1) / splits * (splits - 1) >= kb) splits /= 2;  // every split gets work
   const int stage_bytes = gemm::kATileBytes + bn * 128;
-  const int budget = (tiles * splits > sms) ? 108 * 1024 : 200 * 1024;  // two CTAs per SM when the grid is larger than the GPU
+  // two CTAs per SM when the grid is larger than the GPU, or than the four fifths of it that clusters of eight find at one CTA per SM
+  const int budget = (tiles * splits > (splits < 8 ? sms : sms * 4 / 5)) ? 108 * 1024 : 200 * 1024;
   int stages = budget / stage_bytes;
   stages = stages < 2 ? 2 : (stages > gemm::kMaxStages ? gemm::kMaxStages : stages);
   const int need = splits > 1 || f32_out ? bn * 512 : bn * 256;  // epilogue staging reuses the ring
