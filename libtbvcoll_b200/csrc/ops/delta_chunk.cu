@@ -124,17 +124,21 @@ __device__ __forceinline__ void make_operands(const Params& p, uint8_t* sm, cons
   using S = Shape<DK>;
   const int tid = w.tid, warp = w.warp, lane = w.lane, r8 = lane >> 2, quad = lane & 3, row16 = w.row16, l16 = w.l16, n = w.n;
   const uint32_t base = smem_addr(sm);
-  const float rate = p.rate[w.h], qscale = rsqrtf(float(p.dim));
+  const float rate2 = -p.rate[w.h] * kLog2e, qscale = rsqrtf(float(p.dim));
   const __nv_bfloat16* qg = static_cast<const __nv_bfloat16*>(p.q) + size_t(w.g) * p.Dp;
   const __nv_bfloat16* kg = static_cast<const __nv_bfloat16*>(p.k) + size_t(w.g) * p.Dp;
   const __nv_bfloat16* vg = static_cast<const __nv_bfloat16*>(p.v) + size_t(w.h) * p.Vp + w.vb;
   const float* zg = p.z + size_t(w.h) * p.Dp;
 
-  // rows of chunk c on their way to shared memory (missing rows: whatever the buffer holds, left out when they are used)
+  // rows of chunk c on their way to shared memory; missing rows are zeros: they decay nothing, write nothing and read nothing
   auto issue = [&](int c) {
     const size_t r = size_t(w.first + c * kC + row16);
     const uint32_t raw = base + S::oZ + (c & 1) * S::kRaw;
-    if (c * kC + row16 >= n) return;
+    if (c * kC + row16 >= n) {
+      for (int x = l16; x < DK / 4; x += 16) st_zero16(raw + (row16 * DK + x * 4) * 4);
+      for (int x = l16; x < DK / 4; x += 16) st_zero16(raw + S::kRq + (x >= DK / 8 ? S::kRk - S::kRq : 0) + (row16 * DK + x % (DK / 8) * 8) * 2);
+      return;
+    }
     for (int x = l16; x < p.Dp / 4; x += 16) cp_async16(raw + (row16 * DK + x * 4) * 4, zg + r * p.ldz + x * 4);
     for (int x = l16; x < p.Dp / 8; x += 16) {
       cp_async16(raw + S::kRq + (row16 * DK + x * 8) * 2, qg + r * p.ld + x * 8);
@@ -182,21 +186,19 @@ __device__ __forceinline__ void make_operands(const Params& p, uint8_t* sm, cons
   const bool odd = quarter & 1, late = quarter & 2, item = warp * 16 < p.Dp;
   auto scores = [&](int c) {
     if (!item) return;
-    const int nt = min(kC, n - c * kC);
     const uint8_t* raw = sm + S::oZ + (c & 1) * S::kRaw;
     const float* factors = factors_of(c);
     f32x2 a[4], q[4], k[4];
 #pragma unroll
     for (int j = 0; j < 4; j++) {
       const int t = quarter * 4 + j;
-      const bool ok = t < nt;
       const float2 z = *reinterpret_cast<const float2*>(raw + (t * DK + d) * 4);
       const uint32_t qb = *reinterpret_cast<const uint32_t*>(raw + S::kRq + (t * DK + d) * 2), kb = *reinterpret_cast<const uint32_t*>(raw + S::kRk + (t * DK + d) * 2);
       const float fq = factors[t], fk = factors[kC + t];
-      const float a0 = delta_ops::decay<__nv_bfloat16>(z.x, rate), a1 = delta_ops::decay<__nv_bfloat16>(z.y, rate);
-      a[j] = ok ? pack2(a0, a1) : pack2(1.f, 1.f);
-      q[j] = ok ? pack2(__uint_as_float(qb << 16) * fq, __uint_as_float(qb & 0xffff0000u) * fq) : 0ull;
-      k[j] = ok ? pack2(__uint_as_float(kb << 16) * fk, __uint_as_float(kb & 0xffff0000u) * fk) : 0ull;
+      const float a0 = vec::pow2<__nv_bfloat16>(z.x * rate2), a1 = vec::pow2<__nv_bfloat16>(z.y * rate2);
+      a[j] = pack2(a0, a1);
+      q[j] = mul2(pack2(__uint_as_float(qb << 16), __uint_as_float(qb & 0xffff0000u)), pack2(fq, fq));
+      k[j] = mul2(pack2(__uint_as_float(kb << 16), __uint_as_float(kb & 0xffff0000u)), pack2(fk, fk));
     }
     // products over quarters: t1 of quarter ^ 1, t23 of the two others
     const f32x2 tot = mul2(mul2(a[0], a[1]), mul2(a[2], a[3]));

@@ -113,15 +113,6 @@ struct ScanParams {
   int inner, N, ldu, ldxz, zoff, lddt, ldbc, boff, coff, ldo, ldc, taps;
 };
 
-// 2^x: the hardware instruction for bf16 models, CUDA's exp2f for fp32 ones
-template <typename T> __device__ __forceinline__ float pow2(float x);
-template <> __device__ __forceinline__ float pow2<float>(float x) { return exp2f(x); }
-template <> __device__ __forceinline__ float pow2<__nv_bfloat16>(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-
 // Replaces the convolution state of channel c by its last taps - 1 inputs; ascending, so an old entry is read before it is overwritten.
 template <typename T>
 __device__ __forceinline__ void roll_conv_state(const ScanParams& p, const T* xz, int first, int count, int slot, bool fresh, int c) {

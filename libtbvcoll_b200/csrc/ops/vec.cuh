@@ -37,6 +37,14 @@ template <> __device__ __forceinline__ float softplus<__nv_bfloat16>(float v) {
   h = fmaf(h, q, 1.f);
   return fmaxf(v, 0.f) + 2.f * r * h;
 }
+// 2^x: the hardware instruction for bf16 models, CUDA's exp2f for fp32 ones
+template <typename T> __device__ __forceinline__ float pow2(float x);
+template <> __device__ __forceinline__ float pow2<float>(float x) { return exp2f(x); }
+template <> __device__ __forceinline__ float pow2<__nv_bfloat16>(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 
 __device__ __forceinline__ void load8(const float* p, float* f) {
   const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
