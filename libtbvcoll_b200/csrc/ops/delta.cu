@@ -179,13 +179,13 @@ __global__ void __launch_bounds__(256) k_delta_norm_gate(const Params p, int row
 }
 
 // One row per segment.  Threads: 4 value columns each, as many groups of keys as fit.
-constexpr int kStepThreads = 256, kStepKeys = 16;
+constexpr int kStepThreads = 256, kStepKeys = 16, kStepTaps = 3;     // kStepTaps: carried inputs of the convolution taken at once
 template <typename T>
 __global__ void __launch_bounds__(kStepThreads) k_delta_step(const Params p) {
   extern __shared__ __align__(16) float sm[];
   __shared__ float red[4][8];
   const int h = blockIdx.x, g = h / (p.heads / p.kv_heads), tid = threadIdx.x, nc = p.Vp / 4, nkg = max(1, kStepThreads / nc);
-  float *qs = sm, *ks = qs + p.Dp, *as = ks + p.Dp, *vs = as + p.Dp, *us = vs + p.Vp, *gs = us + p.Vp, *acc = gs + p.Vp, *la = acc + 2 * nkg * p.Vp, *lg = la + p.rank;
+  float *qs = sm, *ks = qs + p.Dp, *vs = ks + p.Dp, *as = vs + p.Vp, *us = as + p.Dp, *gs = us + p.Vp, *acc = gs + p.Vp, *la = acc + 2 * nkg * p.Vp, *lg = la + p.rank;
   pdl::launch_dependents();
   pdl::grid_dependency_wait();
   const int* seg = p.segs + 4 * blockIdx.y;
@@ -205,30 +205,53 @@ __global__ void __launch_bounds__(kStepThreads) k_delta_step(const Params p) {
     la[i] = to_f((i < p.rank ? static_cast<const T*>(p.low_a) : static_cast<const T*>(p.low_g) - p.rank)[size_t(row) * p.ldx + i]);
   // q, k, v of this head; the convolution over the carried inputs first, if it was not done before
   float sq = 0.f, sk = 0.f, sd = 0.f;
-  auto value = [&](const void* base, int c, int column) {
-    const T* x = static_cast<const T*>(base) + size_t(row) * p.ld + c;
-    float v = to_f(*x);
-    if (p.taps_w) {
-      float* past = p.conv + size_t(slot) * (p.taps - 1) * p.C + column;
-      float a = 0.f;
-      for (int j = 0; j < p.taps - 1; j++) {
-        const float in = fresh ? 0.f : past[size_t(j) * p.C];
-        a = fmaf(p.taps_w[size_t(j) * p.C + column], in, a);
-        if (j > 0) past[size_t(j - 1) * p.C] = in;
+  // (all loads of a thread's two values come before its stores: one round trip)
+  const int K = p.kv_heads * p.Dp, total = 2 * p.Dp + p.Vp, keep = p.taps_w ? p.taps - 1 : 0;
+  for (int i0 = tid; i0 < total; i0 += 2 * kStepThreads) {
+    float cur[2], in[2][kStepTaps], w[2][kStepTaps], last[2];
+    int column[2];
+#pragma unroll
+    for (int e = 0; e < 2; e++) {
+      const int i = i0 + e * kStepThreads;
+      if (i >= total) continue;
+      const int part = i < p.Dp ? 0 : (i < 2 * p.Dp ? 1 : 2), c = part == 2 ? h * p.Vp + i - 2 * p.Dp : g * p.Dp + i - part * p.Dp;
+      column[e] = part * K + c;
+      cur[e] = to_f((part == 0 ? static_cast<const T*>(p.q) : (part == 1 ? static_cast<const T*>(p.k) : static_cast<const T*>(p.v)))[size_t(row) * p.ld + c]);
+      if (!p.taps_w) continue;
+      last[e] = p.taps_w[size_t(keep) * p.C + column[e]];
+      const float* past = p.conv + size_t(slot) * keep * p.C + column[e];
+#pragma unroll
+      for (int j = 0; j < kStepTaps; j++) {
+        in[e][j] = j < keep && !fresh ? past[size_t(j) * p.C] : 0.f;
+        w[e][j] = j < keep ? p.taps_w[size_t(j) * p.C + column[e]] : 0.f;
       }
-      a = fmaf(p.taps_w[size_t(p.taps - 1) * p.C + column], v, a);
-      if (p.taps > 1) past[size_t(p.taps - 2) * p.C] = v;
-      T o;
-      from_f(o, vec::gate<T>(a));               // rounded as where the convolution is a kernel of its own
-      v = to_f(o);
     }
-    return v;
-  };
-  const int K = p.kv_heads * p.Dp;
-  for (int i = tid; i < 2 * p.Dp + p.Vp; i += kStepThreads) {
-    if (i < p.Dp) qs[i] = value(p.q, g * p.Dp + i, g * p.Dp + i);
-    else if (i < 2 * p.Dp) ks[i - p.Dp] = value(p.k, g * p.Dp + i - p.Dp, K + g * p.Dp + i - p.Dp);
-    else vs[i - 2 * p.Dp] = value(p.v, h * p.Vp + i - 2 * p.Dp, 2 * K + h * p.Vp + i - 2 * p.Dp);
+#pragma unroll
+    for (int e = 0; e < 2; e++) {
+      const int i = i0 + e * kStepThreads;
+      if (i >= total) continue;
+      float v = cur[e];
+      if (p.taps_w) {
+        float* past = p.conv + size_t(slot) * keep * p.C + column[e];
+        float a = 0.f;
+#pragma unroll
+        for (int j = 0; j < kStepTaps; j++) {
+          a = fmaf(w[e][j], in[e][j], a);
+          if (j > 0 && j < keep) past[size_t(j - 1) * p.C] = in[e][j];
+        }
+        for (int j = kStepTaps; j < keep; j++) {
+          const float x = fresh ? 0.f : past[size_t(j) * p.C];
+          a = fmaf(p.taps_w[size_t(j) * p.C + column[e]], x, a);
+          past[size_t(j - 1) * p.C] = x;
+        }
+        a = fmaf(last[e], v, a);
+        if (keep) past[size_t(keep - 1) * p.C] = v;
+        T o;
+        from_f(o, vec::gate<T>(a));              // rounded as where the convolution is a kernel of its own
+        v = to_f(o);
+      }
+      qs[i] = v;                                 // q, k and v one after the other
+    }
   }
   __syncthreads();
   const float rate = p.rate[h];

@@ -31,6 +31,7 @@ namespace {
 constexpr int kThreads = 512;
 constexpr int kMaxUnits = 16;       // float4 units of a row per thread: width <= 512 * 16 * 4
 constexpr int kMaxTop = 64;
+constexpr int kNear = 3;            // carried inputs of the convolution taken at once
 
 struct ResidualParams {
   // embedding
@@ -106,7 +107,8 @@ __device__ __forceinline__ float block_total(const float* red) {
   return v;
 }
 
-template <typename T, bool EMBED, bool POST, int U>
+// NEAR: with the convolution (an instance of its own: it holds more registers)
+template <typename T, bool EMBED, bool POST, bool NEAR, int U>
 __global__ void __launch_bounds__(kThreads) k_residual(const ResidualParams p) {
   __shared__ float red[16], red_b[16], red_s[16], sw[kMaxTop];
   __shared__ int sp[kMaxTop], so[kMaxTop];
@@ -123,6 +125,25 @@ __global__ void __launch_bounds__(kThreads) k_residual(const ResidualParams p) {
     __syncthreads();
   }
   float* xr = p.x + row * p.ld;
+  // carried inputs of the convolution: requested here where registers allow, long before they are used
+  constexpr bool kEarly = NEAR && U <= 2;
+  float4 pre[kEarly ? U : 1][kNear];
+  float* past = nullptr;
+  bool fresh = true;
+  if constexpr (NEAR) {
+    past = p.past + size_t(p.segs[4 * blockIdx.x + 2]) * (p.taps - 1) * p.ld;
+    fresh = p.positions[row] == 0;
+    if (kEarly) {
+#pragma unroll
+      for (int k = 0; k < U; k++)
+#pragma unroll
+        for (int j = 0; j < kNear; j++) {
+          const int i = threadIdx.x + k * blockDim.x;
+          pre[kEarly ? k : 0][j] = make_float4(0.f, 0.f, 0.f, 0.f);
+          if (i < units && j < p.taps - 1 && !fresh) pre[kEarly ? k : 0][j] = load4(past + size_t(j) * p.ld + i * 4);
+        }
+    }
+  }
   float4 u[U], b[POST ? U : 1];
   if constexpr (POST) {
     float sb = 0.f, sq = 0.f;
@@ -214,12 +235,7 @@ __global__ void __launch_bounds__(kThreads) k_residual(const ResidualParams p) {
     __syncthreads();
   }
   if (!p.h1 && !p.h2) return;
-  float *shift = nullptr, *past = nullptr;
-  bool fresh = true;
-  if (p.near) {
-    past = p.past + size_t(p.segs[4 * blockIdx.x + 2]) * (p.taps - 1) * p.ld;
-    fresh = p.positions[row] == 0;
-  }
+  float* shift = nullptr;
   if (p.mu) {
     shift = p.shift + size_t(p.segs[4 * blockIdx.x + 2]) * p.ld;
     fresh = p.positions[row] == 0;
@@ -233,12 +249,24 @@ __global__ void __launch_bounds__(kThreads) k_residual(const ResidualParams p) {
         const float4 g = load4(p.g1 + i * 4);
         v = make_float4(u[k].x * r * g.x, u[k].y * r * g.y, u[k].z * r * g.z, u[k].w * r * g.w);
       }
-      if (p.near) {
-        float4 c = make_float4(0.f, 0.f, 0.f, 0.f);
-        for (int j = 0; j < p.taps - 1; j++) {
-          const float4 in = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : load4(past + size_t(j) * p.ld + i * 4);
-          mul_add4(c, load4(p.near + size_t(j) * p.ld + i * 4), in);
-          if (j > 0) store4(past + size_t(j - 1) * p.ld + i * 4, in);
+      if constexpr (NEAR) {
+        float4 c = make_float4(0.f, 0.f, 0.f, 0.f), in[kNear], w[kNear];    // loads before stores: one round trip
+#pragma unroll
+        for (int j = 0; j < kNear; j++)
+          if (j < p.taps - 1) {
+            w[j] = load4(p.near + size_t(j) * p.ld + i * 4);
+            in[j] = kEarly ? pre[kEarly ? k : 0][j] : (fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : load4(past + size_t(j) * p.ld + i * 4));
+          }
+#pragma unroll
+        for (int j = 0; j < kNear; j++)
+          if (j < p.taps - 1) {
+            mul_add4(c, w[j], in[j]);
+            if (j > 0) store4(past + size_t(j - 1) * p.ld + i * 4, in[j]);
+          }
+        for (int j = kNear; j < p.taps - 1; j++) {
+          const float4 x = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : load4(past + size_t(j) * p.ld + i * 4);
+          mul_add4(c, load4(p.near + size_t(j) * p.ld + i * 4), x);
+          store4(past + size_t(j - 1) * p.ld + i * 4, x);
         }
         mul_add4(c, load4(p.near + size_t(p.taps - 1) * p.ld + i * 4), v);
         if (p.taps > 1) store4(past + size_t(p.taps - 2) * p.ld + i * 4, v);
@@ -284,8 +312,8 @@ __global__ void __launch_bounds__(256) k_token_shift(const float* __restrict__ h
   for (int s = 0; s < nmix; s++) store4(mixes + (size_t(row) * nmix + s) * ld + i, mix4(v, prev, load4(mu + size_t(s) * ld + i)));
 }
 
-template <typename T, bool EMBED, bool POST>
-cudaError_t launch_u(const ResidualParams& p, int rows, cudaStream_t st) {
+template <typename T, bool EMBED, bool POST, bool NEAR>
+cudaError_t launch_n(const ResidualParams& p, int rows, cudaStream_t st) {
   const int units = p.ld / 4;
   const int per = units <= 64 ? 1 : (units <= kThreads * 2 ? 2 : (units <= kThreads * 4 ? 4 : (units <= kThreads * 8 ? 8 : 16)));
   int threads = ((units + per - 1) / per + 31) / 32 * 32;
@@ -293,12 +321,16 @@ cudaError_t launch_u(const ResidualParams& p, int rows, cudaStream_t st) {
   if (threads < kMaxTop) threads = kMaxTop;
   const dim3 grid(rows), blk(threads);
   switch (per) {
-    case 1: return pdl::launch(k_residual<T, EMBED, POST, 1>, grid, blk, 0, st, 1, p);
-    case 2: return pdl::launch(k_residual<T, EMBED, POST, 2>, grid, blk, 0, st, 1, p);
-    case 4: return pdl::launch(k_residual<T, EMBED, POST, 4>, grid, blk, 0, st, 1, p);
-    case 8: return pdl::launch(k_residual<T, EMBED, POST, 8>, grid, blk, 0, st, 1, p);
-    default: return pdl::launch(k_residual<T, EMBED, POST, 16>, grid, blk, 0, st, 1, p);
+    case 1: return pdl::launch(k_residual<T, EMBED, POST, NEAR, 1>, grid, blk, 0, st, 1, p);
+    case 2: return pdl::launch(k_residual<T, EMBED, POST, NEAR, 2>, grid, blk, 0, st, 1, p);
+    case 4: return pdl::launch(k_residual<T, EMBED, POST, NEAR, 4>, grid, blk, 0, st, 1, p);
+    case 8: return pdl::launch(k_residual<T, EMBED, POST, NEAR, 8>, grid, blk, 0, st, 1, p);
+    default: return pdl::launch(k_residual<T, EMBED, POST, NEAR, 16>, grid, blk, 0, st, 1, p);
   }
+}
+template <typename T, bool EMBED, bool POST>
+cudaError_t launch_u(const ResidualParams& p, int rows, cudaStream_t st) {
+  return p.near ? launch_n<T, EMBED, POST, true>(p, rows, st) : launch_n<T, EMBED, POST, false>(p, rows, st);
 }
 template <typename T>
 cudaError_t launch_t(const ResidualParams& p, int rows, cudaStream_t st) {
