@@ -113,7 +113,9 @@ def kernel_numbers(size: str, T: int, seqs: int, ctx: int, only: str = "") -> li
         q, kk, v = _w(T, C).split((K, K, H * V), 1)
         z, gate, o, beta = torch.rand(T, H * D, device=dev) * 0.1, _w(T, H * V), zeros(T, H * V), wide[:, C + 2 * R:]
         gr = torch.from_numpy(scan_groups(segs.cpu().numpy(), model.scan_group_rows(segs[:, 1].cpu().numpy()))).to(dev)
-        return lambda: ops.delta_scan(q, kk, v, beta, z, gate, rate, norm, st, o, out, segs, pos, groups=gr, **args)
+        size = ops.delta_sets(T, seqs, st)
+        sets = torch.empty(size, dtype=torch.uint8, device=dev) if size else None
+        return lambda: ops.delta_scan(q, kk, v, beta, z, gate, rate, norm, st, o, out, segs, pos, groups=gr, sets=sets, **args)
     matrix = seqs * H * D * V * 4
     if decode:
         k.time("scan", "lugizen delta step (convolution, products, norm, gate)", mk_rec,

@@ -18,6 +18,7 @@
 #include "../pdl.cuh"
 #include "attn_mma.cuh"
 #include "delta.cuh"
+#include "ops.h"
 
 using namespace vec;
 using delta_ops::decay;
@@ -375,9 +376,10 @@ cudaError_t scan(const Params& p, int nseg, cudaStream_t st) {
 extern "C" {
 
 // Many rows per segment: q, k, v [rows, ld] behind convolution and SiLU, beta [rows, ldb], z fp32 [rows, ldz] = softplus of the decay inputs, gate [rows, ldg]; o fp32 scratch [rows, heads * Vp].
-// groups (bf16; null: the sequential kernel): the segments as the chunked kernel takes them, [ngroups, 4].
+// groups (bf16; null: the sequential kernel): the segments as the chunked kernels take them, [ngroups, 4]; sets: scratch of tbv_op_delta_sets bytes, or null (see
+// delta_chunk.cu).
 int tbv_op_delta_scan(const void* q, const void* k, const void* v, const void* beta, const void* z, const void* gate, const void* rate, const void* norm,
-                      void* state, void* o, void* out, const void* segs, const void* positions, const void* groups, int ngroups, int rows, int nseg, int heads,
+                      void* state, void* o, void* out, const void* segs, const void* positions, const void* groups, int ngroups, void* sets, int rows, int nseg, int heads,
                       int kv_heads, int Dp, int Vp, int dim, int vdim, int ld, int ldb, int ldz, int ldg, int ldo, float eps, int bf16, void* stream) {
   if (rows <= 0 || nseg <= 0) return 0;
   Params p{};
@@ -389,7 +391,7 @@ int tbv_op_delta_scan(const void* q, const void* k, const void* v, const void* b
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   cudaError_t e;
   bool finished = false;
-  if (bf16 && groups && delta_ops::chunk_fits(p)) e = delta_ops::chunk_scan(p, static_cast<const int*>(groups), ngroups, &finished, st);
+  if (bf16 && groups && delta_ops::chunk_fits(p)) e = delta_ops::chunk_scan(p, static_cast<const int*>(groups), ngroups, rows, sets, &finished, st);
   else e = bf16 ? scan<__nv_bfloat16>(p, nseg, st) : scan<float>(p, nseg, st);
   if (e == cudaSuccess && !finished) {
     const dim3 grid(unsigned(((long long)rows * heads + 7) / 8));
@@ -397,6 +399,14 @@ int tbv_op_delta_scan(const void* q, const void* k, const void* v, const void* b
   }
   if (e != cudaSuccess) fprintf(stderr, "[tbvops] delta scan launch failed: %s\n", cudaGetErrorString(e));
   return e == cudaSuccess ? 0 : -1;
+}
+
+// Bytes of `sets` that the form for few sequences and heads needs; 0: the sizes do not take the chunked kernels, or the GPU is busy enough without it.
+long long tbv_op_delta_sets(int rows, int ngroups, int heads, int Dp, int Vp) {
+  Params p{};
+  p.heads = heads; p.Dp = Dp; p.Vp = Vp;
+  if (!delta_ops::chunk_fits(p) || 2 * ngroups * heads * ((Vp + 127) / 128) > tbvops::sm_count()) return 0;
+  return (long long)delta_ops::chunk_sets(p, rows, ngroups);
 }
 
 // One row per segment.  beta, low_a, low_g: columns of rows ldx apart; w_a [heads * Dp, rank], b_a [heads * Dp], w_g [heads * Vp, rank].  taps_w [taps, C] (C = the

@@ -38,9 +38,11 @@ inline bool sizes_ok(const Params& p) {
          p.Vp % 16 == 0 && p.dim > 0 && p.dim <= p.Dp && p.vdim > 0 && p.vdim <= p.Vp;
 }
 
-// delta_chunk.cu: many rows of a bf16 model, in chunks on tensor cores; groups [ngroups, 4]: (first row, rows, state slot, flags).  *finished: head norm and gate
-// are done too (p.out), otherwise o is left in p.o.
+// delta_chunk.cu: many rows of a bf16 model, in chunks on tensor cores; groups [ngroups, 4]: (first row, rows, state slot, -), together `rows` rows.  sets:
+// null, or chunk_sets() bytes for the operands of all chunks (the form for few sequences and heads).  *finished: head norm and gate are done too (p.out),
+// otherwise o is left in p.o.
 bool chunk_fits(const Params& p);
-cudaError_t chunk_scan(const Params& p, const int* groups, int ngroups, bool* finished, cudaStream_t st);
+size_t chunk_sets(const Params& p, int rows, int ngroups);
+cudaError_t chunk_scan(const Params& p, const int* groups, int ngroups, int rows, void* sets, bool* finished, cudaStream_t st);
 
 }  // namespace delta_ops

@@ -16,9 +16,14 @@
 // Eight warps of a CTA make the chunks' operands (they do not depend on the state), eight others take them through the products, one or two chunks behind; two sets
 // of operands pass between them.  The two groups meet in named barriers only: `full` (operands of a set are there) and `empty` (its products are done).  If a
 // CTA owns all value columns of its head, head norm, weight and gate follow here as well.
+//
+// With few sequences and heads most of the GPU would idle and every chunk would cost a maker's latency.  Then the two halves are kernels of their own: the sets
+// of all chunks are made in parallel into memory (k_delta_make), and the products, their value columns shared out over several CTAs, find them there
+// (k_delta_multiply: four warps fetch, four sets in flight).
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
+#include <type_traits>
 
 #include "../pdl.cuh"
 #include "attn_mma.cuh"
@@ -36,6 +41,7 @@ namespace {
 
 constexpr int kC = 16, kNW = 8, kNT = kNW * 32, kCols = kNW * 16;    // tokens of a chunk, warps and threads of a group, value columns of a CTA
 constexpr int kParts = 3;
+constexpr int kFetch = 128, kMakeChunks = 8;      // threads that fetch sets; chunks of a CTA that makes them
 
 template <int DK>
 struct Shape {
@@ -48,29 +54,39 @@ struct Shape {
   static constexpr int oQ = 0;                                     // q P                 [2][16][pitch]
   static constexpr int oK = oQ + 2 * kC * kPitch;                  // k P                 [parts][16][pitch]
   static constexpr int oR = oK + kParts * kC * kPitch;             // k R                 [parts][16][pitch]
-  static constexpr int oV = oR + kParts * kC * kPitch;             // v                   [16][vpitch]
-  static constexpr int oA = oV + kC * kVPitch;                     // A                   [2][16][apitch]
+  static constexpr int oA = oR + kParts * kC * kPitch;             // A                   [2][16][apitch]
   static constexpr int oT = oA + 2 * kC * kAPitch;                 // T                   [parts][16][apitch]
   static constexpr int oE = oT + kParts * kC * kAPitch;            // P_16                [DK] fp32
-  static constexpr int oL = oE + DK * 4;                           // diag(beta) B        [16][17] fp32
+  static constexpr int kStored = oE + DK * 4;                      // what a set in memory holds
+  static constexpr int oV = kStored;                               // v                   [16][vpitch]
+  static constexpr int oL = oV + kC * kVPitch;                     // diag(beta) B        [16][17] fp32
   static constexpr int oB = oL + 16 * 17 * 4;                      // step sizes          [16] fp32
   static constexpr int kSet = oB + kC * 4;
-  // dynamic shared memory: two sets, then what one of the groups has for itself
-  static constexpr int oTa = 2 * kSet;                             // blocks: left rows   [parts][2 kinds][16][pitch]  (8 of q, 8 of k)
+  static_assert(kStored % 16 == 0 && kSet % 16 == 0, "16-byte copies");
+};
+// Dynamic shared memory of a CTA that makes operands: its sets, then what the makers have for themselves.
+template <int DK, int SETS, int RAWS>
+struct Layout : Shape<DK> {
+  using B = Shape<DK>;
+  using B::kItems;
+  using B::kPitch;
+  static constexpr int oTa = SETS * B::kSet;                            // blocks: left rows   [parts][2 kinds][16][pitch]  (8 of q, 8 of k)
   static constexpr int oTb = oTa + kParts * 32 * kPitch;           //         right rows  [parts][2 kinds][8][pitch]
-  static constexpr int oZ = oTb + kParts * 16 * kPitch;            // raw decay inputs [16][DK] fp32, q and k [16][DK] bf16 each; two chunks
+  static constexpr int oZ = oTb + kParts * 16 * kPitch;            // raw decay inputs [16][DK] fp32, q and k [16][DK] bf16 each; RAWS chunks
   static constexpr int kRq = kC * DK * 4, kRk = kRq + kC * DK * 2, kRaw = kRk + kC * DK * 2;
-  static constexpr int oF = oZ + 2 * kRaw;                         // factors of q, of k, step sizes [2 chunks][3][16] fp32
+  static constexpr int oF = oZ + RAWS * kRaw;                         // factors of q, of k, step sizes [2 chunks][3][16] fp32
   static constexpr int oTri = oF + 6 * kC * 4;                     // diagonal blocks     [items][4 quarters][16] fp32
   static constexpr int oOff = oTri + (kItems + 1) * 256;           // the other blocks' sums [warps][2][16][8] fp32
   static constexpr int oI = oOff + kNW * 1024;                     // I + diag(beta) B inverted [16][17] fp32, a product [8][17]
-  static constexpr int oO = oI + 24 * 17 * 4;                      // o                   [16][opitch] fp32
-  static constexpr int kBytes = oO + kC * kOPitch * 4;
-  static_assert(kSet % 16 == 0 && oO % 16 == 0 && kBytes <= int(kMaxSmem), "shared memory");
+  static constexpr int oO = oI + 24 * 17 * 4;                      // o                   [16][opitch] fp32 (both halves in one kernel)
+  static constexpr int kBytes = oO + (SETS == 2 ? kC * B::kOPitch * 4 : 0);
+  static_assert(oTa % 16 == 0 && oZ % 16 == 0 && oF % 16 == 0 && oO % 16 == 0 && kBytes <= (SETS == 2 ? int(kMaxSmem) : 113 * 1024), "shared memory; two CTAs per SM");
 };
+template <int DK> using Both = Layout<DK, 2, 2>;
+template <int DK> using Make = Layout<DK, 1, 1>;
 
-// Named barriers (0 is __syncthreads): one inside each group, `full` and `empty` of each set of operands.
-enum Bar : int { kMakers = 1, kProducts = 2, kFull = 3, kEmpty = 5 };
+// Named barriers (0 is __syncthreads): one inside each group, `full` and `empty` of up to four sets of operands.
+enum Bar : int { kMakers = 1, kProducts = 2, kFull = 3, kEmpty = 7 };
 __device__ __forceinline__ void bar_sync(int id, int threads) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
 __device__ __forceinline__ void bar_arrive(int id, int threads) { asm volatile("bar.arrive %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
 
@@ -117,11 +133,32 @@ struct Job {                        // what one CTA works on, and where a thread
   int h, g, first, n, nc, slot, vb, cols;  // vb: first of its value columns
   int tid, warp, lane, row16, l16;  // 16 lanes per row of a chunk
 };
+__device__ __forceinline__ Job job_of(const Params& p, const int* group, int h, int vb, int cols, int tid) {
+  Job w;
+  w.h = h;
+  w.g = h / (p.heads / p.kv_heads);
+  w.first = group[0];
+  w.n = group[1];
+  w.slot = group[2];
+  w.nc = (w.n + kC - 1) / kC;
+  w.vb = vb;
+  w.cols = cols;
+  w.tid = tid;
+  w.warp = tid >> 5;
+  w.lane = tid & 31;
+  w.row16 = tid >> 4;
+  w.l16 = tid & 15;
+  return w;
+}
+// Sets in memory: that of chunk c of group gi, head h is number (first / 16 + gi + c) * heads + h (different for all chunks of a batch).
+__device__ __forceinline__ int first_set(const Job& w, int gi) { return w.first / kC + gi; }
 
 // ---- the makers -----------------------------------------------------------------------------------------------------------
-template <int DK>
-__device__ __forceinline__ void make_operands(const Params& p, uint8_t* sm, const Job& w) {
-  using S = Shape<DK>;
+// Chunks c0 .. c1 - 1.  sets null: they go to the products of this CTA; otherwise to memory, chunk c to sets + c * stride.
+template <int DK, bool STORE>
+__device__ __forceinline__ void make_operands(const Params& p, uint8_t* sm, const Job& w, int c0, int c1, uint8_t* sets, size_t stride) {
+  using S = typename std::conditional<STORE, Make<DK>, Both<DK>>::type;
+  constexpr int kRaws = STORE ? 0 : 1;          // mask of the raw buffers
   const int tid = w.tid, warp = w.warp, lane = w.lane, r8 = lane >> 2, quad = lane & 3, row16 = w.row16, l16 = w.l16, n = w.n;
   const uint32_t base = smem_addr(sm);
   const float rate2 = -p.rate[w.h] * kLog2e, qscale = rsqrtf(float(p.dim));
@@ -133,7 +170,7 @@ __device__ __forceinline__ void make_operands(const Params& p, uint8_t* sm, cons
   // rows of chunk c on their way to shared memory; missing rows are zeros: they decay nothing, write nothing and read nothing
   auto issue = [&](int c) {
     const size_t r = size_t(w.first + c * kC + row16);
-    const uint32_t raw = base + S::oZ + (c & 1) * S::kRaw;
+    const uint32_t raw = base + S::oZ + (c & kRaws) * S::kRaw;
     if (c * kC + row16 >= n) {
       for (int x = l16; x < DK / 4; x += 16) st_zero16(raw + (row16 * DK + x * 4) * 4);
       for (int x = l16; x < DK / 4; x += 16) st_zero16(raw + S::kRq + (x >= DK / 8 ? S::kRk - S::kRq : 0) + (row16 * DK + x % (DK / 8) * 8) * 2);
@@ -158,7 +195,7 @@ __device__ __forceinline__ void make_operands(const Params& p, uint8_t* sm, cons
   // factors that make rows of q and k unit vectors (of rows that this thread's own copies brought), step sizes
   auto factors_of = [&](int c) { return reinterpret_cast<float*>(sm + S::oF) + (c & 1) * 3 * kC; };
   auto norms = [&](int c) {
-    const uint8_t* raw = sm + S::oZ + (c & 1) * S::kRaw;
+    const uint8_t* raw = sm + S::oZ + (c & kRaws) * S::kRaw;
     float *factors = factors_of(c), sq = 0.f, sk = 0.f;
     for (int x = l16; x < p.Dp / 8; x += 16) {
       float f[8], k[8];
@@ -186,7 +223,7 @@ __device__ __forceinline__ void make_operands(const Params& p, uint8_t* sm, cons
   const bool odd = quarter & 1, late = quarter & 2, item = warp * 16 < p.Dp;
   auto scores = [&](int c) {
     if (!item) return;
-    const uint8_t* raw = sm + S::oZ + (c & 1) * S::kRaw;
+    const uint8_t* raw = sm + S::oZ + (c & kRaws) * S::kRaw;
     const float* factors = factors_of(c);
     f32x2 a[4], q[4], k[4];
 #pragma unroll
@@ -326,61 +363,7 @@ __device__ __forceinline__ void make_operands(const Params& p, uint8_t* sm, cons
     reinterpret_cast<float*>(set_p + S::oL)[t * 17 + s] = s < t ? vk * factors[2 * kC + t] : 0.f;
     if (tid < kC) reinterpret_cast<float*>(set_p + S::oB)[tid] = factors[2 * kC + tid];
   };
-  issue(0);
-  cp_async_commit();
-  fetch_beta(0);
-  for (int i = tid; i < S::oZ / 16; i += kNT) st_zero16(base + i * 16);     // operand rows of channels beyond Dp stay zero
-  cp_async_wait<0>();
-  norms(0);
-  bar_sync(kMakers, kNT);
-  for (int c = 0; c < w.nc; c++) {                                  // the raw rows of chunk c are there, and their factors
-    const int b = c & 1;
-    uint8_t* set_p = sm + b * S::kSet;
-    const uint32_t set = base + b * S::kSet;
-    if (c + 1 < w.nc) {
-      issue(c + 1);
-      fetch_beta(c + 1);
-    }
-    cp_async_commit();
-    scores(c);
-    bar_sync(kMakers, kNT);
-    if (c >= 2) bar_sync(kEmpty + b, 2 * kNT);                      // the products of chunk c - 2 are done
-    issue_v(c, set);
-    cp_async_commit();
-    blocks();
-    operands(set, set_p);
-    bar_sync(kMakers, kNT);
-    assemble(set_p, factors_of(c));
-    if (c + 1 < w.nc) {
-      cp_async_wait<1>();
-      norms(c + 1);
-    }
-    bar_sync(kMakers, kNT);
-    cp_async_wait<0>();                                             // v
-    bar_arrive(kFull + b, 2 * kNT);
-  }
-}
-
-// ---- the products -----------------------------------------------------------------------------------------------------------
-template <int DK>
-__device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job& w) {
-  using S = Shape<DK>;
-  const int lane = w.lane, r8 = lane >> 2, quad = lane & 3, row16 = w.row16, l16 = w.l16, n = w.n;
-  const uint32_t base = smem_addr(sm);
-  const bool fresh = p.positions[w.first] == 0, fused = p.o == nullptr;
-  const int v0 = w.vb + w.warp * 16;                                // first value column of the warp
-  const bool mma_warp = w.warp * 16 < w.cols && v0 < p.Vp;
-  float st[DK / 8][4];      // S^T: value column v0 + r8 (+ 8), channels 8 i + 2 quad (+ 1)
-  float* state = p.state + (size_t(w.slot) * p.heads + w.h) * p.Dp * p.Vp;
-#pragma unroll
-  for (int i = 0; i < DK / 8; i++)
-#pragma unroll
-    for (int j = 0; j < 4; j++) {
-      const int d = i * 8 + quad * 2 + (j & 1), v = v0 + r8 + (j >> 1) * 8;
-      st[i][j] = !mma_warp || fresh || d >= p.Dp ? 0.f : state[size_t(d) * p.Vp + v];
-    }
-  const uint32_t brow = (lane & 7) + ((lane >> 4) << 3), bcol = ((lane >> 3) & 1) * 16;    // right operands stored [n][k]
-  // T, by one warp (the last one, which has no columns of its own where they are shared out)
+  // T, by one warp
   auto invert = [&](uint32_t set, const uint8_t* set_p) {
     const float *L = reinterpret_cast<const float*>(set_p + S::oL), *beta = reinterpret_cast<const float*>(set_p + S::oB);
     float *I = reinterpret_cast<float*>(sm + S::oI), *M = I + 16 * 17;
@@ -428,19 +411,86 @@ __device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job
     out(8 + r8, c, m0, m1);
     out(8 + r8, 8 + c, I[(8 + r8) * 17 + 8 + c], I[(8 + r8) * 17 + 8 + c + 1]);
   };
+  issue(c0);
+  cp_async_commit();
+  fetch_beta(c0);
+  for (int i = tid; i < S::oZ / 16; i += kNT) st_zero16(base + i * 16);     // operand rows of channels beyond Dp stay zero
+  cp_async_wait<0>();
+  norms(c0);
+  bar_sync(kMakers, kNT);
+  for (int c = c0; c < c1; c++) {                                   // the raw rows of chunk c are there, and their factors
+    const int b = STORE ? 0 : c & 1;
+    uint8_t* set_p = sm + b * S::kSet;
+    const uint32_t set = base + b * S::kSet;
+    auto next = [&]() {
+      if (c + 1 < c1) {
+        issue(c + 1);
+        fetch_beta(c + 1);
+      }
+      cp_async_commit();
+    };
+    if (!STORE) next();
+    scores(c);
+    bar_sync(kMakers, kNT);
+    if (STORE) next();                                              // into the rows just read
+    if (!STORE) {
+      if (c >= 2) bar_sync(kEmpty + b, 2 * kNT);                    // the products of chunk c - 2 are done
+      issue_v(c, set);
+      cp_async_commit();
+    }
+    blocks();
+    operands(set, set_p);
+    bar_sync(kMakers, kNT);
+    assemble(set_p, factors_of(c));
+    if (c + 1 < c1) {
+      cp_async_wait<STORE ? 0 : 1>();
+      norms(c + 1);
+    }
+    bar_sync(kMakers, kNT);
+    if (warp == 0) invert(set, set_p);
+    if (STORE) {
+      bar_sync(kMakers, kNT);
+      uint4* to = reinterpret_cast<uint4*>(sets + c * stride);
+      for (int i = tid; i < S::kStored / 16; i += kNT) to[i] = reinterpret_cast<const uint4*>(set_p)[i];
+    } else {
+      cp_async_wait<0>();                                           // v
+      bar_arrive(kFull + b, 2 * kNT);
+    }
+  }
+  cp_async_wait<0>();
+}
+
+// ---- the products -----------------------------------------------------------------------------------------------------------
+// SETS 2: beside the makers, o of a chunk stays here for its norm if p.o is null.  SETS 4: beside the warps that fetch.
+template <int DK, int SETS>
+__device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job& w) {
+  using S = Both<DK>;
+  constexpr int kMeet = SETS == 2 ? 2 * kNT : kNT + kFetch;        // threads that meet in a barrier of a set
+  const int lane = w.lane, r8 = lane >> 2, quad = lane & 3, row16 = w.row16, l16 = w.l16, n = w.n;
+  const uint32_t base = smem_addr(sm);
+  const bool fresh = p.positions[w.first] == 0, fused = SETS == 2 && p.o == nullptr;
+  const int v0 = w.vb + w.warp * 16;                                // first value column of the warp
+  const bool mma_warp = w.warp * 16 < w.cols && v0 < p.Vp;
+  float st[DK / 8][4];      // S^T: value column v0 + r8 (+ 8), channels 8 i + 2 quad (+ 1)
+  float* state = p.state + (size_t(w.slot) * p.heads + w.h) * p.Dp * p.Vp;
+#pragma unroll
+  for (int i = 0; i < DK / 8; i++)
+#pragma unroll
+    for (int j = 0; j < 4; j++) {
+      const int d = i * 8 + quad * 2 + (j & 1), v = v0 + r8 + (j >> 1) * 8;
+      st[i][j] = !mma_warp || fresh || d >= p.Dp ? 0.f : state[size_t(d) * p.Vp + v];
+    }
+  const uint32_t brow = (lane & 7) + ((lane >> 4) << 3), bcol = ((lane >> 3) & 1) * 16;    // right operands stored [n][k]
   for (int c = 0; c < w.nc; c++) {
-    const int b = c & 1, at = c * kC;
+    const int b = c % SETS, at = c * kC;
     const uint32_t set = base + b * S::kSet;
     vec::Raw8<__nv_bfloat16> gate;
     if (fused && at + row16 < n && l16 * 8 < p.Vp)
       gate.load(static_cast<const __nv_bfloat16*>(p.gate) + size_t(w.first + at + row16) * p.ldg + size_t(w.h) * p.Vp + l16 * 8);
-    bar_sync(kFull + b, 2 * kNT);
-    if (w.warp == kNW - 1) invert(set, sm + b * S::kSet);
-    uint32_t l[kParts][4], f[4];
-    float o[2][2][4] = {};
+    bar_sync(kFull + b, kMeet);
     if (mma_warp) {
       // (q P) S and (k P) S, two sums each for even and odd k steps: value column as above, tokens 8 i + 2 quad (+ 1)
-      float x[2][2][4] = {};
+      float o[2][2][4] = {}, x[2][2][4] = {};
 #pragma unroll
       for (int ks = 0; ks < DK / 16; ks += 2) {
         uint32_t s[2][kParts][4], r[2][4];
@@ -471,6 +521,7 @@ __device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job
             }
         }
       }
+      uint32_t l[kParts][4], f[4];
       ldmatrix_x4_trans(set + S::oV + brow * S::kVPitch + w.warp * 32 + bcol, f);      // v^T: stored [token][column]
 #pragma unroll
       for (int j = 0; j < 4; j++) {
@@ -479,11 +530,8 @@ __device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job
         y[0] = __uint_as_float(f[j] << 16) - (y[0] + z[0]);
         y[1] = __uint_as_float(f[j] & 0xffff0000u) - (y[1] + z[1]);
       }
-      as_left<kParts>(x[0], l);
-    }
-    bar_sync(kProducts, kNT);                                       // T is there
-    if (mma_warp) {
       float u[2][4] = {};
+      as_left<kParts>(x[0], l);
 #pragma unroll
       for (int j = kParts - 1; j >= 0; j--) {
         ldmatrix_x4(set + S::oT + (j * kC + brow) * S::kAPitch + bcol, f);
@@ -533,7 +581,7 @@ __device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job
           else if (at + t < n) p.o[(size_t(w.first + at + t) * p.heads + w.h) * p.Vp + v0 + v] = y;
         }
     }
-    if (c + 2 < w.nc) bar_arrive(kEmpty + b, 2 * kNT);
+    if (c + SETS < w.nc) bar_arrive(kEmpty + b, kMeet);
     if (!fused) continue;
     // head norm, weight and gate; a row per 16 lanes, 8 columns per lane.  (The next chunk's o is written behind its `full`, which waits for all of these warps.)
     bar_sync(kProducts, kNT);
@@ -569,45 +617,107 @@ __device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job
   }
 }
 
+// Four warps that bring sets from memory, and the values of their columns, three chunks ahead.
 template <int DK>
-__global__ void __launch_bounds__(2 * kNT, 1) k_delta_chunk(const Params p, const int* groups, int cols) {
+__device__ __forceinline__ void fetch_operands(const Params& p, uint8_t* sm, const Job& w, const uint8_t* sets, size_t stride) {
+  using S = Shape<DK>;
+  const uint32_t base = smem_addr(sm);
+  const int units = min(w.cols, p.Vp - w.vb) / 8;
+  const __nv_bfloat16* vg = static_cast<const __nv_bfloat16*>(p.v) + size_t(w.h) * p.Vp + w.vb;
+  auto issue = [&](int c) {
+    if (c < w.nc) {
+      const uint32_t set = base + (c & 3) * S::kSet;
+      const uint8_t* from = sets + c * stride;
+      for (int i = w.tid; i < S::kStored / 16; i += kFetch) cp_async16(set + i * 16, from + i * 16);
+      for (int i = w.tid; i < kC * units; i += kFetch) {            // missing rows are zeros
+        const int t = i / units, x = i - t * units;
+        const uint32_t dst = set + S::oV + t * S::kVPitch + x * 16;
+        if (c * kC + t < w.n) cp_async16(dst, vg + size_t(w.first + c * kC + t) * p.ld + x * 8);
+        else st_zero16(dst);
+      }
+    }
+    cp_async_commit();
+  };
+  for (int c = 0; c < 3; c++) issue(c);
+  for (int c = 0; c < w.nc; c++) {
+    cp_async_wait<2>();                                             // chunk c
+    bar_arrive(kFull + (c & 3), kNT + kFetch);
+    if (c >= 1 && c + 3 < w.nc) bar_sync(kEmpty + ((c + 3) & 3), kNT + kFetch);   // the products of chunk c - 1 are done
+    issue(c + 3);
+  }
+  cp_async_wait<0>();
+}
+
+// registers of the launch, 128 per thread, shared out anew
+template <int N> __device__ __forceinline__ void more_registers() { asm volatile("setmaxnreg.inc.sync.aligned.u32 %0;" ::"n"(N)); }
+template <int N> __device__ __forceinline__ void fewer_registers() { asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;" ::"n"(N)); }
+
+template <int DK>
+__global__ void __launch_bounds__(2 * kNT, 1) k_delta_chunk(const Params p, const int* groups) {
   extern __shared__ __align__(16) uint8_t sm[];
   pdl::launch_dependents();
   pdl::grid_dependency_wait();
-  Job w;
-  w.h = blockIdx.y;
-  w.g = w.h / (p.heads / p.kv_heads);
-  w.first = groups[4 * blockIdx.x];
-  w.n = groups[4 * blockIdx.x + 1];
-  w.slot = groups[4 * blockIdx.x + 2];
-  w.nc = (w.n + kC - 1) / kC;
-  w.vb = blockIdx.z * cols;
-  w.cols = cols;
-  w.tid = threadIdx.x % kNT;
-  w.warp = w.tid >> 5;
-  w.lane = w.tid & 31;
-  w.row16 = w.tid >> 4;
-  w.l16 = w.tid & 15;
-  // registers of the launch, 128 per thread, shared out anew
+  const Job w = job_of(p, groups + 4 * blockIdx.x, blockIdx.y, blockIdx.z * kCols, kCols, threadIdx.x % kNT);
   if (threadIdx.x < kNT) {
-    asm volatile("setmaxnreg.inc.sync.aligned.u32 152;");
-    multiply<DK>(p, sm, w);
+    more_registers<152>();
+    multiply<DK, 2>(p, sm, w);
   } else {
-    asm volatile("setmaxnreg.dec.sync.aligned.u32 104;");
-    make_operands<DK>(p, sm, w);
+    fewer_registers<104>();
+    make_operands<DK, false>(p, sm, w, 0, w.nc, nullptr, 0);
+  }
+}
+
+// CTA (x, head): the sets numbered x * kMakeChunks .. of all groups
+template <int DK>
+__global__ void __launch_bounds__(kNT, 2) k_delta_make(const Params p, const int* groups, int ngroups, uint8_t* sets) {
+  extern __shared__ __align__(16) uint8_t sm[];
+  pdl::launch_dependents();
+  pdl::grid_dependency_wait();
+  const size_t stride = size_t(p.heads) * Shape<DK>::kStored;
+  for (int gi = 0; gi < ngroups; gi++) {
+    const Job w = job_of(p, groups + 4 * gi, blockIdx.y, 0, kCols, threadIdx.x);
+    const int s0 = first_set(w, gi), c0 = max(0, int(blockIdx.x) * kMakeChunks - s0), c1 = min(w.nc, int(blockIdx.x + 1) * kMakeChunks - s0);
+    if (c0 < c1) {
+      make_operands<DK, true>(p, sm, w, c0, c1, sets + s0 * stride + size_t(w.h) * Shape<DK>::kStored, stride);
+      __syncthreads();
+    }
   }
 }
 
 template <int DK>
-cudaError_t launch(Params p, const int* groups, int ngroups, bool* finished, cudaStream_t st) {
-  static bool done = false;
-  // few CTAs: the value columns of a head are shared out (every CTA makes the operands), and the head norm becomes a kernel of its own
+__global__ void __launch_bounds__(kNT + kFetch, 1) k_delta_multiply(const Params p, const int* groups, const uint8_t* sets, int cols) {
+  extern __shared__ __align__(16) uint8_t sm[];
+  pdl::launch_dependents();
+  pdl::grid_dependency_wait();
+  const Job w = job_of(p, groups + 4 * blockIdx.x, blockIdx.y, blockIdx.z * cols, cols, threadIdx.x % kNT);
+  const size_t stride = size_t(p.heads) * Shape<DK>::kStored;
+  if (threadIdx.x < kNT) multiply<DK, 4>(p, sm, w);
+  else fetch_operands<DK>(p, sm, w, sets + first_set(w, blockIdx.x) * stride + size_t(w.h) * Shape<DK>::kStored, stride);
+}
+
+template <int DK>
+size_t sets_bytes(const Params& p, int rows, int ngroups) { return size_t(rows / kC + ngroups + 1) * p.heads * Shape<DK>::kStored; }
+
+template <int DK>
+cudaError_t launch(Params p, const int* groups, int ngroups, int rows, uint8_t* sets, bool* finished, cudaStream_t st) {
+  static bool done[3] = {};
+  cudaError_t e;
+  if (!sets) {
+    *finished = p.Vp <= kCols;
+    if (*finished) p.o = nullptr;
+    e = allow_smem(k_delta_chunk<DK>, Both<DK>::kBytes, &done[0]);
+    return e != cudaSuccess ? e : pdl::launch(k_delta_chunk<DK>, dim3(ngroups, p.heads, (p.Vp + kCols - 1) / kCols), dim3(2 * kNT), Both<DK>::kBytes, st, 1, p, groups);
+  }
+  *finished = false;
+  e = allow_smem(k_delta_make<DK>, Make<DK>::kBytes, &done[1]);
+  const int all = rows / kC + ngroups;
+  if (e == cudaSuccess) e = pdl::launch(k_delta_make<DK>, dim3((all + kMakeChunks - 1) / kMakeChunks, p.heads), dim3(kNT), Make<DK>::kBytes, st, 1, p, groups, ngroups, sets);
+  // as many CTAs per head as find room: the fewer value columns, the shorter a chunk's products
   int cols = kCols;
-  while (cols > 32 && cols / 2 < p.Vp && 2 * ngroups * p.heads * ((p.Vp + cols - 1) / cols) <= tbvops::sm_count()) cols /= 2;
-  *finished = p.Vp <= cols;
-  if (*finished) p.o = nullptr;
-  cudaError_t e = allow_smem(k_delta_chunk<DK>, Shape<DK>::kBytes, &done);
-  return e != cudaSuccess ? e : pdl::launch(k_delta_chunk<DK>, dim3(ngroups, p.heads, (p.Vp + cols - 1) / cols), dim3(2 * kNT), Shape<DK>::kBytes, st, 1, p, groups, cols);
+  while (cols > 32 && cols / 2 < p.Vp && ngroups * p.heads * ((p.Vp + cols / 2 - 1) / (cols / 2)) <= tbvops::sm_count()) cols /= 2;
+  if (e == cudaSuccess) e = allow_smem(k_delta_multiply<DK>, 4 * Shape<DK>::kSet, &done[2]);
+  return e != cudaSuccess ? e : pdl::launch(k_delta_multiply<DK>, dim3(ngroups, p.heads, (p.Vp + cols - 1) / cols), dim3(kNT + kFetch), 4 * Shape<DK>::kSet, st, 1, p, groups,
+                                            static_cast<const uint8_t*>(sets), cols);
 }
 
 }  // namespace
@@ -616,10 +726,15 @@ namespace delta_ops {
 
 bool chunk_fits(const Params& p) { return p.Dp <= 128; }
 
-cudaError_t chunk_scan(const Params& p, const int* groups, int ngroups, bool* finished, cudaStream_t st) {
-  if (p.Dp <= 32) return launch<32>(p, groups, ngroups, finished, st);
-  if (p.Dp <= 64) return launch<64>(p, groups, ngroups, finished, st);
-  return launch<128>(p, groups, ngroups, finished, st);
+size_t chunk_sets(const Params& p, int rows, int ngroups) {
+  return p.Dp <= 32 ? sets_bytes<32>(p, rows, ngroups) : (p.Dp <= 64 ? sets_bytes<64>(p, rows, ngroups) : sets_bytes<128>(p, rows, ngroups));
+}
+
+cudaError_t chunk_scan(const Params& p, const int* groups, int ngroups, int rows, void* sets, bool* finished, cudaStream_t st) {
+  uint8_t* s = static_cast<uint8_t*>(sets);
+  if (p.Dp <= 32) return launch<32>(p, groups, ngroups, rows, s, finished, st);
+  if (p.Dp <= 64) return launch<64>(p, groups, ngroups, rows, s, finished, st);
+  return launch<128>(p, groups, ngroups, rows, s, finished, st);
 }
 
 }  // namespace delta_ops

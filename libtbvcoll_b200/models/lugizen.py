@@ -103,6 +103,14 @@ class Lugizen(StreamDecoder, LatentAttention):
             return 0
         return -(-int(rows.max()) // self.SCAN_CHUNK) * self.SCAN_CHUNK
 
+    def _sets_scratch(self, size: int) -> Optional[torch.Tensor]:
+        """Operands of all chunks of a recurrence, grown on demand (never inside a captured step)."""
+        if not size:
+            return None
+        if "sets" not in self._flat or self._flat["sets"].numel() < size:
+            self._flat["sets"] = torch.empty(size, dtype=torch.uint8, device=self.device)
+        return self._flat["sets"]
+
     def layer_splits(self, m, rows: int, splits: int) -> int:
         """CTAs per row of an attention layer, at most ``splits``: what runs at once (an SM holds two CTAs of the kernel over paired rows, one over latents), and at
         least 64 visible keys for each."""
@@ -134,7 +142,8 @@ class Lugizen(StreamDecoder, LatentAttention):
             z, gate = self._buf("z", T, w[p + "a2"].shape[0]), self._buf("gate", T, V)
             ops.linear(low_a, w[p + "a2"], z, bias=w[p + "dt_bias"], act=ops.ACT_SOFTPLUS)
             ops.linear(low_g, w[p + "g2"], gate)
-            ops.delta_scan(q, k, v, beta, z, gate, w[p + "rate"], w[p + "norm"], self.state[i], self._buf("o", T, V), out, b.segs, b.positions, groups=b.scan_groups, **args)
+            ops.delta_scan(q, k, v, beta, z, gate, w[p + "rate"], w[p + "norm"], self.state[i], self._buf("o", T, V), out, b.segs, b.positions, groups=b.scan_groups,
+                           sets=None if b.scan_groups is None else self._sets_scratch(ops.delta_sets(T, b.scan_groups.shape[0], self.state[i])), **args)
         return self._project(b, i, out)
 
     def _attention(self, b: StepBatch, i: int, m: HeadAttentionSpec) -> dict:

@@ -60,7 +60,9 @@ def lib():
     l.tbv_op_latent_prep.argtypes = [c_vp] * 9 + [I] * 14 + [F, F, I, c_vp]
     l.tbv_op_latent_attn_rows.argtypes = [c_vp] * 7 + [I] * 8 + [F, I, I, c_vp]
     l.tbv_op_short_conv.argtypes = [c_vp] * 7 + [I] * 7 + [c_vp]
-    l.tbv_op_delta_scan.argtypes = [c_vp] * 14 + [I] * 14 + [F, I, c_vp]
+    l.tbv_op_delta_scan.argtypes = [c_vp] * 14 + [I, c_vp] + [I] * 13 + [F, I, c_vp]
+    l.tbv_op_delta_sets.argtypes = [I] * 5
+    l.tbv_op_delta_sets.restype = LL
     l.tbv_op_delta_step.argtypes = [c_vp] * 17 + [I] * 12 + [F, I, c_vp]
     l.tbv_op_head_attn_prep.argtypes = [c_vp] * 9 + [I] * 10 + [F, I, c_vp]
     l.tbv_op_latent_gather.argtypes = [c_vp] * 4 + [I] * 3 + [c_vp]
@@ -455,7 +457,7 @@ def prefill_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
     return out
 
 
-from .mixers import (DECAY_RANK_MAX, SHARED_PREFILL_MAX_DIM, causal_conv_silu, decay_powers, decay_scan, decay_step, delta_scan, delta_step,  # noqa: E402,F401
+from .mixers import (DECAY_RANK_MAX, SHARED_PREFILL_MAX_DIM, causal_conv_silu, decay_powers, decay_scan, decay_step, delta_scan, delta_sets, delta_step,  # noqa: E402,F401
                      fixed_decay_scan, fixed_decay_step, fixed_decay_sums, frequency_turns, head_attention_prep, hyper_embed, hyper_mix,
                      latent_attention_prefill, latent_attention_rows, latent_gather, latent_prefill_fits, latent_prep, latent_row, moe_place_table, moe_route,
                      moe_table_layers, paired_attention_prefill, paired_attention_prep, paired_attention_rows, paired_prefill_fits, position_turns, residual,

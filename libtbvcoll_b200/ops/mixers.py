@@ -297,22 +297,31 @@ def fixed_decay_step(q, k, v, g, norm, powers, state, out, sums, segs, positions
 
 
 # ---- gated delta rule with a decay per key channel -----------------------------------------------------------------------------------
-def delta_scan(q, k, v, beta, z, gate, rate, norm, state, o, out, segs, positions, kv_heads: int, dim: int, vdim: int, eps: float, groups=None) -> None:
+def delta_sets(rows: int, groups: int, state: torch.Tensor) -> int:
+    """Bytes of scratch with which ``delta_scan`` makes the operands of all chunks in parallel; 0 where the sizes do not allow it or enough sequences and heads
+    keep the GPU busy."""
+    _, H, Dp, Vp = state.shape
+    return lib().tbv_op_delta_sets(rows, groups, H, Dp, Vp)
+
+
+def delta_scan(q, k, v, beta, z, gate, rate, norm, state, o, out, segs, positions, kv_heads: int, dim: int, vdim: int, eps: float, groups=None, sets=None) -> None:
     """Per head, q and k of its key head made unit vectors (q times dim^-0.5), S' = diag(exp(-rate z_t)) S_{t-1}, u = sigmoid(beta_t) (v_t - S'^T k_t),
     S_t = S' + k_t u^T over the rows of every segment; out = RMSNorm(S_t^T q_t) * norm * sigmoid(gate).
 
     q, k [rows, kv_heads * Dp] and v [rows, heads * Vp]: column views of one buffer, behind convolution and SiLU; beta [rows, >= heads], gate [rows, heads * Vp] in the
     activation type; z fp32 [rows, heads * Dp] (softplus of the decay inputs), rate fp32 [heads], norm fp32 [Vp]; state fp32 [slots, heads, Dp, Vp] is replaced; o fp32 scratch [rows, heads * Vp].
-    ``groups`` (bf16): the segments, int32 [n, 4] (engine.batch.scan_groups), for the chunked tensor-core kernel where the sizes allow."""
+    ``groups`` (bf16): the segments, int32 [n, 4] (engine.batch.scan_groups), for the chunked tensor-core kernels where the sizes allow; ``sets``: uint8 scratch of
+    ``delta_sets`` bytes (16-byte aligned) for their form with few sequences and heads."""
     _, H, Dp, Vp = state.shape
     rows = q.shape[0]
     assert q.stride(0) == k.stride(0) == v.stride(0) and q.shape[1] == k.shape[1] == kv_heads * Dp and v.shape[1] == gate.shape[1] == H * Vp and z.shape[1] == H * Dp
     assert state.dtype is z.dtype is rate.dtype is norm.dtype is o.dtype is torch.float32 and o.numel() >= rows * H * Vp and norm.shape[0] == Vp and rate.shape[0] == H
+    assert sets is None or (groups is not None and sets.dtype is torch.uint8)
     assert q.dtype is beta.dtype is gate.dtype is out.dtype and beta.shape[1] >= H and (groups is None or (q.dtype is torch.bfloat16 and groups.dtype is torch.int32))
     _chk(lib().tbv_op_delta_scan(_p(q), _p(k), _p(v), _p(beta), _p(z), _p(gate), _p(rate), _p(norm), _p(state), _p(o), _p(out), _p(segs), _p(positions), _p(groups),
-                                 0 if groups is None else groups.shape[0], rows, segs.shape[0], H, kv_heads, Dp, Vp, dim, vdim, q.stride(0), beta.stride(0), z.stride(0),
+                                 0 if groups is None else groups.shape[0], _p(sets), rows, segs.shape[0], H, kv_heads, Dp, Vp, dim, vdim, q.stride(0), beta.stride(0), z.stride(0),
                                  gate.stride(0), out.stride(0), eps, _is_bf16(q), _st()), "tbv_op_delta_scan")
-    _count(2)
+    _count(1 if sets is None and Vp <= 128 and Dp <= 128 and groups is not None else (3 if sets is not None else 2))
 
 
 def delta_step(q, k, v, beta, low_a, low_g, w_a, b_a, w_g, rate, norm, state, out, segs, positions, kv_heads: int, dim: int, vdim: int, eps: float, conv=None) -> None:

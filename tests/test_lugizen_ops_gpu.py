@@ -335,15 +335,19 @@ class Delta:
     def common(self):
         return dict(kv_heads=self.G, dim=self.D, vdim=self.V, eps=self.eps)
 
-    def scan(self, rows, segs, pos, state, chunked):
+    def scan(self, rows, segs, pos, state, form):
+        """``form``: sequential, chunks (one kernel) or apart (operands of all chunks first)."""
         from libtbvcoll_b200 import ops
         q, k, v, al, gl, beta = self.split(self.wide(rows))
         T, n = q.shape[0], self.H
         z = padded(oracle.softplus((self.al[rows].double() @ self.wa.double().T + self.ba.double())).float().view(-1, n, self.D), self.Dp, F32).flatten(1)
         gate = pad_heads((self.gl[rows].double() @ self.wg.double().T).float().view(-1, n, self.V), self.dtype)
         out = torch.zeros(T, n * self.Vp, dtype=self.dtype, device=DEV)
+        size = ops.delta_sets(T, segs.shape[0], state) if form == "apart" else 0
+        sets = torch.full((size,), 255, dtype=torch.uint8, device=DEV) if size else None        # NaN wherever it is not written
+        assert sets is not None or form != "apart" or self.Dp > 128
         ops.delta_scan(q, k, v, beta, z, gate, self.rate.to(DEV), padded(self.norm, self.Vp, F32), state, torch.empty(T, n * self.Vp, device=DEV), out, segs, pos,
-                       groups=segs if chunked else None, **self.common)
+                       groups=None if form in ("fp32", "sequential") else segs, sets=sets, **self.common)
         got = out.view(T, n, self.Vp)
         assert not got[..., self.V:].any()
         return got[..., : self.V].cpu()
@@ -354,10 +358,10 @@ SIZES = [(4, 2, 24, 36), (3, 3, 64, 64), (2, 1, 128, 128), (2, 2, 96, 200), (1, 
 
 @pytest.mark.parametrize("kind", ["plain", "strong", "slow"])
 @pytest.mark.parametrize("H,G,D,V", SIZES + [(2, 1, 200, 48), (1, 1, 256, 20)])
-@pytest.mark.parametrize("form", ["fp32", "sequential", "chunks"])
+@pytest.mark.parametrize("form", ["fp32", "sequential", "chunks", "apart"])
 def test_delta_recurrence_in_portions(form, H, G, D, V, kind):
     """Whole, and in portions down to one row, the state handed over in a slot that holds something else at first."""
-    dtype, chunked = F32 if form == "fp32" else BF, form == "chunks"
+    dtype = F32 if form == "fp32" else BF
     N = 117
     d = Delta(H, G, D, V, N, dtype, kind=kind)
     want = d.want()
@@ -367,7 +371,7 @@ def test_delta_recurrence_in_portions(form, H, G, D, V, kind):
         st, at, got = d.state(), 0, []
         for n in portions:
             segs, _, pos = ragged([n], [at], [2])
-            got.append(d.scan(slice(at, at + n), segs, pos, st, chunked))
+            got.append(d.scan(slice(at, at + n), segs, pos, st, form))
             at += n
         close(torch.cat(got), want, dtype, tol)
         assert float(st[[0, 1, 3]].min()) == 7.0
@@ -382,7 +386,7 @@ def test_delta_chunks_with_many_heads_and_sequences(H, seqs):
     N, D, V = 45, 64, 128
     d = Delta(H, H, D, V, N, BF, seqs=seqs, kind="slow")
     segs, _, pos = ragged([N] * seqs, [0] * seqs, list(range(1, seqs + 1)))
-    got = d.scan(slice(None), segs, pos, d.state(seqs + 1), True)
+    got = d.scan(slice(None), segs, pos, d.state(seqs + 1), "chunks")
     for s in (0, 1, seqs - 1):
         rows = slice(s * N, s * N + N)
         close(got[rows], d.want(rows), BF)
@@ -390,9 +394,9 @@ def test_delta_chunks_with_many_heads_and_sequences(H, seqs):
     st = d.state(seqs + 1)
     cut = 20
     segs, _, pos = ragged([cut], [0], [1])
-    a = d.scan(slice(0, cut), segs, pos, st, True)
+    a = d.scan(slice(0, cut), segs, pos, st, "chunks")
     segs, _, pos = ragged([N - cut] + [N] * (seqs - 1), [cut] + [0] * (seqs - 1), list(range(1, seqs + 1)))
-    b = d.scan(slice(cut, N * seqs), segs, pos, st, True)
+    b = d.scan(slice(cut, N * seqs), segs, pos, st, "chunks")
     close(torch.cat((a, b)), got, BF)
 
 
@@ -400,9 +404,21 @@ def test_delta_chunks_of_a_long_sequence():
     """Hundreds of chunks: the state stays what the sequential form makes of it, rounding of thousands of decays aside."""
     d = Delta(2, 2, 128, 64, 3000, BF, kind="slow")
     segs, _, pos = ragged([3000], [0], [1])
-    a, b = d.state(), d.state()
-    x, y = d.scan(slice(None), segs, pos, a, True), d.scan(slice(None), segs, pos, b, False)
-    assert float((a[1] - b[1]).norm() / b[1].norm()) < 5e-5
+    a, b, c = d.state(), d.state(), d.state()
+    x, y, z = (d.scan(slice(None), segs, pos, st, f) for st, f in ((a, "chunks"), (b, "sequential"), (c, "apart")))
+    assert float((a[1] - b[1]).norm() / b[1].norm()) < 5e-5 and torch.equal(a, c)
+    close(x, y, BF)
+    close(z, y, BF)
+
+
+def test_delta_sets_of_ragged_segments():
+    """Segments that begin and end anywhere in the chunks of the batch, as operands made apart: each has sets of its own."""
+    lens, starts, slots = [5, 40, 1, 16, 130, 3], [0, 7, 100, 0, 0, 64], [3, 1, 6, 2, 5, 4]
+    d = Delta(3, 1, 40, 70, sum(lens), BF, kind="slow")
+    segs, _, pos = ragged(lens, starts, slots)
+    a, b = d.state(7), d.state(7)
+    x, y = d.scan(slice(None), segs, pos, a, "apart"), d.scan(slice(None), segs, pos, b, "sequential")
+    assert float((a - b).norm() / b.norm()) < 1e-5
     close(x, y, BF)
 
 
