@@ -462,22 +462,25 @@ __device__ __forceinline__ void make_operands(const Params& p, uint8_t* sm, cons
 
 // ---- the products -----------------------------------------------------------------------------------------------------------
 // SETS 2: beside the makers, o of a chunk stays here for its norm if p.o is null.  SETS 4: beside the warps that fetch.
-template <int DK, int SETS>
-__device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job& w) {
+// DS warps share the 16 value columns of a warp: each has DK / DS of the channels, their readouts are summed through shared memory (at `xch`).
+template <int DK, int SETS, int DS>
+__device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job& w, float* xch) {
   using S = Both<DK>;
   constexpr int kMeet = SETS == 2 ? 2 * kNT : kNT + kFetch;        // threads that meet in a barrier of a set
   const int lane = w.lane, r8 = lane >> 2, quad = lane & 3, row16 = w.row16, l16 = w.l16, n = w.n;
   const uint32_t base = smem_addr(sm);
   const bool fresh = p.positions[w.first] == 0, fused = SETS == 2 && p.o == nullptr;
-  const int v0 = w.vb + w.warp * 16;                                // first value column of the warp
-  const bool mma_warp = w.warp * 16 < w.cols && v0 < p.Vp;
-  float st[DK / 8][4];      // S^T: value column v0 + r8 (+ 8), channels 8 i + 2 quad (+ 1)
+  constexpr int DW = DK / DS;
+  const int part = w.warp % DS, own = w.warp / DS, d0 = part * DW;  // channels from d0 on
+  const int v0 = w.vb + own * 16;                                   // first value column of the warp
+  const bool mma_warp = own * 16 < w.cols && v0 < p.Vp;
+  float st[DW / 8][4];      // S^T: value column v0 + r8 (+ 8), channels d0 + 8 i + 2 quad (+ 1)
   float* state = p.state + (size_t(w.slot) * p.heads + w.h) * p.Dp * p.Vp;
 #pragma unroll
-  for (int i = 0; i < DK / 8; i++)
+  for (int i = 0; i < DW / 8; i++)
 #pragma unroll
     for (int j = 0; j < 4; j++) {
-      const int d = i * 8 + quad * 2 + (j & 1), v = v0 + r8 + (j >> 1) * 8;
+      const int d = d0 + i * 8 + quad * 2 + (j & 1), v = v0 + r8 + (j >> 1) * 8;
       st[i][j] = !mma_warp || fresh || d >= p.Dp ? 0.f : state[size_t(d) * p.Vp + v];
     }
   const uint32_t brow = (lane & 7) + ((lane >> 4) << 3), bcol = ((lane >> 3) & 1) * 16;    // right operands stored [n][k]
@@ -488,18 +491,18 @@ __device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job
     if (fused && at + row16 < n && l16 * 8 < p.Vp)
       gate.load(static_cast<const __nv_bfloat16*>(p.gate) + size_t(w.first + at + row16) * p.ldg + size_t(w.h) * p.Vp + l16 * 8);
     bar_sync(kFull + b, kMeet);
+    float o[2][2][4] = {}, x[2][2][4] = {};
     if (mma_warp) {
       // (q P) S and (k P) S, two sums each for even and odd k steps: value column as above, tokens 8 i + 2 quad (+ 1)
-      float o[2][2][4] = {}, x[2][2][4] = {};
 #pragma unroll
-      for (int ks = 0; ks < DK / 16; ks += 2) {
+      for (int ks = 0; ks < DW / 16; ks += 2) {
         uint32_t s[2][kParts][4], r[2][4];
         as_left<kParts>(st + 2 * ks, s[0]);
         as_left<kParts>(st + 2 * ks + 2, s[1]);
 #pragma unroll
         for (int j = kParts - 1; j >= 0; j--) {
 #pragma unroll
-          for (int e = 0; e < 2; e++) ldmatrix_x4(set + S::oK + (j * kC + brow) * S::kPitch + bcol + (ks + e) * 32, r[e]);
+          for (int e = 0; e < 2; e++) ldmatrix_x4(set + S::oK + (j * kC + brow) * S::kPitch + bcol + d0 * 2 + (ks + e) * 32, r[e]);
 #pragma unroll
           for (int i = kParts - 1 - j; i >= 0; i--)
 #pragma unroll
@@ -511,7 +514,7 @@ __device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job
 #pragma unroll
         for (int j = 1; j >= 0; j--) {
 #pragma unroll
-          for (int e = 0; e < 2; e++) ldmatrix_x4(set + S::oQ + (j * kC + brow) * S::kPitch + bcol + (ks + e) * 32, r[e]);
+          for (int e = 0; e < 2; e++) ldmatrix_x4(set + S::oQ + (j * kC + brow) * S::kPitch + bcol + d0 * 2 + (ks + e) * 32, r[e]);
 #pragma unroll
           for (int i = 1 - j; i >= 0; i--)
 #pragma unroll
@@ -521,14 +524,36 @@ __device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job
             }
         }
       }
+#pragma unroll
+      for (int i = 0; i < 2; i++)
+#pragma unroll
+        for (int j = 0; j < 4; j++) { x[0][i][j] += x[1][i][j]; o[0][i][j] += o[1][i][j]; }
+      if constexpr (DS > 1) {
+        float* mine = xch + w.warp * 512 + lane;
+#pragma unroll
+        for (int i = 0; i < 16; i++) mine[i * 32] = i < 8 ? x[0][i >> 2][i & 3] : o[0][(i >> 2) & 1][i & 3];
+      }
+    }
+    if constexpr (DS > 1) bar_sync(kProducts, kNT);
+    if (mma_warp) {
+      if constexpr (DS > 1) {                   // in the same order in all of them
+        float sum[16];
+#pragma unroll
+        for (int i = 0; i < 16; i++) {
+          sum[i] = 0.f;
+#pragma unroll
+          for (int k = 0; k < DS; k++) sum[i] += xch[(own * DS + k) * 512 + i * 32 + lane];
+          if (i < 8) x[0][i >> 2][i & 3] = sum[i];
+          else o[0][(i >> 2) & 1][i & 3] = sum[i];
+        }
+      }
       uint32_t l[kParts][4], f[4];
-      ldmatrix_x4_trans(set + S::oV + brow * S::kVPitch + w.warp * 32 + bcol, f);      // v^T: stored [token][column]
+      ldmatrix_x4_trans(set + S::oV + brow * S::kVPitch + own * 32 + bcol, f);      // v^T: stored [token][column]
 #pragma unroll
       for (int j = 0; j < 4; j++) {
         float* y = &x[0][j >> 1][(j & 1) * 2];
-        const float* z = &x[1][j >> 1][(j & 1) * 2];
-        y[0] = __uint_as_float(f[j] << 16) - (y[0] + z[0]);
-        y[1] = __uint_as_float(f[j] & 0xffff0000u) - (y[1] + z[1]);
+        y[0] = __uint_as_float(f[j] << 16) - y[0];
+        y[1] = __uint_as_float(f[j] & 0xffff0000u) - y[1];
       }
       float u[2][4] = {};
       as_left<kParts>(x[0], l);
@@ -542,27 +567,34 @@ __device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job
         }
       }
 #pragma unroll
-      for (int i = 0; i < DK / 8; i++) {
-        const float2 e = *reinterpret_cast<const float2*>(sm + b * S::kSet + S::oE + (i * 8 + quad * 2) * 4);
+      for (int i = 0; i < DW / 8; i++) {
+        const float2 e = *reinterpret_cast<const float2*>(sm + b * S::kSet + S::oE + (d0 + i * 8 + quad * 2) * 4);
         st[i][0] *= e.x; st[i][1] *= e.y; st[i][2] *= e.x; st[i][3] *= e.y;
       }
       as_left<kParts>(u, l);
+      if (part == 0) {
+        float q[2][4] = {};
 #pragma unroll
-      for (int j = 1; j >= 0; j--) {
-        ldmatrix_x4(set + S::oA + (j * kC + brow) * S::kAPitch + bcol, f);
+        for (int j = 1; j >= 0; j--) {
+          ldmatrix_x4(set + S::oA + (j * kC + brow) * S::kAPitch + bcol, f);
 #pragma unroll
-        for (int i = 1 - j; i >= 0; i--) {
-          mma_bf16(o[i][0], l[i], f[0], f[1]);
-          mma_bf16(o[i][1], l[i], f[2], f[3]);
+          for (int i = 1 - j; i >= 0; i--) {
+            mma_bf16(i ? q[0] : o[0][0], l[i], f[0], f[1]);
+            mma_bf16(i ? q[1] : o[0][1], l[i], f[2], f[3]);
+          }
         }
+#pragma unroll
+        for (int i = 0; i < 2; i++)
+#pragma unroll
+          for (int j = 0; j < 4; j++) o[0][i][j] += q[i][j];
       }
 #pragma unroll
-      for (int i = 0; i < DK / 16; i += 2)
+      for (int i = 0; i < DW / 16; i += 2)
 #pragma unroll
         for (int j = kParts - 1; j >= 0; j--) {                     // smallest part first
           uint32_t r[2][4];
 #pragma unroll
-          for (int e = 0; e < 2; e++) ldmatrix_x4_trans(set + S::oR + (j * kC + (lane & 15)) * S::kPitch + (i + e) * 32 + (lane >> 4) * 16, r[e]);
+          for (int e = 0; e < 2; e++) ldmatrix_x4_trans(set + S::oR + (j * kC + (lane & 15)) * S::kPitch + d0 * 2 + (i + e) * 32 + (lane >> 4) * 16, r[e]);
 #pragma unroll
           for (int y = kParts - 1 - j; y >= 0; y--)
 #pragma unroll
@@ -576,8 +608,9 @@ __device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job
 #pragma unroll
         for (int j = 0; j < 4; j++) {
           const int t = i * 8 + quad * 2 + (j & 1), v = r8 + (j >> 1) * 8;
-          const float y = o[0][i][j] + o[1][i][j];
-          if (fused) reinterpret_cast<float*>(sm + S::oO)[t * S::kOPitch + w.warp * 16 + v] = y;
+          const float y = o[0][i][j];
+          if (part != 0) continue;
+          if (fused) reinterpret_cast<float*>(sm + S::oO)[t * S::kOPitch + own * 16 + v] = y;
           else if (at + t < n) p.o[(size_t(w.first + at + t) * p.heads + w.h) * p.Vp + v0 + v] = y;
         }
     }
@@ -608,10 +641,10 @@ __device__ __forceinline__ void multiply(const Params& p, uint8_t* sm, const Job
   }
   if (mma_warp) {
 #pragma unroll
-    for (int i = 0; i < DK / 8; i++)
+    for (int i = 0; i < DW / 8; i++)
 #pragma unroll
       for (int j = 0; j < 4; j++) {
-        const int d = i * 8 + quad * 2 + (j & 1), v = v0 + r8 + (j >> 1) * 8;
+        const int d = d0 + i * 8 + quad * 2 + (j & 1), v = v0 + r8 + (j >> 1) * 8;
         if (d < p.Dp) state[size_t(d) * p.Vp + v] = st[i][j];
       }
   }
@@ -660,7 +693,7 @@ __global__ void __launch_bounds__(2 * kNT, 1) k_delta_chunk(const Params p, cons
   const Job w = job_of(p, groups + 4 * blockIdx.x, blockIdx.y, blockIdx.z * kCols, kCols, threadIdx.x % kNT);
   if (threadIdx.x < kNT) {
     more_registers<152>();
-    multiply<DK, 2>(p, sm, w);
+    multiply<DK, 2, 1>(p, sm, w, nullptr);
   } else {
     fewer_registers<104>();
     make_operands<DK, false>(p, sm, w, 0, w.nc, nullptr, 0);
@@ -684,23 +717,30 @@ __global__ void __launch_bounds__(kNT, 2) k_delta_make(const Params p, const int
   }
 }
 
-template <int DK>
+template <int DK, int DS>
 __global__ void __launch_bounds__(kNT + kFetch, 1) k_delta_multiply(const Params p, const int* groups, const uint8_t* sets, int cols) {
   extern __shared__ __align__(16) uint8_t sm[];
   pdl::launch_dependents();
   pdl::grid_dependency_wait();
   const Job w = job_of(p, groups + 4 * blockIdx.x, blockIdx.y, blockIdx.z * cols, cols, threadIdx.x % kNT);
   const size_t stride = size_t(p.heads) * Shape<DK>::kStored;
-  if (threadIdx.x < kNT) multiply<DK, 4>(p, sm, w);
+  if (threadIdx.x < kNT) multiply<DK, 4, DS>(p, sm, w, reinterpret_cast<float*>(sm + 4 * Shape<DK>::kSet));
   else fetch_operands<DK>(p, sm, w, sets + first_set(w, blockIdx.x) * stride + size_t(w.h) * Shape<DK>::kStored, stride);
 }
 
 template <int DK>
 size_t sets_bytes(const Params& p, int rows, int ngroups) { return size_t(rows / kC + ngroups + 1) * p.heads * Shape<DK>::kStored; }
 
+template <int DK, int DS>
+cudaError_t launch_multiply(const Params& p, const int* groups, const uint8_t* sets, int cols, dim3 grid, cudaStream_t st) {
+  static bool done = false;
+  constexpr size_t smem = 4 * Shape<DK>::kSet + (DS > 1 ? kNW * 512 * 4 : 0);
+  cudaError_t e = allow_smem(k_delta_multiply<DK, DS>, smem, &done);
+  return e != cudaSuccess ? e : pdl::launch(k_delta_multiply<DK, DS>, grid, dim3(kNT + kFetch), smem, st, 1, p, groups, sets, cols);
+}
 template <int DK>
 cudaError_t launch(Params p, const int* groups, int ngroups, int rows, uint8_t* sets, bool* finished, cudaStream_t st) {
-  static bool done[3] = {};
+  static bool done[2] = {};
   cudaError_t e;
   if (!sets) {
     *finished = p.Vp <= kCols;
@@ -712,12 +752,19 @@ cudaError_t launch(Params p, const int* groups, int ngroups, int rows, uint8_t* 
   e = allow_smem(k_delta_make<DK>, Make<DK>::kBytes, &done[1]);
   const int all = rows / kC + ngroups;
   if (e == cudaSuccess) e = pdl::launch(k_delta_make<DK>, dim3((all + kMakeChunks - 1) / kMakeChunks, p.heads), dim3(kNT), Make<DK>::kBytes, st, 1, p, groups, ngroups, sets);
-  // as many CTAs per head as find room: the fewer value columns, the shorter a chunk's products
+  if (e != cudaSuccess) return e;
+  // as many CTAs per head as find room, and as many warps per 16 value columns as there are channels for: the shorter a chunk's products
+  const auto ctas = [&](int cols) { return ngroups * p.heads * ((p.Vp + cols - 1) / cols); };
   int cols = kCols;
-  while (cols > 32 && cols / 2 < p.Vp && ngroups * p.heads * ((p.Vp + cols / 2 - 1) / (cols / 2)) <= tbvops::sm_count()) cols /= 2;
-  if (e == cudaSuccess) e = allow_smem(k_delta_multiply<DK>, 4 * Shape<DK>::kSet, &done[2]);
-  return e != cudaSuccess ? e : pdl::launch(k_delta_multiply<DK>, dim3(ngroups, p.heads, (p.Vp + cols - 1) / cols), dim3(kNT + kFetch), 4 * Shape<DK>::kSet, st, 1, p, groups,
-                                            static_cast<const uint8_t*>(sets), cols);
+  while (cols > 16 && cols / 2 < p.Vp && ctas(cols / 2) <= tbvops::sm_count()) cols /= 2;
+  const int ds = cols > 64 || DK < 64 ? 1 : (cols > 16 || DK < 128 ? 2 : 4);
+  const dim3 grid(ngroups, p.heads, (p.Vp + cols - 1) / cols);
+  if (ds == 1) return launch_multiply<DK, 1>(p, groups, sets, cols, grid, st);
+  if constexpr (DK >= 64) {
+    if (ds == 2) return launch_multiply<DK, 2>(p, groups, sets, cols, grid, st);
+  }
+  if constexpr (DK >= 128) return launch_multiply<DK, 4>(p, groups, sets, cols, grid, st);
+  return cudaErrorInvalidValue;
 }
 
 }  // namespace
